@@ -41,6 +41,15 @@ class ForgeSampling(C.Structure):
                 ("seed", C.c_uint64)]
 
 
+class ForgeCheckpointInfo(C.Structure):
+    _fields_ = [("architecture", C.c_char * 64), ("hidden_size", C.c_int32), ("vocab_size", C.c_int32), ("num_layers", C.c_int32),
+                ("num_weight_layers", C.c_int32), ("parameters", C.c_int64), ("cache_values_per_token", C.c_int64)]
+
+
+class ForgeStepEntry(C.Structure):
+    _fields_ = [("seq", C.c_int32), ("n_tokens", C.c_int32), ("n_want", C.c_int32)]
+
+
 # name -> (restype, argtypes); every symbol the public header declares
 SIGNATURES = {
     "forge_last_error": (C.c_char_p, []),
@@ -83,6 +92,9 @@ SIGNATURES = {
     "forge_gguf_export_weights_bin": (i32, [vp, vp, sz]),
     "forge_weights_bin_size": (sz, [C.POINTER(ForgeModelConfig)]),
     "forge_model_create": (i32, [C.POINTER(ForgeModelConfig), vp, sz, i32, C.POINTER(vp)]),
+    "forge_checkpoint_info": (i32, [C.c_char_p, C.POINTER(ForgeCheckpointInfo)]),
+    "forge_model_open": (i32, [C.c_char_p, i32, i32, C.POINTER(vp)]),
+    "forge_model_info": (i32, [vp, C.POINTER(ForgeCheckpointInfo)]),
     "forge_model_destroy": (None, [vp]),
     "forge_model_stream": (vp, [vp]),
     "forge_model_vocab_size": (sz, [vp]),
@@ -98,6 +110,9 @@ SIGNATURES = {
     "forge_model_set_prefill_mode": (i32, [vp, i32]),
     "forge_model_set_wait_limit": (i32, [vp, u32]),
     "forge_kv_create": (i32, [vp, i32, i32, C.POINTER(vp)]),
+    "forge_kv_create_pool": (i32, [vp, i32, i32, i32, C.POINTER(vp)]),
+    "forge_kv_free_seq": (i32, [vp, i32]),
+    "forge_kv_free_tokens": (C.c_int64, [vp]),
     "forge_kv_reset": (i32, [vp]),
     "forge_kv_len": (i32, [vp, i32]),
     "forge_kv_destroy": (None, [vp]),
@@ -110,6 +125,7 @@ SIGNATURES = {
     "forge_forward_seq": (i32, [vp, vp, i32, u32, vp]),
     "forge_forward_prefill_seq": (i32, [vp, vp, i32, vp, sz, vp]),
     "forge_forward_batch": (i32, [vp, vp, i32, vp, vp]),
+    "forge_step": (i32, [vp, vp, C.POINTER(ForgeStepEntry), i32, vp, vp, vp]),
     "forge_generate_greedy": (i32, [vp, vp, vp, sz, i32, vp]),
     "forge_decode_greedy_batch": (i32, [vp, vp, i32, vp, i32, vp]),
     "forge_hidden_trace_enable": (i32, [vp, i32]),

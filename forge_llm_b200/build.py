@@ -4,6 +4,7 @@
 """
 from __future__ import annotations
 
+import hashlib
 import os
 import subprocess
 import sys
@@ -13,8 +14,10 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(CSRC, "build")
 LIB = os.path.join(HERE, "libforge_b200.so")
+STAMP = LIB + ".sha256"
 SOURCES = ["pack.cu", "gemv_tc.cu", "gemv_batch.cu", "elementwise.cu", "attn_decode.cu", "attn_prefill_tc5.cu", "gemm_mma.cu", "gemm_tc5.cu",
-           "tp_comm.cu", "gguf_reader.cu", "kquant_host.cu", "sampler.cu", "api_ops.cu", "model.cu"]
+           "tp_comm.cu", "gguf_reader.cu", "kquant_host.cu", "sampler.cu", "api_ops.cu", "model.cu",
+           "checkpoint.cu", "gemm_dense.cu", "mla.cu", "mla_decode.cu", "attn_prefill_kv.cu", "stack_model.cu"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC,-fopenmp,-O3", "-Xptxas", "-v"]
 
@@ -59,7 +62,31 @@ def build_library(force: bool = False, verbose: bool = False) -> str:
                            capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
+    with open(STAMP, "w") as f:
+        f.write(_digest() + "\n")
     return LIB
+
+
+def _digest() -> str:
+    """Content hash of everything the library is built from."""
+    h = hashlib.sha256()
+    files = sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cu", ".cuh", ".h")))
+    for f in files + [os.path.join(HERE, "..", "include", "forge_b200.h"), os.path.abspath(__file__)]:
+        h.update(os.path.basename(f).encode())
+        with open(f, "rb") as fh:
+            h.update(fh.read())
+    return h.hexdigest()
+
+
+def ensure_library() -> str:
+    """Builds the library if it is missing or was built from other sources (by content, not by file times)."""
+    try:
+        with open(STAMP) as f:
+            if f.read().strip() == _digest() and os.path.exists(LIB):
+                return LIB
+    except OSError:
+        pass
+    return build_library()
 
 
 if __name__ == "__main__":

@@ -1,0 +1,252 @@
+// Prompt attention over keys and values formed for this call (latent attention), bfloat16, tcgen05.  The structure is that
+// of attn_prefill_tc5.cu - S = Q K^T in tensor memory, lazy running maximum, probabilities back into tensor memory as the
+// operand of O += P V, three overlapped stages - with these differences: the query / key width (an unrotated part per head
+// plus a rotated part whose keys all heads share) and the value width are independent run-time sizes, several sequences'
+// tiles run in one launch (a table gives each tile's rows, position and context), and the epilogue applies the output gate.
+// Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = softmax, rescale, store.
+// Tensor memory: S [0, 64), P0 [64, 96), P1 [96, 128), O from 128.
+#include <algorithm>
+
+#include "mla.cuh"
+#include "tc5.cuh"
+
+namespace forge {
+
+namespace {
+
+using namespace tc5;
+
+constexpr int BM = 128, BN = 64, kThreads = 192;
+constexpr uint32_t kColS = 0, kColP = 64, kColO = 128;
+constexpr float kLazy = 8.f;
+
+struct Params {
+    LatentDims d;
+    PromptAttnArgs a;
+    float scale2;
+    int stages;
+};
+
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+template <uint32_t COLS>
+__global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+                                                                   const __grid_constant__ CUtensorMap map_r, const __grid_constant__ CUtensorMap map_v, const __grid_constant__ Params p) {
+    constexpr int Q_CHUNK = BM * 128, KV_CHUNK = BN * 128, kMaxStages = 3;
+    const LatentDims& d = p.d;
+    const int kch = d.dim_p / 64, rch = d.rot_p / 64, vch = d.vdim_p / 64, qch = kch + rch;
+    const int stage_bytes = (qch + vch) * KV_CHUNK, KVS = p.stages;
+    extern __shared__ __align__(1024) unsigned char smem_raw[];
+    unsigned char* sQ = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+    unsigned char* sKV = sQ + qch * Q_CHUNK;
+    __shared__ uint64_t q_full, kv_full[kMaxStages], kv_empty[kMaxStages], s_full, s_free, p_full[2], pv_done[2];
+    __shared__ uint32_t s_tmem;
+    __shared__ int s_err;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int h = blockIdx.x;
+    const PromptTile t = p.a.tiles[blockIdx.y];
+    const int nblk = (t.pos0 + t.rows - 1) / BN + 1;
+
+    if (tid == 0) {
+        mbar_init(&q_full, 1);
+        for (int s = 0; s < kMaxStages; ++s) { mbar_init(&kv_full[s], 1); mbar_init(&kv_empty[s], 1); }
+        mbar_init(&s_full, 1);
+        mbar_init(&s_free, 4);
+        for (int s = 0; s < 2; ++s) { mbar_init(&p_full[s], 4); mbar_init(&pv_done[s], 1); }
+        s_err = 0;
+        mbar_fence_init();
+    }
+    if (warp == 1) tmem_alloc<COLS>(&s_tmem);
+    fence_before();
+    __syncthreads();
+    fence_after();
+    const uint32_t tmem = s_tmem;
+
+    if (warp == 0) {
+        if (lane == 0) {
+            mbar_expect_tx(&q_full, uint32_t(qch * Q_CHUNK));
+            for (int c = 0; c < qch; ++c) tma_3d(sQ + c * Q_CHUNK, &map_q, c * 64, h, t.row0, &q_full);
+            for (int j = 0; j < nblk; ++j) {
+                const int s = j % KVS, use = j / KVS;
+                if (use > 0 && !mbar_wait(&kv_empty[s], (use - 1) & 1, &s_err)) { atomicExch(&s_err, 1); break; }
+                const int row = t.ctx0 + j * BN;
+                unsigned char* dst = sKV + size_t(s) * stage_bytes;
+                mbar_expect_tx(&kv_full[s], uint32_t(stage_bytes));
+                for (int c = 0; c < kch; ++c) tma_3d(dst + c * KV_CHUNK, &map_k, c * 64, h, row, &kv_full[s]);
+                for (int c = 0; c < rch; ++c) tma_2d(dst + (kch + c) * KV_CHUNK, &map_r, c * 64, row, &kv_full[s]);
+                for (int c = 0; c < vch; ++c) tma_3d(dst + (qch + c) * KV_CHUNK, &map_v, c * 64, h, row, &kv_full[s]);
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            bool ok = mbar_wait(&q_full, 0, &s_err);
+            const uint32_t q_base = smem_u32(sQ);
+            const int ks = (d.dim + 15) / 16, rs = (d.rot + 15) / 16;   // sixteen-wide steps that hold anything
+            auto issue_s = [&](int j) {
+                const uint32_t k_base = smem_u32(sKV + size_t(j % KVS) * stage_bytes);
+                for (int i = 0; i < ks + rs; ++i) {
+                    const int step = i < ks ? i : kch * 4 + (i - ks);
+                    const uint32_t off = uint32_t(step / 4), in = uint32_t((step % 4) * 32);
+                    umma_ss(tmem + kColS, desc_kmajor(q_base + off * Q_CHUNK + in), desc_kmajor(k_base + off * KV_CHUNK + in), idesc_bf16(BN), i > 0 ? 1u : 0u);
+                }
+                umma_commit(&s_full);
+            };
+            if (ok && mbar_wait(&kv_full[0], 0, &s_err)) { fence_after(); issue_s(0); }
+            else ok = false;
+            const uint32_t id_v = idesc_bf16(d.vdim_p, true);
+            for (int j = 0; j < nblk && ok; ++j) {
+                if (j + 1 < nblk) {
+                    if (!mbar_wait(&kv_full[(j + 1) % KVS], ((j + 1) / KVS) & 1, &s_err) || !mbar_wait(&s_free, j & 1, &s_err)) { ok = false; break; }
+                    fence_after();
+                    issue_s(j + 1);
+                }
+                if (!mbar_wait(&p_full[j & 1], (j >> 1) & 1, &s_err)) { ok = false; break; }
+                fence_after();
+                const uint32_t v_base = smem_u32(sKV + size_t(j % KVS) * stage_bytes) + qch * KV_CHUNK;
+#pragma unroll
+                for (int k16 = 0; k16 < BN / 16; ++k16)
+                    umma_ts(tmem + kColO, tmem + kColP + uint32_t((j & 1) * 32 + k16 * 8), desc_mnmajor(v_base + k16 * 2048, KV_CHUNK), id_v, (j > 0 || k16 > 0) ? 1u : 0u);
+                umma_commit(&pv_done[j & 1]);
+                umma_commit(&kv_empty[j % KVS]);
+            }
+            if (!ok) atomicExch(&s_err, 1);
+        }
+    } else {
+        const int quad = warp & 3;
+        const int r = quad * 32 + lane;
+        const int pq = t.pos0 + r;
+        const uint32_t lane_addr = tmem + (uint32_t(quad * 32) << 16);
+        float m_ref = -INFINITY, l_run = 0.f;
+        bool ok = true;
+        for (int j = 0; j < nblk; ++j) {
+            const int t0 = j * BN;
+            if (ok && !mbar_wait(&s_full, j & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
+            fence_after();
+            uint32_t sv[2][32];
+            tmem_ld32(lane_addr + kColS, sv[0]);
+            tmem_ld32(lane_addr + kColS + 32, sv[1]);
+            wait_ld();
+            fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&s_free);
+            if (t0 + BN - 1 > t.pos0) {
+#pragma unroll
+                for (int c = 0; c < 64; ++c)
+                    if (t0 + c > pq) sv[c >> 5][c & 31] = 0xff800000u;  // -inf
+            }
+            float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+            for (int c = 0; c < 64; ++c) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(sv[c >> 5][c & 31]) * p.scale2);   // the scale may have either sign
+            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+            float alpha = 1.f;
+            if (m_ref == -INFINITY) m_ref = mx;
+            else if (mx > m_ref + kLazy) { alpha = ex2(m_ref - mx); m_ref = mx; }
+            const float m_use = m_ref == -INFINITY ? 0.f : m_ref;
+            float sum4[4] = {0.f, 0.f, 0.f, 0.f};
+            uint32_t ph[32];
+#pragma unroll
+            for (int c = 0; c < 64; c += 2) {
+                const float p0 = ex2(fmaf(__uint_as_float(sv[c >> 5][c & 31]), p.scale2, -m_use));
+                const float p1 = ex2(fmaf(__uint_as_float(sv[c >> 5][(c & 31) + 1]), p.scale2, -m_use));
+                sum4[(c >> 1) & 3] += p0 + p1;
+                ph[c >> 1] = pack_bf2(p0, p1);
+            }
+            l_run = l_run * alpha + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
+            if (j >= 2 && ok && !mbar_wait(&pv_done[j & 1], ((j >> 1) - 1) & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
+            if (j > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
+                if (ok && !mbar_wait(&pv_done[(j - 1) & 1], ((j - 1) >> 1) & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
+                fence_after();
+                for (int c0 = 0; c0 < d.vdim_p; c0 += 32) {
+                    uint32_t o[32];
+                    tmem_ld32(lane_addr + kColO + c0, o);
+                    wait_ld();
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
+                    tmem_st32(lane_addr + kColO + c0, o);
+                }
+            }
+            fence_after();
+            tmem_st32(lane_addr + kColP + uint32_t((j & 1) * 32), ph);
+            wait_st();
+            fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&p_full[j & 1]);
+        }
+        if (ok && !mbar_wait(&pv_done[(nblk - 1) & 1], ((nblk - 1) >> 1) & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
+        fence_after();
+        const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+        const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(p.a.gate) + size_t(t.row0 + r) * p.a.gate_ld + h * d.vdim;
+        __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.a.out) + size_t(t.row0 + r) * p.a.out_ld + h * d.vdim;
+        const bool vec = !(d.vdim & 7) && !(p.a.gate_ld & 7) && !(p.a.out_ld & 7);   // 16-byte pieces stay aligned
+        for (int c0 = 0; c0 < d.vdim; c0 += 32) {
+            uint32_t o[32];
+            tmem_ld32(lane_addr + kColO + c0, o);
+            wait_ld();
+            if (r < t.rows && ok) {
+                const int nc = min(32, d.vdim - c0);
+                if (vec) {
+#pragma unroll
+                    for (int i = 0; i < 32; i += 8)
+                        if (i < nc) {
+                            const uint4 g4 = *reinterpret_cast<const uint4*>(gate + c0 + i);
+                            const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&g4);
+                            uint32_t w[4];
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                const float2 g = __bfloat1622float2(g2[e]);
+                                w[e] = pack_bf2(__uint_as_float(o[i + 2 * e]) * inv * g.x, __uint_as_float(o[i + 2 * e + 1]) * inv * g.y);
+                            }
+                            *reinterpret_cast<uint4*>(out + c0 + i) = make_uint4(w[0], w[1], w[2], w[3]);
+                        }
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i)
+                        if (i < nc) out[c0 + i] = __float2bfloat16_rn(__uint_as_float(o[i]) * inv * __bfloat162float(gate[c0 + i]));
+                }
+            }
+        }
+        fence_before();
+    }
+    __syncthreads();
+    if (warp == 1) {
+        fence_after();
+        tmem_free<COLS>(tmem);
+    }
+    if (tid == 0 && s_err && p.a.err) atomicExch(p.a.err, 1);
+}
+
+size_t smem_bytes(const LatentDims& d, int stages) {
+    const int qch = (d.dim_p + d.rot_p) / 64, vch = d.vdim_p / 64;
+    return size_t(qch) * BM * 128 + size_t(stages) * (qch + vch) * BN * 128 + 1024;
+}
+
+}  // namespace
+
+bool attn_prefill_kv_supported(const LatentDims& d) { return d.vdim_p <= 256 && smem_bytes(d, 2) <= 220 * 1024; }
+
+int32_t attn_prefill_kv(const LatentDims& d, const PromptAttnArgs& a, cudaStream_t st) {
+    if (a.n_tiles <= 0) return FORGE_OK;
+    if (!attn_prefill_kv_supported(d)) { set_error("prompt attention: head sizes %d + %d / %d unsupported", d.dim, d.rot, d.vdim); return FORGE_ERR_SHAPE; }
+    CUtensorMap mq, mk, mr, mv;
+    const uint64_t qd = uint64_t(d.dim_p + d.rot_p), H = uint64_t(d.heads);
+    FORGE_TRY(make_map_3d(&mq, a.q, qd, H, uint64_t(a.q_rows), qd * 2, H * qd * 2, BM));
+    FORGE_TRY(make_map_3d(&mk, a.k, uint64_t(d.dim_p), H, uint64_t(a.ctx_rows), uint64_t(d.dim_p) * 2, H * d.dim_p * 2, BN));
+    if (d.rot_p == 0) mr = mk;   // no rotated part: never read
+    else FORGE_TRY(make_map_2d(&mr, a.krot, uint64_t(d.rot_p), uint64_t(a.ctx_rows), uint64_t(d.rot_p) * 2, BN));
+    FORGE_TRY(make_map_3d(&mv, a.v, uint64_t(d.vdim_p), H, uint64_t(a.ctx_rows), uint64_t(d.vdim_p) * 2, H * d.vdim_p * 2, BN));
+    Params p{d, a, d.scale * 1.4426950408889634f, smem_bytes(d, 3) <= 220 * 1024 ? 3 : 2};
+    const size_t smem = smem_bytes(d, p.stages);
+    auto go = [&](auto kern) -> int32_t {
+        FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+        kern<<<dim3(d.heads, a.n_tiles), kThreads, smem, st>>>(mq, mk, mr, mv, p);
+        FORGE_LAUNCH_CHECK();
+        return FORGE_OK;
+    };
+    return d.vdim_p <= 128 ? go(attn_prefill_kv_kernel<256>) : go(attn_prefill_kv_kernel<512>);
+}
+
+}  // namespace forge

@@ -2,7 +2,9 @@
 // Reference statements (crates/forgellm-codegen-cpu/src/emit.rs): rms_norm :327-334,
 // rope :509-528, silu_mul :381-386, residual_add :455-459, embedding :586-589, bias adds
 // :4108-4118, cache write :4136-4153 (fp16 here instead of int8), argmax project.rs:501-503.
-#include "common.cuh"
+#include <cmath>
+
+#include "dense.cuh"
 
 namespace forge {
 
@@ -162,6 +164,28 @@ __global__ void embedding_kernel(float* out, const float* table, const uint32_t*
     const float4* src = reinterpret_cast<const float4*>(table + size_t(tokens[blockIdx.x]) * h);
     float4* dst = reinterpret_cast<float4*>(out + size_t(blockIdx.x) * h);
     for (int i = threadIdx.x; i < h / 4; i += blockDim.x) dst[i] = src[i];
+}
+
+// embedding row -> residual stream f32, and its Dynamic Tanh norm tanh(alpha x) w + b as the first layer's input
+template <typename T>
+__global__ void embed_dyt_kernel(float* __restrict__ x, T* __restrict__ h, int h_ld, const T* __restrict__ table, const uint32_t* __restrict__ tokens, int width, float alpha,
+                                 const float* __restrict__ w, const float* __restrict__ b, uint32_t* hist, const int32_t* step) {
+    const int r = blockIdx.x;
+    if (hist && threadIdx.x == 0) hist[size_t(*step) * gridDim.x + r] = tokens[r];
+    const T* src = table + size_t(tokens[r]) * width;
+    for (int i = threadIdx.x; i < h_ld; i += blockDim.x) {
+        float n = 0.f;
+        if (i < width) {
+            const float v = float(src[i]);
+            x[size_t(r) * width + i] = v;
+            n = tanhf(alpha * v) * w[i] + b[i];
+        }
+        h[size_t(r) * h_ld + i] = T(n);
+    }
+}
+
+__global__ void gather_act_kernel(uint4* dst, const uint4* src, const int32_t* idx, int ld16) {
+    for (int i = threadIdx.x; i < ld16; i += blockDim.x) dst[size_t(blockIdx.x) * ld16 + i] = src[size_t(idx[blockIdx.x]) * ld16 + i];
 }
 
 __global__ void kv_append_contig_kernel(__half* kc, __half* vc, const float* k, const float* v, size_t n, size_t off) {
@@ -534,6 +558,36 @@ int32_t gather_rows_f16(float* out, const __half* pool, const int32_t* page_row,
     if (n == 0) return FORGE_OK;
     gather_rows_kernel<<<grid_for(n), 256, 0, st>>>(out, pool, page_row, len, kvd);
     FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+
+int32_t embed_dyt(float* x, void* h, int h_ld, const void* table, int dtype, const uint32_t* tokens, int rows, int width, float alpha,
+                  const float* w, const float* b, uint32_t* hist, const int32_t* step, cudaStream_t st) {
+    if (rows <= 0) return FORGE_OK;
+    if (dtype == FORGE_F32)
+        embed_dyt_kernel<float><<<rows, 256, 0, st>>>(x, static_cast<float*>(h), h_ld, static_cast<const float*>(table), tokens, width, alpha, w, b, hist, step);
+    else
+        embed_dyt_kernel<__nv_bfloat16><<<rows, 256, 0, st>>>(x, static_cast<__nv_bfloat16*>(h), h_ld, static_cast<const __nv_bfloat16*>(table), tokens, width, alpha, w, b, hist, step);
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+int32_t gather_act_rows(void* dst, const void* src, const int32_t* idx, int rows, int ld, int dtype, cudaStream_t st) {
+    if (rows <= 0) return FORGE_OK;
+    gather_act_kernel<<<rows, 128, 0, st>>>(static_cast<uint4*>(dst), static_cast<const uint4*>(src), idx, int(ld * dense_size(dtype) / 16));
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+// {cos, sin} of p / base^(2 i / dims), angles formed in double
+int32_t rope_half_table(float* table, int n_pos, int dims, double base) {
+    const int half = dims / 2;
+    for (int i = 0; i < half; ++i) {
+        const double f = std::pow(base, -2.0 * i / dims);
+        for (int p = 0; p < n_pos; ++p) {
+            const double a = p * f;
+            table[(size_t(p) * half + i) * 2] = float(std::cos(a));
+            table[(size_t(p) * half + i) * 2 + 1] = float(std::sin(a));
+        }
+    }
     return FORGE_OK;
 }
 

@@ -1,0 +1,396 @@
+// Dense linear layers of the layer-list models: out[token][row] = act[token][K] . W[row][K]^T.
+//
+// bfloat16 (gemm_dense_kernel): tcgen05 with both operands in shared memory.  A tile is 128 weight rows (MMA M) x NT
+// tokens (MMA N = 16 .. 256); one kernel serves a decode step (NT = 16: a weight stream, 16 KB of weights per K step and
+// SM in a ring of up to eleven stages) and a prompt (NT = 256).  The work is dealt in K steps of 64: CTA i of G takes the
+// steps [i U / G, (i + 1) U / G) of the U = tiles * K / 64 steps of the whole product, so every SM streams the same amount
+// whatever the number of tiles.  A tile that several CTAs share is finished by the last of them to arrive (ticket): every
+// share is left in scratch memory and added in K order, so the result does not depend on the order of arrival.  Nobody
+// waits for another CTA.
+// Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = epilogue (TMEM lane = weight row).
+// Accumulators are double buffered in tensor memory: the epilogue of one tile runs under the products of the next.
+// The weight stages of the ring are requested before the dependency wait of a programmatic launch, the activations after.
+//
+// float32 (gemm_f32_kernel): a tiled product on the CUDA cores in plain f32 fused multiply-adds.
+#include <algorithm>
+#include <cstring>
+
+#include "dense.cuh"
+#include "tc5.cuh"
+
+namespace forge {
+
+namespace {
+
+using namespace tc5;
+
+constexpr int BK = 64;
+constexpr int kThreads = 192;
+
+template <typename T> __device__ __forceinline__ T to_t(float v);
+template <> __device__ __forceinline__ float to_t<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 to_t<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+
+__device__ __forceinline__ int find_seg(const DenseOut& o, int row) {
+    int s = -1;
+    for (int i = 0; i < o.nseg; ++i)
+        if (row >= o.seg[i].row0 && row < o.seg[i].row0 + o.seg[i].rows) s = i;
+    return s;
+}
+
+// one finished value of a segment that is not SEG_CLAMPED_GLU; r = row in the segment
+template <typename T>
+__device__ __forceinline__ void seg_store(const OutSeg& g, int r, size_t token, float v, float resid, float nw, float nb) {
+    if (g.kind == SEG_F32) {
+        static_cast<float*>(g.dst)[token * g.ld + r] = v;
+    } else if (g.kind == SEG_CAST) {
+        const int c = g.group ? (r / g.group) * g.group_ld + r % g.group : r;
+        static_cast<T*>(g.dst)[token * g.ld + c] = to_t<T>(v);
+    } else if (g.kind == SEG_SIGMOID) {
+        static_cast<T*>(g.dst)[token * g.ld + r] = to_t<T>(1.0f / (1.0f + expf(-v)));
+    } else {
+        const float x = resid + v;
+        static_cast<float*>(g.dst)[token * g.ld + r] = x;
+        if (g.next) static_cast<T*>(g.next)[token * g.next_ld + r] = to_t<T>(tanhf(g.alpha * x) * nw + nb);
+    }
+}
+
+struct GemmParams {
+    DenseOut out;
+    int m, N, nk;            // tokens, rows, K steps per tile
+    int tt_count;            // token tiles
+    long long units;         // tiles * nk
+    float* part; int* tickets;
+    int* err;
+};
+
+__device__ __forceinline__ long long share_begin(long long units, int g, int grid) { return units * g / grid; }
+__device__ __forceinline__ int share_of(long long units, long long u, int grid) { return int(((u + 1) * grid - 1) / units); }
+
+template <int NT> struct Ring {
+    static constexpr int X_BYTES = NT * 128, STAGE = 16384 + X_BYTES;
+    static constexpr int STAGES = (200 * 1024) / STAGE > 11 ? 11 : (200 * 1024) / STAGE;
+    static constexpr uint32_t COLS = NT <= 16 ? 32 : 2 * NT;   // two accumulators
+};
+
+template <int NT>
+__global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
+                                                                 const __grid_constant__ GemmParams p) {
+    constexpr int STAGE = Ring<NT>::STAGE, STAGES = Ring<NT>::STAGES;
+    constexpr uint32_t kCols = Ring<NT>::COLS;
+    extern __shared__ __align__(1024) unsigned char smem_raw[];
+    unsigned char* ring = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+    __shared__ uint64_t full[STAGES], empty[STAGES], acc_full[2], acc_empty[2];
+    __shared__ uint32_t s_tmem;
+    __shared__ int s_err, s_last;
+
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const long long u0 = share_begin(p.units, blockIdx.x, gridDim.x), u1 = share_begin(p.units, blockIdx.x + 1, gridDim.x);
+    if (tid == 0) {
+        for (int s = 0; s < STAGES; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
+        for (int s = 0; s < 2; ++s) { mbar_init(&acc_full[s], 1); mbar_init(&acc_empty[s], 4); }
+        s_err = 0;
+        mbar_fence_init();
+    }
+    if (warp == 1) tmem_alloc<kCols>(&s_tmem);
+    fence_before();
+    __syncthreads();
+    fence_after();
+    const uint32_t tmem = s_tmem;
+    pdl_trigger();
+
+    if (warp == 0) {
+        if (lane == 0) {
+            const int total = int(u1 - u0);
+            auto coords = [&](int i, int& kt, int& row0, int& tok0) {
+                const long long u = u0 + i;
+                const int tile = int(u / p.nk);
+                kt = int(u - (long long)tile * p.nk);
+                row0 = (tile / p.tt_count) * 128;
+                tok0 = (tile % p.tt_count) * NT;
+            };
+            const int ahead = min(total, STAGES);
+            int kt, row0, tok0;
+            for (int i = 0; i < ahead; ++i) {   // constant weights: may overlap the kernel in front
+                coords(i, kt, row0, tok0);
+                mbar_expect_tx(&full[i], uint32_t(STAGE));
+                tma_2d(ring + size_t(i) * STAGE, &map_w, kt * BK, row0, &full[i]);
+            }
+            pdl_wait();
+            for (int i = 0; i < total; ++i) {
+                const int s = i % STAGES, use = i / STAGES;
+                coords(i, kt, row0, tok0);
+                unsigned char* dst = ring + size_t(s) * STAGE;
+                if (use > 0) {
+                    if (!mbar_wait(&empty[s], (use - 1) & 1, &s_err)) { atomicExch(&s_err, 1); break; }
+                    mbar_expect_tx(&full[s], uint32_t(STAGE));
+                    tma_2d(dst, &map_w, kt * BK, row0, &full[s]);
+                }
+                tma_2d(dst + 16384, &map_x, kt * BK, tok0, &full[s]);
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            int i = 0;
+            bool ok = true;
+            int seg = 0;
+            for (long long u = u0; u < u1 && ok; ++seg) {
+                const long long tile_end = (u / p.nk + 1) * p.nk;
+                const int n = int(min(u1, tile_end) - u), buf = seg & 1;
+                if (seg >= 2 && !mbar_wait(&acc_empty[buf], ((seg >> 1) - 1) & 1, &s_err)) { ok = false; break; }
+                fence_after();
+                for (int k = 0; k < n; ++k, ++i) {
+                    const int s = i % STAGES;
+                    if (!mbar_wait(&full[s], (i / STAGES) & 1, &s_err)) { ok = false; break; }
+                    fence_after();
+                    const uint32_t base = smem_u32(ring + size_t(s) * STAGE);
+#pragma unroll
+                    for (int k16 = 0; k16 < BK / 16; ++k16)
+                        umma_ss(tmem + uint32_t(buf * NT), desc_kmajor(base + k16 * 32), desc_kmajor(base + 16384 + k16 * 32), idesc_bf16(NT),
+                                (k > 0 || k16 > 0) ? 1u : 0u);
+                    umma_commit(&empty[s]);
+                }
+                if (ok) umma_commit(&acc_full[buf]);
+                u += n;
+            }
+            if (!ok) atomicExch(&s_err, 1);
+        }
+    } else {
+        pdl_wait();
+        const int quad = warp & 3;
+        const uint32_t lane_addr = tmem + (uint32_t(quad * 32) << 16);
+        constexpr int CH = NT < 32 ? NT : 32;   // columns per read
+        int seg_i = 0;
+        for (long long u = u0; u < u1; ++seg_i) {
+            const int tile = int(u / p.nk);
+            const long long t_begin = (long long)tile * p.nk, t_end = t_begin + p.nk;
+            const int n = int(min(u1, t_end) - u), buf = seg_i & 1;
+            const int row0 = (tile / p.tt_count) * 128 + quad * 32, tok0 = (tile % p.tt_count) * NT;
+            const int row = row0 + lane;
+            const int cols = min(NT, p.m - tok0);
+            // the four warps meet at the barriers of a shared tile: one whose wait gave up must not leave the loop alone
+            if (!mbar_wait(&acc_full[buf], (seg_i >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
+            fence_after();
+            // every warp's rows lie in one segment (segments start at multiples of 32 rows)
+            const int si = find_seg(p.out, row0);
+            const OutSeg& g = p.out.seg[si < 0 ? 0 : si];
+            const int r = row - g.row0;
+            const bool row_ok = si >= 0 && r < g.rows;
+            float nw = 0.f, nb = 0.f;
+            if (row_ok && g.kind == SEG_RESID && g.next) { nw = g.norm_w[r]; nb = g.norm_b[r]; }
+            auto finish = [&](int c0, const float (&v)[CH]) {
+                if (g.kind == SEG_CLAMPED_GLU) {
+                    // neighbouring lanes hold gate_j and up_j: the even lane takes the first half of the columns
+                    const bool even = !(lane & 1);
+                    const int j = r >> 1;
+#pragma unroll
+                    for (int c = 0; c < CH / 2; ++c) {
+                        const float got = __shfl_xor_sync(0xffffffffu, even ? v[CH / 2 + c] : v[c], 1);
+                        const float ga = even ? v[c] : got, up = even ? got : v[CH / 2 + c];
+                        const int t = c0 + (even ? c : CH / 2 + c);
+                        if (row_ok && t < cols) static_cast<__nv_bfloat16*>(g.dst)[size_t(tok0 + t) * g.ld + j] = __float2bfloat16_rn(clamped_glu(ga, up, g.limit));
+                    }
+                } else if (row_ok) {
+                    float rv[CH];
+                    if (g.kind == SEG_RESID) {   // all loads before the first store
+#pragma unroll
+                        for (int c = 0; c < CH; ++c) rv[c] = c0 + c < cols ? static_cast<const float*>(g.dst)[size_t(tok0 + c0 + c) * g.ld + r] : 0.f;
+                    }
+#pragma unroll
+                    for (int c = 0; c < CH; ++c)
+                        if (c0 + c < cols) seg_store<__nv_bfloat16>(g, r, size_t(tok0 + c0 + c), v[c], g.kind == SEG_RESID ? rv[c] : 0.f, nw, nb);
+                }
+            };
+            auto load = [&](int c0, float (&v)[CH]) {
+                uint32_t t[CH];
+                if constexpr (CH == 16) tmem_ld16(lane_addr + uint32_t(buf * NT + c0), t);
+                else tmem_ld32(lane_addr + uint32_t(buf * NT + c0), t);
+                wait_ld();
+#pragma unroll
+                for (int c = 0; c < CH; ++c) v[c] = __uint_as_float(t[c]);
+            };
+            if (n == p.nk) {
+#pragma unroll 1
+                for (int c0 = 0; c0 < NT && c0 < cols; c0 += CH) {
+                    float v[CH];
+                    load(c0, v);
+                    finish(c0, v);
+                }
+            } else {
+                // a shared tile: this CTA's part goes to its slot (0: the part its share starts with, 1: the other one)
+                float* mine = p.part + (size_t(blockIdx.x) * 2 + (u0 >= t_begin ? 0 : 1)) * (NT * 128);
+#pragma unroll 1
+                for (int c0 = 0; c0 < NT && c0 < cols; c0 += CH) {
+                    float v[CH];
+                    load(c0, v);
+#pragma unroll
+                    for (int c = 0; c < CH; ++c) __stcg(mine + size_t(c0 + c) * 128 + quad * 32 + lane, v[c]);
+                }
+                const int first = share_of(p.units, t_begin, gridDim.x), last = share_of(p.units, t_end - 1, gridDim.x);
+                __threadfence();
+                asm volatile("bar.sync 1, 128;" ::: "memory");
+                if (tid == 64) {
+                    const int old = atomicAdd(p.tickets + tile, 1);
+                    s_last = old == last - first;
+                    if (s_last) p.tickets[tile] = 0;
+                }
+                asm volatile("bar.sync 1, 128;" ::: "memory");
+                if (s_last) {
+                    __threadfence();
+#pragma unroll 1
+                    for (int c0 = 0; c0 < NT && c0 < cols; c0 += CH) {
+                        float v[CH];
+#pragma unroll
+                        for (int c = 0; c < CH; ++c) v[c] = 0.f;
+                        for (int q = first; q <= last; ++q) {
+                            const float* src = p.part + (size_t(q) * 2 + (share_begin(p.units, q, gridDim.x) >= t_begin ? 0 : 1)) * (NT * 128) + quad * 32 + lane;
+#pragma unroll
+                            for (int c = 0; c < CH; ++c) v[c] += __ldcg(src + size_t(c0 + c) * 128);
+                        }
+                        finish(c0, v);
+                    }
+                }
+                asm volatile("bar.sync 1, 128;" ::: "memory");   // s_last is read before it is written again
+            }
+            fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&acc_empty[buf]);
+            u += n;
+        }
+        fence_before();
+    }
+    __syncthreads();
+    if (warp == 1) {
+        fence_after();
+        tmem_free<kCols>(tmem);
+    }
+    if (tid == 0 && s_err && p.err) atomicExch(p.err, 1);
+}
+
+template <int NT>
+int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmParams& p, int sms, cudaStream_t st) {
+    CUtensorMap mx;
+    FORGE_TRY(make_map_2d(&mx, act, uint64_t(w.K), uint64_t(p.m), uint64_t(act_ld) * 2, NT));
+    CUtensorMap mw;
+    memcpy(&mw, w.map, sizeof(mw));
+    p.tt_count = (p.m + NT - 1) / NT;
+    const long long tiles = (long long)((w.N + 127) / 128) * p.tt_count;
+    p.units = tiles * p.nk;
+    const int grid = int(std::max(1LL, std::min((long long)sms, p.units / 4)));
+    const size_t smem = size_t(Ring<NT>::STAGES) * Ring<NT>::STAGE + 1024;
+    auto kern = gemm_dense_kernel<NT>;
+    FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+    FORGE_CUDA(launch_pdl(kern, dim3(grid), dim3(kThreads), smem, st, mw, mx, p));
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+
+// ------------------------------------------------------------------------------------------------ float32
+// 64 rows x TM tokens per CTA, K in steps of 16, 256 threads
+template <int TM>
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ w, const float* __restrict__ x, int ldx, int K, int m, int N, const DenseOut out) {
+    constexpr int TN = 64, KS = 16, PT = TM / 16;   // tokens per thread
+    __shared__ float sw[KS][TN + 4], sx[KS][TM + 4];
+    const int tid = threadIdx.x, rr = (tid & 15) * 4, tt = (tid >> 4) * PT;
+    const int row0 = blockIdx.x * TN, tok0 = blockIdx.y * TM;
+    float acc[4][PT];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < PT; ++j) acc[i][j] = 0.f;
+    for (int k0 = 0; k0 < K; k0 += KS) {
+        for (int i = tid; i < TN * KS; i += 256) {
+            const int r = i / KS, k = i % KS;
+            sw[k][r] = row0 + r < N ? w[size_t(row0 + r) * K + k0 + k] : 0.f;
+        }
+        for (int i = tid; i < TM * KS; i += 256) {
+            const int t = i / KS, k = i % KS;
+            sx[k][t] = tok0 + t < m ? x[size_t(tok0 + t) * ldx + k0 + k] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < KS; ++k) {
+            float a[4], b[PT];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) a[i] = sw[k][rr + i];
+#pragma unroll
+            for (int j = 0; j < PT; ++j) b[j] = sx[k][tt + j];
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < PT; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+    const int si = find_seg(out, row0 + rr);   // four consecutive rows lie in one segment or past its end
+    if (si < 0) return;
+    const OutSeg& g = out.seg[si];
+#pragma unroll
+    for (int j = 0; j < PT; ++j) {
+        const int t = tok0 + tt + j;
+        if (t >= m) continue;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int r = row0 + rr + i - g.row0;
+            if (r >= g.rows) continue;
+            if (g.kind == SEG_CLAMPED_GLU) {
+                if (!(i & 1)) static_cast<float*>(g.dst)[size_t(t) * g.ld + (r >> 1)] = clamped_glu(acc[i][j], acc[i + 1][j], g.limit);
+            } else {
+                const bool rs = g.kind == SEG_RESID;
+                const float nw = rs && g.next ? g.norm_w[r] : 0.f, nb = rs && g.next ? g.norm_b[r] : 0.f;
+                seg_store<float>(g, r, size_t(t), acc[i][j], rs ? static_cast<const float*>(g.dst)[size_t(t) * g.ld + r] : 0.f, nw, nb);
+            }
+        }
+    }
+}
+
+}  // namespace
+
+int32_t dense_make_map(DenseWeight& w) {
+    static_assert(sizeof(CUtensorMap) == sizeof(w.map), "CUtensorMap is 128 bytes");
+    if (w.dtype != FORGE_BF16) return FORGE_OK;
+    CUtensorMap m;
+    FORGE_TRY(make_map_2d(&m, w.w, uint64_t(w.K), uint64_t(w.N), uint64_t(w.K) * 2, 128));
+    memcpy(w.map, &m, sizeof(m));
+    return FORGE_OK;
+}
+
+int32_t dense_gemm(const DenseWeight& w, const void* act, int act_ld, int m, const DenseOut& out, const DenseScratch& sc, int* err, cudaStream_t st) {
+    if (m <= 0) return FORGE_OK;
+    if (w.K % kDensePad || act_ld < w.K || act_ld % kDensePad) { set_error("dense product: K=%d, activation rows of %d", w.K, act_ld); return FORGE_ERR_SHAPE; }
+    for (int i = 0; i < out.nseg; ++i)
+        if (out.seg[i].row0 % kSegAlign || out.seg[i].row0 + out.seg[i].rows > w.N || (out.seg[i].kind == SEG_CLAMPED_GLU && out.seg[i].rows % 2)) {
+            set_error("dense product: bad output segment %d", i);
+            return FORGE_ERR_SHAPE;
+        }
+    if (w.dtype == FORGE_F32) {
+        const float* wf = static_cast<const float*>(w.w);
+        const float* xf = static_cast<const float*>(act);
+        if (m <= 16) gemm_f32_kernel<16><<<dim3((w.N + 63) / 64, 1), 256, 0, st>>>(wf, xf, act_ld, w.K, m, w.N, out);
+        else gemm_f32_kernel<64><<<dim3((w.N + 63) / 64, (m + 63) / 64), 256, 0, st>>>(wf, xf, act_ld, w.K, m, w.N, out);
+        FORGE_LAUNCH_CHECK();
+        return FORGE_OK;
+    }
+    int dev = 0, sms = 148;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    sms = std::min(sms, 148);
+    GemmParams p{};
+    p.out = out; p.m = m; p.N = w.N; p.nk = w.K / BK; p.part = sc.part; p.tickets = sc.tickets; p.err = err;
+    const int nt = m <= 16 ? 16 : m <= 32 ? 32 : m <= 64 ? 64 : m <= 128 ? 128 : 256;
+    if (size_t((w.N + 127) / 128) * ((m + nt - 1) / nt) > sc.tickets_cap) { set_error("dense product: too many tiles for the ticket array"); return FORGE_ERR_SHAPE; }
+    switch (nt) {
+        case 16: return launch_dense<16>(w, act, act_ld, p, sms, st);
+        case 32: return launch_dense<32>(w, act, act_ld, p, sms, st);
+        case 64: return launch_dense<64>(w, act, act_ld, p, sms, st);
+        case 128: return launch_dense<128>(w, act, act_ld, p, sms, st);
+    }
+    return launch_dense<256>(w, act, act_ld, p, sms, st);
+}
+
+}  // namespace forge

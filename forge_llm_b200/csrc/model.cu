@@ -11,7 +11,7 @@
 #include <string>
 #include <vector>
 
-#include "gemv_core.cuh"
+#include "model.cuh"
 
 namespace forge {
 
@@ -31,96 +31,7 @@ void set_error(const char* fmt, ...) {
 
 using namespace forge;
 
-// ------------------------------------------------------------------------------ structures
-struct ForgeLayer {
-    float* attn_norm = nullptr;
-    QWeight qkv;           // rows: [q ; k ; v] of this rank (row-major split layout: prefill GEMM)
-    QTiled qkv_t;          // the same matrix in the tiled streaming layout (decode GEMV)
-    QTiled v_t;            // only when v_proj is stored in another format than q/k: qkv holds [q ; k], this holds v
-    float* qkv_bias = nullptr;
-    QWeight o;
-    QTiled o_t;
-    float* ffn_norm = nullptr;
-    QWeight gateup;        // rows interleaved: 2j = gate_j, 2j+1 = up_j
-    QTiled gateup_t;
-    QWeight down;
-    QTiled down_t;
-};
-
-struct ForgeModel {
-    ForgeModelConfig cfg;
-    int device = 0;
-    cudaStream_t stream = nullptr;
-    // local (per tensor-parallel rank) sizes
-    int h = 0, qk = 0, kv = 0, ff = 0, V = 0, hd = 0, nq = 0, nkv = 0;
-    float* embed = nullptr;
-    std::vector<ForgeLayer> layers;
-    float* final_norm = nullptr;
-    QWeight lm_head;
-    QTiled lm_head_t;
-    int* d_err = nullptr;  // set by a kernel whose bounded wait gave up
-    GemvSplit split;       // split-K scratch shared by the decode GEMVs (one launch at a time on the stream)
-    GemvSplit bsplit;      // the same for the batched decode products
-    uint2* d_bact = nullptr;  // packed activations of one batched product (sixteen rows)
-    float* rope = nullptr;  // [max_seq][hd/2]{cos,sin}
-    int max_seq = 0;
-    std::vector<void*> allocs;
-    // prefill scratch (grown on demand)
-    int scratch_rows = 0, tok_cap = 0;
-    float* p_hidden = nullptr; __half* p_normed = nullptr; float* p_qkv = nullptr; __half* p_q16 = nullptr; __half* p_q16_lo = nullptr;
-    __half* p_attn16 = nullptr; float* p_gu = nullptr; __half* p_act16 = nullptr; uint32_t* p_tokens = nullptr;
-    __half* p_normed_lo = nullptr; __half* p_attn16_lo = nullptr; __half* p_act16_lo = nullptr;
-    float* p_parts = nullptr;   // [4][rows][h] partial products of the K-sliced o / down projections
-    float* p_qkv_parts = nullptr;   // [4][rows][qk + 2 kv] the same for the QKV projection
-    int gemm_passes = 3;  // 3: split-precision prefill GEMMs (default); 1: single fp16 pass
-    std::vector<struct ForgeKV*> caches;   // live caches of this model (released with it if the caller did not)
-    int pq[8] = {0, 0, 0, 0, 0, 0, 0, 0};  // storage format of q, k, v, o, gate, up, down, lm_head (cfg.proj_quant or cfg.quant)
-    bool uniform_basic = true;             // every projection is stored in cfg.quant (Q8_0 / Q4_0): what the whole-step kernel takes
-    bool per_token_prefill = false;        // no batched layout for this mix of formats: the prompt always runs token by token
-    bool any_kquant = false;               // a projection is stored as Q4_K / Q6_K
-    bool kquant_batched = false;           // K-quant models: prompt through the batched GEMMs (forge_model_set_prefill_mode)
-    TpComm* tp = nullptr;  // tensor-parallel communicator (cfg.tp_world > 1)
-    // peer-memory exchange of the decode step (forge_model_tp_exchange_*): local buffer, peers' mappings, device tables
-    void* tpx_local = nullptr; std::vector<void*> tpx_peer; bool tpx_ready = false;
-    uint2** d_tpx_ll = nullptr; uint32_t* d_tpx_step = nullptr;  // peers' buffers (device table), decode step counter
-    float* p_part = nullptr; float* d_part = nullptr;  // this rank's partial sums of a row-sliced projection
-    uint32_t wait_limit = 1u << 20;     // polls per device-side peer wait (forge_model_set_wait_limit)
-    // decode scratch (per batch row).  Growing it moves every buffer: scratch_gen counts the moves, and whatever holds the
-    // old addresses (a cache's captured decode graph) is rebuilt when its generation differs.
-    int dec_batch = 0; int scratch_gen = 0;
-    float* d_hidden2 = nullptr;
-    float* d_hidden = nullptr; float* d_q = nullptr; float* d_attn = nullptr; float* d_act = nullptr; float* d_logits = nullptr;
-    uint32_t* d_tok = nullptr; uint32_t* d_hist = nullptr; int hist_cap = 0; int32_t* d_step = nullptr;
-    float* d_amax_val = nullptr; int* d_amax_idx = nullptr; int* d_amax_ticket = nullptr;
-    // parity trace
-    bool trace_on = false; float* trace = nullptr; size_t trace_cap = 0; int trace_rows = 0;
-    // timing of the last generate call
-    cudaEvent_t ev[3] = {nullptr, nullptr, nullptr};
-    float prefill_ms = 0.f, decode_ms = 0.f; long long last_launches = 0;
-};
-
-struct ForgeKV {
-    ForgeModel* model = nullptr;
-    int max_seq = 0, batch = 0, pages_per_seq = 0, num_pages = 0;
-    __half* k_pool = nullptr; __half* v_pool = nullptr;
-    size_t layer_stride = 0;  // halfs per layer pool
-    int32_t* d_page_table = nullptr; int32_t* d_seq_len = nullptr;
-    std::vector<int32_t> h_page_table; std::vector<int> free_pages; std::vector<int> pages_used; std::vector<int> len;
-    float* attn_ws = nullptr; int* attn_counters = nullptr; int splits = 1;
-    alignas(64) unsigned char k_map[128], v_map[128];   // CUtensorMap of the two pools (all layers), for the decode attention's page copies
-    cudaGraphExec_t graph = nullptr; int graph_batch = 0; bool graph_greedy = false; int graph_gen = -1;  // scratch generation the graph was captured with
-};
-
 namespace {
-
-template <typename T>
-int32_t dev_alloc(ForgeModel* m, T** p, size_t count) {
-    void* q = nullptr;
-    FORGE_CUDA(cudaMalloc(&q, std::max<size_t>(count, 1) * sizeof(T)));
-    m->allocs.push_back(q);
-    *p = static_cast<T*>(q);
-    return FORGE_OK;
-}
 
 int32_t alloc_qweight(ForgeModel* m, QWeight& w, int quant, int K, int N) {
     w.K = K; w.N = N; w.quant = quant;
@@ -197,6 +108,10 @@ int32_t ensure_prefill_scratch(ForgeModel* m, int rows) {
     return FORGE_OK;
 }
 
+}  // namespace
+
+namespace forge {
+
 int32_t ensure_decode_scratch(ForgeModel* m, int batch) {
     if (batch <= m->dec_batch) return FORGE_OK;
     size_t b = size_t(batch);
@@ -213,7 +128,7 @@ int32_t ensure_decode_scratch(ForgeModel* m, int batch) {
     FORGE_CUDA(cudaMemsetAsync(m->d_amax_ticket, 0, sizeof(int) * b, m->stream));
     if (!m->d_step) { FORGE_TRY(dev_alloc(m, &m->d_step, 1)); }
     if (m->cfg.tp_world > 1) FORGE_TRY(dev_alloc(m, &m->d_part, b * m->h));
-    if (batch >= 2) {   // batched steps keep their q/k/v and gate/up rows in the prompt scratch; their buffers must exist before a capture
+    if (batch >= 2 && !m->stack) {   // batched steps keep their q/k/v and gate/up rows in the prompt scratch; their buffers must exist before a capture
         FORGE_TRY(ensure_prefill_scratch(m, batch));
         FORGE_TRY(ensure_batch_buffers(m));
     }
@@ -232,7 +147,6 @@ int32_t ensure_trace(ForgeModel* m, int rows) {
     return FORGE_OK;
 }
 
-// hand out pages so that sequence `seq` can hold `new_len` positions; uploads the table row if it changed
 int32_t ensure_pages(ForgeKV* kv, int seq, int new_len) {
     if (new_len > kv->max_seq) { set_error("KV cache full: position %d >= max_seq %d", new_len - 1, kv->max_seq); return FORGE_ERR_KV_FULL; }
     int need = (new_len + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE;
@@ -259,9 +173,6 @@ int32_t upload_len(ForgeKV* kv) {
     return FORGE_OK;
 }
 
-// The synchronisation point of a session call.  Also reads the word the bounded device-side waits raise when they give
-// up (a pipeline stage, a peer's contribution or another CTA's result never arrived): the call then fails with
-// FORGE_ERR_TIMEOUT, the word is cleared and the device-side positions are put back to the host's (`kv`, may be null).
 int32_t sync_and_check(ForgeModel* m, ForgeKV* kv) {
     int herr = 0;
     FORGE_CUDA(cudaMemcpyAsync(&herr, m->d_err, sizeof(int), cudaMemcpyDeviceToHost, m->stream));
@@ -273,6 +184,16 @@ int32_t sync_and_check(ForgeModel* m, ForgeKV* kv) {
     set_error("a bounded device-side wait gave up: the step did not complete");
     return FORGE_ERR_TIMEOUT;
 }
+
+int32_t check_seq(const ForgeKV* kv, int seq) {
+    if (!kv || seq < 0 || seq >= kv->batch) { set_error("sequence index out of range"); return FORGE_ERR_INVALID_ARG; }
+    if (!kv->model) { set_error("the model of this cache has been destroyed"); return FORGE_ERR_INVALID_ARG; }
+    return FORGE_OK;
+}
+
+}  // namespace forge
+
+namespace {
 
 // hidden += W x for a projection whose K dimension is sliced over the tensor-parallel ranks: the ranks' partial
 // products are summed (all-reduce) before the residual is added, so every rank holds the same hidden state
@@ -328,6 +249,7 @@ int32_t prefill_seq(ForgeModel* m, ForgeKV* kv, int seq, const uint32_t* tokens_
     cudaStream_t st = m->stream;
     const int base = kv->len[seq];
     FORGE_TRY(ensure_pages(kv, seq, base + n));
+    if (m->stack) return stack_prefill(m, kv, seq, tokens_host, n);
     if (m->per_token_prefill || (m->any_kquant && !m->kquant_batched)) return prefill_per_token(m, kv, seq, tokens_host, n);
     FORGE_TRY(ensure_prefill_scratch(m, n));
     FORGE_TRY(ensure_decode_scratch(m, 1));
@@ -538,6 +460,7 @@ int32_t decode_launches_gemm(ForgeModel* m, ForgeKV* kv, int batch, bool greedy,
 }
 
 int32_t decode_launches(ForgeModel* m, ForgeKV* kv, int batch, bool greedy, bool record, const PrefillToken* pt = nullptr) {
+    if (m->stack) return stack_decode_launches(m, kv, batch, greedy, record);
     const ForgeModelConfig& c = m->cfg;
     cudaStream_t st = m->stream;
     const int32_t* page_table = kv->d_page_table + (pt ? size_t(pt->seq) * kv->pages_per_seq : 0);
@@ -672,6 +595,7 @@ int32_t decode_step_graph(ForgeModel* m, ForgeKV* kv, int batch, bool greedy) {
         cudaError_t ce = cudaStreamEndCapture(m->stream, &g);
         if (rc != FORGE_OK) { if (g) cudaGraphDestroy(g); return rc; }
         if (ce != cudaSuccess) { set_error("graph capture: %s", cudaGetErrorString(ce)); return FORGE_ERR_CUDA; }
+        kv->graph_kernels = g_launches - before;
         g_launches = before;  // captured, not launched
         cudaError_t ie = cudaGraphInstantiate(&kv->graph, g, 0);
         cudaGraphDestroy(g);
@@ -679,14 +603,7 @@ int32_t decode_step_graph(ForgeModel* m, ForgeKV* kv, int batch, bool greedy) {
         kv->graph_batch = batch; kv->graph_greedy = greedy; kv->graph_gen = m->scratch_gen;
     }
     FORGE_CUDA(cudaGraphLaunch(kv->graph, m->stream));
-    // kernels inside one replay: embedding + 5 per layer + lm_head + (argmax) + advance
-    g_launches += 1 + 5LL * m->cfg.num_layers + 1 + (greedy ? 1 : 0) + 1;
-    return FORGE_OK;
-}
-
-int32_t check_seq(const ForgeKV* kv, int seq) {
-    if (!kv || seq < 0 || seq >= kv->batch) { set_error("sequence index out of range"); return FORGE_ERR_INVALID_ARG; }
-    if (!kv->model) { set_error("the model of this cache has been destroyed"); return FORGE_ERR_INVALID_ARG; }
+    g_launches += kv->graph_kernels;
     return FORGE_OK;
 }
 
@@ -877,6 +794,7 @@ void forge_model_destroy(ForgeModel* m) {
     if (m->stream) cudaStreamSynchronize(m->stream);
     for (ForgeKV* kv : m->caches) kv_release_device(kv);
     m->caches.clear();
+    stack_destroy(m);
     tp_destroy(m->tp);
     for (void* q : m->tpx_peer) if (q) cudaIpcCloseMemHandle(q);
     if (m->tpx_local) cudaFree(m->tpx_local);
@@ -952,6 +870,13 @@ int32_t forge_model_tp_init(ForgeModel* m, const uint8_t* id) {
 
 int32_t forge_kv_create(ForgeModel* m, int32_t max_seq, int32_t batch, ForgeKV** out) {
     if (!m || !out || max_seq <= 0 || batch <= 0) { set_error("bad argument to forge_kv_create"); return FORGE_ERR_INVALID_ARG; }
+    const long long pages = (long long)((std::min(max_seq, m->max_seq) + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE) * batch;
+    if (pages * FORGE_KV_PAGE > INT32_MAX) { set_error("a cache of %d x %d positions is too large", batch, max_seq); return FORGE_ERR_SHAPE; }
+    return forge_kv_create_pool(m, int32_t(pages * FORGE_KV_PAGE), max_seq, batch, out);
+}
+
+int32_t forge_kv_create_pool(ForgeModel* m, int32_t pool_tokens, int32_t max_seq, int32_t batch, ForgeKV** out) {
+    if (!m || !out || max_seq <= 0 || batch <= 0 || pool_tokens <= 0) { set_error("bad argument to forge_kv_create_pool"); return FORGE_ERR_INVALID_ARG; }
     *out = nullptr;
     FORGE_CUDA(cudaSetDevice(m->device));
     ForgeKV* kv = new ForgeKV();
@@ -959,10 +884,15 @@ int32_t forge_kv_create(ForgeModel* m, int32_t max_seq, int32_t batch, ForgeKV**
     kv->max_seq = std::min(max_seq, m->max_seq);
     kv->batch = batch;
     kv->pages_per_seq = (kv->max_seq + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE;
-    kv->num_pages = kv->pages_per_seq * batch;
+    kv->num_pages = (pool_tokens - 1) / FORGE_KV_PAGE + 1;
+    const size_t table = size_t(kv->pages_per_seq) * batch;
     kv->layer_stride = size_t(kv->num_pages) * FORGE_KV_PAGE * m->kv;
     size_t pool = kv->layer_stride * m->cfg.num_layers;
     auto fail = [&](int32_t code) { forge_kv_destroy(kv); return code; };
+    if (m->stack) {
+        int32_t rc = stack_cache_create(kv);
+        if (rc != FORGE_OK) return fail(rc);
+    } else {
     if (cudaMalloc(&kv->k_pool, pool * sizeof(__half)) != cudaSuccess || cudaMalloc(&kv->v_pool, pool * sizeof(__half)) != cudaSuccess) {
         set_error("KV pool allocation of %zu bytes failed", 2 * pool * sizeof(__half)); cudaGetLastError(); return fail(FORGE_ERR_CUDA);
     }
@@ -975,21 +905,24 @@ int32_t forge_kv_create(ForgeModel* m, int32_t max_seq, int32_t batch, ForgeKV**
     }
     cudaMemsetAsync(kv->k_pool, 0, pool * sizeof(__half), m->stream);
     cudaMemsetAsync(kv->v_pool, 0, pool * sizeof(__half), m->stream);
-    if (cudaMalloc(&kv->d_page_table, sizeof(int32_t) * kv->num_pages) != cudaSuccess || cudaMalloc(&kv->d_seq_len, sizeof(int32_t) * batch) != cudaSuccess)
+    }
+    if (cudaMalloc(&kv->d_page_table, sizeof(int32_t) * table) != cudaSuccess || cudaMalloc(&kv->d_seq_len, sizeof(int32_t) * batch) != cudaSuccess)
         { set_error("KV table allocation failed"); return fail(FORGE_ERR_CUDA); }
-    cudaMemsetAsync(kv->d_page_table, 0, sizeof(int32_t) * kv->num_pages, m->stream);
+    cudaMemsetAsync(kv->d_page_table, 0, sizeof(int32_t) * table, m->stream);
     cudaMemsetAsync(kv->d_seq_len, 0, sizeof(int32_t) * batch, m->stream);
-    kv->h_page_table.assign(kv->num_pages, 0);
+    kv->h_page_table.assign(table, 0);
     kv->pages_used.assign(batch, 0);
     kv->len.assign(batch, 0);
     for (int i = kv->num_pages - 1; i >= 0; --i) kv->free_pages.push_back(i);
     // split-KV: enough CTAs to fill the SMs
+    if (!m->stack) {
     int sms = 148;
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, m->device);
     kv->splits = attn_decode_splits(kv->pages_per_seq, batch * m->nkv, sms, m->hd, m->nq / m->nkv);
     if (cudaMalloc(&kv->attn_ws, sizeof(float) * attn_decode_ws_floats(batch, m->nq, m->hd, kv->splits)) != cudaSuccess ||
         cudaMalloc(&kv->attn_counters, sizeof(int) * batch * m->nkv) != cudaSuccess) { set_error("attention workspace allocation failed"); return fail(FORGE_ERR_CUDA); }
     cudaMemsetAsync(kv->attn_counters, 0, sizeof(int) * batch * m->nkv, m->stream);
+    }
     if (cudaStreamSynchronize(m->stream) != cudaSuccess) { set_error("KV init failed"); return fail(FORGE_ERR_CUDA); }
     m->caches.push_back(kv);
     *out = kv;
@@ -1007,6 +940,18 @@ int32_t forge_kv_reset(ForgeKV* kv) {
     return upload_len(kv);
 }
 
+int32_t forge_kv_free_seq(ForgeKV* kv, int32_t seq) {
+    FORGE_TRY(check_seq(kv, seq));
+    FORGE_CUDA(cudaSetDevice(kv->model->device));
+    FORGE_CUDA(cudaStreamSynchronize(kv->model->stream));
+    for (int i = 0; i < kv->pages_used[seq]; ++i) kv->free_pages.push_back(kv->h_page_table[size_t(seq) * kv->pages_per_seq + i]);
+    kv->pages_used[seq] = 0;
+    kv->len[seq] = 0;
+    return upload_len(kv);
+}
+
+int64_t forge_kv_free_tokens(const ForgeKV* kv) { return kv && kv->model ? int64_t(kv->free_pages.size()) * FORGE_KV_PAGE : -1; }
+
 int32_t forge_kv_len(const ForgeKV* kv, int32_t seq) { return (kv && seq >= 0 && seq < kv->batch) ? kv->len[seq] : -1; }
 
 void forge_kv_destroy(ForgeKV* kv) {
@@ -1017,6 +962,7 @@ void forge_kv_destroy(ForgeKV* kv) {
     auto& reg = kv->model->caches;
     reg.erase(std::remove(reg.begin(), reg.end(), kv), reg.end());
     if (kv->graph) cudaGraphExecDestroy(kv->graph);
+    stack_cache_destroy(kv);
     cudaFree(kv->k_pool); cudaFree(kv->v_pool); cudaFree(kv->d_page_table); cudaFree(kv->d_seq_len);
     cudaFree(kv->attn_ws); cudaFree(kv->attn_counters);
     delete kv;
@@ -1025,6 +971,7 @@ void forge_kv_destroy(ForgeKV* kv) {
 // device memory of a cache whose model is being destroyed; the handle itself stays valid for forge_kv_destroy
 static void kv_release_device(ForgeKV* kv) {
     if (kv->graph) cudaGraphExecDestroy(kv->graph);
+    stack_cache_destroy(kv);
     cudaFree(kv->k_pool); cudaFree(kv->v_pool); cudaFree(kv->d_page_table); cudaFree(kv->d_seq_len);
     cudaFree(kv->attn_ws); cudaFree(kv->attn_counters);
     kv->graph = nullptr; kv->k_pool = kv->v_pool = nullptr; kv->d_page_table = kv->d_seq_len = nullptr;
@@ -1039,6 +986,7 @@ int32_t forge_kv_read(ForgeKV* kv, int32_t seq, int32_t layer, int32_t which, fl
     FORGE_CUDA(cudaSetDevice(m->device));
     int len = kv->len[seq];
     if (len == 0) return FORGE_OK;
+    if (m->stack) return stack_kv_read(kv, seq, layer, which, out_host);
     float* tmp = nullptr;
     FORGE_CUDA(cudaMalloc(&tmp, sizeof(float) * len * m->kv));
     const __half* pool = (which ? kv->v_pool : kv->k_pool) + size_t(layer) * kv->layer_stride;
@@ -1075,6 +1023,7 @@ int32_t forge_score_chunk(ForgeModel* m, ForgeKV* kv, const uint32_t* chunk, siz
 // ---- persistence (project.rs:456-499)
 namespace {
 constexpr char kKvMagic[4] = {'F', 'K', 'V', '1'};
+constexpr char kLatentMagic[4] = {'F', 'K', 'L', '1'};   // a layer-list model's cache
 // 24 bytes on disk: magic 'FKV1' | u32 layers | u32 width (values per cache row) | u32 zero | u64 positions
 struct KvHeader { char magic[4]; uint32_t layers, width, reserved; uint64_t len; };
 static_assert(sizeof(KvHeader) == 24, "the saved-cache header is a fixed 24-byte layout");
@@ -1099,6 +1048,7 @@ int32_t kv_copy_rows(ForgeKV* kv, int seq, int layer, int which, int len, __half
 size_t forge_kv_save_size(const ForgeKV* kv, int32_t seq) {
     if (!kv || !kv->model || seq < 0 || seq >= kv->batch) return 0;
     const ForgeModel* m = kv->model;
+    if (m->stack) return sizeof(KvHeader) + stack_kv_bytes_per_token(kv) * kv->len[seq];
     return sizeof(KvHeader) + size_t(2) * m->cfg.num_layers * kv->len[seq] * m->kv * sizeof(__half);
 }
 
@@ -1110,6 +1060,11 @@ int32_t forge_kv_save(ForgeKV* kv, int32_t seq, void* out_host, size_t capacity)
     FORGE_CUDA(cudaSetDevice(m->device));
     const int len = kv->len[seq], L = m->cfg.num_layers;
     KvHeader h{};
+    if (m->stack) {   // the rows of every layer as they lie in the cache, width = bytes per position
+        memcpy(h.magic, kLatentMagic, 4); h.layers = uint32_t(L); h.width = uint32_t(stack_kv_bytes_per_token(kv)); h.len = uint64_t(len);
+        memcpy(out_host, &h, sizeof(h));
+        return stack_kv_copy(kv, seq, len, static_cast<char*>(out_host) + sizeof(h), true);
+    }
     memcpy(h.magic, kKvMagic, 4); h.layers = uint32_t(L); h.width = uint32_t(m->kv); h.len = uint64_t(len);
     memcpy(out_host, &h, sizeof(h));
     __half* dst = reinterpret_cast<__half*>(static_cast<char*>(out_host) + sizeof(h));
@@ -1130,6 +1085,18 @@ int32_t forge_kv_load(ForgeKV* kv, int32_t seq, const void* data_host, size_t n)
     const uint8_t* p = static_cast<const uint8_t*>(data_host);
     std::vector<__half> rows;  // [2][L][len][W]
     uint64_t len = 0;
+    if (m->stack) {
+        KvHeader h;
+        if (n < sizeof(h)) { set_error("forge_kv_load: no data"); return FORGE_ERR_INVALID_ARG; }
+        memcpy(&h, p, sizeof(h));
+        if (memcmp(h.magic, kLatentMagic, 4) || h.layers != uint32_t(L) || h.width != uint32_t(stack_kv_bytes_per_token(kv))) { set_error("forge_kv_load: not a cache file of this model"); return FORGE_ERR_SHAPE; }
+        if (h.len > uint64_t(kv->max_seq) || n != sizeof(h) + size_t(h.width) * h.len) { set_error("forge_kv_load: bad length"); return FORGE_ERR_SHAPE; }
+        FORGE_TRY(forge_kv_free_seq(kv, seq));
+        FORGE_TRY(ensure_pages(kv, seq, int(h.len)));
+        FORGE_TRY(stack_kv_copy(kv, seq, int(h.len), reinterpret_cast<char*>(const_cast<uint8_t*>(p)) + sizeof(h), false));
+        kv->len[seq] = int(h.len);
+        return upload_len(kv);
+    }
     if (n >= sizeof(KvHeader) && memcmp(p, kKvMagic, 4) == 0) {
         KvHeader h;
         memcpy(&h, p, sizeof(h));
@@ -1172,7 +1139,7 @@ int32_t forge_forward_prefill_seq(ForgeModel* m, ForgeKV* kv, int32_t seq, const
     FORGE_CUDA(cudaSetDevice(m->device));
     for (size_t i = 0; i < n; ++i) if (tokens[i] >= uint32_t(m->V)) { set_error("token id %u out of vocabulary", tokens[i]); return FORGE_ERR_INVALID_ARG; }
     if (kv->len[seq] + int(n) > kv->max_seq) { set_error("KV cache full: %d + %zu > max_seq %d", kv->len[seq], n, kv->max_seq); return FORGE_ERR_KV_FULL; }
-    if (n < FORGE_PREFILL_BATCH_THRESHOLD && !m->trace_on) {
+    if (n < FORGE_PREFILL_BATCH_THRESHOLD && !m->trace_on && !m->stack) {
         // emit.rs:4581: short prompts take the per-token path
         for (size_t i = 0; i < n; ++i) FORGE_TRY(forge_forward_seq(m, kv, seq, tokens[i], (i + 1 == n) ? logits_host : nullptr));
         return FORGE_OK;
@@ -1199,6 +1166,7 @@ int32_t forge_forward_seq(ForgeModel* m, ForgeKV* kv, int32_t seq, uint32_t toke
     if (token >= uint32_t(m->V)) { set_error("token id %u out of vocabulary", token); return FORGE_ERR_INVALID_ARG; }
     FORGE_CUDA(cudaSetDevice(m->device));
     FORGE_TRY(ensure_decode_scratch(m, 1));
+    if (m->stack) FORGE_TRY(stack_ensure_decode(m, kv, 1));
     FORGE_TRY(ensure_pages(kv, seq, kv->len[seq] + 1));
     if (m->trace_on) FORGE_TRY(ensure_trace(m, 1));
     FORGE_CUDA(cudaMemcpyAsync(m->d_tok, &token, sizeof(uint32_t), cudaMemcpyHostToDevice, m->stream));
@@ -1228,6 +1196,7 @@ int32_t forge_forward_batch(ForgeModel* m, ForgeKV* kv, int32_t batch, const uin
     for (int b = 0; b < batch; ++b) if (tokens[b] >= uint32_t(m->V)) { set_error("token id %u out of vocabulary", tokens[b]); return FORGE_ERR_INVALID_ARG; }
     FORGE_CUDA(cudaSetDevice(m->device));
     FORGE_TRY(ensure_decode_scratch(m, batch));
+    if (m->stack) FORGE_TRY(stack_ensure_decode(m, kv, batch));
     FORGE_TRY(decode_prepare(kv, batch));
     if (m->trace_on) FORGE_TRY(ensure_trace(m, batch));
     FORGE_CUDA(cudaMemcpyAsync(m->d_tok, tokens, sizeof(uint32_t) * batch, cudaMemcpyHostToDevice, m->stream));
@@ -1236,6 +1205,48 @@ int32_t forge_forward_batch(ForgeModel* m, ForgeKV* kv, int32_t batch, const uin
     FORGE_TRY(sync_and_check(m, kv));
     for (int b = 0; b < batch; ++b) kv->len[b] += 1;
     return FORGE_OK;
+}
+
+int32_t forge_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, int32_t n_entries, const uint32_t* tokens, const int32_t* want, float* logits_host) {
+    if (!m || !kv || !entries || n_entries <= 0 || !tokens || kv->model != m) { set_error("bad argument to forge_step"); return FORGE_ERR_INVALID_ARG; }
+    std::vector<char> seen(size_t(kv->batch), 0);
+    size_t n_tok = 0, n_want = 0;
+    long long new_pages = 0;
+    for (int i = 0; i < n_entries; ++i) {
+        const ForgeStepEntry& e = entries[i];
+        FORGE_TRY(check_seq(kv, e.seq));
+        if (seen[e.seq] || e.n_tokens <= 0 || e.n_tokens > (1 << 20) || e.n_want < 0 || (e.n_want && !want)) { set_error("forge_step: bad entry %d", i); return FORGE_ERR_INVALID_ARG; }
+        seen[e.seq] = 1;
+        for (int k = 0; k < e.n_tokens; ++k) if (tokens[n_tok + k] >= uint32_t(m->V)) { set_error("token id %u out of vocabulary", tokens[n_tok + k]); return FORGE_ERR_INVALID_ARG; }
+        for (int k = 0; k < e.n_want; ++k) {
+            const int w = want[n_want + k];
+            if (w < 0 || w >= e.n_tokens) { set_error("forge_step: entry %d asks for place %d of %d", i, w, e.n_tokens); return FORGE_ERR_INVALID_ARG; }
+            if (!m->stack && (w != e.n_tokens - 1 || e.n_want > 1)) { set_error("forge_step: this model gives the logits of an entry's last token only"); return FORGE_ERR_UNSUPPORTED; }
+        }
+        if (kv->len[e.seq] + e.n_tokens > kv->max_seq) { set_error("KV cache full: %d + %d > max_seq %d", kv->len[e.seq], e.n_tokens, kv->max_seq); return FORGE_ERR_KV_FULL; }
+        new_pages += std::max(0, (kv->len[e.seq] + e.n_tokens + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE - kv->pages_used[e.seq]);
+        n_tok += e.n_tokens; n_want += e.n_want;
+    }
+    if (n_want && !logits_host) { set_error("forge_step: no buffer for the logits"); return FORGE_ERR_INVALID_ARG; }
+    if (new_pages > (long long)kv->free_pages.size()) { set_error("KV page pool exhausted"); return FORGE_ERR_KV_FULL; }
+    FORGE_CUDA(cudaSetDevice(m->device));
+    if (!m->stack) {
+        for (int i = 0; i < n_entries; ++i) {
+            FORGE_TRY(forge_forward_prefill_seq(m, kv, entries[i].seq, tokens, size_t(entries[i].n_tokens), entries[i].n_want ? logits_host : nullptr));
+            tokens += entries[i].n_tokens;
+            if (entries[i].n_want) logits_host += m->V;
+        }
+        return FORGE_OK;
+    }
+    for (int i = 0; i < n_entries; ++i) FORGE_TRY(ensure_pages(kv, entries[i].seq, kv->len[entries[i].seq] + entries[i].n_tokens));
+    const int trace_rows = m->trace_on && n_entries == 1 ? entries[0].n_tokens : 0;
+    if (trace_rows) FORGE_TRY(ensure_trace(m, trace_rows));
+    float* d_logits = nullptr;
+    FORGE_TRY(stack_step(m, kv, entries, n_entries, tokens, want, &d_logits, trace_rows, 0));
+    if (n_want) FORGE_CUDA(cudaMemcpyAsync(logits_host, d_logits, sizeof(float) * n_want * m->V, cudaMemcpyDeviceToHost, m->stream));
+    FORGE_TRY(sync_and_check(m, kv));
+    for (int i = 0; i < n_entries; ++i) kv->len[entries[i].seq] += entries[i].n_tokens;
+    return upload_len(kv);
 }
 
 static int32_t ensure_hist(ForgeModel* m, int n) {
@@ -1251,6 +1262,7 @@ int32_t forge_decode_greedy_batch(ForgeModel* m, ForgeKV* kv, int32_t batch, con
         if (kv->len[b] + n_new > kv->max_seq) { set_error("KV cache full: %d + %d > max_seq %d", kv->len[b], n_new, kv->max_seq); return FORGE_ERR_KV_FULL; }
     }
     FORGE_TRY(ensure_decode_scratch(m, batch));
+    if (m->stack) FORGE_TRY(stack_ensure_decode(m, kv, batch));
     FORGE_TRY(ensure_hist(m, n_new * batch));
     long long l0 = g_launches;
     FORGE_CUDA(cudaMemcpyAsync(m->d_tok, first_tokens, sizeof(uint32_t) * batch, cudaMemcpyHostToDevice, m->stream));
@@ -1289,7 +1301,7 @@ int32_t forge_generate_greedy(ForgeModel* m, ForgeKV* kv, const uint32_t* prompt
     long long l0 = g_launches;
     const int len_entry = kv->len[0];
     FORGE_CUDA(cudaEventRecord(m->ev[0], m->stream));
-    if (n < FORGE_PREFILL_BATCH_THRESHOLD) {
+    if (n < FORGE_PREFILL_BATCH_THRESHOLD && !m->stack) {
         for (size_t i = 0; i < n; ++i) FORGE_TRY(forge_forward_seq(m, kv, 0, prompt[i], nullptr));
     } else {
         FORGE_TRY(prefill_seq(m, kv, 0, prompt, int(n)));

@@ -11,10 +11,12 @@ library copies to and from the GPU itself.
 from __future__ import annotations
 
 import ctypes as C
+import json
+import os
 
 import numpy as np
 
-from ._lib import ForgeError, ForgeModelConfig, check, lib
+from ._lib import ForgeCheckpointInfo, ForgeError, ForgeModelConfig, ForgeStepEntry, check, lib
 
 
 def _cfg_struct(c: dict, tp_rank: int = 0, tp_world: int = 1) -> ForgeModelConfig:
@@ -60,12 +62,25 @@ def quantize_kquant(quant: int, x: np.ndarray) -> np.ndarray:
 class KVCache:
     """``KVCache`` of the generated module (emit.rs:3954-4015): fp16, paged, ``batch`` sequences."""
 
-    def __init__(self, model: "Model", max_seq: int | None = None, batch: int = 1):
+    def __init__(self, model: "Model", max_seq: int | None = None, batch: int = 1, pool_tokens: int | None = None):
+        """``pool_tokens``: positions the sequences share (default: room for ``batch`` full sequences)."""
         self.model = model
         self.batch = batch
         h = C.c_void_p()
-        check(lib.forge_kv_create(model._h, int(max_seq or model.cfg["max_seq_len"]), batch, C.byref(h)))
+        n = int(max_seq or model.cfg["max_seq_len"])
+        if pool_tokens is None:
+            check(lib.forge_kv_create(model._h, n, batch, C.byref(h)))
+        else:
+            check(lib.forge_kv_create_pool(model._h, int(pool_tokens), n, batch, C.byref(h)))
         self._h = h
+
+    def free_seq(self, seq: int) -> None:
+        """Sequence ``seq`` back to length 0, its pages to the pool."""
+        check(lib.forge_kv_free_seq(self._h, seq))
+
+    def free_tokens(self) -> int:
+        """Positions the pool can still take, in whole pages."""
+        return int(lib.forge_kv_free_tokens(self._h))
 
     def reset(self) -> None:
         check(lib.forge_kv_reset(self._h))
@@ -74,7 +89,11 @@ class KVCache:
         return int(lib.forge_kv_len(self._h, seq))
 
     def read(self, layer: int, which: int, seq: int = 0) -> np.ndarray:
-        kvd = self.model.cfg["num_kv_heads"] * self.model.cfg["head_dim"] // self.model.tp_world
+        if "layers" in self.model.cfg:   # latents (which = 0) or rotated key parts (1)
+            m = self.model.cfg["layers"][layer]["mixer"]
+            kvd = m["rot_dim"] if which else m["kv_rank"]
+        else:
+            kvd = self.model.cfg["num_kv_heads"] * self.model.cfg["head_dim"] // self.model.tp_world
         out = np.empty((self.len(seq), kvd), np.float32)
         check(lib.forge_kv_read(self._h, seq, layer, which, _p(out)))
         return out
@@ -102,6 +121,17 @@ class KVCache:
             pass
 
 
+DTYPES = {"bfloat16": 30, "float32": 32}  # FORGE_BF16, FORGE_F32
+
+
+def checkpoint_info(path: str) -> dict:
+    """What a checkpoint folder (config.json, model.safetensors) holds, checked; needs no device."""
+    i = ForgeCheckpointInfo()
+    check(lib.forge_checkpoint_info(os.fsencode(path), C.byref(i)))
+    return {"architecture": i.architecture.decode(), "hidden_size": i.hidden_size, "vocab_size": i.vocab_size, "num_layers": i.num_layers,
+            "num_weight_layers": i.num_weight_layers, "parameters": i.parameters, "cache_values_per_token": i.cache_values_per_token}
+
+
 TP_ID_BYTES = 128  # FORGE_TP_ID_BYTES
 TP_HANDLE_BYTES = 64  # FORGE_TP_HANDLE_BYTES
 
@@ -118,6 +148,24 @@ class Model:
         check(lib.forge_model_create(C.byref(s), _p(blob), blob.size, device, C.byref(h)))
         self._h = h
         self.device = device
+
+    @classmethod
+    def open(cls, path: str, dtype: str = "bfloat16", device: int = 0) -> "Model":
+        """A layer-list model from a checkpoint folder; config.json chooses the architecture."""
+        if dtype not in DTYPES:
+            raise ValueError(f"dtype must be one of {sorted(DTYPES)}")
+        m = cls.__new__(cls)
+        h = C.c_void_p()
+        check(lib.forge_model_open(os.fsencode(path), DTYPES[dtype], device, C.byref(h)))
+        m._h = h
+        i = ForgeCheckpointInfo()
+        check(lib.forge_model_info(h, C.byref(i)))
+        with open(os.path.join(path, "config.json")) as f:
+            m.cfg = json.load(f)
+        m.cfg.update(hidden_size=i.hidden_size, vocab_size=i.vocab_size, num_layers=i.num_layers, max_seq_len=4096, dtype=dtype)
+        m.tp_world = 1
+        m.device = device
+        return m
 
     @property
     def stream(self) -> int:
@@ -150,8 +198,21 @@ class Model:
             raise ValueError("one handle per rank, in rank order")
         check(lib.forge_model_tp_exchange_attach(self._h, _p(h)))
 
-    def new_cache(self, max_seq: int | None = None, batch: int = 1) -> KVCache:
-        return KVCache(self, max_seq, batch)
+    def new_cache(self, max_seq: int | None = None, batch: int = 1, pool_tokens: int | None = None) -> KVCache:
+        return KVCache(self, max_seq, batch, pool_tokens)
+
+    def step(self, entries, cache: KVCache) -> list[np.ndarray]:
+        """One mixed batch: ``entries`` = [(seq, tokens, wanted places)]; returns the wanted logits of every entry."""
+        arr = (ForgeStepEntry * len(entries))(*[ForgeStepEntry(int(s), len(t), len(w)) for s, t, w in entries])
+        toks = np.fromiter((x for _, t, _ in entries for x in t), np.uint32)
+        want = np.fromiter((x for _, _, w in entries for x in w), np.int32)
+        logits = np.empty((want.size, self.cfg["vocab_size"]), np.float32)
+        check(lib.forge_step(self._h, cache._h, arr, len(entries), _p(toks), _p(want), _p(logits) if want.size else None))
+        out, at = [], 0
+        for _, _, w in entries:
+            out.append(logits[at:at + len(w)])
+            at += len(w)
+        return out
 
     def forward(self, token: int, cache: KVCache, seq: int = 0, want_logits: bool = True):
         logits = np.empty(self.cfg["vocab_size"], np.float32) if want_logits else None

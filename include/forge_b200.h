@@ -50,6 +50,10 @@ typedef enum ForgeStatus {
 #define FORGE_Q6_K 14 /* 210 bytes {u8 ql[128]; u8 qh[64]; i8 scales[16]; f16 d},
                          value = d*scales[i/16]*(q6-32)                             (E:3542-3546, WL:997-1060) */
 
+/* Storage and compute types of the layer-list models (forge_model_open). */
+#define FORGE_BF16 30 /* bfloat16 weights, activations and cache; f32 accumulation, residual, norms and attention scores */
+#define FORGE_F32 32  /* everything in f32 (no reduced-precision matrix mode) */
+
 #define FORGE_PREFILL_BATCH_THRESHOLD 8 /* E:203-206 */
 #define FORGE_KV_PAGE 64                /* positions per KV page (= FLASH_ATTN_BLOCK_SIZE, E:199-202) */
 
@@ -218,6 +222,27 @@ void forge_model_destroy(ForgeModel* model);
 /* The CUDA stream (cudaStream_t) all work of this model is launched on. */
 void* forge_model_stream(ForgeModel* model);
 
+/* ---- Layer-list models: a checkpoint folder with config.json and model.safetensors.  config.json names an architecture
+ * and lists the layers, each with its mixer, the mixer's sizes and its feed-forward; sizes and constants are read from
+ * there.  Every session call below takes such a model like any other.  (No counterpart in the reference, whose models are
+ * GGUF decoders.)  Registered architectures: "Bolenex" (latent attention and a clamped gated feed-forward in parallel behind
+ * one Dynamic Tanh norm).  An unknown architecture, mixer or feed-forward returns FORGE_ERR_UNSUPPORTED; a missing key, a
+ * missing tensor or a wrong shape FORGE_ERR_SHAPE. */
+typedef struct ForgeCheckpointInfo {
+    char architecture[64];
+    int32_t hidden_size;
+    int32_t vocab_size;
+    int32_t num_layers;              /* layer runs */
+    int32_t num_weight_layers;       /* layers with tensors of their own */
+    int64_t parameters;              /* values in the checkpoint's tensors */
+    int64_t cache_values_per_token;  /* values the cache keeps per position, padding included */
+} ForgeCheckpointInfo;
+/* Reads and checks a checkpoint folder without a device. */
+int32_t forge_checkpoint_info(const char* dir, ForgeCheckpointInfo* out);
+/* Loads it; dtype: FORGE_BF16 or FORGE_F32. */
+int32_t forge_model_open(const char* dir, int32_t dtype, int32_t device, ForgeModel** out);
+int32_t forge_model_info(const ForgeModel* model, ForgeCheckpointInfo* out);
+
 /* Tensor parallelism (one process per GPU, cfg.tp_world ranks).  The attention-output and FFN-down projections are
  * row-sliced, so their results are summed over the ranks (an NCCL all-reduce on the model's stream) before the
  * residual is added; every rank ends with the same hidden state and computes the full logits.
@@ -266,13 +291,21 @@ int32_t forge_model_set_wait_limit(ForgeModel* model, uint32_t polls);
 /* KVCache::new (E:3978-4000) for `batch` independent sequences of up to max_seq positions,
  * fp16, paged (FORGE_KV_PAGE positions per page, pages handed out on demand). */
 int32_t forge_kv_create(ForgeModel* model, int32_t max_seq, int32_t batch, ForgeKV** out);
+/* The same with a page pool smaller than batch * max_seq: `pool_tokens` positions (rounded up to whole pages) are shared by
+ * the `batch` sequences; a call that needs a page when none is left returns FORGE_ERR_KV_FULL. */
+int32_t forge_kv_create_pool(ForgeModel* model, int32_t pool_tokens, int32_t max_seq, int32_t batch, ForgeKV** out);
+/* Sequence `seq` back to length 0; its pages return to the pool. */
+int32_t forge_kv_free_seq(ForgeKV* kv, int32_t seq);
+/* Positions the pool can still take in whole pages; -1 on a bad argument. */
+int64_t forge_kv_free_tokens(const ForgeKV* kv);
 /* KVCache::reset (E:4002-4005): all sequences back to length 0, pages returned. */
 int32_t forge_kv_reset(ForgeKV* kv);
 /* cache.len of sequence `seq`; -1 on a bad argument. */
 int32_t forge_kv_len(const ForgeKV* kv, int32_t seq);
 void forge_kv_destroy(ForgeKV* kv);
 /* Copy K (which = 0) or V (1) rows [0, len) of `layer`, sequence `seq`, widened to f32, into
- * a host buffer [len][num_kv_heads*head_dim] (used by parity tests). */
+ * a host buffer [len][num_kv_heads*head_dim] (used by parity tests).  Latent attention: the latents (0, [len][kv_rank]) or
+ * the rotated key parts (1, [len][rot_dim]). */
 int32_t forge_kv_read(ForgeKV* kv, int32_t seq, int32_t layer, int32_t which, float* out_host);
 
 /* KV cache persistence (save_kv_cache / load_kv_cache of the generated main.rs, project.rs:456-499).
@@ -301,6 +334,19 @@ int32_t forge_forward_prefill_seq(ForgeModel* model, ForgeKV* kv, int32_t seq, c
  * logits_host: [batch][V] or NULL. */
 int32_t forge_forward_batch(ForgeModel* model, ForgeKV* kv, int32_t batch, const uint32_t* tokens,
                             float* logits_host);
+/* One step of a mixed batch: portions of prompts beside single decoded tokens.  entries[i] brings the next n_tokens tokens
+ * of sequence entries[i].seq (each sequence at most once) and asks for the logits behind n_want of them; `tokens` holds the
+ * entries' tokens one after another, `want` the wanted places, each counted from the start of its entry.
+ * logits_host: [sum of n_want][V] in that order (may be NULL if nothing is wanted).  On an error no sequence has advanced.
+ * Layer-list models run the entries as one batch; a quantised decoder serves them one after another and can be asked
+ * for an entry's last place only (FORGE_ERR_UNSUPPORTED otherwise). */
+typedef struct ForgeStepEntry {
+    int32_t seq;
+    int32_t n_tokens;
+    int32_t n_want;
+} ForgeStepEntry;
+int32_t forge_step(ForgeModel* model, ForgeKV* kv, const ForgeStepEntry* entries, int32_t n_entries, const uint32_t* tokens,
+                   const int32_t* want, float* logits_host);
 /* The generated main's greedy loop (P:714-751 with temperature 0 and repeat penalty 1.0):
  * prefill the prompt, then n_new times {argmax, forward}, token selection on the device.
  * out_tokens: host u32 [n_new]. */

@@ -1,0 +1,239 @@
+"""Plain restatement of the layer-list models (a ``config.json`` whose "layers" entry lists mixers and feed-forwards):
+one function per mechanism, numpy, written from the equations, slow on purpose.  The Bolenex design: latent attention
+and a clamped gated feed-forward in parallel behind one Dynamic Tanh norm.
+
+TEST INFRASTRUCTURE ONLY, like the rest of this folder; it shares no code with the shipped package.  Everything is computed in
+``dtype`` (float64 by default).  A sequence is evaluated as a whole: there is no cache, no page and no batch here.
+"""
+from __future__ import annotations
+
+import json
+import math
+import os
+import struct
+
+import numpy as np
+
+
+# ---------------------------------------------------------------------------------------------- mechanisms
+def rms_norm(x, weight, eps):
+    """x / sqrt(mean(x^2) + eps) * weight over the last axis."""
+    return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps) * weight
+
+
+def dynamic_tanh(x, alpha, weight, bias):
+    """Element by element: tanh(alpha x) weight + bias."""
+    return np.tanh(alpha * x) * weight + bias
+
+
+def rotate_half(x, positions, base, dims):
+    """Rotary positions on the first ``dims`` entries of the last axis; entry i turns with entry i + dims/2.
+    x: [tokens, ..., n], positions: [tokens]."""
+    half = dims // 2
+    freq = np.array([base ** (-2.0 * i / dims) for i in range(half)], np.float64)
+    ang = np.asarray(positions, np.float64)[:, None] * freq[None, :]
+    shape = (len(positions),) + (1,) * (x.ndim - 2) + (half,)
+    c, s = np.cos(ang).reshape(shape).astype(x.dtype), np.sin(ang).reshape(shape).astype(x.dtype)
+    out = x.copy()
+    u, v = x[..., :half], x[..., half:dims]
+    out[..., :half] = u * c - v * s
+    out[..., half:dims] = v * c + u * s
+    return out
+
+
+def causal_softmax_attention(q, k, v, scale):
+    """q, k: [tokens, heads, d], v: [tokens, heads, dv]; position i sees every j <= i."""
+    n, heads, _ = q.shape
+    out = np.zeros((n, heads, v.shape[2]), q.dtype)
+    for h in range(heads):
+        s = (q[:, h] @ k[:, h].T) * q.dtype.type(scale)
+        for i in range(n):
+            row = s[i, : i + 1]
+            w = np.exp(row - row.max())
+            out[i, h] = (w / w.sum()) @ v[: i + 1, h]
+    return out
+
+
+def sigmoid(z):
+    return 1.0 / (1.0 + np.exp(-z))
+
+
+def latent_attention(h, w, m, eps, positions=None):
+    """h: [tokens, width]; ``w(name)`` gives a tensor of the mixer, ``m`` its sizes."""
+    n = h.shape[0]
+    H, d, r, dv, rank = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    pos = np.arange(n) if positions is None else positions
+    q = (h @ w("q").T).reshape(n, H, d + r)
+    down = h @ w("dkv").T
+    c = rms_norm(down[:, :rank], w("dkv.norm"), eps)
+    rot = m["rot"]
+    k_rot = rotate_half(down[:, rank:], pos, rot["base"], rot["dims"])
+    q_rot = rotate_half(q[:, :, d:], pos, rot["base"], rot["dims"])
+    k_un = (c @ w("uk").T).reshape(n, H, d)
+    v = (c @ w("uv").T).reshape(n, H, dv)
+    qq = np.concatenate([q[:, :, :d], q_rot], axis=2)
+    kk = np.concatenate([k_un, np.broadcast_to(k_rot[:, None, :], (n, H, r))], axis=2)
+    o = causal_softmax_attention(qq, kk, v, m["scale"]).reshape(n, H * dv)
+    return (o * sigmoid(h @ w("g").T)) @ w("o").T
+
+
+def clamped_glu(gate, up, limit):
+    """g sigmoid(1.702 g) (u + 1) with g = min(gate, limit) and u = up held within +-limit."""
+    g = np.minimum(gate, limit)
+    u = np.clip(up, -limit, limit)
+    return g * sigmoid(1.702 * g) * (u + 1.0)
+
+
+def dense_ff(h, w, m):
+    return clamped_glu(h @ w("gate").T, h @ w("up").T, h.dtype.type(m["limit"])) @ w("down").T
+
+
+# ---------------------------------------------------------------------------------------------- the model
+class LayerStack:
+    """``config``: the parsed config.json; ``tensors``: name -> array."""
+
+    def __init__(self, config: dict, tensors: dict, dtype=np.float64):
+        self.cfg = config
+        self.t = {k: np.asarray(v, dtype) for k, v in tensors.items()}
+        self.dtype = dtype
+
+    def norm(self, x, name):
+        return dynamic_tanh(x, self.t[name + ".alpha"], self.t[name], self.t[name + ".b"])
+
+    def layer(self, x, i):
+        L = self.cfg["layers"][i]
+        p = f"l{L.get('weights_of', i)}."
+        h = self.norm(x, p + "norm1")
+        y = latent_attention(h, lambda n: self.t[p + "mix." + n], L["mixer"], self.cfg["norm"]["eps"])
+        if L.get("mlp"):
+            y = y + dense_ff(h, lambda n: self.t[p + "mlp." + n], L["mlp"])
+        return x + y
+
+    def residuals(self, tokens):
+        """The residual stream after every layer: [layers, tokens, width]."""
+        x = self.t["embed"][np.asarray(tokens, np.int64)]
+        out = []
+        for i in range(len(self.cfg["layers"])):
+            x = self.layer(x, i)
+            out.append(x)
+        return np.stack(out)
+
+    def logits(self, tokens):
+        """[tokens, vocab]: the logits behind every position."""
+        return self.norm(self.residuals(tokens)[-1], "final.norm") @ self.t["head"].T
+
+    def generate_greedy(self, prompt, n_new):
+        """The next n_new tokens, the last index winning a tie."""
+        toks = [int(t) for t in prompt]
+        for _ in range(n_new):
+            row = self.logits(toks)[-1]
+            toks.append(int(np.flatnonzero(row == row.max())[-1]))
+        return toks[len(prompt):]
+
+
+# ---------------------------------------------------------------------------------------------- files
+def bf16_bits(x):
+    """float32 -> bfloat16 bit patterns, round to nearest even."""
+    u = np.ascontiguousarray(x, np.float32).view(np.uint32).astype(np.uint64)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+
+def bf16_round(x):
+    return (bf16_bits(x).astype(np.uint32) << 16).view(np.float32)
+
+
+def read_safetensors(path):
+    with open(path, "rb") as f:
+        n = struct.unpack("<Q", f.read(8))[0]
+        head = json.loads(f.read(n))
+        data = f.read()
+    out = {}
+    for name, d in head.items():
+        if name == "__metadata__":
+            continue
+        a, b = d["data_offsets"]
+        raw = data[a:b]
+        if d["dtype"] == "BF16":
+            arr = (np.frombuffer(raw, np.uint16).astype(np.uint32) << 16).view(np.float32)
+        else:
+            arr = np.frombuffer(raw, {"F32": np.float32, "F16": np.float16, "I32": np.int32}[d["dtype"]])
+        out[name] = arr.reshape(d["shape"])
+    return out
+
+
+def write_model(folder, config, tensors):
+    """config.json and model.safetensors (bfloat16, the tensors as they are given)."""
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(config, f, indent=1)
+    head, blobs, off = {}, [], 0
+    for name, arr in tensors.items():
+        b = bf16_bits(arr).tobytes()
+        head[name] = {"dtype": "BF16", "shape": list(np.shape(arr)), "data_offsets": [off, off + len(b)]}
+        blobs.append(b)
+        off += len(b)
+    h = json.dumps(head).encode()
+    with open(os.path.join(folder, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(h)))
+        f.write(h)
+        for b in blobs:
+            f.write(b)
+
+
+def load(folder, dtype=np.float64):
+    with open(os.path.join(folder, "config.json")) as f:
+        cfg = json.load(f)
+    return LayerStack(cfg, read_safetensors(os.path.join(folder, "model.safetensors")), dtype)
+
+
+# ---------------------------------------------------------------------------------------------- seeded models
+def mixer(heads=3, dim=24, rot_dim=8, vdim=40, kv_rank=56, base=5000.0, scale=None):
+    return {"dim": dim, "heads": heads, "kv_rank": kv_rank, "rot": {"base": float(base), "dims": rot_dim}, "rot_dim": rot_dim,
+            "scale": float(scale if scale is not None else 1.0 / math.sqrt(dim + rot_dim)), "vdim": vdim}
+
+
+def make_config(width=136, vocab=203, layers=(), eps=1e-5):
+    """``layers``: (mixer, ff size or None, limit, weights_of or None) per layer."""
+    out = []
+    for mx, ff, limit, of in layers:
+        e = {"mixer": mx, "mlp": None if ff is None else {"ff": ff, "kind": "dense", "limit": float(limit)}, "type": "latent_attention"}
+        if of is not None:
+            e["weights_of"] = of
+        out.append(e)
+    return {"architecture": "Bolenex", "layers": out, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def random_tensors(cfg, seed=0):
+    """Seeded weights, rounded to bfloat16, in which every factor matters (norm weights and biases away from 1 and 0)."""
+    rng = np.random.default_rng(seed)
+    W = cfg["width"]
+    t = {}
+
+    def mat(name, out, inp, gain=1.0):
+        t[name] = bf16_round(rng.standard_normal((out, inp)) * (gain / math.sqrt(inp)))
+
+    def norm(name):
+        t[name] = bf16_round(1.0 + 0.3 * rng.standard_normal(W))
+        t[name + ".b"] = bf16_round(0.2 * rng.standard_normal(W))
+        t[name + ".alpha"] = bf16_round(np.asarray(0.5 + 0.4 * rng.random()))
+
+    t["embed"] = bf16_round(rng.standard_normal((cfg["vocab"], W)))
+    for i, L in enumerate(cfg["layers"]):
+        if "weights_of" in L:
+            continue
+        p, m = f"l{i}.", L["mixer"]
+        norm(p + "norm1")
+        mat(p + "mix.q", m["heads"] * (m["dim"] + m["rot_dim"]), W, 1.5)
+        mat(p + "mix.dkv", m["kv_rank"] + m["rot_dim"], W)
+        t[p + "mix.dkv.norm"] = bf16_round(1.0 + 0.3 * rng.standard_normal(m["kv_rank"]))
+        mat(p + "mix.uk", m["heads"] * m["dim"], m["kv_rank"], 1.5)
+        mat(p + "mix.uv", m["heads"] * m["vdim"], m["kv_rank"])
+        mat(p + "mix.g", m["heads"] * m["vdim"], W, 2.0)
+        mat(p + "mix.o", W, m["heads"] * m["vdim"], 2.0)
+        if L.get("mlp"):
+            mat(p + "mlp.gate", L["mlp"]["ff"], W, 1.5)
+            mat(p + "mlp.up", L["mlp"]["ff"], W, 1.5)
+            mat(p + "mlp.down", W, L["mlp"]["ff"], 1.0)
+    norm("final.norm")
+    mat("head", cfg["vocab"], W)
+    return t
