@@ -2,6 +2,7 @@
 """Benchmark of the quantized forward path on B200.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
+    python bench.py --design bolenex          (another model design, one GPU; the default workload is unchanged)
 
 One GPU (the default).  Headline workload: the Llama-3.2-1B-shaped Q4_0 decoder of the benchmark definition - one
 "step" is one request: a 1501-token uniform-random prompt through the batched prefill path, then 128 greedy decode
@@ -403,6 +404,110 @@ def run_single(args, device: int):
     print(json.dumps(line), flush=True)
 
 
+# ---------------------------------------------------------------------------- one GPU: the Bolenex design beside a Llama-shaped decoder
+# (width, layers, heads of 128, ff): a 1B- and a 7B-shaped layer
+BOLENEX_SIZES = {"w2048": (2048, 16, 16, 8192), "w4096": (4096, 8, 32, 11008)}
+BOLENEX_VOCAB, BOLENEX_PROMPT, BOLENEX_DECODE = 32768, 2048, 64
+
+
+def bolenex_work(cfg: dict, ctx: int, m: int):
+    """(bytes of a batch-1 decode step: weights once; cache bytes of one sequence at `ctx`; useful flops of an m-token prompt)."""
+    W, V = cfg["width"], cfg["vocab"]
+    w = kv = flops = 0.0
+    for L in cfg["layers"]:
+        x, ff = L["mixer"], L["mlp"]["ff"]
+        qk, hv = x["dim"] + x["rot_dim"], x["heads"] * x["vdim"]
+        lin = W * (x["heads"] * qk + x["kv_rank"] + x["rot_dim"] + hv + 2 * ff) + W * (hv + ff)
+        exp = x["kv_rank"] * x["heads"] * (x["dim"] + x["vdim"])
+        w += 2 * (lin + exp)
+        kv += 2 * (x["kv_rank"] + x["rot_dim"])
+        flops += 2.0 * m * (lin + exp) + 2.0 * x["heads"] * (qk + x["vdim"]) * m * (m + 1) / 2
+    return w + 2 * V * W, kv * ctx, flops + 2.0 * V * W
+
+
+def run_bolenex(args, device: int):
+    """Prefill and decode rates of the Bolenex design and, at equal width, depth, heads and feed-forward, of the framework's closest
+    decoder (multi-head, head_dim 128, Q8_0), each against its own roofline."""
+    import torch
+    from forge_llm_b200 import configs, runtime, synth
+    peaks = load_peaks()
+    sampler = ClockSampler(device)
+    t0 = time.time()
+    out, launches = {}, 0
+
+    def measure(model, batch, n_prompt, n_dec, bytes_w, bytes_kv, flops, vocab):
+        kv = model.new_cache(max_seq=n_prompt + n_dec + 8, batch=batch)
+        rng = np.random.default_rng(3)
+        prompts = [rng.integers(0, vocab, n_prompt).astype(np.uint32) for _ in range(batch)]
+        pre, dec, host, nl = [], [], [], 0
+        for it in range(args.warmup + args.steps):
+            kv.reset()
+            if batch == 1:
+                h0 = time.perf_counter()
+                model.generate_greedy(prompts[0], n_dec, kv)
+                h1 = time.perf_counter()
+                p, d, l = model.last_timing()
+            else:
+                torch.cuda.synchronize()
+                h0 = time.perf_counter()
+                first = []
+                for b in range(batch):
+                    lg = model.forward_prefill(prompts[b], kv, seq=b)
+                    first.append(int(lg.argmax()))
+                p = 1e3 * (time.perf_counter() - h0)
+                model.decode_greedy_batch(np.array(first, np.uint32), n_dec, kv)
+                h1 = time.perf_counter()
+                _, d, l = model.last_timing()
+            if it >= args.warmup:
+                pre.append(p); dec.append(d); host.append(h1 - h0); nl += l
+        kv.close()
+        step = statistics.median(dec) / n_dec * 1e-3
+        gbs = (bytes_w + batch * bytes_kv) / step / 1e9
+        tf = batch * flops / (statistics.median(pre) * 1e-3) / 1e12
+        return {"batch": batch, "decode_tok_s": batch / step, "us_per_step": step * 1e6,
+                "decode_roofline": {"bound": "hbm", "achieved": gbs, "peak": peaks["hbm_gbs"], "unit": "GB/s", "frac": gbs / peaks["hbm_gbs"]},
+                "prefill_tok_s": batch * n_prompt / (statistics.median(pre) * 1e-3), "prefill_timing": "device" if batch == 1 else "host, around the C-ABI calls",
+                "prefill_roofline": {"bound": "tensor", "achieved": tf, "peak": peaks["bf16_tflops"], "unit": "TFLOP/s", "frac": tf / peaks["bf16_tflops"]},
+                "e2e_s_per_request": statistics.median(host) / batch}, nl
+
+    for name in args.sizes.split(","):
+        width, layers, heads, ff = BOLENEX_SIZES[name]
+        n_prompt, n_dec = args.prompt_tokens or BOLENEX_PROMPT, args.decode_steps or BOLENEX_DECODE
+        if args.layers:
+            layers = args.layers
+        ctx = n_prompt + n_dec // 2
+        rec = {"shape": f"width {width}, {layers} layers, {heads} heads of 128, ff {ff}, vocab {BOLENEX_VOCAB}, {n_prompt}-token prompts, {n_dec} decode steps"}
+        batches = [int(b) for b in args.batches.split(",")]
+        if "bolenex" in args.arms:
+            cfg = synth.bolenex_config(width, layers, heads, ff, BOLENEX_VOCAB)
+            folder = os.path.join(CACHE_DIR, f"bolenex-{width}-{layers}-{os.getpid()}")
+            synth.write_bolenex(folder, cfg)
+            model = runtime.Model.open(folder, "bfloat16", device)
+            shutil.rmtree(folder)
+            rec["bolenex bf16"] = []
+            for b in batches:
+                r, nl = measure(model, b, n_prompt, n_dec, *bolenex_work(cfg, ctx, n_prompt), BOLENEX_VOCAB)
+                rec["bolenex bf16"].append(r)
+                launches += nl
+            model.close()
+        if "llama" in args.arms:
+            c = configs._cfg(f"llama-shape-{width}", width, layers, heads, heads, 128, ff, BOLENEX_VOCAB, 1e4, 8)
+            model = runtime.Model(c, synth.make_weights_bin(c, seed=0, quantize_fn=lambda q, w: runtime.quantize_q8_0(w), repeat_layers=True), device=device)
+            rec["llama-shaped q8_0"] = []
+            w = configs.decode_bytes_per_token(c, 0)
+            for b in batches:
+                r, _ = measure(model, b, n_prompt, n_dec, w, configs.decode_bytes_per_token(c, ctx) - w, configs.prefill_flops(c, n_prompt), BOLENEX_VOCAB)
+                rec["llama-shaped q8_0"].append(r)
+            model.close()
+        out[name] = rec
+        print(f"[bench] {name}: {json.dumps(rec)}", file=sys.stderr, flush=True)
+    clocks = sampler.stop(t0, time.time())
+    first = out[args.sizes.split(",")[0]].get("bolenex bf16", [{}])[0]
+    print(json.dumps({"metric": "bolenex_decode_tok_s", "value": first.get("decode_tok_s"), "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+                      "higher_is_better": True, "dtype": "bf16", "data": "synthetic", "sizes": out, "gpu_launches": int(launches), "clocks": clocks,
+                      "config": {"l2": "every decode step streams weights larger than L2 once", "parallelism": "one GPU"}}), flush=True)
+
+
 # ---------------------------------------------------------------------------- N GPUs: request sharding + tensor parallel
 def run_multi(args, rank: int, world: int, local_rank: int):
     import torch
@@ -575,6 +680,11 @@ def main():
     ap.add_argument("--prompt-tokens", type=int, default=None, help="override the headline prompt length (profiling / experiments)")
     ap.add_argument("--decode-steps", type=int, default=None, help="override the headline number of decode steps")
     ap.add_argument("--profile", action="store_true", help="short run for ncu: no side configurations, no CPU baseline; prints a non-benchmark line")
+    ap.add_argument("--design", default="headline", choices=["headline", "bolenex"], help="bolenex: the Bolenex design beside a Llama-shaped decoder of equal size (one GPU)")
+    ap.add_argument("--sizes", default="w2048,w4096", help="with --design bolenex: which sizes")
+    ap.add_argument("--batches", default="1,16", help="with --design bolenex: sequences decoded together")
+    ap.add_argument("--arms", default="bolenex,llama", help="with --design bolenex: which models")
+    ap.add_argument("--layers", type=int, default=None, help="with --design bolenex: override the depth (profiling)")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
@@ -594,7 +704,9 @@ def main():
         print(f"bench.py: WORLD_SIZE={world} but --gpus {args.gpus}; using WORLD_SIZE", file=sys.stderr)
     if args.gpus > 1 and world == 1:
         raise SystemExit("bench.py: launch multi-GPU runs with torch.distributed.run (one rank per GPU)")
-    if world == 1:
+    if args.design == "bolenex":
+        run_bolenex(args, local_rank)
+    elif world == 1:
         run_single(args, local_rank)
     else:
         run_multi(args, rank, world, local_rank)

@@ -194,3 +194,69 @@ def make_weights_bin(c: dict, seed: int = 0, std: float = 0.02, chunk_rows: int 
 def prompt_tokens(c: dict, n: int, seed: int = 1) -> np.ndarray:
     """Uniform token ids, ``numpy.random.default_rng(seed).integers(0, V)``."""
     return np.random.default_rng(seed).integers(0, c["vocab_size"], size=n).astype(np.uint32)
+
+
+# ------------------------------------------------------------------------------------------------ layer-list models
+def bolenex_config(width: int, layers: int, heads: int, ff: int, vocab: int, dim: int = 128, rot_dim: int = 64, vdim: int = 128, kv_rank: int = 512) -> dict:
+    """config.json of a uniform Bolenex stack."""
+    mixer = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "rot": {"base": 10000.0, "dims": rot_dim},
+             "scale": float((dim + rot_dim) ** -0.5)}
+    entry = {"type": "latent_attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}}
+    return {"architecture": "Bolenex", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "layers": [dict(entry) for _ in range(layers)]}
+
+
+def bolenex_shapes(cfg: dict, layer: int) -> dict:
+    """Tensor shapes of one layer, without its prefix."""
+    W, L = cfg["width"], cfg["layers"][layer]
+    m, f = L["mixer"], L.get("mlp")
+    hv = m["heads"] * m["vdim"]
+    s = {"norm1": (W,), "norm1.b": (W,), "norm1.alpha": (), "mix.q": (m["heads"] * (m["dim"] + m["rot_dim"]), W),
+         "mix.dkv": (m["kv_rank"] + m["rot_dim"], W), "mix.dkv.norm": (m["kv_rank"],), "mix.uk": (m["heads"] * m["dim"], m["kv_rank"]),
+         "mix.uv": (hv, m["kv_rank"]), "mix.g": (hv, W), "mix.o": (W, hv)}
+    if f:
+        s.update({"mlp.gate": (f["ff"], W), "mlp.up": (f["ff"], W), "mlp.down": (W, f["ff"])})
+    return s
+
+
+def write_bolenex(folder: str, cfg: dict, seed: int = 0, repeat_layers: bool = True) -> None:
+    """config.json and model.safetensors (bfloat16): matrices ~ N(0, 1/inputs), norm weights 1, biases 0, alpha 0.5.  With
+    ``repeat_layers`` layer 0's values are drawn and stored again for every later layer (of the same sizes)."""
+    import json
+    import os
+    import struct
+    rng = np.random.default_rng(seed)
+
+    def draw(name, shape):
+        if name.endswith("alpha"):
+            x = np.full(shape, 0.5, np.float32)
+        elif len(shape) < 2:
+            x = np.zeros(shape, np.float32) if name.endswith(".b") else np.ones(shape, np.float32)
+        else:
+            x = rng.standard_normal(shape, np.float32) * np.float32(shape[1] ** -0.5)
+        return (np.ascontiguousarray(x).view(np.uint32) >> 16).astype(np.uint16)
+
+    W, V = cfg["width"], cfg["vocab"]
+    parts = [(n, s) for n, s in (("embed", (V, W)), ("head", (V, W)), ("final.norm", (W,)), ("final.norm.b", (W,)), ("final.norm.alpha", ()))]
+    for i, L in enumerate(cfg["layers"]):
+        if "weights_of" not in L:
+            parts += [(f"l{i}.{n}", s) for n, s in bolenex_shapes(cfg, i).items()]
+    head, off = {}, 0
+    for n, s in parts:
+        size = 2 * int(np.prod(s, dtype=np.int64))
+        head[n] = {"dtype": "BF16", "shape": list(s), "data_offsets": [off, off + size]}
+        off += size
+    os.makedirs(folder, exist_ok=True)
+    text = json.dumps(head).encode()
+    kept: dict = {}
+    with open(os.path.join(folder, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(text)) + text)
+        for n, s in parts:
+            key = (n.split(".", 1)[1], s) if n.startswith("l") and repeat_layers else None
+            data = kept.get(key) if key else None
+            if data is None:
+                data = draw(n, s).tobytes()
+                if key:
+                    kept[key] = data
+            f.write(data)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
