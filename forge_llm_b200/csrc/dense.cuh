@@ -16,10 +16,10 @@ constexpr int kSegAlign = 32;    // output segments start at multiples of a warp
 inline int pad_to(int x, int a) { return (x + a - 1) / a * a; }
 
 struct DenseWeight {
-    void* w = nullptr;           // [N][K] of the model's type, padding columns and rows are zero
+    void* w = nullptr;           // [N][K] of the model's type, padding columns and rows are zero (f32 products, and where a kernel reads rows)
+    void* tiles = nullptr;       // bf16: the same matrix as dense_tile_image
     int N = 0, K = 0;            // K: padded
     int dtype = FORGE_BF16;
-    alignas(64) unsigned char map[128];   // CUtensorMap of w (bf16), box {64, 128}
 };
 
 // What becomes of the rows [row0, row0 + rows) of a product.  T: the model's activation type.
@@ -47,7 +47,8 @@ struct DenseOut { int nseg = 0; OutSeg seg[kMaxSegs]; };
 struct DenseScratch { float* part = nullptr; int* tickets = nullptr; size_t tickets_cap = 0; };
 constexpr size_t kDensePartFloats = size_t(148) * 2 * 256 * 128;
 
-int32_t dense_make_map(DenseWeight& w);
+inline size_t dense_tile_bytes(int N, int K) { return size_t((N + 127) / 128) * 128 * K * 2; }
+void dense_tile_image(void* dst, const void* rows, int N, int K);
 // act: [m][w.K] of the model's type (rows w.K apart unless act_ld says otherwise).  max_rows: rows the buffer holds.
 int32_t dense_gemm(const DenseWeight& w, const void* act, int act_ld, int m, const DenseOut& out, const DenseScratch& sc, int* err, cudaStream_t st);
 

@@ -171,9 +171,9 @@ template <typename T>
 __global__ void embed_dyt_kernel(float* __restrict__ x, T* __restrict__ h, int h_ld, const T* __restrict__ table, const uint32_t* __restrict__ tokens, int width, float alpha,
                                  const float* __restrict__ w, const float* __restrict__ b, uint32_t* hist, const int32_t* step) {
     const int r = blockIdx.x;
-    if (hist && threadIdx.x == 0) hist[size_t(*step) * gridDim.x + r] = tokens[r];
+    if (hist && blockIdx.y == 0 && threadIdx.x == 0) hist[size_t(*step) * gridDim.x + r] = tokens[r];
     const T* src = table + size_t(tokens[r]) * width;
-    for (int i = threadIdx.x; i < h_ld; i += blockDim.x) {
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < h_ld; i += gridDim.y * blockDim.x) {
         float n = 0.f;
         if (i < width) {
             const float v = float(src[i]);
@@ -565,9 +565,9 @@ int32_t embed_dyt(float* x, void* h, int h_ld, const void* table, int dtype, con
                   const float* w, const float* b, uint32_t* hist, const int32_t* step, cudaStream_t st) {
     if (rows <= 0) return FORGE_OK;
     if (dtype == FORGE_F32)
-        embed_dyt_kernel<float><<<rows, 256, 0, st>>>(x, static_cast<float*>(h), h_ld, static_cast<const float*>(table), tokens, width, alpha, w, b, hist, step);
+        embed_dyt_kernel<float><<<dim3(rows, rows < 64 ? (h_ld + 255) / 256 : 1), 256, 0, st>>>(x, static_cast<float*>(h), h_ld, static_cast<const float*>(table), tokens, width, alpha, w, b, hist, step);
     else
-        embed_dyt_kernel<__nv_bfloat16><<<rows, 256, 0, st>>>(x, static_cast<__nv_bfloat16*>(h), h_ld, static_cast<const __nv_bfloat16*>(table), tokens, width, alpha, w, b, hist, step);
+        embed_dyt_kernel<__nv_bfloat16><<<dim3(rows, rows < 64 ? (h_ld + 255) / 256 : 1), 256, 0, st>>>(x, static_cast<__nv_bfloat16*>(h), h_ld, static_cast<const __nv_bfloat16*>(table), tokens, width, alpha, w, b, hist, step);
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }

@@ -8,6 +8,7 @@
 // share is left in scratch memory and added in K order, so the result does not depend on the order of arrival.  Nobody
 // waits for another CTA.
 // Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = epilogue (TMEM lane = weight row).
+// The weights lie in memory as the very images the ring holds (dense_tile_image), so a stage is one contiguous 16 KB bulk copy.
 // Accumulators are double buffered in tensor memory: the epilogue of one tile runs under the products of the next.
 // The weight stages of the ring are requested before the dependency wait of a programmatic launch, the activations after.
 //
@@ -36,32 +37,45 @@ __device__ __forceinline__ float clamped_glu(float gate, float up, float limit) 
     return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
 }
 
-__device__ __forceinline__ int find_seg(const DenseOut& o, int row) {
+
+// The fields of a segment this thread's row needs, in registers: a store through a pointer may not make the compiler fetch them
+// again for every value.
+template <typename T>
+struct RowOut {
+    int kind;
+    bool ok;                 // the row belongs to a segment
+    size_t ld;
+    float* f32; T* t;        // the row's place of token 0
+    T* next; size_t next_ld;
+    float limit, alpha, nw, nb;
+};
+template <typename T>
+__device__ __forceinline__ RowOut<T> row_out(const DenseOut& o, int row, int first_row) {
+    RowOut<T> q{};
     int s = -1;
     for (int i = 0; i < o.nseg; ++i)
-        if (row >= o.seg[i].row0 && row < o.seg[i].row0 + o.seg[i].rows) s = i;
-    return s;
-}
-
-// one finished value of a segment that is not SEG_CLAMPED_GLU; r = row in the segment
-template <typename T>
-__device__ __forceinline__ void seg_store(const OutSeg& g, int r, size_t token, float v, float resid, float nw, float nb) {
-    if (g.kind == SEG_F32) {
-        static_cast<float*>(g.dst)[token * g.ld + r] = v;
-    } else if (g.kind == SEG_CAST) {
-        const int c = g.group ? (r / g.group) * g.group_ld + r % g.group : r;
-        static_cast<T*>(g.dst)[token * g.ld + c] = to_t<T>(v);
-    } else if (g.kind == SEG_SIGMOID) {
-        static_cast<T*>(g.dst)[token * g.ld + r] = to_t<T>(1.0f / (1.0f + expf(-v)));
-    } else {
-        const float x = resid + v;
-        static_cast<float*>(g.dst)[token * g.ld + r] = x;
-        if (g.next) static_cast<T*>(g.next)[token * g.next_ld + r] = to_t<T>(tanhf(g.alpha * x) * nw + nb);
+        if (first_row >= o.seg[i].row0 && first_row < o.seg[i].row0 + o.seg[i].rows) s = i;
+    q.kind = -1;
+    if (s < 0) return q;
+    const int r = row - o.seg[s].row0, group = o.seg[s].group;
+    q.kind = o.seg[s].kind;
+    q.ok = r < o.seg[s].rows;
+    q.ld = size_t(o.seg[s].ld);
+    const int col = q.kind == SEG_CLAMPED_GLU ? r >> 1 : (q.kind == SEG_CAST && group) ? (r / group) * o.seg[s].group_ld + r % group : r;
+    q.f32 = static_cast<float*>(o.seg[s].dst) + col;
+    q.t = static_cast<T*>(o.seg[s].dst) + col;
+    q.limit = o.seg[s].limit;
+    if (q.kind == SEG_RESID && o.seg[s].next && q.ok) {
+        q.alpha = o.seg[s].alpha; q.nw = o.seg[s].norm_w[r]; q.nb = o.seg[s].norm_b[r];
+        q.next = static_cast<T*>(o.seg[s].next) + r; q.next_ld = size_t(o.seg[s].next_ld);
     }
+    return q;
 }
+__device__ __forceinline__ float sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
 
 struct GemmParams {
     DenseOut out;
+    const void* w;           // weight images
     int m, N, nk;            // tokens, rows, K steps per tile
     int tt_count;            // token tiles
     long long units;         // tiles * nk
@@ -79,8 +93,7 @@ template <int NT> struct Ring {
 };
 
 template <int NT>
-__global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
-                                                                 const __grid_constant__ GemmParams p) {
+__global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ GemmParams p) {
     constexpr int STAGE = Ring<NT>::STAGE, STAGES = Ring<NT>::STAGES;
     constexpr uint32_t kCols = Ring<NT>::COLS;
     extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -107,36 +120,35 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
     if (warp == 0) {
         if (lane == 0) {
             const int total = int(u1 - u0);
-            auto coords = [&](int i, int& kt, int& row0, int& tok0) {
-                const long long u = u0 + i;
-                const int tile = int(u / p.nk);
-                kt = int(u - (long long)tile * p.nk);
-                row0 = (tile / p.tt_count) * 128;
-                tok0 = (tile % p.tt_count) * NT;
+            // position of the next weight stage and of the next activation stage, advanced without divisions
+            const int tile0 = int(u0 / p.nk);
+            int kt_w = int(u0 - (long long)tile0 * p.nk), rt_w = tile0 / p.tt_count, tt_w = tile0 % p.tt_count;
+            int kt_x = kt_w, tt_x = tt_w;
+            const unsigned char* const weights = static_cast<const unsigned char*>(p.w);
+            auto weight_stage = [&](int s) {   // one contiguous image of 128 rows x 64 columns, already swizzled
+                mbar_expect_tx(&full[s], uint32_t(STAGE));
+                bulk_load(ring + size_t(s) * STAGE, weights + (size_t(rt_w) * p.nk + kt_w) * 16384, 16384, &full[s]);
+                if (++kt_w == p.nk) { kt_w = 0; if (++tt_w == p.tt_count) { tt_w = 0; ++rt_w; } }
             };
             const int ahead = min(total, STAGES);
-            int kt, row0, tok0;
-            for (int i = 0; i < ahead; ++i) {   // constant weights: may overlap the kernel in front
-                coords(i, kt, row0, tok0);
-                mbar_expect_tx(&full[i], uint32_t(STAGE));
-                tma_2d(ring + size_t(i) * STAGE, &map_w, kt * BK, row0, &full[i]);
-            }
+            for (int i = 0; i < ahead; ++i) weight_stage(i);   // constant: may overlap the kernel in front
             pdl_wait();
+            int s = 0;
+            uint32_t phase = 1;   // parity of the round in front of the current one
             for (int i = 0; i < total; ++i) {
-                const int s = i % STAGES, use = i / STAGES;
-                coords(i, kt, row0, tok0);
-                unsigned char* dst = ring + size_t(s) * STAGE;
-                if (use > 0) {
-                    if (!mbar_wait(&empty[s], (use - 1) & 1, &s_err)) { atomicExch(&s_err, 1); break; }
-                    mbar_expect_tx(&full[s], uint32_t(STAGE));
-                    tma_2d(dst, &map_w, kt * BK, row0, &full[s]);
+                if (i >= STAGES) {
+                    if (!mbar_wait(&empty[s], phase, &s_err)) { atomicExch(&s_err, 1); break; }
+                    weight_stage(s);
                 }
-                tma_2d(dst + 16384, &map_x, kt * BK, tok0, &full[s]);
+                tma_2d(ring + size_t(s) * STAGE + 16384, &map_x, kt_x * BK, tt_x * NT, &full[s]);
+                if (++kt_x == p.nk) { kt_x = 0; if (++tt_x == p.tt_count) tt_x = 0; }
+                if (++s == STAGES) { s = 0; phase ^= 1; }
             }
         }
     } else if (warp == 1) {
         if (lane == 0) {
-            int i = 0;
+            int s = 0;
+            uint32_t phase = 0;
             bool ok = true;
             int seg = 0;
             for (long long u = u0; u < u1 && ok; ++seg) {
@@ -144,9 +156,8 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
                 const int n = int(min(u1, tile_end) - u), buf = seg & 1;
                 if (seg >= 2 && !mbar_wait(&acc_empty[buf], ((seg >> 1) - 1) & 1, &s_err)) { ok = false; break; }
                 fence_after();
-                for (int k = 0; k < n; ++k, ++i) {
-                    const int s = i % STAGES;
-                    if (!mbar_wait(&full[s], (i / STAGES) & 1, &s_err)) { ok = false; break; }
+                for (int k = 0; k < n; ++k) {
+                    if (!mbar_wait(&full[s], phase, &s_err)) { ok = false; break; }
                     fence_after();
                     const uint32_t base = smem_u32(ring + size_t(s) * STAGE);
 #pragma unroll
@@ -154,6 +165,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
                         umma_ss(tmem + uint32_t(buf * NT), desc_kmajor(base + k16 * 32), desc_kmajor(base + 16384 + k16 * 32), idesc_bf16(NT),
                                 (k > 0 || k16 > 0) ? 1u : 0u);
                     umma_commit(&empty[s]);
+                    if (++s == STAGES) { s = 0; phase ^= 1; }
                 }
                 if (ok) umma_commit(&acc_full[buf]);
                 u += n;
@@ -177,33 +189,45 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
             if (!mbar_wait(&acc_full[buf], (seg_i >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
             fence_after();
             // every warp's rows lie in one segment (segments start at multiples of 32 rows)
-            const int si = find_seg(p.out, row0);
-            const OutSeg& g = p.out.seg[si < 0 ? 0 : si];
-            const int r = row - g.row0;
-            const bool row_ok = si >= 0 && r < g.rows;
-            float nw = 0.f, nb = 0.f;
-            if (row_ok && g.kind == SEG_RESID && g.next) { nw = g.norm_w[r]; nb = g.norm_b[r]; }
+            const RowOut<__nv_bfloat16> g = row_out<__nv_bfloat16>(p.out, row, row0);
             auto finish = [&](int c0, const float (&v)[CH]) {
+                const int n_c = cols - c0;
+                const size_t t0 = size_t(tok0 + c0);
                 if (g.kind == SEG_CLAMPED_GLU) {
                     // neighbouring lanes hold gate_j and up_j: the even lane takes the first half of the columns
                     const bool even = !(lane & 1);
-                    const int j = r >> 1;
+                    __nv_bfloat16* dst = g.t + (t0 + (even ? 0 : CH / 2)) * g.ld;
 #pragma unroll
                     for (int c = 0; c < CH / 2; ++c) {
                         const float got = __shfl_xor_sync(0xffffffffu, even ? v[CH / 2 + c] : v[c], 1);
                         const float ga = even ? v[c] : got, up = even ? got : v[CH / 2 + c];
-                        const int t = c0 + (even ? c : CH / 2 + c);
-                        if (row_ok && t < cols) static_cast<__nv_bfloat16*>(g.dst)[size_t(tok0 + t) * g.ld + j] = __float2bfloat16_rn(clamped_glu(ga, up, g.limit));
+                        if (g.ok && (even ? c : CH / 2 + c) < n_c) dst[c * g.ld] = __float2bfloat16_rn(clamped_glu(ga, up, g.limit));
                     }
-                } else if (row_ok) {
-                    float rv[CH];
-                    if (g.kind == SEG_RESID) {   // all loads before the first store
+                } else if (!g.ok) {
+                } else if (g.kind == SEG_F32) {
+                    float* dst = g.f32 + t0 * g.ld;
 #pragma unroll
-                        for (int c = 0; c < CH; ++c) rv[c] = c0 + c < cols ? static_cast<const float*>(g.dst)[size_t(tok0 + c0 + c) * g.ld + r] : 0.f;
+                    for (int c = 0; c < CH; ++c) if (c < n_c) dst[c * g.ld] = v[c];
+                } else if (g.kind == SEG_CAST) {
+                    __nv_bfloat16* dst = g.t + t0 * g.ld;
+#pragma unroll
+                    for (int c = 0; c < CH; ++c) if (c < n_c) dst[c * g.ld] = __float2bfloat16_rn(v[c]);
+                } else if (g.kind == SEG_SIGMOID) {
+                    __nv_bfloat16* dst = g.t + t0 * g.ld;
+#pragma unroll
+                    for (int c = 0; c < CH; ++c) if (c < n_c) dst[c * g.ld] = __float2bfloat16_rn(sigmoid(v[c]));
+                } else {
+                    float* dst = g.f32 + t0 * g.ld;
+                    float x[CH];
+#pragma unroll
+                    for (int c = 0; c < CH; ++c) x[c] = c < n_c ? dst[c * g.ld] : 0.f;   // all loads before the first store
+#pragma unroll
+                    for (int c = 0; c < CH; ++c) { x[c] += v[c]; if (c < n_c) dst[c * g.ld] = x[c]; }
+                    if (g.next) {
+                        __nv_bfloat16* nx = g.next + t0 * g.next_ld;
+#pragma unroll
+                        for (int c = 0; c < CH; ++c) if (c < n_c) nx[c * g.next_ld] = __float2bfloat16_rn(tanhf(g.alpha * x[c]) * g.nw + g.nb);
                     }
-#pragma unroll
-                    for (int c = 0; c < CH; ++c)
-                        if (c0 + c < cols) seg_store<__nv_bfloat16>(g, r, size_t(tok0 + c0 + c), v[c], g.kind == SEG_RESID ? rv[c] : 0.f, nw, nb);
                 }
             };
             auto load = [&](int c0, float (&v)[CH]) {
@@ -276,8 +300,6 @@ template <int NT>
 int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmParams& p, int sms, cudaStream_t st) {
     CUtensorMap mx;
     FORGE_TRY(make_map_2d(&mx, act, uint64_t(w.K), uint64_t(p.m), uint64_t(act_ld) * 2, NT));
-    CUtensorMap mw;
-    memcpy(&mw, w.map, sizeof(mw));
     p.tt_count = (p.m + NT - 1) / NT;
     const long long tiles = (long long)((w.N + 127) / 128) * p.tt_count;
     p.units = tiles * p.nk;
@@ -285,7 +307,7 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmPara
     const size_t smem = size_t(Ring<NT>::STAGES) * Ring<NT>::STAGE + 1024;
     auto kern = gemm_dense_kernel<NT>;
     FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
-    FORGE_CUDA(launch_pdl(kern, dim3(grid), dim3(kThreads), smem, st, mw, mx, p));
+    FORGE_CUDA(launch_pdl(kern, dim3(grid), dim3(kThreads), smem, st, mx, p));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
@@ -327,23 +349,28 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
         }
         __syncthreads();
     }
-    const int si = find_seg(out, row0 + rr);   // four consecutive rows lie in one segment or past its end
-    if (si < 0) return;
-    const OutSeg& g = out.seg[si];
+    RowOut<float> g[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) g[i] = row_out<float>(out, row0 + rr + i, row0 + rr);   // four consecutive rows lie in one segment or past its end
 #pragma unroll
     for (int j = 0; j < PT; ++j) {
-        const int t = tok0 + tt + j;
-        if (t >= m) continue;
+        const size_t t = size_t(tok0 + tt + j);
+        if (int(t) >= m) continue;
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-            const int r = row0 + rr + i - g.row0;
-            if (r >= g.rows) continue;
-            if (g.kind == SEG_CLAMPED_GLU) {
-                if (!(i & 1)) static_cast<float*>(g.dst)[size_t(t) * g.ld + (r >> 1)] = clamped_glu(acc[i][j], acc[i + 1][j], g.limit);
-            } else {
-                const bool rs = g.kind == SEG_RESID;
-                const float nw = rs && g.next ? g.norm_w[r] : 0.f, nb = rs && g.next ? g.norm_b[r] : 0.f;
-                seg_store<float>(g, r, size_t(t), acc[i][j], rs ? static_cast<const float*>(g.dst)[size_t(t) * g.ld + r] : 0.f, nw, nb);
+            if (!g[i].ok) continue;
+            float* dst = g[i].f32 + t * g[i].ld;
+            const float v = acc[i][j];
+            switch (g[i].kind) {
+                case SEG_CLAMPED_GLU: if (!(i & 1)) *dst = clamped_glu(v, acc[i | 1][j], g[i].limit); break;
+                case SEG_SIGMOID: *dst = sigmoid(v); break;
+                case SEG_RESID: {
+                    const float x = *dst + v;
+                    *dst = x;
+                    if (g[i].next) g[i].next[t * g[i].next_ld] = tanhf(g[i].alpha * x) * g[i].nw + g[i].nb;
+                    break;
+                }
+                default: *dst = v;
             }
         }
     }
@@ -351,13 +378,18 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 
 }  // namespace
 
-int32_t dense_make_map(DenseWeight& w) {
-    static_assert(sizeof(CUtensorMap) == sizeof(w.map), "CUtensorMap is 128 bytes");
-    if (w.dtype != FORGE_BF16) return FORGE_OK;
-    CUtensorMap m;
-    FORGE_TRY(make_map_2d(&m, w.w, uint64_t(w.K), uint64_t(w.N), uint64_t(w.K) * 2, 128));
-    memcpy(w.map, &m, sizeof(m));
-    return FORGE_OK;
+// Load-time image of a bf16 matrix [N][K]: per 128 rows and 64 columns the 16 KB a stage of the ring holds, 128-byte rows with
+// their 16-byte pieces at piece ^ (row & 7) (what a SWIZZLE_128B copy would write), K steps of a row tile one after another.
+void dense_tile_image(void* dst, const void* rows, int N, int K) {
+    const int nk = K / BK;
+    const uint8_t* src = static_cast<const uint8_t*>(rows);
+    uint8_t* out = static_cast<uint8_t*>(dst);
+    memset(out, 0, dense_tile_bytes(N, K));
+    for (int r = 0; r < N; ++r) {
+        uint8_t* tile = out + size_t(r / 128) * nk * 16384 + size_t(r % 128) * 128;
+        for (int kt = 0; kt < nk; ++kt)
+            for (int c = 0; c < 8; ++c) memcpy(tile + size_t(kt) * 16384 + ((c ^ (r & 7)) << 4), src + (size_t(r) * K + kt * BK) * 2 + c * 16, 16);
+    }
 }
 
 int32_t dense_gemm(const DenseWeight& w, const void* act, int act_ld, int m, const DenseOut& out, const DenseScratch& sc, int* err, cudaStream_t st) {
@@ -381,7 +413,7 @@ int32_t dense_gemm(const DenseWeight& w, const void* act, int act_ld, int m, con
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
     sms = std::min(sms, 148);
     GemmParams p{};
-    p.out = out; p.m = m; p.N = w.N; p.nk = w.K / BK; p.part = sc.part; p.tickets = sc.tickets; p.err = err;
+    p.out = out; p.w = w.tiles; p.m = m; p.N = w.N; p.nk = w.K / BK; p.part = sc.part; p.tickets = sc.tickets; p.err = err;
     const int nt = m <= 16 ? 16 : m <= 32 ? 32 : m <= 64 ? 64 : m <= 128 ? 128 : 256;
     if (size_t((w.N + 127) / 128) * ((m + nt - 1) / nt) > sc.tickets_cap) { set_error("dense product: too many tiles for the ticket array"); return FORGE_ERR_SHAPE; }
     switch (nt) {

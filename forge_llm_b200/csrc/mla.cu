@@ -16,6 +16,17 @@ template <> __device__ __forceinline__ __nv_bfloat16 to_t<__nv_bfloat16>(float v
 __device__ __forceinline__ float to_f(float v) { return v; }
 __device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+// eight consecutive values
+__device__ __forceinline__ void load8(float (&v)[8], const float* p) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void load8(float (&v)[8], const __nv_bfloat16* p) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h[i]); v[2 * i] = f.x; v[2 * i + 1] = f.y; }
+}
 __device__ __forceinline__ float2 load2(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
 
 constexpr int kThreads = 256;
@@ -63,7 +74,7 @@ template <typename T, int RB>
 __global__ void __launch_bounds__(kThreads) latent_post_kernel(const LatentDims d, const float* __restrict__ proj, int ldp, int dkv_col, const float* __restrict__ kv_norm,
                                                                const float2* __restrict__ rope, const T* __restrict__ uk, int uk_ld, T* __restrict__ qabs, T* __restrict__ cache,
                                                                const StepRows rows) {
-    extern __shared__ float sm[];   // queries [RB][dim], then partial sums [4][RB][128]
+    extern __shared__ float sm[];   // queries [RB][dim], then partial sums [8][RB][128]
     __shared__ float red[32];
     const int nrb = (d.rank_p + kAbsorbCols - 1) / kAbsorbCols;
     const int r0 = blockIdx.x * RB, nr = min(RB, rows.n - r0);
@@ -91,25 +102,41 @@ __global__ void __launch_bounds__(kThreads) latent_post_kernel(const LatentDims 
         sq[i] = j < nr ? proj[size_t(r0 + j) * ldp + h * qd + e] : 0.f;
     }
     __syncthreads();
-    const int col = (threadIdx.x & 63) * 2, part = threadIdx.x >> 6;
-    float a0[RB], a1[RB];
+    // sixteen threads cover the columns, sixteen groups of them share the dimensions
+    const int col = (threadIdx.x & 15) * 8, part = threadIdx.x >> 4;
+    float a[RB][8];
 #pragma unroll
-    for (int j = 0; j < RB; ++j) { a0[j] = 0.f; a1[j] = 0.f; }
+    for (int j = 0; j < RB; ++j)
+#pragma unroll
+        for (int c = 0; c < 8; ++c) a[j][c] = 0.f;
     if (c0 + col < d.rank_p) {
 #pragma unroll 8
-        for (int e = part; e < d.dim; e += 4) {
-            const float2 v = load2(w + size_t(e) * uk_ld + col);
+        for (int e = part; e < d.dim; e += 16) {
+            float v[8];
+            load8(v, w + size_t(e) * uk_ld + col);
 #pragma unroll
-            for (int j = 0; j < RB; ++j) { const float q = sq[j * d.dim + e]; a0[j] = fmaf(q, v.x, a0[j]); a1[j] = fmaf(q, v.y, a1[j]); }
+            for (int j = 0; j < RB; ++j) {
+                const float q = sq[j * d.dim + e];
+#pragma unroll
+                for (int c = 0; c < 8; ++c) a[j][c] = fmaf(q, v[c], a[j][c]);
+            }
         }
     }
 #pragma unroll
-    for (int j = 0; j < RB; ++j) { sp[(part * RB + j) * 128 + col] = a0[j]; sp[(part * RB + j) * 128 + col + 1] = a1[j]; }
+    for (int j = 0; j < RB; ++j) {   // lanes l and l + 16 hold the same columns
+#pragma unroll
+        for (int c = 0; c < 8; ++c) a[j][c] += __shfl_xor_sync(0xffffffffu, a[j][c], 16);
+        if (!(threadIdx.x & 16))
+#pragma unroll
+            for (int c = 0; c < 8; ++c) sp[((threadIdx.x >> 5) * RB + j) * 128 + col + c] = a[j][c];
+    }
     __syncthreads();
     for (int i = threadIdx.x; i < RB * 128; i += kThreads) {
         const int j = i >> 7, c = i & 127;
         if (j < nr && c0 + c < d.rank_p) {
-            const float s = (sp[j * 128 + c] + sp[(RB + j) * 128 + c]) + (sp[(2 * RB + j) * 128 + c] + sp[(3 * RB + j) * 128 + c]);
+            float s = 0.f;
+#pragma unroll
+            for (int q = 0; q < 8; ++q) s += sp[(q * RB + j) * 128 + c];
             qabs[(size_t(r0 + j) * d.heads + h) * d.row() + c0 + c] = to_t<T>(s);
         }
     }
@@ -215,8 +242,8 @@ constexpr int kValueRows = 32;   // rows of W_uv per CTA
 
 template <typename T, int RB>
 __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentDims d, const float* __restrict__ part, const float2* __restrict__ ml, int splits,
-                                                                const T* __restrict__ uv, int uv_ld, const T* __restrict__ gate, int gate_ld, T* __restrict__ out, int out_ld, int rows) {
-    extern __shared__ float sm[];   // merged latents [RB][rank_p], split factors [RB][splits]
+                                                                const T* __restrict__ uv, int uv_ld, const T* __restrict__ gate, int gate_ld, T* __restrict__ out, int out_ld, int rows, const int32_t* __restrict__ rows_pos) {
+    extern __shared__ __align__(16) float sm[];   // merged latents [RB][rank_p], split factors [RB][splits]
     const int h = blockIdx.y, v0 = blockIdx.z * kValueRows, r0 = blockIdx.x * RB, nr = min(RB, rows - r0);
     const int nv = min(kValueRows, d.vdim - v0);
     const T* w = uv + (size_t(h) * d.vdim + v0) * uv_ld;
@@ -248,39 +275,62 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentDims
         for (int s = lane; s < splits; s += 32) fac[warp * splits + s] *= inv;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < nr * d.rank_p; i += kThreads) {
-        const int j = i / d.rank_p, c = i % d.rank_p;
-        const float* p = part + (size_t(r0 + j) * d.heads + h) * splits * d.rank_p + c;
-        float v = 0.f;
-#pragma unroll 4
-        for (int s = 0; s < splits; ++s) {
-            const float f = fac[j * splits + s];
-            if (f != 0.f) v = fmaf(p[size_t(s) * d.rank_p], f, v);   // a split without keys left nothing to read
+    {
+        // four latents per thread; with room to spare two threads share a quad's splits (rank_p / 4 is a multiple of 16)
+        const int quads = d.rank_p / 4, halves = nr * quads * 2 <= kThreads ? 2 : 1;
+        for (int i = threadIdx.x; i < nr * quads * halves; i += kThreads) {
+            const int hf = halves == 2 ? (i >> 4) & 1 : 0, q = halves == 2 ? (i >> 5) * 16 + (i & 15) : i;
+            const int j = q / quads, c = (q % quads) * 4;
+            const int n = min(splits, rows_pos[r0 + j] / FORGE_KV_PAGE + 1);   // splits that own a page
+            const float* p = part + (size_t(r0 + j) * d.heads + h) * splits * d.rank_p + c;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+            for (int s = hf; s < n; s += halves) {
+                const float f = fac[j * splits + s];
+                const float4 x = *reinterpret_cast<const float4*>(p + size_t(s) * d.rank_p);
+                v.x = fmaf(x.x, f, v.x); v.y = fmaf(x.y, f, v.y); v.z = fmaf(x.z, f, v.z); v.w = fmaf(x.w, f, v.w);
+            }
+            if (halves == 2) {   // whole warps are in the loop (a multiple of 32 items)
+                v.x += __shfl_xor_sync(0xffffffffu, v.x, 16); v.y += __shfl_xor_sync(0xffffffffu, v.y, 16);
+                v.z += __shfl_xor_sync(0xffffffffu, v.z, 16); v.w += __shfl_xor_sync(0xffffffffu, v.w, 16);
+            }
+            if (!hf) *reinterpret_cast<float4*>(lat + j * d.rank_p + c) = v;
         }
-        lat[i] = v;
+        for (int i = nr * d.rank_p + threadIdx.x; i < RB * d.rank_p; i += kThreads) lat[i] = 0.f;
     }
     __syncthreads();
-    for (int v = warp; v < nv; v += kThreads / 32) {
-        float acc[RB];
+    // four rows of W_uv per warp: their loads are in flight together
+    constexpr int VR = kValueRows / (kThreads / 32);
+    float acc[VR][RB];
 #pragma unroll
-        for (int j = 0; j < RB; ++j) acc[j] = 0.f;
-        const T* wr = w + size_t(v) * uv_ld;
-#pragma unroll 4
-        for (int c = lane * 2; c < d.rank_p; c += 64) {
-            const float2 a = load2(wr + c);
+    for (int v = 0; v < VR; ++v)
 #pragma unroll
-            for (int j = 0; j < RB; ++j) { acc[j] = fmaf(a.x, lat[j * d.rank_p + c], acc[j]); acc[j] = fmaf(a.y, lat[j * d.rank_p + c + 1], acc[j]); }
+        for (int j = 0; j < RB; ++j) acc[v][j] = 0.f;
+    for (int c = lane * 8; c < d.rank_p; c += 256) {
+        float a[VR][8];
+#pragma unroll
+        for (int v = 0; v < VR; ++v) load8(a[v], w + size_t(min(warp * VR + v, nv - 1)) * uv_ld + c);
+#pragma unroll
+        for (int j = 0; j < RB; ++j) {
+            float x[8];
+            load8(x, lat + j * d.rank_p + c);
+#pragma unroll
+            for (int v = 0; v < VR; ++v)
+#pragma unroll
+                for (int e = 0; e < 8; ++e) acc[v][j] = fmaf(a[v][e], x[e], acc[v][j]);
         }
+    }
+#pragma unroll
+    for (int v = 0; v < VR; ++v)
 #pragma unroll
         for (int j = 0; j < RB; ++j) {
 #pragma unroll
-            for (int o = 16; o > 0; o >>= 1) acc[j] += __shfl_xor_sync(0xffffffffu, acc[j], o);
-            if (lane == 0 && j < nr) {
-                const int col = h * d.vdim + v0 + v;
-                out[size_t(r0 + j) * out_ld + col] = to_t<T>(acc[j] * to_f(gate[size_t(r0 + j) * gate_ld + col]));
+            for (int o = 16; o > 0; o >>= 1) acc[v][j] += __shfl_xor_sync(0xffffffffu, acc[v][j], o);
+            if (lane == 0 && j < nr && warp * VR + v < nv) {
+                const int col = h * d.vdim + v0 + warp * VR + v;
+                out[size_t(r0 + j) * out_ld + col] = to_t<T>(acc[v][j] * to_f(gate[size_t(r0 + j) * gate_ld + col]));
             }
         }
-    }
 }
 
 __global__ void __launch_bounds__(128) latent_gather_kernel(const LatentDims d, const uint4* __restrict__ cache, const int32_t* __restrict__ pages, uint4* __restrict__ c, uint4* __restrict__ krot) {
@@ -297,7 +347,7 @@ int32_t post_t(const LatentDims& d, const float* proj, int ldp, int dkv_col, con
                const StepRows& rows, cudaStream_t st) {
     const int nrb = (d.rank_p + kAbsorbCols - 1) / kAbsorbCols;
     auto go = [&](auto kern, int rb) -> int32_t {
-        const size_t smem = sizeof(float) * size_t(rb) * (d.dim + 4 * 128);
+        const size_t smem = sizeof(float) * size_t(rb) * (d.dim + 8 * 128);
         if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
         FORGE_CUDA(launch_pdl(kern, dim3((rows.n + rb - 1) / rb, d.heads * nrb + 1), dim3(kThreads), smem, st, d, proj, ldp, dkv_col, kv_norm, reinterpret_cast<const float2*>(rope),
                               static_cast<const T*>(uk), uk_ld, static_cast<T*>(qabs), static_cast<T*>(cache), rows));
@@ -309,12 +359,13 @@ int32_t post_t(const LatentDims& d, const float* proj, int ldp, int dkv_col, con
 }
 
 template <typename T>
-int32_t value_t(const LatentDims& d, const float* part, const float2* ml, int splits, const void* uv, int uv_ld, const void* gate, int gate_ld, void* out, int out_ld, int rows, cudaStream_t st) {
+int32_t value_t(const LatentDims& d, const float* part, const float2* ml, int splits, const void* uv, int uv_ld, const void* gate, int gate_ld, void* out, int out_ld, const StepRows& sr, cudaStream_t st) {
+    const int rows = sr.n;
     auto go = [&](auto kern, int rb) -> int32_t {
         const size_t smem = sizeof(float) * size_t(rb) * (d.rank_p + splits);
         if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
         FORGE_CUDA(launch_pdl(kern, dim3((rows + rb - 1) / rb, d.heads, (d.vdim + kValueRows - 1) / kValueRows), dim3(kThreads), smem, st, d, part, ml, splits,
-                              static_cast<const T*>(uv), uv_ld, static_cast<const T*>(gate), gate_ld, static_cast<T*>(out), out_ld, rows));
+                              static_cast<const T*>(uv), uv_ld, static_cast<const T*>(gate), gate_ld, static_cast<T*>(out), out_ld, rows, sr.pos));
         FORGE_LAUNCH_CHECK();
         return FORGE_OK;
     };
@@ -350,9 +401,9 @@ int32_t latent_attn_rows(const LatentDims& d, int dtype, const void* qabs, const
     if (rows.n <= 0) return FORGE_OK;
     return dtype == FORGE_F32 ? attn_t<float>(d, qabs, cache, rows, splits, part, ml, st) : attn_t<__nv_bfloat16>(d, qabs, cache, rows, splits, part, ml, st);
 }
-int32_t latent_value(const LatentDims& d, int dtype, const float* part, const float2* ml, int splits, const void* uv, int uv_ld, const void* gate, int gate_ld, void* out, int out_ld, int rows,
-                     cudaStream_t st) {
-    if (rows <= 0) return FORGE_OK;
+int32_t latent_value(const LatentDims& d, int dtype, const float* part, const float2* ml, int splits, const void* uv, int uv_ld, const void* gate, int gate_ld, void* out, int out_ld,
+                     const StepRows& rows, cudaStream_t st) {
+    if (rows.n <= 0) return FORGE_OK;
     return dtype == FORGE_F32 ? value_t<float>(d, part, ml, splits, uv, uv_ld, gate, gate_ld, out, out_ld, rows, st)
                               : value_t<__nv_bfloat16>(d, part, ml, splits, uv, uv_ld, gate, gate_ld, out, out_ld, rows, st);
 }

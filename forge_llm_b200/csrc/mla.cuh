@@ -40,7 +40,7 @@ int32_t latent_cache_map(void* map_out, const void* cache, const LatentDims& d, 
 int32_t latent_decode_tc(const LatentDims& d, const void* qabs, const void* map, const StepRows& rows, int splits, float* part, float2* ml, int* err, cudaStream_t st);
 // out[row][head * vdim + v] = gate * (W_uv (sum of the splits)) as T
 int32_t latent_value(const LatentDims& d, int dtype, const float* part, const float2* ml, int splits, const void* uv, int uv_ld, const void* gate, int gate_ld,
-                     void* out, int out_ld, int rows, cudaStream_t st);
+                     void* out, int out_ld, const StepRows& rows, cudaStream_t st);
 
 // ---- prompts (bfloat16): keys and values of the heads are formed once per prompt portion, then a tcgen05 flash attention
 // c[r] = latents of context row r, krot[r] = its rotated key part (rows gathered through page list `pages`)

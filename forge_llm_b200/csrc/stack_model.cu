@@ -255,10 +255,16 @@ int32_t load_dyt(ForgeModel* m, DytNorm* n, const TensorView& w, const TensorVie
     FORGE_TRY(upload_f32(m, &n->w, w));
     return upload_f32(m, &n->b, b);
 }
-int32_t load_dense(ForgeModel* m, DenseWeight* w, int N, int K, int dtype, const std::vector<uint8_t>& img) {
+// row_reads: some kernel reads rows of the matrix, so it is kept in rows as well
+int32_t load_dense(ForgeModel* m, DenseWeight* w, int N, int K, int dtype, const std::vector<uint8_t>& img, bool row_reads = false) {
     w->N = N; w->K = K; w->dtype = dtype;
-    FORGE_TRY(upload(m, &w->w, img));
-    return dense_make_map(*w);
+    if (dtype == FORGE_F32 || row_reads) FORGE_TRY(upload(m, &w->w, img));
+    if (dtype == FORGE_BF16) {
+        std::vector<uint8_t> tiles(dense_tile_bytes(N, K));
+        dense_tile_image(tiles.data(), img.data(), N, K);
+        FORGE_TRY(upload(m, &w->tiles, tiles));
+    }
+    return FORGE_OK;
 }
 
 int32_t load_layer(ForgeModel* m, const LayerSpec& L, const LayerTensors& t, LayerWeights* w) {
@@ -286,7 +292,7 @@ int32_t load_layer(ForgeModel* m, const LayerSpec& L, const LayerTensors& t, Lay
         std::vector<uint8_t> img(size_t(n) * d.rank_p * es, 0);
         put_rows(img, S.dtype, d.rank_p, *t.uk, 0);
         put_rows(img, S.dtype, d.rank_p, *t.uv, w->uv_row);
-        FORGE_TRY(load_dense(m, &w->kv, n, d.rank_p, S.dtype, img));
+        FORGE_TRY(load_dense(m, &w->kv, n, d.rank_p, S.dtype, img, true));
     }
     {
         w->heads_k = pad_to(d.heads * d.vdim, kDensePad);
@@ -338,11 +344,11 @@ int32_t grow(ForgeModel* m, StackModel::Buf& b, size_t bytes) {
 
 bool tensor_core_rows(const StackModel& S, const LatentDims& d) { return S.dtype == FORGE_BF16 && latent_decode_tc_supported(d); }
 
-// splits of the row attention: one CTA per SM over all rows and head groups, no more than there are pages
+// splits of the row attention: at most one CTA per SM over all rows and head groups, no more than there are pages
 int row_splits(const StackModel& S, int rows, int pages) {
     int groups = 1;
     for (const LayerSpec& L : S.spec.layers) groups = std::max(groups, tensor_core_rows(S, L.mix) ? (L.mix.heads + 15) / 16 : L.mix.heads);
-    return std::max(1, std::min(pages, (148 + rows * groups - 1) / std::max(1, rows * groups)));
+    return std::max(1, std::min(pages, 148 / std::max(1, rows * groups)));
 }
 
 int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt, int ctx_rows) {
@@ -435,7 +441,7 @@ int32_t run_layers(ForgeModel* m, ForgeKV* kv, const Step& s) {
             FORGE_TRY(latent_post(d, dt, proj, ldp, w.dkv_row, w.kv_norm, rope, w.kv.w, w.kv.K, S.q.p, run.pool, single, st));
             if (tensor_core_rows(S, d)) FORGE_TRY(latent_decode_tc(d, S.q.p, run.map, single, s.splits, part, ml, m->d_err, st));
             else FORGE_TRY(latent_attn_rows(d, dt, S.q.p, run.pool, single, s.splits, part, ml, st));
-            FORGE_TRY(latent_value(d, dt, part, ml, s.splits, at(w.kv.w, size_t(w.uv_row) * w.kv.K, dt), w.kv.K, S.gate.p, gate_ld, S.mid.p, mid_ld, s.single, st));
+            FORGE_TRY(latent_value(d, dt, part, ml, s.splits, at(w.kv.w, size_t(w.uv_row) * w.kv.K, dt), w.kv.K, S.gate.p, gate_ld, S.mid.p, mid_ld, single, st));
         }
         const int np = n - s.single;
         if (np > 0) {
