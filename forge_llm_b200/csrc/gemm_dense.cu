@@ -28,10 +28,6 @@ using namespace tc5;
 constexpr int BK = 64;
 constexpr int kThreads = 192;
 
-template <typename T> __device__ __forceinline__ T to_t(float v);
-template <> __device__ __forceinline__ float to_t<float>(float v) { return v; }
-template <> __device__ __forceinline__ __nv_bfloat16 to_t<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
-
 __device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
     return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
@@ -185,11 +181,11 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
             const int row0 = (tile / p.tt_count) * 128 + quad * 32, tok0 = (tile % p.tt_count) * NT;
             const int row = row0 + lane;
             const int cols = min(NT, p.m - tok0);
+            // every warp's rows lie in one segment (segments start at multiples of 32 rows)
+            const RowOut<__nv_bfloat16> g = row_out<__nv_bfloat16>(p.out, row, row0);
             // the four warps meet at the barriers of a shared tile: one whose wait gave up must not leave the loop alone
             if (!mbar_wait(&acc_full[buf], (seg_i >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
             fence_after();
-            // every warp's rows lie in one segment (segments start at multiples of 32 rows)
-            const RowOut<__nv_bfloat16> g = row_out<__nv_bfloat16>(p.out, row, row0);
             auto finish = [&](int c0, const float (&v)[CH]) {
                 const int n_c = cols - c0;
                 const size_t t0 = size_t(tok0 + c0);
@@ -253,7 +249,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
                     float v[CH];
                     load(c0, v);
 #pragma unroll
-                    for (int c = 0; c < CH; ++c) __stcg(mine + size_t(c0 + c) * 128 + quad * 32 + lane, v[c]);
+                    for (int c = 0; c < CH; ++c) if (c < cols - c0) __stcg(mine + size_t(c0 + c) * 128 + quad * 32 + lane, v[c]);
                 }
                 const int first = share_of(p.units, t_begin, gridDim.x), last = share_of(p.units, t_end - 1, gridDim.x);
                 __threadfence();
@@ -271,10 +267,22 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
                         float v[CH];
 #pragma unroll
                         for (int c = 0; c < CH; ++c) v[c] = 0.f;
-                        for (int q = first; q <= last; ++q) {
-                            const float* src = p.part + (size_t(q) * 2 + (share_begin(p.units, q, gridDim.x) >= t_begin ? 0 : 1)) * (NT * 128) + quad * 32 + lane;
+                        // only the first share of the tile may be the second part of its CTA; loads of QB shares in flight together
+                        constexpr int QB = CH == 16 ? 4 : 2;
+                        const int n_c = cols - c0;
+                        const int first_slot = share_begin(p.units, first, gridDim.x) >= t_begin ? 0 : 1;
+                        for (int q = first; q <= last; q += QB) {
+                            float t[QB][CH];
 #pragma unroll
-                            for (int c = 0; c < CH; ++c) v[c] += __ldcg(src + size_t(c0 + c) * 128);
+                            for (int b = 0; b < QB; ++b) {
+                                const float* src = p.part + (size_t(q + b) * 2 + (q + b == first ? first_slot : 0)) * (NT * 128) + quad * 32 + lane + size_t(c0) * 128;
+#pragma unroll
+                                for (int c = 0; c < CH; ++c) t[b][c] = q + b <= last && c < n_c ? __ldcg(src + size_t(c) * 128) : 0.f;
+                            }
+#pragma unroll
+                            for (int b = 0; b < QB; ++b)
+#pragma unroll
+                                for (int c = 0; c < CH; ++c) v[c] += t[b][c];
                         }
                         finish(c0, v);
                     }

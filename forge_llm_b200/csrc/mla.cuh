@@ -20,6 +20,7 @@ struct StepRows {
     int n = 0;
     const int32_t* pos = nullptr; const int32_t* seq = nullptr;   // device
     const int32_t* page_table = nullptr; int pages_per_seq = 0;
+    int fresh = 1;                 // most rows one sequence has in this step
 };
 
 // proj: f32 rows [q | ... | dkv | ...] of ldp floats; q at column 0, W_dkv h at column dkv_col.

@@ -63,7 +63,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
     }
     __syncthreads();
     pdl_trigger();
-    pdl_wait();
+    // positions and page tables are written in front of the step's first kernel, which is launched without overlap
     const int pos = rows.pos[r], seq = rows.seq ? rows.seq[r] : r;
     const int pages = pos / kPage + 1;
     const int n = pages > split ? (pages - split + splits - 1) / splits : 0;
@@ -71,15 +71,23 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
     if (warp == 8) {
         if (lane == 0) {
             const int32_t* pt = rows.page_table + size_t(seq) * rows.pages_per_seq;
-            for (int i = 0; i < n; ++i) {
-                const int s = i % kStages, use = i / kStages;
-                if (use > 0 && !mbar_wait(&empty[s], (use - 1) & 1, &s_err)) { atomicExch(&s_err, 1); break; }
+            auto request = [&](int i) {
+                const int s = i % kStages, y = pt[split + i * splits] * kPage;
                 mbar_expect_tx(&full[s], uint32_t(stage_bytes));
-                const int y = pt[split + i * splits] * kPage;
                 for (int c = 0; c < W / 64; ++c) tma_2d(ring + size_t(s) * stage_bytes + c * (kPage * 128), &map, c * 64, y, &full[s]);
+            };
+            // pages that hold no row of this step are complete already: the first ones are requested before the wait
+            const int complete = (pos - rows.fresh + 1) / kPage;   // (rounds towards zero: 0 if nothing is older than the step)
+            int i = 0;
+            for (; i < n && i < kStages && split + i * splits < complete; ++i) request(i);
+            pdl_wait();
+            for (; i < n; ++i) {
+                if (i >= kStages && !mbar_wait(&empty[i % kStages], (i / kStages - 1) & 1, &s_err)) { atomicExch(&s_err, 1); break; }
+                request(i);
             }
         }
     } else {
+        pdl_wait();
         // queries into shared memory (heads past the last are zero), then this warp's half of them into registers
         for (int i = tid; i < 16 * (W / 8); i += kConsumers) {
             const int hh = i / (W / 8), c = i % (W / 8);

@@ -622,6 +622,7 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
     Step s;
     s.tokens = reinterpret_cast<const uint32_t*>(dm);
     s.rows = StepRows{rows, dm + rows, dm + 2 * rows, kv->d_page_table, kv->pages_per_seq};
+    for (int i = 0; i < n_entries; ++i) if (!is_prompt(i)) s.rows.fresh = std::max(s.rows.fresh, int(entries[i].n_tokens));
     s.single = single; s.splits = splits;
     s.ctx_pages = dm + o_pages; s.ctx_rows = ctx_rows;
     s.tiles = reinterpret_cast<const PromptTile*>(dm + o_tiles); s.n_tiles = int(tiles.size());
