@@ -135,7 +135,7 @@ class LayerStack:
 def bf16_bits(x):
     """float32 -> bfloat16 bit patterns, round to nearest even."""
     u = np.ascontiguousarray(x, np.float32).view(np.uint32).astype(np.uint64)
-    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16).reshape(np.shape(x))
 
 
 def bf16_round(x):
