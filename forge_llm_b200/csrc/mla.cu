@@ -68,8 +68,8 @@ __device__ __forceinline__ size_t cache_row(const StepRows& rows, int r, int pos
 
 constexpr int kAbsorbCols = 128;   // latent columns per CTA
 
-// blockIdx.x: group of RB rows.  blockIdx.y < heads * col blocks: queries of one head into 128 latent columns; the last
-// blockIdx.y appends the rows to the cache.
+// blockIdx.x: group of RB rows.  blockIdx.y < heads * col blocks: queries of one head into 128 latent columns; the last RB
+// values of blockIdx.y append one row each to the cache.
 template <typename T, int RB>
 __global__ void __launch_bounds__(kThreads) latent_post_kernel(const LatentDims d, const float* __restrict__ proj, int ldp, int dkv_col, const float* __restrict__ kv_norm,
                                                                const float2* __restrict__ rope, const T* __restrict__ uk, int uk_ld, T* __restrict__ qabs, T* __restrict__ cache,
@@ -78,13 +78,13 @@ __global__ void __launch_bounds__(kThreads) latent_post_kernel(const LatentDims 
     __shared__ float red[32];
     const int nrb = (d.rank_p + kAbsorbCols - 1) / kAbsorbCols;
     const int r0 = blockIdx.x * RB, nr = min(RB, rows.n - r0);
-    if (int(blockIdx.y) == d.heads * nrb) {
+    if (int(blockIdx.y) >= d.heads * nrb) {
+        const int r = r0 + int(blockIdx.y) - d.heads * nrb;
         pdl_trigger();
         pdl_wait();
-        for (int j = 0; j < nr; ++j) {
-            const int pos = rows.pos[r0 + j];
-            append_row<T>(d, proj + size_t(r0 + j) * ldp + dkv_col, kv_norm, rope + size_t(pos) * (d.rot_dims / 2), cache + cache_row(rows, r0 + j, pos) * d.row(), red);
-            __syncthreads();
+        if (r < rows.n) {
+            const int pos = rows.pos[r];
+            append_row<T>(d, proj + size_t(r) * ldp + dkv_col, kv_norm, rope + size_t(pos) * (d.rot_dims / 2), cache + cache_row(rows, r, pos) * d.row(), red);
         }
         return;
     }
@@ -349,7 +349,7 @@ int32_t post_t(const LatentDims& d, const float* proj, int ldp, int dkv_col, con
     auto go = [&](auto kern, int rb) -> int32_t {
         const size_t smem = sizeof(float) * size_t(rb) * (d.dim + 8 * 128);
         if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
-        FORGE_CUDA(launch_pdl(kern, dim3((rows.n + rb - 1) / rb, d.heads * nrb + 1), dim3(kThreads), smem, st, d, proj, ldp, dkv_col, kv_norm, reinterpret_cast<const float2*>(rope),
+        FORGE_CUDA(launch_pdl(kern, dim3((rows.n + rb - 1) / rb, d.heads * nrb + rb), dim3(kThreads), smem, st, d, proj, ldp, dkv_col, kv_norm, reinterpret_cast<const float2*>(rope),
                               static_cast<const T*>(uk), uk_ld, static_cast<T*>(qabs), static_cast<T*>(cache), rows));
         FORGE_LAUNCH_CHECK();
         return FORGE_OK;
