@@ -37,6 +37,7 @@ int32_t latent_post_prompt(const LatentDims& d, const float* proj, int ldp, int 
 int32_t latent_attn_rows(const LatentDims& d, int dtype, const void* qabs, const void* cache, const StepRows& rows, int splits, float* part, float2* ml, cudaStream_t st);
 // the same on the tensor cores (bfloat16); map: tensor map of the layer's cache rows, see latent_cache_map
 bool latent_decode_tc_supported(const LatentDims& d);
+int latent_decode_head_groups(const LatentDims& d);   // CTAs per row and split
 int32_t latent_cache_map(void* map_out, const void* cache, const LatentDims& d, size_t rows);
 int32_t latent_decode_tc(const LatentDims& d, const void* qabs, const void* map, const StepRows& rows, int splits, float* part, float2* ml, int* err, cudaStream_t st);
 // out[row][head * vdim + v] = gate * (W_uv (sum of the splits)) as T

@@ -347,7 +347,7 @@ bool tensor_core_rows(const StackModel& S, const LatentDims& d) { return S.dtype
 // splits of the row attention: at most one CTA per SM over all rows and head groups, no more than there are pages
 int row_splits(const StackModel& S, int rows, int pages) {
     int groups = 1;
-    for (const LayerSpec& L : S.spec.layers) groups = std::max(groups, tensor_core_rows(S, L.mix) ? (L.mix.heads + 15) / 16 : L.mix.heads);
+    for (const LayerSpec& L : S.spec.layers) groups = std::max(groups, tensor_core_rows(S, L.mix) ? latent_decode_head_groups(L.mix) : L.mix.heads);
     return std::max(1, std::min(pages, 148 / std::max(1, rows * groups)));
 }
 
