@@ -159,16 +159,14 @@ __global__ void __launch_bounds__(kThreads) latent_prompt_kernel(const LatentDim
     append_row<__nv_bfloat16>(d, src + dkv_col, kv_norm, cs, cache + cache_row(rows, r, pos) * d.row(), red);
     const int qd = d.dim + d.rot, qp = d.dim_p + d.rot_p;
     __nv_bfloat16* dst = q + size_t(r) * d.heads * qp;
-    for (int i = threadIdx.x; i < d.heads * qp / 2; i += kThreads) {
-        const int h = (2 * i) / qp, e0 = (2 * i) % qp;
+    const int lane = threadIdx.x & 31;
+    for (int h = threadIdx.x >> 5; h < d.heads; h += kThreads / 32) {   // a warp per head
         const float* x = src + h * qd;
-        float v[2];
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-            const int e = e0 + j, t = e - d.dim_p;
-            v[j] = t < 0 ? (e < d.dim ? x[e] : 0.f) : (t < d.rot ? rotated(x + d.dim, t, d.rot_dims, cs) : 0.f);
-        }
-        reinterpret_cast<__nv_bfloat162*>(dst)[i] = __floats2bfloat162_rn(v[0], v[1]);
+        __nv_bfloat162* out = reinterpret_cast<__nv_bfloat162*>(dst + h * qp);
+#pragma unroll 4
+        for (int e = 2 * lane; e < d.dim_p; e += 64) out[e >> 1] = __floats2bfloat162_rn(e < d.dim ? x[e] : 0.f, e + 1 < d.dim ? x[e + 1] : 0.f);
+        for (int t = 2 * lane; t < d.rot_p; t += 64)
+            out[(d.dim_p + t) >> 1] = __floats2bfloat162_rn(t < d.rot ? rotated(x + d.dim, t, d.rot_dims, cs) : 0.f, t + 1 < d.rot ? rotated(x + d.dim, t + 1, d.rot_dims, cs) : 0.f);
     }
 }
 

@@ -6,8 +6,8 @@
 // this kernel was bound by the tensor pipe at 16 heads).  A page has 64 rows, the MMA 128: the upper half of S is formed
 // from whatever follows in shared memory (always inside the CTA's allocation) and never read.
 //
-// One CTA = N heads of one row and one split of its pages.  Warp roles (224 threads): 0 = TMA producer (64-column boxes,
-// SWIZZLE_128B, a two-stage ring; pages of earlier steps are requested before the dependency wait), 1 = TMEM allocation and
+// One CTA = N heads of one row and one split of its pages.  Warp roles (224 threads): 0 = TMA producer (a page is one box of
+// 64-column chunks, SWIZZLE_128B, a two-stage ring; pages of earlier steps are requested before the dependency wait), 1 = TMEM allocation and
 // the products of S, 2..5 = softmax, 6 = the products of O (two issuing threads: with one, a page's O would wait for the
 // arrival of the next page).  S is turned in shared memory so that 128 / N lanes share a head's 64 scores; the
 // probabilities go to shared memory as the next B operand.  The running maximum is lazy (as in attn_prefill_tc5.cu): O is
@@ -54,21 +54,22 @@ template <int N> __device__ __forceinline__ void tmem_st(uint32_t addr, const ui
 }
 
 template <int N, uint32_t COLS>
-__global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap map, const LatentDims d, const __nv_bfloat16* __restrict__ qabs,
-                                                                    const StepRows rows, float scale2, float* __restrict__ part, float2* __restrict__ ml, int* err) {
+__global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_constant__ CUtensorMap map_q, const LatentDims d, const StepRows rows,
+                                                                    float scale2, float* __restrict__ part, float2* __restrict__ ml, int* err) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     const int W = d.row(), nch = W / 64, stage_bytes = nch * kChunk, tiles = (d.rank_p + 127) / 128;
     unsigned char* ring = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     unsigned char* sQ = ring + kStages * stage_bytes;          // [chunk][head][64 columns], swizzled
     unsigned char* sP = sQ + nch * N * 128;                    // [2][head][64 keys], swizzled
     float* sS = reinterpret_cast<float*>(sP + 2 * N * 128);    // [head][key]
-    __shared__ uint64_t full[kStages], empty[kStages], s_full[2], s_free[2], p_full[2], pv_done[2];
+    __shared__ uint64_t full[kStages], empty[kStages], q_full, s_full[2], s_free[2], p_full[2], pv_done[2];
     __shared__ float s_alpha[N];
     __shared__ uint32_t s_tmem;
     __shared__ int s_err;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int split = blockIdx.x, splits = gridDim.x, h0 = blockIdx.y * N, r = blockIdx.z;
     if (tid == 0) {
+        mbar_init(&q_full, 1);
         for (int s = 0; s < kStages; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
         for (int s = 0; s < 2; ++s) { mbar_init(&s_full[s], 1); mbar_init(&s_free[s], 2); mbar_init(&p_full[s], 4); mbar_init(&pv_done[s], 1); }
         s_err = 0;
@@ -86,40 +87,38 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
     const int n = pages > split ? (pages - split + splits - 1) / splits : 0;
 
     if (warp == 0) {
-        if (lane == 0) {
-            const int32_t* pt = rows.page_table + size_t(seq) * rows.pages_per_seq;
-            auto request = [&](int i) {
-                const int s = i % kStages, y = pt[split + i * splits] * kPage;
+        // the warp reads 32 entries of the page table at a time; lane 0 requests the pages
+        const int32_t* pt = rows.page_table + size_t(seq) * rows.pages_per_seq;
+        int entry = lane < n ? pt[split + lane * splits] : 0;
+        auto request = [&](int i) {
+            const int s = i % kStages, y = __shfl_sync(0xffffffffu, entry, i & 31) * kPage;
+            if (lane == 0) {
                 mbar_expect_tx(&full[s], uint32_t(stage_bytes));
-                for (int c = 0; c < nch; ++c) tma_2d(ring + size_t(s) * stage_bytes + c * kChunk, &map, c * 64, y, &full[s]);
-            };
-            // pages that hold no row of this step are complete already: the first ones are requested before the wait
-            const int complete = (pos - rows.fresh + 1) / kPage;   // (rounds towards zero: 0 if nothing is older than the step)
-            int i = 0;
-            for (; i < n && i < kStages && split + i * splits < complete; ++i) request(i);
-            pdl_wait();
-            for (; i < n; ++i) {
-                if (i >= kStages && !mbar_wait(&empty[i % kStages], (i / kStages - 1) & 1, &s_err)) { atomicExch(&s_err, 1); break; }
-                request(i);
+                tma_3d(ring + size_t(s) * stage_bytes, &map, 0, y, 0, &full[s]);
             }
+            __syncwarp();
+        };
+        // pages that hold no row of this step are complete already: the first ones are requested before the wait
+        const int complete = (pos - rows.fresh + 1) / kPage;   // (rounds towards zero: 0 if nothing is older than the step)
+        int i = 0;
+        for (; i < n && i < kStages && split + i * splits < complete; ++i) request(i);
+        pdl_wait();
+            // the row's queries (heads past the last read the next row's, or zero past the end: their columns are not used)
+        if (n > 0 && lane == 0) {
+            mbar_expect_tx(&q_full, uint32_t(nch * N * 128));
+            tma_3d(sQ, &map_q, 0, r * d.heads + h0, 0, &q_full);
+        }
+        for (; i < n; ++i) {
+            if ((i & 31) == 0 && i > 0) entry = i + lane < n ? pt[split + (i + lane) * splits] : 0;
+            const bool ok = i < kStages || mbar_wait(&empty[i % kStages], (i / kStages - 1) & 1, &s_err);
+            if (!__all_sync(0xffffffffu, ok)) { atomicExch(&s_err, 1); break; }
+            request(i);
         }
     }
-    if (warp != 0) pdl_wait();
-    if (warp >= 2 && warp < 6) {
-        // queries as the B operand; heads past the last are zero
-#pragma unroll 5
-        for (int i = tid - 64; i < N * (W / 8); i += 128) {
-            const int hh = i / (W / 8), c = i % (W / 8);
-            const uint4 v = h0 + hh < d.heads ? reinterpret_cast<const uint4*>(qabs + (size_t(r) * d.heads + h0 + hh) * W)[c] : make_uint4(0, 0, 0, 0);
-            *reinterpret_cast<uint4*>(sQ + (c >> 3) * (N * 128) + hh * 128 + (((c & 7) ^ (hh & 7)) << 4)) = v;
-        }
-        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-    }
-    if (warp != 0 && warp != 6) asm volatile("bar.sync 2, 160;" ::: "memory");
-
     if (warp == 1) {
         if (lane == 0 && n > 0) {
             const uint64_t q_desc = desc_kmajor(smem_u32(sQ));
+            if (!mbar_wait(&q_full, 0, &s_err)) atomicExch(&s_err, 1);
             for (int j = 0; j < n; ++j) {
                 if (!mbar_wait(&full[j % kStages], (j / kStages) & 1, &s_err) || (j >= 2 && !mbar_wait(&s_free[j & 1], ((j >> 1) - 1) & 1, &s_err))) { atomicExch(&s_err, 1); break; }
                 fence_after();
@@ -147,6 +146,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
             }
         }
     } else if (warp >= 2) {
+        pdl_wait();   // the results overwrite what an earlier layer's merge reads
         const int quad = warp & 3, tt = tid - 64;
         const uint32_t lane_addr = uint32_t(quad * 32) << 16;
         constexpr int HL = 128 / N, KL = kPage / HL;   // lanes of one head, keys per lane
@@ -228,10 +228,12 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
                 tmem_ld<N>(t_o + lane_addr + uint32_t(t * N), o);
                 wait_ld();
                 const int col = t * 128 + quad * 32 + lane;
-                if (col < d.rank_p)
+                float* dst = part + ((size_t(r) * d.heads + h0) * splits + split) * d.rank_p + col;
+                const size_t step = size_t(splits) * d.rank_p;
+                const int nh = col < d.rank_p ? min(N, d.heads - h0) : 0;
 #pragma unroll
-                    for (int h = 0; h < N; ++h)
-                        if (h0 + h < d.heads) part[((size_t(r) * d.heads + h0 + h) * splits + split) * d.rank_p + col] = __uint_as_float(o[h]);
+                for (int h = 0; h < N; ++h, dst += step)
+                    if (h < nh) *dst = __uint_as_float(o[h]);
             }
             fence_before();
         }
@@ -251,14 +253,23 @@ size_t decode_smem(const LatentDims& d, int n) {
     return size_t(kStages) * d.row() * 128 + std::max<size_t>(extra, kChunk) + 1024;   // at least a chunk behind the ring: see the header
 }
 
+// {64 columns, rows, chunks}: one box brings `box_rows` whole rows as chunks of swizzled 128-byte rows
+int32_t chunked_map(CUtensorMap* m, const void* base, const LatentDims& d, uint64_t rows, uint32_t box_rows) {
+    const uint32_t nch = uint32_t(d.row() / 64);
+    const uint64_t dims[3] = {64, rows, nch}, strides[2] = {uint64_t(d.row()) * 2, 128};
+    const uint32_t box[3] = {64, box_rows, nch};
+    return make_map(m, base, 3, dims, strides, box);
+}
+
 template <int N, uint32_t COLS>
 int32_t launch(const LatentDims& d, const void* qabs, const void* map, const StepRows& rows, int splits, float* part, float2* ml, int* err, cudaStream_t st) {
-    CUtensorMap m;
+    CUtensorMap m, mq;
     memcpy(&m, map, sizeof(m));
+    FORGE_TRY(chunked_map(&mq, qabs, d, uint64_t(rows.n) * d.heads, N));
     auto kern = latent_decode_kernel<N, COLS>;
     const size_t smem = decode_smem(d, N);
     FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
-    FORGE_CUDA(launch_pdl(kern, dim3(splits, (d.heads + N - 1) / N, rows.n), dim3(kThreads), smem, st, m, d, static_cast<const __nv_bfloat16*>(qabs), rows,
+    FORGE_CUDA(launch_pdl(kern, dim3(splits, (d.heads + N - 1) / N, rows.n), dim3(kThreads), smem, st, m, mq, d, rows,
                           d.scale * 1.4426950408889634f, part, ml, err));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
@@ -271,7 +282,7 @@ int latent_decode_head_groups(const LatentDims& d) { return (d.heads + head_tile
 
 int32_t latent_cache_map(void* map_out, const void* cache, const LatentDims& d, size_t rows) {
     CUtensorMap m;
-    FORGE_TRY(make_map_2d(&m, cache, uint64_t(d.row()), uint64_t(rows), uint64_t(d.row()) * 2, kPage));
+    FORGE_TRY(chunked_map(&m, cache, d, rows, kPage));
     memcpy(map_out, &m, sizeof(m));
     return FORGE_OK;
 }
