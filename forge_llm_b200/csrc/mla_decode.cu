@@ -1,18 +1,12 @@
-// Latent attention of single rows (decode, short portions) on the tensor cores (tcgen05 + TMEM), bfloat16.  All heads of a row
-// share the cached latents, and a page is the operand of both products, read once:
-//   S[key][head]    = C Q_abs^T   the page as the K-major A operand (M = keys), the queries of N = 16 or 32 heads as B;
-//   O[latent][head] += C^T P      the same page as the MN-major A operand (M = 128 latent columns), the probabilities as B.
-// The few heads are the N side of the products, so a decode step does not pay for a 128-row query tile (an mma.sync form of
-// this kernel was bound by the tensor pipe at 16 heads).  A page has 64 rows, the MMA 128: the upper half of S is formed
-// from whatever follows in shared memory (always inside the CTA's allocation) and never read.
+// Latent attention of single rows (decode, short portions) on the tensor cores, bfloat16.  All heads of a row share the
+// cached latents, so sixteen heads form one MMA tile: S[head][key] = Q_abs C^T over the whole cache row (latent and rotated
+// part), O[head][latent] += P C with the SAME page as the value operand - a page is read once for both.
 //
-// One CTA = N heads of one row and one split of its pages.  Warp roles (224 threads): 0 = TMA producer (a page is one box of
-// 64-column chunks, SWIZZLE_128B, a two-stage ring; pages of earlier steps are requested before the dependency wait), 1 = TMEM allocation and
-// the products of S, 2..5 = softmax, 6 = the products of O (two issuing threads: with one, a page's O would wait for the
-// arrival of the next page).  S is turned in shared memory so that 128 / N lanes share a head's 64 scores; the
-// probabilities go to shared memory as the next B operand.  The running maximum is lazy (as in attn_prefill_tc5.cu): O is
-// rescaled in tensor memory only when a maximum has grown by more than 2^8.  The partial results of the splits are merged by
-// the value projection's kernel.
+// One CTA = sixteen heads of one row and one split of its pages.  A producer warp requests a page (one box of 64-column chunks,
+// SWIZZLE_128B) per stage of a two-stage ring; eight consumer warps form the scores (four groups of sixteen keys x two halves
+// of the columns, the query fragments stay in registers), the running softmax (two heads per warp) and the sums (sixteen
+// latent columns at a time per warp).  mma.sync m16n8k16: sixteen heads are an eighth of a tcgen05 tile, and the kernel is
+// bound by the cache stream.  The partial results are merged by the value projection's kernel.
 #include <algorithm>
 #include <cstring>
 
@@ -25,68 +19,56 @@ namespace {
 
 using namespace tc5;
 
-constexpr int kThreads = 224, kStages = 2, kPage = FORGE_KV_PAGE;
-constexpr int kChunk = kPage * 128;      // bytes of one 64-column chunk of a page
-constexpr int kSLd = 68;
-constexpr float kLazy = 8.f;
+constexpr int kConsumers = 256, kThreads = kConsumers + 32;
+constexpr int kStages = 2;
+constexpr int kPage = FORGE_KV_PAGE;
+constexpr int kSLd = 68, kPLd = 72;
 
-// A MN-major (bit 15), B K-major
-__device__ __forceinline__ constexpr uint32_t idesc_a_mn(int n) { return idesc_bf16(n) | (1u << 15); }
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void consumer_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
-__device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
-__device__ __forceinline__ bool softmax_sync_or(bool v) {
-    uint32_t r;
-    asm volatile("{\n.reg .pred p, q;\nsetp.ne.u32 p, %1, 0;\nbar.red.or.pred q, 1, 128, p;\nselp.u32 %0, 1, 0, q;\n}" : "=r"(r) : "r"(uint32_t(v)) : "memory");
-    return r != 0;
-}
-template <int N> __device__ __forceinline__ void tmem_ld(uint32_t addr, uint32_t (&v)[N]) {
-    if constexpr (N == 16) tmem_ld16(addr, v);
-    else tmem_ld32(addr, v);
-}
-__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&v)[16]) {
-    asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
-                 ::"r"(taddr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]),
-                   "r"(v[9]), "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15]) : "memory");
-}
-template <int N> __device__ __forceinline__ void tmem_st(uint32_t addr, const uint32_t (&v)[N]) {
-    if constexpr (N == 16) tmem_st16(addr, v);
-    else tmem_st32(addr, v);
+// byte offset of (key, col) in a page stage: 64-column chunks of 64 swizzled 128-byte rows
+__device__ __forceinline__ uint32_t page_off(int key, int col) {
+    return uint32_t((col >> 6) * (kPage * 128) + key * 128 + ((((col & 63) >> 3) ^ (key & 7)) << 4));
 }
 
-template <int N, uint32_t COLS>
-__global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_constant__ CUtensorMap map_q, const LatentDims d, const StepRows rows,
-                                                                    float scale2, float* __restrict__ part, float2* __restrict__ ml, int* err) {
+// NCH: most 64-column chunks of a cache row
+template <int NCH>
+__global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid_constant__ CUtensorMap map, const LatentDims d, const __nv_bfloat16* __restrict__ qabs,
+                                                                    const StepRows rows, float scale2, float* __restrict__ part, float2* __restrict__ ml, int* err) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
-    const int W = d.row(), nch = W / 64, stage_bytes = nch * kChunk, tiles = (d.rank_p + 127) / 128;
+    const int W = d.row(), stage_bytes = W * kPage * 2, ldq = W + 8;
     unsigned char* ring = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-    unsigned char* sQ = ring + kStages * stage_bytes;          // [chunk][head][64 columns], swizzled
-    unsigned char* sP = sQ + nch * N * 128;                    // [2][head][64 keys], swizzled
-    float* sS = reinterpret_cast<float*>(sP + 2 * N * 128);    // [head][key]
-    __shared__ uint64_t full[kStages], empty[kStages], q_full, s_full[2], s_free[2], p_full[2], pv_done[2];
-    __shared__ float s_alpha[N];
-    __shared__ uint32_t s_tmem;
+    __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(ring + kStages * stage_bytes);
+    float* sS = reinterpret_cast<float*>(sQ + 16 * ldq);
+    __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(sS + 2 * 16 * kSLd);
+    __shared__ uint64_t full[kStages], empty[kStages];
+    __shared__ float s_alpha[16];
     __shared__ int s_err;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int split = blockIdx.x, splits = gridDim.x, h0 = blockIdx.y * N, r = blockIdx.z;
+    const int split = blockIdx.x, splits = gridDim.x, h0 = blockIdx.y * 16, r = blockIdx.z;
     if (tid == 0) {
-        mbar_init(&q_full, 1);
-        for (int s = 0; s < kStages; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
-        for (int s = 0; s < 2; ++s) { mbar_init(&s_full[s], 1); mbar_init(&s_free[s], 2); mbar_init(&p_full[s], 4); mbar_init(&pv_done[s], 1); }
+        for (int s = 0; s < kStages; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 8); }
         s_err = 0;
         mbar_fence_init();
     }
-    if (warp == 1) tmem_alloc<COLS>(&s_tmem);
-    fence_before();
     __syncthreads();
-    fence_after();
-    const uint32_t tmem = s_tmem, t_o = tmem + 2 * N;
     pdl_trigger();
     // positions and page tables are written in front of the step's first kernel, which is launched without overlap
     const int pos = rows.pos[r], seq = rows.seq ? rows.seq[r] : r;
     const int pages = pos / kPage + 1;
     const int n = pages > split ? (pages - split + splits - 1) / splits : 0;
 
-    if (warp == 0) {
+    if (warp == 8) {
         // the warp reads 32 entries of the page table at a time; lane 0 requests the pages
         const int32_t* pt = rows.page_table + size_t(seq) * rows.pages_per_seq;
         int entry = lane < n ? pt[split + lane * splits] : 0;
@@ -103,173 +85,143 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const __grid
         int i = 0;
         for (; i < n && i < kStages && split + i * splits < complete; ++i) request(i);
         pdl_wait();
-            // the row's queries (heads past the last read the next row's, or zero past the end: their columns are not used)
-        if (n > 0 && lane == 0) {
-            mbar_expect_tx(&q_full, uint32_t(nch * N * 128));
-            tma_3d(sQ, &map_q, 0, r * d.heads + h0, 0, &q_full);
-        }
         for (; i < n; ++i) {
             if ((i & 31) == 0 && i > 0) entry = i + lane < n ? pt[split + (i + lane) * splits] : 0;
             const bool ok = i < kStages || mbar_wait(&empty[i % kStages], (i / kStages - 1) & 1, &s_err);
             if (!__all_sync(0xffffffffu, ok)) { atomicExch(&s_err, 1); break; }
             request(i);
         }
-    }
-    if (warp == 1) {
-        if (lane == 0 && n > 0) {
-            const uint64_t q_desc = desc_kmajor(smem_u32(sQ));
-            if (!mbar_wait(&q_full, 0, &s_err)) atomicExch(&s_err, 1);
-            for (int j = 0; j < n; ++j) {
-                if (!mbar_wait(&full[j % kStages], (j / kStages) & 1, &s_err) || (j >= 2 && !mbar_wait(&s_free[j & 1], ((j >> 1) - 1) & 1, &s_err))) { atomicExch(&s_err, 1); break; }
-                fence_after();
-                uint64_t a = desc_kmajor(smem_u32(ring + size_t(j % kStages) * stage_bytes)), b = q_desc;
-                const uint32_t t_s = tmem + uint32_t((j & 1) * N);
-                for (int c = 0; c < nch; ++c, a += kChunk >> 4, b += (N * 128) >> 4)
+    } else {
+        pdl_wait();
+        // queries into shared memory (heads past the last are zero), then this warp's half of them into registers
+        {
+            const uint4* src = reinterpret_cast<const uint4*>(qabs + (size_t(r) * d.heads + h0) * W);
+            const int per = W / 8, have = min(16, d.heads - h0) * per;
+            uint4 v[5];   // every load before the first store; a row has at most nine chunks of eight pieces
 #pragma unroll
-                    for (int k = 0; k < 4; ++k) umma_ss(t_s, a + uint64_t(k * 2), b + uint64_t(k * 2), idesc_bf16(N), (c > 0 || k > 0) ? 1u : 0u);
-                umma_commit(&s_full[j & 1]);
+            for (int u = 0; u < 5; ++u) v[u] = tid + u * kConsumers < have ? src[tid + u * kConsumers] : make_uint4(0, 0, 0, 0);
+#pragma unroll
+            for (int u = 0; u < 5; ++u) {
+                const int i = tid + u * kConsumers;
+                if (i < 16 * per) *reinterpret_cast<uint4*>(sQ + (i / per) * ldq + (i % per) * 8) = v[u];
             }
         }
-    } else if (warp == 6) {
-        if (lane == 0) {
-            for (int j = 0; j < n; ++j) {
-                if (!mbar_wait(&p_full[j & 1], (j >> 1) & 1, &s_err)) { atomicExch(&s_err, 1); break; }
-                fence_after();
-                uint64_t a = desc_mnmajor(smem_u32(ring + size_t(j % kStages) * stage_bytes), kChunk);
-                const uint64_t b = desc_kmajor(smem_u32(sP) + uint32_t((j & 1) * N * 128));
-                for (int t = 0; t < tiles; ++t, a += (2 * kChunk) >> 4)
+        consumer_sync();
+        const int kg = warp & 3, kh = warp >> 2;
+        const int half = W / 32;                 // sixteen-column steps of one half
+        const int j = lane >> 3, jr = lane & 7;
+        uint32_t qf[NCH * 2][4];
 #pragma unroll
-                    for (int k16 = 0; k16 < kPage / 16; ++k16)
-                        umma_ss(t_o + uint32_t(t * N), a + uint64_t(k16 * 2048 >> 4), b + uint64_t(k16 * 2), idesc_a_mn(N), (j > 0 || k16 > 0) ? 1u : 0u);
-                umma_commit(&pv_done[j & 1]);
-                umma_commit(&empty[j % kStages]);
-            }
-        }
-    } else if (warp >= 2) {
-        pdl_wait();   // the results overwrite what an earlier layer's merge reads
-        const int quad = warp & 3, tt = tid - 64;
-        const uint32_t lane_addr = uint32_t(quad * 32) << 16;
-        constexpr int HL = 128 / N, KL = kPage / HL;   // lanes of one head, keys per lane
-        const int sh = tt / HL, sl = tt % HL;
-        float m_ref = -INFINITY, l_run = 0.f;
-        // (a wait that gave up must not leave the loop alone: the four warps meet at barriers)
-        for (int j = 0; j < n; ++j) {
-            if (!mbar_wait(&s_full[j & 1], (j >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
-            fence_after();
-            if (quad < 2) {   // the quadrants that hold the page's 64 keys
-                uint32_t v[N];
-                tmem_ld<N>(tmem + lane_addr + uint32_t((j & 1) * N), v);
-                wait_ld();
-                fence_before();
-                __syncwarp();
-                if (lane == 0) mbar_arrive(&s_free[j & 1]);
+        for (int i = 0; i < NCH * 2; ++i)
+            if (i < half) ldsm4(qf[i], smem_u32(sQ + ((j & 1) * 8 + jr) * ldq + (kh * half + i) * 16 + (j >> 1) * 8));
+        float acc[4][2][4];
 #pragma unroll
-                for (int h = 0; h < N; ++h) sS[h * kSLd + quad * 32 + lane] = __uint_as_float(v[h]);
-            }
-            softmax_sync();
-            const int key0 = (split + j * splits) * kPage;
-            float v[KL], mx = -INFINITY;
+        for (int t = 0; t < 4; ++t)
 #pragma unroll
-            for (int e = 0; e < KL; e += 4) {
-                const float4 x = *reinterpret_cast<const float4*>(sS + sh * kSLd + sl * KL + e);
-                v[e] = x.x * scale2; v[e + 1] = x.y * scale2; v[e + 2] = x.z * scale2; v[e + 3] = x.w * scale2;
-            }
+            for (int b = 0; b < 2; ++b)
 #pragma unroll
-            for (int e = 0; e < KL; ++e) { if (key0 + sl * KL + e > pos) v[e] = -INFINITY; mx = fmaxf(mx, v[e]); }
+                for (int e = 0; e < 4; ++e) acc[t][b][e] = 0.f;
+        const int nt = d.rank_p / 16;            // sixteen-column tiles of the latent; this warp: warp, warp + 8, ...
+        float m_run = -INFINITY, l_run = 0.f;    // of head 2 warp + (lane >> 4), kept by sixteen lanes
+        const int sh = 2 * warp + (lane >> 4), sl = lane & 15;
+        for (int i = 0; i < n; ++i) {
+            const int s = i % kStages;
+            // every warp of the CTA meets at the barriers below, so a wait that gave up must not leave the loop alone
+            if (!mbar_wait(&full[s], (i / kStages) & 1, &s_err)) atomicExch(&s_err, 1);
+            const uint32_t page = smem_u32(ring + size_t(s) * stage_bytes);
+            float sc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
-            for (int o = HL / 2; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-            float alpha = 1.f;
-            if (j == 0) m_ref = mx;   // a page of the split holds at least one visible key
-            else if (mx > m_ref + kLazy) { alpha = exp2f(m_ref - mx); m_ref = mx; }
-            if (sl == 0) s_alpha[sh] = alpha;
-            // this buffer of probabilities was last read by the product of page j - 2
-            if (j >= 2 && !mbar_wait(&pv_done[j & 1], ((j >> 1) - 1) & 1, &s_err)) atomicExch(&s_err, 1);
-            float sum = 0.f;
-            unsigned char* prow = sP + (j & 1) * (N * 128) + sh * 128;
-#pragma unroll
-            for (int e = 0; e < KL; e += 8) {
-                uint32_t w[4];
-#pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const float p0 = exp2f(v[e + 2 * i] - m_ref), p1 = exp2f(v[e + 2 * i + 1] - m_ref);
-                    sum += p0 + p1;
-                    w[i] = pack_bf2(p0, p1);
+            for (int k = 0; k < NCH * 2; ++k)
+                if (k < half) {
+                    uint32_t b[4];
+                    ldsm4(b, page + page_off(kg * 16 + (j >> 1) * 8 + jr, (kh * half + k) * 16 + (j & 1) * 8));
+                    mma(sc[0], qf[k], b[0], b[1]);
+                    mma(sc[1], qf[k], b[2], b[3]);
                 }
-                const int piece = (sl * KL + e) >> 3;
-                *reinterpret_cast<uint4*>(prow + ((piece ^ (sh & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
-            }
+            {
+                float* dst = sS + kh * 16 * kSLd + (lane >> 2) * kSLd + kg * 16 + (lane & 3) * 2;
 #pragma unroll
-            for (int o = HL / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-            l_run = l_run * alpha + sum;
-            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-            if (softmax_sync_or(alpha != 1.f)) {
-                // O changes scale: every product issued so far must be complete (the next one waits for this page's probabilities)
-                if (!mbar_wait(&pv_done[(j - 1) & 1], ((j - 1) >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
-                fence_after();
-                for (int t = 0; t < tiles; ++t) {
-                    uint32_t o[N];
-                    tmem_ld<N>(t_o + lane_addr + uint32_t(t * N), o);
-                    wait_ld();
-#pragma unroll
-                    for (int h = 0; h < N; ++h) o[h] = __float_as_uint(__uint_as_float(o[h]) * s_alpha[h]);
-                    tmem_st<N>(t_o + lane_addr + uint32_t(t * N), o);
+                for (int b = 0; b < 2; ++b) {
+                    *reinterpret_cast<float2*>(dst + b * 8) = make_float2(sc[b][0], sc[b][1]);
+                    *reinterpret_cast<float2*>(dst + 8 * kSLd + b * 8) = make_float2(sc[b][2], sc[b][3]);
                 }
-                wait_st();
-                fence_before();
+            }
+            consumer_sync();
+            {
+                const int key0 = (split + i * splits) * kPage;
+                const float4 a = *reinterpret_cast<const float4*>(sS + sh * kSLd + sl * 4), b = *reinterpret_cast<const float4*>(sS + (16 + sh) * kSLd + sl * 4);
+                float v[4] = {(a.x + b.x) * scale2, (a.y + b.y) * scale2, (a.z + b.z) * scale2, (a.w + b.w) * scale2};
+                float mx = -INFINITY;
+#pragma unroll
+                for (int e = 0; e < 4; ++e) { if (key0 + sl * 4 + e > pos) v[e] = -INFINITY; mx = fmaxf(mx, v[e]); }
+#pragma unroll
+                for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+                const float mn = fmaxf(m_run, mx), alpha = exp2f(m_run - mn);   // a page of the split holds at least one visible key
+                float sum = 0.f;
+#pragma unroll
+                for (int e = 0; e < 4; ++e) { v[e] = exp2f(v[e] - mn); sum += v[e]; }
+#pragma unroll
+                for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+                l_run = l_run * alpha + sum;
+                m_run = mn;
+                *reinterpret_cast<uint2*>(sP + sh * kPLd + sl * 4) = make_uint2(pack_bf2(v[0], v[1]), pack_bf2(v[2], v[3]));
+                if (sl == 0) s_alpha[sh] = alpha;
+            }
+            consumer_sync();
+            const float al0 = s_alpha[lane >> 2], al1 = s_alpha[(lane >> 2) + 8];
+            uint32_t pf[4][4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) ldsm4(pf[k], smem_u32(sP + ((j & 1) * 8 + jr) * kPLd + k * 16 + (j >> 1) * 8));
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                const int tile = warp + t * 8;
+                if (tile < nt) {
+#pragma unroll
+                    for (int b = 0; b < 2; ++b) { acc[t][b][0] *= al0; acc[t][b][1] *= al0; acc[t][b][2] *= al1; acc[t][b][3] *= al1; }
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        uint32_t b[4];
+                        ldsm4t(b, page + page_off(k * 16 + (j & 1) * 8 + jr, tile * 16 + (j >> 1) * 8));
+                        mma(acc[t][0], pf[k], b[0], b[1]);
+                        mma(acc[t][1], pf[k], b[2], b[3]);
+                    }
+                }
             }
             __syncwarp();
-            if (lane == 0) mbar_arrive(&p_full[j & 1]);
+            if (lane == 0) mbar_arrive(&empty[s]);
         }
-        if (n > 0) {
-            if (!mbar_wait(&pv_done[(n - 1) & 1], ((n - 1) >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
-            fence_after();
-            for (int t = 0; t < tiles; ++t) {
-                uint32_t o[N];
-                tmem_ld<N>(t_o + lane_addr + uint32_t(t * N), o);
-                wait_ld();
-                const int col = t * 128 + quad * 32 + lane;
-                float* dst = part + ((size_t(r) * d.heads + h0) * splits + split) * d.rank_p + col;
-                const size_t step = size_t(splits) * d.rank_p;
-                const int nh = col < d.rank_p ? min(N, d.heads - h0) : 0;
 #pragma unroll
-                for (int h = 0; h < N; ++h, dst += step)
-                    if (h < nh) *dst = __uint_as_float(o[h]);
-            }
-            fence_before();
+        for (int t = 0; t < 4; ++t) {
+            const int tile = warp + t * 8;
+            if (n > 0 && tile < nt)
+#pragma unroll
+                for (int b = 0; b < 2; ++b)
+#pragma unroll
+                    for (int hf = 0; hf < 2; ++hf) {
+                        const int h = h0 + (lane >> 2) + hf * 8;
+                        if (h < d.heads)
+                            *reinterpret_cast<float2*>(part + ((size_t(r) * d.heads + h) * splits + split) * d.rank_p + tile * 16 + b * 8 + (lane & 3) * 2) =
+                                make_float2(acc[t][b][2 * hf], acc[t][b][2 * hf + 1]);
+                    }
         }
-        if (sl == 0 && h0 + sh < d.heads) ml[(size_t(r) * d.heads + h0 + sh) * splits + split] = make_float2(m_ref, l_run);
+        if (sl == 0 && h0 + sh < d.heads) ml[(size_t(r) * d.heads + h0 + sh) * splits + split] = make_float2(m_run, l_run);
     }
     __syncthreads();
-    if (warp == 1) {
-        fence_after();
-        tmem_free<COLS>(tmem);
-    }
     if (tid == 0 && s_err && err) atomicExch(err, 1);
 }
 
-int head_tile(const LatentDims& d) { return d.heads > 16 ? 32 : 16; }
-size_t decode_smem(const LatentDims& d, int n) {
-    const size_t extra = size_t(d.row() / 64) * n * 128 + size_t(2) * n * 128 + sizeof(float) * n * kSLd;
-    return size_t(kStages) * d.row() * 128 + std::max<size_t>(extra, kChunk) + 1024;   // at least a chunk behind the ring: see the header
+size_t decode_smem(const LatentDims& d) {
+    return size_t(kStages) * d.row() * kPage * 2 + size_t(16) * (d.row() + 8) * 2 + sizeof(float) * 2 * 16 * kSLd + size_t(16) * kPLd * 2 + 1024;
 }
 
-// {64 columns, rows, chunks}: one box brings `box_rows` whole rows as chunks of swizzled 128-byte rows
-int32_t chunked_map(CUtensorMap* m, const void* base, const LatentDims& d, uint64_t rows, uint32_t box_rows) {
-    const uint32_t nch = uint32_t(d.row() / 64);
-    const uint64_t dims[3] = {64, rows, nch}, strides[2] = {uint64_t(d.row()) * 2, 128};
-    const uint32_t box[3] = {64, box_rows, nch};
-    return make_map(m, base, 3, dims, strides, box);
-}
-
-template <int N, uint32_t COLS>
+template <int NCH>
 int32_t launch(const LatentDims& d, const void* qabs, const void* map, const StepRows& rows, int splits, float* part, float2* ml, int* err, cudaStream_t st) {
-    CUtensorMap m, mq;
+    CUtensorMap m;
     memcpy(&m, map, sizeof(m));
-    FORGE_TRY(chunked_map(&mq, qabs, d, uint64_t(rows.n) * d.heads, N));
-    auto kern = latent_decode_kernel<N, COLS>;
-    const size_t smem = decode_smem(d, N);
+    auto kern = latent_decode_kernel<NCH>;
+    const size_t smem = decode_smem(d);
     FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
-    FORGE_CUDA(launch_pdl(kern, dim3(splits, (d.heads + N - 1) / N, rows.n), dim3(kThreads), smem, st, m, mq, d, rows,
+    FORGE_CUDA(launch_pdl(kern, dim3(splits, (d.heads + 15) / 16, rows.n), dim3(kThreads), smem, st, m, d, static_cast<const __nv_bfloat16*>(qabs), rows,
                           d.scale * 1.4426950408889634f, part, ml, err));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
@@ -277,12 +229,15 @@ int32_t launch(const LatentDims& d, const void* qabs, const void* map, const Ste
 
 }  // namespace
 
-bool latent_decode_tc_supported(const LatentDims& d) { return decode_smem(d, head_tile(d)) <= 224 * 1024; }
-int latent_decode_head_groups(const LatentDims& d) { return (d.heads + head_tile(d) - 1) / head_tile(d); }
+bool latent_decode_tc_supported(const LatentDims& d) { return d.row() <= 9 * 64 && d.rank_p <= 512; }
+int latent_decode_head_groups(const LatentDims& d) { return (d.heads + 15) / 16; }
 
 int32_t latent_cache_map(void* map_out, const void* cache, const LatentDims& d, size_t rows) {
     CUtensorMap m;
-    FORGE_TRY(chunked_map(&m, cache, d, rows, kPage));
+    // {64 columns, rows, chunks}: one box brings a whole page as chunks of swizzled 128-byte rows
+    const uint64_t dims[3] = {64, rows, uint64_t(d.row() / 64)}, strides[2] = {uint64_t(d.row()) * 2, 128};
+    const uint32_t box[3] = {64, kPage, uint32_t(d.row() / 64)};
+    FORGE_TRY(make_map(&m, cache, 3, dims, strides, box));
     memcpy(map_out, &m, sizeof(m));
     return FORGE_OK;
 }
@@ -290,9 +245,10 @@ int32_t latent_cache_map(void* map_out, const void* cache, const LatentDims& d, 
 int32_t latent_decode_tc(const LatentDims& d, const void* qabs, const void* map, const StepRows& rows, int splits, float* part, float2* ml, int* err, cudaStream_t st) {
     if (rows.n <= 0) return FORGE_OK;
     if (!latent_decode_tc_supported(d)) { set_error("latent decode: rows of %d values unsupported", d.row()); return FORGE_ERR_SHAPE; }
-    const int n = head_tile(d), cols = (2 + (d.rank_p + 127) / 128) * n;
-    if (n == 16) return cols <= 128 ? launch<16, 128>(d, qabs, map, rows, splits, part, ml, err, st) : launch<16, 256>(d, qabs, map, rows, splits, part, ml, err, st);
-    return cols <= 256 ? launch<32, 256>(d, qabs, map, rows, splits, part, ml, err, st) : launch<32, 512>(d, qabs, map, rows, splits, part, ml, err, st);
+    const int nch = d.row() / 64;
+    if (nch <= 3) return launch<3>(d, qabs, map, rows, splits, part, ml, err, st);
+    if (nch <= 5) return launch<5>(d, qabs, map, rows, splits, part, ml, err, st);
+    return launch<9>(d, qabs, map, rows, splits, part, ml, err, st);
 }
 
 }  // namespace forge
