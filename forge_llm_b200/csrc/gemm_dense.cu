@@ -2,11 +2,12 @@
 //
 // bfloat16 (gemm_dense_kernel): tcgen05 with both operands in shared memory.  A tile is 128 weight rows (MMA M) x NT
 // tokens (MMA N = 16 .. 256); one kernel serves a decode step (NT = 16: a weight stream, 16 KB of weights per K step and
-// SM in a ring of up to eleven stages) and a prompt (NT = 256).  The work is dealt in K steps of 64: CTA i of G takes the
-// steps [i U / G, (i + 1) U / G) of the U = tiles * K / 64 steps of the whole product, so every SM streams the same amount
-// whatever the number of tiles.  A tile that several CTAs share is finished by the last of them to arrive (ticket): every
-// share is left in scratch memory and added in K order, so the result does not depend on the order of arrival.  Nobody
-// waits for another CTA.
+// SM in a ring of up to eleven stages) and a prompt (NT = 256).  Of T tiles over G CTAs the first G floor(T / G) are, for prompts,
+// whole tiles dealt in turn (neighbouring CTAs then work on the same weight rows, which come from L2 once); the K steps of 64 of
+// the remaining tiles are dealt evenly, CTA i of S taking the steps [i U / S, (i + 1) U / S) of their U, so every SM streams the
+// same amount whatever the number of tiles.  A tile that several CTAs share is finished by the last of them to arrive
+// (ticket): every share is left in scratch memory and added in K order, so the result does not depend on the order of
+// arrival.  Nobody waits for another CTA.
 // Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = epilogue (TMEM lane = weight row).
 // The weights lie in memory as the very images the ring holds (dense_tile_image), so a stage is one contiguous 16 KB bulk copy.
 // Accumulators are double buffered in tensor memory: the epilogue of one tile runs under the products of the next.
@@ -74,13 +75,35 @@ struct GemmParams {
     const void* w;           // weight images
     int m, N, nk;            // tokens, rows, K steps per tile
     int tt_count;            // token tiles
-    long long units;         // tiles * nk
+    int waves;               // whole tiles per CTA
+    uint32_t units;          // K steps of the tiles after them, dealt to the first `sharers` CTAs (at most one per step: no share is empty)
+    int sharers;
     float* part; int* tickets;
     int* err;
 };
 
-__device__ __forceinline__ long long share_begin(long long units, int g, int grid) { return units * g / grid; }
-__device__ __forceinline__ int share_of(long long units, long long u, int grid) { return int(((u + 1) * grid - 1) / units); }
+// (32-bit: the host checks that units * sharers fits; 64-bit divisions in front of the first load cost microseconds)
+__device__ __forceinline__ uint32_t share_begin(uint32_t units, uint32_t g, uint32_t sharers) { return units * g / sharers; }
+__device__ __forceinline__ int share_of(uint32_t units, uint32_t u, uint32_t sharers) { return int(((u + 1) * sharers - 1) / units); }
+
+// the pieces of work of one CTA, in order: [k0, k0 + n) K steps of `tile`
+struct Work {
+    int cta, grid, waves, nk, wave = 0;
+    uint32_t u, u1;
+    int tile, k0, n;
+    __device__ __forceinline__ Work(const GemmParams& p, uint32_t u_begin, uint32_t u_end)
+        : cta(blockIdx.x), grid(gridDim.x), waves(p.waves), nk(p.nk), u(u_begin), u1(u_end) {}
+    __device__ __forceinline__ bool next() {
+        if (wave < waves) { tile = wave++ * grid + cta; k0 = 0; n = nk; return true; }
+        if (u >= u1) return false;
+        const int t = int(u / uint32_t(nk));
+        k0 = int(u) - t * nk;
+        n = min(int(u1 - u), nk - k0);
+        tile = waves * grid + t;
+        u += uint32_t(n);
+        return true;
+    }
+};
 
 template <int NT> struct Ring {
     static constexpr int X_BYTES = NT * 128, STAGE = 16384 + X_BYTES;
@@ -99,7 +122,8 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
     __shared__ int s_err, s_last;
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const long long u0 = share_begin(p.units, blockIdx.x, gridDim.x), u1 = share_begin(p.units, blockIdx.x + 1, gridDim.x);
+    uint32_t u0 = 0, u1 = 0;   // this CTA's share of the dealt-out K steps
+    if (int(blockIdx.x) < p.sharers) { u0 = share_begin(p.units, blockIdx.x, p.sharers); u1 = share_begin(p.units, blockIdx.x + 1, p.sharers); }
     if (tid == 0) {
         for (int s = 0; s < STAGES; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
         for (int s = 0; s < 2; ++s) { mbar_init(&acc_full[s], 1); mbar_init(&acc_empty[s], 4); }
@@ -115,30 +139,33 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
 
     if (warp == 0) {
         if (lane == 0) {
-            const int total = int(u1 - u0);
-            // position of the next weight stage and of the next activation stage, advanced without divisions
-            const int tile0 = int(u0 / p.nk);
-            int kt_w = int(u0 - (long long)tile0 * p.nk), rt_w = tile0 / p.tt_count, tt_w = tile0 % p.tt_count;
-            int kt_x = kt_w, tt_x = tt_w;
+            // two walks over the same pieces: weight stages run up to a whole ring ahead of the dependency wait
+            Work ww(p, u0, u1), wx = ww;
+            int kw = 0, row_tile = 0;
+            bool more = ww.next();
+            if (more) row_tile = ww.tile / p.tt_count;
             const unsigned char* const weights = static_cast<const unsigned char*>(p.w);
             auto weight_stage = [&](int s) {   // one contiguous image of 128 rows x 64 columns, already swizzled
                 mbar_expect_tx(&full[s], uint32_t(STAGE));
-                bulk_load(ring + size_t(s) * STAGE, weights + (size_t(rt_w) * p.nk + kt_w) * 16384, 16384, &full[s]);
-                if (++kt_w == p.nk) { kt_w = 0; if (++tt_w == p.tt_count) { tt_w = 0; ++rt_w; } }
+                bulk_load(ring + size_t(s) * STAGE, weights + (size_t(row_tile) * p.nk + ww.k0 + kw) * 16384, 16384, &full[s]);
+                if (++kw == ww.n) { kw = 0; more = ww.next(); if (more) row_tile = ww.tile / p.tt_count; }
             };
-            const int ahead = min(total, STAGES);
-            for (int i = 0; i < ahead; ++i) weight_stage(i);   // constant: may overlap the kernel in front
+            int ahead = 0;
+            for (; ahead < STAGES && more; ++ahead) weight_stage(ahead);   // constant: may overlap the kernel in front
             pdl_wait();
-            int s = 0;
+            int s = 0, i = 0;
             uint32_t phase = 1;   // parity of the round in front of the current one
-            for (int i = 0; i < total; ++i) {
-                if (i >= STAGES) {
-                    if (!mbar_wait(&empty[s], phase, &s_err)) { atomicExch(&s_err, 1); break; }
-                    weight_stage(s);
+            bool ok = true;
+            while (ok && wx.next()) {
+                const int tok0 = (wx.tile % p.tt_count) * NT;
+                for (int k = 0; k < wx.n; ++k, ++i) {
+                    if (i >= ahead) {
+                        if (!mbar_wait(&empty[s], phase, &s_err)) { atomicExch(&s_err, 1); ok = false; break; }
+                        weight_stage(s);
+                    }
+                    tma_2d(ring + size_t(s) * STAGE + 16384, &map_x, (wx.k0 + k) * BK, tok0, &full[s]);
+                    if (++s == STAGES) { s = 0; phase ^= 1; }
                 }
-                tma_2d(ring + size_t(s) * STAGE + 16384, &map_x, kt_x * BK, tt_x * NT, &full[s]);
-                if (++kt_x == p.nk) { kt_x = 0; if (++tt_x == p.tt_count) tt_x = 0; }
-                if (++s == STAGES) { s = 0; phase ^= 1; }
             }
         }
     } else if (warp == 1) {
@@ -147,9 +174,8 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
             uint32_t phase = 0;
             bool ok = true;
             int seg = 0;
-            for (long long u = u0; u < u1 && ok; ++seg) {
-                const long long tile_end = (u / p.nk + 1) * p.nk;
-                const int n = int(min(u1, tile_end) - u), buf = seg & 1;
+            for (Work w(p, u0, u1); ok && w.next(); ++seg) {
+                const int n = w.n, buf = seg & 1;
                 if (seg >= 2 && !mbar_wait(&acc_empty[buf], ((seg >> 1) - 1) & 1, &s_err)) { ok = false; break; }
                 fence_after();
                 for (int k = 0; k < n; ++k) {
@@ -164,7 +190,6 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
                     if (++s == STAGES) { s = 0; phase ^= 1; }
                 }
                 if (ok) umma_commit(&acc_full[buf]);
-                u += n;
             }
             if (!ok) atomicExch(&s_err, 1);
         }
@@ -174,10 +199,9 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
         const uint32_t lane_addr = tmem + (uint32_t(quad * 32) << 16);
         constexpr int CH = NT < 32 ? NT : 32;   // columns per read
         int seg_i = 0;
-        for (long long u = u0; u < u1; ++seg_i) {
-            const int tile = int(u / p.nk);
-            const long long t_begin = (long long)tile * p.nk, t_end = t_begin + p.nk;
-            const int n = int(min(u1, t_end) - u), buf = seg_i & 1;
+        for (Work w(p, u0, u1); w.next(); ++seg_i) {
+            const int tile = w.tile, n = w.n, buf = seg_i & 1;
+            const uint32_t t_begin = uint32_t((tile - p.waves * int(gridDim.x)) * p.nk), t_end = t_begin + uint32_t(p.nk);   // among the dealt-out steps
             const int row0 = (tile / p.tt_count) * 128 + quad * 32, tok0 = (tile % p.tt_count) * NT;
             const int row = row0 + lane;
             const int cols = min(NT, p.m - tok0);
@@ -251,7 +275,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
 #pragma unroll
                     for (int c = 0; c < CH; ++c) if (c < cols - c0) __stcg(mine + size_t(c0 + c) * 128 + quad * 32 + lane, v[c]);
                 }
-                const int first = share_of(p.units, t_begin, gridDim.x), last = share_of(p.units, t_end - 1, gridDim.x);
+                const int first = share_of(p.units, t_begin, p.sharers), last = share_of(p.units, t_end - 1, p.sharers);
                 __threadfence();
                 asm volatile("bar.sync 1, 128;" ::: "memory");
                 if (tid == 64) {
@@ -270,7 +294,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
                         // only the first share of the tile may be the second part of its CTA; loads of QB shares in flight together
                         constexpr int QB = CH == 16 ? 4 : 2;
                         const int n_c = cols - c0;
-                        const int first_slot = share_begin(p.units, first, gridDim.x) >= t_begin ? 0 : 1;
+                        const int first_slot = share_begin(p.units, first, p.sharers) >= t_begin ? 0 : 1;
                         for (int q = first; q <= last; q += QB) {
                             float t[QB][CH];
 #pragma unroll
@@ -292,7 +316,6 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
             fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(&acc_empty[buf]);
-            u += n;
         }
         fence_before();
     }
@@ -310,8 +333,12 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmPara
     FORGE_TRY(make_map_2d(&mx, act, uint64_t(w.K), uint64_t(p.m), uint64_t(act_ld) * 2, NT));
     p.tt_count = (p.m + NT - 1) / NT;
     const long long tiles = (long long)((w.N + 127) / 128) * p.tt_count;
-    p.units = tiles * p.nk;
-    const int grid = int(std::max(1LL, std::min((long long)sms, p.units / 4)));
+    const int grid = int(std::max(1LL, std::min((long long)sms, tiles * p.nk / 4)));
+    p.waves = NT >= 128 ? int(tiles / grid) : 0;   // a weight stream gains nothing from whole tiles in turn
+    const long long units = (tiles - (long long)p.waves * grid) * p.nk;
+    if (tiles * p.nk > INT32_MAX || (units + 1) * grid > INT32_MAX) { set_error("dense product: %lld tiles of %d K steps are too many", tiles, p.nk); return FORGE_ERR_SHAPE; }
+    p.units = uint32_t(units);
+    p.sharers = int(std::min((long long)grid, (units + 1) / 2));
     const size_t smem = size_t(Ring<NT>::STAGES) * Ring<NT>::STAGE + 1024;
     auto kern = gemm_dense_kernel<NT>;
     FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
