@@ -339,6 +339,9 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmPara
     if (tiles * p.nk > INT32_MAX || (units + 1) * grid > INT32_MAX) { set_error("dense product: %lld tiles of %d K steps are too many", tiles, p.nk); return FORGE_ERR_SHAPE; }
     p.units = uint32_t(units);
     p.sharers = int(std::min((long long)grid, (units + 1) / 2));
+    // leaving and adding shares costs about NT / 32 K steps: where whole tiles are no dearer, every CTA takes at most one
+    const long long rest = tiles - (long long)p.waves * grid;
+    if (rest > 0 && rest <= grid && p.nk <= units / grid + NT / 32) p.sharers = int(rest);
     const size_t smem = size_t(Ring<NT>::STAGES) * Ring<NT>::STAGE + 1024;
     auto kern = gemm_dense_kernel<NT>;
     FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));

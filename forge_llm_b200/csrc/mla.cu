@@ -70,6 +70,21 @@ constexpr int kAbsorbCols = 128;   // latent columns per CTA
 
 // blockIdx.x: group of RB rows.  blockIdx.y < heads * col blocks: queries of one head into 128 latent columns; the last RB
 // values of blockIdx.y append one row each to the cache.
+// Eight consecutive constant weights held in registers from in front of the dependency wait.  bf16 and one row per CTA only: a
+// float32 model loads them where they are used, and with several rows the registers are worth more (the weights are then
+// only asked towards L2).
+template <typename T> struct Held { static constexpr bool on = false; __device__ __forceinline__ void fetch(const T*) {} __device__ __forceinline__ void get(float (&)[8]) const {} };
+template <> struct Held<__nv_bfloat16> {
+    static constexpr bool on = true;
+    uint4 u;
+    __device__ __forceinline__ void fetch(const __nv_bfloat16* p) { u = *reinterpret_cast<const uint4*>(p); }
+    __device__ __forceinline__ void get(float (&v)[8]) const {
+        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h[i]); v[2 * i] = f.x; v[2 * i + 1] = f.y; }
+    }
+};
+
 template <typename T, int RB>
 __global__ void __launch_bounds__(kThreads) latent_post_kernel(const LatentDims d, const float* __restrict__ proj, int ldp, int dkv_col, const float* __restrict__ kv_norm,
                                                                const float2* __restrict__ rope, const T* __restrict__ uk, int uk_ld, T* __restrict__ qabs, T* __restrict__ cache,
@@ -90,8 +105,19 @@ __global__ void __launch_bounds__(kThreads) latent_post_kernel(const LatentDims 
     }
     const int h = blockIdx.y / nrb, c0 = (blockIdx.y % nrb) * kAbsorbCols;
     const T* w = uk + size_t(h) * d.dim * uk_ld + c0;
-    for (int i = threadIdx.x; i < d.dim * 2; i += kThreads)   // the weights are constant: towards L2 while the kernel in front runs
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(w + size_t(i >> 1) * uk_ld) + (i & 1) * 128));
+    // sixteen threads cover the columns, sixteen groups of them share the dimensions; the weights are constant: the first
+    // kHeld rows of every thread are fetched while the kernel in front runs
+    constexpr int kHeld = 8;
+    constexpr bool kHold = Held<T>::on && RB == 1;
+    const int col = (threadIdx.x & 15) * 8, group = threadIdx.x >> 4;
+    const bool col_ok = c0 + col < d.rank_p;
+    Held<T> held[kHeld];
+    if (!kHold)
+        for (int i = threadIdx.x; i < d.dim * 2; i += kThreads)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(w + size_t(i >> 1) * uk_ld) + (i & 1) * 128));
+    if (kHold && col_ok)
+#pragma unroll
+        for (int i = 0; i < kHeld; ++i) if (group + 16 * i < d.dim) held[i].fetch(w + size_t(group + 16 * i) * uk_ld + col);
     pdl_trigger();
     pdl_wait();
     float* sq = sm;
@@ -102,25 +128,26 @@ __global__ void __launch_bounds__(kThreads) latent_post_kernel(const LatentDims 
         sq[i] = j < nr ? proj[size_t(r0 + j) * ldp + h * qd + e] : 0.f;
     }
     __syncthreads();
-    // sixteen threads cover the columns, sixteen groups of them share the dimensions
-    const int col = (threadIdx.x & 15) * 8, part = threadIdx.x >> 4;
     float a[RB][8];
 #pragma unroll
     for (int j = 0; j < RB; ++j)
 #pragma unroll
         for (int c = 0; c < 8; ++c) a[j][c] = 0.f;
-    if (c0 + col < d.rank_p) {
-#pragma unroll 8
-        for (int e = part; e < d.dim; e += 16) {
-            float v[8];
-            load8(v, w + size_t(e) * uk_ld + col);
+    if (col_ok) {
+        auto add = [&](int e, const float (&v)[8]) {
 #pragma unroll
             for (int j = 0; j < RB; ++j) {
                 const float q = sq[j * d.dim + e];
 #pragma unroll
                 for (int c = 0; c < 8; ++c) a[j][c] = fmaf(q, v[c], a[j][c]);
             }
-        }
+        };
+        float v[8];
+        if (kHold)
+#pragma unroll
+            for (int i = 0; i < kHeld; ++i) if (group + 16 * i < d.dim) { held[i].get(v); add(group + 16 * i, v); }
+#pragma unroll 8
+        for (int e = group + (kHold ? 16 * kHeld : 0); e < d.dim; e += 16) { load8(v, w + size_t(e) * uk_ld + col); add(e, v); }
     }
 #pragma unroll
     for (int j = 0; j < RB; ++j) {   // lanes l and l + 16 hold the same columns
@@ -245,14 +272,25 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentDims
     const int h = blockIdx.y, v0 = blockIdx.z * kValueRows, r0 = blockIdx.x * RB, nr = min(RB, rows - r0);
     const int nv = min(kValueRows, d.vdim - v0);
     const T* w = uv + (size_t(h) * d.vdim + v0) * uv_ld;
-    const int lines = int((size_t(d.rank_p) * sizeof(T) + 127) / 128);
-    for (int i = threadIdx.x; i < nv * lines; i += kThreads)
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(w + size_t(i / lines) * uv_ld) + (i % lines) * 128));
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    // four rows of W_uv per warp; their first kHeld pieces are fetched while the kernel in front runs
+    constexpr int VR = kValueRows / (kThreads / 32), kHeld = 2, kUnroll = RB == 1 ? 16 : 4;
+    constexpr bool kHold = Held<T>::on && RB == 1;
+    Held<T> held[VR][kHeld];
+    if (!kHold) {
+        const int lines = int((size_t(d.rank_p) * sizeof(T) + 127) / 128);
+        for (int i = threadIdx.x; i < nv * lines; i += kThreads)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(w + size_t(i / lines) * uv_ld) + (i % lines) * 128));
+    }
+    if (kHold)
+#pragma unroll
+    for (int v = 0; v < VR; ++v)
+#pragma unroll
+        for (int i = 0; i < kHeld; ++i) if (lane * 8 + 256 * i < d.rank_p) held[v][i].fetch(w + size_t(min(warp * VR + v, nv - 1)) * uv_ld + lane * 8 + 256 * i);
     pdl_trigger();
     pdl_wait();
     float* lat = sm;
     float* fac = sm + RB * d.rank_p;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (warp < nr) {   // RB <= 8 warps: one row each
         const float2* p = ml + (size_t(r0 + warp) * d.heads + h) * splits;
         float mt = -INFINITY;
@@ -282,7 +320,7 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentDims
             const int n = min(splits, rows_pos[r0 + j] / FORGE_KV_PAGE + 1);   // splits that own a page
             const float* p = part + (size_t(r0 + j) * d.heads + h) * splits * d.rank_p + c;
             float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
+#pragma unroll kUnroll
             for (int s = hf; s < n; s += halves) {
                 const float f = fac[j * splits + s];
                 const float4 x = *reinterpret_cast<const float4*>(p + size_t(s) * d.rank_p);
@@ -297,17 +335,12 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentDims
         for (int i = nr * d.rank_p + threadIdx.x; i < RB * d.rank_p; i += kThreads) lat[i] = 0.f;
     }
     __syncthreads();
-    // four rows of W_uv per warp: their loads are in flight together
-    constexpr int VR = kValueRows / (kThreads / 32);
     float acc[VR][RB];
 #pragma unroll
     for (int v = 0; v < VR; ++v)
 #pragma unroll
         for (int j = 0; j < RB; ++j) acc[v][j] = 0.f;
-    for (int c = lane * 8; c < d.rank_p; c += 256) {
-        float a[VR][8];
-#pragma unroll
-        for (int v = 0; v < VR; ++v) load8(a[v], w + size_t(min(warp * VR + v, nv - 1)) * uv_ld + c);
+    auto add = [&](int c, const float (&a)[VR][8]) {
 #pragma unroll
         for (int j = 0; j < RB; ++j) {
             float x[8];
@@ -317,6 +350,20 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentDims
 #pragma unroll
                 for (int e = 0; e < 8; ++e) acc[v][j] = fmaf(a[v][e], x[e], acc[v][j]);
         }
+    };
+    float a[VR][8];
+    if (kHold)
+#pragma unroll
+        for (int i = 0; i < kHeld; ++i)
+            if (lane * 8 + 256 * i < d.rank_p) {
+#pragma unroll
+                for (int v = 0; v < VR; ++v) held[v][i].get(a[v]);
+                add(lane * 8 + 256 * i, a);
+            }
+    for (int c = lane * 8 + (kHold ? 256 * kHeld : 0); c < d.rank_p; c += 256) {
+#pragma unroll
+        for (int v = 0; v < VR; ++v) load8(a[v], w + size_t(min(warp * VR + v, nv - 1)) * uv_ld + c);
+        add(c, a);
     }
 #pragma unroll
     for (int v = 0; v < VR; ++v)
