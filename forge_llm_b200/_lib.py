@@ -43,7 +43,8 @@ class ForgeSampling(C.Structure):
 
 class ForgeCheckpointInfo(C.Structure):
     _fields_ = [("architecture", C.c_char * 64), ("hidden_size", C.c_int32), ("vocab_size", C.c_int32), ("num_layers", C.c_int32),
-                ("num_weight_layers", C.c_int32), ("parameters", C.c_int64), ("cache_values_per_token", C.c_int64)]
+                ("num_weight_layers", C.c_int32), ("parameters", C.c_int64), ("cache_values_per_token", C.c_int64),
+                ("state_values_per_sequence", C.c_int64)]
 
 
 class ForgeStepEntry(C.Structure):
@@ -116,6 +117,9 @@ SIGNATURES = {
     "forge_kv_reset": (i32, [vp]),
     "forge_kv_len": (i32, [vp, i32]),
     "forge_kv_destroy": (None, [vp]),
+    "forge_kv_width": (i32, [vp, i32, i32]),
+    "forge_kv_state_values": (C.c_int64, [vp, i32]),
+    "forge_kv_state_read": (i32, [vp, i32, i32, vp]),
     "forge_kv_read": (i32, [vp, i32, i32, i32, vp]),
     "forge_kv_save_size": (sz, [vp, i32]),
     "forge_kv_save": (i32, [vp, i32, vp, sz]),

@@ -1,13 +1,15 @@
-// Prompt attention over keys and values formed for this call (latent attention), bfloat16, tcgen05.  The structure is that
-// of attn_prefill_tc5.cu - S = Q K^T in tensor memory, lazy running maximum, probabilities back into tensor memory as the
-// operand of O += P V, three overlapped stages - with these differences: the query / key width (an unrotated part per head
-// plus a rotated part whose keys all heads share) and the value width are independent run-time sizes, several sequences'
-// tiles run in one launch (a table gives each tile's rows, position and context), and the epilogue applies the output gate.
+// Prompt attention of the layer-list models, bfloat16, tcgen05: over keys and values formed for this call (latent attention) or over
+// the pages of the cache (a page is one key tile).  The structure is that of attn_prefill_tc5.cu - S = Q K^T in tensor memory,
+// lazy running maximum, probabilities back into tensor memory as the operand of O += P V, three overlapped stages - with these
+// differences: the query / key width (a part per head plus, optionally, a part whose keys all heads share) and the value width
+// are independent run-time sizes, several query heads may share a key head, the scores may be capped and the keys limited to the
+// query's chunk, several sequences' tiles run in one launch (a table gives each tile's rows, position and context), and the
+// epilogue applies an output gate per value or per head.
 // Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = softmax, rescale, store.
 // Tensor memory: S [0, 64), P0 [64, 96), P1 [96, 128), O from 128.
 #include <algorithm>
 
-#include "mla.cuh"
+#include "attn_prompt.cuh"
 #include "tc5.cuh"
 
 namespace forge {
@@ -21,7 +23,7 @@ constexpr uint32_t kColS = 0, kColP = 64, kColO = 128;
 constexpr float kLazy = 8.f;
 
 struct Params {
-    LatentDims d;
+    PromptDims d;
     PromptAttnArgs a;
     float scale2;
     int stages;
@@ -37,7 +39,7 @@ template <uint32_t COLS>
 __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                                                                    const __grid_constant__ CUtensorMap map_r, const __grid_constant__ CUtensorMap map_v, const __grid_constant__ Params p) {
     constexpr int Q_CHUNK = BM * 128, KV_CHUNK = BN * 128, kMaxStages = 3;
-    const LatentDims& d = p.d;
+    const PromptDims& d = p.d;
     const int kch = d.dim_p / 64, rch = d.rot_p / 64, vch = d.vdim_p / 64, qch = kch + rch;
     const int stage_bytes = (qch + vch) * KV_CHUNK, KVS = p.stages;
     extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -49,7 +51,8 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = blockIdx.x;
     const PromptTile t = p.a.tiles[blockIdx.y];
-    const int nblk = (t.pos0 + t.rows - 1) / BN + 1;
+    const int jb = (d.chunk > 0 ? t.pos0 / d.chunk * d.chunk : 0) / BN;   // the first key tile anybody sees
+    const int nblk = (t.pos0 + t.rows - 1) / BN + 1 - jb;
 
     if (tid == 0) {
         mbar_init(&q_full, 1);
@@ -73,12 +76,12 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
             for (int j = 0; j < nblk; ++j) {
                 const int s = j % KVS, use = j / KVS;
                 if (use > 0 && !mbar_wait(&kv_empty[s], (use - 1) & 1, &s_err)) { atomicExch(&s_err, 1); break; }
-                const int row = t.ctx0 + j * BN;
+                const int row = p.a.pages ? p.a.pages[t.ctx0 / BN + jb + j] * BN : t.ctx0 + (jb + j) * BN, hk = h / d.share;
                 unsigned char* dst = sKV + size_t(s) * stage_bytes;
                 mbar_expect_tx(&kv_full[s], uint32_t(stage_bytes));
-                for (int c = 0; c < kch; ++c) tma_3d(dst + c * KV_CHUNK, &map_k, c * 64, h, row, &kv_full[s]);
+                for (int c = 0; c < kch; ++c) tma_3d(dst + c * KV_CHUNK, &map_k, c * 64, hk, row, &kv_full[s]);
                 for (int c = 0; c < rch; ++c) tma_2d(dst + (kch + c) * KV_CHUNK, &map_r, c * 64, row, &kv_full[s]);
-                for (int c = 0; c < vch; ++c) tma_3d(dst + (qch + c) * KV_CHUNK, &map_v, c * 64, h, row, &kv_full[s]);
+                for (int c = 0; c < vch; ++c) tma_3d(dst + (qch + c) * KV_CHUNK, &map_v, c * 64, hk, row, &kv_full[s]);
             }
         }
     } else if (warp == 1) {
@@ -118,12 +121,15 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
     } else {
         const int quad = warp & 3;
         const int r = quad * 32 + lane;
-        const int pq = t.pos0 + r;
+        const int pq = t.pos0 + r, lo = d.chunk > 0 ? pq / d.chunk * d.chunk : 0;
+        const int lo_last = d.chunk > 0 ? (t.pos0 + t.rows - 1) / d.chunk * d.chunk : 0;   // of the tile's last row
+        const float scale2 = d.softcap > 0.f ? d.softcap * 1.4426950408889634f : p.scale2, cap2 = d.softcap > 0.f ? 2.f * p.scale2 / d.softcap : 0.f;
         const uint32_t lane_addr = tmem + (uint32_t(quad * 32) << 16);
+        const uint32_t masked = scale2 < 0.f ? 0x7f800000u : 0xff800000u;   // -inf behind the scale
         float m_ref = -INFINITY, l_run = 0.f;
         bool ok = true;
         for (int j = 0; j < nblk; ++j) {
-            const int t0 = j * BN;
+            const int t0 = (jb + j) * BN;
             if (ok && !mbar_wait(&s_full, j & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
             fence_after();
             uint32_t sv[2][32];
@@ -133,14 +139,18 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
             fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(&s_free);
-            if (t0 + BN - 1 > t.pos0) {
+            if (d.softcap > 0.f) {   // tanh(x) = 1 - 2 / (1 + exp(2 x)); scale2 then holds the cap
+#pragma unroll
+                for (int c = 0; c < 64; ++c) sv[c >> 5][c & 31] = __float_as_uint(1.f - __fdividef(2.f, 1.f + ex2(fminf(__uint_as_float(sv[c >> 5][c & 31]) * cap2, 120.f))));
+            }
+            if (t0 + BN - 1 > t.pos0 || t0 < lo_last) {
 #pragma unroll
                 for (int c = 0; c < 64; ++c)
-                    if (t0 + c > pq) sv[c >> 5][c & 31] = 0xff800000u;  // -inf
+                    if (t0 + c > pq || t0 + c < lo) sv[c >> 5][c & 31] = masked;
             }
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-            for (int c = 0; c < 64; ++c) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(sv[c >> 5][c & 31]) * p.scale2);   // the scale may have either sign
+            for (int c = 0; c < 64; ++c) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(sv[c >> 5][c & 31]) * scale2);   // the scale may have either sign
             const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
             float alpha = 1.f;
             if (m_ref == -INFINITY) m_ref = mx;
@@ -150,8 +160,8 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
             uint32_t ph[32];
 #pragma unroll
             for (int c = 0; c < 64; c += 2) {
-                const float p0 = ex2(fmaf(__uint_as_float(sv[c >> 5][c & 31]), p.scale2, -m_use));
-                const float p1 = ex2(fmaf(__uint_as_float(sv[c >> 5][(c & 31) + 1]), p.scale2, -m_use));
+                const float p0 = ex2(fmaf(__uint_as_float(sv[c >> 5][c & 31]), scale2, -m_use));
+                const float p1 = ex2(fmaf(__uint_as_float(sv[c >> 5][(c & 31) + 1]), scale2, -m_use));
                 sum4[(c >> 1) & 3] += p0 + p1;
                 ph[c >> 1] = pack_bf2(p0, p1);
             }
@@ -178,7 +188,9 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
         }
         if (ok && !mbar_wait(&pv_done[(nblk - 1) & 1], ((nblk - 1) >> 1) & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
         fence_after();
-        const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+        const bool per_value = p.a.gate != nullptr;
+        const float head_gate = per_value || r >= t.rows ? 1.f : p.a.head_gate[size_t(t.row0 + r) * d.heads + h];
+        const float inv = l_run > 0.f ? head_gate / l_run : 0.f;
         const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(p.a.gate) + size_t(t.row0 + r) * p.a.gate_ld + h * d.vdim;
         __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.a.out) + size_t(t.row0 + r) * p.a.out_ld + h * d.vdim;
         const bool vec = !(d.vdim & 7) && !(p.a.gate_ld & 7) && !(p.a.out_ld & 7);   // 16-byte pieces stay aligned
@@ -192,7 +204,7 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
 #pragma unroll
                     for (int i = 0; i < 32; i += 8)
                         if (i < nc) {
-                            const uint4 g4 = *reinterpret_cast<const uint4*>(gate + c0 + i);
+                            const uint4 g4 = per_value ? *reinterpret_cast<const uint4*>(gate + c0 + i) : make_uint4(0x3f803f80u, 0x3f803f80u, 0x3f803f80u, 0x3f803f80u);   // ones
                             const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&g4);
                             uint32_t w[4];
 #pragma unroll
@@ -205,7 +217,7 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
                 } else {
 #pragma unroll
                     for (int i = 0; i < 32; ++i)
-                        if (i < nc) out[c0 + i] = __float2bfloat16_rn(__uint_as_float(o[i]) * inv * __bfloat162float(gate[c0 + i]));
+                        if (i < nc) out[c0 + i] = __float2bfloat16_rn(__uint_as_float(o[i]) * inv * (per_value ? __bfloat162float(gate[c0 + i]) : 1.f));
                 }
             }
         }
@@ -219,25 +231,26 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
     if (tid == 0 && s_err && p.a.err) atomicExch(p.a.err, 1);
 }
 
-size_t smem_bytes(const LatentDims& d, int stages) {
+size_t smem_bytes(const PromptDims& d, int stages) {
     const int qch = (d.dim_p + d.rot_p) / 64, vch = d.vdim_p / 64;
     return size_t(qch) * BM * 128 + size_t(stages) * (qch + vch) * BN * 128 + 1024;
 }
 
 }  // namespace
 
-bool attn_prefill_kv_supported(const LatentDims& d) { return d.vdim_p <= 256 && smem_bytes(d, 2) <= 220 * 1024; }
+bool attn_prefill_kv_supported(const PromptDims& d) { return d.vdim_p <= 256 && smem_bytes(d, 2) <= 220 * 1024; }
 
-int32_t attn_prefill_kv(const LatentDims& d, const PromptAttnArgs& a, cudaStream_t st) {
+int32_t attn_prefill_kv(const PromptDims& d, const PromptAttnArgs& a, cudaStream_t st) {
     if (a.n_tiles <= 0) return FORGE_OK;
     if (!attn_prefill_kv_supported(d)) { set_error("prompt attention: head sizes %d + %d / %d unsupported", d.dim, d.rot, d.vdim); return FORGE_ERR_SHAPE; }
     CUtensorMap mq, mk, mr, mv;
-    const uint64_t qd = uint64_t(d.dim_p + d.rot_p), H = uint64_t(d.heads);
+    const uint64_t qd = uint64_t(d.dim_p + d.rot_p), H = uint64_t(d.heads), G = H / d.share;
+    const uint64_t k_row = a.pages ? uint64_t(a.page_row) * 2 : G * d.dim_p * 2, v_row = a.pages ? k_row : G * d.vdim_p * 2;
     FORGE_TRY(make_map_3d(&mq, a.q, qd, H, uint64_t(a.q_rows), qd * 2, H * qd * 2, BM));
-    FORGE_TRY(make_map_3d(&mk, a.k, uint64_t(d.dim_p), H, uint64_t(a.ctx_rows), uint64_t(d.dim_p) * 2, H * d.dim_p * 2, BN));
+    FORGE_TRY(make_map_3d(&mk, a.k, uint64_t(d.dim_p), G, uint64_t(a.ctx_rows), uint64_t(d.dim_p) * 2, k_row, BN));
     if (d.rot_p == 0) mr = mk;   // no rotated part: never read
     else FORGE_TRY(make_map_2d(&mr, a.krot, uint64_t(d.rot_p), uint64_t(a.ctx_rows), uint64_t(d.rot_p) * 2, BN));
-    FORGE_TRY(make_map_3d(&mv, a.v, uint64_t(d.vdim_p), H, uint64_t(a.ctx_rows), uint64_t(d.vdim_p) * 2, H * d.vdim_p * 2, BN));
+    FORGE_TRY(make_map_3d(&mv, a.v, uint64_t(d.vdim_p), G, uint64_t(a.ctx_rows), uint64_t(d.vdim_p) * 2, v_row, BN));
     Params p{d, a, d.scale * 1.4426950408889634f, smem_bytes(d, 3) <= 220 * 1024 ? 3 : 2};
     const size_t smem = smem_bytes(d, p.stages);
     auto go = [&](auto kern) -> int32_t {

@@ -41,6 +41,8 @@ public:
     const Json& config() const { return config_; }
     // null and an error message if it is absent or has another shape ({} = scalar)
     const TensorView* tensor(const std::string& name, const std::vector<int64_t>& shape) const;
+    // null if it is absent
+    const TensorView* find(const std::string& name) const { auto it = tensors_.find(name); return it == tensors_.end() ? nullptr : &it->second; }
     int64_t parameters() const;
 
 private:

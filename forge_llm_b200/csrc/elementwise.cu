@@ -166,21 +166,21 @@ __global__ void embedding_kernel(float* out, const float* table, const uint32_t*
     for (int i = threadIdx.x; i < h / 4; i += blockDim.x) dst[i] = src[i];
 }
 
-// embedding row -> residual stream f32, and its Dynamic Tanh norm tanh(alpha x) w + b as the first layer's input
+// embedding row -> residual stream f32, what its first reader takes, and the step's bookkeeping
 template <typename T>
-__global__ void embed_dyt_kernel(float* __restrict__ x, T* __restrict__ h, int h_ld, const T* __restrict__ table, const uint32_t* __restrict__ tokens, int width, float alpha,
-                                 const float* __restrict__ w, const float* __restrict__ b, uint32_t* hist, const int32_t* step) {
+__global__ void embed_rows_kernel(const EmbedArgs a) {
     const int r = blockIdx.x;
-    if (hist && blockIdx.y == 0 && threadIdx.x == 0) hist[size_t(*step) * gridDim.x + r] = tokens[r];
-    const T* src = table + size_t(tokens[r]) * width;
-    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < h_ld; i += gridDim.y * blockDim.x) {
-        float n = 0.f;
-        if (i < width) {
-            const float v = float(src[i]);
-            x[size_t(r) * width + i] = v;
-            n = tanhf(alpha * v) * w[i] + b[i];
-        }
-        h[size_t(r) * h_ld + i] = T(n);
+    if (blockIdx.y == 0 && threadIdx.x == 0) {
+        if (a.hist) a.hist[size_t(*a.step) * gridDim.x + r] = a.tokens[r];
+        if (a.place) a.place[r] = int32_t(cache_row(a.rows, r, a.rows.pos[r]));
+    }
+    const T* src = static_cast<const T*>(a.table) + size_t(a.tokens[r]) * a.width;
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < a.width_p; i += gridDim.y * blockDim.x) {
+        const float v = i < a.width ? to_f(src[i]) : 0.f;
+        if (i < a.width) a.x[size_t(r) * a.width + i] = v;
+        static_cast<T*>(a.after.dst)[size_t(r) * a.after.ld + i] =
+            to_t<T>(i >= a.width ? 0.f : a.after.kind == AFTER_DYT ? dynamic_tanh(v, a.after.alpha, a.after.w[i], a.after.b[i]) : v);
+        if (a.x0) static_cast<T*>(a.x0)[size_t(r) * a.x0_ld + i] = to_t<T>(v);
     }
 }
 
@@ -561,13 +561,12 @@ int32_t gather_rows_f16(float* out, const __half* pool, const int32_t* page_row,
     return FORGE_OK;
 }
 
-int32_t embed_dyt(float* x, void* h, int h_ld, const void* table, int dtype, const uint32_t* tokens, int rows, int width, float alpha,
-                  const float* w, const float* b, uint32_t* hist, const int32_t* step, cudaStream_t st) {
+int32_t embed_rows(const EmbedArgs& a, int dtype, cudaStream_t st) {
+    const int rows = a.rows.n;
     if (rows <= 0) return FORGE_OK;
-    if (dtype == FORGE_F32)
-        embed_dyt_kernel<float><<<dim3(rows, rows < 64 ? (h_ld + 255) / 256 : 1), 256, 0, st>>>(x, static_cast<float*>(h), h_ld, static_cast<const float*>(table), tokens, width, alpha, w, b, hist, step);
-    else
-        embed_dyt_kernel<__nv_bfloat16><<<dim3(rows, rows < 64 ? (h_ld + 255) / 256 : 1), 256, 0, st>>>(x, static_cast<__nv_bfloat16*>(h), h_ld, static_cast<const __nv_bfloat16*>(table), tokens, width, alpha, w, b, hist, step);
+    const dim3 grid(rows, rows < 64 ? (a.width_p + 255) / 256 : 1);
+    if (dtype == FORGE_F32) embed_rows_kernel<float><<<grid, 256, 0, st>>>(a);
+    else embed_rows_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(a);
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }

@@ -34,17 +34,20 @@ __device__ __forceinline__ float clamped_glu(float gate, float up, float limit) 
     return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
 }
 
-
 // The fields of a segment this thread's row needs, in registers: a store through a pointer may not make the compiler fetch them
 // again for every value.
 template <typename T>
 struct RowOut {
     int kind;
     bool ok;                 // the row belongs to a segment
+    bool fresh;
     size_t ld;
     float* f32; T* t;        // the row's place of token 0
+    const int32_t* place;
+    int after;
     T* next; size_t next_ld;
-    float limit, alpha, nw, nb;
+    float limit, mul, add, alpha, nw, nb;
+    __device__ __forceinline__ float next_value(float x) const { return after == AFTER_DYT ? dynamic_tanh(x, alpha, nw, nb) : x; }
 };
 template <typename T>
 __device__ __forceinline__ RowOut<T> row_out(const DenseOut& o, int row, int first_row) {
@@ -54,21 +57,34 @@ __device__ __forceinline__ RowOut<T> row_out(const DenseOut& o, int row, int fir
         if (first_row >= o.seg[i].row0 && first_row < o.seg[i].row0 + o.seg[i].rows) s = i;
     q.kind = -1;
     if (s < 0) return q;
-    const int r = row - o.seg[s].row0, group = o.seg[s].group;
-    q.kind = o.seg[s].kind;
-    q.ok = r < o.seg[s].rows;
-    q.ld = size_t(o.seg[s].ld);
-    const int col = q.kind == SEG_CLAMPED_GLU ? r >> 1 : (q.kind == SEG_CAST && group) ? (r / group) * o.seg[s].group_ld + r % group : r;
-    q.f32 = static_cast<float*>(o.seg[s].dst) + col;
-    q.t = static_cast<T*>(o.seg[s].dst) + col;
-    q.limit = o.seg[s].limit;
-    if (q.kind == SEG_RESID && o.seg[s].next && q.ok) {
-        q.alpha = o.seg[s].alpha; q.nw = o.seg[s].norm_w[r]; q.nb = o.seg[s].norm_b[r];
-        q.next = static_cast<T*>(o.seg[s].next) + r; q.next_ld = size_t(o.seg[s].next_ld);
+    const OutSeg& g = o.seg[s];
+    const int r = row - g.row0, group = g.group;
+    q.kind = g.kind;
+    q.ok = r < g.rows;
+    q.ld = size_t(g.ld);
+    q.fresh = g.fresh;
+    const int col = (q.kind == SEG_CLAMPED_GLU || q.kind == SEG_SILU_GLU) ? r >> 1 : (q.kind == SEG_CAST && group) ? (r / group) * g.group_ld + r % group : r;
+    q.f32 = static_cast<float*>(g.dst) + col;
+    q.t = static_cast<T*>(g.dst) + col;
+    q.place = g.place;
+    q.limit = g.limit;
+    if (q.ok) {
+        if (g.mul) q.mul = g.mul[r];
+        if (g.add) q.add = g.add[r];
+        if (q.kind == SEG_RESID) {
+            q.after = g.after.kind;
+            if (q.after == AFTER_DYT) { q.alpha = g.after.alpha; q.nw = g.after.w[r]; q.nb = g.after.b[r]; }
+            q.next = static_cast<T*>(g.after.dst) + r; q.next_ld = size_t(g.after.ld);
+        }
     }
     return q;
 }
-__device__ __forceinline__ float sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
+// column of the activations the rows of the tile at `row` are multiplied with
+__device__ __forceinline__ int act_col(const DenseOut& o, int row) {
+    int c = 0;
+    for (int i = 0; i < o.nseg; ++i) if (o.seg[i].row0 <= row) c = o.seg[i].act_col;
+    return c;
+}
 
 struct GemmParams {
     DenseOut out;
@@ -157,13 +173,13 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
             uint32_t phase = 1;   // parity of the round in front of the current one
             bool ok = true;
             while (ok && wx.next()) {
-                const int tok0 = (wx.tile % p.tt_count) * NT;
+                const int tok0 = (wx.tile % p.tt_count) * NT, col0 = act_col(p.out, wx.tile / p.tt_count * 128);
                 for (int k = 0; k < wx.n; ++k, ++i) {
                     if (i >= ahead) {
                         if (!mbar_wait(&empty[s], phase, &s_err)) { atomicExch(&s_err, 1); ok = false; break; }
                         weight_stage(s);
                     }
-                    tma_2d(ring + size_t(s) * STAGE + 16384, &map_x, (wx.k0 + k) * BK, tok0, &full[s]);
+                    tma_2d(ring + size_t(s) * STAGE + 16384, &map_x, col0 + (wx.k0 + k) * BK, tok0, &full[s]);
                     if (++s == STAGES) { s = 0; phase ^= 1; }
                 }
             }
@@ -213,40 +229,52 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
             auto finish = [&](int c0, const float (&v)[CH]) {
                 const int n_c = cols - c0;
                 const size_t t0 = size_t(tok0 + c0);
-                if (g.kind == SEG_CLAMPED_GLU) {
+                auto put_t = [&](auto f) {
+                    __nv_bfloat16* dst = g.t + t0 * g.ld;
+#pragma unroll
+                    for (int c = 0; c < CH; ++c) if (c < n_c) dst[c * g.ld] = __float2bfloat16_rn(f(v[c]));
+                };
+                auto put_f = [&](auto f) {
+                    float* dst = g.f32 + t0 * g.ld;
+#pragma unroll
+                    for (int c = 0; c < CH; ++c) if (c < n_c) dst[c * g.ld] = f(v[c]);
+                };
+                if (g.kind == SEG_CLAMPED_GLU || g.kind == SEG_SILU_GLU) {
                     // neighbouring lanes hold gate_j and up_j: the even lane takes the first half of the columns
-                    const bool even = !(lane & 1);
+                    const bool even = !(lane & 1), clamped = g.kind == SEG_CLAMPED_GLU;
                     __nv_bfloat16* dst = g.t + (t0 + (even ? 0 : CH / 2)) * g.ld;
 #pragma unroll
                     for (int c = 0; c < CH / 2; ++c) {
                         const float got = __shfl_xor_sync(0xffffffffu, even ? v[CH / 2 + c] : v[c], 1);
                         const float ga = even ? v[c] : got, up = even ? got : v[CH / 2 + c];
-                        if (g.ok && (even ? c : CH / 2 + c) < n_c) dst[c * g.ld] = __float2bfloat16_rn(clamped_glu(ga, up, g.limit));
+                        if (g.ok && (even ? c : CH / 2 + c) < n_c) dst[c * g.ld] = __float2bfloat16_rn(clamped ? clamped_glu(ga, up, g.limit) : silu(ga) * up);
                     }
-                } else if (!g.ok) {
-                } else if (g.kind == SEG_F32) {
-                    float* dst = g.f32 + t0 * g.ld;
+                } else if (g.ok) switch (g.kind) {
+                    case SEG_F32: put_f([](float x) { return x; }); break;
+                    case SEG_CAST:
+                        if (g.place) {
 #pragma unroll
-                    for (int c = 0; c < CH; ++c) if (c < n_c) dst[c * g.ld] = v[c];
-                } else if (g.kind == SEG_CAST) {
-                    __nv_bfloat16* dst = g.t + t0 * g.ld;
+                            for (int c = 0; c < CH; ++c) if (c < n_c) g.t[size_t(g.place[t0 + c]) * g.ld] = __float2bfloat16_rn(v[c]);
+                        } else put_t([](float x) { return x; });
+                        break;
+                    case SEG_SIGMOID: put_t([](float x) { return sigmoid(x); }); break;
+                    case SEG_SILU: put_t([](float x) { return silu(x); }); break;
+                    case SEG_TANH: put_t([](float x) { return tanhf(x); }); break;
+                    case SEG_SIGMOID_F32: put_f([](float x) { return sigmoid(x); }); break;
+                    case SEG_DECAY: put_f([&](float x) { return -g.mul * softplus(x + g.add); }); break;
+                    case SEG_EXP_DECAY: put_f([&](float x) { return -expf(x + g.add); }); break;
+                    default: {
+                        float* dst = g.f32 + t0 * g.ld;
+                        float x[CH];
 #pragma unroll
-                    for (int c = 0; c < CH; ++c) if (c < n_c) dst[c * g.ld] = __float2bfloat16_rn(v[c]);
-                } else if (g.kind == SEG_SIGMOID) {
-                    __nv_bfloat16* dst = g.t + t0 * g.ld;
+                        for (int c = 0; c < CH; ++c) x[c] = c < n_c && !g.fresh ? dst[c * g.ld] : 0.f;   // all loads before the first store
 #pragma unroll
-                    for (int c = 0; c < CH; ++c) if (c < n_c) dst[c * g.ld] = __float2bfloat16_rn(sigmoid(v[c]));
-                } else {
-                    float* dst = g.f32 + t0 * g.ld;
-                    float x[CH];
+                        for (int c = 0; c < CH; ++c) { x[c] += v[c] + g.add; if (c < n_c) dst[c * g.ld] = x[c]; }
+                        if (g.after) {
+                            __nv_bfloat16* nx = g.next + t0 * g.next_ld;
 #pragma unroll
-                    for (int c = 0; c < CH; ++c) x[c] = c < n_c ? dst[c * g.ld] : 0.f;   // all loads before the first store
-#pragma unroll
-                    for (int c = 0; c < CH; ++c) { x[c] += v[c]; if (c < n_c) dst[c * g.ld] = x[c]; }
-                    if (g.next) {
-                        __nv_bfloat16* nx = g.next + t0 * g.next_ld;
-#pragma unroll
-                        for (int c = 0; c < CH; ++c) if (c < n_c) nx[c * g.next_ld] = __float2bfloat16_rn(tanhf(g.alpha * x[c]) * g.nw + g.nb);
+                            for (int c = 0; c < CH; ++c) if (c < n_c) nx[c * g.next_ld] = __float2bfloat16_rn(g.next_value(x[c]));
+                        }
                     }
                 }
             };
@@ -330,7 +358,9 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
 template <int NT>
 int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmParams& p, int sms, cudaStream_t st) {
     CUtensorMap mx;
-    FORGE_TRY(make_map_2d(&mx, act, uint64_t(w.K), uint64_t(p.m), uint64_t(act_ld) * 2, NT));
+    int last_col = 0;
+    for (int i = 0; i < p.out.nseg; ++i) last_col = std::max(last_col, p.out.seg[i].act_col);
+    FORGE_TRY(make_map_2d(&mx, act, uint64_t(last_col + w.K), uint64_t(p.m), uint64_t(act_ld) * 2, NT));
     p.tt_count = (p.m + NT - 1) / NT;
     const long long tiles = (long long)((w.N + 127) / 128) * p.tt_count;
     const int grid = int(std::max(1LL, std::min((long long)sms, tiles * p.nk / 4)));
@@ -358,6 +388,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
     __shared__ float sw[KS][TN + 4], sx[KS][TM + 4];
     const int tid = threadIdx.x, rr = (tid & 15) * 4, tt = (tid >> 4) * PT;
     const int row0 = blockIdx.x * TN, tok0 = blockIdx.y * TM;
+    x += act_col(out, row0);
     float acc[4][PT];
 #pragma unroll
     for (int i = 0; i < 4; ++i)
@@ -401,11 +432,17 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
             const float v = acc[i][j];
             switch (g[i].kind) {
                 case SEG_CLAMPED_GLU: if (!(i & 1)) *dst = clamped_glu(v, acc[i | 1][j], g[i].limit); break;
-                case SEG_SIGMOID: *dst = sigmoid(v); break;
+                case SEG_SILU_GLU: if (!(i & 1)) *dst = silu(v) * acc[i | 1][j]; break;
+                case SEG_SIGMOID: case SEG_SIGMOID_F32: *dst = sigmoid(v); break;
+                case SEG_SILU: *dst = silu(v); break;
+                case SEG_TANH: *dst = tanhf(v); break;
+                case SEG_DECAY: *dst = -g[i].mul * softplus(v + g[i].add); break;
+                case SEG_EXP_DECAY: *dst = -expf(v + g[i].add); break;
+                case SEG_CAST: g[i].f32[size_t(g[i].place ? g[i].place[t] : int(t)) * g[i].ld] = v; break;
                 case SEG_RESID: {
-                    const float x = *dst + v;
+                    const float x = (g[i].fresh ? 0.f : *dst) + v + g[i].add;
                     *dst = x;
-                    if (g[i].next) g[i].next[t * g[i].next_ld] = tanhf(g[i].alpha * x) * g[i].nw + g[i].nb;
+                    if (g[i].after) g[i].next[t * g[i].next_ld] = g[i].next_value(x);
                     break;
                 }
                 default: *dst = v;
@@ -433,11 +470,15 @@ void dense_tile_image(void* dst, const void* rows, int N, int K) {
 int32_t dense_gemm(const DenseWeight& w, const void* act, int act_ld, int m, const DenseOut& out, const DenseScratch& sc, int* err, cudaStream_t st) {
     if (m <= 0) return FORGE_OK;
     if (w.K % kDensePad || act_ld < w.K || act_ld % kDensePad) { set_error("dense product: K=%d, activation rows of %d", w.K, act_ld); return FORGE_ERR_SHAPE; }
-    for (int i = 0; i < out.nseg; ++i)
-        if (out.seg[i].row0 % kSegAlign || out.seg[i].row0 + out.seg[i].rows > w.N || (out.seg[i].kind == SEG_CLAMPED_GLU && out.seg[i].rows % 2)) {
+    for (int i = 0; i < out.nseg; ++i) {
+        const OutSeg& g = out.seg[i];
+        const bool glu = g.kind == SEG_CLAMPED_GLU || g.kind == SEG_SILU_GLU, moved = g.act_col != (i ? out.seg[i - 1].act_col : 0);
+        if (g.row0 % kSegAlign || g.row0 + g.rows > w.N || (glu && g.rows % 2) || (i && g.row0 < out.seg[i - 1].row0 + out.seg[i - 1].rows) ||
+            g.act_col % kDensePad || g.act_col + w.K > act_ld || (i && moved && g.row0 % 128)) {
             set_error("dense product: bad output segment %d", i);
             return FORGE_ERR_SHAPE;
         }
+    }
     if (w.dtype == FORGE_F32) {
         const float* wf = static_cast<const float*>(w.w);
         const float* xf = static_cast<const float*>(act);

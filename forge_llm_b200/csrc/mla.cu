@@ -10,23 +10,7 @@ namespace forge {
 
 namespace {
 
-template <typename T> __device__ __forceinline__ T to_t(float v);
-template <> __device__ __forceinline__ float to_t<float>(float v) { return v; }
-template <> __device__ __forceinline__ __nv_bfloat16 to_t<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
-__device__ __forceinline__ float to_f(float v) { return v; }
-__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
-// eight consecutive values
-__device__ __forceinline__ void load8(float (&v)[8], const float* p) {
-    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-__device__ __forceinline__ void load8(float (&v)[8], const __nv_bfloat16* p) {
-    const uint4 u = *reinterpret_cast<const uint4*>(p);
-    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
-#pragma unroll
-    for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h[i]); v[2 * i] = f.x; v[2 * i + 1] = f.y; }
-}
 __device__ __forceinline__ float2 load2(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
 
 constexpr int kThreads = 256;
@@ -59,11 +43,6 @@ __device__ void append_row(const LatentDims& d, const float* down, const float* 
     const float inv = 1.0f / sqrtf(ss / float(d.rank) + d.eps);
     for (int i = threadIdx.x; i < d.rank_p; i += blockDim.x) dst[i] = to_t<T>(i < d.rank ? down[i] * inv * kv_norm[i] : 0.f);
     for (int i = threadIdx.x; i < d.rot_p; i += blockDim.x) dst[d.rank_p + i] = to_t<T>(i < d.rot ? rotated(down + d.rank, i, d.rot_dims, cs) : 0.f);
-}
-
-__device__ __forceinline__ size_t cache_row(const StepRows& rows, int r, int pos) {
-    const int seq = rows.seq ? rows.seq[r] : r;
-    return size_t(rows.page_table[size_t(seq) * rows.pages_per_seq + pos / FORGE_KV_PAGE]) * FORGE_KV_PAGE + pos % FORGE_KV_PAGE;
 }
 
 constexpr int kAbsorbCols = 128;   // latent columns per CTA

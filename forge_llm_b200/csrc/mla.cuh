@@ -15,14 +15,6 @@ struct LatentDims {
     __host__ __device__ int row() const { return rank_p + rot_p; }
 };
 
-// Rows of a step and where their sequence lives.  Row r belongs to sequence seq[r] (null: sequence r) at position pos[r].
-struct StepRows {
-    int n = 0;
-    const int32_t* pos = nullptr; const int32_t* seq = nullptr;   // device
-    const int32_t* page_table = nullptr; int pages_per_seq = 0;
-    int fresh = 1;                 // most rows one sequence has in this step
-};
-
 // proj: f32 rows [q | ... | dkv | ...] of ldp floats; q at column 0, W_dkv h at column dkv_col.
 // The latent is normed, the key part rotated, and both are appended to the cache; the queries are rotated and carried into
 // the latent space, qabs[row][head] = [W_uk^T q_unrotated | zeros | q_rotated | zeros] as T.
@@ -44,18 +36,8 @@ int32_t latent_decode_tc(const LatentDims& d, const void* qabs, const void* map,
 int32_t latent_value(const LatentDims& d, int dtype, const float* part, const float2* ml, int splits, const void* uv, int uv_ld, const void* gate, int gate_ld,
                      void* out, int out_ld, const StepRows& rows, cudaStream_t st);
 
-// ---- prompts (bfloat16): keys and values of the heads are formed once per prompt portion, then a tcgen05 flash attention
+// ---- prompts (bfloat16): keys and values of the heads are formed once per prompt portion, then a tcgen05 flash attention (attn_prompt.cuh)
 // c[r] = latents of context row r, krot[r] = its rotated key part (rows gathered through page list `pages`)
 int32_t latent_gather_context(const LatentDims& d, const void* cache, const int32_t* pages, int rows, void* c, void* krot, cudaStream_t st);
-struct PromptTile { int32_t row0, rows, pos0, ctx0; };   // query rows of the step, position of the first, first context row of its sequence
-struct PromptAttnArgs {
-    const void* q; const void* k; const void* krot; const void* v;   // [q_rows][heads][dim_p + rot_p], [ctx][heads][dim_p], [ctx][rot_p], [ctx][heads][vdim_p]
-    const void* gate; int gate_ld; void* out; int out_ld;            // out[row][head * vdim + i] = gate * attention
-    int q_rows, ctx_rows;
-    const PromptTile* tiles; int n_tiles;                             // device
-    int* err;
-};
-bool attn_prefill_kv_supported(const LatentDims& d);
-int32_t attn_prefill_kv(const LatentDims& d, const PromptAttnArgs& a, cudaStream_t st);
 
 }  // namespace forge

@@ -181,13 +181,25 @@ int32_t sync_and_check(ForgeModel* m, ForgeKV* kv) {
     FORGE_CUDA(cudaMemsetAsync(m->d_err, 0, sizeof(int), m->stream));
     if (kv) FORGE_TRY(upload_len(kv));
     FORGE_CUDA(cudaStreamSynchronize(m->stream));
+    if (kv) mark_lost(kv);
     set_error("a bounded device-side wait gave up: the step did not complete");
     return FORGE_ERR_TIMEOUT;
+}
+
+void mark_lost(ForgeKV* kv) {
+    if (!kv->model->stack || !stack_has_state(kv->model)) return;
+    for (int b = 0; b < kv->batch; ++b) if (kv->len[b] > 0) kv->lost[b] = 1;   // a sequence of length 0 starts from nothing
 }
 
 int32_t check_seq(const ForgeKV* kv, int seq) {
     if (!kv || seq < 0 || seq >= kv->batch) { set_error("sequence index out of range"); return FORGE_ERR_INVALID_ARG; }
     if (!kv->model) { set_error("the model of this cache has been destroyed"); return FORGE_ERR_INVALID_ARG; }
+    return FORGE_OK;
+}
+// may the sequence go on?
+static int32_t check_live(const ForgeKV* kv, int seq) {
+    FORGE_TRY(check_seq(kv, seq));
+    if (kv->lost[seq]) { set_error("a failed step has left the recurrent state of sequence %d undefined: free, reset or load it", seq); return FORGE_ERR_INVALID_ARG; }
     return FORGE_OK;
 }
 
@@ -913,6 +925,7 @@ int32_t forge_kv_create_pool(ForgeModel* m, int32_t pool_tokens, int32_t max_seq
     kv->h_page_table.assign(table, 0);
     kv->pages_used.assign(batch, 0);
     kv->len.assign(batch, 0);
+    kv->lost.assign(batch, 0);
     for (int i = kv->num_pages - 1; i >= 0; --i) kv->free_pages.push_back(i);
     // split-KV: enough CTAs to fill the SMs
     if (!m->stack) {
@@ -934,6 +947,7 @@ int32_t forge_kv_reset(ForgeKV* kv) {
     FORGE_CUDA(cudaSetDevice(kv->model->device));
     FORGE_CUDA(cudaStreamSynchronize(kv->model->stream));
     std::fill(kv->len.begin(), kv->len.end(), 0);
+    std::fill(kv->lost.begin(), kv->lost.end(), 0);
     std::fill(kv->pages_used.begin(), kv->pages_used.end(), 0);
     kv->free_pages.clear();
     for (int i = kv->num_pages - 1; i >= 0; --i) kv->free_pages.push_back(i);
@@ -947,6 +961,7 @@ int32_t forge_kv_free_seq(ForgeKV* kv, int32_t seq) {
     for (int i = 0; i < kv->pages_used[seq]; ++i) kv->free_pages.push_back(kv->h_page_table[size_t(seq) * kv->pages_per_seq + i]);
     kv->pages_used[seq] = 0;
     kv->len[seq] = 0;
+    kv->lost[seq] = 0;
     return upload_len(kv);
 }
 
@@ -995,6 +1010,21 @@ int32_t forge_kv_read(ForgeKV* kv, int32_t seq, int32_t layer, int32_t which, fl
                            cudaStreamSynchronize(m->stream) != cudaSuccess)) { set_error("kv read copy failed"); rc = FORGE_ERR_CUDA; }
     cudaFree(tmp);
     return rc;
+}
+
+int32_t forge_kv_width(const ForgeKV* kv, int32_t layer, int32_t which) {
+    if (!kv || !kv->model || layer < 0 || layer >= kv->model->cfg.num_layers) return -1;
+    return kv->model->stack ? stack_kv_width(kv, layer, which) : kv->model->kv;
+}
+int64_t forge_kv_state_values(const ForgeKV* kv, int32_t layer) {
+    if (!kv || !kv->model || layer < 0 || layer >= kv->model->cfg.num_layers) return -1;
+    return kv->model->stack ? int64_t(stack_state_values(kv, layer)) : 0;
+}
+int32_t forge_kv_state_read(ForgeKV* kv, int32_t seq, int32_t layer, float* out_host) {
+    FORGE_TRY(check_seq(kv, seq));
+    if (forge_kv_state_values(kv, layer) <= 0 || !out_host) { set_error("bad argument to forge_kv_state_read"); return FORGE_ERR_INVALID_ARG; }
+    FORGE_CUDA(cudaSetDevice(kv->model->device));
+    return stack_state_read(kv, seq, layer, out_host);
 }
 
 // ---- corpus scoring (--score-corpus, project.rs:652-712): per-token forward() over one chunk from an empty cache; the
@@ -1048,7 +1078,7 @@ int32_t kv_copy_rows(ForgeKV* kv, int seq, int layer, int which, int len, __half
 size_t forge_kv_save_size(const ForgeKV* kv, int32_t seq) {
     if (!kv || !kv->model || seq < 0 || seq >= kv->batch) return 0;
     const ForgeModel* m = kv->model;
-    if (m->stack) return sizeof(KvHeader) + stack_kv_bytes_per_token(kv) * kv->len[seq];
+    if (m->stack) return sizeof(KvHeader) + stack_kv_bytes_per_token(kv) * kv->len[seq] + stack_kv_bytes_per_seq(kv);
     return sizeof(KvHeader) + size_t(2) * m->cfg.num_layers * kv->len[seq] * m->kv * sizeof(__half);
 }
 
@@ -1060,7 +1090,7 @@ int32_t forge_kv_save(ForgeKV* kv, int32_t seq, void* out_host, size_t capacity)
     FORGE_CUDA(cudaSetDevice(m->device));
     const int len = kv->len[seq], L = m->cfg.num_layers;
     KvHeader h{};
-    if (m->stack) {   // the rows of every layer as they lie in the cache, width = bytes per position
+    if (m->stack) {   // of every layer run its rows as they lie in the cache (width = bytes per position, all runs) and its state
         memcpy(h.magic, kLatentMagic, 4); h.layers = uint32_t(L); h.width = uint32_t(stack_kv_bytes_per_token(kv)); h.len = uint64_t(len);
         memcpy(out_host, &h, sizeof(h));
         return stack_kv_copy(kv, seq, len, static_cast<char*>(out_host) + sizeof(h), true);
@@ -1090,7 +1120,7 @@ int32_t forge_kv_load(ForgeKV* kv, int32_t seq, const void* data_host, size_t n)
         if (n < sizeof(h)) { set_error("forge_kv_load: no data"); return FORGE_ERR_INVALID_ARG; }
         memcpy(&h, p, sizeof(h));
         if (memcmp(h.magic, kLatentMagic, 4) || h.layers != uint32_t(L) || h.width != uint32_t(stack_kv_bytes_per_token(kv))) { set_error("forge_kv_load: not a cache file of this model"); return FORGE_ERR_SHAPE; }
-        if (h.len > uint64_t(kv->max_seq) || n != sizeof(h) + size_t(h.width) * h.len) { set_error("forge_kv_load: bad length"); return FORGE_ERR_SHAPE; }
+        if (h.len > uint64_t(kv->max_seq) || n != sizeof(h) + size_t(h.width) * h.len + stack_kv_bytes_per_seq(kv)) { set_error("forge_kv_load: bad length"); return FORGE_ERR_SHAPE; }
         FORGE_TRY(forge_kv_free_seq(kv, seq));
         FORGE_TRY(ensure_pages(kv, seq, int(h.len)));
         FORGE_TRY(stack_kv_copy(kv, seq, int(h.len), reinterpret_cast<char*>(const_cast<uint8_t*>(p)) + sizeof(h), false));
@@ -1134,7 +1164,7 @@ int32_t forge_kv_load(ForgeKV* kv, int32_t seq, const void* data_host, size_t n)
 
 int32_t forge_forward_prefill_seq(ForgeModel* m, ForgeKV* kv, int32_t seq, const uint32_t* tokens, size_t n, float* logits_host) {
     if (!m || !tokens || n == 0 || n > (1u << 20)) { set_error("bad argument to forge_forward_prefill"); return FORGE_ERR_INVALID_ARG; }
-    FORGE_TRY(check_seq(kv, seq));
+    FORGE_TRY(check_live(kv, seq));
     if (kv->model != m) { set_error("kv belongs to another model"); return FORGE_ERR_INVALID_ARG; }
     FORGE_CUDA(cudaSetDevice(m->device));
     for (size_t i = 0; i < n; ++i) if (tokens[i] >= uint32_t(m->V)) { set_error("token id %u out of vocabulary", tokens[i]); return FORGE_ERR_INVALID_ARG; }
@@ -1161,7 +1191,7 @@ int32_t forge_forward_prefill(ForgeModel* m, ForgeKV* kv, const uint32_t* tokens
 // single sequence `seq` of a multi-sequence cache: runs the batch-1 launch sequence on views of that sequence
 int32_t forge_forward_seq(ForgeModel* m, ForgeKV* kv, int32_t seq, uint32_t token, float* logits_host) {
     if (!m) { set_error("null model"); return FORGE_ERR_INVALID_ARG; }
-    FORGE_TRY(check_seq(kv, seq));
+    FORGE_TRY(check_live(kv, seq));
     if (kv->model != m) { set_error("kv belongs to another model"); return FORGE_ERR_INVALID_ARG; }
     if (token >= uint32_t(m->V)) { set_error("token id %u out of vocabulary", token); return FORGE_ERR_INVALID_ARG; }
     FORGE_CUDA(cudaSetDevice(m->device));
@@ -1174,6 +1204,7 @@ int32_t forge_forward_seq(ForgeModel* m, ForgeKV* kv, int32_t seq, uint32_t toke
     ForgeKV view = *kv;
     view.d_page_table = kv->d_page_table + size_t(seq) * kv->pages_per_seq;
     view.d_seq_len = kv->d_seq_len + seq;
+    view.slot0 = seq;
     view.graph = nullptr;
     int32_t rc;
     if (seq == 0 && kv->batch >= 1 && !m->trace_on) {
@@ -1197,6 +1228,7 @@ int32_t forge_forward_batch(ForgeModel* m, ForgeKV* kv, int32_t batch, const uin
     FORGE_CUDA(cudaSetDevice(m->device));
     FORGE_TRY(ensure_decode_scratch(m, batch));
     if (m->stack) FORGE_TRY(stack_ensure_decode(m, kv, batch));
+    for (int b = 0; b < batch; ++b) FORGE_TRY(check_live(kv, b));
     FORGE_TRY(decode_prepare(kv, batch));
     if (m->trace_on) FORGE_TRY(ensure_trace(m, batch));
     FORGE_CUDA(cudaMemcpyAsync(m->d_tok, tokens, sizeof(uint32_t) * batch, cudaMemcpyHostToDevice, m->stream));
@@ -1214,7 +1246,7 @@ int32_t forge_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
     long long new_pages = 0;
     for (int i = 0; i < n_entries; ++i) {
         const ForgeStepEntry& e = entries[i];
-        FORGE_TRY(check_seq(kv, e.seq));
+        FORGE_TRY(check_live(kv, e.seq));
         if (seen[e.seq] || e.n_tokens <= 0 || e.n_tokens > (1 << 20) || e.n_want < 0 || (e.n_want && !want)) { set_error("forge_step: bad entry %d", i); return FORGE_ERR_INVALID_ARG; }
         seen[e.seq] = 1;
         for (int k = 0; k < e.n_tokens; ++k) if (tokens[n_tok + k] >= uint32_t(m->V)) { set_error("token id %u out of vocabulary", tokens[n_tok + k]); return FORGE_ERR_INVALID_ARG; }
@@ -1258,6 +1290,7 @@ int32_t forge_decode_greedy_batch(ForgeModel* m, ForgeKV* kv, int32_t batch, con
     if (!m || !kv || !first_tokens || !out_tokens || batch <= 0 || batch > kv->batch || n_new <= 0 || kv->model != m) { set_error("bad argument to forge_decode_greedy_batch"); return FORGE_ERR_INVALID_ARG; }
     FORGE_CUDA(cudaSetDevice(m->device));
     for (int b = 0; b < batch; ++b) {
+        FORGE_TRY(check_live(kv, b));
         if (first_tokens[b] >= uint32_t(m->V)) { set_error("token id out of vocabulary"); return FORGE_ERR_INVALID_ARG; }
         if (kv->len[b] + n_new > kv->max_seq) { set_error("KV cache full: %d + %d > max_seq %d", kv->len[b], n_new, kv->max_seq); return FORGE_ERR_KV_FULL; }
     }
@@ -1278,7 +1311,7 @@ int32_t forge_decode_greedy_batch(ForgeModel* m, ForgeKV* kv, int32_t batch, con
         if (rc == FORGE_OK) for (int b = 0; b < batch; ++b) kv->len[b] += 1;
     }
     m->trace_on = saved_trace;
-    if (rc != FORGE_OK) { cudaStreamSynchronize(m->stream); kv->len = len0; upload_len(kv); return rc; }
+    if (rc != FORGE_OK) { cudaStreamSynchronize(m->stream); kv->len = len0; mark_lost(kv); upload_len(kv); return rc; }
     FORGE_CUDA(cudaEventRecord(m->ev[2], m->stream));
     FORGE_CUDA(cudaMemcpyAsync(out_tokens, m->d_hist, sizeof(uint32_t) * size_t(n_new) * batch, cudaMemcpyDeviceToHost, m->stream));
     {

@@ -91,7 +91,9 @@ struct ForgeKV {
     int32_t* d_page_table = nullptr; int32_t* d_seq_len = nullptr;
     std::vector<int32_t> h_page_table; std::vector<int> free_pages; std::vector<int> pages_used; std::vector<int> len;
     float* attn_ws = nullptr; int* attn_counters = nullptr; int splits = 1;
-    StackCache* stack = nullptr;   // cache rows of a layer-list model (then k_pool and v_pool stay empty)
+    StackCache* stack = nullptr;   // cache rows and states of a layer-list model (then k_pool and v_pool stay empty)
+    int slot0 = 0;                 // of a view of single sequences: the first one's state slot
+    std::vector<char> lost;        // sequences whose recurrent state a failed step has left undefined
     alignas(64) unsigned char k_map[128], v_map[128];   // CUtensorMap of the two pools (all layers), for the decode attention's page copies
     cudaGraphExec_t graph = nullptr; int graph_batch = 0; bool graph_greedy = false; int graph_gen = -1;  // scratch generation the graph was captured with
     long long graph_kernels = 0;   // kernels of one replay
@@ -119,6 +121,8 @@ int32_t sync_and_check(ForgeModel* m, ForgeKV* kv);
 int32_t ensure_decode_scratch(ForgeModel* m, int batch);
 int32_t ensure_trace(ForgeModel* m, int rows);
 int32_t check_seq(const ForgeKV* kv, int seq);
+// a failed step of a model with recurrent state: the sequences that hold one must start over (or be loaded)
+void mark_lost(ForgeKV* kv);
 
 // ------------------------------------------------------------------ layer-list models (stack_model.cu)
 void stack_destroy(ForgeModel* m);
@@ -135,8 +139,13 @@ int32_t stack_prefill(ForgeModel* m, ForgeKV* kv, int seq, const uint32_t* token
 // decode step of `batch` sequences from device-side tokens and positions (captured into the cache's graph)
 int32_t stack_ensure_decode(ForgeModel* m, ForgeKV* kv, int batch);
 int32_t stack_decode_launches(ForgeModel* m, ForgeKV* kv, int batch, bool greedy, bool record);
-int32_t stack_kv_read(ForgeKV* kv, int seq, int layer, int which, float* out_host);
+bool stack_has_state(const ForgeModel* m);
+int stack_kv_width(const ForgeKV* kv, int run, int which);
+int32_t stack_kv_read(ForgeKV* kv, int seq, int run, int which, float* out_host);
+size_t stack_state_values(const ForgeKV* kv, int run);
+int32_t stack_state_read(ForgeKV* kv, int seq, int run, float* out_host);
 size_t stack_kv_bytes_per_token(const ForgeKV* kv);
+size_t stack_kv_bytes_per_seq(const ForgeKV* kv);
 int32_t stack_kv_copy(ForgeKV* kv, int seq, int len, char* host, bool to_host);
 
 }  // namespace forge

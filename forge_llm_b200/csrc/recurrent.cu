@@ -1,0 +1,444 @@
+// Recurrent mixers in f32 arithmetic: single tokens (decode), segments token by token, and the row operators around them.
+// T is the model's type (bfloat16 or float32); states, decays, step sizes, unit norms and sums are f32 in either.
+#include <cooperative_groups.h>
+
+#include <algorithm>
+
+#include "recurrent.cuh"
+
+namespace forge {
+
+namespace {
+
+namespace cg = cooperative_groups;
+
+constexpr int kConvTile = 32;     // tokens per warp; taps - 1 of them at most reach behind the segment
+
+// ------------------------------------------------------------------------------------------------ decode
+// One CTA = 32 value columns of one head of one row; the CTAs of a head form a cluster for the norm of its output.  A thread holds
+// the state of one column in the rows warp, warp + 8, ... of it; state, weights and what the convolution keeps are read before
+// the dependency wait.
+template <typename T, bool DELTA, bool CHANNEL, int RPT>
+__global__ void __launch_bounds__(256) recur_decode_kernel(const RecurDims d, const RecurArgs a, const StepRows rows) {
+    extern __shared__ float sm[];
+    float* sq = sm;                 // [dim] queries, keys, decays
+    float* sk = sq + d.dim;
+    float* sg = sk + d.dim;
+    float* sv = sg + d.dim;         // [32]
+    __shared__ float red[8][33], redo[8][33], wsum[8][3], part;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int split = blockIdx.x, splits = gridDim.x, h = blockIdx.y, r = blockIdx.z;
+    const int g = h / (d.heads / d.groups), c0 = split * 32, nc = min(32, d.vdim - c0);
+    pdl_trigger();
+    // positions are written in front of the step's first kernel, the state in the last step: both are complete
+    const int pos = rows.pos[r], slot = state_slot(rows, r);
+    float* S = a.state + (size_t(slot) * d.heads + h) * d.dim * d.vdim + c0 + lane;
+    float st[RPT];
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+        const int row = warp + 8 * i;
+        st[i] = pos > 0 && row < d.dim && lane < nc ? S[size_t(row) * d.vdim] : 0.f;
+    }
+    const int n_in = 2 * d.dim + nc;      // this CTA's channels: q, k, its values
+    auto channel = [&](int i) { return i < d.dim ? g * d.dim + i : i < 2 * d.dim ? d.qk() + g * d.dim + i - d.dim : 2 * d.qk() + h * d.vdim + c0 + i - 2 * d.dim; };
+    auto place = [&](int i) { return i < d.dim ? sq + i : i < 2 * d.dim ? sk + i - d.dim : sv + i - 2 * d.dim; };
+    if constexpr (DELTA) {
+        const T* ring = static_cast<const T*>(a.ring) + size_t(slot) * d.ring_values();
+        for (int i = tid; i < n_in; i += 256) {
+            const int ch = channel(i);
+            float v = 0.f;
+            for (int j = 0; j < d.taps - 1; ++j) {
+                const int p = pos - (d.taps - 1 - j);
+                if (p >= 0) v = fmaf(a.conv[size_t(ch) * d.taps + j], to_f(ring[size_t(p % d.taps) * d.channels() + ch]), v);
+            }
+            *place(i) = v;
+        }
+    }
+    pdl_wait();
+    const T* x = static_cast<const T*>(a.x) + size_t(r) * a.x_ld;
+    const float gate = lane < nc ? to_f(static_cast<const T*>(a.gate)[size_t(r) * a.gate_ld + h * d.vdim + c0 + lane]) : 0.f;
+    for (int i = tid; i < n_in; i += 256) {
+        const int ch = channel(i);
+        const T in = x[ch];
+        if constexpr (DELTA) {
+            const float v = fmaf(a.conv[size_t(ch) * d.taps + d.taps - 1], to_f(in), *place(i));
+            *place(i) = to_f(to_t<T>(silu(v)));
+            // one CTA keeps each input
+            if (i >= 2 * d.dim || (split == 0 && h % (d.heads / d.groups) == 0)) static_cast<T*>(a.ring)[size_t(slot) * d.ring_values() + size_t(pos % d.taps) * d.channels() + ch] = in;
+        } else *place(i) = to_f(in);
+    }
+    if constexpr (CHANNEL) {
+        for (int i = tid; i < d.dim; i += 256) sg[i] = expf(a.decay[size_t(r) * a.decay_ld + h * d.dim + i]);
+    }
+    const float g1 = CHANNEL ? 0.f : expf(a.decay[size_t(r) * a.decay_ld + h]);
+    const float beta = DELTA ? a.beta[size_t(r) * d.heads + h] : 0.f;
+    __syncthreads();
+    // sums over the head's channels: q q and k k, or q bonus k
+    {
+        float s0 = 0.f, s1 = 0.f;
+        for (int i = tid; i < d.dim; i += 256) {
+            if constexpr (DELTA) { s0 = fmaf(sq[i], sq[i], s0); s1 = fmaf(sk[i], sk[i], s1); }
+            else s0 = fmaf(sq[i] * a.bonus[h * d.dim + i], sk[i], s0);
+        }
+        s0 = warp_sum(s0);
+        if constexpr (DELTA) s1 = warp_sum(s1);
+        if (lane == 0) { wsum[warp][0] = s0; wsum[warp][1] = s1; }
+    }
+    __syncthreads();
+    float t0 = 0.f, t1 = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) { t0 += wsum[w][0]; t1 += wsum[w][1]; }
+    const float qs = DELTA ? d.q_scale / sqrtf(t0 + 1e-6f) : 1.f, ks = DELTA ? 1.0f / sqrtf(t1 + 1e-6f) : 1.f;
+    float o;
+    if constexpr (DELTA) {
+        float dot = 0.f;
+#pragma unroll
+        for (int i = 0; i < RPT; ++i) {
+            const int row = warp + 8 * i;
+            if (row < d.dim) {
+                st[i] *= CHANNEL ? sg[row] : g1;
+                dot = fmaf(st[i], sk[row] * ks, dot);
+            }
+        }
+        red[warp][lane] = dot;
+        __syncthreads();
+        dot = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) dot += red[w][lane];
+        const float u = lane < nc ? beta * (sv[lane] - dot) : 0.f;
+        o = 0.f;
+#pragma unroll
+        for (int i = 0; i < RPT; ++i) {
+            const int row = warp + 8 * i;
+            if (row < d.dim) {
+                st[i] = fmaf(sk[row] * ks, u, st[i]);
+                o = fmaf(st[i], sq[row] * qs, o);
+                if (lane < nc) S[size_t(row) * d.vdim] = st[i];
+            }
+        }
+    } else {
+        const float v = lane < nc ? sv[lane] : 0.f;
+        o = 0.f;
+#pragma unroll
+        for (int i = 0; i < RPT; ++i) {
+            const int row = warp + 8 * i;
+            if (row < d.dim) {
+                o = fmaf(st[i], sq[row], o);
+                st[i] = fmaf(sk[row], v, st[i] * (CHANNEL ? sg[row] : g1));
+                if (lane < nc) S[size_t(row) * d.vdim] = st[i];
+            }
+        }
+    }
+    redo[warp][lane] = o;
+    __syncthreads();
+    o = 0.f;
+    if (warp == 0) {
+#pragma unroll
+        for (int w = 0; w < 8; ++w) o += redo[w][lane];
+        if constexpr (!DELTA) o = fmaf(t0, lane < nc ? sv[lane] : 0.f, o);
+        const float ss = warp_sum(lane < nc ? o * o : 0.f);
+        if (lane == 0) part = ss;
+    }
+    float total;
+    if (splits > 1) {
+        cg::cluster_group cl = cg::this_cluster();
+        cl.sync();
+        total = 0.f;
+        if (warp == 0)
+            for (int s = 0; s < splits; ++s) total += *cl.map_shared_rank(&part, s);
+        cl.sync();   // nobody leaves while its part is read
+    } else {
+        __syncthreads();
+        total = part;
+    }
+    if (warp == 0 && lane < nc) {
+        const float inv = 1.0f / sqrtf(total / float(d.vdim) + d.eps);
+        static_cast<T*>(a.out)[size_t(r) * a.out_ld + h * d.vdim + c0 + lane] = to_t<T>(o * inv * a.norm[size_t(h) * a.norm_head + c0 + lane] * gate);
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ segments
+// Convolution, silu and the factors that make q and k unit vectors.  A warp = a tile of tokens of one unit (a head of q or k, or
+// up to 128 values).  The first tile's warp alone reads what the ring keeps of its channels and then leaves there the segment's
+// last inputs.
+template <typename T>
+__global__ void __launch_bounds__(256) conv_rows_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs) {
+    const ScanSeg s = segs[blockIdx.z];
+    const int t0 = blockIdx.x * kConvTile, lane = threadIdx.x & 31;
+    if (t0 >= s.n) return;
+    const int vblocks = (d.heads * d.vdim + 127) / 128, unit = blockIdx.y * 8 + (threadIdx.x >> 5);
+    if (unit >= 2 * d.groups + vblocks) return;
+    const bool is_v = unit >= 2 * d.groups;
+    const int ch0 = is_v ? 2 * d.qk() + (unit - 2 * d.groups) * 128 : unit * d.dim;
+    const int nch = is_v ? min(128, d.channels() - ch0) : d.dim;
+    const T* x = static_cast<const T*>(a.x) + size_t(s.row0) * a.x_ld;
+    T* y = static_cast<T*>(sc.conv) + size_t(s.row0) * d.channels();
+    T* ring = static_cast<T*>(a.ring) + size_t(s.slot) * d.ring_values();
+    for (int t = t0; t < min(s.n, t0 + kConvTile); ++t) {
+        float sum = 0.f;
+        for (int c = lane; c < nch; c += 32) {
+            const int ch = ch0 + c;
+            float v = 0.f;
+            for (int j = 0; j < d.taps; ++j) {
+                const int q = t - (d.taps - 1 - j), p = s.pos0 + q;
+                float in = 0.f;
+                if (q >= 0) in = to_f(x[size_t(q) * a.x_ld + ch]);
+                else if (p >= 0) in = to_f(ring[size_t(p % d.taps) * d.channels() + ch]);
+                v = fmaf(a.conv[size_t(ch) * d.taps + j], in, v);
+            }
+            const T o = to_t<T>(silu(v));
+            y[size_t(t) * d.channels() + ch] = o;
+            sum = fmaf(to_f(o), to_f(o), sum);
+        }
+        if (!is_v) {
+            sum = warp_sum(sum);
+            if (lane == 0) sc.unit[size_t(s.row0 + t) * 2 * d.groups + unit] = (unit < d.groups ? d.q_scale : 1.f) / sqrtf(sum + 1e-6f);
+        }
+    }
+    if (blockIdx.x == 0)
+        for (int c = lane; c < nch; c += 32)
+            for (int t = max(0, s.n - d.taps); t < s.n; ++t) ring[size_t((s.pos0 + t) % d.taps) * d.channels() + ch0 + c] = x[size_t(t) * a.x_ld + ch0 + c];
+}
+
+// Token by token: a warp carries four value columns of one head, its lanes share the rows of the state.
+template <typename T, bool DELTA, bool CHANNEL, int RPL>
+__global__ void __launch_bounds__(128) scan_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs) {
+    const ScanSeg s = segs[blockIdx.z];
+    const int lane = threadIdx.x & 31, h = blockIdx.y, c0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * 4;
+    if (c0 >= d.vdim) return;
+    const int nc = min(4, d.vdim - c0), g = h / (d.heads / d.groups);
+    float* S = a.state + (size_t(s.slot) * d.heads + h) * d.dim * d.vdim + c0;
+    const T* x = DELTA ? static_cast<const T*>(sc.conv) + size_t(s.row0) * d.channels() : static_cast<const T*>(a.x) + size_t(s.row0) * a.x_ld;
+    const size_t ld = DELTA ? d.channels() : a.x_ld;
+    float st[RPL][4], bonus[RPL];
+#pragma unroll
+    for (int i = 0; i < RPL; ++i) {
+        const int row = lane + 32 * i;
+        bonus[i] = !DELTA && row < d.dim ? a.bonus[h * d.dim + row] : 0.f;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) st[i][c] = s.pos0 > 0 && row < d.dim && c < nc ? S[size_t(row) * d.vdim + c] : 0.f;
+    }
+    struct In { T q[RPL], k[RPL], v[4]; float g[CHANNEL ? RPL : 1], beta, qs, ks; };
+    auto load = [&](int t, In& in) {
+        const T* xr = x + size_t(t) * ld;
+#pragma unroll
+        for (int i = 0; i < RPL; ++i) {
+            const int row = lane + 32 * i;
+            const bool ok = row < d.dim;
+            in.q[i] = ok ? xr[g * d.dim + row] : to_t<T>(0.f);
+            in.k[i] = ok ? xr[d.qk() + g * d.dim + row] : to_t<T>(0.f);
+            if (CHANNEL) in.g[i] = ok ? a.decay[size_t(s.row0 + t) * a.decay_ld + h * d.dim + row] : 0.f;
+        }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) in.v[c] = c < nc ? xr[2 * d.qk() + h * d.vdim + c0 + c] : to_t<T>(0.f);
+        if (!CHANNEL) in.g[0] = a.decay[size_t(s.row0 + t) * a.decay_ld + h];
+        if (DELTA) {
+            in.beta = a.beta[size_t(s.row0 + t) * d.heads + h];
+            in.qs = sc.unit[size_t(s.row0 + t) * 2 * d.groups + g];
+            in.ks = sc.unit[size_t(s.row0 + t) * 2 * d.groups + d.groups + g];
+        }
+    };
+    In in, next;
+    load(0, in);
+    for (int t = 0; t < s.n; ++t) {
+        load(min(t + 1, s.n - 1), next);
+        float o[4] = {0.f, 0.f, 0.f, 0.f};
+        if constexpr (DELTA) {
+            float dot[4] = {0.f, 0.f, 0.f, 0.f};
+            const float g1 = CHANNEL ? 0.f : expf(in.g[0]);
+#pragma unroll
+            for (int i = 0; i < RPL; ++i) {
+                const float w = CHANNEL ? expf(in.g[CHANNEL ? i : 0]) : g1, k = to_f(in.k[i]) * in.ks;
+#pragma unroll
+                for (int c = 0; c < 4; ++c) { st[i][c] *= w; dot[c] = fmaf(st[i][c], k, dot[c]); }
+            }
+#pragma unroll
+            for (int c = 0; c < 4; ++c) dot[c] = in.beta * (to_f(in.v[c]) - warp_sum(dot[c]));
+#pragma unroll
+            for (int i = 0; i < RPL; ++i) {
+                const float k = to_f(in.k[i]) * in.ks, q = to_f(in.q[i]) * in.qs;
+#pragma unroll
+                for (int c = 0; c < 4; ++c) { st[i][c] = fmaf(k, dot[c], st[i][c]); o[c] = fmaf(st[i][c], q, o[c]); }
+            }
+        } else {
+            float own = 0.f;
+            const float g1 = CHANNEL ? 0.f : expf(in.g[0]);
+#pragma unroll
+            for (int i = 0; i < RPL; ++i) {
+                const float w = CHANNEL ? expf(in.g[CHANNEL ? i : 0]) : g1, k = to_f(in.k[i]), q = to_f(in.q[i]);
+                own = fmaf(q * bonus[i], k, own);
+#pragma unroll
+                for (int c = 0; c < 4; ++c) { o[c] = fmaf(st[i][c], q, o[c]); st[i][c] = fmaf(k, to_f(in.v[c]), st[i][c] * w); }
+            }
+#pragma unroll
+            for (int c = 0; c < 4; ++c) o[c] = fmaf(own, to_f(in.v[c]), o[c]);
+        }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            o[c] = warp_sum(o[c]);
+            if (lane == c && c < nc) sc.o[(size_t(s.row0 + t) * d.heads + h) * d.vdim + c0 + c] = o[c];
+        }
+        in = next;
+    }
+#pragma unroll
+    for (int i = 0; i < RPL; ++i) {
+        const int row = lane + 32 * i;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) if (row < d.dim && c < nc) S[size_t(row) * d.vdim + c] = st[i][c];
+    }
+}
+
+// out = rms norm(o) * norm * gate per head; a warp per (row, head)
+template <typename T>
+__global__ void __launch_bounds__(256) head_norm_kernel(const RecurDims d, const RecurArgs a, const float* __restrict__ o, int row0, int rows) {
+    const int i = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (i >= rows * d.heads) return;
+    const int r = row0 + i / d.heads, h = i % d.heads;
+    const float* src = o + (size_t(r) * d.heads + h) * d.vdim;
+    float ss = 0.f;
+    for (int c = lane; c < d.vdim; c += 32) ss = fmaf(src[c], src[c], ss);
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / float(d.vdim) + d.eps);
+    const T* gate = static_cast<const T*>(a.gate) + size_t(r) * a.gate_ld + h * d.vdim;
+    T* out = static_cast<T*>(a.out) + size_t(r) * a.out_ld + h * d.vdim;
+    for (int c = lane; c < d.vdim; c += 32) out[c] = to_t<T>(src[c] * inv * a.norm[size_t(h) * a.norm_head + c] * to_f(gate[c]));
+}
+
+// ------------------------------------------------------------------------------------------------ token shift
+// One CTA = 256 columns of one row (single rows) or of up to kShiftRows rows of a segment; the thread that reads what is kept of the row
+// before a segment is the one that leaves the segment's last row there.
+constexpr int kShiftRows = 16;
+template <typename T>
+__global__ void __launch_bounds__(256) token_shift_kernel(T* __restrict__ dst, int ld, int width, int width_p, int n_mix, const float* __restrict__ mu, T* __restrict__ prev, const StepRows rows,
+                                                          const ScanSeg* __restrict__ segs) {
+    const int c = blockIdx.y * 256 + threadIdx.x;
+    ScanSeg s;
+    if (segs) s = segs[blockIdx.z];
+    else s = ScanSeg{int(blockIdx.x), 1, state_slot(rows, blockIdx.x), rows.pos[blockIdx.x]};
+    const int t0 = segs ? blockIdx.x * kShiftRows : 0;
+    pdl_trigger();
+    pdl_wait();
+    if (c >= width || t0 >= s.n) return;
+    T* at = dst + size_t(s.row0) * ld + c;
+    T* keep = prev + size_t(s.slot) * width + c;
+    float before = t0 > 0 ? to_f(at[size_t(t0 - 1) * ld]) : s.pos0 > 0 ? to_f(*keep) : 0.f;
+    if (t0 == 0) *keep = at[size_t(s.n - 1) * ld];
+    float m[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) m[i] = i < n_mix ? mu[size_t(i) * width + c] : 0.f;
+    for (int t = t0; t < min(s.n, t0 + kShiftRows); ++t) {
+        const float h = to_f(at[size_t(t) * ld]);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) if (i < n_mix) at[size_t(t) * ld + size_t(i + 1) * width_p] = to_t<T>(fmaf(before - h, m[i], h));
+        before = h;
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ sum of two normed rows
+template <typename T>
+__global__ void __launch_bounds__(256) add_normed_pair_kernel(float* __restrict__ x, const float* __restrict__ ab, int width, float eps, const float* __restrict__ wa, const float* __restrict__ wb, const After after) {
+    __shared__ float red[8][2];
+    const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    pdl_trigger();
+    pdl_wait();
+    const float* a = ab + size_t(r) * 2 * width;
+    const float* b = a + width;
+    float sa = 0.f, sb = 0.f;
+    for (int i = threadIdx.x; i < width; i += 256) { sa = fmaf(a[i], a[i], sa); sb = fmaf(b[i], b[i], sb); }
+    sa = warp_sum(sa); sb = warp_sum(sb);
+    if (lane == 0) { red[warp][0] = sa; red[warp][1] = sb; }
+    __syncthreads();
+    sa = sb = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) { sa += red[w][0]; sb += red[w][1]; }
+    const float ia = 0.5f / sqrtf(sa / float(width) + eps), ib = 0.5f / sqrtf(sb / float(width) + eps);
+    for (int i = threadIdx.x; i < width; i += 256) {
+        const float v = x[size_t(r) * width + i] + a[i] * ia * wa[i] + b[i] * ib * wb[i];
+        x[size_t(r) * width + i] = v;
+        if (after.kind != AFTER_NONE)
+            static_cast<T*>(after.dst)[size_t(r) * after.ld + i] = to_t<T>(after.kind == AFTER_DYT ? dynamic_tanh(v, after.alpha, after.w[i], after.b[i]) : v);
+    }
+}
+
+template <typename T, bool DELTA, bool CHANNEL, int RPT>
+int32_t launch_decode(const RecurDims& d, const RecurArgs& a, const StepRows& rows, cudaStream_t st) {
+    const int splits = (d.vdim + 31) / 32;
+    FORGE_CUDA(launch_pdl_cluster(recur_decode_kernel<T, DELTA, CHANNEL, RPT>, dim3(splits, d.heads, rows.n), dim3(256), splits, sizeof(float) * (3 * size_t(d.dim) + 32), st, d, a, rows));
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+template <typename T, bool DELTA, bool CHANNEL>
+int32_t decode_t(const RecurDims& d, const RecurArgs& a, const StepRows& rows, cudaStream_t st) {
+    if (d.dim <= 64) return launch_decode<T, DELTA, CHANNEL, 8>(d, a, rows, st);
+    if (d.dim <= 128) return launch_decode<T, DELTA, CHANNEL, 16>(d, a, rows, st);
+    return launch_decode<T, DELTA, CHANNEL, 32>(d, a, rows, st);
+}
+template <typename T, bool DELTA, bool CHANNEL>
+int32_t scan_t(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, const ScanSeg* segs, int n_segs, cudaStream_t st) {
+    const dim3 grid((d.vdim + 15) / 16, d.heads, n_segs);
+    if (d.dim <= 32) scan_kernel<T, DELTA, CHANNEL, 1><<<grid, 128, 0, st>>>(d, a, sc, segs);
+    else if (d.dim <= 64) scan_kernel<T, DELTA, CHANNEL, 2><<<grid, 128, 0, st>>>(d, a, sc, segs);
+    else if (d.dim <= 128) scan_kernel<T, DELTA, CHANNEL, 4><<<grid, 128, 0, st>>>(d, a, sc, segs);
+    else scan_kernel<T, DELTA, CHANNEL, 8><<<grid, 128, 0, st>>>(d, a, sc, segs);
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+template <typename T>
+int32_t segments_t(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, const ScanSeg* segs, int n_segs, int max_n, int row0, int rows, cudaStream_t st) {
+    if (d.delta) {
+        const int units = 2 * d.groups + (d.heads * d.vdim + 127) / 128;
+        conv_rows_kernel<T><<<dim3((max_n + kConvTile - 1) / kConvTile, (units + 7) / 8, n_segs), 256, 0, st>>>(d, a, sc, segs);
+        FORGE_LAUNCH_CHECK();
+        FORGE_TRY(d.channel ? (scan_t<T, true, true>(d, a, sc, segs, n_segs, st)) : (scan_t<T, true, false>(d, a, sc, segs, n_segs, st)));
+    } else FORGE_TRY((scan_t<T, false, true>(d, a, sc, segs, n_segs, st)));
+    head_norm_kernel<T><<<(rows * d.heads + 7) / 8, 256, 0, st>>>(d, a, sc.o, row0, rows);
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+
+}  // namespace
+
+bool recur_supported(const RecurDims& d) { return d.dim <= 256 && d.vdim <= 256 && d.taps <= kConvTile && (d.delta ? d.taps >= 1 : d.channel && d.taps == 0); }
+
+int32_t recur_decode(const RecurDims& d, int dtype, const RecurArgs& a, const StepRows& rows, cudaStream_t st) {
+    if (rows.n <= 0) return FORGE_OK;
+    auto go = [&](auto t) -> int32_t {
+        using T = decltype(t);
+        if (!d.delta) return decode_t<T, false, true>(d, a, rows, st);
+        return d.channel ? decode_t<T, true, true>(d, a, rows, st) : decode_t<T, true, false>(d, a, rows, st);
+    };
+    return dtype == FORGE_F32 ? go(float{}) : go(__nv_bfloat16{});
+}
+
+int32_t recur_segments(const RecurDims& d, int dtype, const RecurArgs& a, const RecurScratch& sc, const ScanSeg* segs, int n_segs, int max_n, int row0, int rows, cudaStream_t st) {
+    if (n_segs <= 0) return FORGE_OK;
+    return dtype == FORGE_F32 ? segments_t<float>(d, a, sc, segs, n_segs, max_n, row0, rows, st) : segments_t<__nv_bfloat16>(d, a, sc, segs, n_segs, max_n, row0, rows, st);
+}
+
+int32_t token_shift(void* dst, int ld, int width, int width_p, int n_mix, const float* mu, void* prev, int dtype, const StepRows& rows, int n_single, const ScanSeg* segs, int n_segs, int max_n,
+                    cudaStream_t st) {
+    if (n_mix > 8) { set_error("token shift: %d mixes", n_mix); return FORGE_ERR_SHAPE; }
+    auto go = [&](auto t) -> int32_t {
+        using T = decltype(t);
+        const int cols = (width + 255) / 256;
+        if (n_single > 0) {
+            FORGE_CUDA(launch_pdl(token_shift_kernel<T>, dim3(n_single, cols), dim3(256), 0, st, static_cast<T*>(dst), ld, width, width_p, n_mix, mu, static_cast<T*>(prev), rows, static_cast<const ScanSeg*>(nullptr)));
+            FORGE_LAUNCH_CHECK();
+        }
+        if (n_segs > 0) {
+            FORGE_CUDA(launch_pdl(token_shift_kernel<T>, dim3((max_n + kShiftRows - 1) / kShiftRows, cols, n_segs), dim3(256), 0, st, static_cast<T*>(dst), ld, width, width_p, n_mix, mu, static_cast<T*>(prev), rows, segs));
+            FORGE_LAUNCH_CHECK();
+        }
+        return FORGE_OK;
+    };
+    return dtype == FORGE_F32 ? go(float{}) : go(__nv_bfloat16{});
+}
+
+int32_t add_normed_pair(float* x, const float* ab, int rows, int width, float eps, const float* wa, const float* wb, const After& after, int dtype, cudaStream_t st) {
+    if (rows <= 0) return FORGE_OK;
+    if (dtype == FORGE_F32) FORGE_CUDA(launch_pdl(add_normed_pair_kernel<float>, dim3(rows), dim3(256), 0, st, x, ab, width, eps, wa, wb, after));
+    else FORGE_CUDA(launch_pdl(add_normed_pair_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, st, x, ab, width, eps, wa, wb, after));
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+
+}  // namespace forge

@@ -1,0 +1,62 @@
+// Recurrent mixers: per head a state S [dim][vdim] in f32 that every token decays, extends and reads.
+//   delta rule     S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+//   time mixing    o = S^T q + (sum_c q_c bonus_c k_c) v;  S <- diag(g) S + k v^T
+// g is one decay per head or one per head and key channel, given by its logarithm.  The delta rule's q, k, v come from a short
+// causal convolution per channel with silu behind it, q and k as unit vectors; its last inputs are kept in a ring of `taps` rows,
+// the input of position p in row p % taps.  A sequence's state counts as zero when its first row of a step is at position 0, so
+// a slot that is used again needs no clearing.
+#pragma once
+
+#include "dense.cuh"
+
+namespace forge {
+
+struct RecurDims {
+    int heads = 0, groups = 0, dim = 0, vdim = 0;   // groups: heads of q and k (head h uses h / (heads / groups))
+    int taps = 0;                                   // 0: no convolution
+    bool delta = false, channel = false;            // channel: a decay per key channel
+    float eps = 0.f, q_scale = 1.f;
+    __host__ __device__ int qk() const { return groups * dim; }
+    __host__ __device__ int channels() const { return 2 * groups * dim + heads * vdim; }
+    size_t state_values() const { return size_t(heads) * dim * vdim; }
+    __host__ __device__ size_t ring_values() const { return size_t(taps) * channels(); }
+};
+
+// consecutive rows of one sequence: rows [row0, row0 + n) of the step at positions pos0, pos0 + 1, ... of state slot `slot`
+struct ScanSeg { int32_t row0, n, slot, pos0; };
+
+struct RecurArgs {
+    const void* x = nullptr; int x_ld = 0;               // T rows [q | k | v]: in front of the convolution, if there is one
+    const float* decay = nullptr; int decay_ld = 0;      // logarithms, [row][heads] or [row][heads * dim]
+    const float* beta = nullptr;                         // [row][heads]
+    const float* bonus = nullptr;                        // [heads][dim]
+    const float* conv = nullptr; void* ring = nullptr;   // [channels][taps]; T [slot][taps][channels]
+    float* state = nullptr;                              // [slot][heads][dim][vdim]
+    const float* norm = nullptr; int norm_head = 0;      // weight of the output's norm, and its step per head
+    const void* gate = nullptr; int gate_ld = 0;         // T rows [heads * vdim]
+    void* out = nullptr; int out_ld = 0;                 // T rows [heads * vdim]: rms norm(o) * norm * gate
+};
+
+// scratch of a step with segments
+struct RecurScratch {
+    void* conv = nullptr;         // T [rows][channels]: behind convolution and silu
+    float* unit = nullptr;        // [rows][2 * groups]: what q and k are multiplied with to be unit vectors (q: times q_scale)
+    float* o = nullptr;           // [rows][heads * vdim]
+};
+
+bool recur_supported(const RecurDims& d);
+// single tokens: row r of `rows` is one token of its sequence
+int32_t recur_decode(const RecurDims& d, int dtype, const RecurArgs& a, const StepRows& rows, cudaStream_t st);
+// segments (device table, at most max_n tokens each) that make up the rows [row0, row0 + rows) of the step
+int32_t recur_segments(const RecurDims& d, int dtype, const RecurArgs& a, const RecurScratch& sc, const ScanSeg* segs, int n_segs, int max_n, int row0, int rows, cudaStream_t st);
+
+// Token shift: dst rows get, next to h in columns [0, width_p), `n_mix` blocks of width_p columns h + (h' - h) mu[i], h' being the
+// sequence's row before (prev [slot][width], zeros at position 0).  h lies in dst's first block already.  prev is left at the
+// sequence's last row.
+int32_t token_shift(void* dst, int ld, int width, int width_p, int n_mix, const float* mu, void* prev, int dtype, const StepRows& rows, int n_single, const ScanSeg* segs, int n_segs, int max_n,
+                    cudaStream_t st);
+
+// x += (rms norm(a) wa + rms norm(b) wb) / 2 over rows of `width` values, then `after`; ab: f32 rows [a | b]
+int32_t add_normed_pair(float* x, const float* ab, int rows, int width, float eps, const float* wa, const float* wb, const After& after, int dtype, cudaStream_t st);
+
+}  // namespace forge

@@ -1,0 +1,321 @@
+// Registry of architectures and the reader of a layer-list model's configuration and tensor names (host code).
+#include <cmath>
+#include <cstdio>
+#include <cstring>
+
+#include "stack.cuh"
+
+namespace forge {
+
+static const Architecture kArchitectures[] = {
+    {"Bolenex", Norm::DynamicTanh, Arrangement::Parallel, Mlp::ClampedGlu},
+    {"Robazen", Norm::DynamicTanh, Arrangement::Sequential, Mlp::SiluGlu},
+};
+static const struct { const char* name; Mixer kind; } kMixers[] = {
+    {"latent_attention", Mixer::Latent}, {"delta", Mixer::Delta}, {"channel_delta", Mixer::ChannelDelta}, {"parallel", Mixer::AttnTimeMix},
+};
+
+namespace {
+
+int32_t need_int(const Json* o, const char* key, int* out, int lo = 1) {
+    const Json* v = o ? o->get(key) : nullptr;
+    if (!v || v->kind != Json::Number || v->num != std::floor(v->num) || v->num < lo || v->num > 1e9) { set_error("config.json: \"%s\" must be an integer of at least %d", key, lo); return FORGE_ERR_SHAPE; }
+    *out = int(v->num);
+    return FORGE_OK;
+}
+int32_t need_num(const Json* o, const char* key, double* out) {
+    const Json* v = o ? o->get(key) : nullptr;
+    if (!v || v->kind != Json::Number) { set_error("config.json: \"%s\" must be a number", key); return FORGE_ERR_SHAPE; }
+    *out = v->num;
+    return FORGE_OK;
+}
+int32_t need_string(const Json* o, const char* key, std::string* out) {
+    const Json* v = o ? o->get(key) : nullptr;
+    if (!v || v->kind != Json::String) { set_error("config.json: \"%s\" must be a string", key); return FORGE_ERR_SHAPE; }
+    *out = v->str;
+    return FORGE_OK;
+}
+
+int32_t parse_latent(const Json* m, float eps, LayerSpec* L) {
+    LatentDims& d = L->mix;
+    double scale;
+    FORGE_TRY(need_int(m, "heads", &d.heads));
+    FORGE_TRY(need_int(m, "dim", &d.dim));
+    FORGE_TRY(need_int(m, "rot_dim", &d.rot, 0));
+    FORGE_TRY(need_int(m, "vdim", &d.vdim));
+    FORGE_TRY(need_int(m, "kv_rank", &d.rank));
+    FORGE_TRY(need_num(m, "scale", &scale));
+    if (d.rot > 0) {
+        const Json* rot = m->get("rot");
+        FORGE_TRY(need_int(rot, "dims", &d.rot_dims, 0));
+        FORGE_TRY(need_num(rot, "base", &L->rot_base));
+        if (d.rot_dims > d.rot || d.rot_dims % 2 || !(L->rot_base > 0)) { set_error("config.json: rot.dims %d does not fit rot_dim %d", d.rot_dims, d.rot); return FORGE_ERR_SHAPE; }
+    }
+    d.scale = float(scale); d.eps = eps;
+    d.rank_p = pad_to(d.rank, 64); d.rot_p = pad_to(d.rot, 64); d.dim_p = pad_to(d.dim, 64); d.vdim_p = pad_to(d.vdim, 64);
+    return FORGE_OK;
+}
+
+int32_t heads_fit(int heads, int groups) {
+    if (heads % groups) { set_error("config.json: %d heads do not share %d kv_heads evenly", heads, groups); return FORGE_ERR_SHAPE; }
+    return FORGE_OK;
+}
+
+int32_t check_recur(const RecurDims& d) {
+    if (recur_supported(d)) return FORGE_OK;
+    set_error("recurrent mixer: head sizes %d / %d with %d taps are not supported", d.dim, d.vdim, d.taps);
+    return FORGE_ERR_UNSUPPORTED;
+}
+
+int32_t parse_delta(const Json* m, float eps, bool channel, LayerSpec* L) {
+    RecurDims& d = L->rec;
+    FORGE_TRY(need_int(m, "heads", &d.heads));
+    FORGE_TRY(need_int(m, "kv_heads", &d.groups));
+    FORGE_TRY(need_int(m, "dim", &d.dim));
+    FORGE_TRY(need_int(m, "vdim", &d.vdim));
+    FORGE_TRY(need_int(m, "conv", &d.taps));
+    FORGE_TRY(heads_fit(d.heads, d.groups));
+    d.delta = true; d.channel = channel; d.eps = eps;
+    d.q_scale = float(1.0 / std::sqrt(double(d.dim)));
+    return check_recur(d);
+}
+
+int32_t parse_attn(const Json* m, AttnDims* d) {
+    double scale, cap = 0;
+    FORGE_TRY(need_int(m, "heads", &d->heads));
+    FORGE_TRY(need_int(m, "kv_heads", &d->groups));
+    FORGE_TRY(need_int(m, "dim", &d->dim));
+    FORGE_TRY(need_int(m, "vdim", &d->vdim));
+    FORGE_TRY(need_num(m, "scale", &scale));
+    const Json* c = m->get("softcap");
+    if (c && c->kind != Json::Null) {
+        FORGE_TRY(need_num(m, "softcap", &cap));
+        if (!(cap > 0)) { set_error("config.json: \"softcap\" must be positive"); return FORGE_ERR_SHAPE; }
+    }
+    const Json* mask = m->get("mask");
+    if (mask && mask->kind != Json::Null) FORGE_TRY(need_int(mask, "size", &d->chunk));
+    FORGE_TRY(heads_fit(d->heads, d->groups));
+    d->scale = float(scale); d->softcap = float(cap);
+    d->dim_p = pad_to(d->dim, 64); d->vdim_p = pad_to(d->vdim, 64);
+    if (attn_rows_supported(*d)) return FORGE_OK;
+    set_error("attention: head sizes %d / %d are not supported", d->dim, d->vdim);
+    return FORGE_ERR_UNSUPPORTED;
+}
+
+int32_t parse_pair(const Json* m, float eps, LayerSpec* L) {
+    const Json* left = m ? m->get("left") : nullptr;
+    const Json* right = m ? m->get("right") : nullptr;
+    FORGE_TRY(parse_attn(left ? left : m, &L->attn));
+    RecurDims& d = L->rec;
+    FORGE_TRY(need_int(right, "heads", &d.heads));
+    FORGE_TRY(need_int(right, "dim", &d.dim));
+    d.groups = d.heads; d.vdim = d.dim; d.channel = true; d.eps = eps;
+    return check_recur(d);
+}
+
+bool same_sizes(const LayerSpec& A, const LayerSpec& B) {
+    const LatentDims &a = A.mix, &b = B.mix;
+    return A.kind == Mixer::Latent && B.kind == Mixer::Latent && a.heads == b.heads && a.dim == b.dim && a.rot == b.rot && a.vdim == b.vdim && a.rank == b.rank && A.ff == B.ff;
+}
+
+}  // namespace
+
+int32_t stack_parse(const Json& c, StackSpec* s) {
+    std::string name;
+    FORGE_TRY(need_string(&c, "architecture", &name));
+    for (const Architecture& a : kArchitectures) if (name == a.name) s->arch = &a;
+    if (!s->arch) { set_error("architecture \"%s\" is not registered", name.c_str()); return FORGE_ERR_UNSUPPORTED; }
+    FORGE_TRY(need_int(&c, "width", &s->width));
+    FORGE_TRY(need_int(&c, "vocab", &s->vocab));
+    double eps;
+    FORGE_TRY(need_num(c.get("norm"), "eps", &eps));
+    s->eps = float(eps);
+    const Json* layers = c.get("layers");
+    if (!layers || layers->kind != Json::Array || layers->items.empty()) { set_error("config.json: \"layers\" must list at least one layer"); return FORGE_ERR_SHAPE; }
+    const int n = int(layers->items.size());
+    for (int i = 0; i < n; ++i) {
+        const Json& e = layers->items[i];
+        LayerSpec L;
+        std::string type;
+        FORGE_TRY(need_string(&e, "type", &type));
+        bool known = false;
+        for (const auto& m : kMixers) if (type == m.name) { L.kind = m.kind; known = true; }
+        if (!known || (s->arch->arrangement == Arrangement::Parallel && L.kind != Mixer::Latent)) { set_error("layer %d: mixer \"%s\" is not supported", i, type.c_str()); return FORGE_ERR_UNSUPPORTED; }
+        const Json* mx = e.get("mixer");
+        if (!mx || mx->kind != Json::Object) { set_error("layer %d: \"mixer\" must be an object", i); return FORGE_ERR_SHAPE; }
+        switch (L.kind) {
+            case Mixer::Latent: FORGE_TRY(parse_latent(mx, s->eps, &L)); break;
+            case Mixer::Delta: FORGE_TRY(parse_delta(mx, s->eps, false, &L)); break;
+            case Mixer::ChannelDelta: FORGE_TRY(parse_delta(mx, s->eps, true, &L)); break;
+            case Mixer::AttnTimeMix: FORGE_TRY(parse_pair(mx, s->eps, &L)); break;
+        }
+        const Json* mlp = e.get("mlp");
+        if (mlp && mlp->kind != Json::Null) {
+            std::string kind;
+            FORGE_TRY(need_string(mlp, "kind", &kind));
+            if (kind != "dense") { set_error("layer %d: feed-forward \"%s\" is not supported", i, kind.c_str()); return FORGE_ERR_UNSUPPORTED; }
+            FORGE_TRY(need_int(mlp, "ff", &L.ff));
+            if (s->arch->dense == Mlp::ClampedGlu) {
+                double limit;
+                FORGE_TRY(need_num(mlp, "limit", &limit));
+                L.limit = float(limit);
+            }
+        }
+        const Json* of = e.get("weights_of");
+        if (of && of->kind != Json::Null) {
+            FORGE_TRY(need_int(&e, "weights_of", &L.weights_of, 0));
+            if (L.weights_of >= n || L.weights_of == i) { set_error("layer %d: weights_of %d is not another layer", i, L.weights_of); return FORGE_ERR_SHAPE; }
+        }
+        s->layers.push_back(L);
+    }
+    for (int i = 0; i < n; ++i) {
+        const LayerSpec& L = s->layers[i];
+        if (L.weights_of < 0) continue;
+        const LayerSpec& O = s->layers[L.weights_of];
+        if (O.weights_of >= 0 || !same_sizes(L, O)) {
+            set_error("layer %d: weights_of %d names a layer of other sizes or without tensors", i, L.weights_of);
+            return FORGE_ERR_SHAPE;
+        }
+    }
+    const Json* loop = c.get("loop");
+    if (loop && loop->kind != Json::Null) {
+        FORGE_TRY(need_int(loop, "start", &s->loop_start, 0));
+        FORGE_TRY(need_int(loop, "stop", &s->loop_stop));
+        FORGE_TRY(need_int(loop, "times", &s->loop_times));
+        if (s->loop_start >= s->loop_stop || s->loop_stop > n || s->loop_times > 4096) { set_error("config.json: loop %d .. %d of %d layers", s->loop_start, s->loop_stop, n); return FORGE_ERR_SHAPE; }
+    }
+    for (int i = 0; i < n; ++i) {
+        if (s->loop_times == 0 || i < s->loop_start || i >= s->loop_stop) { s->runs.push_back({i, -1}); continue; }
+        for (int t = 0; t < s->loop_times; ++t)
+            for (int l = s->loop_start; l < s->loop_stop; ++l) s->runs.push_back({l, l == s->loop_start ? t : -1});
+        i = s->loop_stop - 1;
+    }
+    return FORGE_OK;
+}
+
+int32_t stack_find_tensors(const Checkpoint& ck, StackSpec* s, StackTensors* t) {
+    const int64_t W = s->width, V = s->vocab;
+    TensorSet* set = &t->top;
+    std::string prefix;
+    auto get = [&](const std::string& name, std::vector<int64_t> shape) -> int32_t {
+        const TensorView* v = ck.tensor(prefix + name, shape);
+        if (!v) return FORGE_ERR_SHAPE;
+        (*set)[name] = v;
+        return FORGE_OK;
+    };
+    auto norm = [&](const std::string& name) -> int32_t {
+        FORGE_TRY(get(name, {W}));
+        FORGE_TRY(get(name + ".b", {W}));
+        return get(name + ".alpha", {});
+    };
+    // rows of a matrix [rank][cols] whose first size only its shape gives
+    auto rank_of = [&](const std::string& name, int* rank) -> int32_t {
+        const TensorView* v = ck.find(prefix + name);
+        if (!v || v->shape.size() != 2 || v->shape[0] < 1 || v->shape[0] > (1 << 20)) { set_error("tensor \"%s\" is missing or no matrix", (prefix + name).c_str()); return FORGE_ERR_SHAPE; }
+        *rank = int(v->shape[0]);
+        return get(name, {v->shape[0], W});
+    };
+    FORGE_TRY(get("embed", {V, W}));
+    FORGE_TRY(get("head", {V, W}));
+    FORGE_TRY(norm("final.norm"));
+    if (s->loop_times) { FORGE_TRY(get("loop.in", {W, 2 * W})); FORGE_TRY(get("loop.step", {s->loop_times, W})); }
+    for (size_t i = 0; i < s->layers.size(); ++i) {
+        t->layers.push_back(TensorSet{});
+        LayerSpec& L = s->layers[i];
+        if (L.weights_of >= 0) continue;
+        set = &t->layers.back();
+        prefix = "l" + std::to_string(i) + ".";
+        FORGE_TRY(norm("norm1"));
+        const RecurDims& r = L.rec;
+        const int64_t H = r.heads, D = int64_t(r.heads) * r.dim, HV = int64_t(r.heads) * r.vdim;
+        switch (L.kind) {
+            case Mixer::Latent: {
+                const LatentDims& d = L.mix;
+                const int64_t hv = int64_t(d.heads) * d.vdim;
+                FORGE_TRY(get("mix.q", {int64_t(d.heads) * (d.dim + d.rot), W}));
+                FORGE_TRY(get("mix.dkv", {d.rank + d.rot, W}));
+                FORGE_TRY(get("mix.dkv.norm", {d.rank}));
+                FORGE_TRY(get("mix.uk", {int64_t(d.heads) * d.dim, d.rank}));
+                FORGE_TRY(get("mix.uv", {hv, d.rank}));
+                FORGE_TRY(get("mix.g", {hv, W}));
+                FORGE_TRY(get("mix.o", {W, hv}));
+                break;
+            }
+            case Mixer::Delta:
+            case Mixer::ChannelDelta: {
+                FORGE_TRY(get("mix.q", {r.qk(), W})); FORGE_TRY(get("mix.q.conv", {r.qk(), r.taps}));
+                FORGE_TRY(get("mix.k", {r.qk(), W})); FORGE_TRY(get("mix.k.conv", {r.qk(), r.taps}));
+                FORGE_TRY(get("mix.v", {HV, W})); FORGE_TRY(get("mix.v.conv", {HV, r.taps}));
+                FORGE_TRY(get("mix.b", {H, W}));
+                FORGE_TRY(get("mix.A_log", {H}));
+                FORGE_TRY(get("mix.norm", {r.vdim}));
+                FORGE_TRY(get("mix.o", {W, HV}));
+                if (L.kind == Mixer::Delta) {
+                    FORGE_TRY(get("mix.a", {H, W})); FORGE_TRY(get("mix.dt_bias", {H}));
+                    FORGE_TRY(get("mix.g", {HV, W}));
+                } else {
+                    FORGE_TRY(rank_of("mix.a1", &L.decay_rank)); FORGE_TRY(get("mix.a2", {D, L.decay_rank}));
+                    FORGE_TRY(get("mix.dt_bias", {D}));
+                    FORGE_TRY(rank_of("mix.g1", &L.gate_rank)); FORGE_TRY(get("mix.g2", {HV, L.gate_rank}));
+                }
+                break;
+            }
+            case Mixer::AttnTimeMix: {
+                const AttnDims& a = L.attn;
+                FORGE_TRY(get("mix.left.q", {int64_t(a.heads) * a.dim, W}));
+                FORGE_TRY(get("mix.left.k", {int64_t(a.groups) * a.dim, W}));
+                FORGE_TRY(get("mix.left.v", {int64_t(a.groups) * a.vdim, W}));
+                FORGE_TRY(get("mix.left.g", {a.heads, W}));
+                FORGE_TRY(get("mix.left.o", {W, int64_t(a.heads) * a.vdim}));
+                FORGE_TRY(get("mix.left.out", {W}));
+                for (const char* x : {"r", "k", "v", "g"}) FORGE_TRY(get(std::string("mix.right.") + x, {D, W}));
+                for (const char* x : {"r", "k", "v", "g", "w"}) FORGE_TRY(get(std::string("mix.right.mu.") + x, {W}));
+                FORGE_TRY(rank_of("mix.right.w1", &L.decay_rank)); FORGE_TRY(get("mix.right.w2", {D, L.decay_rank}));
+                FORGE_TRY(get("mix.right.w0", {D}));
+                FORGE_TRY(get("mix.right.u", {H, r.dim}));
+                FORGE_TRY(get("mix.right.norm", {D}));
+                FORGE_TRY(get("mix.right.o", {W, D}));
+                FORGE_TRY(get("mix.right.out", {W}));
+                break;
+            }
+        }
+        if (L.ff) {
+            if (s->arch->arrangement == Arrangement::Sequential) FORGE_TRY(norm("norm2"));
+            FORGE_TRY(get("mlp.gate", {L.ff, W}));
+            FORGE_TRY(get("mlp.up", {L.ff, W}));
+            FORGE_TRY(get("mlp.down", {W, L.ff}));
+        }
+    }
+    return FORGE_OK;
+}
+
+void stack_fill_info(const StackSpec& s, ForgeCheckpointInfo* out) {
+    memset(out, 0, sizeof(*out));
+    snprintf(out->architecture, sizeof out->architecture, "%s", s.arch->name);
+    out->hidden_size = s.width; out->vocab_size = s.vocab; out->num_layers = int32_t(s.runs.size());
+    out->parameters = s.parameters;
+    for (const LayerSpec& L : s.layers) out->num_weight_layers += L.weights_of < 0;
+    for (const LayerRun& r : s.runs) {
+        const LayerSpec& L = s.layers[r.layer];
+        out->cache_values_per_token += L.cache_row();
+        if (L.has_state()) out->state_values_per_sequence += int64_t(L.rec.state_values() + L.rec.ring_values()) + (L.kind == Mixer::AttnTimeMix ? s.width : 0);
+    }
+}
+
+}  // namespace forge
+
+// ------------------------------------------------------------------------------------------------ C API
+using namespace forge;
+
+extern "C" int32_t forge_checkpoint_info(const char* dir, ForgeCheckpointInfo* out) {
+    if (!dir || !out) { set_error("bad argument to forge_checkpoint_info"); return FORGE_ERR_INVALID_ARG; }
+    Checkpoint ck;
+    StackSpec s;
+    StackTensors t;
+    FORGE_TRY(ck.open(dir));
+    FORGE_TRY(stack_parse(ck.config(), &s));
+    FORGE_TRY(stack_find_tensors(ck, &s, &t));
+    s.parameters = ck.parameters();
+    stack_fill_info(s, out);
+    return FORGE_OK;
+}

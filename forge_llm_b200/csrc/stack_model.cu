@@ -1,62 +1,47 @@
-// Layer-list models: a checkpoint's config.json names an architecture and lists layers, each with a mixer, the mixer's sizes
-// and a feed-forward.  This file holds the registry, the reader of the configuration, the loader, the cache rows and the
-// launch sequences; the session calls (model.cu) - cache, prompt, decode graph, greedy loop, sampling, mixed steps - take
-// such a model like a quantised decoder.
+// Layer-list models: loader, cache and state, launch sequences.  The session calls (model.cu) - cache, prompt, decode graph, greedy
+// loop, sampling, mixed steps - take such a model like a quantised decoder.
 //
-// One layer of the parallel arrangement (x += mixer(h) + ff(h), one norm in front) is two dense products and, between them,
-// the attention:
-//   in    one product of h over the stacked rows [q | dkv | g | gate, up interleaved]; its epilogue leaves q and dkv as f32,
-//         sigmoid(g), and the gated feed-forward activation;
-//   post  latent norm, rotations, cache append, queries into the latent space (rows of their own) or in prompt layout;
-//   attention over the latent cache (single rows) or over keys and values formed for the portion (prompts);
-//   out   one product over the concatenated columns [o | down] of [gated heads | feed-forward activation]: both sublayers
-//         are summed by the product itself; its epilogue adds the residual and applies the next layer's Dynamic Tanh norm,
-//         which needs no statistics of the row.
+// A sublayer is a dense product of its normed input (all projections of a mixer in one), the mechanism, and a dense product
+// whose epilogue adds the residual and leaves what the next reader of the stream takes (After): its Dynamic Tanh norm, or the
+// stream itself where a pass of the loop begins.
+//   parallel arrangement   the `in` product also holds the feed-forward's rows, and `out` runs over the concatenated columns
+//                          [o | down] of [gated heads | activation], so both sublayers are summed by the product itself;
+//   delta rules            in [q k v | gate | beta | decay] (a second product for two-step gates and decays), recurrence, out;
+//   attention | time mix   the input's columns are [h | five shifted mixes] and every row of `in` reads the block it belongs to; keys
+//                          and values go from the epilogue into the cache; two out products, then the sum of their norms.
 #include <algorithm>
 #include <cmath>
 #include <cstring>
 #include <map>
 #include <memory>
 
-#include "checkpoint.cuh"
-#include "mla.cuh"
 #include "model.cuh"
+#include "stack.cuh"
 
 // ------------------------------------------------------------------------------------------------ structures
 namespace forge {
 
-enum class Norm { DynamicTanh };
-enum class Arrangement { Parallel };
-enum class Mlp { ClampedGlu };
-struct Architecture { const char* name; Norm norm; Arrangement arrangement; Mlp dense; };
-static const Architecture kArchitectures[] = {
-    {"Bolenex", Norm::DynamicTanh, Arrangement::Parallel, Mlp::ClampedGlu},
-};
-
-struct LayerSpec {
-    LatentDims mix;
-    double rot_base = 1.0;
-    int ff = 0;            // 0: no feed-forward
-    float limit = 0.f;
-    int weights_of = -1;   // layer whose tensors are used
-};
-struct StackSpec {
-    const Architecture* arch = nullptr;
-    int width = 0, vocab = 0;
-    float eps = 0.f;
-    std::vector<LayerSpec> layers;
-    int64_t parameters = 0;
-};
-
 struct DytNorm { float* w = nullptr; float* b = nullptr; float alpha = 0.f; };
 
 struct LayerWeights {
-    DytNorm norm;
-    DenseWeight in, out, kv;      // kv: rows [uk | uv] over the latent
+    DytNorm norm1, norm2;
+    DenseWeight in, out;
+    DenseWeight ff_in, ff_out;    // sequential arrangement
+    // latent attention
+    DenseWeight kv;               // rows [uk | uv] over the latent
     int q_rows = 0, dkv_row = 0, g_row = 0, glu_row = 0, uv_row = 0;   // first rows of the segments of `in` / `kv`
     int heads_k = 0;              // columns of `out` in front of the feed-forward's
     float* kv_norm = nullptr;
-    float* rope = nullptr;        // of this layer's base and dims
+    // recurrent mixers
+    int gate_row = 0, beta_row = 0, decay_row = 0, low_gate_row = 0;   // first rows of the segments of `in`
+    int decay_k = 0;              // columns of the decay's inner values in front of the gate's
+    int low_row = 0;              // first row of the gate in `low`
+    DenseWeight low;              // second step of decay [and gate]
+    float *conv = nullptr, *decay_mul = nullptr, *decay_add = nullptr, *bonus = nullptr, *head_norm = nullptr;
+    // attention beside time mixing
+    int k_row = 0, v_row = 0, hg_row = 0, r_row = 0, rk_row = 0, rv_row = 0;
+    DenseWeight out_r;
+    float *mu = nullptr, *norm_l = nullptr, *norm_r = nullptr;
 };
 
 struct StackModel {
@@ -66,157 +51,29 @@ struct StackModel {
     void* embed = nullptr;
     std::vector<LayerWeights> w;                       // by layer; empty for a layer with weights_of
     DytNorm final_norm;
-    DenseWeight head;
+    DenseWeight head, loop_in;
+    float* loop_step = nullptr;                        // [times][width]
     std::map<std::pair<double, int>, std::pair<int, float*>> ropes;   // (base, dims) -> positions, table
     int rope_positions = 0;
     DenseScratch scratch;
     // step buffers, grown on demand (scratch_gen of the model counts the moves)
     struct Buf { void* p = nullptr; size_t cap = 0; };
-    Buf x, h, proj, gate, mid, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, sel, logits, meta;
-    std::vector<Buf*> all() { return {&x, &h, &proj, &gate, &mid, &q, &part, &ml, &ctx_c, &ctx_r, &ctx_k, &ctx_v, &sel, &logits, &meta}; }
+    Buf x, h, cat, proj, gate, mid, mid_r, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, hgate, decay, beta, low, conv, unit, o, pair, place, sel, logits, meta;
+    std::vector<Buf*> all() {
+        return {&x, &h, &cat, &proj, &gate, &mid, &mid_r, &q, &part, &ml, &ctx_c, &ctx_r, &ctx_k, &ctx_v, &hgate, &decay, &beta, &low, &conv, &unit, &o, &pair, &place, &sel, &logits, &meta};
+    }
+    const LayerWeights& weights(int layer) const { return w[spec.layers[layer].weights_of >= 0 ? spec.layers[layer].weights_of : layer]; }
 };
 
-// Cache rows of every layer run: [pages][FORGE_KV_PAGE][row] of the model's type, one pool per run.
+// What a layer run keeps: cache rows in pages of the pool, [pages][FORGE_KV_PAGE][row] of the model's type, and per sequence a
+// recurrent state (f32), the last inputs of its convolution and the last row of its token shift (the model's type).
 struct StackCache {
-    struct Run { void* pool = nullptr; alignas(64) unsigned char map[128]; };
+    struct Run { void* pool = nullptr; alignas(64) unsigned char map[128]; float* state = nullptr; void* ring = nullptr; void* prev = nullptr; };
     std::vector<Run> runs;
     int splits = 1;     // of a captured decode step
 };
 
 namespace {
-
-// ------------------------------------------------------------------------------------------------ configuration
-int32_t need_int(const Json* o, const char* key, int* out, int lo = 1) {
-    const Json* v = o ? o->get(key) : nullptr;
-    if (!v || v->kind != Json::Number || v->num != std::floor(v->num) || v->num < lo || v->num > 1e9) { set_error("config.json: \"%s\" must be an integer of at least %d", key, lo); return FORGE_ERR_SHAPE; }
-    *out = int(v->num);
-    return FORGE_OK;
-}
-int32_t need_num(const Json* o, const char* key, double* out) {
-    const Json* v = o ? o->get(key) : nullptr;
-    if (!v || v->kind != Json::Number) { set_error("config.json: \"%s\" must be a number", key); return FORGE_ERR_SHAPE; }
-    *out = v->num;
-    return FORGE_OK;
-}
-int32_t need_string(const Json* o, const char* key, std::string* out) {
-    const Json* v = o ? o->get(key) : nullptr;
-    if (!v || v->kind != Json::String) { set_error("config.json: \"%s\" must be a string", key); return FORGE_ERR_SHAPE; }
-    *out = v->str;
-    return FORGE_OK;
-}
-
-int32_t parse_latent(const Json* m, float eps, LayerSpec* L) {
-    LatentDims& d = L->mix;
-    double scale;
-    FORGE_TRY(need_int(m, "heads", &d.heads));
-    FORGE_TRY(need_int(m, "dim", &d.dim));
-    FORGE_TRY(need_int(m, "rot_dim", &d.rot, 0));
-    FORGE_TRY(need_int(m, "vdim", &d.vdim));
-    FORGE_TRY(need_int(m, "kv_rank", &d.rank));
-    FORGE_TRY(need_num(m, "scale", &scale));
-    if (d.rot > 0) {
-        const Json* rot = m->get("rot");
-        FORGE_TRY(need_int(rot, "dims", &d.rot_dims, 0));
-        FORGE_TRY(need_num(rot, "base", &L->rot_base));
-        if (d.rot_dims > d.rot || d.rot_dims % 2 || !(L->rot_base > 0)) { set_error("config.json: rot.dims %d does not fit rot_dim %d", d.rot_dims, d.rot); return FORGE_ERR_SHAPE; }
-    }
-    d.scale = float(scale); d.eps = eps;
-    d.rank_p = pad_to(d.rank, 64); d.rot_p = pad_to(d.rot, 64); d.dim_p = pad_to(d.dim, 64); d.vdim_p = pad_to(d.vdim, 64);
-    return FORGE_OK;
-}
-
-int32_t parse_spec(const Json& c, StackSpec* s) {
-    std::string name;
-    FORGE_TRY(need_string(&c, "architecture", &name));
-    for (const Architecture& a : kArchitectures) if (name == a.name) s->arch = &a;
-    if (!s->arch) { set_error("architecture \"%s\" is not registered", name.c_str()); return FORGE_ERR_UNSUPPORTED; }
-    FORGE_TRY(need_int(&c, "width", &s->width));
-    FORGE_TRY(need_int(&c, "vocab", &s->vocab));
-    double eps;
-    FORGE_TRY(need_num(c.get("norm"), "eps", &eps));
-    s->eps = float(eps);
-    const Json* layers = c.get("layers");
-    if (!layers || layers->kind != Json::Array || layers->items.empty()) { set_error("config.json: \"layers\" must list at least one layer"); return FORGE_ERR_SHAPE; }
-    for (size_t i = 0; i < layers->items.size(); ++i) {
-        const Json& e = layers->items[i];
-        LayerSpec L;
-        std::string type;
-        FORGE_TRY(need_string(&e, "type", &type));
-        if (type != "latent_attention") { set_error("layer %zu: mixer \"%s\" is not supported", i, type.c_str()); return FORGE_ERR_UNSUPPORTED; }
-        FORGE_TRY(parse_latent(e.get("mixer"), s->eps, &L));
-        const Json* mlp = e.get("mlp");
-        if (mlp && mlp->kind != Json::Null) {
-            std::string kind;
-            FORGE_TRY(need_string(mlp, "kind", &kind));
-            if (kind != "dense") { set_error("layer %zu: feed-forward \"%s\" is not supported", i, kind.c_str()); return FORGE_ERR_UNSUPPORTED; }
-            double limit;
-            FORGE_TRY(need_int(mlp, "ff", &L.ff));
-            FORGE_TRY(need_num(mlp, "limit", &limit));
-            L.limit = float(limit);
-        }
-        const Json* of = e.get("weights_of");
-        if (of && of->kind != Json::Null) {
-            FORGE_TRY(need_int(&e, "weights_of", &L.weights_of, 0));
-            if (L.weights_of >= int(layers->items.size()) || L.weights_of == int(i)) { set_error("layer %zu: weights_of %d is not another layer", i, L.weights_of); return FORGE_ERR_SHAPE; }
-        }
-        s->layers.push_back(L);
-    }
-    for (size_t i = 0; i < s->layers.size(); ++i) {
-        const LayerSpec& L = s->layers[i];
-        if (L.weights_of < 0) continue;
-        const LayerSpec& O = s->layers[L.weights_of];
-        const LatentDims &a = L.mix, &b = O.mix;
-        if (O.weights_of >= 0 || a.heads != b.heads || a.dim != b.dim || a.rot != b.rot || a.vdim != b.vdim || a.rank != b.rank || L.ff != O.ff) {
-            set_error("layer %zu: weights_of %d names a layer of other sizes or without tensors", i, L.weights_of);
-            return FORGE_ERR_SHAPE;
-        }
-    }
-    return FORGE_OK;
-}
-
-// every tensor of the design, with its shape
-struct LayerTensors { const TensorView *norm, *norm_b, *norm_a, *q, *dkv, *kvn, *uk, *uv, *g, *o, *gate, *up, *down; };
-struct StackTensors { const TensorView *embed, *head, *fn, *fb, *fa; std::vector<LayerTensors> layers; };
-
-int32_t find_tensors(const Checkpoint& ck, const StackSpec& s, StackTensors* t) {
-#define GET(dst, ...) do { dst = ck.tensor(__VA_ARGS__); if (!dst) return FORGE_ERR_SHAPE; } while (0)
-    const int64_t W = s.width, V = s.vocab;
-    GET(t->embed, "embed", {V, W});
-    GET(t->head, "head", {V, W});
-    GET(t->fn, "final.norm", {W}); GET(t->fb, "final.norm.b", {W}); GET(t->fa, "final.norm.alpha", {});
-    for (size_t i = 0; i < s.layers.size(); ++i) {
-        t->layers.push_back(LayerTensors{});
-        const LayerSpec& L = s.layers[i];
-        if (L.weights_of >= 0) continue;
-        LayerTensors& o = t->layers.back();
-        const LatentDims& d = L.mix;
-        const std::string p = "l" + std::to_string(i) + ".", x = p + "mix.";
-        const int64_t HV = int64_t(d.heads) * d.vdim;
-        GET(o.norm, p + "norm1", {W}); GET(o.norm_b, p + "norm1.b", {W}); GET(o.norm_a, p + "norm1.alpha", {});
-        GET(o.q, x + "q", {int64_t(d.heads) * (d.dim + d.rot), W});
-        GET(o.dkv, x + "dkv", {d.rank + d.rot, W});
-        GET(o.kvn, x + "dkv.norm", {d.rank});
-        GET(o.uk, x + "uk", {int64_t(d.heads) * d.dim, d.rank});
-        GET(o.uv, x + "uv", {HV, d.rank});
-        GET(o.g, x + "g", {HV, W});
-        GET(o.o, x + "o", {W, HV});
-        if (L.ff) {
-            GET(o.gate, p + "mlp.gate", {L.ff, W});
-            GET(o.up, p + "mlp.up", {L.ff, W});
-            GET(o.down, p + "mlp.down", {W, L.ff});
-        }
-    }
-#undef GET
-    return FORGE_OK;
-}
-
-void fill_info(const StackSpec& s, ForgeCheckpointInfo* out) {
-    memset(out, 0, sizeof(*out));
-    snprintf(out->architecture, sizeof out->architecture, "%s", s.arch->name);
-    out->hidden_size = s.width; out->vocab_size = s.vocab; out->num_layers = int32_t(s.layers.size());
-    out->parameters = s.parameters;
-    for (const LayerSpec& L : s.layers) { out->num_weight_layers += L.weights_of < 0; out->cache_values_per_token += L.mix.row(); }
-}
 
 // ------------------------------------------------------------------------------------------------ loading
 void store(void* dst, int dtype, size_t i, const TensorView& t, size_t j) {
@@ -250,11 +107,6 @@ int32_t upload_f32(ForgeModel* m, float** dst, const TensorView& t) {
     FORGE_CUDA(cudaStreamSynchronize(m->stream));
     return FORGE_OK;
 }
-int32_t load_dyt(ForgeModel* m, DytNorm* n, const TensorView& w, const TensorView& b, const TensorView& a) {
-    n->alpha = a.at(0);
-    FORGE_TRY(upload_f32(m, &n->w, w));
-    return upload_f32(m, &n->b, b);
-}
 // row_reads: some kernel reads rows of the matrix, so it is kept in rows as well
 int32_t load_dense(ForgeModel* m, DenseWeight* w, int N, int K, int dtype, const std::vector<uint8_t>& img, bool row_reads = false) {
     w->N = N; w->K = K; w->dtype = dtype;
@@ -267,40 +119,151 @@ int32_t load_dense(ForgeModel* m, DenseWeight* w, int N, int K, int dtype, const
     return FORGE_OK;
 }
 
-int32_t load_layer(ForgeModel* m, const LayerSpec& L, const LayerTensors& t, LayerWeights* w) {
+int32_t upload_values(ForgeModel* m, float** dst, const std::vector<float>& v) {
+    FORGE_TRY(dev_alloc(m, dst, v.size()));
+    FORGE_CUDA(cudaMemcpyAsync(*dst, v.data(), v.size() * 4, cudaMemcpyHostToDevice, m->stream));
+    FORGE_CUDA(cudaStreamSynchronize(m->stream));
+    return FORGE_OK;
+}
+
+// the host image of a matrix of N rows and K (padded) columns, filled piece by piece
+struct Image {
+    std::vector<uint8_t> img;
+    int N, K, dtype;
+    Image(int n, int k, int dt) : img(size_t(n) * k * dense_size(dt), 0), N(n), K(k), dtype(dt) {}
+    void put(const TensorView* t, int row0, int step = 1, int col0 = 0) { put_rows(img, dtype, K, *t, row0, step, col0); }
+    int32_t load(ForgeModel* m, DenseWeight* w, bool row_reads = false) const { return load_dense(m, w, N, K, dtype, img, row_reads); }
+};
+
+int32_t load_norm(ForgeModel* m, DytNorm* n, const TensorSet& t, const std::string& name) {
+    n->alpha = t.at(name + ".alpha")->at(0);
+    FORGE_TRY(upload_f32(m, &n->w, *t.at(name)));
+    return upload_f32(m, &n->b, *t.at(name + ".b"));
+}
+
+int32_t load_latent(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
     StackModel& S = *m->stack;
     const LatentDims& d = L.mix;
-    const size_t es = dense_size(S.dtype);
-    FORGE_TRY(load_dyt(m, &w->norm, *t.norm, *t.norm_b, *t.norm_a));
-    FORGE_TRY(upload_f32(m, &w->kv_norm, *t.kvn));
+    const int ff = S.spec.arch->arrangement == Arrangement::Parallel ? L.ff : 0;
+    FORGE_TRY(upload_f32(m, &w->kv_norm, *t.at("mix.dkv.norm")));
     w->q_rows = d.heads * (d.dim + d.rot);
     w->dkv_row = pad_to(w->q_rows, kSegAlign);
     w->g_row = w->dkv_row + pad_to(d.rank + d.rot, kSegAlign);
     w->glu_row = w->g_row + pad_to(d.heads * d.vdim, kSegAlign);
-    const int n_in = w->glu_row + 2 * L.ff;
+    Image in(w->glu_row + 2 * ff, S.width_p, S.dtype);
+    in.put(t.at("mix.q"), 0);
+    in.put(t.at("mix.dkv"), w->dkv_row);
+    in.put(t.at("mix.g"), w->g_row);
+    if (ff) { in.put(t.at("mlp.gate"), w->glu_row, 2); in.put(t.at("mlp.up"), w->glu_row + 1, 2); }
+    FORGE_TRY(in.load(m, &w->in));
+    w->uv_row = pad_to(d.heads * d.dim, kSegAlign);
+    Image kv(w->uv_row + d.heads * d.vdim, d.rank_p, S.dtype);
+    kv.put(t.at("mix.uk"), 0);
+    kv.put(t.at("mix.uv"), w->uv_row);
+    FORGE_TRY(kv.load(m, &w->kv, true));
+    w->heads_k = pad_to(d.heads * d.vdim, kDensePad);
+    Image out(S.spec.width, w->heads_k + pad_to(ff, kDensePad), S.dtype);
+    out.put(t.at("mix.o"), 0);
+    if (ff) out.put(t.at("mlp.down"), 0, 1, w->heads_k);
+    return out.load(m, &w->out);
+}
+
+int32_t load_delta(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
+    StackModel& S = *m->stack;
+    const RecurDims& d = L.rec;
+    const int H = d.heads, HV = d.heads * d.vdim;
     {
-        std::vector<uint8_t> img(size_t(n_in) * S.width_p * es, 0);
-        put_rows(img, S.dtype, S.width_p, *t.q, 0);
-        put_rows(img, S.dtype, S.width_p, *t.dkv, w->dkv_row);
-        put_rows(img, S.dtype, S.width_p, *t.g, w->g_row);
-        if (L.ff) { put_rows(img, S.dtype, S.width_p, *t.gate, w->glu_row, 2); put_rows(img, S.dtype, S.width_p, *t.up, w->glu_row + 1, 2); }
-        FORGE_TRY(load_dense(m, &w->in, n_in, S.width_p, S.dtype, img));
+        std::vector<float> conv;
+        for (const char* n : {"mix.q.conv", "mix.k.conv", "mix.v.conv"}) for (int64_t i = 0; i < t.at(n)->count(); ++i) conv.push_back(t.at(n)->at(size_t(i)));
+        FORGE_TRY(upload_values(m, &w->conv, conv));
+        // a decay's logarithm is -exp(A_log of the head) softplus(its row's value + dt_bias)
+        const int per = d.channel ? d.dim : 1;
+        std::vector<float> mul(size_t(H) * per);
+        for (int h = 0; h < H; ++h) for (int i = 0; i < per; ++i) mul[size_t(h) * per + i] = float(std::exp(double(t.at("mix.A_log")->at(h))));
+        FORGE_TRY(upload_values(m, &w->decay_mul, mul));
+        FORGE_TRY(upload_f32(m, &w->decay_add, *t.at("mix.dt_bias")));
+        FORGE_TRY(upload_f32(m, &w->head_norm, *t.at("mix.norm")));
     }
-    {
-        w->uv_row = pad_to(d.heads * d.dim, kSegAlign);
-        const int n = w->uv_row + d.heads * d.vdim;
-        std::vector<uint8_t> img(size_t(n) * d.rank_p * es, 0);
-        put_rows(img, S.dtype, d.rank_p, *t.uk, 0);
-        put_rows(img, S.dtype, d.rank_p, *t.uv, w->uv_row);
-        FORGE_TRY(load_dense(m, &w->kv, n, d.rank_p, S.dtype, img, true));
+    int row = pad_to(d.channels(), kSegAlign);
+    auto take = [&](int rows) { const int at = row; row += pad_to(rows, kSegAlign); return at; };
+    if (d.channel) {
+        w->beta_row = take(H); w->decay_row = take(L.decay_rank); w->low_gate_row = take(L.gate_rank);
+    } else {
+        w->gate_row = take(HV); w->beta_row = take(H); w->decay_row = take(H);
     }
-    {
-        w->heads_k = pad_to(d.heads * d.vdim, kDensePad);
-        const int k = w->heads_k + pad_to(L.ff, kDensePad);
-        std::vector<uint8_t> img(size_t(S.spec.width) * k * es, 0);
-        put_rows(img, S.dtype, k, *t.o, 0);
-        if (L.ff) put_rows(img, S.dtype, k, *t.down, 0, 1, w->heads_k);
-        FORGE_TRY(load_dense(m, &w->out, S.spec.width, k, S.dtype, img));
+    Image in(row, S.width_p, S.dtype);
+    in.put(t.at("mix.q"), 0); in.put(t.at("mix.k"), d.qk()); in.put(t.at("mix.v"), 2 * d.qk());
+    in.put(t.at("mix.b"), w->beta_row);
+    if (d.channel) {
+        in.put(t.at("mix.a1"), w->decay_row); in.put(t.at("mix.g1"), w->low_gate_row);
+        // rows [a2 | g2]; each reads its own block of the inner values, K is the wider of the two
+        w->decay_k = pad_to(L.decay_rank, kDensePad);
+        w->low_row = pad_to(H * d.dim, 128);
+        Image low(w->low_row + HV, std::max(w->decay_k, pad_to(L.gate_rank, kDensePad)), S.dtype);
+        low.put(t.at("mix.a2"), 0);
+        low.put(t.at("mix.g2"), w->low_row);
+        FORGE_TRY(low.load(m, &w->low));
+    } else {
+        in.put(t.at("mix.g"), w->gate_row); in.put(t.at("mix.a"), w->decay_row);
+    }
+    FORGE_TRY(in.load(m, &w->in));
+    Image out(S.spec.width, pad_to(HV, kDensePad), S.dtype);
+    out.put(t.at("mix.o"), 0);
+    return out.load(m, &w->out);
+}
+
+constexpr int kMixes = 5;   // r, k, v, g, w
+
+int32_t load_pair(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
+    StackModel& S = *m->stack;
+    const AttnDims& a = L.attn;
+    const RecurDims& d = L.rec;
+    const int D = d.heads * d.dim;
+    int row = 0;
+    auto take = [&](int rows, int align) { row = pad_to(row, align); const int at = row; row += rows; return at; };
+    const int q_row = take(a.heads * a.dim, kSegAlign);
+    w->k_row = take(a.groups * a.dim, kSegAlign); w->v_row = take(a.groups * a.vdim, kSegAlign); w->hg_row = take(a.heads, kSegAlign);
+    // a tile of rows reads one block of the activations
+    w->r_row = take(D, 128); w->rk_row = take(D, 128); w->rv_row = take(D, 128); w->gate_row = take(D, 128); w->decay_row = take(L.decay_rank, 128);
+    Image in(row, S.width_p, S.dtype);
+    in.put(t.at("mix.left.q"), q_row); in.put(t.at("mix.left.k"), w->k_row); in.put(t.at("mix.left.v"), w->v_row); in.put(t.at("mix.left.g"), w->hg_row);
+    in.put(t.at("mix.right.r"), w->r_row); in.put(t.at("mix.right.k"), w->rk_row); in.put(t.at("mix.right.v"), w->rv_row);
+    in.put(t.at("mix.right.g"), w->gate_row); in.put(t.at("mix.right.w1"), w->decay_row);
+    FORGE_TRY(in.load(m, &w->in));
+    Image low(D, pad_to(L.decay_rank, kDensePad), S.dtype);
+    low.put(t.at("mix.right.w2"), 0);
+    FORGE_TRY(low.load(m, &w->low));
+    Image out(S.spec.width, pad_to(a.heads * a.vdim, kDensePad), S.dtype);
+    out.put(t.at("mix.left.o"), 0);
+    FORGE_TRY(out.load(m, &w->out));
+    Image out_r(S.spec.width, pad_to(D, kDensePad), S.dtype);
+    out_r.put(t.at("mix.right.o"), 0);
+    FORGE_TRY(out_r.load(m, &w->out_r));
+    std::vector<float> mu;
+    for (const char* n : {"r", "k", "v", "g", "w"}) { const TensorView* v = t.at(std::string("mix.right.mu.") + n); for (int i = 0; i < S.spec.width; ++i) mu.push_back(v->at(size_t(i))); }
+    FORGE_TRY(upload_values(m, &w->mu, mu));
+    FORGE_TRY(upload_f32(m, &w->decay_add, *t.at("mix.right.w0")));
+    FORGE_TRY(upload_f32(m, &w->bonus, *t.at("mix.right.u")));
+    FORGE_TRY(upload_f32(m, &w->head_norm, *t.at("mix.right.norm")));
+    FORGE_TRY(upload_f32(m, &w->norm_l, *t.at("mix.left.out")));
+    return upload_f32(m, &w->norm_r, *t.at("mix.right.out"));
+}
+
+int32_t load_layer(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
+    StackModel& S = *m->stack;
+    FORGE_TRY(load_norm(m, &w->norm1, t, "norm1"));
+    switch (L.kind) {
+        case Mixer::Latent: FORGE_TRY(load_latent(m, L, t, w)); break;
+        case Mixer::Delta: case Mixer::ChannelDelta: FORGE_TRY(load_delta(m, L, t, w)); break;
+        case Mixer::AttnTimeMix: FORGE_TRY(load_pair(m, L, t, w)); break;
+    }
+    if (L.ff && S.spec.arch->arrangement == Arrangement::Sequential) {
+        FORGE_TRY(load_norm(m, &w->norm2, t, "norm2"));
+        Image in(2 * L.ff, S.width_p, S.dtype), out(S.spec.width, pad_to(L.ff, kDensePad), S.dtype);
+        in.put(t.at("mlp.gate"), 0, 2); in.put(t.at("mlp.up"), 1, 2);
+        FORGE_TRY(in.load(m, &w->ff_in));
+        out.put(t.at("mlp.down"), 0);
+        FORGE_TRY(out.load(m, &w->ff_out));
     }
     return FORGE_OK;
 }
@@ -312,6 +275,7 @@ int32_t ensure_rope(ForgeModel* m, int n) {
     n = pad_to(n, 1024);
     FORGE_CUDA(cudaStreamSynchronize(m->stream));
     for (const LayerSpec& L : S.spec.layers) {
+        if (!L.has_latent()) continue;
         auto& e = S.ropes[{L.rot_base, L.mix.rot_dims}];
         if (e.first >= n) continue;
         std::vector<float> tab(std::max<size_t>(1, size_t(n) * L.mix.rot_dims));
@@ -347,45 +311,58 @@ bool tensor_core_rows(const StackModel& S, const LatentDims& d) { return S.dtype
 // splits of the row attention: at most one CTA per SM over all rows and head groups, no more than there are pages
 int row_splits(const StackModel& S, int rows, int pages) {
     int groups = 1;
-    for (const LayerSpec& L : S.spec.layers) groups = std::max(groups, tensor_core_rows(S, L.mix) ? latent_decode_head_groups(L.mix) : L.mix.heads);
+    for (const LayerSpec& L : S.spec.layers) if (L.has_latent()) groups = std::max(groups, tensor_core_rows(S, L.mix) ? latent_decode_head_groups(L.mix) : L.mix.heads);
     return std::max(1, std::min(pages, 148 / std::max(1, rows * groups)));
 }
 
-int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt, int ctx_rows) {
+int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt, int ctx_rows, int seg_rows) {
     StackModel& S = *m->stack;
-    const size_t es = dense_size(S.dtype), r = size_t(rows);
-    size_t proj = 0, gate = 0, mid = 0, qa = 0, part = 0, heads = 0, qp = 0, cc = 0, cr = 0, ck = 0, cv = 0;
+    const size_t es = dense_size(S.dtype), r = size_t(rows), W = size_t(S.spec.width), WP = size_t(S.width_p);
+    // bytes, rows times the widest layer
+    size_t h = WP * es, proj = 0, gate = 0, mid = 0, mid_r = 0, q = 0, part = 0, heads = 0, cc = 0, cr = 0, ck = 0, cv = 0, hgate = 0, decay = 0, beta = 0, low = 0, conv = 0, unit = 0, o = 0, pair = 0;
+    auto most = [](size_t& a, size_t b) { a = std::max(a, b); };
+    size_t n_max = size_t(S.head.N);
     for (size_t i = 0; i < S.spec.layers.size(); ++i) {
         const LayerSpec& L = S.spec.layers[i];
-        const LayerWeights& w = S.w[L.weights_of >= 0 ? L.weights_of : int(i)];
-        const LatentDims& d = L.mix;
-        proj = std::max(proj, size_t(w.g_row));
-        gate = std::max(gate, size_t(d.heads) * d.vdim);
-        mid = std::max(mid, size_t(w.out.K));
-        qa = std::max(qa, size_t(d.heads) * d.row());
-        part = std::max(part, size_t(d.heads) * d.rank_p);
-        heads = std::max(heads, size_t(d.heads));
-        qp = std::max(qp, size_t(d.heads) * (d.dim_p + d.rot_p));
-        cc = std::max(cc, size_t(d.rank_p)); cr = std::max(cr, size_t(std::max(d.rot_p, 64)));
-        ck = std::max(ck, size_t(d.heads) * d.dim_p); cv = std::max(cv, size_t(d.heads) * d.vdim_p);
+        const LayerWeights& w = S.weights(int(i));
+        for (const DenseWeight* d : {&w.in, &w.out, &w.kv, &w.low, &w.out_r, &w.ff_in, &w.ff_out}) most(n_max, size_t(d->N));
+        most(mid, r * std::max(w.out.K, w.ff_out.K) * es);
+        if (L.has_latent()) {
+            const LatentDims& d = L.mix;
+            most(proj, r * w.g_row * 4);
+            most(gate, r * d.heads * d.vdim * es);
+            most(q, std::max(size_t(single) * d.heads * d.row(), size_t(prompt) * d.heads * (d.dim_p + d.rot_p)) * es);
+            most(part, size_t(single) * d.heads * d.rank_p * splits * 4);
+            most(heads, size_t(single) * d.heads * splits * sizeof(float2));
+            most(cc, size_t(ctx_rows) * d.rank_p * es); most(cr, size_t(ctx_rows) * std::max(d.rot_p, 64) * es);
+            most(ck, size_t(ctx_rows) * d.heads * d.dim_p * es); most(cv, size_t(ctx_rows) * d.heads * d.vdim_p * es);
+            continue;
+        }
+        const RecurDims& d = L.rec;
+        const size_t HV = size_t(d.heads) * d.vdim;
+        most(proj, r * d.channels() * es);
+        most(gate, r * HV * es);
+        most(decay, r * (d.channel ? size_t(d.heads) * d.dim : d.heads) * 4);
+        most(beta, r * d.heads * 4);
+        most(low, r * (w.decay_k + w.low.K) * es);
+        most(o, r * HV * 4);
+        if (d.delta && seg_rows) { most(conv, r * d.channels() * es); most(unit, r * 2 * d.groups * 4); }
+        if (L.has_attn()) {
+            most(h, (1 + kMixes) * WP * es);
+            most(q, r * L.attn.heads * L.attn.dim_p * es);
+            most(hgate, r * L.attn.heads * 4);
+            most(mid_r, r * w.out_r.K * es);
+            most(pair, r * 2 * W * 4);
+        }
     }
-    FORGE_TRY(grow(m, S.x, r * S.spec.width * 4));
-    FORGE_TRY(grow(m, S.h, r * S.width_p * es));
-    FORGE_TRY(grow(m, S.proj, r * proj * 4));
-    FORGE_TRY(grow(m, S.gate, r * gate * es));
-    FORGE_TRY(grow(m, S.mid, r * mid * es));
-    FORGE_TRY(grow(m, S.q, std::max(size_t(single) * qa * es, size_t(prompt) * qp * es)));
-    FORGE_TRY(grow(m, S.part, size_t(single) * part * splits * 4));
-    FORGE_TRY(grow(m, S.ml, size_t(single) * heads * splits * sizeof(float2)));
-    if (ctx_rows) {
-        FORGE_TRY(grow(m, S.ctx_c, size_t(ctx_rows) * cc * es));
-        FORGE_TRY(grow(m, S.ctx_r, size_t(ctx_rows) * cr * es));
-        FORGE_TRY(grow(m, S.ctx_k, size_t(ctx_rows) * ck * es));
-        FORGE_TRY(grow(m, S.ctx_v, size_t(ctx_rows) * cv * es));
-    }
+    FORGE_TRY(grow(m, S.x, r * W * 4));
+    FORGE_TRY(grow(m, S.h, r * h));
+    if (S.spec.loop_times) FORGE_TRY(grow(m, S.cat, r * 2 * WP * es));
+    FORGE_TRY(grow(m, S.place, r * sizeof(int32_t)));
+    const std::pair<StackModel::Buf*, size_t> sizes[] = {{&S.proj, proj}, {&S.gate, gate}, {&S.mid, mid}, {&S.mid_r, mid_r}, {&S.q, q}, {&S.part, part}, {&S.ml, heads}, {&S.hgate, hgate}, {&S.decay, decay},
+        {&S.beta, beta}, {&S.low, low}, {&S.conv, conv}, {&S.unit, unit}, {&S.o, o}, {&S.pair, pair}, {&S.ctx_c, cc}, {&S.ctx_r, cr}, {&S.ctx_k, ck}, {&S.ctx_v, cv}};
+    for (const auto& e : sizes) FORGE_TRY(grow(m, *e.first, e.second));
     // one ticket per output tile of the largest product (128 rows x at least 16 tokens)
-    size_t n_max = size_t(S.head.N);
-    for (const LayerWeights& w : S.w) n_max = std::max({n_max, size_t(w.in.N), size_t(w.out.N), size_t(w.kv.N)});
     const size_t tiles = ((n_max + 127) / 128) * std::max<size_t>(1, (size_t(std::max(rows, ctx_rows)) + 127) / 128);
     if (tiles > S.scratch.tickets_cap) {
         FORGE_TRY(dev_alloc(m, &S.scratch.tickets, tiles));
@@ -399,7 +376,10 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
 struct Step {
     const uint32_t* tokens = nullptr;        // device
     StepRows rows;
+    int ones = 0;                            // rows [0, ones): one token of its sequence each
     int single = 0, splits = 1;              // rows [0, single): attention row by row; the rest are prompt rows
+    int max_keys = 1;                        // most keys a row of [0, single) has
+    const ScanSeg* segs = nullptr; int n_segs = 0, max_seg = 0;   // the rows [ones, n)
     const PromptTile* tiles = nullptr; int n_tiles = 0;
     const int32_t* ctx_pages = nullptr; int ctx_rows = 0;
     uint32_t* hist = nullptr; const int32_t* step = nullptr;
@@ -408,30 +388,84 @@ struct Step {
 
 char* at(void* p, size_t elems, int dtype) { return static_cast<char*>(p) + elems * dense_size(dtype); }
 
-// the whole stack for the rows of a step; leaves the final norm's rows in S.h
-int32_t run_layers(ForgeModel* m, ForgeKV* kv, const Step& s) {
-    StackModel& S = *m->stack;
-    cudaStream_t st = m->stream;
-    const int n = s.rows.n, W = S.spec.width, dt = S.dtype, nl = int(S.spec.layers.size());
-    auto weights = [&](int l) -> const LayerWeights& { return S.w[S.spec.layers[l].weights_of >= 0 ? S.spec.layers[l].weights_of : l]; };
-    auto norm_of = [&](int l) -> const DytNorm& { return l < nl ? weights(l).norm : S.final_norm; };
-    FORGE_TRY(embed_dyt(static_cast<float*>(S.x.p), S.h.p, S.width_p, S.embed, dt, s.tokens, n, W, norm_of(0).alpha, norm_of(0).w, norm_of(0).b, s.hist, s.step, st));
-    for (int l = 0; l < nl; ++l) {
-        const LayerSpec& L = S.spec.layers[l];
-        const LayerWeights& w = weights(l);
+// The launch sequence of one step.
+struct Sequence {
+    ForgeModel* m;
+    ForgeKV* kv;
+    const Step& s;
+    StackModel& S;
+    cudaStream_t st;
+    const int n, W, WP, dt;
+    const bool sequential;
+    Sequence(ForgeModel* m_, ForgeKV* kv_, const Step& s_)
+        : m(m_), kv(kv_), s(s_), S(*m_->stack), st(m_->stream), n(s_.rows.n), W(S.spec.width), WP(S.width_p), dt(S.dtype), sequential(S.spec.arch->arrangement == Arrangement::Sequential) {}
+
+    int32_t gemm(const DenseWeight& w, const void* act, int ld, const DenseOut& o, int rows) { return dense_gemm(w, act, ld, rows, o, S.scratch, m->d_err, st); }
+    int32_t gemm(const DenseWeight& w, const void* act, int ld, const DenseOut& o) { return gemm(w, act, ld, o, n); }
+
+    After dyt(const DytNorm& d, int ld) { After a; a.kind = AFTER_DYT; a.alpha = d.alpha; a.w = d.w; a.b = d.b; a.dst = S.h.p; a.ld = ld; return a; }
+    int h_ld(int layer) const { return S.spec.layers[layer].has_attn() ? (1 + kMixes) * WP : WP; }
+    After norm1(int layer) { return dyt(S.weights(layer).norm1, h_ld(layer)); }
+    // what the first reader of the stream in front of run i takes
+    After into(size_t i) {
+        if (i == S.spec.runs.size()) return dyt(S.final_norm, WP);
+        if (S.spec.runs[i].pass < 0) return norm1(S.spec.runs[i].layer);
+        After a;
+        a.kind = AFTER_CAST; a.dst = S.cat.p; a.ld = 2 * WP;
+        return a;
+    }
+    static void resid(DenseOut* o, float* x, int W, const After& after) { o->add(SEG_RESID, 0, W, x, W).after = after; }
+    float* x() { return static_cast<float*>(S.x.p); }
+
+    int32_t run() {
+        EmbedArgs e;
+        e.x = x(); e.table = S.embed; e.tokens = s.tokens; e.width = W; e.width_p = WP;
+        e.after = into(0);
+        if (S.spec.loop_times) { e.x0 = at(S.cat.p, size_t(WP), dt); e.x0_ld = 2 * WP; }
+        e.place = static_cast<int32_t*>(S.place.p); e.rows = s.rows; e.hist = s.hist; e.step = s.step;
+        FORGE_TRY(embed_rows(e, dt, st));
+        for (size_t i = 0; i < S.spec.runs.size(); ++i) {
+            const LayerRun& r = S.spec.runs[i];
+            const LayerSpec& L = S.spec.layers[r.layer];
+            const LayerWeights& w = S.weights(r.layer);
+            StackCache::Run& run = kv->stack->runs[i];
+            if (r.pass >= 0) {
+                DenseOut o;
+                OutSeg& g = o.add(SEG_RESID, 0, W, x(), W);
+                g.fresh = true; g.add = S.loop_step + size_t(r.pass) * W; g.after = norm1(r.layer);
+                FORGE_TRY(gemm(S.loop_in, S.cat.p, 2 * WP, o));
+            }
+            const bool ff = sequential && L.ff;
+            const After after = ff ? dyt(w.norm2, WP) : into(i + 1);
+            switch (L.kind) {
+                case Mixer::Latent: FORGE_TRY(latent(L, w, run, after)); break;
+                case Mixer::Delta: case Mixer::ChannelDelta: FORGE_TRY(delta(L, w, run, after)); break;
+                case Mixer::AttnTimeMix: FORGE_TRY(pair(L, w, run, after)); break;
+            }
+            if (ff) {
+                DenseOut in, out;
+                in.add(S.spec.arch->dense == Mlp::ClampedGlu ? SEG_CLAMPED_GLU : SEG_SILU_GLU, 0, 2 * L.ff, S.mid.p, w.ff_out.K).limit = L.limit;
+                FORGE_TRY(gemm(w.ff_in, S.h.p, WP, in));
+                resid(&out, x(), W, into(i + 1));
+                FORGE_TRY(gemm(w.ff_out, S.mid.p, w.ff_out.K, out));
+            }
+            if (s.trace) FORGE_CUDA(cudaMemcpyAsync(s.trace + i * s.trace_stride, S.x.p, sizeof(float) * n * W, cudaMemcpyDeviceToDevice, st));
+        }
+        return FORGE_OK;
+    }
+
+    int32_t latent(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
         const LatentDims& d = L.mix;
-        const int ldp = w.g_row, gate_ld = d.heads * d.vdim, mid_ld = w.out.K;
+        const int ldp = w.g_row, gate_ld = d.heads * d.vdim, mid_ld = w.out.K, ff = sequential ? 0 : L.ff;
         float* proj = static_cast<float*>(S.proj.p);
         const float* rope = S.ropes.at({L.rot_base, d.rot_dims}).second;
-        StackCache::Run& run = kv->stack->runs[l];
         {
             DenseOut o;
-            auto add = [&](int kind, int row0, int rows, void* dst, int ld) -> OutSeg& { OutSeg& g = o.seg[o.nseg++]; g.kind = kind; g.row0 = row0; g.rows = rows; g.dst = dst; g.ld = ld; return g; };
-            add(SEG_F32, 0, w.q_rows, proj, ldp);
-            add(SEG_F32, w.dkv_row, d.rank + d.rot, proj + w.dkv_row, ldp);
-            add(SEG_SIGMOID, w.g_row, gate_ld, S.gate.p, gate_ld);
-            if (L.ff) add(SEG_CLAMPED_GLU, w.glu_row, 2 * L.ff, at(S.mid.p, w.heads_k, dt), mid_ld).limit = L.limit;
-            FORGE_TRY(dense_gemm(w.in, S.h.p, S.width_p, n, o, S.scratch, m->d_err, st));
+            o.add(SEG_F32, 0, w.q_rows, proj, ldp);
+            o.add(SEG_F32, w.dkv_row, d.rank + d.rot, proj + w.dkv_row, ldp);
+            o.add(SEG_SIGMOID, w.g_row, gate_ld, S.gate.p, gate_ld);
+            if (ff) o.add(S.spec.arch->dense == Mlp::ClampedGlu ? SEG_CLAMPED_GLU : SEG_SILU_GLU, w.glu_row, 2 * ff, at(S.mid.p, w.heads_k, dt), mid_ld).limit = L.limit;
+            FORGE_TRY(gemm(w.in, S.h.p, WP, o));
         }
         StepRows single = s.rows;
         single.n = s.single;
@@ -450,28 +484,126 @@ int32_t run_layers(ForgeModel* m, ForgeKV* kv, const Step& s) {
             FORGE_TRY(latent_post_prompt(d, proj + size_t(s.single) * ldp, ldp, w.dkv_row, w.kv_norm, rope, S.q.p, run.pool, pr, st));
             FORGE_TRY(latent_gather_context(d, run.pool, s.ctx_pages, s.ctx_rows, S.ctx_c.p, S.ctx_r.p, st));
             DenseOut o;
-            o.nseg = 2;
-            o.seg[0].kind = o.seg[1].kind = SEG_CAST;
-            o.seg[0].rows = d.heads * d.dim; o.seg[0].dst = S.ctx_k.p; o.seg[0].ld = d.heads * d.dim_p; o.seg[0].group = d.dim; o.seg[0].group_ld = d.dim_p;
-            o.seg[1].row0 = w.uv_row; o.seg[1].rows = d.heads * d.vdim; o.seg[1].dst = S.ctx_v.p; o.seg[1].ld = d.heads * d.vdim_p; o.seg[1].group = d.vdim; o.seg[1].group_ld = d.vdim_p;
-            FORGE_TRY(dense_gemm(w.kv, S.ctx_c.p, d.rank_p, s.ctx_rows, o, S.scratch, m->d_err, st));
-            PromptAttnArgs a{S.q.p, S.ctx_k.p, S.ctx_r.p, S.ctx_v.p, at(S.gate.p, size_t(s.single) * gate_ld, dt), gate_ld, at(S.mid.p, size_t(s.single) * mid_ld, dt), mid_ld,
-                             np, s.ctx_rows, s.tiles, s.n_tiles, m->d_err};
-            FORGE_TRY(attn_prefill_kv(d, a, st));
+            OutSeg& k = o.add(SEG_CAST, 0, d.heads * d.dim, S.ctx_k.p, d.heads * d.dim_p);
+            k.group = d.dim; k.group_ld = d.dim_p;
+            OutSeg& v = o.add(SEG_CAST, w.uv_row, d.heads * d.vdim, S.ctx_v.p, d.heads * d.vdim_p);
+            v.group = d.vdim; v.group_ld = d.vdim_p;
+            FORGE_TRY(gemm(w.kv, S.ctx_c.p, d.rank_p, o, s.ctx_rows));
+            PromptAttnArgs a;
+            a.q = S.q.p; a.k = S.ctx_k.p; a.krot = S.ctx_r.p; a.v = S.ctx_v.p;
+            a.gate = at(S.gate.p, size_t(s.single) * gate_ld, dt); a.gate_ld = gate_ld;
+            a.out = at(S.mid.p, size_t(s.single) * mid_ld, dt); a.out_ld = mid_ld;
+            a.q_rows = np; a.ctx_rows = s.ctx_rows; a.tiles = s.tiles; a.n_tiles = s.n_tiles; a.err = m->d_err;
+            FORGE_TRY(attn_prefill_kv(PromptDims(d), a, st));
+        }
+        DenseOut o;
+        resid(&o, x(), W, after);
+        return gemm(w.out, S.mid.p, mid_ld, o);
+    }
+
+    // single tokens and segments of a recurrent mixer
+    int32_t recur(const RecurDims& d, const RecurArgs& a) {
+        StepRows ones = s.rows;
+        ones.n = s.ones;
+        FORGE_TRY(recur_decode(d, dt, a, ones, st));
+        RecurScratch sc;
+        sc.conv = S.conv.p; sc.unit = static_cast<float*>(S.unit.p); sc.o = static_cast<float*>(S.o.p);
+        return recur_segments(d, dt, a, sc, s.segs, s.n_segs, s.max_seg, s.ones, n - s.ones, st);
+    }
+    RecurArgs recur_args(const RecurDims& d, const LayerWeights& w, StackCache::Run& run) {
+        RecurArgs a;
+        a.x = S.proj.p; a.x_ld = d.channels();
+        a.decay = static_cast<float*>(S.decay.p); a.decay_ld = d.channel ? d.heads * d.dim : d.heads;
+        a.beta = static_cast<float*>(S.beta.p); a.bonus = w.bonus; a.conv = w.conv; a.ring = run.ring; a.state = run.state;
+        a.norm = w.head_norm;
+        a.gate = S.gate.p; a.gate_ld = d.heads * d.vdim;
+        return a;
+    }
+
+    int32_t delta(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
+        const RecurDims& d = L.rec;
+        const int H = d.heads, HV = H * d.vdim, low_ld = w.decay_k + w.low.K;
+        DenseOut o;
+        o.add(SEG_CAST, 0, d.channels(), S.proj.p, d.channels());
+        if (!d.channel) {
+            o.add(SEG_SILU, w.gate_row, HV, S.gate.p, HV);
+            o.add(SEG_SIGMOID_F32, w.beta_row, H, S.beta.p, H);
+            OutSeg& g = o.add(SEG_DECAY, w.decay_row, H, S.decay.p, H);
+            g.mul = w.decay_mul; g.add = w.decay_add;
+            FORGE_TRY(gemm(w.in, S.h.p, WP, o));
+        } else {
+            o.add(SEG_SIGMOID_F32, w.beta_row, H, S.beta.p, H);
+            o.add(SEG_CAST, w.decay_row, L.decay_rank, S.low.p, low_ld);
+            o.add(SEG_CAST, w.low_gate_row, L.gate_rank, at(S.low.p, w.decay_k, dt), low_ld);
+            FORGE_TRY(gemm(w.in, S.h.p, WP, o));
+            DenseOut lo;
+            OutSeg& g = lo.add(SEG_DECAY, 0, H * d.dim, S.decay.p, H * d.dim);
+            g.mul = w.decay_mul; g.add = w.decay_add;
+            lo.add(SEG_SIGMOID, w.low_row, HV, S.gate.p, HV).act_col = w.decay_k;
+            FORGE_TRY(gemm(w.low, S.low.p, low_ld, lo));
+        }
+        RecurArgs a = recur_args(d, w, run);
+        a.out = S.mid.p; a.out_ld = w.out.K;
+        FORGE_TRY(recur(d, a));
+        DenseOut out;
+        resid(&out, x(), W, after);
+        return gemm(w.out, S.mid.p, w.out.K, out);
+    }
+
+    int32_t pair(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
+        const AttnDims& t = L.attn;
+        const RecurDims& d = L.rec;
+        const int D = d.heads * d.dim, ld = (1 + kMixes) * WP;
+        float* hgate = static_cast<float*>(S.hgate.p);
+        FORGE_TRY(token_shift(S.h.p, ld, W, WP, kMixes, w.mu, run.prev, dt, s.rows, s.ones, s.segs, s.n_segs, s.max_seg, st));
+        DenseOut o;
+        {
+            const int32_t* place = static_cast<const int32_t*>(S.place.p);
+            OutSeg& q = o.add(SEG_CAST, 0, t.heads * t.dim, S.q.p, t.heads * t.dim_p);
+            q.group = t.dim; q.group_ld = t.dim_p;
+            OutSeg& k = o.add(SEG_CAST, w.k_row, t.groups * t.dim, run.pool, t.row());
+            k.group = t.dim; k.group_ld = t.dim_p; k.place = place;
+            OutSeg& v = o.add(SEG_CAST, w.v_row, t.groups * t.vdim, at(run.pool, size_t(t.groups) * t.dim_p, dt), t.row());
+            v.group = t.vdim; v.group_ld = t.vdim_p; v.place = place;
+            o.add(SEG_SIGMOID_F32, w.hg_row, t.heads, hgate, t.heads);
+            o.add(SEG_CAST, w.r_row, D, S.proj.p, 3 * D).act_col = WP;
+            o.add(SEG_CAST, w.rk_row, D, at(S.proj.p, D, dt), 3 * D).act_col = 2 * WP;
+            o.add(SEG_CAST, w.rv_row, D, at(S.proj.p, 2 * D, dt), 3 * D).act_col = 3 * WP;
+            o.add(SEG_SILU, w.gate_row, D, S.gate.p, D).act_col = 4 * WP;
+            o.add(SEG_TANH, w.decay_row, L.decay_rank, S.low.p, w.low.K).act_col = 5 * WP;
+            FORGE_TRY(gemm(w.in, S.h.p, ld, o));
         }
         {
-            const DytNorm& nx = norm_of(l + 1);
-            DenseOut o;
-            o.nseg = 1;
-            OutSeg& g = o.seg[0];
-            g.kind = SEG_RESID; g.rows = W; g.dst = S.x.p; g.ld = W;
-            g.alpha = nx.alpha; g.norm_w = nx.w; g.norm_b = nx.b; g.next = S.h.p; g.next_ld = S.width_p;
-            FORGE_TRY(dense_gemm(w.out, S.mid.p, mid_ld, n, o, S.scratch, m->d_err, st));
+            DenseOut lo;
+            lo.add(SEG_EXP_DECAY, 0, D, S.decay.p, D).add = w.decay_add;
+            FORGE_TRY(gemm(w.low, S.low.p, w.low.K, lo));
         }
-        if (s.trace) FORGE_CUDA(cudaMemcpyAsync(s.trace + size_t(l) * s.trace_stride, S.x.p, sizeof(float) * n * W, cudaMemcpyDeviceToDevice, st));
+        StepRows single = s.rows;
+        single.n = s.single;
+        FORGE_TRY(attn_rows(t, dt, S.q.p, run.pool, hgate, S.mid.p, w.out.K, single, t.chunk ? std::min(t.chunk, s.max_keys) : s.max_keys, st));
+        const int np = n - s.single;
+        if (np > 0) {
+            PromptAttnArgs a;
+            a.q = at(S.q.p, size_t(s.single) * t.heads * t.dim_p, dt); a.k = run.pool; a.v = at(run.pool, size_t(t.groups) * t.dim_p, dt);
+            a.head_gate = hgate + size_t(s.single) * t.heads;
+            a.out = at(S.mid.p, size_t(s.single) * w.out.K, dt); a.out_ld = w.out.K;
+            a.q_rows = np; a.ctx_rows = kv->num_pages * FORGE_KV_PAGE; a.tiles = s.tiles; a.n_tiles = s.n_tiles;
+            a.pages = s.ctx_pages; a.page_row = t.row(); a.err = m->d_err;
+            FORGE_TRY(attn_prefill_kv(PromptDims(t), a, st));
+        }
+        RecurArgs a = recur_args(d, w, run);
+        a.norm_head = d.dim;
+        a.out = S.mid_r.p; a.out_ld = w.out_r.K;
+        FORGE_TRY(recur(d, a));
+        float* both = static_cast<float*>(S.pair.p);
+        DenseOut left, right;
+        left.add(SEG_F32, 0, W, both, 2 * W);
+        right.add(SEG_F32, 0, W, both + W, 2 * W);
+        FORGE_TRY(gemm(w.out, S.mid.p, w.out.K, left));
+        FORGE_TRY(gemm(w.out_r, S.mid_r.p, w.out_r.K, right));
+        return add_normed_pair(x(), both, n, W, S.spec.eps, w.norm_l, w.norm_r, after, dt, st);
     }
-    return FORGE_OK;
-}
+};
 
 int32_t run_head(ForgeModel* m, const void* h, int n, float* logits) {
     StackModel& S = *m->stack;
@@ -481,8 +613,8 @@ int32_t run_head(ForgeModel* m, const void* h, int n, float* logits) {
     return dense_gemm(S.head, h, S.width_p, n, o, S.scratch, m->d_err, m->stream);
 }
 
-// Entries of fewer tokens than this run row by row over the latent cache: forming the keys and values of the whole context
-// does not pay for them.
+// The attention of entries of fewer tokens than this runs row by row over the cache: forming the keys and values of the whole
+// context (latent attention), or filling a tile of 128 queries, does not pay for them.
 constexpr int kPromptRows = 32;
 constexpr int kPortion = 4096;      // rows of a prompt per pass
 
@@ -497,20 +629,37 @@ void stack_destroy(ForgeModel* m) {
 }
 
 // ------------------------------------------------------------------------------------------------ cache
+static size_t state_bytes(const StackModel& S, const LayerSpec& L) { return L.has_state() ? L.rec.state_values() * 4 : 0; }
+static size_t ring_bytes(const StackModel& S, const LayerSpec& L) { return L.has_state() ? L.rec.ring_values() * dense_size(S.dtype) : 0; }
+static size_t prev_bytes(const StackModel& S, const LayerSpec& L) { return L.kind == Mixer::AttnTimeMix ? size_t(S.spec.width) * dense_size(S.dtype) : 0; }
+
 int32_t stack_cache_create(ForgeKV* kv) {
     ForgeModel* m = kv->model;
     StackModel& S = *m->stack;
     FORGE_TRY(ensure_rope(m, kv->max_seq));
     kv->stack = new StackCache();
-    kv->stack->runs.resize(S.spec.layers.size());
-    const size_t rows = size_t(kv->num_pages) * FORGE_KV_PAGE;
-    for (size_t i = 0; i < S.spec.layers.size(); ++i) {
-        const LatentDims& d = S.spec.layers[i].mix;
+    kv->stack->runs.resize(S.spec.runs.size());
+    const size_t rows = size_t(kv->num_pages) * FORGE_KV_PAGE, slots = size_t(kv->batch);
+    auto alloc = [&](auto** p, size_t bytes) -> int32_t {
+        if (!bytes) return FORGE_OK;
+        void* q = nullptr;
+        FORGE_CUDA(cudaMalloc(&q, bytes));
+        *p = static_cast<std::remove_reference_t<decltype(**p)>*>(q);
+        FORGE_CUDA(cudaMemsetAsync(q, 0, bytes, m->stream));
+        return FORGE_OK;
+    };
+    for (size_t i = 0; i < S.spec.runs.size(); ++i) {
+        const LayerSpec& L = S.spec.layers[S.spec.runs[i].layer];
         StackCache::Run& r = kv->stack->runs[i];
-        const size_t bytes = rows * d.row() * dense_size(S.dtype);
-        FORGE_CUDA(cudaMalloc(&r.pool, bytes));
-        FORGE_CUDA(cudaMemsetAsync(r.pool, 0, bytes, m->stream));
-        if (tensor_core_rows(S, d)) FORGE_TRY(latent_cache_map(r.map, r.pool, d, rows));
+        char *pool = nullptr, *ring = nullptr, *prev = nullptr;
+        FORGE_TRY(alloc(&pool, rows * L.cache_row() * dense_size(S.dtype)));
+        r.pool = pool;
+        if (L.has_latent() && tensor_core_rows(S, L.mix)) FORGE_TRY(latent_cache_map(r.map, r.pool, L.mix, rows));
+        FORGE_TRY(alloc(&r.state, slots * state_bytes(S, L)));
+        FORGE_TRY(alloc(&ring, slots * ring_bytes(S, L)));
+        r.ring = ring;
+        FORGE_TRY(alloc(&prev, slots * prev_bytes(S, L)));
+        r.prev = prev;
     }
     kv->stack->splits = row_splits(S, kv->batch, kv->pages_per_seq);
     return FORGE_OK;
@@ -518,25 +667,43 @@ int32_t stack_cache_create(ForgeKV* kv) {
 
 void stack_cache_destroy(ForgeKV* kv) {
     if (!kv->stack) return;
-    for (StackCache::Run& r : kv->stack->runs) if (r.pool) cudaFree(r.pool);
+    for (StackCache::Run& r : kv->stack->runs) for (void* p : {r.pool, static_cast<void*>(r.state), r.ring, r.prev}) if (p) cudaFree(p);
     delete kv->stack;
     kv->stack = nullptr;
 }
 
-int32_t stack_kv_read(ForgeKV* kv, int seq, int layer, int which, float* out_host) {
+bool stack_has_state(const ForgeModel* m) {
+    for (const LayerSpec& L : m->stack->spec.layers) if (L.has_state()) return true;
+    return false;
+}
+
+int stack_kv_width(const ForgeKV* kv, int run, int which) {
+    const StackModel& S = *kv->model->stack;
+    const LayerSpec& L = S.spec.layers[S.spec.runs[run].layer];
+    if (L.has_latent()) return which ? L.mix.rot : L.mix.rank;
+    return L.has_attn() ? L.attn.groups * (which ? L.attn.vdim : L.attn.dim) : 0;
+}
+
+int32_t stack_kv_read(ForgeKV* kv, int seq, int run, int which, float* out_host) {
     ForgeModel* m = kv->model;
     const StackModel& S = *m->stack;
-    const LatentDims& d = S.spec.layers[layer].mix;
-    const int len = kv->len[seq], n = which ? d.rot : d.rank, col = which ? d.rank_p : 0;
-    const size_t es = dense_size(S.dtype), row = size_t(d.row()) * es;
+    const LayerSpec& L = S.spec.layers[S.spec.runs[run].layer];
+    const int n = stack_kv_width(kv, run, which), len = kv->len[seq];
+    if (n == 0) return FORGE_OK;
+    auto column = [&](int i) {
+        if (L.has_latent()) return (which ? L.mix.rank_p : 0) + i;
+        const AttnDims& a = L.attn;
+        return which ? a.groups * a.dim_p + i / a.vdim * a.vdim_p + i % a.vdim : i / a.dim * a.dim_p + i % a.dim;
+    };
+    const size_t es = dense_size(S.dtype), row = size_t(L.cache_row()) * es;
     std::vector<uint8_t> page(row * FORGE_KV_PAGE);
     for (int t0 = 0; t0 < len; t0 += FORGE_KV_PAGE) {
         const int pg = kv->h_page_table[size_t(seq) * kv->pages_per_seq + t0 / FORGE_KV_PAGE];
-        FORGE_CUDA(cudaMemcpyAsync(page.data(), static_cast<char*>(kv->stack->runs[layer].pool) + size_t(pg) * page.size(), page.size(), cudaMemcpyDeviceToHost, m->stream));
+        FORGE_CUDA(cudaMemcpyAsync(page.data(), static_cast<char*>(kv->stack->runs[run].pool) + size_t(pg) * page.size(), page.size(), cudaMemcpyDeviceToHost, m->stream));
         FORGE_CUDA(cudaStreamSynchronize(m->stream));
         for (int t = t0; t < std::min(len, t0 + FORGE_KV_PAGE); ++t)
             for (int i = 0; i < n; ++i) {
-                const uint8_t* p = page.data() + (t - t0) * row + (col + i) * es;
+                const uint8_t* p = page.data() + (t - t0) * row + column(i) * es;
                 float& v = out_host[size_t(t) * n + i];
                 if (es == 4) memcpy(&v, p, 4);
                 else { uint16_t h; memcpy(&h, p, 2); const uint32_t u = uint32_t(h) << 16; memcpy(&v, &u, 4); }
@@ -545,25 +712,52 @@ int32_t stack_kv_read(ForgeKV* kv, int seq, int layer, int which, float* out_hos
     return FORGE_OK;
 }
 
+size_t stack_state_values(const ForgeKV* kv, int run) {
+    const StackModel& S = *kv->model->stack;
+    return state_bytes(S, S.spec.layers[S.spec.runs[run].layer]) / 4;
+}
+int32_t stack_state_read(ForgeKV* kv, int seq, int run, float* out_host) {
+    const size_t n = stack_state_values(kv, run);
+    if (n == 0) return FORGE_OK;
+    if (kv->len[seq] == 0) { std::fill(out_host, out_host + n, 0.f); return FORGE_OK; }   // what a slot holds then counts as zero
+    FORGE_CUDA(cudaMemcpyAsync(out_host, kv->stack->runs[run].state + size_t(seq) * n, n * 4, cudaMemcpyDeviceToHost, kv->model->stream));
+    FORGE_CUDA(cudaStreamSynchronize(kv->model->stream));
+    return FORGE_OK;
+}
+
 size_t stack_kv_bytes_per_token(const ForgeKV* kv) {
     const StackModel& S = *kv->model->stack;
     size_t n = 0;
-    for (const LayerSpec& L : S.spec.layers) n += L.mix.row();
+    for (const LayerRun& r : S.spec.runs) n += S.spec.layers[r.layer].cache_row();
     return n * dense_size(S.dtype);
+}
+size_t stack_kv_bytes_per_seq(const ForgeKV* kv) {
+    const StackModel& S = *kv->model->stack;
+    size_t n = 0;
+    for (const LayerRun& r : S.spec.runs) { const LayerSpec& L = S.spec.layers[r.layer]; n += state_bytes(S, L) + ring_bytes(S, L) + prev_bytes(S, L); }
+    return n;
 }
 
 int32_t stack_kv_copy(ForgeKV* kv, int seq, int len, char* host, bool to_host) {
     ForgeModel* m = kv->model;
     const StackModel& S = *m->stack;
-    for (size_t l = 0; l < S.spec.layers.size(); ++l) {
-        const size_t row = size_t(S.spec.layers[l].mix.row()) * dense_size(S.dtype);
-        for (int t0 = 0; t0 < len; t0 += FORGE_KV_PAGE) {
+    auto copy = [&](char* dev, size_t bytes) -> int32_t {
+        if (!bytes) return FORGE_OK;
+        FORGE_CUDA(to_host ? cudaMemcpyAsync(host, dev, bytes, cudaMemcpyDeviceToHost, m->stream) : cudaMemcpyAsync(dev, host, bytes, cudaMemcpyHostToDevice, m->stream));
+        host += bytes;
+        return FORGE_OK;
+    };
+    for (size_t l = 0; l < S.spec.runs.size(); ++l) {
+        const LayerSpec& L = S.spec.layers[S.spec.runs[l].layer];
+        const StackCache::Run& r = kv->stack->runs[l];
+        const size_t row = size_t(L.cache_row()) * dense_size(S.dtype);
+        for (int t0 = 0; row && t0 < len; t0 += FORGE_KV_PAGE) {
             const int pg = kv->h_page_table[size_t(seq) * kv->pages_per_seq + t0 / FORGE_KV_PAGE];
-            char* dev = static_cast<char*>(kv->stack->runs[l].pool) + size_t(pg) * FORGE_KV_PAGE * row;
-            const size_t bytes = row * std::min(FORGE_KV_PAGE, len - t0);
-            FORGE_CUDA(to_host ? cudaMemcpyAsync(host, dev, bytes, cudaMemcpyDeviceToHost, m->stream) : cudaMemcpyAsync(dev, host, bytes, cudaMemcpyHostToDevice, m->stream));
-            host += bytes;
+            FORGE_TRY(copy(static_cast<char*>(r.pool) + size_t(pg) * FORGE_KV_PAGE * row, row * std::min(FORGE_KV_PAGE, len - t0)));
         }
+        FORGE_TRY(copy(reinterpret_cast<char*>(r.state) + size_t(seq) * state_bytes(S, L), state_bytes(S, L)));
+        FORGE_TRY(copy(static_cast<char*>(r.ring) + size_t(seq) * ring_bytes(S, L), ring_bytes(S, L)));
+        FORGE_TRY(copy(static_cast<char*>(r.prev) + size_t(seq) * prev_bytes(S, L), prev_bytes(S, L)));
     }
     FORGE_CUDA(cudaStreamSynchronize(m->stream));
     return FORGE_OK;
@@ -574,24 +768,31 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
                    int trace_rows, int trace_row0) {
     StackModel& S = *m->stack;
     bool prompt_ok = S.dtype == FORGE_BF16;
-    for (const LayerSpec& L : S.spec.layers) prompt_ok = prompt_ok && attn_prefill_kv_supported(L.mix);
-    // rows: the short entries first, then the prompt portions
+    for (const LayerSpec& L : S.spec.layers)
+        prompt_ok = prompt_ok && (L.has_latent() ? attn_prefill_kv_supported(PromptDims(L.mix)) : !L.has_attn() || attn_prefill_kv_supported(PromptDims(L.attn)));
+    // rows: the single tokens first, then the short entries, then the prompt portions
     struct Place { int row, tok, want; };
     std::vector<Place> at_entry(n_entries);
-    int tok = 0, wants = 0, rows = 0, single = 0, max_pages = 1;
+    int tok = 0, wants = 0, rows = 0, ones = 0, single = 0, max_keys = 1;
     for (int i = 0; i < n_entries; ++i) { at_entry[i] = {0, tok, wants}; tok += entries[i].n_tokens; wants += entries[i].n_want; }
     auto is_prompt = [&](int i) { return prompt_ok && entries[i].n_tokens >= kPromptRows; };
-    for (int pass = 0; pass < 2; ++pass)
+    auto pass_of = [&](int i) { return is_prompt(i) ? 2 : entries[i].n_tokens > 1 ? 1 : 0; };
+    for (int pass = 0; pass < 3; ++pass) {
         for (int i = 0; i < n_entries; ++i)
-            if (is_prompt(i) == (pass == 1)) {
+            if (pass_of(i) == pass) {
                 at_entry[i].row = rows;
                 rows += entries[i].n_tokens;
-                if (pass == 0) { single = rows; max_pages = std::max(max_pages, (kv->len[entries[i].seq] + entries[i].n_tokens + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE); }
+                if (pass < 2) max_keys = std::max(max_keys, kv->len[entries[i].seq] + entries[i].n_tokens);
             }
-    // one upload: tokens | positions | sequences | wanted rows | context pages | prompt tiles
+        if (pass == 0) ones = rows;
+        if (pass < 2) single = rows;
+    }
+    // one upload: tokens | positions | sequences | wanted rows | context pages | prompt tiles | segments
     std::vector<int32_t> meta(size_t(3) * rows + wants);
     std::vector<int32_t> pages;
     std::vector<PromptTile> tiles;
+    std::vector<ScanSeg> segs;
+    int max_seg = 0;
     for (int i = 0; i < n_entries; ++i) {
         const ForgeStepEntry& e = entries[i];
         const int base = kv->len[e.seq], r0 = at_entry[i].row;
@@ -601,6 +802,7 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
             meta[2 * rows + r0 + k] = e.seq;
         }
         for (int k = 0; k < e.n_want; ++k) meta[3 * rows + at_entry[i].want + k] = r0 + want[at_entry[i].want + k];
+        if (e.n_tokens > 1) { segs.push_back({r0, e.n_tokens, e.seq, base}); max_seg = std::max(max_seg, int(e.n_tokens)); }
         if (is_prompt(i)) {
             const int ctx0 = int(pages.size()) * FORGE_KV_PAGE, np = (base + e.n_tokens + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE;
             for (int p = 0; p < np; ++p) pages.push_back(kv->h_page_table[size_t(e.seq) * kv->pages_per_seq + p]);
@@ -608,12 +810,13 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
         }
     }
     std::stable_sort(tiles.begin(), tiles.end(), [](const PromptTile& a, const PromptTile& b) { return a.pos0 + a.rows > b.pos0 + b.rows; });   // the longest first
-    const size_t o_pages = (meta.size() + 3) & ~size_t(3), o_tiles = (o_pages + pages.size() + 3) & ~size_t(3), total = o_tiles + tiles.size() * 4;
+    const size_t o_pages = (meta.size() + 3) & ~size_t(3), o_tiles = (o_pages + pages.size() + 3) & ~size_t(3), o_segs = o_tiles + tiles.size() * 4, total = o_segs + segs.size() * 4;
     meta.resize(total);
     std::copy(pages.begin(), pages.end(), meta.begin() + o_pages);
     if (!tiles.empty()) memcpy(meta.data() + o_tiles, tiles.data(), tiles.size() * sizeof(PromptTile));
-    const int splits = row_splits(S, std::max(1, single), max_pages), ctx_rows = int(pages.size()) * FORGE_KV_PAGE;
-    FORGE_TRY(ensure_step(m, std::max(rows, wants), single, splits, rows - single, ctx_rows));
+    if (!segs.empty()) memcpy(meta.data() + o_segs, segs.data(), segs.size() * sizeof(ScanSeg));
+    const int splits = row_splits(S, std::max(1, single), (max_keys + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE), ctx_rows = int(pages.size()) * FORGE_KV_PAGE;
+    FORGE_TRY(ensure_step(m, std::max(rows, wants), single, splits, rows - single, ctx_rows, rows - ones));
     FORGE_TRY(grow(m, S.meta, total * 4));
     FORGE_TRY(grow(m, S.sel, size_t(wants) * S.width_p * dense_size(S.dtype)));
     FORGE_TRY(grow(m, S.logits, size_t(wants) * S.spec.vocab * 4));
@@ -623,11 +826,12 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
     s.tokens = reinterpret_cast<const uint32_t*>(dm);
     s.rows = StepRows{rows, dm + rows, dm + 2 * rows, kv->d_page_table, kv->pages_per_seq};
     for (int i = 0; i < n_entries; ++i) if (!is_prompt(i)) s.rows.fresh = std::max(s.rows.fresh, int(entries[i].n_tokens));
-    s.single = single; s.splits = splits;
+    s.ones = ones; s.single = single; s.splits = splits; s.max_keys = max_keys;
+    s.segs = reinterpret_cast<const ScanSeg*>(dm + o_segs); s.n_segs = int(segs.size()); s.max_seg = max_seg;
     s.ctx_pages = dm + o_pages; s.ctx_rows = ctx_rows;
     s.tiles = reinterpret_cast<const PromptTile*>(dm + o_tiles); s.n_tiles = int(tiles.size());
     if (trace_rows) { s.trace = m->trace + size_t(trace_row0) * S.spec.width; s.trace_stride = size_t(trace_rows) * S.spec.width; }
-    FORGE_TRY(run_layers(m, kv, s));
+    FORGE_TRY(Sequence(m, kv, s).run());
     if (wants) {
         FORGE_TRY(gather_act_rows(S.sel.p, S.h.p, dm + 3 * rows, wants, S.width_p, S.dtype, m->stream));
         FORGE_TRY(run_head(m, S.sel.p, wants, static_cast<float*>(S.logits.p)));
@@ -651,21 +855,22 @@ int32_t stack_prefill(ForgeModel* m, ForgeKV* kv, int seq, const uint32_t* token
         if (rc == FORGE_OK && last && cudaMemcpyAsync(m->d_logits, lg, sizeof(float) * m->V, cudaMemcpyDeviceToDevice, m->stream) != cudaSuccess) { set_error("logits copy failed"); rc = FORGE_ERR_CUDA; }
         if (rc == FORGE_OK) kv->len[seq] += k;
     }
-    if (rc != FORGE_OK) kv->len[seq] = len0;
+    if (rc != FORGE_OK) { kv->len[seq] = len0; mark_lost(kv); }
     return rc;
 }
 
-int32_t stack_ensure_decode(ForgeModel* m, ForgeKV* kv, int batch) { return ensure_step(m, batch, batch, kv->stack->splits, 0, 0); }
+int32_t stack_ensure_decode(ForgeModel* m, ForgeKV* kv, int batch) { return ensure_step(m, batch, batch, kv->stack->splits, 0, 0, 0); }
 
 int32_t stack_decode_launches(ForgeModel* m, ForgeKV* kv, int batch, bool greedy, bool record) {
     StackModel& S = *m->stack;
     Step s;
     s.tokens = m->d_tok;
     s.rows = StepRows{batch, kv->d_seq_len, nullptr, kv->d_page_table, kv->pages_per_seq};
-    s.single = batch; s.splits = kv->stack->splits;
+    s.rows.slot0 = kv->slot0;
+    s.ones = s.single = batch; s.splits = kv->stack->splits; s.max_keys = kv->max_seq;
     if (record) { s.hist = m->d_hist; s.step = m->d_step; }
     if (m->trace_on) { s.trace = m->trace; s.trace_stride = size_t(batch) * S.spec.width; }
-    FORGE_TRY(run_layers(m, kv, s));
+    FORGE_TRY(Sequence(m, kv, s).run());
     FORGE_TRY(run_head(m, S.h.p, batch, m->d_logits));
     if (greedy) FORGE_TRY(argmax_slices(m->d_tok, m->d_logits, m->V, batch, m->d_amax_val, m->d_amax_idx, m->d_amax_ticket, m->stream));
     return step_advance(kv->d_seq_len, batch, m->d_step, m->stream);
@@ -676,23 +881,10 @@ int32_t stack_decode_launches(ForgeModel* m, ForgeKV* kv, int batch, bool greedy
 // ------------------------------------------------------------------------------------------------ C API
 extern "C" {
 
-int32_t forge_checkpoint_info(const char* dir, ForgeCheckpointInfo* out) {
-    if (!dir || !out) { set_error("bad argument to forge_checkpoint_info"); return FORGE_ERR_INVALID_ARG; }
-    Checkpoint ck;
-    StackSpec s;
-    StackTensors t;
-    FORGE_TRY(ck.open(dir));
-    FORGE_TRY(parse_spec(ck.config(), &s));
-    FORGE_TRY(find_tensors(ck, s, &t));
-    s.parameters = ck.parameters();
-    fill_info(s, out);
-    return FORGE_OK;
-}
-
 int32_t forge_model_info(const ForgeModel* m, ForgeCheckpointInfo* out) {
     if (!m || !out) { set_error("bad argument to forge_model_info"); return FORGE_ERR_INVALID_ARG; }
     if (!m->stack) { set_error("not a layer-list model"); return FORGE_ERR_UNSUPPORTED; }
-    fill_info(m->stack->spec, out);
+    stack_fill_info(m->stack->spec, out);
     return FORGE_OK;
 }
 
@@ -704,8 +896,8 @@ int32_t forge_model_open(const char* dir, int32_t dtype, int32_t device, ForgeMo
     StackSpec spec;
     StackTensors t;
     FORGE_TRY(ck.open(dir));
-    FORGE_TRY(parse_spec(ck.config(), &spec));
-    FORGE_TRY(find_tensors(ck, spec, &t));
+    FORGE_TRY(stack_parse(ck.config(), &spec));
+    FORGE_TRY(stack_find_tensors(ck, &spec, &t));
     spec.parameters = ck.parameters();
     const int ndev = forge_device_count();
     if (ndev == 0) { set_error("no CUDA device: this backend has no CPU fallback"); return FORGE_ERR_CUDA; }
@@ -713,7 +905,7 @@ int32_t forge_model_open(const char* dir, int32_t dtype, int32_t device, ForgeMo
     FORGE_CUDA(cudaSetDevice(device));
     ForgeModel* m = new ForgeModel();
     m->cfg = ForgeModelConfig{};
-    m->cfg.hidden_size = spec.width; m->cfg.num_layers = int32_t(spec.layers.size()); m->cfg.vocab_size = spec.vocab;
+    m->cfg.hidden_size = spec.width; m->cfg.num_layers = int32_t(spec.runs.size()); m->cfg.vocab_size = spec.vocab;
     m->cfg.max_seq_len = 1 << 20; m->cfg.tp_world = 1; m->cfg.quant = dtype;
     m->device = device; m->h = spec.width; m->V = spec.vocab; m->max_seq = 1 << 20;
     m->uniform_basic = false;
@@ -729,15 +921,24 @@ int32_t forge_model_open(const char* dir, int32_t dtype, int32_t device, ForgeMo
         const size_t es = dense_size(dtype);
         {
             std::vector<uint8_t> img(size_t(spec.vocab) * spec.width * es);
-            put_rows(img, dtype, spec.width, *t.embed, 0);
+            put_rows(img, dtype, spec.width, *t.top.at("embed"), 0);
             FORGE_TRY(upload(m, &S.embed, img));
         }
         {
-            std::vector<uint8_t> img(size_t(spec.vocab) * S.width_p * es, 0);
-            put_rows(img, dtype, S.width_p, *t.head, 0);
-            FORGE_TRY(load_dense(m, &S.head, spec.vocab, S.width_p, dtype, img));
+            Image head(spec.vocab, S.width_p, dtype);
+            head.put(t.top.at("head"), 0);
+            FORGE_TRY(head.load(m, &S.head));
         }
-        FORGE_TRY(load_dyt(m, &S.final_norm, *t.fn, *t.fb, *t.fa));
+        if (spec.loop_times) {   // columns [stream | embedding], each padded
+            const TensorView& in = *t.top.at("loop.in");
+            Image img(spec.width, 2 * S.width_p, dtype);
+            for (int r = 0; r < spec.width; ++r)
+                for (int c = 0; c < 2 * spec.width; ++c)
+                    store(img.img.data(), dtype, size_t(r) * img.K + (c < spec.width ? c : S.width_p + c - spec.width), in, size_t(r) * 2 * spec.width + c);
+            FORGE_TRY(img.load(m, &S.loop_in));
+            FORGE_TRY(upload_f32(m, &S.loop_step, *t.top.at("loop.step")));
+        }
+        FORGE_TRY(load_norm(m, &S.final_norm, t.top, "final.norm"));
         S.w.resize(spec.layers.size());
         for (size_t i = 0; i < spec.layers.size(); ++i)
             if (spec.layers[i].weights_of < 0) FORGE_TRY(load_layer(m, spec.layers[i], t.layers[i], &S.w[i]));

@@ -89,13 +89,15 @@ class KVCache:
         return int(lib.forge_kv_len(self._h, seq))
 
     def read(self, layer: int, which: int, seq: int = 0) -> np.ndarray:
-        if "layers" in self.model.cfg:   # latents (which = 0) or rotated key parts (1)
-            m = self.model.cfg["layers"][layer]["mixer"]
-            kvd = m["rot_dim"] if which else m["kv_rank"]
-        else:
-            kvd = self.model.cfg["num_kv_heads"] * self.model.cfg["head_dim"] // self.model.tp_world
-        out = np.empty((self.len(seq), kvd), np.float32)
+        out = np.empty((self.len(seq), lib.forge_kv_width(self._h, layer, which)), np.float32)
         check(lib.forge_kv_read(self._h, seq, layer, which, _p(out)))
+        return out
+
+    def read_state(self, layer: int, seq: int = 0) -> np.ndarray:
+        """A recurrent layer run's state, flat [heads * dim * vdim] (empty if it has none)."""
+        out = np.empty(int(lib.forge_kv_state_values(self._h, layer)), np.float32)
+        if out.size:
+            check(lib.forge_kv_state_read(self._h, seq, layer, _p(out)))
         return out
 
     def save(self, seq: int = 0) -> np.ndarray:
@@ -129,7 +131,8 @@ def checkpoint_info(path: str) -> dict:
     i = ForgeCheckpointInfo()
     check(lib.forge_checkpoint_info(os.fsencode(path), C.byref(i)))
     return {"architecture": i.architecture.decode(), "hidden_size": i.hidden_size, "vocab_size": i.vocab_size, "num_layers": i.num_layers,
-            "num_weight_layers": i.num_weight_layers, "parameters": i.parameters, "cache_values_per_token": i.cache_values_per_token}
+            "num_weight_layers": i.num_weight_layers, "parameters": i.parameters, "cache_values_per_token": i.cache_values_per_token,
+            "state_values_per_sequence": i.state_values_per_sequence}
 
 
 TP_ID_BYTES = 128  # FORGE_TP_ID_BYTES

@@ -226,7 +226,8 @@ void* forge_model_stream(ForgeModel* model);
  * and lists the layers, each with its mixer, the mixer's sizes and its feed-forward; sizes and constants are read from
  * there.  Every session call below takes such a model like any other.  (No counterpart in the reference, whose models are
  * GGUF decoders.)  Registered architectures: "Bolenex" (latent attention and a clamped gated feed-forward in parallel behind
- * one Dynamic Tanh norm).  An unknown architecture, mixer or feed-forward returns FORGE_ERR_UNSUPPORTED; a missing key, a
+ * one Dynamic Tanh norm), "Robazen" (gated delta rules, with one decay per head or per key channel, and pairs of chunked attention
+ * and time mixing, a SiLU-gated feed-forward behind its own norm, and a range of layers that may run several times).  An unknown architecture, mixer or feed-forward returns FORGE_ERR_UNSUPPORTED; a missing key, a
  * missing tensor or a wrong shape FORGE_ERR_SHAPE. */
 typedef struct ForgeCheckpointInfo {
     char architecture[64];
@@ -236,6 +237,7 @@ typedef struct ForgeCheckpointInfo {
     int32_t num_weight_layers;       /* layers with tensors of their own */
     int64_t parameters;              /* values in the checkpoint's tensors */
     int64_t cache_values_per_token;  /* values the cache keeps per position, padding included */
+    int64_t state_values_per_sequence; /* values of the recurrent states, independent of the length */
 } ForgeCheckpointInfo;
 /* Reads and checks a checkpoint folder without a device. */
 int32_t forge_checkpoint_info(const char* dir, ForgeCheckpointInfo* out);
@@ -305,8 +307,15 @@ int32_t forge_kv_len(const ForgeKV* kv, int32_t seq);
 void forge_kv_destroy(ForgeKV* kv);
 /* Copy K (which = 0) or V (1) rows [0, len) of `layer`, sequence `seq`, widened to f32, into
  * a host buffer [len][num_kv_heads*head_dim] (used by parity tests).  Latent attention: the latents (0, [len][kv_rank]) or
- * the rotated key parts (1, [len][rot_dim]). */
+ * the rotated key parts (1, [len][rot_dim]).  A layer without cache rows gives nothing. */
 int32_t forge_kv_read(ForgeKV* kv, int32_t seq, int32_t layer, int32_t which, float* out_host);
+/* Values per position forge_kv_read gives; -1 on a bad argument. */
+int32_t forge_kv_width(const ForgeKV* kv, int32_t layer, int32_t which);
+/* Recurrent state of a sequence in a layer run, f32 [heads][dim][vdim]: number of values (0: the run has none; -1: bad argument)
+ * and a copy.  When a step fails after it has begun (FORGE_ERR_TIMEOUT), the states of all sequences that hold one are undefined:
+ * forwards of these sequences then return FORGE_ERR_INVALID_ARG until forge_kv_free_seq, forge_kv_reset or forge_kv_load. */
+int64_t forge_kv_state_values(const ForgeKV* kv, int32_t layer);
+int32_t forge_kv_state_read(ForgeKV* kv, int32_t seq, int32_t layer, float* out_host);
 
 /* KV cache persistence (save_kv_cache / load_kv_cache of the generated main.rs, project.rs:456-499).
  * forge_kv_save writes sequence `seq` as {"FKV1", u32 layers, u32 kv_width, u64 len} followed by the K rows of every

@@ -1,6 +1,9 @@
 """Plain restatement of the layer-list models (a ``config.json`` whose "layers" entry lists mixers and feed-forwards):
-one function per mechanism, numpy, written from the equations, slow on purpose.  The Bolenex design: latent attention
-and a clamped gated feed-forward in parallel behind one Dynamic Tanh norm.
+one function per mechanism, numpy, written from the equations, slow on purpose.
+
+Bolenex: latent attention and a clamped gated feed-forward in parallel behind one Dynamic Tanh norm.
+Robazen: mixer and feed-forward one after the other, each behind its own Dynamic Tanh norm; mixers are gated delta rules (one
+decay per head or per key channel) and a pair of chunked attention and time mixing; some layers run several times.
 
 TEST INFRASTRUCTURE ONLY, like the rest of this folder; it shares no code with the shipped package.  Everything is computed in
 ``dtype`` (float64 by default).  A sequence is evaluated as a whole: there is no cache, no page and no batch here.
@@ -88,6 +91,144 @@ def dense_ff(h, w, m):
     return clamped_glu(h @ w("gate").T, h @ w("up").T, h.dtype.type(m["limit"])) @ w("down").T
 
 
+# ------------------------------------------------------------------------------------ recurrent mixers and their neighbours
+def silu(z):
+    return z * sigmoid(z)
+
+
+def softplus(z):
+    return np.maximum(z, 0.0) + np.log1p(np.exp(-np.abs(z)))
+
+
+def short_convolution(x, taps):
+    """Causal, per channel: y[t, c] = sum_j taps[c, j] x[t - (n - 1 - j), c], zeros before the start.  x: [tokens, channels]."""
+    n = taps.shape[1]
+    y = np.zeros_like(x)
+    for t in range(x.shape[0]):
+        for j in range(n):
+            s = t - (n - 1 - j)
+            if s >= 0:
+                y[t] += taps[:, j] * x[s]
+    return y
+
+
+def unit(x, eps=1e-6):
+    return x / np.sqrt((x * x).sum(-1, keepdims=True) + eps)
+
+
+def delta_rule(q, k, v, beta, g):
+    """Token by token: the state decays, is corrected towards v at k, and is read at q behind the write.
+    q, k: [tokens, heads, d], v: [tokens, heads, dv], beta: [tokens, heads], g: [tokens, heads, d] (rows of the state)."""
+    n, heads, d = q.shape
+    out = np.zeros_like(v)
+    for h in range(heads):
+        S = np.zeros((d, v.shape[2]), q.dtype)
+        for t in range(n):
+            S = g[t, h][:, None] * S
+            u = beta[t, h] * (v[t, h] - S.T @ k[t, h])
+            S = S + np.outer(k[t, h], u)
+            out[t, h] = S.T @ q[t, h]
+    return out
+
+
+def _delta_inputs(h, w, m):
+    n, H, G, d, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q, k, v = (silu(short_convolution(h @ w(t).T, w(t + ".conv"))) for t in "qkv")
+    head = np.arange(H) // (H // G)
+    q = unit(q.reshape(n, G, d))[:, head] * d ** -0.5
+    k = unit(k.reshape(n, G, d))[:, head]
+    return q, k, v.reshape(n, H, dv), sigmoid(h @ w("b").T)
+
+
+def gated_delta(h, w, m, eps):
+    q, k, v, beta = _delta_inputs(h, w, m)
+    n, H, dv = v.shape
+    g = np.exp(-np.exp(w("A_log")) * softplus(h @ w("a").T + w("dt_bias")))
+    o = delta_rule(q, k, v, beta, np.broadcast_to(g[:, :, None], k.shape))
+    o = rms_norm(o, w("norm"), eps) * silu(h @ w("g").T).reshape(n, H, dv)
+    return o.reshape(n, H * dv) @ w("o").T
+
+
+def channel_delta(h, w, m, eps):
+    q, k, v, beta = _delta_inputs(h, w, m)
+    n, H, dv = v.shape
+    z = ((h @ w("a1").T) @ w("a2").T + w("dt_bias")).reshape(n, H, m["dim"])
+    o = delta_rule(q, k, v, beta, np.exp(-np.exp(w("A_log"))[None, :, None] * softplus(z)))
+    o = rms_norm(o, w("norm"), eps) * sigmoid((h @ w("g1").T) @ w("g2").T).reshape(n, H, dv)
+    return o.reshape(n, H * dv) @ w("o").T
+
+
+def chunked_attention(q, k, v, scale, softcap, chunk):
+    """q: [tokens, heads, d], k: [tokens, kv heads, d], v: [tokens, kv heads, dv]; position i sees the keys j <= i of its own chunk."""
+    n, H, _ = q.shape
+    G = k.shape[1]
+    out = np.zeros((n, H, v.shape[2]), q.dtype)
+    for h in range(H):
+        kh, vh = k[:, h // (H // G)], v[:, h // (H // G)]
+        for i in range(n):
+            j0 = i // chunk * chunk
+            s = kh[j0:i + 1] @ q[i, h] * q.dtype.type(scale)
+            s = softcap * np.tanh(s / softcap)
+            e = np.exp(s - s.max())
+            out[i, h] = (e / e.sum()) @ vh[j0:i + 1]
+    return out
+
+
+def gated_attention(h, w, m):
+    n, H, G = h.shape[0], m["heads"], m["kv_heads"]
+    o = chunked_attention((h @ w("q").T).reshape(n, H, m["dim"]), (h @ w("k").T).reshape(n, G, m["dim"]), (h @ w("v").T).reshape(n, G, m["vdim"]),
+                          m["scale"], m["softcap"], m["mask"]["size"])
+    o = o * sigmoid(h @ w("g").T)[:, :, None]
+    return o.reshape(n, H * m["vdim"]) @ w("o").T
+
+
+def token_shift(h, mu):
+    """h + (h' - h) mu with h' the row before (zeros in front of the first)."""
+    before = np.concatenate([np.zeros_like(h[:1]), h[:-1]])
+    return h + (before - h) * mu
+
+
+def time_mixing(h, w, m, eps):
+    n, H, d = h.shape[0], m["heads"], m["dim"]
+    r, k, v = ((token_shift(h, w("mu." + s)) @ w(s).T).reshape(n, H, d) for s in "rkv")
+    gate = silu(token_shift(h, w("mu.g")) @ w("g").T)
+    dec = np.exp(-np.exp(np.tanh(token_shift(h, w("mu.w")) @ w("w1").T) @ w("w2").T + w("w0"))).reshape(n, H, d)
+    o = np.zeros_like(v)
+    for i in range(H):
+        S = np.zeros((d, d), h.dtype)
+        for t in range(n):
+            o[t, i] = S.T @ r[t, i] + (r[t, i] * w("u")[i] * k[t, i]).sum() * v[t, i]
+            S = dec[t, i][:, None] * S + np.outer(k[t, i], v[t, i])
+    o = rms_norm(o, 1.0, eps).reshape(n, H * d) * w("norm") * gate
+    return o @ w("o").T
+
+
+def parallel_pair(h, w, m, eps):
+    left = gated_attention(h, lambda t: w("left." + t), m["left"])
+    right = time_mixing(h, lambda t: w("right." + t), m["right"], eps)
+    return 0.5 * (rms_norm(left, w("left.out"), eps) + rms_norm(right, w("right.out"), eps))
+
+
+def silu_glu_ff(h, w):
+    return (silu(h @ w("gate").T) * (h @ w("up").T)) @ w("down").T
+
+
+def mixer_of(kind, h, w, m, eps):
+    if kind == "latent_attention":
+        return latent_attention(h, w, m, eps)
+    return {"delta": gated_delta, "channel_delta": channel_delta, "parallel": parallel_pair}[kind](h, w, m, eps)
+
+
+def layer_runs(cfg):
+    """[(layer, pass that starts in front of it or None)] in the order of running."""
+    n, loop = len(cfg["layers"]), cfg.get("loop")
+    if not loop:
+        return [(i, None) for i in range(n)]
+    a, b = loop["start"], loop["stop"]
+    body = [(i, t if i == a else None) for t in range(loop["times"]) for i in range(a, b)]
+    return [(i, None) for i in range(a)] + body + [(i, None) for i in range(b, n)]
+
+
 # ---------------------------------------------------------------------------------------------- the model
 class LayerStack:
     """``config``: the parsed config.json; ``tensors``: name -> array."""
@@ -103,17 +244,23 @@ class LayerStack:
     def layer(self, x, i):
         L = self.cfg["layers"][i]
         p = f"l{L.get('weights_of', i)}."
+        mix, mlp = (lambda n: self.t[p + "mix." + n]), (lambda n: self.t[p + "mlp." + n])
         h = self.norm(x, p + "norm1")
-        y = latent_attention(h, lambda n: self.t[p + "mix." + n], L["mixer"], self.cfg["norm"]["eps"])
-        if L.get("mlp"):
-            y = y + dense_ff(h, lambda n: self.t[p + "mlp." + n], L["mlp"])
-        return x + y
+        y = mixer_of(L["type"], h, mix, L["mixer"], self.cfg["norm"]["eps"])
+        if self.cfg["architecture"] == "Bolenex":
+            if L.get("mlp"):
+                y = y + dense_ff(h, mlp, L["mlp"])
+            return x + y
+        x = x + y
+        return x + silu_glu_ff(self.norm(x, p + "norm2"), mlp) if L.get("mlp") else x
 
     def residuals(self, tokens):
-        """The residual stream after every layer: [layers, tokens, width]."""
-        x = self.t["embed"][np.asarray(tokens, np.int64)]
+        """The residual stream after every layer run: [runs, tokens, width]."""
+        x0 = x = self.t["embed"][np.asarray(tokens, np.int64)]
         out = []
-        for i in range(len(self.cfg["layers"])):
+        for i, start in layer_runs(self.cfg):
+            if start is not None:
+                x = np.concatenate([x, x0], axis=1) @ self.t["loop.in"].T + self.t["loop.step"][start]
             x = self.layer(x, i)
             out.append(x)
         return np.stack(out)
