@@ -2,7 +2,7 @@
 """Benchmark of the quantized forward path on B200.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
-    python bench.py --design bolenex          (another model design, one GPU; the default workload is unchanged)
+    python bench.py --design bolenex|robazen  (another model design, one GPU; the default workload is unchanged)
 
 One GPU (the default).  Headline workload: the Llama-3.2-1B-shaped Q4_0 decoder of the benchmark definition - one
 "step" is one request: a 1501-token uniform-random prompt through the batched prefill path, then 128 greedy decode
@@ -404,10 +404,10 @@ def run_single(args, device: int):
     print(json.dumps(line), flush=True)
 
 
-# ---------------------------------------------------------------------------- one GPU: the Bolenex design beside a Llama-shaped decoder
+# ---------------------------------------------------------------------------- one GPU: a layer-list design beside a Llama-shaped decoder
 # (width, layers, heads of 128, ff): a 1B- and a 7B-shaped layer
-BOLENEX_SIZES = {"w2048": (2048, 16, 16, 8192), "w4096": (4096, 8, 32, 11008)}
-BOLENEX_VOCAB, BOLENEX_PROMPT, BOLENEX_DECODE = 32768, 2048, 64
+DESIGN_SIZES = {"w2048": (2048, 16, 16, 8192), "w4096": (4096, 8, 32, 11008)}
+DESIGN_VOCAB, DESIGN_PROMPT, DESIGN_DECODE = 32768, 2048, 64
 
 
 def bolenex_work(cfg: dict, ctx: int, m: int):
@@ -425,8 +425,38 @@ def bolenex_work(cfg: dict, ctx: int, m: int):
     return w + 2 * V * W, kv * ctx, flops + 2.0 * V * W
 
 
-def run_bolenex(args, device: int):
-    """Prefill and decode rates of the Bolenex design and, at equal width, depth, heads and feed-forward, of the framework's closest
+def robazen_work(cfg: dict, ctx: int, m: int):
+    """The same; a layer that runs twice streams its weights twice.  Per sequence: the keys and values of the chunk `ctx` lies in, and every
+    recurrent state read and written.  A recurrence counts with the products of its token-by-token form (decay aside): read-out,
+    write and, for a delta rule, the correction."""
+    from forge_llm_b200 import synth
+    W, V = cfg["width"], cfg["vocab"]
+    shapes = synth.stack_shapes(cfg)
+    loop = cfg.get("loop") or {"start": 0, "stop": 0, "times": 1}
+    w, kv, flops = 2.0 * V * W, 0.0, 2.0 * V * W
+    if loop["stop"]:
+        w += loop["times"] * 4.0 * W * W
+        flops += loop["times"] * 4.0 * W * W * m
+    for i, L in enumerate(cfg["layers"]):
+        n = loop["times"] if loop["start"] <= i < loop["stop"] else 1
+        lin = sum(s[0] * s[1] for k, s in shapes.items() if k.startswith(f"l{i}.") and len(s) == 2 and not k.endswith((".conv", ".u")))
+        x = L["mixer"]
+        rec = x["right"] if L["type"] == "parallel" else x
+        state = rec["heads"] * rec["dim"] * rec.get("vdim", rec["dim"])
+        w += n * 2.0 * lin
+        kv += n * 8.0 * state
+        flops += n * (2.0 * m * lin + (4.0 if L["type"] == "parallel" else 6.0) * m * state)
+        if L["type"] == "parallel":
+            a = x["left"]
+            c = a["mask"]["size"]
+            kv += n * 2.0 * a["kv_heads"] * (a["dim"] + a["vdim"]) * (ctx % c + 1)
+            pairs = (m // c) * c * (c + 1) / 2 + (m % c) * (m % c + 1) / 2
+            flops += n * 2.0 * a["heads"] * (a["dim"] + a["vdim"]) * pairs
+    return w, kv, flops
+
+
+def run_design(args, device: int):
+    """Prefill and decode rates of a layer-list design and, at equal width, depth, heads and feed-forward, of the framework's closest
     decoder (multi-head, head_dim 128, Q8_0), each against its own roofline."""
     import torch
     from forge_llm_b200 import configs, runtime, synth
@@ -434,6 +464,9 @@ def run_bolenex(args, device: int):
     sampler = ClockSampler(device)
     t0 = time.time()
     out, launches = {}, 0
+    design = args.design
+    make_config, work = {"bolenex": (synth.bolenex_config, bolenex_work), "robazen": (synth.robazen_config, robazen_work)}[design]
+    arm = f"{design} bf16"
 
     def measure(model, batch, n_prompt, n_dec, bytes_w, bytes_kv, flops, vocab):
         kv = model.new_cache(max_seq=n_prompt + n_dec + 8, batch=batch)
@@ -471,39 +504,39 @@ def run_bolenex(args, device: int):
                 "e2e_s_per_request": statistics.median(host) / batch}, nl
 
     for name in args.sizes.split(","):
-        width, layers, heads, ff = BOLENEX_SIZES[name]
-        n_prompt, n_dec = args.prompt_tokens or BOLENEX_PROMPT, args.decode_steps or BOLENEX_DECODE
+        width, layers, heads, ff = DESIGN_SIZES[name]
+        n_prompt, n_dec = args.prompt_tokens or DESIGN_PROMPT, args.decode_steps or DESIGN_DECODE
         if args.layers:
             layers = args.layers
         ctx = n_prompt + n_dec // 2
-        rec = {"shape": f"width {width}, {layers} layers, {heads} heads of 128, ff {ff}, vocab {BOLENEX_VOCAB}, {n_prompt}-token prompts, {n_dec} decode steps"}
+        rec = {"shape": f"width {width}, {layers} layers, {heads} heads of 128, ff {ff}, vocab {DESIGN_VOCAB}, {n_prompt}-token prompts, {n_dec} decode steps"}
         batches = [int(b) for b in args.batches.split(",")]
-        if "bolenex" in args.arms:
-            cfg = synth.bolenex_config(width, layers, heads, ff, BOLENEX_VOCAB)
-            folder = os.path.join(CACHE_DIR, f"bolenex-{width}-{layers}-{os.getpid()}")
-            synth.write_bolenex(folder, cfg)
+        if "design" in args.arms or design in args.arms:
+            cfg = make_config(width, layers, heads, ff, DESIGN_VOCAB)
+            folder = os.path.join(CACHE_DIR, f"{design}-{width}-{layers}-{os.getpid()}")
+            synth.write_stack(folder, cfg)
             model = runtime.Model.open(folder, "bfloat16", device)
             shutil.rmtree(folder)
-            rec["bolenex bf16"] = []
+            rec[arm] = []
             for b in batches:
-                r, nl = measure(model, b, n_prompt, n_dec, *bolenex_work(cfg, ctx, n_prompt), BOLENEX_VOCAB)
-                rec["bolenex bf16"].append(r)
+                r, nl = measure(model, b, n_prompt, n_dec, *work(cfg, ctx, n_prompt), DESIGN_VOCAB)
+                rec[arm].append(r)
                 launches += nl
             model.close()
         if "llama" in args.arms:
-            c = configs._cfg(f"llama-shape-{width}", width, layers, heads, heads, 128, ff, BOLENEX_VOCAB, 1e4, 8)
+            c = configs._cfg(f"llama-shape-{width}", width, layers, heads, heads, 128, ff, DESIGN_VOCAB, 1e4, 8)
             model = runtime.Model(c, synth.make_weights_bin(c, seed=0, quantize_fn=lambda q, w: runtime.quantize_q8_0(w), repeat_layers=True), device=device)
             rec["llama-shaped q8_0"] = []
             w = configs.decode_bytes_per_token(c, 0)
             for b in batches:
-                r, _ = measure(model, b, n_prompt, n_dec, w, configs.decode_bytes_per_token(c, ctx) - w, configs.prefill_flops(c, n_prompt), BOLENEX_VOCAB)
+                r, _ = measure(model, b, n_prompt, n_dec, w, configs.decode_bytes_per_token(c, ctx) - w, configs.prefill_flops(c, n_prompt), DESIGN_VOCAB)
                 rec["llama-shaped q8_0"].append(r)
             model.close()
         out[name] = rec
         print(f"[bench] {name}: {json.dumps(rec)}", file=sys.stderr, flush=True)
     clocks = sampler.stop(t0, time.time())
-    first = out[args.sizes.split(",")[0]].get("bolenex bf16", [{}])[0]
-    print(json.dumps({"metric": "bolenex_decode_tok_s", "value": first.get("decode_tok_s"), "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+    first = out[args.sizes.split(",")[0]].get(arm, [{}])[0]
+    print(json.dumps({"metric": f"{design}_decode_tok_s", "value": first.get("decode_tok_s"), "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
                       "higher_is_better": True, "dtype": "bf16", "data": "synthetic", "sizes": out, "gpu_launches": int(launches), "clocks": clocks,
                       "config": {"l2": "every decode step streams weights larger than L2 once", "parallelism": "one GPU"}}), flush=True)
 
@@ -680,11 +713,11 @@ def main():
     ap.add_argument("--prompt-tokens", type=int, default=None, help="override the headline prompt length (profiling / experiments)")
     ap.add_argument("--decode-steps", type=int, default=None, help="override the headline number of decode steps")
     ap.add_argument("--profile", action="store_true", help="short run for ncu: no side configurations, no CPU baseline; prints a non-benchmark line")
-    ap.add_argument("--design", default="headline", choices=["headline", "bolenex"], help="bolenex: the Bolenex design beside a Llama-shaped decoder of equal size (one GPU)")
-    ap.add_argument("--sizes", default="w2048,w4096", help="with --design bolenex: which sizes")
-    ap.add_argument("--batches", default="1,16", help="with --design bolenex: sequences decoded together")
-    ap.add_argument("--arms", default="bolenex,llama", help="with --design bolenex: which models")
-    ap.add_argument("--layers", type=int, default=None, help="with --design bolenex: override the depth (profiling)")
+    ap.add_argument("--design", default="headline", choices=["headline", "bolenex", "robazen"], help="bolenex, robazen: that design beside a Llama-shaped decoder of equal size (one GPU)")
+    ap.add_argument("--sizes", default="w2048,w4096", help="with --design: which sizes")
+    ap.add_argument("--batches", default="1,16", help="with --design: sequences decoded together")
+    ap.add_argument("--arms", default="design,llama", help="with --design: which models")
+    ap.add_argument("--layers", type=int, default=None, help="with --design: override the depth (profiling)")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
@@ -704,8 +737,8 @@ def main():
         print(f"bench.py: WORLD_SIZE={world} but --gpus {args.gpus}; using WORLD_SIZE", file=sys.stderr)
     if args.gpus > 1 and world == 1:
         raise SystemExit("bench.py: launch multi-GPU runs with torch.distributed.run (one rank per GPU)")
-    if args.design == "bolenex":
-        run_bolenex(args, local_rank)
+    if args.design != "headline":
+        run_design(args, local_rank)
     elif world == 1:
         run_single(args, local_rank)
     else:

@@ -363,7 +363,7 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmPara
     FORGE_TRY(make_map_2d(&mx, act, uint64_t(last_col + w.K), uint64_t(p.m), uint64_t(act_ld) * 2, NT));
     p.tt_count = (p.m + NT - 1) / NT;
     const long long tiles = (long long)((w.N + 127) / 128) * p.tt_count;
-    const int grid = int(std::max(1LL, std::min((long long)sms, tiles * p.nk / 4)));
+    const int grid = int(std::max(1LL, std::min((long long)sms, std::max(NT >= 128 ? tiles : 1, tiles * p.nk / 4))));
     p.waves = NT >= 128 ? int(tiles / grid) : 0;   // a weight stream gains nothing from whole tiles in turn
     const long long units = (tiles - (long long)p.waves * grid) * p.nk;
     if (tiles * p.nk > INT32_MAX || (units + 1) * grid > INT32_MAX) { set_error("dense product: %lld tiles of %d K steps are too many", tiles, p.nk); return FORGE_ERR_SHAPE; }

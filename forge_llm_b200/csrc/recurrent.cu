@@ -3,6 +3,7 @@
 #include <cooperative_groups.h>
 
 #include <algorithm>
+#include <type_traits>
 
 #include "recurrent.cuh"
 
@@ -200,6 +201,70 @@ __global__ void __launch_bounds__(256) conv_rows_kernel(const RecurDims d, const
             for (int t = max(0, s.n - d.taps); t < s.n; ++t) ring[size_t((s.pos0 + t) % d.taps) * d.channels() + ch0 + c] = x[size_t(t) * a.x_ld + ch0 + c];
 }
 
+// The same for bfloat16 sizes in whole 16-byte pieces and at most four taps: a thread carries eight channels over eight tokens at a time.
+constexpr int kConvRun = 8;
+__global__ void __launch_bounds__(128) conv_rows8_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs) {
+    using bf16 = __nv_bfloat16;
+    const ScanSeg s = segs[blockIdx.z];
+    const int t0 = blockIdx.x * kConvTile, ch = (blockIdx.y * 128 + threadIdx.x) * 8, channels = d.channels();
+    if (t0 >= s.n) return;
+    const bool ok = ch < channels;
+    const bf16* x = static_cast<const bf16*>(a.x) + size_t(s.row0) * a.x_ld + ch;
+    bf16* y = static_cast<bf16*>(sc.conv) + size_t(s.row0) * channels + ch;
+    bf16* ring = static_cast<bf16*>(a.ring) + size_t(s.slot) * d.ring_values() + ch;
+    float w[4][8], past[3][8];   // past[2]: the token before
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) w[j][e] = ok && j >= 4 - d.taps ? a.conv[size_t(ch + e) * d.taps + j - (4 - d.taps)] : 0.f;
+#pragma unroll
+    for (int j = 0; j < 3; ++j) {
+        const int q = t0 - 3 + j, p = s.pos0 + q;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) past[j][e] = 0.f;
+        if (ok && j >= 4 - d.taps && p >= 0) load8(past[j], q >= 0 ? x + size_t(q) * a.x_ld : ring + size_t(p % d.taps) * channels);
+    }
+    const int lanes = d.dim / 8, unit = ch / d.dim;   // threads of a head of q or k
+    const bool is_qk = ok && unit < 2 * d.groups;
+    for (int t1 = t0; t1 < min(s.n, t0 + kConvTile); t1 += kConvRun) {
+        uint4 in[kConvRun];
+#pragma unroll
+        for (int i = 0; i < kConvRun; ++i) in[i] = ok && t1 + i < s.n ? *reinterpret_cast<const uint4*>(x + size_t(t1 + i) * a.x_ld) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+        for (int i = 0; i < kConvRun; ++i) {
+            const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&in[i]);
+            uint4 out;
+            __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&out);
+            float sum = 0.f;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float2 f = __bfloat1622float2(h[e]);
+                const float now[2] = {f.x, f.y};
+                float v[2];
+#pragma unroll
+                for (int b = 0; b < 2; ++b) {
+                    const int c = 2 * e + b;
+                    v[b] = silu(fmaf(w[3][c], now[b], fmaf(w[2][c], past[2][c], fmaf(w[1][c], past[1][c], w[0][c] * past[0][c]))));
+                    past[0][c] = past[1][c]; past[1][c] = past[2][c]; past[2][c] = now[b];
+                }
+                o[e] = __floats2bfloat162_rn(v[0], v[1]);
+                const float2 r = __bfloat1622float2(o[e]);
+                sum = fmaf(r.x, r.x, fmaf(r.y, r.y, sum));
+            }
+            if (ok && t1 + i < s.n) *reinterpret_cast<uint4*>(y + size_t(t1 + i) * channels) = out;
+            for (int m = lanes >> 1; m > 0; m >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, m);
+            if (is_qk && t1 + i < s.n && (threadIdx.x & (lanes - 1)) == 0)
+                sc.unit[size_t(s.row0 + t1 + i) * 2 * d.groups + unit] = (unit < d.groups ? d.q_scale : 1.f) / sqrtf(sum + 1e-6f);
+        }
+    }
+    if (ok && blockIdx.x == 0)
+        for (int t = max(0, s.n - d.taps); t < s.n; ++t) *reinterpret_cast<uint4*>(ring + size_t((s.pos0 + t) % d.taps) * channels) = *reinterpret_cast<const uint4*>(x + size_t(t) * a.x_ld);
+}
+bool conv_rows8_supported(const RecurDims& d) {
+    const int lanes = d.dim / 8;
+    return d.taps <= 4 && d.dim % 8 == 0 && d.vdim % 8 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0;
+}
+
 // Token by token: a warp carries four value columns of one head, its lanes share the rows of the state.
 template <typename T, bool DELTA, bool CHANNEL, int RPL>
 __global__ void __launch_bounds__(128) scan_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs) {
@@ -303,6 +368,23 @@ __global__ void __launch_bounds__(256) head_norm_kernel(const RecurDims d, const
     for (int c = lane; c < d.vdim; c += 32) out[c] = to_t<T>(src[c] * inv * a.norm[size_t(h) * a.norm_head + c] * to_f(gate[c]));
 }
 
+// the same in 16-byte pieces for vdim = 4 * a power of two up to 128: vdim / 4 lanes per (row, head)
+__global__ void __launch_bounds__(256) head_norm4_kernel(const RecurDims d, const RecurArgs a, const float* __restrict__ o, int row0, int rows) {
+    const int lanes = d.vdim / 4, i = int((blockIdx.x * 256 + threadIdx.x) / lanes), c = int(threadIdx.x & (lanes - 1)) * 4;
+    const bool ok = i < rows * d.heads;
+    const int r = row0 + (ok ? i : 0) / d.heads, h = (ok ? i : 0) % d.heads;
+    const float4 v = *reinterpret_cast<const float4*>(o + (size_t(r) * d.heads + h) * d.vdim + c);
+    const uint2 g2 = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(a.gate) + size_t(r) * a.gate_ld + h * d.vdim + c);
+    const float4 w = *reinterpret_cast<const float4*>(a.norm + size_t(h) * a.norm_head + c);
+    float ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+    for (int m = lanes >> 1; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+    const float inv = 1.0f / sqrtf(ss / float(d.vdim) + d.eps);
+    const float2 ga = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&g2.x)), gb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&g2.y));
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x * inv * w.x * ga.x, v.y * inv * w.y * ga.y), hi = __floats2bfloat162_rn(v.z * inv * w.z * gb.x, v.w * inv * w.w * gb.y);
+    if (ok) *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(a.out) + size_t(r) * a.out_ld + h * d.vdim + c) =
+        make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+
 // ------------------------------------------------------------------------------------------------ token shift
 // One CTA = 256 columns of one row (single rows) or of up to kShiftRows rows of a segment; the thread that reads what is kept of the row
 // before a segment is the one that leaves the segment's last row there.
@@ -313,7 +395,7 @@ __global__ void __launch_bounds__(256) token_shift_kernel(T* __restrict__ dst, i
     const int c = blockIdx.y * 256 + threadIdx.x;
     ScanSeg s;
     if (segs) s = segs[blockIdx.z];
-    else s = ScanSeg{int(blockIdx.x), 1, state_slot(rows, blockIdx.x), rows.pos[blockIdx.x]};
+    else s = ScanSeg{int(blockIdx.x), 1, state_slot(rows, blockIdx.x), rows.pos[blockIdx.x], 0, {}};
     const int t0 = segs ? blockIdx.x * kShiftRows : 0;
     pdl_trigger();
     pdl_wait();
@@ -383,14 +465,24 @@ int32_t scan_t(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, c
     return FORGE_OK;
 }
 template <typename T>
-int32_t segments_t(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, const ScanSeg* segs, int n_segs, int max_n, int row0, int rows, cudaStream_t st) {
+int32_t segments_t(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, const SegTable& t, cudaStream_t st) {
+    constexpr bool half = std::is_same<T, __nv_bfloat16>::value;
     if (d.delta) {
-        const int units = 2 * d.groups + (d.heads * d.vdim + 127) / 128;
-        conv_rows_kernel<T><<<dim3((max_n + kConvTile - 1) / kConvTile, (units + 7) / 8, n_segs), 256, 0, st>>>(d, a, sc, segs);
+        const int tiles = (t.max_n + kConvTile - 1) / kConvTile, units = 2 * d.groups + (d.heads * d.vdim + 127) / 128;
+        if (half && conv_rows8_supported(d)) conv_rows8_kernel<<<dim3(tiles, (d.channels() + 1023) / 1024, t.n), 128, 0, st>>>(d, a, sc, t.segs);
+        else conv_rows_kernel<T><<<dim3(tiles, (units + 7) / 8, t.n), 256, 0, st>>>(d, a, sc, t.segs);
         FORGE_LAUNCH_CHECK();
-        FORGE_TRY(d.channel ? (scan_t<T, true, true>(d, a, sc, segs, n_segs, st)) : (scan_t<T, true, false>(d, a, sc, segs, n_segs, st)));
-    } else FORGE_TRY((scan_t<T, false, true>(d, a, sc, segs, n_segs, st)));
-    head_norm_kernel<T><<<(rows * d.heads + 7) / 8, 256, 0, st>>>(d, a, sc.o, row0, rows);
+    }
+    const int walked = half && recur_chunked_supported(d) ? t.n_short : t.n;   // token by token
+    if (walked > 0) {
+        if (!d.delta) FORGE_TRY((scan_t<T, false, true>(d, a, sc, t.segs, walked, st)));
+        else FORGE_TRY(d.channel ? (scan_t<T, true, true>(d, a, sc, t.segs, walked, st)) : (scan_t<T, true, false>(d, a, sc, t.segs, walked, st)));
+    }
+    FORGE_TRY(recur_chunked(d, a, sc, t.segs + walked, t.n - walked, t.n_chunks, st));
+    const int lanes = d.vdim / 4;
+    if (half && d.vdim % 4 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0 && a.gate_ld % 4 == 0 && a.out_ld % 4 == 0)
+        head_norm4_kernel<<<unsigned((size_t(t.rows) * d.heads * lanes + 255) / 256), 256, 0, st>>>(d, a, sc.o, t.row0, t.rows);
+    else head_norm_kernel<T><<<(t.rows * d.heads + 7) / 8, 256, 0, st>>>(d, a, sc.o, t.row0, t.rows);
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
@@ -409,23 +501,22 @@ int32_t recur_decode(const RecurDims& d, int dtype, const RecurArgs& a, const St
     return dtype == FORGE_F32 ? go(float{}) : go(__nv_bfloat16{});
 }
 
-int32_t recur_segments(const RecurDims& d, int dtype, const RecurArgs& a, const RecurScratch& sc, const ScanSeg* segs, int n_segs, int max_n, int row0, int rows, cudaStream_t st) {
-    if (n_segs <= 0) return FORGE_OK;
-    return dtype == FORGE_F32 ? segments_t<float>(d, a, sc, segs, n_segs, max_n, row0, rows, st) : segments_t<__nv_bfloat16>(d, a, sc, segs, n_segs, max_n, row0, rows, st);
+int32_t recur_segments(const RecurDims& d, int dtype, const RecurArgs& a, const RecurScratch& sc, const SegTable& t, cudaStream_t st) {
+    if (t.n <= 0) return FORGE_OK;
+    return dtype == FORGE_F32 ? segments_t<float>(d, a, sc, t, st) : segments_t<__nv_bfloat16>(d, a, sc, t, st);
 }
 
-int32_t token_shift(void* dst, int ld, int width, int width_p, int n_mix, const float* mu, void* prev, int dtype, const StepRows& rows, int n_single, const ScanSeg* segs, int n_segs, int max_n,
-                    cudaStream_t st) {
+int32_t token_shift(void* dst, int ld, int width, int width_p, int n_mix, const float* mu, void* prev, int dtype, const StepRows& rows, int n_single, const SegTable& t, cudaStream_t st) {
     if (n_mix > 8) { set_error("token shift: %d mixes", n_mix); return FORGE_ERR_SHAPE; }
-    auto go = [&](auto t) -> int32_t {
-        using T = decltype(t);
+    auto go = [&](auto type) -> int32_t {
+        using T = decltype(type);
         const int cols = (width + 255) / 256;
         if (n_single > 0) {
             FORGE_CUDA(launch_pdl(token_shift_kernel<T>, dim3(n_single, cols), dim3(256), 0, st, static_cast<T*>(dst), ld, width, width_p, n_mix, mu, static_cast<T*>(prev), rows, static_cast<const ScanSeg*>(nullptr)));
             FORGE_LAUNCH_CHECK();
         }
-        if (n_segs > 0) {
-            FORGE_CUDA(launch_pdl(token_shift_kernel<T>, dim3((max_n + kShiftRows - 1) / kShiftRows, cols, n_segs), dim3(256), 0, st, static_cast<T*>(dst), ld, width, width_p, n_mix, mu, static_cast<T*>(prev), rows, segs));
+        if (t.n > 0) {
+            FORGE_CUDA(launch_pdl(token_shift_kernel<T>, dim3((t.max_n + kShiftRows - 1) / kShiftRows, cols, t.n), dim3(256), 0, st, static_cast<T*>(dst), ld, width, width_p, n_mix, mu, static_cast<T*>(prev), rows, t.segs));
             FORGE_LAUNCH_CHECK();
         }
         return FORGE_OK;

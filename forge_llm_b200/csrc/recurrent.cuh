@@ -22,8 +22,13 @@ struct RecurDims {
     __host__ __device__ size_t ring_values() const { return size_t(taps) * channels(); }
 };
 
-// consecutive rows of one sequence: rows [row0, row0 + n) of the step at positions pos0, pos0 + 1, ... of state slot `slot`
-struct ScanSeg { int32_t row0, n, slot, pos0; };
+constexpr int kRecurChunk = 64;     // tokens of a chunk (recurrent_chunk.cu)
+constexpr int kChunkedRows = 16;    // segments of fewer tokens go token by token
+// consecutive rows of one sequence: rows [row0, row0 + n) of the step at positions pos0, pos0 + 1, ... of state slot `slot`; chunk0: number
+// of its first chunk among all chunks of the step (segments of at least kChunkedRows)
+struct ScanSeg { int32_t row0, n, slot, pos0, chunk0, unused[3]; };
+// a step's segments (device table), the n_short short ones first; together they are the rows [row0, row0 + rows)
+struct SegTable { const ScanSeg* segs = nullptr; int n = 0, n_short = 0, max_n = 0, n_chunks = 0, row0 = 0, rows = 0; };
 
 struct RecurArgs {
     const void* x = nullptr; int x_ld = 0;               // T rows [q | k | v]: in front of the convolution, if there is one
@@ -37,24 +42,31 @@ struct RecurArgs {
     void* out = nullptr; int out_ld = 0;                 // T rows [heads * vdim]: rms norm(o) * norm * gate
 };
 
+// per chunk and head, see recurrent_chunk.cu
+struct ChunkScratch { __nv_bfloat16* tp = nullptr; float* scal = nullptr; float* end = nullptr; __nv_bfloat16* dec = nullptr; };
+struct ChunkBytes { size_t tp, scal, end, dec; };   // of one chunk, all heads
 // scratch of a step with segments
 struct RecurScratch {
     void* conv = nullptr;         // T [rows][channels]: behind convolution and silu
     float* unit = nullptr;        // [rows][2 * groups]: what q and k are multiplied with to be unit vectors (q: times q_scale)
     float* o = nullptr;           // [rows][heads * vdim]
+    ChunkScratch chunk;
 };
 
 bool recur_supported(const RecurDims& d);
 // single tokens: row r of `rows` is one token of its sequence
 int32_t recur_decode(const RecurDims& d, int dtype, const RecurArgs& a, const StepRows& rows, cudaStream_t st);
-// segments (device table, at most max_n tokens each) that make up the rows [row0, row0 + rows) of the step
-int32_t recur_segments(const RecurDims& d, int dtype, const RecurArgs& a, const RecurScratch& sc, const ScanSeg* segs, int n_segs, int max_n, int row0, int rows, cudaStream_t st);
+// segments of any length
+int32_t recur_segments(const RecurDims& d, int dtype, const RecurArgs& a, const RecurScratch& sc, const SegTable& t, cudaStream_t st);
+// the walk of the long segments by chunks (bfloat16; called by recur_segments): leaves o and the state
+bool recur_chunked_supported(const RecurDims& d);
+ChunkBytes recur_chunk_bytes(const RecurDims& d);
+int32_t recur_chunked(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, const ScanSeg* segs, int n_segs, int n_chunks, cudaStream_t st);
 
 // Token shift: dst rows get, next to h in columns [0, width_p), `n_mix` blocks of width_p columns h + (h' - h) mu[i], h' being the
 // sequence's row before (prev [slot][width], zeros at position 0).  h lies in dst's first block already.  prev is left at the
 // sequence's last row.
-int32_t token_shift(void* dst, int ld, int width, int width_p, int n_mix, const float* mu, void* prev, int dtype, const StepRows& rows, int n_single, const ScanSeg* segs, int n_segs, int max_n,
-                    cudaStream_t st);
+int32_t token_shift(void* dst, int ld, int width, int width_p, int n_mix, const float* mu, void* prev, int dtype, const StepRows& rows, int n_single, const SegTable& t, cudaStream_t st);
 
 // x += (rms norm(a) wa + rms norm(b) wb) / 2 over rows of `width` values, then `after`; ab: f32 rows [a | b]
 int32_t add_normed_pair(float* x, const float* ab, int rows, int width, float eps, const float* wa, const float* wb, const After& after, int dtype, cudaStream_t st);

@@ -58,9 +58,9 @@ struct StackModel {
     DenseScratch scratch;
     // step buffers, grown on demand (scratch_gen of the model counts the moves)
     struct Buf { void* p = nullptr; size_t cap = 0; };
-    Buf x, h, cat, proj, gate, mid, mid_r, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, hgate, decay, beta, low, conv, unit, o, pair, place, sel, logits, meta;
+    Buf x, h, cat, proj, gate, mid, mid_r, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, hgate, decay, beta, low, conv, unit, o, pair, place, c_tp, c_scal, c_end, c_dec, sel, logits, meta;
     std::vector<Buf*> all() {
-        return {&x, &h, &cat, &proj, &gate, &mid, &mid_r, &q, &part, &ml, &ctx_c, &ctx_r, &ctx_k, &ctx_v, &hgate, &decay, &beta, &low, &conv, &unit, &o, &pair, &place, &sel, &logits, &meta};
+        return {&x, &h, &cat, &proj, &gate, &mid, &mid_r, &q, &part, &ml, &ctx_c, &ctx_r, &ctx_k, &ctx_v, &hgate, &decay, &beta, &low, &conv, &unit, &o, &pair, &place, &c_tp, &c_scal, &c_end, &c_dec, &sel, &logits, &meta};
     }
     const LayerWeights& weights(int layer) const { return w[spec.layers[layer].weights_of >= 0 ? spec.layers[layer].weights_of : layer]; }
 };
@@ -315,11 +315,12 @@ int row_splits(const StackModel& S, int rows, int pages) {
     return std::max(1, std::min(pages, 148 / std::max(1, rows * groups)));
 }
 
-int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt, int ctx_rows, int seg_rows) {
+int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt, int ctx_rows, int seg_rows, int chunks) {
     StackModel& S = *m->stack;
     const size_t es = dense_size(S.dtype), r = size_t(rows), W = size_t(S.spec.width), WP = size_t(S.width_p);
     // bytes, rows times the widest layer
     size_t h = WP * es, proj = 0, gate = 0, mid = 0, mid_r = 0, q = 0, part = 0, heads = 0, cc = 0, cr = 0, ck = 0, cv = 0, hgate = 0, decay = 0, beta = 0, low = 0, conv = 0, unit = 0, o = 0, pair = 0;
+    ChunkBytes cb{0, 0, 0, 0};
     auto most = [](size_t& a, size_t b) { a = std::max(a, b); };
     size_t n_max = size_t(S.head.N);
     for (size_t i = 0; i < S.spec.layers.size(); ++i) {
@@ -346,6 +347,10 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
         most(beta, r * d.heads * 4);
         most(low, r * (w.decay_k + w.low.K) * es);
         most(o, r * HV * 4);
+        if (chunks && recur_chunked_supported(d)) {
+            const ChunkBytes b = recur_chunk_bytes(d);
+            most(cb.tp, chunks * b.tp); most(cb.scal, chunks * b.scal); most(cb.end, chunks * b.end); most(cb.dec, chunks * b.dec);
+        }
         if (d.delta && seg_rows) { most(conv, r * d.channels() * es); most(unit, r * 2 * d.groups * 4); }
         if (L.has_attn()) {
             most(h, (1 + kMixes) * WP * es);
@@ -360,7 +365,7 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
     if (S.spec.loop_times) FORGE_TRY(grow(m, S.cat, r * 2 * WP * es));
     FORGE_TRY(grow(m, S.place, r * sizeof(int32_t)));
     const std::pair<StackModel::Buf*, size_t> sizes[] = {{&S.proj, proj}, {&S.gate, gate}, {&S.mid, mid}, {&S.mid_r, mid_r}, {&S.q, q}, {&S.part, part}, {&S.ml, heads}, {&S.hgate, hgate}, {&S.decay, decay},
-        {&S.beta, beta}, {&S.low, low}, {&S.conv, conv}, {&S.unit, unit}, {&S.o, o}, {&S.pair, pair}, {&S.ctx_c, cc}, {&S.ctx_r, cr}, {&S.ctx_k, ck}, {&S.ctx_v, cv}};
+        {&S.beta, beta}, {&S.low, low}, {&S.conv, conv}, {&S.unit, unit}, {&S.o, o}, {&S.pair, pair}, {&S.c_tp, cb.tp}, {&S.c_scal, cb.scal}, {&S.c_end, cb.end}, {&S.c_dec, cb.dec}, {&S.ctx_c, cc}, {&S.ctx_r, cr}, {&S.ctx_k, ck}, {&S.ctx_v, cv}};
     for (const auto& e : sizes) FORGE_TRY(grow(m, *e.first, e.second));
     // one ticket per output tile of the largest product (128 rows x at least 16 tokens)
     const size_t tiles = ((n_max + 127) / 128) * std::max<size_t>(1, (size_t(std::max(rows, ctx_rows)) + 127) / 128);
@@ -379,7 +384,7 @@ struct Step {
     int ones = 0;                            // rows [0, ones): one token of its sequence each
     int single = 0, splits = 1;              // rows [0, single): attention row by row; the rest are prompt rows
     int max_keys = 1;                        // most keys a row of [0, single) has
-    const ScanSeg* segs = nullptr; int n_segs = 0, max_seg = 0;   // the rows [ones, n)
+    SegTable segs;                           // the rows [ones, n)
     const PromptTile* tiles = nullptr; int n_tiles = 0;
     const int32_t* ctx_pages = nullptr; int ctx_rows = 0;
     uint32_t* hist = nullptr; const int32_t* step = nullptr;
@@ -508,7 +513,9 @@ struct Sequence {
         FORGE_TRY(recur_decode(d, dt, a, ones, st));
         RecurScratch sc;
         sc.conv = S.conv.p; sc.unit = static_cast<float*>(S.unit.p); sc.o = static_cast<float*>(S.o.p);
-        return recur_segments(d, dt, a, sc, s.segs, s.n_segs, s.max_seg, s.ones, n - s.ones, st);
+        sc.chunk.tp = static_cast<__nv_bfloat16*>(S.c_tp.p); sc.chunk.scal = static_cast<float*>(S.c_scal.p); sc.chunk.end = static_cast<float*>(S.c_end.p);
+        sc.chunk.dec = static_cast<__nv_bfloat16*>(S.c_dec.p);
+        return recur_segments(d, dt, a, sc, s.segs, st);
     }
     RecurArgs recur_args(const RecurDims& d, const LayerWeights& w, StackCache::Run& run) {
         RecurArgs a;
@@ -555,7 +562,7 @@ struct Sequence {
         const RecurDims& d = L.rec;
         const int D = d.heads * d.dim, ld = (1 + kMixes) * WP;
         float* hgate = static_cast<float*>(S.hgate.p);
-        FORGE_TRY(token_shift(S.h.p, ld, W, WP, kMixes, w.mu, run.prev, dt, s.rows, s.ones, s.segs, s.n_segs, s.max_seg, st));
+        FORGE_TRY(token_shift(S.h.p, ld, W, WP, kMixes, w.mu, run.prev, dt, s.rows, s.ones, s.segs, st));
         DenseOut o;
         {
             const int32_t* place = static_cast<const int32_t*>(S.place.p);
@@ -802,7 +809,7 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
             meta[2 * rows + r0 + k] = e.seq;
         }
         for (int k = 0; k < e.n_want; ++k) meta[3 * rows + at_entry[i].want + k] = r0 + want[at_entry[i].want + k];
-        if (e.n_tokens > 1) { segs.push_back({r0, e.n_tokens, e.seq, base}); max_seg = std::max(max_seg, int(e.n_tokens)); }
+        if (e.n_tokens > 1) { segs.push_back({r0, e.n_tokens, e.seq, base, 0, {}}); max_seg = std::max(max_seg, int(e.n_tokens)); }
         if (is_prompt(i)) {
             const int ctx0 = int(pages.size()) * FORGE_KV_PAGE, np = (base + e.n_tokens + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE;
             for (int p = 0; p < np; ++p) pages.push_back(kv->h_page_table[size_t(e.seq) * kv->pages_per_seq + p]);
@@ -810,13 +817,18 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
         }
     }
     std::stable_sort(tiles.begin(), tiles.end(), [](const PromptTile& a, const PromptTile& b) { return a.pos0 + a.rows > b.pos0 + b.rows; });   // the longest first
-    const size_t o_pages = (meta.size() + 3) & ~size_t(3), o_tiles = (o_pages + pages.size() + 3) & ~size_t(3), o_segs = o_tiles + tiles.size() * 4, total = o_segs + segs.size() * 4;
+    const auto first_long = std::stable_partition(segs.begin(), segs.end(), [](const ScanSeg& g) { return g.n < kChunkedRows; });
+    const int n_short = int(first_long - segs.begin());
+    int chunks = 0;
+    for (auto g = first_long; g != segs.end(); ++g) { g->chunk0 = chunks; chunks += (g->n + kRecurChunk - 1) / kRecurChunk; }
+    static_assert(sizeof(ScanSeg) == 32, "eight words");
+    const size_t o_pages = (meta.size() + 3) & ~size_t(3), o_tiles = (o_pages + pages.size() + 3) & ~size_t(3), o_segs = o_tiles + tiles.size() * 4, total = o_segs + segs.size() * 8;
     meta.resize(total);
     std::copy(pages.begin(), pages.end(), meta.begin() + o_pages);
     if (!tiles.empty()) memcpy(meta.data() + o_tiles, tiles.data(), tiles.size() * sizeof(PromptTile));
     if (!segs.empty()) memcpy(meta.data() + o_segs, segs.data(), segs.size() * sizeof(ScanSeg));
     const int splits = row_splits(S, std::max(1, single), (max_keys + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE), ctx_rows = int(pages.size()) * FORGE_KV_PAGE;
-    FORGE_TRY(ensure_step(m, std::max(rows, wants), single, splits, rows - single, ctx_rows, rows - ones));
+    FORGE_TRY(ensure_step(m, std::max(rows, wants), single, splits, rows - single, ctx_rows, rows - ones, chunks));
     FORGE_TRY(grow(m, S.meta, total * 4));
     FORGE_TRY(grow(m, S.sel, size_t(wants) * S.width_p * dense_size(S.dtype)));
     FORGE_TRY(grow(m, S.logits, size_t(wants) * S.spec.vocab * 4));
@@ -827,7 +839,7 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
     s.rows = StepRows{rows, dm + rows, dm + 2 * rows, kv->d_page_table, kv->pages_per_seq};
     for (int i = 0; i < n_entries; ++i) if (!is_prompt(i)) s.rows.fresh = std::max(s.rows.fresh, int(entries[i].n_tokens));
     s.ones = ones; s.single = single; s.splits = splits; s.max_keys = max_keys;
-    s.segs = reinterpret_cast<const ScanSeg*>(dm + o_segs); s.n_segs = int(segs.size()); s.max_seg = max_seg;
+    s.segs = SegTable{reinterpret_cast<const ScanSeg*>(dm + o_segs), int(segs.size()), n_short, max_seg, chunks, ones, rows - ones};
     s.ctx_pages = dm + o_pages; s.ctx_rows = ctx_rows;
     s.tiles = reinterpret_cast<const PromptTile*>(dm + o_tiles); s.n_tiles = int(tiles.size());
     if (trace_rows) { s.trace = m->trace + size_t(trace_row0) * S.spec.width; s.trace_stride = size_t(trace_rows) * S.spec.width; }
@@ -859,7 +871,7 @@ int32_t stack_prefill(ForgeModel* m, ForgeKV* kv, int seq, const uint32_t* token
     return rc;
 }
 
-int32_t stack_ensure_decode(ForgeModel* m, ForgeKV* kv, int batch) { return ensure_step(m, batch, batch, kv->stack->splits, 0, 0, 0); }
+int32_t stack_ensure_decode(ForgeModel* m, ForgeKV* kv, int batch) { return ensure_step(m, batch, batch, kv->stack->splits, 0, 0, 0, 0); }
 
 int32_t stack_decode_launches(ForgeModel* m, ForgeKV* kv, int batch, bool greedy, bool record) {
     StackModel& S = *m->stack;

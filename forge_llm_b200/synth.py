@@ -218,9 +218,74 @@ def bolenex_shapes(cfg: dict, layer: int) -> dict:
     return s
 
 
-def write_bolenex(folder: str, cfg: dict, seed: int = 0, repeat_layers: bool = True) -> None:
-    """config.json and model.safetensors (bfloat16): matrices ~ N(0, 1/inputs), norm weights 1, biases 0, alpha 0.5.  With
-    ``repeat_layers`` layer 0's values are drawn and stored again for every later layer (of the same sizes)."""
+def robazen_config(width: int, layers: int, heads: int, ff: int, vocab: int, dim: int = 128, chunk: int = 1024, loop: bool = True) -> dict:
+    """config.json of a Robazen stack of ``layers`` layer runs (a multiple of four): groups of (attention beside time mixing, delta, channel
+    delta, delta), each with a feed-forward.  With ``loop`` a quarter of the groups (at least one) runs twice with the same weights."""
+    pair = {"left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": dim, "scale": float(dim ** -0.5), "softcap": 50.0, "mask": {"size": chunk}},
+            "right": {"heads": heads * dim // 64, "dim": 64}}
+    rec = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": 4}
+    mlp = {"kind": "dense", "ff": ff}
+    group = [("parallel", pair), ("delta", rec), ("channel_delta", rec), ("delta", rec)]
+    n = layers // 4
+    twice = max(1, n // 4) if loop and n >= 2 else 0
+    out = [{"type": t, "mixer": dict(m), "mlp": dict(mlp)} for _ in range(n - twice) for t, m in group]
+    cfg = {"architecture": "Robazen", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "layers": out, "loop": None}
+    if twice:
+        cfg["loop"] = {"start": len(out) - 4 * twice, "stop": len(out), "times": 2}
+    return cfg
+
+
+def robazen_shapes(cfg: dict, layer: int, rank: int = 64) -> dict:
+    """Tensor shapes of one layer, without its prefix; ``rank``: inner size of the two-step projections."""
+    W, L = cfg["width"], cfg["layers"][layer]
+    m, f = L["mixer"], L.get("mlp")
+
+    def norm(n):
+        return {n: (W,), n + ".b": (W,), n + ".alpha": ()}
+
+    s = norm("norm1")
+    if L["type"] == "parallel":
+        a, r = m["left"], m["right"]
+        d = r["heads"] * r["dim"]
+        s.update({"mix.left.q": (a["heads"] * a["dim"], W), "mix.left.k": (a["kv_heads"] * a["dim"], W), "mix.left.v": (a["kv_heads"] * a["vdim"], W),
+                  "mix.left.g": (a["heads"], W), "mix.left.o": (W, a["heads"] * a["vdim"]), "mix.left.out": (W,), "mix.right.out": (W,)})
+        s.update({"mix.right." + x: (d, W) for x in "rkvg"})
+        s.update({"mix.right.mu." + x: (W,) for x in "rkvgw"})
+        s.update({"mix.right.w1": (rank, W), "mix.right.w2": (d, rank), "mix.right.w0": (d,), "mix.right.u": (r["heads"], r["dim"]),
+                  "mix.right.norm": (d,), "mix.right.o": (W, d)})
+    else:
+        H, D, hv = m["heads"], m["heads"] * m["dim"], m["heads"] * m["vdim"]
+        for x, n in (("q", m["kv_heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", hv)):
+            s.update({"mix." + x: (n, W), f"mix.{x}.conv": (n, m["conv"])})
+        s.update({"mix.b": (H, W), "mix.A_log": (H,), "mix.norm": (m["vdim"],), "mix.o": (W, hv)})
+        if L["type"] == "delta":
+            s.update({"mix.a": (H, W), "mix.dt_bias": (H,), "mix.g": (hv, W)})
+        else:
+            s.update({"mix.a1": (rank, W), "mix.a2": (D, rank), "mix.dt_bias": (D,), "mix.g1": (rank, W), "mix.g2": (hv, rank)})
+    if f:
+        s.update(norm("norm2"))
+        s.update({"mlp.gate": (f["ff"], W), "mlp.up": (f["ff"], W), "mlp.down": (W, f["ff"])})
+    return s
+
+
+LAYER_SHAPES = {"Bolenex": bolenex_shapes, "Robazen": robazen_shapes}
+
+
+def stack_shapes(cfg: dict) -> dict:
+    """Tensor shapes of a layer-list model."""
+    W, V = cfg["width"], cfg["vocab"]
+    out = {"embed": (V, W), "head": (V, W), "final.norm": (W,), "final.norm.b": (W,), "final.norm.alpha": ()}
+    if cfg.get("loop"):
+        out.update({"loop.in": (W, 2 * W), "loop.step": (cfg["loop"]["times"], W)})
+    for i, L in enumerate(cfg["layers"]):
+        if "weights_of" not in L:
+            out.update({f"l{i}.{n}": s for n, s in LAYER_SHAPES[cfg["architecture"]](cfg, i).items()})
+    return out
+
+
+def write_stack(folder: str, cfg: dict, seed: int = 0, repeat_layers: bool = True) -> None:
+    """config.json and model.safetensors (bfloat16): matrices ~ N(0, 1/inputs), norm weights 1, biases and mixes 0, alpha 0.5.  With
+    ``repeat_layers`` a layer's values are stored again for later tensors of the same name and shape."""
     import json
     import os
     import struct
@@ -230,16 +295,12 @@ def write_bolenex(folder: str, cfg: dict, seed: int = 0, repeat_layers: bool = T
         if name.endswith("alpha"):
             x = np.full(shape, 0.5, np.float32)
         elif len(shape) < 2:
-            x = np.zeros(shape, np.float32) if name.endswith(".b") else np.ones(shape, np.float32)
+            x = np.zeros(shape, np.float32) if name.endswith((".b", "A_log", "dt_bias", ".w0")) or ".mu." in name else np.ones(shape, np.float32)
         else:
             x = rng.standard_normal(shape, np.float32) * np.float32(shape[1] ** -0.5)
         return (np.ascontiguousarray(x).view(np.uint32) >> 16).astype(np.uint16)
 
-    W, V = cfg["width"], cfg["vocab"]
-    parts = [(n, s) for n, s in (("embed", (V, W)), ("head", (V, W)), ("final.norm", (W,)), ("final.norm.b", (W,)), ("final.norm.alpha", ()))]
-    for i, L in enumerate(cfg["layers"]):
-        if "weights_of" not in L:
-            parts += [(f"l{i}.{n}", s) for n, s in bolenex_shapes(cfg, i).items()]
+    parts = list(stack_shapes(cfg).items())
     head, off = {}, 0
     for n, s in parts:
         size = 2 * int(np.prod(s, dtype=np.int64))
@@ -251,7 +312,7 @@ def write_bolenex(folder: str, cfg: dict, seed: int = 0, repeat_layers: bool = T
     with open(os.path.join(folder, "model.safetensors"), "wb") as f:
         f.write(struct.pack("<Q", len(text)) + text)
         for n, s in parts:
-            key = (n.split(".", 1)[1], s) if n.startswith("l") and repeat_layers else None
+            key = (n.split(".", 1)[1], s) if n.startswith("l") and not n.startswith("loop") and repeat_layers else None
             data = kept.get(key) if key else None
             if data is None:
                 data = draw(n, s).tobytes()

@@ -350,8 +350,99 @@ def make_config(width=136, vocab=203, layers=(), eps=1e-5):
     return {"architecture": "Bolenex", "layers": out, "norm": {"eps": eps}, "vocab": vocab, "width": width}
 
 
+def delta_mixer(heads=4, kv_heads=2, dim=24, vdim=40, conv=4):
+    return {"conv": conv, "dim": dim, "heads": heads, "kv_heads": kv_heads, "vdim": vdim}
+
+
+def pair_mixer(heads=6, kv_heads=2, dim=24, vdim=40, chunk=48, softcap=20.0, scale=None, heads_r=3, dim_r=40):
+    return {"left": {"dim": dim, "heads": heads, "kv_heads": kv_heads, "mask": {"size": chunk}, "scale": float(scale if scale is not None else dim ** -0.5),
+                     "softcap": float(softcap), "vdim": vdim}, "right": {"dim": dim_r, "heads": heads_r}}
+
+
+def make_robazen(width=136, vocab=203, layers=(), loop=None, eps=1e-5):
+    """``layers``: (type, mixer, ff size or None) per layer; ``loop``: (start, stop, times)."""
+    out = [{"mixer": mx, "mlp": None if ff is None else {"ff": ff, "kind": "dense"}, "type": t} for t, mx, ff in layers]
+    return {"architecture": "Robazen", "layers": out, "loop": None if loop is None else dict(zip(("start", "stop", "times"), loop)), "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def random_robazen(cfg, seed=0, rank=20):
+    """Seeded weights of a Robazen model, rounded to bfloat16: decays between almost none and almost all, every factor away from 1 and 0."""
+    rng = np.random.default_rng(seed)
+    W = cfg["width"]
+    t = {}
+
+    def mat(name, out, inp, gain=1.0):
+        t[name] = bf16_round(rng.standard_normal((out, inp)) * (gain / math.sqrt(inp)))
+
+    def vec(name, n, mean, dev):
+        t[name] = bf16_round(mean + dev * rng.standard_normal(n))
+
+    def norm(name):
+        vec(name, W, 1.0, 0.3)
+        vec(name + ".b", W, 0.0, 0.2)
+        t[name + ".alpha"] = bf16_round(np.asarray(0.5 + 0.4 * rng.random()))
+
+    t["embed"] = bf16_round(rng.standard_normal((cfg["vocab"], W)))
+    if cfg.get("loop"):
+        mat("loop.in", W, 2 * W, 1.3)
+        t["loop.step"] = bf16_round(0.5 * rng.standard_normal((cfg["loop"]["times"], W)))
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        norm(p + "norm1")
+        x = p + "mix."
+        if L["type"] == "parallel":
+            a, r = m["left"], m["right"]
+            D = r["heads"] * r["dim"]
+            mat(x + "left.q", a["heads"] * a["dim"], W, 1.5)
+            mat(x + "left.k", a["kv_heads"] * a["dim"], W, 1.5)
+            mat(x + "left.v", a["kv_heads"] * a["vdim"], W)
+            mat(x + "left.g", a["heads"], W, 2.0)
+            mat(x + "left.o", W, a["heads"] * a["vdim"], 2.0)
+            for n in "rkvgw":
+                t[x + "right.mu." + n] = bf16_round(rng.random(W))
+            for n in "rkvg":
+                mat(x + "right." + n, D, W)
+            mat(x + "right.w1", rank, W)
+            mat(x + "right.w2", D, rank, 1.5)
+            vec(x + "right.w0", D, -2.0, 1.5)
+            t[x + "right.u"] = bf16_round(rng.standard_normal((r["heads"], r["dim"])))
+            vec(x + "right.norm", D, 1.0, 0.3)
+            mat(x + "right.o", W, D)
+            vec(x + "left.out", W, 0.8, 0.3)
+            vec(x + "right.out", W, 1.2, 0.3)
+        else:
+            H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            for n, c in (("q", G * d), ("k", G * d), ("v", H * dv)):
+                mat(x + n, c, W, 1.5)
+                t[x + n + ".conv"] = bf16_round(0.6 * rng.standard_normal((c, m["conv"])))
+            mat(x + "b", H, W, 2.0)
+            vec(x + "A_log", H, -1.0, 1.5)
+            vec(x + "norm", dv, 1.0, 0.3)
+            mat(x + "o", W, H * dv, 1.5)
+            if L["type"] == "delta":
+                mat(x + "a", H, W, 2.0)
+                vec(x + "dt_bias", H, -1.0, 1.0)
+                mat(x + "g", H * dv, W, 1.5)
+            else:
+                mat(x + "a1", rank, W)
+                mat(x + "a2", H * d, rank, 2.0)
+                vec(x + "dt_bias", H * d, -1.0, 1.5)
+                mat(x + "g1", rank + 4, W)
+                mat(x + "g2", H * dv, rank + 4, 2.0)
+        if L.get("mlp"):
+            norm(p + "norm2")
+            mat(p + "mlp.gate", L["mlp"]["ff"], W, 1.5)
+            mat(p + "mlp.up", L["mlp"]["ff"], W, 1.5)
+            mat(p + "mlp.down", W, L["mlp"]["ff"])
+    norm("final.norm")
+    mat("head", cfg["vocab"], W)
+    return t
+
+
 def random_tensors(cfg, seed=0):
     """Seeded weights, rounded to bfloat16, in which every factor matters (norm weights and biases away from 1 and 0)."""
+    if cfg["architecture"] == "Robazen":
+        return random_robazen(cfg, seed)
     rng = np.random.default_rng(seed)
     W = cfg["width"]
     t = {}

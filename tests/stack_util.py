@@ -31,6 +31,25 @@ CONFIGS = {
 }
 
 
+_delta, _pair = LS.delta_mixer, LS.pair_mixer
+ROBAZEN = {
+    # every mixer, with and without a feed-forward, the middle layers twice
+    "all": LS.make_robazen(136, 203, [("parallel", _pair(), 72), ("delta", _delta(), None), ("channel_delta", _delta(heads=6, kv_heads=3, dim=16, vdim=24, conv=3), 56), ("delta", _delta(conv=2), 40)],
+                           (1, 3, 2), eps=1e-3),
+    # the loop is the whole model, three passes; one head; no history in the convolution
+    "loop_all": LS.make_robazen(72, 67, [("channel_delta", _delta(1, 1, 8, 8, 1), 24), ("parallel", _pair(1, 1, 8, 16, 7, 5.0, 0.9, 1, 8), None)], (0, 2, 3), eps=1e-2),
+    # one pass only, at the end; sizes no multiple of eight (token by token everywhere)
+    "odd": LS.make_robazen(70, 91, [("parallel", _pair(3, 1, 9, 13, 33, 11.0, None, 2, 11), 21), ("delta", _delta(3, 1, 13, 11, 5), 30), ("channel_delta", _delta(2, 2, 10, 7, 6), None)], (2, 3, 1)),
+    # no loop; a real model's head sizes
+    "wide": LS.make_robazen(128, 150, [("delta", _delta(2, 1, 128, 128, 4), 64), ("parallel", _pair(8, 2, 128, 128, 80, 30.0, None, 2, 64), None), ("channel_delta", _delta(2, 2, 128, 64, 4), 64)]),
+    # wide heads and values beyond the chunked kernels, many query heads on one key head, a chunk larger than the prompt
+    "beyond": LS.make_robazen(96, 110, [("delta", _delta(2, 2, 160, 200, 4), None), ("parallel", _pair(10, 1, 72, 136, 1000, 50.0, None, 1, 136), 40), ("channel_delta", _delta(1, 1, 136, 40, 7), None)]),
+}
+CONFIGS.update({"robazen_" + k: v for k, v in ROBAZEN.items()})
+ROBAZEN_NAMES = ["robazen_" + k for k in ROBAZEN]
+BOLENEX_NAMES = [k for k in CONFIGS if k not in ROBAZEN_NAMES]
+
+
 def sharp(tensors, cfg, gain=5.0):
     """Query weights scaled up, so that single keys decide the attention."""
     return {k: (LS.bf16_round(v * gain) if k.endswith(".mix.q") else v) for k, v in tensors.items()}

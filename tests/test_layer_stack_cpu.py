@@ -273,7 +273,7 @@ def test_command_line_info(tmp_path, capsys):
 def test_shapes_of_the_synthetic_writer_agree(tmp_path):
     from forge_llm_b200 import synth
     cfg = synth.bolenex_config(64, 2, 3, 48, 77, dim=16, rot_dim=8, vdim=24, kv_rank=32)
-    synth.write_bolenex(str(tmp_path), cfg)
+    synth.write_stack(str(tmp_path), cfg)
     i = _info(str(tmp_path))
     assert i["num_layers"] == 2 and i["vocab_size"] == 77
     t = LS.read_safetensors(os.path.join(str(tmp_path), "model.safetensors"))
