@@ -118,9 +118,11 @@ def unit(x, eps=1e-6):
 
 def delta_rule(q, k, v, beta, g):
     """Token by token: the state decays, is corrected towards v at k, and is read at q behind the write.
-    q, k: [tokens, heads, d], v: [tokens, heads, dv], beta: [tokens, heads], g: [tokens, heads, d] (rows of the state)."""
+    q, k: [tokens, heads, d], v: [tokens, heads, dv], beta: [tokens, heads], g: [tokens, heads, d] (rows of the state).
+    Returns what is read and the last states [heads, d, dv]."""
     n, heads, d = q.shape
     out = np.zeros_like(v)
+    last = []
     for h in range(heads):
         S = np.zeros((d, v.shape[2]), q.dtype)
         for t in range(n):
@@ -128,7 +130,8 @@ def delta_rule(q, k, v, beta, g):
             u = beta[t, h] * (v[t, h] - S.T @ k[t, h])
             S = S + np.outer(k[t, h], u)
             out[t, h] = S.T @ q[t, h]
-    return out
+        last.append(S)
+    return out, np.stack(last)
 
 
 def _delta_inputs(h, w, m):
@@ -140,20 +143,30 @@ def _delta_inputs(h, w, m):
     return q, k, v.reshape(n, H, dv), sigmoid(h @ w("b").T)
 
 
-def gated_delta(h, w, m, eps):
+def gated_delta_states(h, w, m):
     q, k, v, beta = _delta_inputs(h, w, m)
     n, H, dv = v.shape
     g = np.exp(-np.exp(w("A_log")) * softplus(h @ w("a").T + w("dt_bias")))
-    o = delta_rule(q, k, v, beta, np.broadcast_to(g[:, :, None], k.shape))
+    return delta_rule(q, k, v, beta, np.broadcast_to(g[:, :, None], k.shape))
+
+
+def gated_delta(h, w, m, eps):
+    o, _ = gated_delta_states(h, w, m)
+    n, H, dv = o.shape
     o = rms_norm(o, w("norm"), eps) * silu(h @ w("g").T).reshape(n, H, dv)
     return o.reshape(n, H * dv) @ w("o").T
 
 
-def channel_delta(h, w, m, eps):
+def channel_delta_states(h, w, m):
     q, k, v, beta = _delta_inputs(h, w, m)
     n, H, dv = v.shape
     z = ((h @ w("a1").T) @ w("a2").T + w("dt_bias")).reshape(n, H, m["dim"])
-    o = delta_rule(q, k, v, beta, np.exp(-np.exp(w("A_log"))[None, :, None] * softplus(z)))
+    return delta_rule(q, k, v, beta, np.exp(-np.exp(w("A_log"))[None, :, None] * softplus(z)))
+
+
+def channel_delta(h, w, m, eps):
+    o, _ = channel_delta_states(h, w, m)
+    n, H, dv = o.shape
     o = rms_norm(o, w("norm"), eps) * sigmoid((h @ w("g1").T) @ w("g2").T).reshape(n, H, dv)
     return o.reshape(n, H * dv) @ w("o").T
 
@@ -188,18 +201,25 @@ def token_shift(h, mu):
     return h + (before - h) * mu
 
 
-def time_mixing(h, w, m, eps):
+def time_mix_states(h, w, m):
+    """What is read, [tokens, heads, d], and the last states [heads, d, d]."""
     n, H, d = h.shape[0], m["heads"], m["dim"]
     r, k, v = ((token_shift(h, w("mu." + s)) @ w(s).T).reshape(n, H, d) for s in "rkv")
-    gate = silu(token_shift(h, w("mu.g")) @ w("g").T)
     dec = np.exp(-np.exp(np.tanh(token_shift(h, w("mu.w")) @ w("w1").T) @ w("w2").T + w("w0"))).reshape(n, H, d)
-    o = np.zeros_like(v)
+    o, last = np.zeros_like(v), []
     for i in range(H):
         S = np.zeros((d, d), h.dtype)
         for t in range(n):
             o[t, i] = S.T @ r[t, i] + (r[t, i] * w("u")[i] * k[t, i]).sum() * v[t, i]
             S = dec[t, i][:, None] * S + np.outer(k[t, i], v[t, i])
-    o = rms_norm(o, 1.0, eps).reshape(n, H * d) * w("norm") * gate
+        last.append(S)
+    return o, np.stack(last)
+
+
+def time_mixing(h, w, m, eps):
+    o, _ = time_mix_states(h, w, m)
+    gate = silu(token_shift(h, w("mu.g")) @ w("g").T)
+    o = rms_norm(o, 1.0, eps).reshape(gate.shape) * w("norm") * gate
     return o @ w("o").T
 
 

@@ -204,7 +204,7 @@ def test_one_key_stands_out(root, dtype, n, key_pos):
 
 # ------------------------------------------------------------------------------------------------ prompts, decoding, portions
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", list(U.CONFIGS))
+@pytest.mark.parametrize("name", U.BOLENEX_NAMES)
 def test_prompt_decode_and_portions(opened, dtype, name):
     m, orc = opened(name, dtype)
     toks = U.tokens(U.CONFIGS[name], 150)
