@@ -43,14 +43,15 @@ struct RecurArgs {
 };
 
 // per chunk and head, see recurrent_chunk.cu
-struct ChunkScratch { __nv_bfloat16* tp = nullptr; float* scal = nullptr; float* end = nullptr; __nv_bfloat16* dec = nullptr; };
-struct ChunkBytes { size_t tp, scal, end, dec; };   // of one chunk, all heads
+struct ChunkScratch { __nv_bfloat16* half = nullptr; float* f32 = nullptr; };
+struct ChunkBytes { size_t half, f32; };   // of one chunk, all heads
 // scratch of a step with segments
 struct RecurScratch {
     void* conv = nullptr;         // T [rows][channels]: behind convolution and silu
     float* unit = nullptr;        // [rows][2 * groups]: what q and k are multiplied with to be unit vectors (q: times q_scale)
     float* o = nullptr;           // [rows][heads * vdim]
     ChunkScratch chunk;
+    int* err = nullptr;           // set when a bounded wait gave up
 };
 
 bool recur_supported(const RecurDims& d);

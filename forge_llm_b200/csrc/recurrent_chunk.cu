@@ -5,11 +5,13 @@
 //                 o_t = S^T (e^{G_t} q_t) + sum_{s <= t} P_ts u_s,         P_ts = sum_c q_tc k_sc e^{G_tc - G_sc}
 //                 S <- e^{G_end} S + sum_s (e^{G_end - G_s} k_s) u_s^T
 //   time mixing   U = V, o_t reads with e^{G_(t-1)} instead of e^{G_t}, and P_tt = sum_c q_tc bonus_c k_tc.
-// chunk_prep_kernel (every chunk and head at once) forms T = (I + L)^-1 and P, and for decays per channel the decayed q and k;
-// chunk_scan_kernel walks a sequence's chunks with a block of the state's columns in registers.
+// chunk_prep_kernel (every chunk and head at once) inverts I + L and leaves P, U0 = (I + L)^-1 diag(beta) V and
+// W = (I + L)^-1 diag(beta) e^G K, so that U = U0 - W S; chunk_scan_kernel walks a sequence's chunks with a block of 32 columns of
+// the state in registers: two dependent products per chunk (U, then S), the read-out beside them.  What the walk reads lies in
+// memory as the tiles its shared memory holds, so a tile is one bulk copy of a producer warp.
 //
-// Precision: q, k and v are the model's bf16 values; every factor that is not (decays, unit norms, T, P, U, the state) enters a product as a
-// bf16 pair hi + lo, three products with f32 sums for two such factors.  Exponents are differences <= 0, so strong decays
+// Precision: q, k and v are the model's bf16 values; every factor that is not (decays, unit norms, W, P, U, the state) enters a product as
+// a bf16 pair hi + lo, three products with f32 sums for two such factors.  Exponents are differences <= 0, so strong decays
 // underflow to zero and nothing overflows: for decays per channel the pairs of a 16-token block are formed directly, and earlier
 // blocks are reached through the sum at the block's start.
 #include <algorithm>
@@ -17,29 +19,52 @@
 
 #include "mma.cuh"
 #include "recurrent.cuh"
+#include "tc5.cuh"
 
 namespace forge {
 
 namespace {
 
 using bf16 = __nv_bfloat16;
+using tc5::bulk_load;
+using tc5::mbar_arrive;
+using tc5::mbar_expect_tx;
+using tc5::mbar_fence_init;
+using tc5::mbar_init;
+using tc5::mbar_wait;
 
 constexpr int C = kRecurChunk;          // tokens of a chunk
-constexpr int LDT = C + 8;
+constexpr int NB = 32;                  // value columns of a CTA of the walk
+constexpr int LDT = C + 8, LDN = NB + 8, TT = C * LDT, VT = C * LDN;
 enum Mode { HEAD_DELTA = 0, CHANNEL_DELTA = 1, TIME_MIX = 2 };
+constexpr float kLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return uint32_t(__cvta_generic_to_shared(p)); }
-
-// per (chunk, head): bf16 [2][64][64] T and P (hi, lo); f32 scal[4][64]; f32 end[dim] = e^{G_end}; decays per channel also
-// bf16 [3][2][64][DK]: k with e^G (delta rule only), q with e^G, k with e^{G_end - G}
-struct ChunkPtr {
-    bf16* T; bf16* P; float* scal; float* end; bf16* dec;
-};
-__device__ __forceinline__ ChunkPtr chunk_ptr(const ChunkScratch& s, int chunk, int heads, int h, int DK) {
-    const size_t i = size_t(chunk) * heads + h;
-    return {s.tp + i * 4 * C * C, s.tp + i * 4 * C * C + 2 * C * C, s.scal + i * 4 * C, s.end + i * DK, s.dec + i * 6 * C * DK};
+__device__ __forceinline__ float ex2(float x) {   // 2^x
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
 }
-constexpr int kScalKin = 0, kScalQin = C, kScalKout = 2 * C, kScalBeta = 3 * C;   // scal: e^G |k|^-1, e^G q scale, e^{G_end - G} |k|^-1, beta
+
+// What one chunk of one head leaves for the walk.  bf16 tiles: W hi, lo (delta rules); q (hi, lo where decays are per channel); k (the same);
+// P hi, lo; v in blocks of 32 columns (time mixing).  f32: U0 in blocks [64][32] (delta rules), scale of q and of k's update per
+// token (decay per head), e^{G_end} per channel.
+template <int DK, int MODE> struct Rec {
+    static constexpr int LDK = DK + 8, KT = C * LDK;
+    static constexpr int nw = MODE == TIME_MIX ? 0 : 2, nx = MODE == HEAD_DELTA ? 1 : 2;
+    static constexpr int oq = nw * KT, ok = oq + nx * KT, op = ok + nx * KT, ov = op + 2 * TT;
+    static __host__ __device__ size_t halves(int nb) { return size_t(ov) + (MODE == TIME_MIX ? size_t(nb) * VT : 0); }
+    static __host__ __device__ size_t floats(int nb) { return (MODE == TIME_MIX ? 0 : size_t(nb) * C * NB) + 2 * C + DK; }
+    bf16* h; float* f;
+    float *scal, *end;
+    __device__ __forceinline__ Rec(const ChunkScratch& s, int chunk, int heads, int head, int nb) {
+        const size_t i = size_t(chunk) * heads + head;
+        h = s.half + i * halves(nb);
+        f = s.f32 + i * floats(nb);
+        scal = f + (MODE == TIME_MIX ? 0 : size_t(nb) * C * NB);
+        end = scal + 2 * C;
+    }
+};
 
 // t = (I + L)^-1 for the strictly lower L in l (what l holds on and above the diagonal is ignored); 64 rows of LDL floats each, the blocks
 // above t's diagonal blocks are not written; tmp: 3 x 16 x 17 floats
@@ -81,72 +106,85 @@ __device__ __forceinline__ void invert_unit_lower(float* t, const float* l, floa
     }
 }
 
-// lower triangle of an f32 matrix (LDL apart) -> [2][64][64] hi, lo with zeros above
+// lower triangle of an f32 matrix (LDL apart), its columns times `col` -> bf16 hi and lo tiles with zeros above
 template <int NT>
-__device__ __forceinline__ void store_lower(bf16* dst, const float* src, int tid) {
+__device__ __forceinline__ void put_lower(bf16* dst, const float* src, const float* col, int tid) {
     for (int e = tid; e < C * C / 2; e += NT) {
         const int r = e / (C / 2), c = (e % (C / 2)) * 2;
         uint32_t hi, lo;
-        split_bf16x2(c <= r ? src[r * LDL + c] : 0.f, c + 1 <= r ? src[r * LDL + c + 1] : 0.f, hi, lo);
-        reinterpret_cast<uint32_t*>(dst)[e] = hi;
-        reinterpret_cast<uint32_t*>(dst + C * C)[e] = lo;
+        split_bf16x2(c <= r ? src[r * LDL + c] * (col ? col[c] : 1.f) : 0.f, c + 1 <= r ? src[r * LDL + c + 1] * (col ? col[c + 1] : 1.f) : 0.f, hi, lo);
+        *reinterpret_cast<uint32_t*>(dst + r * LDT + c) = hi;
+        *reinterpret_cast<uint32_t*>(dst + TT + r * LDT + c) = lo;
     }
 }
 
 template <int DK, int MODE> struct Prep {
     static constexpr int NT = MODE == HEAD_DELTA ? 256 : 512, LDK = DK + 8;
     static constexpr bool CH = MODE != HEAD_DELTA;
-    static constexpr size_t tiles = size_t(2) * C * LDK * 2;                          // q, k
-    static constexpr size_t mats = size_t(2) * C * LDL * 4 + 3 * 272 * 4;             // L / T, P, tmp
-    static constexpr size_t chan = CH ? size_t(C) * DK * 4 + size_t(5) * DK * 4 + size_t(2) * (32 + 48) * LDK * 2 : 0;   // sums, block sums, operands of one block row
+    static constexpr size_t tiles = size_t(2) * C * LDK * 2;                          // q (later v), k
+    static constexpr size_t mats = size_t(2) * C * LDL * 4 + 3 * 272 * 4;             // L (later (I + L)^-1 as hi, lo), P (later (I + L)^-1), tmp
+    static constexpr size_t chan = CH ? size_t(C) * DK * 4 + size_t(5) * DK * 4 + size_t(2) * (32 + 48) * LDK * 2 : 0;   // sums, block sums, operands of one block row (later decayed k)
     static constexpr size_t smem = tiles + mats + chan;
+    static_assert(size_t(2) * TT * 2 <= size_t(C) * LDL * 4 + 3 * 272 * 4, "hi and lo fit where L and tmp lay");
 };
 
 template <int DK, int MODE>
 __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs, int n_segs) {
     using L = Prep<DK, MODE>;
-    constexpr int NT = L::NT, LDK = L::LDK, NW = NT / 32;
+    using R = Rec<DK, MODE>;
+    constexpr int NT = L::NT, LDK = L::LDK, NW = NT / 32, KT = R::KT;
     extern __shared__ __align__(16) unsigned char sm_raw[];
     bf16* sq = reinterpret_cast<bf16*>(sm_raw);
     bf16* sk = sq + C * LDK;
-    float* sl = reinterpret_cast<float*>(sm_raw + L::tiles);
-    float* sp = sl + C * LDL;
-    float* tmp = sp + C * LDL;
-    float* sg = tmp + 3 * 272;                 // [64][DK] sums of the log decays inside their 16-token block
+    float* sp = reinterpret_cast<float*>(sm_raw + L::tiles);
+    float* sl = sp + C * LDL;
+    float* tmp = sl + C * LDL;                 // behind sl: both give way to the inverse's bf16 tiles
+    float* sg = tmp + 3 * 272;                 // [64][DK] sums of the log decays inside their 16-token block (base 2)
     float* sb = sg + C * DK;                   // [5][DK] sums in front of each block, and the chunk's
     bf16* sa = reinterpret_cast<bf16*>(sb + 5 * DK);   // [2][32][LDK] rows k, then q, of a block row
     bf16* so = sa + 2 * 32 * LDK;              // [2][48][LDK] keys in front of it
-    __shared__ float s_scal[4][C], s_gt[C];
-    __shared__ int s_find[3];
+    bf16* st = reinterpret_cast<bf16*>(sl);    // [2][64][LDT]
+    __shared__ float s_ks[C], s_qs[C], s_beta[C], s_gt[C], s_col[C];
+    __shared__ int s_seg;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int chunk = blockIdx.x, h = blockIdx.y, g = h / (d.heads / d.groups);
-    if (tid < n_segs && segs[tid].chunk0 <= chunk && chunk < segs[tid].chunk0 + (segs[tid].n + C - 1) / C) s_find[0] = tid;
-    for (int i = tid + NT; i < n_segs; i += NT) if (segs[i].chunk0 <= chunk && chunk < segs[i].chunk0 + (segs[i].n + C - 1) / C) s_find[0] = i;
+    const int chunk = blockIdx.x, h = blockIdx.y, g = h / (d.heads / d.groups), nb = (d.vdim + NB - 1) / NB;
+    for (int i = tid; i < n_segs; i += NT) if (segs[i].chunk0 <= chunk && chunk < segs[i].chunk0 + (segs[i].n + C - 1) / C) s_seg = i;
     __syncthreads();
-    const ScanSeg s = segs[s_find[0]];
+    const ScanSeg s = segs[s_seg];
     const int t0 = (chunk - s.chunk0) * C, n = min(C, s.n - t0), row0 = s.row0 + t0;
-    const ChunkPtr out = chunk_ptr(sc.chunk, chunk, d.heads, h, DK);
+    const R out(sc.chunk, chunk, d.heads, h, nb);
     const bf16* x = MODE == TIME_MIX ? static_cast<const bf16*>(a.x) : static_cast<const bf16*>(sc.conv);
     const size_t ld = MODE == TIME_MIX ? a.x_ld : d.channels();
-    for (int i = tid; i < 2 * C * (DK / 8); i += NT) {
-        const int which = i / (C * (DK / 8)), t = i / (DK / 8) % C, c = (i % (DK / 8)) * 8;
-        const bool ok = t < n && c < d.dim;
-        cp_async16(smem_addr((which ? sk : sq) + t * LDK + c), ok ? x + size_t(row0 + t) * ld + which * d.qk() + g * d.dim + c : x, ok);
-    }
+    // [64] rows of the step, `cols` of its columns from col0 (zeros past `valid`)
+    auto fetch = [&](bf16* dst, int l, int col0, int cols, int valid) {
+        for (int i = tid; i < C * (cols / 8); i += NT) {
+            const int t = i / (cols / 8), c = (i % (cols / 8)) * 8;
+            const bool ok = t < n && c < valid;
+            cp_async16(smem_addr(dst + t * l + c), ok ? x + size_t(row0 + t) * ld + col0 + c : x, ok);
+        }
+    };
+    fetch(sq, LDK, g * d.dim, DK, d.dim);
+    fetch(sk, LDK, d.qk() + g * d.dim, DK, d.dim);
     cp_commit();
     if (tid < C) {
         const bool ok = tid < n;
+        s_ks[tid] = s_qs[tid] = s_beta[tid] = 1.f;
         if constexpr (MODE != TIME_MIX) {
-            s_scal[0][tid] = ok ? sc.unit[size_t(row0 + tid) * 2 * d.groups + d.groups + g] : 0.f;   // |k|^-1
-            s_scal[1][tid] = ok ? sc.unit[size_t(row0 + tid) * 2 * d.groups + g] : 0.f;              // q scale
-            s_scal[3][tid] = ok ? a.beta[size_t(row0 + tid) * d.heads + h] : 0.f;
-        } else { s_scal[0][tid] = s_scal[1][tid] = 1.f; }
-        if constexpr (MODE == HEAD_DELTA) s_gt[tid] = ok ? a.decay[size_t(row0 + tid) * a.decay_ld + h] : 0.f;
+            s_ks[tid] = ok ? sc.unit[size_t(row0 + tid) * 2 * d.groups + d.groups + g] : 0.f;   // |k|^-1
+            s_qs[tid] = ok ? sc.unit[size_t(row0 + tid) * 2 * d.groups + g] : 0.f;              // q scale
+            s_beta[tid] = ok ? a.beta[size_t(row0 + tid) * d.heads + h] : 0.f;
+        }
+        if constexpr (MODE == HEAD_DELTA) s_gt[tid] = ok ? a.decay[size_t(row0 + tid) * a.decay_ld + h] * kLog2e : 0.f;
     }
     if constexpr (L::CH) {
-        for (int i = tid; i < C * DK; i += NT) {
-            const int t = i / DK, c = i % DK;
-            sg[i] = t < n && c < d.dim ? a.decay[size_t(row0 + t) * a.decay_ld + h * d.dim + c] : 0.f;
+        // sums inside the blocks: a thread per block and channel
+        for (int i = tid; i < 4 * DK; i += NT) {
+            const int b = i / DK, c = i % DK;
+            float v[16], sum = 0.f;
+#pragma unroll
+            for (int t = 0; t < 16; ++t) v[t] = b * 16 + t < n && c < d.dim ? a.decay[size_t(row0 + b * 16 + t) * a.decay_ld + h * d.dim + c] : 0.f;
+#pragma unroll
+            for (int t = 0; t < 16; ++t) { sum = fmaf(v[t], kLog2e, sum); sg[(b * 16 + t) * DK + c] = sum; }
         }
     }
     cp_wait<0>();
@@ -176,12 +214,12 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
             uint32_t fa[4];
             (is_q ? mq : mk).a(fa, mt * 16, kt * 16, lane);
 #pragma unroll
-            for (int nb = 0; nb < 4; ++nb)
-                if (nb <= mt) {
+            for (int b = 0; b < 4; ++b)
+                if (b <= mt) {
                     uint32_t fb[4];
-                    mk.b(fb, nb * 16, kt * 16, lane);
-                    mma(acc[2 * nb], fa, fb[0], fb[1]);
-                    mma(acc[2 * nb + 1], fa, fb[2], fb[3]);
+                    mk.b(fb, b * 16, kt * 16, lane);
+                    mma(acc[2 * b], fa, fb[0], fb[1]);
+                    mma(acc[2 * b + 1], fa, fb[2], fb[3]);
                 }
         }
         __syncthreads();
@@ -192,356 +230,353 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
             for (int e = 0; e < 4; ++e) {
                 const int t = mt * 16 + lr + (e >> 1) * 8, c = i * 8 + lc + (e & 1);
                 if (i / 2 > mt) continue;
-                float v = 0.f;
-                if (is_q ? c <= t : c < t) v = acc[i][e] * s_scal[0][c] * expf(s_gt[t] - s_gt[c]) * (is_q ? s_scal[1][t] : s_scal[0][t] * s_scal[3][t]);
-                dst[t * LDL + c] = v;
+                dst[t * LDL + c] = c <= t ? acc[i][e] * s_ks[c] * ex2(s_gt[t] - s_gt[c]) * (is_q ? s_qs[t] : s_ks[t] * s_beta[t]) : 0.f;
             }
-        __syncthreads();
         if (tid < C) {
-            const float e = expf(s_gt[tid]);
-            out.scal[kScalKin + tid] = e * s_scal[0][tid];
-            out.scal[kScalQin + tid] = e * s_scal[1][tid];
-            out.scal[kScalKout + tid] = expf(s_gt[C - 1] - s_gt[tid]) * s_scal[0][tid];
-            out.scal[kScalBeta + tid] = s_scal[3][tid];
+            const float e = ex2(s_gt[tid]);
+            s_col[tid] = e * s_ks[tid];
+            out.scal[tid] = e * s_qs[tid];
+            out.scal[C + tid] = ex2(s_gt[C - 1] - s_gt[tid]) * s_ks[tid];
         }
-        if (tid < DK) out.end[tid] = expf(s_gt[C - 1]);
-    } else {
-        // sums inside the blocks, then in front of them
-        for (int i = tid; i < 4 * DK; i += NT) {
-            const int b = i / DK, c = i % DK;
-            float sum = 0.f;
-#pragma unroll
-            for (int t = 0; t < 16; ++t) { sum += sg[(b * 16 + t) * DK + c]; sg[(b * 16 + t) * DK + c] = sum; }
-        }
+        if (tid < DK) out.end[tid] = ex2(s_gt[C - 1]);
+        for (int i = tid; i < 2 * KT / 8; i += NT) reinterpret_cast<uint4*>(out.h + R::oq)[i] = reinterpret_cast<const uint4*>(sq)[i];   // q, k as they are (padding columns too)
         __syncthreads();
+    } else {
         for (int c = tid; c < DK; c += NT) {
             float sum = 0.f;
 #pragma unroll
             for (int b = 0; b < 4; ++b) { sb[b * DK + c] = sum; sum += sg[(b * 16 + 15) * DK + c]; }
             sb[4 * DK + c] = sum;
-            out.end[c] = expf(sum);
+            out.end[c] = ex2(sum);
         }
-        __syncthreads();
-        // exponent of a query row inside its block: up to and including its own decay, or for time mixing without it
-        auto sum_q = [&](int t, int c) { return MODE == TIME_MIX ? (t & 15 ? sg[(t - 1) * DK + c] : 0.f) : sg[t * DK + c]; };
-        // pairs inside a block: a warp per row, lanes share the channels
+        // exponents of a query row inside its block: up to and including its own decay, or for time mixing without it
+        auto sum_q = [&](int t) { return MODE == TIME_MIX ? sg + (t - 1) * DK : sg + t * DK; };
+        auto first = [](int t) { return MODE == TIME_MIX && !(t & 15); };   // then they are zero
+        // pairs inside a block: a warp per row, DK / 32 neighbouring channels per lane, sixteen partners at once
+        constexpr int PL = DK / 32;
         for (int t = warp; t < C; t += NW) {
-            constexpr int PL = DK / 32;
-            float qv[PL], kv[PL], eq[PL], ek[PL];
+            float qv[PL], kv[PL], eq[PL];
+            const int c = lane * PL;
 #pragma unroll
             for (int i = 0; i < PL; ++i) {
-                const int c = lane + 32 * i;
-                qv[i] = __bfloat162float(sq[t * LDK + c]); kv[i] = __bfloat162float(sk[t * LDK + c]);
-                eq[i] = sum_q(t, c); ek[i] = sg[t * DK + c];
+                qv[i] = __bfloat162float(sq[t * LDK + c + i]); kv[i] = __bfloat162float(sk[t * LDK + c + i]);
+                eq[i] = first(t) ? 0.f : sum_q(t)[c + i];
             }
-            for (int u = t & ~15; u <= t; ++u) {
-                float pq = 0.f, pk = 0.f;
+            float part[32];   // P of the sixteen partners, then L
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+                const int u = (t & ~15) + j;
+                part[j] = part[16 + j] = 0.f;
+                if (u > t) continue;
 #pragma unroll
                 for (int i = 0; i < PL; ++i) {
-                    const int c = lane + 32 * i;
-                    const float ku = __bfloat162float(sk[u * LDK + c]), gu = sg[u * DK + c];
-                    if constexpr (MODE == TIME_MIX) pq = fmaf(qv[i] * ku, u < t ? expf(eq[i] - gu) : c < d.dim ? a.bonus[h * d.dim + c] : 0.f, pq);
-                    else { const float e = expf(ek[i] - gu) * ku; pq = fmaf(qv[i], e, pq); pk = fmaf(kv[i], e, pk); }
-                }
-                pq = warp_sum(pq);
-                if constexpr (MODE != TIME_MIX) pk = warp_sum(pk);
-                if (lane == 0) {
-                    sp[t * LDL + u] = pq * s_scal[1][t] * s_scal[0][u];
-                    if constexpr (MODE != TIME_MIX) sl[t * LDL + u] = pk * s_scal[3][t] * s_scal[0][t] * s_scal[0][u];
+                    const float ku = __bfloat162float(sk[u * LDK + c + i]), gu = sg[u * DK + c + i];
+                    if constexpr (MODE == TIME_MIX) part[j] = fmaf(qv[i] * ku, u < t ? ex2(eq[i] - gu) : c + i < d.dim ? a.bonus[h * d.dim + c + i] : 0.f, part[j]);
+                    else { const float e = ex2(eq[i] - gu) * ku; part[j] = fmaf(qv[i], e, part[j]); part[16 + j] = fmaf(kv[i], e, part[16 + j]); }
                 }
             }
+            // lane l ends with the sum of part[l]
+#pragma unroll
+            for (int w = 16; w > 0; w >>= 1)
+#pragma unroll
+                for (int i = 0; i < w; ++i) {
+                    const bool up = lane & w;
+                    const float send = up ? part[i] : part[i + w], mine = up ? part[i + w] : part[i];
+                    part[i] = mine + __shfl_xor_sync(0xffffffffu, send, w);
+                }
+            const int j = lane & 15, u = (t & ~15) + j;
+            if (u <= t) {
+                if (lane < 16) sp[t * LDL + u] = part[0] * s_qs[t] * s_ks[u];
+                else if (MODE != TIME_MIX) sl[t * LDL + u] = part[0] * s_beta[t] * s_ks[t] * s_ks[u];
+            }
         }
+        __syncthreads();
         // earlier blocks, reached through the sum at the block's start
         for (int b = 1; b < 4; ++b) {
-            __syncthreads();
             for (int i = tid; i < (32 + 16 * b) * (DK / 2); i += NT) {
-                const int r = i / (DK / 2), c = (i % (DK / 2)) * 2;
-                float v[2];
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    if (r < 16) v[e] = __bfloat162float(sk[(b * 16 + r) * LDK + c + e]) * expf(sg[(b * 16 + r) * DK + c + e]);
-                    else if (r < 32) v[e] = __bfloat162float(sq[(b * 16 + r - 16) * LDK + c + e]) * expf(sum_q(b * 16 + r - 16, c + e));
-                    else {
-                        const int u = r - 32;
-                        v[e] = __bfloat162float(sk[u * LDK + c + e]) * expf(sb[b * DK + c + e] - sb[(u >> 4) * DK + c + e] - sg[u * DK + c + e]);
-                    }
+                const int r = i / (DK / 2), c = (i % (DK / 2)) * 2, t = b * 16 + (r & 15), u = r - 32;
+                const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>((r < 16 ? sk + t * LDK : r < 32 ? sq + t * LDK : sk + u * LDK) + c));
+                float2 e;
+                if (r < 16) e = *reinterpret_cast<const float2*>(sg + t * DK + c);
+                else if (r < 32) e = first(t) ? make_float2(0.f, 0.f) : *reinterpret_cast<const float2*>(sum_q(t) + c);
+                else {
+                    const float2 f = *reinterpret_cast<const float2*>(sb + b * DK + c), o = *reinterpret_cast<const float2*>(sb + (u >> 4) * DK + c), w = *reinterpret_cast<const float2*>(sg + u * DK + c);
+                    e = make_float2(f.x - o.x - w.x, f.y - o.y - w.y);
                 }
                 uint32_t hi, lo;
-                split_bf16x2(v[0], v[1], hi, lo);
-                bf16* dst = r < 32 ? sa + r * LDK + c : so + (r - 32) * LDK + c;
+                split_bf16x2(v.x * ex2(e.x), v.y * ex2(e.y), hi, lo);
+                bf16* dst = r < 32 ? sa + r * LDK + c : so + u * LDK + c;
                 *reinterpret_cast<uint32_t*>(dst) = hi;
                 *reinterpret_cast<uint32_t*>(dst + (r < 32 ? 32 : 48) * LDK) = lo;
             }
             __syncthreads();
             const SmemMat ah{smem_addr(sa), LDK}, al{smem_addr(sa + 32 * LDK), LDK}, bh{smem_addr(so), LDK}, bl{smem_addr(so + 48 * LDK), LDK};
-            for (int w = warp; w < 2 * b; w += NW) {   // (k or q) x 16 earlier keys
-                const int is_q = w & 1, nb = w >> 1;
+            for (int w = warp; w < 4 * b; w += NW) {   // (k or q) x 8 earlier keys
+                const int is_q = w & 1, n8 = w >> 1;
                 if (MODE == TIME_MIX && !is_q) continue;
-                float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+                float acc[3][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
                 for (int kt = 0; kt < DK / 16; ++kt) {
                     uint32_t fh[4], fl[4], gh[4], gl[4];
                     ah.a(fh, is_q * 16, kt * 16, lane); al.a(fl, is_q * 16, kt * 16, lane);
-                    bh.b(gh, nb * 16, kt * 16, lane); bl.b(gl, nb * 16, kt * 16, lane);
-#pragma unroll
-                    for (int j = 0; j < 2; ++j) {
-                        mma(acc[j], fl, gh[2 * j], gh[2 * j + 1]);
-                        mma(acc[j], fh, gl[2 * j], gl[2 * j + 1]);
-                        mma(acc[j], fh, gh[2 * j], gh[2 * j + 1]);
-                    }
+                    bh.b(gh, (n8 >> 1) * 16, kt * 16, lane); bl.b(gl, (n8 >> 1) * 16, kt * 16, lane);
+                    const int j = (n8 & 1) * 2;
+                    mma(acc[0], fl, j ? gh[2] : gh[0], j ? gh[3] : gh[1]);
+                    mma(acc[1], fh, j ? gl[2] : gl[0], j ? gl[3] : gl[1]);
+                    mma(acc[2], fh, j ? gh[2] : gh[0], j ? gh[3] : gh[1]);
                 }
                 float* dst = is_q ? sp : sl;
 #pragma unroll
-                for (int j = 0; j < 2; ++j)
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        const int t = b * 16 + lr + (e >> 1) * 8, u = nb * 16 + j * 8 + lc + (e & 1);
-                        dst[t * LDL + u] = acc[j][e] * s_scal[0][u] * (is_q ? s_scal[1][t] : s_scal[0][t] * s_scal[3][t]);
-                    }
+                for (int e = 0; e < 4; ++e) {
+                    const int t = b * 16 + lr + (e >> 1) * 8, u = n8 * 8 + lc + (e & 1);
+                    dst[t * LDL + u] = (acc[0][e] + acc[1][e] + acc[2][e]) * s_ks[u] * (is_q ? s_qs[t] : s_ks[t] * s_beta[t]);
+                }
             }
+            __syncthreads();
         }
-        // q and k with their decays, for the walk over the state
+        // q and k with their decays: for the walk, and k as an operand of W
         for (int i = tid; i < C * (DK / 2); i += NT) {
             const int t = i / (DK / 2), c = (i % (DK / 2)) * 2, b = t >> 4;
-            const __nv_bfloat162 q2 = *reinterpret_cast<const __nv_bfloat162*>(sq + t * LDK + c), k2 = *reinterpret_cast<const __nv_bfloat162*>(sk + t * LDK + c);
-            const float2 q = __bfloat1622float2(q2), k = __bfloat1622float2(k2);
-            const float f0 = sb[b * DK + c], f1 = sb[b * DK + c + 1], g0 = sg[t * DK + c], g1 = sg[t * DK + c + 1];
-            const float ks = s_scal[0][t], qs = s_scal[1][t];
+            const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sq + t * LDK + c)), k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sk + t * LDK + c));
+            const float2 f = *reinterpret_cast<const float2*>(sb + b * DK + c), w = *reinterpret_cast<const float2*>(sg + t * DK + c), end = *reinterpret_cast<const float2*>(sb + 4 * DK + c);
+            const float2 wq = first(t) ? make_float2(0.f, 0.f) : *reinterpret_cast<const float2*>(sum_q(t) + c);
+            const float ks = s_ks[t], qs = s_qs[t];
             uint32_t hi, lo;
-            uint32_t* dst = reinterpret_cast<uint32_t*>(out.dec) + i;
-            constexpr int M = C * DK / 2;
+            split_bf16x2(q.x * qs * ex2(f.x + wq.x), q.y * qs * ex2(f.y + wq.y), hi, lo);
+            uint32_t* dst = reinterpret_cast<uint32_t*>(out.h + R::oq + t * LDK + c);
+            dst[0] = hi; dst[KT / 2] = lo;
+            split_bf16x2(k.x * ks * ex2(end.x - f.x - w.x), k.y * ks * ex2(end.y - f.y - w.y), hi, lo);
+            dst = reinterpret_cast<uint32_t*>(out.h + R::ok + t * LDK + c);
+            dst[0] = hi; dst[KT / 2] = lo;
             if constexpr (MODE != TIME_MIX) {
-                split_bf16x2(k.x * ks * expf(f0 + g0), k.y * ks * expf(f1 + g1), hi, lo);
-                dst[0] = hi; dst[M] = lo;
+                split_bf16x2(k.x * ks * ex2(f.x + w.x), k.y * ks * ex2(f.y + w.y), hi, lo);
+                dst = reinterpret_cast<uint32_t*>(sa + t * LDK + c);
+                dst[0] = hi; dst[KT / 2] = lo;
             }
-            split_bf16x2(q.x * qs * expf(f0 + sum_q(t, c)), q.y * qs * expf(f1 + sum_q(t, c + 1)), hi, lo);
-            dst[2 * M] = hi; dst[3 * M] = lo;
-            split_bf16x2(k.x * ks * expf(sb[4 * DK + c] - f0 - g0), k.y * ks * expf(sb[4 * DK + c + 1] - f1 - g1), hi, lo);
-            dst[4 * M] = hi; dst[5 * M] = lo;
         }
-        if constexpr (MODE != TIME_MIX) if (tid < C) out.scal[kScalBeta + tid] = s_scal[3][tid];
-        __syncthreads();
+        if constexpr (MODE == TIME_MIX) {   // v as the walk's tiles
+            for (int i = tid; i < nb * C * (NB / 8); i += NT) {
+                const int blk = i / (C * (NB / 8)), t = i / (NB / 8) % C, c = (i % (NB / 8)) * 8;
+                const bool ok = t < n && blk * NB + c < d.vdim;
+                *reinterpret_cast<uint4*>(out.h + R::ov + size_t(blk) * VT + t * LDN + c) =
+                    ok ? *reinterpret_cast<const uint4*>(x + size_t(row0 + t) * ld + 2 * d.qk() + h * d.vdim + blk * NB + c) : make_uint4(0, 0, 0, 0);
+            }
+        }
     }
-    store_lower<NT>(out.P, sp, tid);
+    put_lower<NT>(out.h + R::op, sp, nullptr, tid);
     if constexpr (MODE != TIME_MIX) {
         __syncthreads();
-        invert_unit_lower<NT>(sp, sl, tmp, tid);   // P is stored: its place takes T
-        store_lower<NT>(out.T, sp, tid);
+        fetch(sq, LDK, 2 * d.qk() + h * d.vdim, DK, d.vdim);   // q gives way to the first columns of v
+        cp_commit();
+        invert_unit_lower<NT>(sp, sl, tmp, tid);               // P is stored: its place takes the inverse
+        put_lower<NT>(st, sp, s_beta, tid);
+        cp_wait<0>();
+        __syncthreads();
+        const SmemMat th{smem_addr(st), LDT}, tl{smem_addr(st + TT), LDT};
+        // [64][cols] = (I + L)^-1 diag(beta) B in blocks of 16 x 16, B as one bf16 matrix or as hi and lo
+        auto product = [&](const bf16* B, bool pair, int cols, auto store) {
+            const SmemMat bh{smem_addr(B), LDK}, bl{smem_addr(B + KT), LDK};
+            for (int w = warp; w < 4 * (cols / 16); w += NW) {
+                const int mt = 3 - (w & 3), n0 = (w >> 2) * 16;
+                float acc[2][2][4];
+#pragma unroll
+                for (int i = 0; i < 16; ++i) acc[i >> 3][(i >> 2) & 1][i & 3] = 0.f;
+#pragma unroll
+                for (int kt = 0; kt < C / 16; ++kt)
+                    if (kt <= mt) {
+                        uint32_t fh[4], fl[4], gh[4], gl[4];
+                        th.a(fh, mt * 16, kt * 16, lane); tl.a(fl, mt * 16, kt * 16, lane);
+                        bh.b_t(gh, kt * 16, n0, lane);
+                        if (pair) bl.b_t(gl, kt * 16, n0, lane);
+#pragma unroll
+                        for (int j = 0; j < 2; ++j) {
+                            mma(acc[0][j], fl, gh[2 * j], gh[2 * j + 1]);
+                            if (pair) mma(acc[0][j], fh, gl[2 * j], gl[2 * j + 1]);
+                            mma(acc[1][j], fh, gh[2 * j], gh[2 * j + 1]);
+                        }
+                    }
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) store(mt * 16 + lr + e * 8, n0 + j * 8 + lc, acc[0][j][2 * e] + acc[1][j][2 * e], acc[0][j][2 * e + 1] + acc[1][j][2 * e + 1]);
+            }
+        };
+        for (int c0 = 0; c0 < d.vdim; c0 += DK) {   // U0
+            if (c0) {
+                __syncthreads();
+                fetch(sq, LDK, 2 * d.qk() + h * d.vdim + c0, DK, d.vdim - c0);
+                cp_commit();
+                cp_wait<0>();
+                __syncthreads();
+            }
+            product(sq, false, min(DK, (d.vdim - c0 + 15) / 16 * 16), [&](int t, int c, float vx, float vy) {
+                *reinterpret_cast<float2*>(out.f + size_t((c0 + c) / NB) * C * NB + t * NB + (c0 + c) % NB) = make_float2(vx, vy);
+            });
+        }
+        if constexpr (MODE == HEAD_DELTA) {         // W: the decay of k goes into the inverse's columns
+            __syncthreads();
+            if (tid < C) s_col[tid] *= s_beta[tid];
+            __syncthreads();
+            put_lower<NT>(st, sp, s_col, tid);
+            __syncthreads();
+        }
+        product(MODE == HEAD_DELTA ? sk : sa, MODE != HEAD_DELTA, DK, [&](int t, int c, float vx, float vy) {
+            uint32_t hi, lo;
+            split_bf16x2(vx, vy, hi, lo);
+            uint32_t* dst = reinterpret_cast<uint32_t*>(out.h + t * LDK + c);
+            dst[0] = hi; dst[KT / 2] = lo;
+        });
     }
 }
 
 // ------------------------------------------------------------------------------------------------ walk over the chunks
-constexpr int NB = 32, LDN = NB + 8;   // value columns of a CTA
-
 template <int DK, int MODE> struct Scan {
-    static constexpr int LDK = DK + 8;
-    static constexpr int KT = C * LDK, TT = C * LDT, VT = C * LDN;            // elements of the tiles
-    // k (two buffers for exact k; hi and lo otherwise), q (one; hi, lo), k for the update (hi, lo)
-    static constexpr int nk = MODE == TIME_MIX ? 0 : 2, nq = MODE == HEAD_DELTA ? 1 : 2, no = MODE == HEAD_DELTA ? 0 : 2;
-    static constexpr int oq = nk * KT, oo = oq + nq * KT, ot = oo + no * KT, op = ot + (MODE == TIME_MIX ? 0 : 2 * TT), ov = op + 2 * TT, os = ov + VT,
-                         orr = os + 2 * DK * LDN, ou = orr + (MODE == TIME_MIX ? 0 : 2 * VT), ow = ou + (MODE == TIME_MIX ? 0 : 2 * VT), total = ow + (MODE == HEAD_DELTA ? 2 * VT : 0);
-    static constexpr size_t smem = size_t(total) * 2 + 2 * (4 * C + DK) * 4;
+    using R = Rec<DK, MODE>;
+    static constexpr int SS = DK * LDN;                              // one half of a state buffer
+    static constexpr int ow = 0, oq = R::nw * R::KT, ok = oq + R::nx * R::KT, op = ok + R::nx * R::KT, ov = op + 2 * TT, os = ov + (MODE == TIME_MIX ? VT : 0),
+                         ou = os + 4 * SS, ox = ou + (MODE == TIME_MIX ? 0 : 2 * VT), total = ox + (MODE == HEAD_DELTA ? 2 * VT : 0);
+    static constexpr size_t smem = size_t(total) * 2 + 16;
 };
 
+constexpr int kScanThreads = 288;   // eight warps of products and a producer
+__device__ __forceinline__ void walk_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+
 template <int DK, int MODE>
-__global__ void __launch_bounds__(256) chunk_scan_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs) {
+__global__ void __launch_bounds__(kScanThreads) chunk_scan_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs, int* err) {
     using L = Scan<DK, MODE>;
-    constexpr int LDK = L::LDK, NT = 256;
+    using R = Rec<DK, MODE>;
+    constexpr int LDK = R::LDK, KT = R::KT;
     extern __shared__ __align__(16) unsigned char sm_raw[];
     bf16* sm = reinterpret_cast<bf16*>(sm_raw);
-    float* s_scal = reinterpret_cast<float*>(sm + L::total);   // [2][4 * 64]
-    float* s_end = s_scal + 2 * 4 * C;                         // [2][DK]
+    enum { BW, BK, BQ, BP, BUFS };
+    __shared__ uint64_t full[BUFS], empty[BUFS];
+    __shared__ int s_err;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lr = lane >> 2, lc = (lane & 3) * 2;
     const ScanSeg s = segs[blockIdx.z];
-    const int h = blockIdx.y, g = h / (d.heads / d.groups), c0 = blockIdx.x * NB;
-    const int chunks = (s.n + C - 1) / C;
-    const bf16* x = MODE == TIME_MIX ? static_cast<const bf16*>(a.x) : static_cast<const bf16*>(sc.conv);
-    const size_t ld = MODE == TIME_MIX ? a.x_ld : d.channels();
-    auto mat = [&](int off, int l) { return SmemMat{smem_addr(sm + off), l}; };
-
-    // [64][cols] bf16 rows of a dense scratch matrix
-    auto copy_rows = [&](int off, int l, const bf16* src, int cols) {
-        for (int i = tid; i < C * (cols / 8); i += NT) {
-            const int r = i / (cols / 8), c = (i % (cols / 8)) * 8;
-            cp_async16(smem_addr(sm + off + r * l + c), src + size_t(r) * cols + c, true);
-        }
-    };
-    // [64][DK] rows of the step's q or k (which = 0, 1), or [64][NB] of v (2)
-    auto copy_x = [&](int off, int l, int ch, int which) {
-        const int cols = which == 2 ? NB : DK, valid = which == 2 ? min(NB, d.vdim - c0) : d.dim;
-        const int col0 = which == 2 ? 2 * d.qk() + h * d.vdim + c0 : which * d.qk() + g * d.dim;
-        for (int i = tid; i < C * (cols / 8); i += NT) {
-            const int r = i / (cols / 8), c = (i % (cols / 8)) * 8;
-            const bool ok = ch * C + r < s.n && c < valid;
-            cp_async16(smem_addr(sm + off + r * l + c), ok ? x + size_t(s.row0 + ch * C + r) * ld + col0 + c : x, ok);
-        }
-    };
-    auto fetch1 = [&](int ch) {   // read by the first products
-        if (ch < chunks) {
-            const ChunkPtr p = chunk_ptr(sc.chunk, s.chunk0 + ch, d.heads, h, DK);
-            if constexpr (MODE == HEAD_DELTA) { copy_x((ch & 1) * L::KT, LDK, ch, 1); copy_x(L::oq, LDK, ch, 0); }
-            else {
-                if constexpr (MODE == CHANNEL_DELTA) for (int i = 0; i < 2; ++i) copy_rows(i * L::KT, LDK, p.dec + i * C * DK, DK);
-                for (int i = 0; i < 2; ++i) copy_rows(L::oq + i * L::KT, LDK, p.dec + (2 + i) * C * DK, DK);
+    const int h = blockIdx.y, c0 = blockIdx.x * NB, nb = gridDim.x, chunks = (s.n + C - 1) / C;
+    if (tid == 0) {
+        for (int i = 0; i < BUFS; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], 8); }
+        s_err = 0;
+        mbar_fence_init();
+    }
+    __syncthreads();
+    if (warp == 8) {
+        if (lane == 0) {
+            bool ok = true;
+            for (int ch = 0; ch < chunks && ok; ++ch) {
+                const R r(sc.chunk, s.chunk0 + ch, d.heads, h, nb);
+                auto load = [&](int buf, int dst, const bf16* src, int elems, const bf16* more = nullptr, int more_dst = 0, int more_elems = 0) {
+                    if (!ok) return;
+                    if (ch > 0 && !mbar_wait(&empty[buf], (ch - 1) & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; return; }
+                    mbar_expect_tx(&full[buf], uint32_t(elems + more_elems) * 2);
+                    bulk_load(sm + dst, src, uint32_t(elems) * 2, &full[buf]);
+                    if (more_elems) bulk_load(sm + more_dst, more, uint32_t(more_elems) * 2, &full[buf]);
+                };
+                if constexpr (MODE != TIME_MIX) load(BW, L::ow, r.h, 2 * KT);
+                load(BK, L::ok, r.h + R::ok, R::nx * KT, r.h + R::ov + size_t(blockIdx.x) * VT, L::ov, MODE == TIME_MIX ? VT : 0);
+                load(BQ, L::oq, r.h + R::oq, R::nx * KT);
+                load(BP, L::op, r.h + R::op, 2 * TT);
             }
-            if constexpr (MODE != TIME_MIX) {
-                copy_x(L::ov, LDN, ch, 2);
-                if (tid < C) cp_async16(smem_addr(s_scal + (ch & 1) * 4 * C + tid * 4), p.scal + tid * 4, true);
-            }
-            if (tid < DK / 4) cp_async16(smem_addr(s_end + (ch & 1) * DK + tid * 4), p.end + tid * 4, true);
         }
-        cp_commit();
-    };
-    auto fetch2 = [&](int ch) {
-        if (MODE != TIME_MIX && ch < chunks) {
-            const ChunkPtr p = chunk_ptr(sc.chunk, s.chunk0 + ch, d.heads, h, DK);
-            for (int i = 0; i < 2; ++i) copy_rows(L::ot + i * L::TT, LDT, p.T + i * C * C, C);
-        }
-        cp_commit();
-    };
-    auto fetch3 = [&](int ch) {   // read by the last products
-        if (ch < chunks) {
-            const ChunkPtr p = chunk_ptr(sc.chunk, s.chunk0 + ch, d.heads, h, DK);
-            for (int i = 0; i < 2; ++i) copy_rows(L::op + i * L::TT, LDT, p.P + i * C * C, C);
-            if constexpr (MODE != HEAD_DELTA) for (int i = 0; i < 2; ++i) copy_rows(L::oo + i * L::KT, LDK, p.dec + (4 + i) * C * DK, DK);
-            if constexpr (MODE == TIME_MIX) copy_x(L::ov, LDN, ch, 2);
-        }
-        cp_commit();
-    };
-
-    // the state: 16 rows and NI times 16 columns per warp
-    constexpr int MW = DK / 16 < 8 ? DK / 16 : 8, NI = NB / 16 / (8 / MW), MI = DK / 16 / MW;
-    static_assert(MI == 1 && NI >= 1, "one row tile per warp");
-    const int sm0 = (warp % MW) * 16, sn0 = (warp / MW) * NI * 16;
-    float st[NI][2][4];
-    float* S = a.state + (size_t(s.slot) * d.heads + h) * d.dim * d.vdim + c0;
-#pragma unroll
-    for (int i = 0; i < NI; ++i)
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int r = sm0 + lr + e * 8, c = sn0 + i * 16 + j * 8 + lc;
-                float2 v = make_float2(0.f, 0.f);
-                if (s.pos0 > 0 && r < d.dim && c0 + c < d.vdim) v = *reinterpret_cast<const float2*>(S + size_t(r) * d.vdim + c);
-                st[i][j][2 * e] = v.x; st[i][j][2 * e + 1] = v.y;
-            }
-    auto put_pair = [&](int off, int tile, int r, int c, float vx, float vy) {   // hi at off, lo `tile` elements behind
-        uint32_t hi, lo;
-        split_bf16x2(vx, vy, hi, lo);
-        *reinterpret_cast<uint32_t*>(sm + off + r * LDN + c) = hi;
-        *reinterpret_cast<uint32_t*>(sm + off + tile + r * LDN + c) = lo;
-    };
-    auto put_state = [&]() {
+    } else {
+        auto mat = [&](int off, int l) { return SmemMat{smem_addr(sm + off), l}; };
+        // every warp meets at the barriers below, so a wait that gave up must not leave the loop alone
+        auto take = [&](int buf, int ch) { if (!mbar_wait(&full[buf], ch & 1, &s_err)) atomicExch(&s_err, 1); };
+        auto give = [&](int buf) { __syncwarp(); if (lane == 0) mbar_arrive(&empty[buf]); };
+        // the state: 16 rows and NI times 16 columns per warp
+        constexpr int MW = DK / 16 < 8 ? DK / 16 : 8, NI = NB / 16 / (8 / MW);
+        static_assert(DK / 16 / MW == 1 && NI >= 1, "one row tile per warp");
+        const int sm0 = (warp % MW) * 16, sn0 = (warp / MW) * NI * 16;
+        float st[NI][2][4];
+        float* S = a.state + (size_t(s.slot) * d.heads + h) * d.dim * d.vdim + c0;
 #pragma unroll
         for (int i = 0; i < NI; ++i)
 #pragma unroll
             for (int j = 0; j < 2; ++j)
 #pragma unroll
-                for (int e = 0; e < 2; ++e) put_pair(L::os, DK * LDN, sm0 + lr + e * 8, sn0 + i * 16 + j * 8 + lc, st[i][j][2 * e], st[i][j][2 * e + 1]);
-    };
-    fetch1(0); fetch2(0); fetch3(0);
-    put_state();
-    cp_wait<2>();
-    __syncthreads();
-
-    const SmemMat sh = mat(L::os, LDN), slo = mat(L::os + DK * LDN, LDN), vt = mat(L::ov, LDN);
-    const SmemMat rh = mat(L::orr, LDN), rl = mat(L::orr + L::VT, LDN), uh = mat(L::ou, LDN), ul = mat(L::ou + L::VT, LDN), wh = mat(L::ow, LDN), wl = mat(L::ow + L::VT, LDN);
-    const SmemMat th = mat(L::ot, LDT), tl = mat(L::ot + L::TT, LDT), ph = mat(L::op, LDT), pl = mat(L::op + L::TT, LDT);
-    // tiles of the products with 64 rows: warps 0..3 k, 4..7 q, two 16-column blocks each; time mixing: a block per warp
-    constexpr int NQ = MODE == TIME_MIX ? 1 : 2;
-    const int mt = warp & 3, half = warp >> 2, qn0 = MODE == TIME_MIX ? half * 16 : 0;
-    const bool is_q = MODE == TIME_MIX || half == 1;
-    for (int ch = 0; ch < chunks; ++ch) {
-        const float* scal = s_scal + (ch & 1) * 4 * C;
-        const int rows = min(C, s.n - ch * C);
-        // decayed k and q against the state
-        float acc[NQ][2][4];
-#pragma unroll
-        for (int i = 0; i < NQ; ++i)
-#pragma unroll
-            for (int j = 0; j < 2; ++j)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
-        {
-            const SmemMat ah = is_q ? mat(L::oq, LDK) : mat(MODE == HEAD_DELTA ? (ch & 1) * L::KT : 0, LDK), al = is_q ? mat(L::oq + L::KT, LDK) : mat(L::KT, LDK);
-#pragma unroll
-            for (int kt = 0; kt < DK / 16; ++kt) {
-                uint32_t fh[4], fl[4];
-                ah.a(fh, mt * 16, kt * 16, lane);
-                if constexpr (MODE != HEAD_DELTA) al.a(fl, mt * 16, kt * 16, lane);
-#pragma unroll
-                for (int i = 0; i < NQ; ++i) {
-                    uint32_t gh[4], gl[4];
-                    sh.b_t(gh, kt * 16, qn0 + i * 16, lane);
-                    slo.b_t(gl, kt * 16, qn0 + i * 16, lane);
-#pragma unroll
-                    for (int j = 0; j < 2; ++j) {
-                        if constexpr (MODE != HEAD_DELTA) mma(acc[i][j], fl, gh[2 * j], gh[2 * j + 1]);
-                        mma(acc[i][j], fh, gl[2 * j], gl[2 * j + 1]);
-                        mma(acc[i][j], fh, gh[2 * j], gh[2 * j + 1]);
-                    }
-                }
-            }
-        }
-        if constexpr (MODE != TIME_MIX) {
-            if (!is_q) {   // R = beta (v - decayed k against the state)
-#pragma unroll
-                for (int i = 0; i < NQ; ++i)
-#pragma unroll
-                    for (int j = 0; j < 2; ++j)
-#pragma unroll
-                        for (int e = 0; e < 2; ++e) {
-                            const int t = mt * 16 + lr + e * 8, c = i * 16 + j * 8 + lc;
-                            const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sm + L::ov + t * LDN + c));
-                            const float k = MODE == HEAD_DELTA ? scal[kScalKin + t] : 1.f, b = scal[kScalBeta + t];
-                            put_pair(L::orr, L::VT, t, c, b * (v.x - k * acc[i][j][2 * e]), b * (v.y - k * acc[i][j][2 * e + 1]));
-                        }
-            }
-            cp_wait<1>();          // T
-            __syncthreads();
-            fetch1(ch + 1);
-            // U = T R, a 16 x 16 block per warp
-            float u[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-#pragma unroll
-            for (int kt = 0; kt < C / 16; ++kt)
-                if (kt <= mt) {
-                    uint32_t fh[4], fl[4], gh[4], gl[4];
-                    th.a(fh, mt * 16, kt * 16, lane); tl.a(fl, mt * 16, kt * 16, lane);
-                    rh.b_t(gh, kt * 16, half * 16, lane); rl.b_t(gl, kt * 16, half * 16, lane);
-#pragma unroll
-                    for (int j = 0; j < 2; ++j) {
-                        mma(u[j], fl, gh[2 * j], gh[2 * j + 1]);
-                        mma(u[j], fh, gl[2 * j], gl[2 * j + 1]);
-                        mma(u[j], fh, gh[2 * j], gh[2 * j + 1]);
-                    }
-                }
-#pragma unroll
-            for (int j = 0; j < 2; ++j)
-#pragma unroll
                 for (int e = 0; e < 2; ++e) {
-                    const int t = mt * 16 + lr + e * 8, c = half * 16 + j * 8 + lc;
-                    put_pair(L::ou, L::VT, t, c, u[j][2 * e], u[j][2 * e + 1]);
-                    if constexpr (MODE == HEAD_DELTA) { const float k = scal[kScalKout + t]; put_pair(L::ow, L::VT, t, c, k * u[j][2 * e], k * u[j][2 * e + 1]); }
+                    const int r = sm0 + lr + e * 8, c = sn0 + i * 16 + j * 8 + lc;
+                    float2 v = make_float2(0.f, 0.f);
+                    if (s.pos0 > 0 && r < d.dim && c0 + c < d.vdim) v = *reinterpret_cast<const float2*>(S + size_t(r) * d.vdim + c);
+                    st[i][j][2 * e] = v.x; st[i][j][2 * e + 1] = v.y;
                 }
-            cp_wait<1>();          // P and the update's k
-            __syncthreads();
-            fetch2(ch + 1);
-        } else {
-            cp_wait<0>();
-            __syncthreads();
-            fetch1(ch + 1);
-            fetch2(ch + 1);
-        }
-        // the state's update
-        {
-            const float* end = s_end + (ch & 1) * DK;
-            const float e0 = end[sm0 + lr], e1 = end[sm0 + lr + 8];
+        auto put_pair = [&](int off, int half, int r, int c, float vx, float vy) {   // hi at off, lo `half` elements behind
+            uint32_t hi, lo;
+            split_bf16x2(vx, vy, hi, lo);
+            *reinterpret_cast<uint32_t*>(sm + off + r * LDN + c) = hi;
+            *reinterpret_cast<uint32_t*>(sm + off + half + r * LDN + c) = lo;
+        };
+        auto put_state = [&](int buf) {
 #pragma unroll
             for (int i = 0; i < NI; ++i)
 #pragma unroll
-                for (int j = 0; j < 2; ++j) { st[i][j][0] *= e0; st[i][j][1] *= e0; st[i][j][2] *= e1; st[i][j][3] *= e1; }
-            const SmemMat kh = MODE == HEAD_DELTA ? mat((ch & 1) * L::KT, LDK) : mat(L::oo, LDK), kl = mat(L::oo + L::KT, LDK);
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) put_pair(L::os + buf * 2 * L::SS, L::SS, sm0 + lr + e * 8, sn0 + i * 16 + j * 8 + lc, st[i][j][2 * e], st[i][j][2 * e + 1]);
+        };
+        put_state(0);
+        walk_sync();
+        // products with 64 rows: 16 rows and 16 columns per warp
+        const int mt = warp & 3, n0 = (warp >> 2) * 16, t_lo = mt * 16 + lr;
+        const SmemMat uh = mat(MODE == TIME_MIX ? L::ov : L::ou, LDN), ul = mat(L::ou + VT, LDN), xh = mat(L::ox, LDN), xl = mat(L::ox + VT, LDN);
+        const SmemMat wh = mat(L::ow, LDK), wl = mat(L::ow + KT, LDK), qh = mat(L::oq, LDK), ql = mat(L::oq + KT, LDK), kh = mat(L::ok, LDK), kl = mat(L::ok + KT, LDK);
+        const SmemMat ph = mat(L::op, LDT), pl = mat(L::op + TT, LDT);
+        // what a thread reads of a chunk by itself, one chunk ahead
+        struct Own { float2 u0[2][2]; float end[2], qd[2], ko[2]; };
+        auto own = [&](int ch) {
+            Own o;
+            const R r(sc.chunk, s.chunk0 + min(ch, chunks - 1), d.heads, h, nb);
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                o.end[e] = r.end[sm0 + lr + 8 * e];
+                if constexpr (MODE == HEAD_DELTA) { o.qd[e] = r.scal[t_lo + 8 * e]; o.ko[e] = r.scal[C + t_lo + 8 * e]; }
+                if constexpr (MODE != TIME_MIX)
+#pragma unroll
+                    for (int j = 0; j < 2; ++j) o.u0[j][e] = *reinterpret_cast<const float2*>(r.f + size_t(blockIdx.x) * C * NB + (t_lo + 8 * e) * NB + n0 + j * 8 + lc);
+            }
+            return o;
+        };
+        Own now = own(0);
+        for (int ch = 0; ch < chunks; ++ch) {
+            const Own next = own(ch + 1);
+            const SmemMat sh = mat(L::os + (ch & 1) * 2 * L::SS, LDN), slo = mat(L::os + (ch & 1) * 2 * L::SS + L::SS, LDN);
+            if constexpr (MODE != TIME_MIX) {   // U = U0 - W S
+                take(BW, ch);
+                float acc[3][2][4];
+#pragma unroll
+                for (int i = 0; i < 24; ++i) acc[i / 8][(i >> 2) & 1][i & 3] = 0.f;
+#pragma unroll
+                for (int kt = 0; kt < DK / 16; ++kt) {
+                    uint32_t fh[4], fl[4], gh[4], gl[4];
+                    wh.a(fh, mt * 16, kt * 16, lane); wl.a(fl, mt * 16, kt * 16, lane);
+                    sh.b_t(gh, kt * 16, n0, lane); slo.b_t(gl, kt * 16, n0, lane);
+#pragma unroll
+                    for (int j = 0; j < 2; ++j) {
+                        mma(acc[0][j], fl, gh[2 * j], gh[2 * j + 1]);
+                        mma(acc[1][j], fh, gl[2 * j], gl[2 * j + 1]);
+                        mma(acc[2][j], fh, gh[2 * j], gh[2 * j + 1]);
+                    }
+                }
+                give(BW);
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const float ux = now.u0[j][e].x - (acc[0][j][2 * e] + acc[1][j][2 * e] + acc[2][j][2 * e]);
+                        const float uy = now.u0[j][e].y - (acc[0][j][2 * e + 1] + acc[1][j][2 * e + 1] + acc[2][j][2 * e + 1]);
+                        put_pair(L::ou, VT, t_lo + 8 * e, n0 + j * 8 + lc, ux, uy);
+                        if constexpr (MODE == HEAD_DELTA) put_pair(L::ox, VT, t_lo + 8 * e, n0 + j * 8 + lc, now.ko[e] * ux, now.ko[e] * uy);
+                    }
+                walk_sync();
+            }
+            take(BK, ch);
+            // the state's update
+#pragma unroll
+            for (int i = 0; i < NI; ++i)
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) st[i][j][e] *= now.end[e >> 1];
 #pragma unroll
             for (int kt = 0; kt < C / 16; ++kt) {
                 uint32_t fh[4], fl[4];
@@ -550,8 +585,8 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(const RecurDims d, cons
 #pragma unroll
                 for (int i = 0; i < NI; ++i) {
                     uint32_t gh[4], gl[4];
-                    (MODE == TIME_MIX ? vt : MODE == HEAD_DELTA ? wh : uh).b_t(gh, kt * 16, sn0 + i * 16, lane);
-                    if constexpr (MODE != TIME_MIX) (MODE == HEAD_DELTA ? wl : ul).b_t(gl, kt * 16, sn0 + i * 16, lane);
+                    (MODE == HEAD_DELTA ? xh : uh).b_t(gh, kt * 16, sn0 + i * 16, lane);
+                    if constexpr (MODE != TIME_MIX) (MODE == HEAD_DELTA ? xl : ul).b_t(gl, kt * 16, sn0 + i * 16, lane);
 #pragma unroll
                     for (int j = 0; j < 2; ++j) {
                         if constexpr (MODE != HEAD_DELTA) mma(st[i][j], fl, gh[2 * j], gh[2 * j + 1]);
@@ -560,58 +595,77 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(const RecurDims d, cons
                     }
                 }
             }
-            put_state();   // read again behind the next barrier only
-        }
-        if (is_q) {        // read-out
-            if constexpr (MODE == HEAD_DELTA) {
-                const float q0 = scal[kScalQin + mt * 16 + lr], q1 = scal[kScalQin + mt * 16 + lr + 8];
+            if constexpr (MODE != TIME_MIX) give(BK);
+            put_state((ch + 1) & 1);
+            // the read-out: q against the state in front of the chunk, then P U
+            take(BQ, ch);
+            float acc[3][2][4];
 #pragma unroll
-                for (int i = 0; i < NQ; ++i)
+            for (int i = 0; i < 24; ++i) acc[i / 8][(i >> 2) & 1][i & 3] = 0.f;
 #pragma unroll
-                    for (int j = 0; j < 2; ++j) { acc[i][j][0] *= q0; acc[i][j][1] *= q0; acc[i][j][2] *= q1; acc[i][j][3] *= q1; }
+            for (int kt = 0; kt < DK / 16; ++kt) {
+                uint32_t fh[4], fl[4], gh[4], gl[4];
+                qh.a(fh, mt * 16, kt * 16, lane);
+                if constexpr (MODE != HEAD_DELTA) ql.a(fl, mt * 16, kt * 16, lane);
+                sh.b_t(gh, kt * 16, n0, lane); slo.b_t(gl, kt * 16, n0, lane);
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+                    if constexpr (MODE != HEAD_DELTA) mma(acc[0][j], fl, gh[2 * j], gh[2 * j + 1]);
+                    mma(acc[1][j], fh, gl[2 * j], gl[2 * j + 1]);
+                    mma(acc[2][j], fh, gh[2 * j], gh[2 * j + 1]);
+                }
             }
+            give(BQ);
+            if constexpr (MODE == HEAD_DELTA) {
+#pragma unroll
+                for (int i = 1; i < 3; ++i)
+#pragma unroll
+                    for (int j = 0; j < 2; ++j)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) acc[i][j][e] *= now.qd[e >> 1];
+            }
+            take(BP, ch);
 #pragma unroll
             for (int kt = 0; kt < C / 16; ++kt)
                 if (kt <= mt) {
-                    uint32_t fh[4], fl[4];
+                    uint32_t fh[4], fl[4], gh[4], gl[4];
                     ph.a(fh, mt * 16, kt * 16, lane); pl.a(fl, mt * 16, kt * 16, lane);
+                    uh.b_t(gh, kt * 16, n0, lane);
+                    if constexpr (MODE != TIME_MIX) ul.b_t(gl, kt * 16, n0, lane);
 #pragma unroll
-                    for (int i = 0; i < NQ; ++i) {
-                        uint32_t gh[4], gl[4];
-                        (MODE == TIME_MIX ? vt : uh).b_t(gh, kt * 16, qn0 + i * 16, lane);
-                        if constexpr (MODE != TIME_MIX) ul.b_t(gl, kt * 16, qn0 + i * 16, lane);
-#pragma unroll
-                        for (int j = 0; j < 2; ++j) {
-                            mma(acc[i][j], fl, gh[2 * j], gh[2 * j + 1]);
-                            if constexpr (MODE != TIME_MIX) mma(acc[i][j], fh, gl[2 * j], gl[2 * j + 1]);
-                            mma(acc[i][j], fh, gh[2 * j], gh[2 * j + 1]);
-                        }
+                    for (int j = 0; j < 2; ++j) {
+                        mma(acc[0][j], fl, gh[2 * j], gh[2 * j + 1]);
+                        if constexpr (MODE != TIME_MIX) mma(acc[1][j], fh, gl[2 * j], gl[2 * j + 1]);
+                        mma(acc[2][j], fh, gh[2 * j], gh[2 * j + 1]);
                     }
                 }
+            give(BP);
+            if constexpr (MODE == TIME_MIX) give(BK);   // v lies with k
+            const int rows = s.n - ch * C;
 #pragma unroll
-            for (int i = 0; i < NQ; ++i)
+            for (int j = 0; j < 2; ++j)
 #pragma unroll
-                for (int j = 0; j < 2; ++j)
-#pragma unroll
-                    for (int e = 0; e < 2; ++e) {
-                        const int t = mt * 16 + lr + e * 8, c = c0 + qn0 + i * 16 + j * 8 + lc;
-                        if (t < rows && c < d.vdim) *reinterpret_cast<float2*>(sc.o + (size_t(s.row0 + ch * C + t) * d.heads + h) * d.vdim + c) = make_float2(acc[i][j][2 * e], acc[i][j][2 * e + 1]);
-                    }
+                for (int e = 0; e < 2; ++e) {
+                    const int t = t_lo + 8 * e, c = c0 + n0 + j * 8 + lc;
+                    if (t < rows && c < d.vdim)
+                        *reinterpret_cast<float2*>(sc.o + (size_t(s.row0 + ch * C + t) * d.heads + h) * d.vdim + c) =
+                            make_float2(acc[0][j][2 * e] + acc[1][j][2 * e] + acc[2][j][2 * e], acc[0][j][2 * e + 1] + acc[1][j][2 * e + 1] + acc[2][j][2 * e + 1]);
+                }
+            now = next;
+            walk_sync();   // the new state is complete, U and the old state are read
         }
-        cp_wait<1>();              // the next chunk's first operands
-        __syncthreads();
-        fetch3(ch + 1);
+#pragma unroll
+        for (int i = 0; i < NI; ++i)
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int r = sm0 + lr + e * 8, c = sn0 + i * 16 + j * 8 + lc;
+                    if (r < d.dim && c0 + c < d.vdim) *reinterpret_cast<float2*>(S + size_t(r) * d.vdim + c) = make_float2(st[i][j][2 * e], st[i][j][2 * e + 1]);
+                }
     }
-    cp_wait<0>();
-#pragma unroll
-    for (int i = 0; i < NI; ++i)
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int r = sm0 + lr + e * 8, c = sn0 + i * 16 + j * 8 + lc;
-                if (r < d.dim && c0 + c < d.vdim) *reinterpret_cast<float2*>(S + size_t(r) * d.vdim + c) = make_float2(st[i][j][2 * e], st[i][j][2 * e + 1]);
-            }
+    __syncthreads();
+    if (tid == 0 && s_err && err) atomicExch(err, 1);
 }
 
 template <int DK, int MODE>
@@ -622,30 +676,35 @@ int32_t launch(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, c
     FORGE_LAUNCH_CHECK();
     auto scan = chunk_scan_kernel<DK, MODE>;
     FORGE_CUDA(cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, int(Scan<DK, MODE>::smem)));
-    scan<<<dim3((d.vdim + NB - 1) / NB, d.heads, n_segs), 256, Scan<DK, MODE>::smem, st>>>(d, a, sc, segs);
+    scan<<<dim3((d.vdim + NB - 1) / NB, d.heads, n_segs), kScanThreads, Scan<DK, MODE>::smem, st>>>(d, a, sc, segs, sc.err);
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
 
-int padded_dim(const RecurDims& d) { return d.dim <= 64 ? 64 : 128; }
+template <typename F> auto dispatch(const RecurDims& d, F f) {
+    auto mode = [&](auto dk) {
+        if (!d.delta) return f(dk, std::integral_constant<int, TIME_MIX>{});
+        return d.channel ? f(dk, std::integral_constant<int, CHANNEL_DELTA>{}) : f(dk, std::integral_constant<int, HEAD_DELTA>{});
+    };
+    return d.dim <= 64 ? mode(std::integral_constant<int, 64>{}) : mode(std::integral_constant<int, 128>{});
+}
 
 }  // namespace
 
 bool recur_chunked_supported(const RecurDims& d) { return d.dim <= 128 && d.dim % 8 == 0 && d.vdim % 8 == 0; }
 
 ChunkBytes recur_chunk_bytes(const RecurDims& d) {
-    const size_t h = size_t(d.heads), dk = size_t(padded_dim(d));
-    return {h * 4 * C * C * 2, h * 4 * C * 4, h * dk * 4, d.channel ? h * 6 * C * dk * 2 : 0};
+    const size_t h = size_t(d.heads);
+    const int nb = (d.vdim + NB - 1) / NB;
+    return dispatch(d, [&](auto dk, auto mode) {
+        using R = Rec<decltype(dk)::value, decltype(mode)::value>;
+        return ChunkBytes{h * R::halves(nb) * 2, h * R::floats(nb) * 4};
+    });
 }
 
 int32_t recur_chunked(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, const ScanSeg* segs, int n_segs, int n_chunks, cudaStream_t st) {
     if (n_segs <= 0) return FORGE_OK;
-    auto go = [&](auto dk) -> int32_t {
-        constexpr int DK = decltype(dk)::value;
-        if (!d.delta) return launch<DK, TIME_MIX>(d, a, sc, segs, n_segs, n_chunks, st);
-        return d.channel ? launch<DK, CHANNEL_DELTA>(d, a, sc, segs, n_segs, n_chunks, st) : launch<DK, HEAD_DELTA>(d, a, sc, segs, n_segs, n_chunks, st);
-    };
-    return padded_dim(d) == 64 ? go(std::integral_constant<int, 64>{}) : go(std::integral_constant<int, 128>{});
+    return dispatch(d, [&](auto dk, auto mode) { return launch<decltype(dk)::value, decltype(mode)::value>(d, a, sc, segs, n_segs, n_chunks, st); });
 }
 
 }  // namespace forge

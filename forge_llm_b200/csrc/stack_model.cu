@@ -58,9 +58,9 @@ struct StackModel {
     DenseScratch scratch;
     // step buffers, grown on demand (scratch_gen of the model counts the moves)
     struct Buf { void* p = nullptr; size_t cap = 0; };
-    Buf x, h, cat, proj, gate, mid, mid_r, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, hgate, decay, beta, low, conv, unit, o, pair, place, c_tp, c_scal, c_end, c_dec, sel, logits, meta;
+    Buf x, h, cat, proj, gate, mid, mid_r, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, hgate, decay, beta, low, conv, unit, o, pair, place, c_half, c_f32, sel, logits, meta;
     std::vector<Buf*> all() {
-        return {&x, &h, &cat, &proj, &gate, &mid, &mid_r, &q, &part, &ml, &ctx_c, &ctx_r, &ctx_k, &ctx_v, &hgate, &decay, &beta, &low, &conv, &unit, &o, &pair, &place, &c_tp, &c_scal, &c_end, &c_dec, &sel, &logits, &meta};
+        return {&x, &h, &cat, &proj, &gate, &mid, &mid_r, &q, &part, &ml, &ctx_c, &ctx_r, &ctx_k, &ctx_v, &hgate, &decay, &beta, &low, &conv, &unit, &o, &pair, &place, &c_half, &c_f32, &sel, &logits, &meta};
     }
     const LayerWeights& weights(int layer) const { return w[spec.layers[layer].weights_of >= 0 ? spec.layers[layer].weights_of : layer]; }
 };
@@ -320,7 +320,7 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
     const size_t es = dense_size(S.dtype), r = size_t(rows), W = size_t(S.spec.width), WP = size_t(S.width_p);
     // bytes, rows times the widest layer
     size_t h = WP * es, proj = 0, gate = 0, mid = 0, mid_r = 0, q = 0, part = 0, heads = 0, cc = 0, cr = 0, ck = 0, cv = 0, hgate = 0, decay = 0, beta = 0, low = 0, conv = 0, unit = 0, o = 0, pair = 0;
-    ChunkBytes cb{0, 0, 0, 0};
+    ChunkBytes cb{0, 0};
     auto most = [](size_t& a, size_t b) { a = std::max(a, b); };
     size_t n_max = size_t(S.head.N);
     for (size_t i = 0; i < S.spec.layers.size(); ++i) {
@@ -349,7 +349,7 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
         most(o, r * HV * 4);
         if (chunks && recur_chunked_supported(d)) {
             const ChunkBytes b = recur_chunk_bytes(d);
-            most(cb.tp, chunks * b.tp); most(cb.scal, chunks * b.scal); most(cb.end, chunks * b.end); most(cb.dec, chunks * b.dec);
+            most(cb.half, chunks * b.half); most(cb.f32, chunks * b.f32);
         }
         if (d.delta && seg_rows) { most(conv, r * d.channels() * es); most(unit, r * 2 * d.groups * 4); }
         if (L.has_attn()) {
@@ -365,7 +365,7 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
     if (S.spec.loop_times) FORGE_TRY(grow(m, S.cat, r * 2 * WP * es));
     FORGE_TRY(grow(m, S.place, r * sizeof(int32_t)));
     const std::pair<StackModel::Buf*, size_t> sizes[] = {{&S.proj, proj}, {&S.gate, gate}, {&S.mid, mid}, {&S.mid_r, mid_r}, {&S.q, q}, {&S.part, part}, {&S.ml, heads}, {&S.hgate, hgate}, {&S.decay, decay},
-        {&S.beta, beta}, {&S.low, low}, {&S.conv, conv}, {&S.unit, unit}, {&S.o, o}, {&S.pair, pair}, {&S.c_tp, cb.tp}, {&S.c_scal, cb.scal}, {&S.c_end, cb.end}, {&S.c_dec, cb.dec}, {&S.ctx_c, cc}, {&S.ctx_r, cr}, {&S.ctx_k, ck}, {&S.ctx_v, cv}};
+        {&S.beta, beta}, {&S.low, low}, {&S.conv, conv}, {&S.unit, unit}, {&S.o, o}, {&S.pair, pair}, {&S.c_half, cb.half}, {&S.c_f32, cb.f32}, {&S.ctx_c, cc}, {&S.ctx_r, cr}, {&S.ctx_k, ck}, {&S.ctx_v, cv}};
     for (const auto& e : sizes) FORGE_TRY(grow(m, *e.first, e.second));
     // one ticket per output tile of the largest product (128 rows x at least 16 tokens)
     const size_t tiles = ((n_max + 127) / 128) * std::max<size_t>(1, (size_t(std::max(rows, ctx_rows)) + 127) / 128);
@@ -513,8 +513,7 @@ struct Sequence {
         FORGE_TRY(recur_decode(d, dt, a, ones, st));
         RecurScratch sc;
         sc.conv = S.conv.p; sc.unit = static_cast<float*>(S.unit.p); sc.o = static_cast<float*>(S.o.p);
-        sc.chunk.tp = static_cast<__nv_bfloat16*>(S.c_tp.p); sc.chunk.scal = static_cast<float*>(S.c_scal.p); sc.chunk.end = static_cast<float*>(S.c_end.p);
-        sc.chunk.dec = static_cast<__nv_bfloat16*>(S.c_dec.p);
+        sc.chunk.half = static_cast<__nv_bfloat16*>(S.c_half.p); sc.chunk.f32 = static_cast<float*>(S.c_f32.p); sc.err = m->d_err;
         return recur_segments(d, dt, a, sc, s.segs, st);
     }
     RecurArgs recur_args(const RecurDims& d, const LayerWeights& w, StackCache::Run& run) {
