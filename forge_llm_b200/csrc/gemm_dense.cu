@@ -7,7 +7,8 @@
 // the remaining tiles are dealt evenly, CTA i of S taking the steps [i U / S, (i + 1) U / S) of their U, so every SM streams the
 // same amount whatever the number of tiles.  A tile that several CTAs share is finished by the last of them to arrive
 // (ticket): every share is left in scratch memory and added in K order, so the result does not depend on the order of
-// arrival.  Nobody waits for another CTA.
+// arrival.  Nobody waits for another CTA.  Up to 32 tokens with at most one tile per SM, the CTAs of a tile form a cluster instead: each takes
+// an equal part of its K steps, and the first adds the parts through distributed shared memory.
 // Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = epilogue (TMEM lane = weight row).
 // The weights lie in memory as the very images the ring holds (dense_tile_image), so a stage is one contiguous 16 KB bulk copy.
 // Accumulators are double buffered in tensor memory: the epilogue of one tile runs under the products of the next.
@@ -94,6 +95,7 @@ struct GemmParams {
     int waves;               // whole tiles per CTA
     uint32_t units;          // K steps of the tiles after them, dealt to the first `sharers` CTAs (at most one per step: no share is empty)
     int sharers;
+    int cluster;             // > 0: CTA i takes part i % cluster of the K steps of tile i / cluster, and nothing is dealt out
     float* part; int* tickets;
     int* err;
 };
@@ -139,7 +141,11 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     uint32_t u0 = 0, u1 = 0;   // this CTA's share of the dealt-out K steps
-    if (int(blockIdx.x) < p.sharers) { u0 = share_begin(p.units, blockIdx.x, p.sharers); u1 = share_begin(p.units, blockIdx.x + 1, p.sharers); }
+    const int rank = p.cluster > 1 ? int(blockIdx.x) % p.cluster : 0;
+    if (p.cluster > 0) {
+        const uint32_t t = blockIdx.x / uint32_t(p.cluster) * uint32_t(p.nk);
+        u0 = t + uint32_t(p.nk * rank / p.cluster); u1 = t + uint32_t(p.nk * (rank + 1) / p.cluster);
+    } else if (int(blockIdx.x) < p.sharers) { u0 = share_begin(p.units, blockIdx.x, p.sharers); u1 = share_begin(p.units, blockIdx.x + 1, p.sharers); }
     if (tid == 0) {
         for (int s = 0; s < STAGES; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
         for (int s = 0; s < 2; ++s) { mbar_init(&acc_full[s], 1); mbar_init(&acc_empty[s], 4); }
@@ -184,6 +190,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
                 }
             }
         }
+        if (p.cluster > 1) { __syncwarp(); cluster_sync(); cluster_sync(); }
     } else if (warp == 1) {
         if (lane == 0) {
             int s = 0;
@@ -209,6 +216,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
             }
             if (!ok) atomicExch(&s_err, 1);
         }
+        if (p.cluster > 1) { __syncwarp(); cluster_sync(); cluster_sync(); }
     } else {
         pdl_wait();
         const int quad = warp & 3;
@@ -223,6 +231,10 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
             const int cols = min(NT, p.m - tok0);
             // every warp's rows lie in one segment (segments start at multiples of 32 rows)
             const RowOut<__nv_bfloat16> g = row_out<__nv_bfloat16>(p.out, row, row0);
+            float x_old[CH];   // few tokens: the residual is on its way while the product is formed
+            if (NT <= 32 && g.kind == SEG_RESID && g.ok && !g.fresh && rank == 0)
+#pragma unroll
+                for (int c = 0; c < CH; ++c) x_old[c] = c < cols ? g.f32[size_t(tok0 + c) * g.ld] : 0.f;
             // the four warps meet at the barriers of a shared tile: one whose wait gave up must not leave the loop alone
             if (!mbar_wait(&acc_full[buf], (seg_i >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
             fence_after();
@@ -267,7 +279,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
                         float* dst = g.f32 + t0 * g.ld;
                         float x[CH];
 #pragma unroll
-                        for (int c = 0; c < CH; ++c) x[c] = c < n_c && !g.fresh ? dst[c * g.ld] : 0.f;   // all loads before the first store
+                        for (int c = 0; c < CH; ++c) x[c] = g.fresh ? 0.f : NT <= 32 ? x_old[c] : c < n_c ? dst[c * g.ld] : 0.f;   // all loads before the first store
 #pragma unroll
                         for (int c = 0; c < CH; ++c) { x[c] += v[c] + g.add; if (c < n_c) dst[c * g.ld] = x[c]; }
                         if (g.after) {
@@ -293,6 +305,36 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
                     load(c0, v);
                     finish(c0, v);
                 }
+            } else if (NT <= 32 && p.cluster > 1) {
+                // [token / 4][row][4] in the ring, which nothing uses any more
+                float* mine = reinterpret_cast<float*>(ring) + (quad * 32 + lane) * 4;
+                float v[CH];
+                load(0, v);
+                if (rank > 0)
+#pragma unroll
+                    for (int c = 0; c < CH; c += 4) *reinterpret_cast<float4*>(mine + c * 128) = make_float4(v[c], v[c + 1], v[c + 2], v[c + 3]);
+                __syncwarp();
+                cluster_sync();
+                if (rank == 0) {
+                    constexpr int QB = CH == 16 ? 4 : 2;   // loads of QB parts in flight together; added in their order
+                    for (int q0 = 1; q0 < p.cluster; q0 += QB) {
+                        float4 t[QB][CH / 4];
+#pragma unroll
+                        for (int q = 0; q < QB; ++q) {
+                            const uint32_t src = cluster_addr(mine, min(q0 + q, p.cluster - 1));
+#pragma unroll
+                            for (int c = 0; c < CH / 4; ++c) t[q][c] = cluster_load4(src + c * 512 * 4);
+                        }
+#pragma unroll
+                        for (int q = 0; q < QB; ++q)
+                            if (q0 + q < p.cluster)
+#pragma unroll
+                                for (int c = 0; c < CH / 4; ++c) { v[4 * c] += t[q][c].x; v[4 * c + 1] += t[q][c].y; v[4 * c + 2] += t[q][c].z; v[4 * c + 3] += t[q][c].w; }
+                    }
+                    finish(0, v);
+                }
+                __syncwarp();
+                cluster_sync();   // nobody leaves while its part is read
             } else {
                 // a shared tile: this CTA's part goes to its slot (0: the part its share starts with, 1: the other one)
                 float* mine = p.part + (size_t(blockIdx.x) * 2 + (u0 >= t_begin ? 0 : 1)) * (NT * 128);
@@ -363,6 +405,31 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmPara
     FORGE_TRY(make_map_2d(&mx, act, uint64_t(last_col + w.K), uint64_t(p.m), uint64_t(act_ld) * 2, NT));
     p.tt_count = (p.m + NT - 1) / NT;
     const long long tiles = (long long)((w.N + 127) / 128) * p.tt_count;
+    auto kern = gemm_dense_kernel<NT>;
+    const size_t smem = size_t(Ring<NT>::STAGES) * Ring<NT>::STAGE + 1024;
+    FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+    if (NT <= 32 && tiles <= sms) {
+        // most parts per tile whose clusters all run at once (a cluster lies within one group of SMs, so large ones leave SMs idle)
+        static int fits[9] = {0};
+        if (!fits[1])
+            for (int c = 1; c <= 8; ++c) {
+                cudaLaunchConfig_t cfg{};
+                cudaLaunchAttribute at[1];
+                cfg.gridDim = dim3(unsigned(c * 148)); cfg.blockDim = dim3(kThreads); cfg.dynamicSmemBytes = smem;
+                at[0].id = cudaLaunchAttributeClusterDimension;
+                at[0].val.clusterDim.x = unsigned(c); at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
+                cfg.attrs = at; cfg.numAttrs = 1;
+                FORGE_CUDA(cudaOccupancyMaxActiveClusters(&fits[c], kern, &cfg));
+            }
+        int parts = 0;
+        for (int c = 1; c <= 8; ++c) if (tiles <= fits[c] && (c == 1 || p.nk >= 2 * c)) parts = c;
+        if (tiles * parts >= 90 || tiles <= fits[8]) {
+            p.cluster = parts;
+            FORGE_CUDA(launch_pdl_cluster(kern, dim3(unsigned(tiles * parts)), dim3(kThreads), parts, smem, st, mx, p));
+            FORGE_LAUNCH_CHECK();
+            return FORGE_OK;
+        }
+    }
     const int grid = int(std::max(1LL, std::min((long long)sms, std::max(NT >= 128 ? tiles : 1, tiles * p.nk / 4))));
     p.waves = NT >= 128 ? int(tiles / grid) : 0;   // a weight stream gains nothing from whole tiles in turn
     const long long units = (tiles - (long long)p.waves * grid) * p.nk;
@@ -372,9 +439,6 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmPara
     // leaving and adding shares costs about NT / 32 K steps: where whole tiles are no dearer, every CTA takes at most one
     const long long rest = tiles - (long long)p.waves * grid;
     if (rest > 0 && rest <= grid && p.nk <= units / grid + NT / 32) p.sharers = int(rest);
-    const size_t smem = size_t(Ring<NT>::STAGES) * Ring<NT>::STAGE + 1024;
-    auto kern = gemm_dense_kernel<NT>;
-    FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
     FORGE_CUDA(launch_pdl(kern, dim3(grid), dim3(kThreads), smem, st, mx, p));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;

@@ -16,6 +16,50 @@ namespace cg = cooperative_groups;
 constexpr int kConvTile = 32;     // tokens per warp; taps - 1 of them at most reach behind the segment
 
 // ------------------------------------------------------------------------------------------------ decode
+// Second step of a two-step projection inside a CTA of 256 threads: put(i, sum of w[i][k] in[k]) for i < n, k < K (a multiple of 64).  `held` keeps the
+// first 16-byte pieces of a bfloat16 matrix: they are fetched in front of the dependency wait.
+template <typename T, int H> struct LowRows {
+    uint4 held[H];
+    const T* w; int n, K, pieces, steps;   // pieces: of eight values per row
+    bool narrow;                           // the pieces of a row lie in one warp
+    __device__ __forceinline__ LowRows(const T* w_, int n_, int K_) : w(w_), n(n_), K(K_), pieces(K_ / 8), steps((n_ * (K_ / 8) + 255) / 256), narrow(K_ == 64 || K_ == 128 || K_ == 256) {
+        if constexpr (std::is_same<T, __nv_bfloat16>::value)
+            if (narrow)
+#pragma unroll
+                for (int j = 0; j < H; ++j) if (int(threadIdx.x) + 256 * j < n * pieces) held[j] = reinterpret_cast<const uint4*>(w)[threadIdx.x + 256 * j];
+    }
+    template <typename F> __device__ __forceinline__ void run(const float* in, F put) {
+        const int lane = threadIdx.x & 31;
+        if (narrow) {
+            auto step = [&](int j, const T* src) {
+                const int i = threadIdx.x + 256 * j, row = i / pieces, pc = i % pieces;
+                float s = 0.f;
+                if (row < n) {
+                    float v[8], x[8];
+                    load8(v, src);
+                    load8(x, in + pc * 8);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) s = fmaf(v[e], x[e], s);
+                }
+                for (int m = pieces >> 1; m > 0; m >>= 1) s += __shfl_xor_sync(0xffffffffu, s, m);
+                if (pc == 0 && row < n) put(row, s);
+            };
+            constexpr bool hold = std::is_same<T, __nv_bfloat16>::value;
+            if constexpr (hold)
+#pragma unroll
+                for (int j = 0; j < H; ++j) if (j < steps) step(j, reinterpret_cast<const T*>(&held[j]));
+            for (int j = hold ? H : 0; j < steps; ++j) step(j, w + (size_t(threadIdx.x) + 256 * j) * 8);
+        } else {
+            for (int row = threadIdx.x >> 5; row < n; row += 8) {
+                float s = 0.f;
+                for (int k = lane; k < K; k += 32) s = fmaf(to_f(w[size_t(row) * K + k]), in[k], s);
+                s = warp_sum(s);
+                if (lane == 0) put(row, s);
+            }
+        }
+    }
+};
+
 // One CTA = 32 value columns of one head of one row; the CTAs of a head form a cluster for the norm of its output.  A thread holds
 // the state of one column in the rows warp, warp + 8, ... of it; state, weights and what the convolution keeps are read before
 // the dependency wait.
@@ -26,6 +70,8 @@ __global__ void __launch_bounds__(256) recur_decode_kernel(const RecurDims d, co
     float* sk = sq + d.dim;
     float* sg = sk + d.dim;
     float* sv = sg + d.dim;         // [32]
+    float* sgate = sv + 32;         // [32]
+    float* slow = sm + ((3 * d.dim + 64 + 3) & ~3);   // [2][low_k] inner values of decay and gate
     __shared__ float red[8][33], redo[8][33], wsum[8][3], part;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int split = blockIdx.x, splits = gridDim.x, h = blockIdx.y, r = blockIdx.z;
@@ -55,9 +101,16 @@ __global__ void __launch_bounds__(256) recur_decode_kernel(const RecurDims d, co
             *place(i) = v;
         }
     }
+    const bool two_step = CHANNEL && a.decay_w, low_gate = two_step && a.gate_w;
+    LowRows<T, 4> low_d(static_cast<const T*>(a.decay_w) + size_t(h) * d.dim * a.low_k, two_step ? d.dim : 0, a.low_k);
+    LowRows<T, 1> low_g(static_cast<const T*>(a.gate_w) + size_t(h * d.vdim + c0) * a.low_k, low_gate ? nc : 0, a.low_k);
     pdl_wait();
+    if (two_step) {
+        const T* in = static_cast<const T*>(a.low) + size_t(r) * a.low_ld;
+        for (int i = tid; i < (low_gate ? 2 : 1) * a.low_k; i += 256) slow[i] = to_f(in[i < a.low_k ? i : a.gate_col + i - a.low_k]);
+    }
     const T* x = static_cast<const T*>(a.x) + size_t(r) * a.x_ld;
-    const float gate = lane < nc ? to_f(static_cast<const T*>(a.gate)[size_t(r) * a.gate_ld + h * d.vdim + c0 + lane]) : 0.f;
+    float gate = lane < nc && !low_gate ? to_f(static_cast<const T*>(a.gate)[size_t(r) * a.gate_ld + h * d.vdim + c0 + lane]) : 0.f;
     for (int i = tid; i < n_in; i += 256) {
         const int ch = channel(i);
         const T in = x[ch];
@@ -69,7 +122,7 @@ __global__ void __launch_bounds__(256) recur_decode_kernel(const RecurDims d, co
         } else *place(i) = to_f(in);
     }
     if constexpr (CHANNEL) {
-        for (int i = tid; i < d.dim; i += 256) sg[i] = expf(a.decay[size_t(r) * a.decay_ld + h * d.dim + i]);
+        if (!two_step) for (int i = tid; i < d.dim; i += 256) sg[i] = expf(a.decay[size_t(r) * a.decay_ld + h * d.dim + i]);
     }
     const float g1 = CHANNEL ? 0.f : expf(a.decay[size_t(r) * a.decay_ld + h]);
     const float beta = DELTA ? a.beta[size_t(r) * d.heads + h] : 0.f;
@@ -85,7 +138,15 @@ __global__ void __launch_bounds__(256) recur_decode_kernel(const RecurDims d, co
         if constexpr (DELTA) s1 = warp_sum(s1);
         if (lane == 0) { wsum[warp][0] = s0; wsum[warp][1] = s1; }
     }
+    if (two_step) {
+        low_d.run(slow, [&](int i, float z) {
+            z += a.decay_add[h * d.dim + i];
+            sg[i] = expf(DELTA ? -a.decay_mul[h * d.dim + i] * softplus(z) : -expf(z));
+        });
+        if (low_gate) low_g.run(slow + a.low_k, [&](int i, float z) { sgate[i] = sigmoid(z); });
+    }
     __syncthreads();
+    if (low_gate && lane < nc) gate = sgate[lane];
     float t0 = 0.f, t1 = 0.f;
 #pragma unroll
     for (int w = 0; w < 8; ++w) { t0 += wsum[w][0]; t1 += wsum[w][1]; }
@@ -416,35 +477,81 @@ __global__ void __launch_bounds__(256) token_shift_kernel(T* __restrict__ dst, i
 }
 
 // ------------------------------------------------------------------------------------------------ sum of two normed rows
-template <typename T>
+// NV: four-value pieces per thread of rows of up to 1024 NV values (a multiple of four); 0: any width
+template <typename T, int NV>
 __global__ void __launch_bounds__(256) add_normed_pair_kernel(float* __restrict__ x, const float* __restrict__ ab, int width, float eps, const float* __restrict__ wa, const float* __restrict__ wb, const After after) {
     __shared__ float red[8][2];
     const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    pdl_trigger();
-    pdl_wait();
     const float* a = ab + size_t(r) * 2 * width;
     const float* b = a + width;
     float sa = 0.f, sb = 0.f;
-    for (int i = threadIdx.x; i < width; i += 256) { sa = fmaf(a[i], a[i], sa); sb = fmaf(b[i], b[i], sb); }
-    sa = warp_sum(sa); sb = warp_sum(sb);
-    if (lane == 0) { red[warp][0] = sa; red[warp][1] = sb; }
-    __syncthreads();
-    sa = sb = 0.f;
+    auto factors = [&]() {
+        sa = warp_sum(sa); sb = warp_sum(sb);
+        if (lane == 0) { red[warp][0] = sa; red[warp][1] = sb; }
+        __syncthreads();
+        sa = sb = 0.f;
 #pragma unroll
-    for (int w = 0; w < 8; ++w) { sa += red[w][0]; sb += red[w][1]; }
-    const float ia = 0.5f / sqrtf(sa / float(width) + eps), ib = 0.5f / sqrtf(sb / float(width) + eps);
-    for (int i = threadIdx.x; i < width; i += 256) {
-        const float v = x[size_t(r) * width + i] + a[i] * ia * wa[i] + b[i] * ib * wb[i];
-        x[size_t(r) * width + i] = v;
-        if (after.kind != AFTER_NONE)
-            static_cast<T*>(after.dst)[size_t(r) * after.ld + i] = to_t<T>(after.kind == AFTER_DYT ? dynamic_tanh(v, after.alpha, after.w[i], after.b[i]) : v);
+        for (int w = 0; w < 8; ++w) { sa += red[w][0]; sb += red[w][1]; }
+        sa = 0.5f / sqrtf(sa / float(width) + eps); sb = 0.5f / sqrtf(sb / float(width) + eps);
+    };
+    auto next = [&](float v, float w, float bias) { return after.kind == AFTER_DYT ? dynamic_tanh(v, after.alpha, w, bias) : v; };
+    pdl_trigger();
+    if constexpr (NV > 0) {
+        float4 va[NV], vb[NV], vx[NV], ca[NV], cb[NV], cw[NV], cz[NV];
+        const int n4 = width / 4;
+        auto get = [&](const float* p, int i) { return reinterpret_cast<const float4*>(p)[i]; };
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            if (i >= n4) continue;
+            ca[j] = get(wa, i); cb[j] = get(wb, i);
+            if (after.kind == AFTER_DYT) { cw[j] = get(after.w, i); cz[j] = get(after.b, i); }
+        }
+        pdl_wait();
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            if (i >= n4) continue;
+            va[j] = get(a, i); vb[j] = get(b, i); vx[j] = get(x + size_t(r) * width, i);
+        }
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            if (int(threadIdx.x) + 256 * j >= n4) continue;
+            sa = fmaf(va[j].x, va[j].x, fmaf(va[j].y, va[j].y, fmaf(va[j].z, va[j].z, fmaf(va[j].w, va[j].w, sa))));
+            sb = fmaf(vb[j].x, vb[j].x, fmaf(vb[j].y, vb[j].y, fmaf(vb[j].z, vb[j].z, fmaf(vb[j].w, vb[j].w, sb))));
+        }
+        factors();
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            if (i >= n4) continue;
+            float4 v = vx[j];
+            v.x += va[j].x * sa * ca[j].x + vb[j].x * sb * cb[j].x; v.y += va[j].y * sa * ca[j].y + vb[j].y * sb * cb[j].y;
+            v.z += va[j].z * sa * ca[j].z + vb[j].z * sb * cb[j].z; v.w += va[j].w * sa * ca[j].w + vb[j].w * sb * cb[j].w;
+            reinterpret_cast<float4*>(x + size_t(r) * width)[i] = v;
+            if (after.kind != AFTER_NONE) {
+                T* dst = static_cast<T*>(after.dst) + size_t(r) * after.ld + 4 * i;
+                dst[0] = to_t<T>(next(v.x, cw[j].x, cz[j].x)); dst[1] = to_t<T>(next(v.y, cw[j].y, cz[j].y));
+                dst[2] = to_t<T>(next(v.z, cw[j].z, cz[j].z)); dst[3] = to_t<T>(next(v.w, cw[j].w, cz[j].w));
+            }
+        }
+    } else {
+        pdl_wait();
+        for (int i = threadIdx.x; i < width; i += 256) { sa = fmaf(a[i], a[i], sa); sb = fmaf(b[i], b[i], sb); }
+        factors();
+        for (int i = threadIdx.x; i < width; i += 256) {
+            const float v = x[size_t(r) * width + i] + a[i] * sa * wa[i] + b[i] * sb * wb[i];
+            x[size_t(r) * width + i] = v;
+            if (after.kind != AFTER_NONE)
+                static_cast<T*>(after.dst)[size_t(r) * after.ld + i] = to_t<T>(next(v, after.kind == AFTER_DYT ? after.w[i] : 0.f, after.kind == AFTER_DYT ? after.b[i] : 0.f));
+        }
     }
 }
 
 template <typename T, bool DELTA, bool CHANNEL, int RPT>
 int32_t launch_decode(const RecurDims& d, const RecurArgs& a, const StepRows& rows, cudaStream_t st) {
     const int splits = (d.vdim + 31) / 32;
-    FORGE_CUDA(launch_pdl_cluster(recur_decode_kernel<T, DELTA, CHANNEL, RPT>, dim3(splits, d.heads, rows.n), dim3(256), splits, sizeof(float) * (3 * size_t(d.dim) + 32), st, d, a, rows));
+    FORGE_CUDA(launch_pdl_cluster(recur_decode_kernel<T, DELTA, CHANNEL, RPT>, dim3(splits, d.heads, rows.n), dim3(256), splits, sizeof(float) * (3 * size_t(d.dim) + 68 + 2 * size_t(a.low_k)), st, d, a, rows));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
@@ -526,10 +633,14 @@ int32_t token_shift(void* dst, int ld, int width, int width_p, int n_mix, const 
 
 int32_t add_normed_pair(float* x, const float* ab, int rows, int width, float eps, const float* wa, const float* wb, const After& after, int dtype, cudaStream_t st) {
     if (rows <= 0) return FORGE_OK;
-    if (dtype == FORGE_F32) FORGE_CUDA(launch_pdl(add_normed_pair_kernel<float>, dim3(rows), dim3(256), 0, st, x, ab, width, eps, wa, wb, after));
-    else FORGE_CUDA(launch_pdl(add_normed_pair_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, st, x, ab, width, eps, wa, wb, after));
-    FORGE_LAUNCH_CHECK();
-    return FORGE_OK;
+    auto go = [&](auto type) -> int32_t {
+        using T = decltype(type);
+        auto kern = width % 4 || width > 4096 ? add_normed_pair_kernel<T, 0> : width <= 2048 ? add_normed_pair_kernel<T, 2> : add_normed_pair_kernel<T, 4>;
+        FORGE_CUDA(launch_pdl(kern, dim3(rows), dim3(256), 0, st, x, ab, width, eps, wa, wb, after));
+        FORGE_LAUNCH_CHECK();
+        return FORGE_OK;
+    };
+    return dtype == FORGE_F32 ? go(float{}) : go(__nv_bfloat16{});
 }
 
 }  // namespace forge

@@ -37,6 +37,12 @@ struct RecurArgs {
     const float* bonus = nullptr;                        // [heads][dim]
     const float* conv = nullptr; void* ring = nullptr;   // [channels][taps]; T [slot][taps][channels]
     float* state = nullptr;                              // [slot][heads][dim][vdim]
+    // second step of two-step decays and gates, for single tokens (then decay, and gate if gate_w is set, are not read): T rows of low_k values per
+    // key channel and per value over the inner values low[row], the gate's from column gate_col; a decay's logarithm is
+    // -mul softplus(z + add) for the delta rule, -exp(z + add) for time mixing
+    const void* decay_w = nullptr; const void* gate_w = nullptr; const void* low = nullptr;
+    int low_ld = 0, low_k = 0, gate_col = 0;
+    const float* decay_mul = nullptr; const float* decay_add = nullptr;
     const float* norm = nullptr; int norm_head = 0;      // weight of the output's norm, and its step per head
     const void* gate = nullptr; int gate_ld = 0;         // T rows [heads * vdim]
     void* out = nullptr; int out_ld = 0;                 // T rows [heads * vdim]: rms norm(o) * norm * gate

@@ -8,7 +8,7 @@
 //                          [o | down] of [gated heads | activation], so both sublayers are summed by the product itself;
 //   delta rules            in [q k v | gate | beta | decay] (a second product for two-step gates and decays), recurrence, out;
 //   attention | time mix   the input's columns are [h | five shifted mixes] and every row of `in` reads the block it belongs to; keys
-//                          and values go from the epilogue into the cache; two out products, then the sum of their norms.
+//                          and values go from the epilogue into the cache; one product with both outputs, then the sum of their norms.
 #include <algorithm>
 #include <cmath>
 #include <cstring>
@@ -40,7 +40,7 @@ struct LayerWeights {
     float *conv = nullptr, *decay_mul = nullptr, *decay_add = nullptr, *bonus = nullptr, *head_norm = nullptr;
     // attention beside time mixing
     int k_row = 0, v_row = 0, hg_row = 0, r_row = 0, rk_row = 0, rv_row = 0;
-    DenseWeight out_r;
+    int out_r_row = 0;            // first row of the second mixer in `out`; it reads the columns behind the first one's
     float *mu = nullptr, *norm_l = nullptr, *norm_r = nullptr;
 };
 
@@ -58,9 +58,9 @@ struct StackModel {
     DenseScratch scratch;
     // step buffers, grown on demand (scratch_gen of the model counts the moves)
     struct Buf { void* p = nullptr; size_t cap = 0; };
-    Buf x, h, cat, proj, gate, mid, mid_r, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, hgate, decay, beta, low, conv, unit, o, pair, place, c_half, c_f32, sel, logits, meta;
+    Buf x, h, cat, proj, gate, mid, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, hgate, decay, beta, low, conv, unit, o, pair, place, c_half, c_f32, sel, logits, meta;
     std::vector<Buf*> all() {
-        return {&x, &h, &cat, &proj, &gate, &mid, &mid_r, &q, &part, &ml, &ctx_c, &ctx_r, &ctx_k, &ctx_v, &hgate, &decay, &beta, &low, &conv, &unit, &o, &pair, &place, &c_half, &c_f32, &sel, &logits, &meta};
+        return {&x, &h, &cat, &proj, &gate, &mid, &q, &part, &ml, &ctx_c, &ctx_r, &ctx_k, &ctx_v, &hgate, &decay, &beta, &low, &conv, &unit, &o, &pair, &place, &c_half, &c_f32, &sel, &logits, &meta};
     }
     const LayerWeights& weights(int layer) const { return w[spec.layers[layer].weights_of >= 0 ? spec.layers[layer].weights_of : layer]; }
 };
@@ -202,7 +202,7 @@ int32_t load_delta(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerW
         Image low(w->low_row + HV, std::max(w->decay_k, pad_to(L.gate_rank, kDensePad)), S.dtype);
         low.put(t.at("mix.a2"), 0);
         low.put(t.at("mix.g2"), w->low_row);
-        FORGE_TRY(low.load(m, &w->low));
+        FORGE_TRY(low.load(m, &w->low, true));
     } else {
         in.put(t.at("mix.g"), w->gate_row); in.put(t.at("mix.a"), w->decay_row);
     }
@@ -232,13 +232,12 @@ int32_t load_pair(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWe
     FORGE_TRY(in.load(m, &w->in));
     Image low(D, pad_to(L.decay_rank, kDensePad), S.dtype);
     low.put(t.at("mix.right.w2"), 0);
-    FORGE_TRY(low.load(m, &w->low));
-    Image out(S.spec.width, pad_to(a.heads * a.vdim, kDensePad), S.dtype);
+    FORGE_TRY(low.load(m, &w->low, true));
+    w->out_r_row = pad_to(S.spec.width, 128);
+    Image out(w->out_r_row + S.spec.width, pad_to(std::max(a.heads * a.vdim, D), kDensePad), S.dtype);
     out.put(t.at("mix.left.o"), 0);
+    out.put(t.at("mix.right.o"), w->out_r_row);
     FORGE_TRY(out.load(m, &w->out));
-    Image out_r(S.spec.width, pad_to(D, kDensePad), S.dtype);
-    out_r.put(t.at("mix.right.o"), 0);
-    FORGE_TRY(out_r.load(m, &w->out_r));
     std::vector<float> mu;
     for (const char* n : {"r", "k", "v", "g", "w"}) { const TensorView* v = t.at(std::string("mix.right.mu.") + n); for (int i = 0; i < S.spec.width; ++i) mu.push_back(v->at(size_t(i))); }
     FORGE_TRY(upload_values(m, &w->mu, mu));
@@ -319,14 +318,14 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
     StackModel& S = *m->stack;
     const size_t es = dense_size(S.dtype), r = size_t(rows), W = size_t(S.spec.width), WP = size_t(S.width_p);
     // bytes, rows times the widest layer
-    size_t h = WP * es, proj = 0, gate = 0, mid = 0, mid_r = 0, q = 0, part = 0, heads = 0, cc = 0, cr = 0, ck = 0, cv = 0, hgate = 0, decay = 0, beta = 0, low = 0, conv = 0, unit = 0, o = 0, pair = 0;
+    size_t h = WP * es, proj = 0, gate = 0, mid = 0, q = 0, part = 0, heads = 0, cc = 0, cr = 0, ck = 0, cv = 0, hgate = 0, decay = 0, beta = 0, low = 0, conv = 0, unit = 0, o = 0, pair = 0;
     ChunkBytes cb{0, 0};
     auto most = [](size_t& a, size_t b) { a = std::max(a, b); };
     size_t n_max = size_t(S.head.N);
     for (size_t i = 0; i < S.spec.layers.size(); ++i) {
         const LayerSpec& L = S.spec.layers[i];
         const LayerWeights& w = S.weights(int(i));
-        for (const DenseWeight* d : {&w.in, &w.out, &w.kv, &w.low, &w.out_r, &w.ff_in, &w.ff_out}) most(n_max, size_t(d->N));
+        for (const DenseWeight* d : {&w.in, &w.out, &w.kv, &w.low, &w.ff_in, &w.ff_out}) most(n_max, size_t(d->N));
         most(mid, r * std::max(w.out.K, w.ff_out.K) * es);
         if (L.has_latent()) {
             const LatentDims& d = L.mix;
@@ -356,7 +355,7 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
             most(h, (1 + kMixes) * WP * es);
             most(q, r * L.attn.heads * L.attn.dim_p * es);
             most(hgate, r * L.attn.heads * 4);
-            most(mid_r, r * w.out_r.K * es);
+            most(mid, r * 2 * w.out.K * es);
             most(pair, r * 2 * W * 4);
         }
     }
@@ -364,7 +363,7 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
     FORGE_TRY(grow(m, S.h, r * h));
     if (S.spec.loop_times) FORGE_TRY(grow(m, S.cat, r * 2 * WP * es));
     FORGE_TRY(grow(m, S.place, r * sizeof(int32_t)));
-    const std::pair<StackModel::Buf*, size_t> sizes[] = {{&S.proj, proj}, {&S.gate, gate}, {&S.mid, mid}, {&S.mid_r, mid_r}, {&S.q, q}, {&S.part, part}, {&S.ml, heads}, {&S.hgate, hgate}, {&S.decay, decay},
+    const std::pair<StackModel::Buf*, size_t> sizes[] = {{&S.proj, proj}, {&S.gate, gate}, {&S.mid, mid}, {&S.q, q}, {&S.part, part}, {&S.ml, heads}, {&S.hgate, hgate}, {&S.decay, decay},
         {&S.beta, beta}, {&S.low, low}, {&S.conv, conv}, {&S.unit, unit}, {&S.o, o}, {&S.pair, pair}, {&S.c_half, cb.half}, {&S.c_f32, cb.f32}, {&S.ctx_c, cc}, {&S.ctx_r, cr}, {&S.ctx_k, ck}, {&S.ctx_v, cv}};
     for (const auto& e : sizes) FORGE_TRY(grow(m, *e.first, e.second));
     // one ticket per output tile of the largest product (128 rows x at least 16 tokens)
@@ -526,9 +525,17 @@ struct Sequence {
         return a;
     }
 
+    // a step of single tokens forms two-step decays and gates inside the recurrence
+    bool all_ones() const { return s.ones == n; }
+    void two_step(RecurArgs* a, const LayerWeights& w, int low_ld) {
+        a->decay_w = w.low.w; a->low = S.low.p; a->low_ld = low_ld; a->low_k = w.low.K;
+        a->decay_mul = w.decay_mul; a->decay_add = w.decay_add;
+    }
+
     int32_t delta(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
         const RecurDims& d = L.rec;
         const int H = d.heads, HV = H * d.vdim, low_ld = w.decay_k + w.low.K;
+        RecurArgs a = recur_args(d, w, run);
         DenseOut o;
         o.add(SEG_CAST, 0, d.channels(), S.proj.p, d.channels());
         if (!d.channel) {
@@ -542,13 +549,17 @@ struct Sequence {
             o.add(SEG_CAST, w.decay_row, L.decay_rank, S.low.p, low_ld);
             o.add(SEG_CAST, w.low_gate_row, L.gate_rank, at(S.low.p, w.decay_k, dt), low_ld);
             FORGE_TRY(gemm(w.in, S.h.p, WP, o));
-            DenseOut lo;
-            OutSeg& g = lo.add(SEG_DECAY, 0, H * d.dim, S.decay.p, H * d.dim);
-            g.mul = w.decay_mul; g.add = w.decay_add;
-            lo.add(SEG_SIGMOID, w.low_row, HV, S.gate.p, HV).act_col = w.decay_k;
-            FORGE_TRY(gemm(w.low, S.low.p, low_ld, lo));
+            if (all_ones()) {
+                two_step(&a, w, low_ld);
+                a.gate_w = at(w.low.w, size_t(w.low_row) * w.low.K, dt); a.gate_col = w.decay_k;
+            } else {
+                DenseOut lo;
+                OutSeg& g = lo.add(SEG_DECAY, 0, H * d.dim, S.decay.p, H * d.dim);
+                g.mul = w.decay_mul; g.add = w.decay_add;
+                lo.add(SEG_SIGMOID, w.low_row, HV, S.gate.p, HV).act_col = w.decay_k;
+                FORGE_TRY(gemm(w.low, S.low.p, low_ld, lo));
+            }
         }
-        RecurArgs a = recur_args(d, w, run);
         a.out = S.mid.p; a.out_ld = w.out.K;
         FORGE_TRY(recur(d, a));
         DenseOut out;
@@ -579,34 +590,35 @@ struct Sequence {
             o.add(SEG_TANH, w.decay_row, L.decay_rank, S.low.p, w.low.K).act_col = 5 * WP;
             FORGE_TRY(gemm(w.in, S.h.p, ld, o));
         }
-        {
+        RecurArgs a = recur_args(d, w, run);
+        const int mid_ld = 2 * w.out.K;
+        if (all_ones()) two_step(&a, w, w.low.K);
+        else {
             DenseOut lo;
             lo.add(SEG_EXP_DECAY, 0, D, S.decay.p, D).add = w.decay_add;
             FORGE_TRY(gemm(w.low, S.low.p, w.low.K, lo));
         }
         StepRows single = s.rows;
         single.n = s.single;
-        FORGE_TRY(attn_rows(t, dt, S.q.p, run.pool, hgate, S.mid.p, w.out.K, single, t.chunk ? std::min(t.chunk, s.max_keys) : s.max_keys, st));
+        FORGE_TRY(attn_rows(t, dt, S.q.p, run.pool, hgate, S.mid.p, mid_ld, single, t.chunk ? std::min(t.chunk, s.max_keys) : s.max_keys, st));
         const int np = n - s.single;
         if (np > 0) {
-            PromptAttnArgs a;
-            a.q = at(S.q.p, size_t(s.single) * t.heads * t.dim_p, dt); a.k = run.pool; a.v = at(run.pool, size_t(t.groups) * t.dim_p, dt);
-            a.head_gate = hgate + size_t(s.single) * t.heads;
-            a.out = at(S.mid.p, size_t(s.single) * w.out.K, dt); a.out_ld = w.out.K;
-            a.q_rows = np; a.ctx_rows = kv->num_pages * FORGE_KV_PAGE; a.tiles = s.tiles; a.n_tiles = s.n_tiles;
-            a.pages = s.ctx_pages; a.page_row = t.row(); a.err = m->d_err;
-            FORGE_TRY(attn_prefill_kv(PromptDims(t), a, st));
+            PromptAttnArgs p;
+            p.q = at(S.q.p, size_t(s.single) * t.heads * t.dim_p, dt); p.k = run.pool; p.v = at(run.pool, size_t(t.groups) * t.dim_p, dt);
+            p.head_gate = hgate + size_t(s.single) * t.heads;
+            p.out = at(S.mid.p, size_t(s.single) * mid_ld, dt); p.out_ld = mid_ld;
+            p.q_rows = np; p.ctx_rows = kv->num_pages * FORGE_KV_PAGE; p.tiles = s.tiles; p.n_tiles = s.n_tiles;
+            p.pages = s.ctx_pages; p.page_row = t.row(); p.err = m->d_err;
+            FORGE_TRY(attn_prefill_kv(PromptDims(t), p, st));
         }
-        RecurArgs a = recur_args(d, w, run);
         a.norm_head = d.dim;
-        a.out = S.mid_r.p; a.out_ld = w.out_r.K;
+        a.out = at(S.mid.p, w.out.K, dt); a.out_ld = mid_ld;
         FORGE_TRY(recur(d, a));
         float* both = static_cast<float*>(S.pair.p);
-        DenseOut left, right;
-        left.add(SEG_F32, 0, W, both, 2 * W);
-        right.add(SEG_F32, 0, W, both + W, 2 * W);
-        FORGE_TRY(gemm(w.out, S.mid.p, w.out.K, left));
-        FORGE_TRY(gemm(w.out_r, S.mid_r.p, w.out_r.K, right));
+        DenseOut out;
+        out.add(SEG_F32, 0, W, both, 2 * W);
+        out.add(SEG_F32, w.out_r_row, W, both + W, 2 * W).act_col = w.out.K;
+        FORGE_TRY(gemm(w.out, S.mid.p, mid_ld, out));
         return add_normed_pair(x(), both, n, W, S.spec.eps, w.norm_l, w.norm_r, after, dt, st);
     }
 };
