@@ -2,13 +2,15 @@
 //
 // bfloat16 (gemm_dense_kernel): tcgen05 with both operands in shared memory.  A tile is 128 weight rows (MMA M) x NT
 // tokens (MMA N = 16 .. 256); one kernel serves a decode step (NT = 16: a weight stream, 16 KB of weights per K step and
-// SM in a ring of up to eleven stages) and a prompt (NT = 256).  Of T tiles over G CTAs the first G floor(T / G) are, for prompts,
+// SM in a ring of five stages) and a prompt (NT = 256).  Of T tiles over G CTAs the first G floor(T / G) are, for prompts,
 // whole tiles dealt in turn (neighbouring CTAs then work on the same weight rows, which come from L2 once); the K steps of 64 of
 // the remaining tiles are dealt evenly, CTA i of S taking the steps [i U / S, (i + 1) U / S) of their U, so every SM streams the
 // same amount whatever the number of tiles.  A tile that several CTAs share is finished by the last of them to arrive
 // (ticket): every share is left in scratch memory and added in K order, so the result does not depend on the order of
 // arrival.  Nobody waits for another CTA.  Up to 32 tokens with at most one tile per SM, the CTAs of a tile form a cluster instead: each takes
-// an equal part of its K steps, and the first adds the parts through distributed shared memory.
+// an equal part of its K steps, and the first adds the parts through distributed shared memory (few columns are stored there by the
+// others; many are fetched).  The ring of the sixteen-token form leaves room for a second CTA on the SM: the next product's weights are
+// requested while this one ends.
 // Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = epilogue (TMEM lane = weight row).
 // The weights lie in memory as the very images the ring holds (dense_tile_image), so a stage is one contiguous 16 KB bulk copy.
 // Accumulators are double buffered in tensor memory: the epilogue of one tile runs under the products of the next.
@@ -87,6 +89,31 @@ __device__ __forceinline__ int act_col(const DenseOut& o, int row) {
     return c;
 }
 
+// the epilogue of one value; `up`: the value of the next row, used by the even rows of gated pairs; `old`: what dst holds, if it is known
+template <typename T>
+__device__ __forceinline__ void put_one(const RowOut<T>& g, float v, float up, size_t t, float old, bool old_known, bool even_row) {
+    float* f = g.f32 + t * g.ld;
+    T* h = g.t + t * g.ld;
+    switch (g.kind) {
+        case SEG_CLAMPED_GLU: if (even_row) *h = to_t<T>(clamped_glu(v, up, g.limit)); break;
+        case SEG_SILU_GLU: if (even_row) *h = to_t<T>(silu(v) * up); break;
+        case SEG_CAST: g.t[(g.place ? size_t(g.place[t]) : t) * g.ld] = to_t<T>(v); break;
+        case SEG_SIGMOID: *h = to_t<T>(sigmoid(v)); break;
+        case SEG_SILU: *h = to_t<T>(silu(v)); break;
+        case SEG_TANH: *h = to_t<T>(tanhf(v)); break;
+        case SEG_SIGMOID_F32: *f = sigmoid(v); break;
+        case SEG_DECAY: *f = -g.mul * softplus(v + g.add); break;
+        case SEG_EXP_DECAY: *f = -expf(v + g.add); break;
+        case SEG_RESID: {
+            const float x = (g.fresh ? 0.f : old_known ? old : *f) + v + g.add;
+            *f = x;
+            if (g.after) g.next[t * g.next_ld] = to_t<T>(g.next_value(x));
+            break;
+        }
+        default: *f = v;
+    }
+}
+
 struct GemmParams {
     DenseOut out;
     const void* w;           // weight images
@@ -96,6 +123,7 @@ struct GemmParams {
     uint32_t units;          // K steps of the tiles after them, dealt to the first `sharers` CTAs (at most one per step: no share is empty)
     int sharers;
     int cluster;             // > 0: CTA i takes part i % cluster of the K steps of tile i / cluster, and nothing is dealt out
+    bool push;               // the parts fit EXCHANGE
     float* part; int* tickets;
     int* err;
 };
@@ -125,12 +153,13 @@ struct Work {
 
 template <int NT> struct Ring {
     static constexpr int X_BYTES = NT * 128, STAGE = 16384 + X_BYTES;
-    static constexpr int STAGES = (200 * 1024) / STAGE > 11 ? 11 : (200 * 1024) / STAGE;
+    static constexpr int STAGES = NT <= 16 ? 5 : (200 * 1024) / STAGE;
+    static constexpr int EXCHANGE = NT <= 16 ? 18432 : 0;   // parts that the other CTAs of a cluster store
     static constexpr uint32_t COLS = NT <= 16 ? 32 : 2 * NT;   // two accumulators
 };
 
 template <int NT>
-__global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ GemmParams p) {
+__global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ GemmParams p) {
     constexpr int STAGE = Ring<NT>::STAGE, STAGES = Ring<NT>::STAGES;
     constexpr uint32_t kCols = Ring<NT>::COLS;
     extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -158,6 +187,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
     fence_after();
     const uint32_t tmem = s_tmem;
     pdl_trigger();
+    if (p.cluster > 1 && p.push) cluster_arrive();   // nobody stores into a CTA that has not begun
 
     if (warp == 0) {
         if (lane == 0) {
@@ -190,7 +220,12 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
                 }
             }
         }
-        if (p.cluster > 1) { __syncwarp(); cluster_sync(); cluster_sync(); }
+        if (p.cluster > 1) {
+            __syncwarp();
+            if (p.push) cluster_wait();
+            else cluster_sync();
+            cluster_sync();
+        }
     } else if (warp == 1) {
         if (lane == 0) {
             int s = 0;
@@ -216,7 +251,12 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
             }
             if (!ok) atomicExch(&s_err, 1);
         }
-        if (p.cluster > 1) { __syncwarp(); cluster_sync(); cluster_sync(); }
+        if (p.cluster > 1) {
+            __syncwarp();
+            if (p.push) cluster_wait();
+            else cluster_sync();
+            cluster_sync();
+        }
     } else {
         pdl_wait();
         const int quad = warp & 3;
@@ -234,7 +274,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
             float x_old[CH];   // few tokens: the residual is on its way while the product is formed
             if (NT <= 32 && g.kind == SEG_RESID && g.ok && !g.fresh && rank == 0)
 #pragma unroll
-                for (int c = 0; c < CH; ++c) x_old[c] = c < cols ? g.f32[size_t(tok0 + c) * g.ld] : 0.f;
+                for (int c = 0; c < CH; ++c) if (c < cols) x_old[c] = g.f32[size_t(tok0 + c) * g.ld];
             // the four warps meet at the barriers of a shared tile: one whose wait gave up must not leave the loop alone
             if (!mbar_wait(&acc_full[buf], (seg_i >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
             fence_after();
@@ -251,7 +291,10 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
 #pragma unroll
                     for (int c = 0; c < CH; ++c) if (c < n_c) dst[c * g.ld] = f(v[c]);
                 };
-                if (g.kind == SEG_CLAMPED_GLU || g.kind == SEG_SILU_GLU) {
+                if (n_c == 1) {   // one token: little code
+                    const float got = __shfl_xor_sync(0xffffffffu, v[0], 1);
+                    if (g.ok) put_one(g, v[0], got, t0, NT <= 32 ? x_old[0] : 0.f, NT <= 32, !(lane & 1));
+                } else if (g.kind == SEG_CLAMPED_GLU || g.kind == SEG_SILU_GLU) {
                     // neighbouring lanes hold gate_j and up_j: the even lane takes the first half of the columns
                     const bool even = !(lane & 1), clamped = g.kind == SEG_CLAMPED_GLU;
                     __nv_bfloat16* dst = g.t + (t0 + (even ? 0 : CH / 2)) * g.ld;
@@ -306,35 +349,55 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_dense_kernel(const __grid_co
                     finish(c0, v);
                 }
             } else if (NT <= 32 && p.cluster > 1) {
-                // [token / 4][row][4] in the ring, which nothing uses any more
-                float* mine = reinterpret_cast<float*>(ring) + (quad * 32 + lane) * 4;
+                // a part: [token / 4][row][4]
+                const int at = (quad * 32 + lane) * 4, groups = (cols + 3) / 4;
                 float v[CH];
                 load(0, v);
-                if (rank > 0)
+                auto add = [&](int c, const float4& t) { v[4 * c] += t.x; v[4 * c + 1] += t.y; v[4 * c + 2] += t.z; v[4 * c + 3] += t.w; };
+                if (p.push) {
+                    float* box = reinterpret_cast<float*>(ring + size_t(STAGES) * STAGE);
+                    cluster_wait();
+                    if (rank > 0) {
+                        const uint32_t dst = cluster_addr(box + (rank - 1) * groups * 512 + at, 0);
 #pragma unroll
-                    for (int c = 0; c < CH; c += 4) *reinterpret_cast<float4*>(mine + c * 128) = make_float4(v[c], v[c + 1], v[c + 2], v[c + 3]);
-                __syncwarp();
-                cluster_sync();
-                if (rank == 0) {
-                    constexpr int QB = CH == 16 ? 4 : 2;   // loads of QB parts in flight together; added in their order
-                    for (int q0 = 1; q0 < p.cluster; q0 += QB) {
-                        float4 t[QB][CH / 4];
-#pragma unroll
-                        for (int q = 0; q < QB; ++q) {
-                            const uint32_t src = cluster_addr(mine, min(q0 + q, p.cluster - 1));
-#pragma unroll
-                            for (int c = 0; c < CH / 4; ++c) t[q][c] = cluster_load4(src + c * 512 * 4);
-                        }
-#pragma unroll
-                        for (int q = 0; q < QB; ++q)
-                            if (q0 + q < p.cluster)
-#pragma unroll
-                                for (int c = 0; c < CH / 4; ++c) { v[4 * c] += t[q][c].x; v[4 * c + 1] += t[q][c].y; v[4 * c + 2] += t[q][c].z; v[4 * c + 3] += t[q][c].w; }
+                        for (int c = 0; c < CH / 4; ++c) if (c < groups) cluster_store4(dst + c * 2048, make_float4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]));
                     }
-                    finish(0, v);
+                    __syncwarp();
+                    cluster_sync();
+                    if (rank == 0) {
+                        for (int q = 1; q < p.cluster; ++q)
+#pragma unroll
+                            for (int c = 0; c < CH / 4; ++c) if (c < groups) add(c, *reinterpret_cast<const float4*>(box + ((q - 1) * groups + c) * 512 + at));
+                        finish(0, v);
+                    }
+                } else {
+                    float* mine = reinterpret_cast<float*>(ring) + at;   // nothing uses the ring any more
+                    if (rank > 0)
+#pragma unroll
+                        for (int c = 0; c < CH / 4; ++c) *reinterpret_cast<float4*>(mine + c * 512) = make_float4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]);
+                    __syncwarp();
+                    cluster_sync();
+                    if (rank == 0) {
+                        constexpr int QB = CH == 16 ? 4 : 2;   // loads of QB parts in flight together; added in their order
+                        for (int q0 = 1; q0 < p.cluster; q0 += QB) {
+                            float4 t[QB][CH / 4];
+#pragma unroll
+                            for (int q = 0; q < QB; ++q) {
+                                const uint32_t src = cluster_addr(mine, min(q0 + q, p.cluster - 1));
+#pragma unroll
+                                for (int c = 0; c < CH / 4; ++c) t[q][c] = cluster_load4(src + c * 2048);
+                            }
+#pragma unroll
+                            for (int q = 0; q < QB; ++q)
+                                if (q0 + q < p.cluster)
+#pragma unroll
+                                    for (int c = 0; c < CH / 4; ++c) add(c, t[q][c]);
+                        }
+                        finish(0, v);
+                    }
+                    __syncwarp();
+                    cluster_sync();   // nobody leaves while its part is read
                 }
-                __syncwarp();
-                cluster_sync();   // nobody leaves while its part is read
             } else {
                 // a shared tile: this CTA's part goes to its slot (0: the part its share starts with, 1: the other one)
                 float* mine = p.part + (size_t(blockIdx.x) * 2 + (u0 >= t_begin ? 0 : 1)) * (NT * 128);
@@ -406,8 +469,8 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmPara
     p.tt_count = (p.m + NT - 1) / NT;
     const long long tiles = (long long)((w.N + 127) / 128) * p.tt_count;
     auto kern = gemm_dense_kernel<NT>;
-    const size_t smem = size_t(Ring<NT>::STAGES) * Ring<NT>::STAGE + 1024;
-    FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+    const size_t smem = size_t(Ring<NT>::STAGES) * Ring<NT>::STAGE + Ring<NT>::EXCHANGE + 1024;
+    FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(std::max(smem, size_t(120) * 1024))));
     if (NT <= 32 && tiles <= sms) {
         // most parts per tile whose clusters all run at once (a cluster lies within one group of SMs, so large ones leave SMs idle)
         static int fits[9] = {0};
@@ -415,7 +478,7 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmPara
             for (int c = 1; c <= 8; ++c) {
                 cudaLaunchConfig_t cfg{};
                 cudaLaunchAttribute at[1];
-                cfg.gridDim = dim3(unsigned(c * 148)); cfg.blockDim = dim3(kThreads); cfg.dynamicSmemBytes = smem;
+                cfg.gridDim = dim3(unsigned(c * 148)); cfg.blockDim = dim3(kThreads); cfg.dynamicSmemBytes = std::max(smem, size_t(120) * 1024);   // one CTA per SM
                 at[0].id = cudaLaunchAttributeClusterDimension;
                 at[0].val.clusterDim.x = unsigned(c); at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
                 cfg.attrs = at; cfg.numAttrs = 1;
@@ -425,6 +488,7 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmPara
         for (int c = 1; c <= 8; ++c) if (tiles <= fits[c] && (c == 1 || p.nk >= 2 * c)) parts = c;
         if (tiles * parts >= 90 || tiles <= fits[8]) {
             p.cluster = parts;
+            p.push = (parts - 1) * ((p.m + 3) / 4) * 2048 <= Ring<NT>::EXCHANGE;
             FORGE_CUDA(launch_pdl_cluster(kern, dim3(unsigned(tiles * parts)), dim3(kThreads), parts, smem, st, mx, p));
             FORGE_LAUNCH_CHECK();
             return FORGE_OK;
@@ -492,25 +556,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             if (!g[i].ok) continue;
-            float* dst = g[i].f32 + t * g[i].ld;
-            const float v = acc[i][j];
-            switch (g[i].kind) {
-                case SEG_CLAMPED_GLU: if (!(i & 1)) *dst = clamped_glu(v, acc[i | 1][j], g[i].limit); break;
-                case SEG_SILU_GLU: if (!(i & 1)) *dst = silu(v) * acc[i | 1][j]; break;
-                case SEG_SIGMOID: case SEG_SIGMOID_F32: *dst = sigmoid(v); break;
-                case SEG_SILU: *dst = silu(v); break;
-                case SEG_TANH: *dst = tanhf(v); break;
-                case SEG_DECAY: *dst = -g[i].mul * softplus(v + g[i].add); break;
-                case SEG_EXP_DECAY: *dst = -expf(v + g[i].add); break;
-                case SEG_CAST: g[i].f32[size_t(g[i].place ? g[i].place[t] : int(t)) * g[i].ld] = v; break;
-                case SEG_RESID: {
-                    const float x = (g[i].fresh ? 0.f : *dst) + v + g[i].add;
-                    *dst = x;
-                    if (g[i].after) g[i].next[t * g[i].next_ld] = g[i].next_value(x);
-                    break;
-                }
-                default: *dst = v;
-            }
+            put_one(g[i], acc[i][j], acc[i | 1][j], t, 0.f, false, !(i & 1));
         }
     }
 }
