@@ -8,8 +8,7 @@
 // same amount whatever the number of tiles.  A tile that several CTAs share is finished by the last of them to arrive
 // (ticket): every share is left in scratch memory and added in K order, so the result does not depend on the order of
 // arrival.  Nobody waits for another CTA.  Up to 32 tokens with at most one tile per SM, the CTAs of a tile form a cluster instead: each takes
-// an equal part of its K steps, and the first adds the parts through distributed shared memory (few columns are stored there by the
-// others; many are fetched).  The ring of the sixteen-token form leaves room for a second CTA on the SM: the next product's weights are
+// an equal part of its K steps and finishes some of its tokens, for which the others store their parts into its shared memory.  The ring of the sixteen-token form leaves room for a second CTA on the SM: the next product's weights are
 // requested while this one ends.
 // Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = epilogue (TMEM lane = weight row).
 // The weights lie in memory as the very images the ring holds (dense_tile_image), so a stage is one contiguous 16 KB bulk copy.
@@ -123,7 +122,6 @@ struct GemmParams {
     uint32_t units;          // K steps of the tiles after them, dealt to the first `sharers` CTAs (at most one per step: no share is empty)
     int sharers;
     int cluster;             // > 0: CTA i takes part i % cluster of the K steps of tile i / cluster, and nothing is dealt out
-    bool push;               // the parts fit EXCHANGE
     float* part; int* tickets;
     int* err;
 };
@@ -154,7 +152,7 @@ struct Work {
 template <int NT> struct Ring {
     static constexpr int X_BYTES = NT * 128, STAGE = 16384 + X_BYTES;
     static constexpr int STAGES = NT <= 16 ? 5 : (200 * 1024) / STAGE;
-    static constexpr int EXCHANGE = NT <= 16 ? 18432 : 0;   // parts that the other CTAs of a cluster store
+    static constexpr int EXCHANGE = NT <= 16 ? 14336 : NT <= 32 ? 20480 : 0;   // parts that the other CTAs of a cluster store: four tokens take 2 KB
     static constexpr uint32_t COLS = NT <= 16 ? 32 : 2 * NT;   // two accumulators
 };
 
@@ -187,7 +185,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
     fence_after();
     const uint32_t tmem = s_tmem;
     pdl_trigger();
-    if (p.cluster > 1 && p.push) cluster_arrive();   // nobody stores into a CTA that has not begun
+    if (p.cluster > 1) cluster_arrive();   // nobody stores into a CTA that has not begun
 
     if (warp == 0) {
         if (lane == 0) {
@@ -222,8 +220,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
         }
         if (p.cluster > 1) {
             __syncwarp();
-            if (p.push) cluster_wait();
-            else cluster_sync();
+            cluster_wait();
             cluster_sync();
         }
     } else if (warp == 1) {
@@ -253,8 +250,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
         }
         if (p.cluster > 1) {
             __syncwarp();
-            if (p.push) cluster_wait();
-            else cluster_sync();
+            cluster_wait();
             cluster_sync();
         }
     } else {
@@ -272,9 +268,9 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
             // every warp's rows lie in one segment (segments start at multiples of 32 rows)
             const RowOut<__nv_bfloat16> g = row_out<__nv_bfloat16>(p.out, row, row0);
             float x_old[CH];   // few tokens: the residual is on its way while the product is formed
-            if (NT <= 32 && g.kind == SEG_RESID && g.ok && !g.fresh && rank == 0)
+            if (NT <= 32 && g.kind == SEG_RESID && g.ok && !g.fresh)
 #pragma unroll
-                for (int c = 0; c < CH; ++c) if (c < cols) x_old[c] = g.f32[size_t(tok0 + c) * g.ld];
+                for (int c = 0; c < CH; ++c) if (c < cols && (p.cluster <= 1 || (c >> 2) % p.cluster == rank)) x_old[c] = g.f32[size_t(tok0 + c) * g.ld];
             // the four warps meet at the barriers of a shared tile: one whose wait gave up must not leave the loop alone
             if (!mbar_wait(&acc_full[buf], (seg_i >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
             fence_after();
@@ -349,54 +345,40 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                     finish(c0, v);
                 }
             } else if (NT <= 32 && p.cluster > 1) {
-                // a part: [token / 4][row][4]
-                const int at = (quad * 32 + lane) * 4, groups = (cols + 3) / 4;
+                // the tokens 4 c .. 4 c + 3 are finished by CTA c % cluster: box [c / cluster][sender][row][4]
+                const int at = (quad * 32 + lane) * 4, groups = (cols + 3) / 4, senders = p.cluster - 1;
+                float* box = reinterpret_cast<float*>(ring + size_t(STAGES) * STAGE);
                 float v[CH];
                 load(0, v);
-                auto add = [&](int c, const float4& t) { v[4 * c] += t.x; v[4 * c + 1] += t.y; v[4 * c + 2] += t.z; v[4 * c + 3] += t.w; };
-                if (p.push) {
-                    float* box = reinterpret_cast<float*>(ring + size_t(STAGES) * STAGE);
-                    cluster_wait();
-                    if (rank > 0) {
-                        const uint32_t dst = cluster_addr(box + (rank - 1) * groups * 512 + at, 0);
+                cluster_wait();
 #pragma unroll
-                        for (int c = 0; c < CH / 4; ++c) if (c < groups) cluster_store4(dst + c * 2048, make_float4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]));
+                for (int c = 0; c < CH / 4; ++c) {
+                    const int to = c % p.cluster;
+                    if (c < groups && to != rank)
+                        cluster_store4(cluster_addr(box + (c / p.cluster * senders + (rank < to ? rank : rank - 1)) * 512 + at, to), make_float4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]));
+                }
+                __syncwarp();
+                cluster_sync();
+#pragma unroll 1
+                for (int k = 0; rank + k * p.cluster < groups; ++k) {
+                    float t[4] = {0.f, 0.f, 0.f, 0.f}, old[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                    for (int c = 0; c < CH / 4; ++c)
+                        if (c == rank + k * p.cluster)
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) { t[e] = v[4 * c + e]; old[e] = x_old[4 * c + e]; }
+                    for (int q = 0; q < senders; ++q) {
+                        const float4 o = *reinterpret_cast<const float4*>(box + (k * senders + q) * 512 + at);
+                        t[0] += o.x; t[1] += o.y; t[2] += o.z; t[3] += o.w;
                     }
-                    __syncwarp();
-                    cluster_sync();
-                    if (rank == 0) {
-                        for (int q = 1; q < p.cluster; ++q)
-#pragma unroll
-                            for (int c = 0; c < CH / 4; ++c) if (c < groups) add(c, *reinterpret_cast<const float4*>(box + ((q - 1) * groups + c) * 512 + at));
-                        finish(0, v);
+                    const int c0 = (rank + k * p.cluster) * 4;
+#pragma unroll 1
+                    for (int e = 0; e < min(4, cols - c0); ++e) {
+                        const float got = __shfl_xor_sync(0xffffffffu, t[0], 1);
+                        if (g.ok) put_one(g, t[0], got, size_t(tok0 + c0 + e), old[0], true, !(lane & 1));
+                        t[0] = t[1]; t[1] = t[2]; t[2] = t[3];
+                        old[0] = old[1]; old[1] = old[2]; old[2] = old[3];
                     }
-                } else {
-                    float* mine = reinterpret_cast<float*>(ring) + at;   // nothing uses the ring any more
-                    if (rank > 0)
-#pragma unroll
-                        for (int c = 0; c < CH / 4; ++c) *reinterpret_cast<float4*>(mine + c * 512) = make_float4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]);
-                    __syncwarp();
-                    cluster_sync();
-                    if (rank == 0) {
-                        constexpr int QB = CH == 16 ? 4 : 2;   // loads of QB parts in flight together; added in their order
-                        for (int q0 = 1; q0 < p.cluster; q0 += QB) {
-                            float4 t[QB][CH / 4];
-#pragma unroll
-                            for (int q = 0; q < QB; ++q) {
-                                const uint32_t src = cluster_addr(mine, min(q0 + q, p.cluster - 1));
-#pragma unroll
-                                for (int c = 0; c < CH / 4; ++c) t[q][c] = cluster_load4(src + c * 2048);
-                            }
-#pragma unroll
-                            for (int q = 0; q < QB; ++q)
-                                if (q0 + q < p.cluster)
-#pragma unroll
-                                    for (int c = 0; c < CH / 4; ++c) add(c, t[q][c]);
-                        }
-                        finish(0, v);
-                    }
-                    __syncwarp();
-                    cluster_sync();   // nobody leaves while its part is read
                 }
             } else {
                 // a shared tile: this CTA's part goes to its slot (0: the part its share starts with, 1: the other one)
@@ -485,10 +467,10 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmPara
                 FORGE_CUDA(cudaOccupancyMaxActiveClusters(&fits[c], kern, &cfg));
             }
         int parts = 0;
-        for (int c = 1; c <= 8; ++c) if (tiles <= fits[c] && (c == 1 || p.nk >= 2 * c)) parts = c;
+        for (int c = 1; c <= 8; ++c)
+            if (tiles <= fits[c] && (c == 1 || (p.nk >= 2 * c && (c - 1) * ((NT / 4 + c - 1) / c) * 2048 <= Ring<NT>::EXCHANGE))) parts = c;
         if (tiles * parts >= 90 || tiles <= fits[8]) {
             p.cluster = parts;
-            p.push = (parts - 1) * ((p.m + 3) / 4) * 2048 <= Ring<NT>::EXCHANGE;
             FORGE_CUDA(launch_pdl_cluster(kern, dim3(unsigned(tiles * parts)), dim3(kThreads), parts, smem, st, mx, p));
             FORGE_LAUNCH_CHECK();
             return FORGE_OK;

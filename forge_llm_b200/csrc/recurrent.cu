@@ -60,31 +60,46 @@ template <typename T, int H> struct LowRows {
     }
 };
 
-// One CTA = 32 value columns of one head of one row; the CTAs of a head form a cluster for the norm of its output.  A thread holds
-// the state of one column in the rows warp, warp + 8, ... of it; state, weights and what the convolution keeps are read before
+// One CTA = 32 CPL value columns of one head of one row; the CTAs of a head form a cluster for the norm of its output.  A thread holds
+// the state of CPL columns in the rows warp, warp + 8, ... of it; state, weights and what the convolution keeps are read before
 // the dependency wait.
-template <typename T, bool DELTA, bool CHANNEL, int RPT>
-__global__ void __launch_bounds__(256) recur_decode_kernel(const RecurDims d, const RecurArgs a, const StepRows rows) {
+template <int N> __device__ __forceinline__ void load_cols(float (&v)[N], const float* p) {
+    if constexpr (N == 4) { const float4 t = *reinterpret_cast<const float4*>(p); v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w; }
+    else if constexpr (N == 2) { const float2 t = *reinterpret_cast<const float2*>(p); v[0] = t.x; v[1] = t.y; }
+    else v[0] = *p;
+}
+template <int N> __device__ __forceinline__ void store_cols(float* p, const float (&v)[N]) {
+    if constexpr (N == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else if constexpr (N == 2) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+    else *p = v[0];
+}
+template <typename T, bool DELTA, bool CHANNEL, int RPT, int CPL>
+__global__ void __launch_bounds__(256, CPL > 1 ? 2 : 1) recur_decode_kernel(const RecurDims d, const RecurArgs a, const StepRows rows) {
     extern __shared__ float sm[];
     float* sq = sm;                 // [dim] queries, keys, decays
     float* sk = sq + d.dim;
     float* sg = sk + d.dim;
-    float* sv = sg + d.dim;         // [32]
-    float* sgate = sv + 32;         // [32]
-    float* slow = sm + ((3 * d.dim + 64 + 3) & ~3);   // [2][low_k] inner values of decay and gate
-    __shared__ float red[8][33], redo[8][33], wsum[8][3], part;
+    float* sv = sg + d.dim;         // [NC]
+    constexpr int NC = 32 * CPL;
+    float* sgate = sv + NC;         // [NC]
+    float* slow = sm + ((3 * d.dim + 2 * NC + 3) & ~3);   // [2][low_k] inner values of decay and gate
+    __shared__ __align__(16) float red[8][NC], redo[8][NC];
+    __shared__ float wsum[8][3], part;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int split = blockIdx.x, splits = gridDim.x, h = blockIdx.y, r = blockIdx.z;
-    const int g = h / (d.heads / d.groups), c0 = split * 32, nc = min(32, d.vdim - c0);
+    const int g = h / (d.heads / d.groups), c0 = split * NC, nc = min(NC, d.vdim - c0), cl = lane * CPL;
+    const bool own = cl < nc;       // this lane's columns (vdim is a multiple of CPL)
     pdl_trigger();
     // positions are written in front of the step's first kernel, the state in the last step: both are complete
     const int pos = rows.pos[r], slot = state_slot(rows, r);
-    float* S = a.state + (size_t(slot) * d.heads + h) * d.dim * d.vdim + c0 + lane;
-    float st[RPT];
+    float* S = a.state + (size_t(slot) * d.heads + h) * d.dim * d.vdim + c0 + cl;
+    float st[RPT][CPL];
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
         const int row = warp + 8 * i;
-        st[i] = pos > 0 && row < d.dim && lane < nc ? S[size_t(row) * d.vdim] : 0.f;
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) st[i][c] = 0.f;
+        if (pos > 0 && row < d.dim && own) load_cols<CPL>(st[i], S + size_t(row) * d.vdim);
     }
     const int n_in = 2 * d.dim + nc;      // this CTA's channels: q, k, its values
     auto channel = [&](int i) { return i < d.dim ? g * d.dim + i : i < 2 * d.dim ? d.qk() + g * d.dim + i - d.dim : 2 * d.qk() + h * d.vdim + c0 + i - 2 * d.dim; };
@@ -103,14 +118,16 @@ __global__ void __launch_bounds__(256) recur_decode_kernel(const RecurDims d, co
     }
     const bool two_step = CHANNEL && a.decay_w, low_gate = two_step && a.gate_w;
     LowRows<T, 4> low_d(static_cast<const T*>(a.decay_w) + size_t(h) * d.dim * a.low_k, two_step ? d.dim : 0, a.low_k);
-    LowRows<T, 1> low_g(static_cast<const T*>(a.gate_w) + size_t(h * d.vdim + c0) * a.low_k, low_gate ? nc : 0, a.low_k);
+    LowRows<T, CPL> low_g(static_cast<const T*>(a.gate_w) + size_t(h * d.vdim + c0) * a.low_k, low_gate ? nc : 0, a.low_k);
     pdl_wait();
     if (two_step) {
         const T* in = static_cast<const T*>(a.low) + size_t(r) * a.low_ld;
         for (int i = tid; i < (low_gate ? 2 : 1) * a.low_k; i += 256) slow[i] = to_f(in[i < a.low_k ? i : a.gate_col + i - a.low_k]);
     }
     const T* x = static_cast<const T*>(a.x) + size_t(r) * a.x_ld;
-    float gate = lane < nc && !low_gate ? to_f(static_cast<const T*>(a.gate)[size_t(r) * a.gate_ld + h * d.vdim + c0 + lane]) : 0.f;
+    float gate[CPL];
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) gate[c] = own && !low_gate ? to_f(static_cast<const T*>(a.gate)[size_t(r) * a.gate_ld + h * d.vdim + c0 + cl + c]) : 0.f;
     for (int i = tid; i < n_in; i += 256) {
         const int ch = channel(i);
         const T in = x[ch];
@@ -146,76 +163,99 @@ __global__ void __launch_bounds__(256) recur_decode_kernel(const RecurDims d, co
         if (low_gate) low_g.run(slow + a.low_k, [&](int i, float z) { sgate[i] = sigmoid(z); });
     }
     __syncthreads();
-    if (low_gate && lane < nc) gate = sgate[lane];
+    if (low_gate && own)
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) gate[c] = sgate[cl + c];
     float t0 = 0.f, t1 = 0.f;
 #pragma unroll
     for (int w = 0; w < 8; ++w) { t0 += wsum[w][0]; t1 += wsum[w][1]; }
     const float qs = DELTA ? d.q_scale / sqrtf(t0 + 1e-6f) : 1.f, ks = DELTA ? 1.0f / sqrtf(t1 + 1e-6f) : 1.f;
-    float o;
+    float o[CPL], sum8[CPL];
+    auto all_warps = [&](float (*buf)[NC], const float (&mine)[CPL]) {   // sum over the warps' rows
+        store_cols<CPL>(&buf[warp][cl], mine);
+        __syncthreads();
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) sum8[c] = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) {
+            float t[CPL];
+            load_cols<CPL>(t, &buf[w][cl]);
+#pragma unroll
+            for (int c = 0; c < CPL; ++c) sum8[c] += t[c];
+        }
+    };
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) o[c] = 0.f;
     if constexpr (DELTA) {
-        float dot = 0.f;
+        float dot[CPL], u[CPL];
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) dot[c] = 0.f;
 #pragma unroll
         for (int i = 0; i < RPT; ++i) {
             const int row = warp + 8 * i;
             if (row < d.dim) {
-                st[i] *= CHANNEL ? sg[row] : g1;
-                dot = fmaf(st[i], sk[row] * ks, dot);
+                const float w = CHANNEL ? sg[row] : g1, k = sk[row] * ks;
+#pragma unroll
+                for (int c = 0; c < CPL; ++c) { st[i][c] *= w; dot[c] = fmaf(st[i][c], k, dot[c]); }
             }
         }
-        red[warp][lane] = dot;
-        __syncthreads();
-        dot = 0.f;
+        all_warps(red, dot);
 #pragma unroll
-        for (int w = 0; w < 8; ++w) dot += red[w][lane];
-        const float u = lane < nc ? beta * (sv[lane] - dot) : 0.f;
-        o = 0.f;
+        for (int c = 0; c < CPL; ++c) u[c] = own ? beta * (sv[cl + c] - sum8[c]) : 0.f;
 #pragma unroll
         for (int i = 0; i < RPT; ++i) {
             const int row = warp + 8 * i;
             if (row < d.dim) {
-                st[i] = fmaf(sk[row] * ks, u, st[i]);
-                o = fmaf(st[i], sq[row] * qs, o);
-                if (lane < nc) S[size_t(row) * d.vdim] = st[i];
+                const float k = sk[row] * ks, q = sq[row] * qs;
+#pragma unroll
+                for (int c = 0; c < CPL; ++c) { st[i][c] = fmaf(k, u[c], st[i][c]); o[c] = fmaf(st[i][c], q, o[c]); }
+                if (own) store_cols<CPL>(S + size_t(row) * d.vdim, st[i]);
             }
         }
     } else {
-        const float v = lane < nc ? sv[lane] : 0.f;
-        o = 0.f;
+        float v[CPL];
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) v[c] = own ? sv[cl + c] : 0.f;
 #pragma unroll
         for (int i = 0; i < RPT; ++i) {
             const int row = warp + 8 * i;
             if (row < d.dim) {
-                o = fmaf(st[i], sq[row], o);
-                st[i] = fmaf(sk[row], v, st[i] * (CHANNEL ? sg[row] : g1));
-                if (lane < nc) S[size_t(row) * d.vdim] = st[i];
+                const float w = CHANNEL ? sg[row] : g1, k = sk[row], q = sq[row];
+#pragma unroll
+                for (int c = 0; c < CPL; ++c) { o[c] = fmaf(st[i][c], q, o[c]); st[i][c] = fmaf(k, v[c], st[i][c] * w); }
+                if (own) store_cols<CPL>(S + size_t(row) * d.vdim, st[i]);
             }
         }
     }
-    redo[warp][lane] = o;
-    __syncthreads();
-    o = 0.f;
+    all_warps(redo, o);
     if (warp == 0) {
+        float ss = 0.f;
 #pragma unroll
-        for (int w = 0; w < 8; ++w) o += redo[w][lane];
-        if constexpr (!DELTA) o = fmaf(t0, lane < nc ? sv[lane] : 0.f, o);
-        const float ss = warp_sum(lane < nc ? o * o : 0.f);
+        for (int c = 0; c < CPL; ++c) {
+            o[c] = sum8[c];
+            if constexpr (!DELTA) o[c] = fmaf(t0, own ? sv[cl + c] : 0.f, o[c]);
+            if (own) ss = fmaf(o[c], o[c], ss);
+        }
+        ss = warp_sum(ss);
         if (lane == 0) part = ss;
     }
     float total;
     if (splits > 1) {
-        cg::cluster_group cl = cg::this_cluster();
-        cl.sync();
+        cg::cluster_group cluster = cg::this_cluster();
+        cluster.sync();
         total = 0.f;
         if (warp == 0)
-            for (int s = 0; s < splits; ++s) total += *cl.map_shared_rank(&part, s);
-        cl.sync();   // nobody leaves while its part is read
+            for (int s = 0; s < splits; ++s) total += *cluster.map_shared_rank(&part, s);
+        cluster.sync();   // nobody leaves while its part is read
     } else {
         __syncthreads();
         total = part;
     }
-    if (warp == 0 && lane < nc) {
+    if (warp == 0 && own) {
         const float inv = 1.0f / sqrtf(total / float(d.vdim) + d.eps);
-        static_cast<T*>(a.out)[size_t(r) * a.out_ld + h * d.vdim + c0 + lane] = to_t<T>(o * inv * a.norm[size_t(h) * a.norm_head + c0 + lane] * gate);
+        T* out = static_cast<T*>(a.out) + size_t(r) * a.out_ld + h * d.vdim + c0 + cl;
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) out[c] = to_t<T>(o[c] * inv * a.norm[size_t(h) * a.norm_head + c0 + cl + c] * gate[c]);
     }
 }
 
@@ -548,18 +588,24 @@ __global__ void __launch_bounds__(256) add_normed_pair_kernel(float* __restrict_
     }
 }
 
-template <typename T, bool DELTA, bool CHANNEL, int RPT>
+template <typename T, bool DELTA, bool CHANNEL, int RPT, int CPL>
 int32_t launch_decode(const RecurDims& d, const RecurArgs& a, const StepRows& rows, cudaStream_t st) {
-    const int splits = (d.vdim + 31) / 32;
-    FORGE_CUDA(launch_pdl_cluster(recur_decode_kernel<T, DELTA, CHANNEL, RPT>, dim3(splits, d.heads, rows.n), dim3(256), splits, sizeof(float) * (3 * size_t(d.dim) + 68 + 2 * size_t(a.low_k)), st, d, a, rows));
+    const int splits = (d.vdim + 32 * CPL - 1) / (32 * CPL);
+    const size_t smem = sizeof(float) * (3 * size_t(d.dim) + 64 * CPL + 4 + 2 * size_t(a.low_k));
+    FORGE_CUDA(launch_pdl_cluster(recur_decode_kernel<T, DELTA, CHANNEL, RPT, CPL>, dim3(splits, d.heads, rows.n), dim3(256), splits, smem, st, d, a, rows));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
 template <typename T, bool DELTA, bool CHANNEL>
 int32_t decode_t(const RecurDims& d, const RecurArgs& a, const StepRows& rows, cudaStream_t st) {
-    if (d.dim <= 64) return launch_decode<T, DELTA, CHANNEL, 8>(d, a, rows, st);
-    if (d.dim <= 128) return launch_decode<T, DELTA, CHANNEL, 16>(d, a, rows, st);
-    return launch_decode<T, DELTA, CHANNEL, 32>(d, a, rows, st);
+    // enough rows to fill the SMs: whole heads (what all columns of a head share is formed once)
+    const bool whole = (long long)rows.n * d.heads >= 148 && d.vdim > 32;
+    if (whole && d.vdim <= 64 && d.vdim % 2 == 0 && d.dim <= 64) return launch_decode<T, DELTA, CHANNEL, 8, 2>(d, a, rows, st);
+    if (whole && d.vdim % 4 == 0 && d.dim <= 64) return launch_decode<T, DELTA, CHANNEL, 8, 4>(d, a, rows, st);
+    if (whole && d.vdim % 4 == 0 && d.dim <= 128) return launch_decode<T, DELTA, CHANNEL, 16, 4>(d, a, rows, st);
+    if (d.dim <= 64) return launch_decode<T, DELTA, CHANNEL, 8, 1>(d, a, rows, st);
+    if (d.dim <= 128) return launch_decode<T, DELTA, CHANNEL, 16, 1>(d, a, rows, st);
+    return launch_decode<T, DELTA, CHANNEL, 32, 1>(d, a, rows, st);
 }
 template <typename T, bool DELTA, bool CHANNEL>
 int32_t scan_t(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, const ScanSeg* segs, int n_segs, cudaStream_t st) {
