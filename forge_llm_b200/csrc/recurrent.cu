@@ -111,7 +111,7 @@ __global__ void __launch_bounds__(256, CPL > 1 ? 2 : 1) recur_decode_kernel(cons
             float v = 0.f;
             for (int j = 0; j < d.taps - 1; ++j) {
                 const int p = pos - (d.taps - 1 - j);
-                if (p >= 0) v = fmaf(a.conv[size_t(ch) * d.taps + j], to_f(ring[size_t(p % d.taps) * d.channels() + ch]), v);
+                if (p >= 0) v = fmaf(a.conv[size_t(j) * d.channels() + ch], to_f(ring[size_t(p % d.taps) * d.channels() + ch]), v);
             }
             *place(i) = v;
         }
@@ -132,7 +132,7 @@ __global__ void __launch_bounds__(256, CPL > 1 ? 2 : 1) recur_decode_kernel(cons
         const int ch = channel(i);
         const T in = x[ch];
         if constexpr (DELTA) {
-            const float v = fmaf(a.conv[size_t(ch) * d.taps + d.taps - 1], to_f(in), *place(i));
+            const float v = fmaf(a.conv[size_t(d.taps - 1) * d.channels() + ch], to_f(in), *place(i));
             *place(i) = to_f(to_t<T>(silu(v)));
             // one CTA keeps each input
             if (i >= 2 * d.dim || (split == 0 && h % (d.heads / d.groups) == 0)) static_cast<T*>(a.ring)[size_t(slot) * d.ring_values() + size_t(pos % d.taps) * d.channels() + ch] = in;
@@ -286,7 +286,7 @@ __global__ void __launch_bounds__(256) conv_rows_kernel(const RecurDims d, const
                 float in = 0.f;
                 if (q >= 0) in = to_f(x[size_t(q) * a.x_ld + ch]);
                 else if (p >= 0) in = to_f(ring[size_t(p % d.taps) * d.channels() + ch]);
-                v = fmaf(a.conv[size_t(ch) * d.taps + j], in, v);
+                v = fmaf(a.conv[size_t(j) * d.channels() + ch], in, v);
             }
             const T o = to_t<T>(silu(v));
             y[size_t(t) * d.channels() + ch] = o;
@@ -302,12 +302,13 @@ __global__ void __launch_bounds__(256) conv_rows_kernel(const RecurDims d, const
             for (int t = max(0, s.n - d.taps); t < s.n; ++t) ring[size_t((s.pos0 + t) % d.taps) * d.channels() + ch0 + c] = x[size_t(t) * a.x_ld + ch0 + c];
 }
 
-// The same for bfloat16 sizes in whole 16-byte pieces and at most four taps: a thread carries eight channels over eight tokens at a time.
+// The same for bfloat16 sizes in whole 16-byte pieces and at most four taps: a thread carries eight channels over eight tokens.
 constexpr int kConvRun = 8;
+__device__ __forceinline__ float fast_silu(float v) { return __fdividef(v, 1.0f + __expf(-v)); }   // far inside a bfloat16 rounding
 __global__ void __launch_bounds__(128) conv_rows8_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs) {
     using bf16 = __nv_bfloat16;
     const ScanSeg s = segs[blockIdx.z];
-    const int t0 = blockIdx.x * kConvTile, ch = (blockIdx.y * 128 + threadIdx.x) * 8, channels = d.channels();
+    const int t0 = blockIdx.x * kConvRun, ch = (blockIdx.y * 128 + threadIdx.x) * 8, channels = d.channels();
     if (t0 >= s.n) return;
     const bool ok = ch < channels;
     const bf16* x = static_cast<const bf16*>(a.x) + size_t(s.row0) * a.x_ld + ch;
@@ -315,9 +316,11 @@ __global__ void __launch_bounds__(128) conv_rows8_kernel(const RecurDims d, cons
     bf16* ring = static_cast<bf16*>(a.ring) + size_t(s.slot) * d.ring_values() + ch;
     float w[4][8], past[3][8];   // past[2]: the token before
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
+    for (int j = 0; j < 4; ++j) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) w[j][e] = ok && j >= 4 - d.taps ? a.conv[size_t(ch + e) * d.taps + j - (4 - d.taps)] : 0.f;
+        for (int e = 0; e < 8; ++e) w[j][e] = 0.f;
+        if (ok && j >= 4 - d.taps) load8(w[j], a.conv + size_t(j - (4 - d.taps)) * channels + ch);
+    }
 #pragma unroll
     for (int j = 0; j < 3; ++j) {
         const int q = t0 - 3 + j, p = s.pos0 + q;
@@ -327,36 +330,34 @@ __global__ void __launch_bounds__(128) conv_rows8_kernel(const RecurDims d, cons
     }
     const int lanes = d.dim / 8, unit = ch / d.dim;   // threads of a head of q or k
     const bool is_qk = ok && unit < 2 * d.groups;
-    for (int t1 = t0; t1 < min(s.n, t0 + kConvTile); t1 += kConvRun) {
-        uint4 in[kConvRun];
+    uint4 in[kConvRun];
 #pragma unroll
-        for (int i = 0; i < kConvRun; ++i) in[i] = ok && t1 + i < s.n ? *reinterpret_cast<const uint4*>(x + size_t(t1 + i) * a.x_ld) : make_uint4(0, 0, 0, 0);
+    for (int i = 0; i < kConvRun; ++i) in[i] = ok && t0 + i < s.n ? *reinterpret_cast<const uint4*>(x + size_t(t0 + i) * a.x_ld) : make_uint4(0, 0, 0, 0);
 #pragma unroll
-        for (int i = 0; i < kConvRun; ++i) {
-            const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&in[i]);
-            uint4 out;
-            __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&out);
-            float sum = 0.f;
+    for (int i = 0; i < kConvRun; ++i) {
+        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&in[i]);
+        uint4 out;
+        __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&out);
+        float sum = 0.f;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const float2 f = __bfloat1622float2(h[e]);
-                const float now[2] = {f.x, f.y};
-                float v[2];
+        for (int e = 0; e < 4; ++e) {
+            const float2 f = __bfloat1622float2(h[e]);
+            const float now[2] = {f.x, f.y};
+            float v[2];
 #pragma unroll
-                for (int b = 0; b < 2; ++b) {
-                    const int c = 2 * e + b;
-                    v[b] = silu(fmaf(w[3][c], now[b], fmaf(w[2][c], past[2][c], fmaf(w[1][c], past[1][c], w[0][c] * past[0][c]))));
-                    past[0][c] = past[1][c]; past[1][c] = past[2][c]; past[2][c] = now[b];
-                }
-                o[e] = __floats2bfloat162_rn(v[0], v[1]);
-                const float2 r = __bfloat1622float2(o[e]);
-                sum = fmaf(r.x, r.x, fmaf(r.y, r.y, sum));
+            for (int b = 0; b < 2; ++b) {
+                const int c = 2 * e + b;
+                v[b] = fast_silu(fmaf(w[3][c], now[b], fmaf(w[2][c], past[2][c], fmaf(w[1][c], past[1][c], w[0][c] * past[0][c]))));
+                past[0][c] = past[1][c]; past[1][c] = past[2][c]; past[2][c] = now[b];
             }
-            if (ok && t1 + i < s.n) *reinterpret_cast<uint4*>(y + size_t(t1 + i) * channels) = out;
-            for (int m = lanes >> 1; m > 0; m >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, m);
-            if (is_qk && t1 + i < s.n && (threadIdx.x & (lanes - 1)) == 0)
-                sc.unit[size_t(s.row0 + t1 + i) * 2 * d.groups + unit] = (unit < d.groups ? d.q_scale : 1.f) / sqrtf(sum + 1e-6f);
+            o[e] = __floats2bfloat162_rn(v[0], v[1]);
+            const float2 r = __bfloat1622float2(o[e]);
+            sum = fmaf(r.x, r.x, fmaf(r.y, r.y, sum));
         }
+        if (ok && t0 + i < s.n) *reinterpret_cast<uint4*>(y + size_t(t0 + i) * channels) = out;
+        for (int m = lanes >> 1; m > 0; m >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, m);
+        if (is_qk && t0 + i < s.n && (threadIdx.x & (lanes - 1)) == 0)
+            sc.unit[size_t(s.row0 + t0 + i) * 2 * d.groups + unit] = (unit < d.groups ? d.q_scale : 1.f) / sqrtf(sum + 1e-6f);
     }
     if (ok && blockIdx.x == 0)
         for (int t = max(0, s.n - d.taps); t < s.n; ++t) *reinterpret_cast<uint4*>(ring + size_t((s.pos0 + t) % d.taps) * channels) = *reinterpret_cast<const uint4*>(x + size_t(t) * a.x_ld);
@@ -622,7 +623,7 @@ int32_t segments_t(const RecurDims& d, const RecurArgs& a, const RecurScratch& s
     constexpr bool half = std::is_same<T, __nv_bfloat16>::value;
     if (d.delta) {
         const int tiles = (t.max_n + kConvTile - 1) / kConvTile, units = 2 * d.groups + (d.heads * d.vdim + 127) / 128;
-        if (half && conv_rows8_supported(d)) conv_rows8_kernel<<<dim3(tiles, (d.channels() + 1023) / 1024, t.n), 128, 0, st>>>(d, a, sc, t.segs);
+        if (half && conv_rows8_supported(d)) conv_rows8_kernel<<<dim3((t.max_n + kConvRun - 1) / kConvRun, (d.channels() + 1023) / 1024, t.n), 128, 0, st>>>(d, a, sc, t.segs);
         else conv_rows_kernel<T><<<dim3(tiles, (units + 7) / 8, t.n), 256, 0, st>>>(d, a, sc, t.segs);
         FORGE_LAUNCH_CHECK();
     }

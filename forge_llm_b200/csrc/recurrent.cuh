@@ -35,7 +35,7 @@ struct RecurArgs {
     const float* decay = nullptr; int decay_ld = 0;      // logarithms, [row][heads] or [row][heads * dim]
     const float* beta = nullptr;                         // [row][heads]
     const float* bonus = nullptr;                        // [heads][dim]
-    const float* conv = nullptr; void* ring = nullptr;   // [channels][taps]; T [slot][taps][channels]
+    const float* conv = nullptr; void* ring = nullptr;   // [taps][channels]; T [slot][taps][channels]
     float* state = nullptr;                              // [slot][heads][dim][vdim]
     // second step of two-step decays and gates, for single tokens (then decay, and gate if gate_w is set, are not read): T rows of low_k values per
     // key channel and per value over the inner values low[row], the gate's from column gate_col; a decay's logarithm is

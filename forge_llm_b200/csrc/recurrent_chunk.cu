@@ -433,7 +433,8 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
 template <int DK, int MODE> struct Scan {
     using R = Rec<DK, MODE>;
     static constexpr int SS = DK * LDN;                              // one half of a state buffer
-    static constexpr int ow = 0, oq = R::nw * R::KT, ok = oq + R::nx * R::KT, op = ok + R::nx * R::KT, ov = op + 2 * TT, os = ov + (MODE == TIME_MIX ? VT : 0),
+    static constexpr int ST = DK <= 64 ? 2 : 1;                      // buffers of every tile
+    static constexpr int ow = 0, oq = R::nw * R::KT, ok = oq + R::nx * R::KT, op = ok + R::nx * R::KT, ov = op + 2 * TT, stage = ov + (MODE == TIME_MIX ? VT : 0), os = ST * stage,
                          ou = os + 4 * SS, ox = ou + (MODE == TIME_MIX ? 0 : 2 * VT), total = ox + (MODE == HEAD_DELTA ? 2 * VT : 0);
     static constexpr size_t smem = size_t(total) * 2 + 16;
 };
@@ -442,20 +443,20 @@ constexpr int kScanThreads = 288;   // eight warps of products and a producer
 __device__ __forceinline__ void walk_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
 template <int DK, int MODE>
-__global__ void __launch_bounds__(kScanThreads) chunk_scan_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs, int* err) {
+__global__ void __launch_bounds__(kScanThreads, 1) chunk_scan_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs, int* err) {
     using L = Scan<DK, MODE>;
     using R = Rec<DK, MODE>;
-    constexpr int LDK = R::LDK, KT = R::KT;
+    constexpr int LDK = R::LDK, KT = R::KT, ST = L::ST;
     extern __shared__ __align__(16) unsigned char sm_raw[];
     bf16* sm = reinterpret_cast<bf16*>(sm_raw);
     enum { BW, BK, BQ, BP, BUFS };
-    __shared__ uint64_t full[BUFS], empty[BUFS];
+    __shared__ uint64_t full[ST][BUFS], empty[ST][BUFS];
     __shared__ int s_err;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lr = lane >> 2, lc = (lane & 3) * 2;
     const ScanSeg s = segs[blockIdx.z];
     const int h = blockIdx.y, c0 = blockIdx.x * NB, nb = gridDim.x, chunks = (s.n + C - 1) / C;
     if (tid == 0) {
-        for (int i = 0; i < BUFS; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], 8); }
+        for (int i = 0; i < ST * BUFS; ++i) { mbar_init(&full[0][i], 1); mbar_init(&empty[0][i], 8); }
         s_err = 0;
         mbar_fence_init();
     }
@@ -467,10 +468,11 @@ __global__ void __launch_bounds__(kScanThreads) chunk_scan_kernel(const RecurDim
                 const R r(sc.chunk, s.chunk0 + ch, d.heads, h, nb);
                 auto load = [&](int buf, int dst, const bf16* src, int elems, const bf16* more = nullptr, int more_dst = 0, int more_elems = 0) {
                     if (!ok) return;
-                    if (ch > 0 && !mbar_wait(&empty[buf], (ch - 1) & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; return; }
-                    mbar_expect_tx(&full[buf], uint32_t(elems + more_elems) * 2);
-                    bulk_load(sm + dst, src, uint32_t(elems) * 2, &full[buf]);
-                    if (more_elems) bulk_load(sm + more_dst, more, uint32_t(more_elems) * 2, &full[buf]);
+                    const int b = ch % ST;
+                    if (ch >= ST && !mbar_wait(&empty[b][buf], (ch / ST - 1) & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; return; }
+                    mbar_expect_tx(&full[b][buf], uint32_t(elems + more_elems) * 2);
+                    bulk_load(sm + b * L::stage + dst, src, uint32_t(elems) * 2, &full[b][buf]);
+                    if (more_elems) bulk_load(sm + b * L::stage + more_dst, more, uint32_t(more_elems) * 2, &full[b][buf]);
                 };
                 if constexpr (MODE != TIME_MIX) load(BW, L::ow, r.h, 2 * KT);
                 load(BK, L::ok, r.h + R::ok, R::nx * KT, r.h + R::ov + size_t(blockIdx.x) * VT, L::ov, MODE == TIME_MIX ? VT : 0);
@@ -481,8 +483,8 @@ __global__ void __launch_bounds__(kScanThreads) chunk_scan_kernel(const RecurDim
     } else {
         auto mat = [&](int off, int l) { return SmemMat{smem_addr(sm + off), l}; };
         // every warp meets at the barriers below, so a wait that gave up must not leave the loop alone
-        auto take = [&](int buf, int ch) { if (!mbar_wait(&full[buf], ch & 1, &s_err)) atomicExch(&s_err, 1); };
-        auto give = [&](int buf) { __syncwarp(); if (lane == 0) mbar_arrive(&empty[buf]); };
+        auto take = [&](int buf, int ch) { if (!mbar_wait(&full[ch % ST][buf], (ch / ST) & 1, &s_err)) atomicExch(&s_err, 1); };
+        auto give = [&](int buf, int ch) { __syncwarp(); if (lane == 0) mbar_arrive(&empty[ch % ST][buf]); };
         // the state: 16 rows and NI times 16 columns per warp
         constexpr int MW = DK / 16 < 8 ? DK / 16 : 8, NI = NB / 16 / (8 / MW);
         static_assert(DK / 16 / MW == 1 && NI >= 1, "one row tile per warp");
@@ -518,9 +520,7 @@ __global__ void __launch_bounds__(kScanThreads) chunk_scan_kernel(const RecurDim
         walk_sync();
         // products with 64 rows: 16 rows and 16 columns per warp
         const int mt = warp & 3, n0 = (warp >> 2) * 16, t_lo = mt * 16 + lr;
-        const SmemMat uh = mat(MODE == TIME_MIX ? L::ov : L::ou, LDN), ul = mat(L::ou + VT, LDN), xh = mat(L::ox, LDN), xl = mat(L::ox + VT, LDN);
-        const SmemMat wh = mat(L::ow, LDK), wl = mat(L::ow + KT, LDK), qh = mat(L::oq, LDK), ql = mat(L::oq + KT, LDK), kh = mat(L::ok, LDK), kl = mat(L::ok + KT, LDK);
-        const SmemMat ph = mat(L::op, LDT), pl = mat(L::op + TT, LDT);
+        const SmemMat xh = mat(L::ox, LDN), xl = mat(L::ox + VT, LDN), ul = mat(L::ou + VT, LDN);
         // what a thread reads of a chunk by itself, one chunk ahead
         struct Own { float2 u0[2][2]; float end[2], qd[2], ko[2]; };
         auto own = [&](int ch) {
@@ -539,7 +539,14 @@ __global__ void __launch_bounds__(kScanThreads) chunk_scan_kernel(const RecurDim
         Own now = own(0);
         for (int ch = 0; ch < chunks; ++ch) {
             const Own next = own(ch + 1);
+            const int at = ch % ST * L::stage;
+            const SmemMat uh = mat(MODE == TIME_MIX ? at + L::ov : L::ou, LDN), ph = mat(at + L::op, LDT), pl = mat(at + L::op + TT, LDT);
+            const SmemMat wh = mat(at + L::ow, LDK), wl = mat(at + L::ow + KT, LDK), qh = mat(at + L::oq, LDK), ql = mat(at + L::oq + KT, LDK), kh = mat(at + L::ok, LDK), kl = mat(at + L::ok + KT, LDK);
             const SmemMat sh = mat(L::os + (ch & 1) * 2 * L::SS, LDN), slo = mat(L::os + (ch & 1) * 2 * L::SS + L::SS, LDN);
+            // the state in front of the chunk as B operands of two products (shared-memory reads bound this kernel)
+            uint32_t gh[DK / 16][4], gl[DK / 16][4];
+#pragma unroll
+            for (int kt = 0; kt < DK / 16; ++kt) { sh.b_t(gh[kt], kt * 16, n0, lane); slo.b_t(gl[kt], kt * 16, n0, lane); }
             if constexpr (MODE != TIME_MIX) {   // U = U0 - W S
                 take(BW, ch);
                 float acc[3][2][4];
@@ -547,17 +554,16 @@ __global__ void __launch_bounds__(kScanThreads) chunk_scan_kernel(const RecurDim
                 for (int i = 0; i < 24; ++i) acc[i / 8][(i >> 2) & 1][i & 3] = 0.f;
 #pragma unroll
                 for (int kt = 0; kt < DK / 16; ++kt) {
-                    uint32_t fh[4], fl[4], gh[4], gl[4];
+                    uint32_t fh[4], fl[4];
                     wh.a(fh, mt * 16, kt * 16, lane); wl.a(fl, mt * 16, kt * 16, lane);
-                    sh.b_t(gh, kt * 16, n0, lane); slo.b_t(gl, kt * 16, n0, lane);
 #pragma unroll
                     for (int j = 0; j < 2; ++j) {
-                        mma(acc[0][j], fl, gh[2 * j], gh[2 * j + 1]);
-                        mma(acc[1][j], fh, gl[2 * j], gl[2 * j + 1]);
-                        mma(acc[2][j], fh, gh[2 * j], gh[2 * j + 1]);
+                        mma(acc[0][j], fl, gh[kt][2 * j], gh[kt][2 * j + 1]);
+                        mma(acc[1][j], fh, gl[kt][2 * j], gl[kt][2 * j + 1]);
+                        mma(acc[2][j], fh, gh[kt][2 * j], gh[kt][2 * j + 1]);
                     }
                 }
-                give(BW);
+                give(BW, ch);
 #pragma unroll
                 for (int j = 0; j < 2; ++j)
 #pragma unroll
@@ -595,7 +601,7 @@ __global__ void __launch_bounds__(kScanThreads) chunk_scan_kernel(const RecurDim
                     }
                 }
             }
-            if constexpr (MODE != TIME_MIX) give(BK);
+            if constexpr (MODE != TIME_MIX) give(BK, ch);
             put_state((ch + 1) & 1);
             // the read-out: q against the state in front of the chunk, then P U
             take(BQ, ch);
@@ -604,18 +610,17 @@ __global__ void __launch_bounds__(kScanThreads) chunk_scan_kernel(const RecurDim
             for (int i = 0; i < 24; ++i) acc[i / 8][(i >> 2) & 1][i & 3] = 0.f;
 #pragma unroll
             for (int kt = 0; kt < DK / 16; ++kt) {
-                uint32_t fh[4], fl[4], gh[4], gl[4];
+                uint32_t fh[4], fl[4];
                 qh.a(fh, mt * 16, kt * 16, lane);
                 if constexpr (MODE != HEAD_DELTA) ql.a(fl, mt * 16, kt * 16, lane);
-                sh.b_t(gh, kt * 16, n0, lane); slo.b_t(gl, kt * 16, n0, lane);
 #pragma unroll
                 for (int j = 0; j < 2; ++j) {
-                    if constexpr (MODE != HEAD_DELTA) mma(acc[0][j], fl, gh[2 * j], gh[2 * j + 1]);
-                    mma(acc[1][j], fh, gl[2 * j], gl[2 * j + 1]);
-                    mma(acc[2][j], fh, gh[2 * j], gh[2 * j + 1]);
+                    if constexpr (MODE != HEAD_DELTA) mma(acc[0][j], fl, gh[kt][2 * j], gh[kt][2 * j + 1]);
+                    mma(acc[1][j], fh, gl[kt][2 * j], gl[kt][2 * j + 1]);
+                    mma(acc[2][j], fh, gh[kt][2 * j], gh[kt][2 * j + 1]);
                 }
             }
-            give(BQ);
+            give(BQ, ch);
             if constexpr (MODE == HEAD_DELTA) {
 #pragma unroll
                 for (int i = 1; i < 3; ++i)
@@ -639,8 +644,8 @@ __global__ void __launch_bounds__(kScanThreads) chunk_scan_kernel(const RecurDim
                         mma(acc[2][j], fh, gh[2 * j], gh[2 * j + 1]);
                     }
                 }
-            give(BP);
-            if constexpr (MODE == TIME_MIX) give(BK);   // v lies with k
+            give(BP, ch);
+            if constexpr (MODE == TIME_MIX) give(BK, ch);   // v lies with k
             const int rows = s.n - ch * C;
 #pragma unroll
             for (int j = 0; j < 2; ++j)

@@ -173,8 +173,10 @@ int32_t load_delta(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerW
     const RecurDims& d = L.rec;
     const int H = d.heads, HV = d.heads * d.vdim;
     {
-        std::vector<float> conv;
-        for (const char* n : {"mix.q.conv", "mix.k.conv", "mix.v.conv"}) for (int64_t i = 0; i < t.at(n)->count(); ++i) conv.push_back(t.at(n)->at(size_t(i)));
+        std::vector<float> conv;   // [taps][channels]
+        for (int j = 0; j < d.taps; ++j)
+            for (const char* n : {"mix.q.conv", "mix.k.conv", "mix.v.conv"})
+                for (int64_t c = 0; c < t.at(n)->shape[0]; ++c) conv.push_back(t.at(n)->at(size_t(c * d.taps + j)));
         FORGE_TRY(upload_values(m, &w->conv, conv));
         // a decay's logarithm is -exp(A_log of the head) softplus(its row's value + dt_bias)
         const int per = d.channel ? d.dim : 1;
