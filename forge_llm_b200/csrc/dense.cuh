@@ -69,7 +69,7 @@ constexpr size_t kDensePartFloats = size_t(148) * 2 * 256 * 128;
 
 inline size_t dense_tile_bytes(int N, int K) { return size_t((N + 127) / 128) * 128 * K * 2; }
 void dense_tile_image(void* dst, const void* rows, int N, int K);
-// act: [m][w.K] of the model's type (rows w.K apart unless act_ld says otherwise).  max_rows: rows the buffer holds.
+// act: [m][w.K] of the model's type, rows act_ld values apart.
 int32_t dense_gemm(const DenseWeight& w, const void* act, int act_ld, int m, const DenseOut& out, const DenseScratch& sc, int* err, cudaStream_t st);
 
 // Rows of a step and where their sequence lives.  Row r belongs to sequence seq[r] (null: sequence r) at position pos[r].

@@ -649,7 +649,7 @@ void stack_destroy(ForgeModel* m) {
 }
 
 // ------------------------------------------------------------------------------------------------ cache
-static size_t state_bytes(const StackModel& S, const LayerSpec& L) { return L.has_state() ? L.rec.state_values() * 4 : 0; }
+static size_t state_bytes(const LayerSpec& L) { return L.has_state() ? L.rec.state_values() * 4 : 0; }
 static size_t ring_bytes(const StackModel& S, const LayerSpec& L) { return L.has_state() ? L.rec.ring_values() * dense_size(S.dtype) : 0; }
 static size_t prev_bytes(const StackModel& S, const LayerSpec& L) { return L.kind == Mixer::AttnTimeMix ? size_t(S.spec.width) * dense_size(S.dtype) : 0; }
 
@@ -675,7 +675,7 @@ int32_t stack_cache_create(ForgeKV* kv) {
         FORGE_TRY(alloc(&pool, rows * L.cache_row() * dense_size(S.dtype)));
         r.pool = pool;
         if (L.has_latent() && tensor_core_rows(S, L.mix)) FORGE_TRY(latent_cache_map(r.map, r.pool, L.mix, rows));
-        FORGE_TRY(alloc(&r.state, slots * state_bytes(S, L)));
+        FORGE_TRY(alloc(&r.state, slots * state_bytes(L)));
         FORGE_TRY(alloc(&ring, slots * ring_bytes(S, L)));
         r.ring = ring;
         FORGE_TRY(alloc(&prev, slots * prev_bytes(S, L)));
@@ -734,7 +734,7 @@ int32_t stack_kv_read(ForgeKV* kv, int seq, int run, int which, float* out_host)
 
 size_t stack_state_values(const ForgeKV* kv, int run) {
     const StackModel& S = *kv->model->stack;
-    return state_bytes(S, S.spec.layers[S.spec.runs[run].layer]) / 4;
+    return state_bytes(S.spec.layers[S.spec.runs[run].layer]) / 4;
 }
 int32_t stack_state_read(ForgeKV* kv, int seq, int run, float* out_host) {
     const size_t n = stack_state_values(kv, run);
@@ -754,7 +754,7 @@ size_t stack_kv_bytes_per_token(const ForgeKV* kv) {
 size_t stack_kv_bytes_per_seq(const ForgeKV* kv) {
     const StackModel& S = *kv->model->stack;
     size_t n = 0;
-    for (const LayerRun& r : S.spec.runs) { const LayerSpec& L = S.spec.layers[r.layer]; n += state_bytes(S, L) + ring_bytes(S, L) + prev_bytes(S, L); }
+    for (const LayerRun& r : S.spec.runs) { const LayerSpec& L = S.spec.layers[r.layer]; n += state_bytes(L) + ring_bytes(S, L) + prev_bytes(S, L); }
     return n;
 }
 
@@ -775,7 +775,7 @@ int32_t stack_kv_copy(ForgeKV* kv, int seq, int len, char* host, bool to_host) {
             const int pg = kv->h_page_table[size_t(seq) * kv->pages_per_seq + t0 / FORGE_KV_PAGE];
             FORGE_TRY(copy(static_cast<char*>(r.pool) + size_t(pg) * FORGE_KV_PAGE * row, row * std::min(FORGE_KV_PAGE, len - t0)));
         }
-        FORGE_TRY(copy(reinterpret_cast<char*>(r.state) + size_t(seq) * state_bytes(S, L), state_bytes(S, L)));
+        FORGE_TRY(copy(reinterpret_cast<char*>(r.state) + size_t(seq) * state_bytes(L), state_bytes(L)));
         FORGE_TRY(copy(static_cast<char*>(r.ring) + size_t(seq) * ring_bytes(S, L), ring_bytes(S, L)));
         FORGE_TRY(copy(static_cast<char*>(r.prev) + size_t(seq) * prev_bytes(S, L), prev_bytes(S, L)));
     }
