@@ -4,6 +4,9 @@ one function per mechanism, numpy, written from the equations, slow on purpose.
 Bolenex: latent attention and a clamped gated feed-forward in parallel behind one Dynamic Tanh norm.
 Robazen: mixer and feed-forward one after the other, each behind its own Dynamic Tanh norm; mixers are gated delta rules (one
 decay per head or per key channel) and a pair of chunked attention and time mixing; some layers run several times.
+Mokatar: mixer and feed-forward side by side, each behind its own RMS norm of the same stream; mixers are softmax attentions with
+normed and rotated queries and keys (a window with kept first tokens and a learned sink per head, or the whole past and a sink of
+score zero) and gated linear attention; feed-forwards may be mixtures of experts; bigram embeddings; some layers run several times.
 
 TEST INFRASTRUCTURE ONLY, like the rest of this folder; it shares no code with the shipped package.  Everything is computed in
 ``dtype`` (float64 by default).  A sequence is evaluated as a whole: there is no cache, no page and no batch here.
@@ -233,9 +236,127 @@ def silu_glu_ff(h, w):
     return (silu(h @ w("gate").T) * (h @ w("up").T)) @ w("down").T
 
 
+# ------------------------------------------------------------------- softmax attention with normed, rotated queries and keys
+def rotation(rot, kind):
+    """(angle per position of every pair, factor on cos and sin) of a rotation; kind: what "scaling" asks for."""
+    d, base = rot["dims"], float(rot["base"])
+    f = np.array([base ** (-2.0 * i / d) for i in range(d // 2)])
+    s = rot.get("scaling")
+    if not s:
+        return f, 1.0
+    if kind == "linear":
+        return f / s["factor"], 1.0
+    turns = lambda t: d * math.log(s["original"] / (2 * math.pi * t)) / (2 * math.log(base))   # the pair that turns t times over the original length
+    lo, hi = max(math.floor(turns(s["fast"])), 0), min(math.ceil(turns(s["slow"])), d - 1)
+    ramp = np.clip((np.arange(d // 2) - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return f / s["factor"] * ramp + f * (1 - ramp), 0.1 * math.log(s["factor"]) + 1.0
+
+
+def rotate(x, positions, freq, factor, interleaved):
+    """x: [tokens, heads, n]; pair i is (2i, 2i + 1) if interleaved, else (i, i + number of pairs); the rest passes."""
+    n = len(freq)
+    a, b = (np.arange(n) * 2, np.arange(n) * 2 + 1) if interleaved else (np.arange(n), np.arange(n) + n)
+    ang = np.asarray(positions, np.float64)[:, None, None] * freq
+    c, s = (np.cos(ang) * factor).astype(x.dtype), (np.sin(ang) * factor).astype(x.dtype)
+    out = x.copy()
+    out[:, :, a] = x[:, :, a] * c - x[:, :, b] * s
+    out[:, :, b] = x[:, :, b] * c + x[:, :, a] * s
+    return out
+
+
+def visible(i, size=None, keep=0):
+    """Which keys j = 0 .. i position i sees: its window of ``size`` positions and the first ``keep``."""
+    j = np.arange(i + 1)
+    return np.ones(i + 1, bool) if size is None else (i - j < size) | (j < keep)
+
+
+def sink_attention(q, k, v, scale, sink, size=None, keep=0):
+    """q: [tokens, heads, d], k: [tokens, kv heads, d], v: [tokens, kv heads, dv]; the denominator holds exp(sink[head]) besides the keys'."""
+    n, H, _ = q.shape
+    G = k.shape[1]
+    out = np.zeros((n, H, v.shape[2]), q.dtype)
+    for h in range(H):
+        kh, vh = k[:, h // (H // G)], v[:, h // (H // G)]
+        s = (q[:, h] @ kh.T) * q.dtype.type(scale)
+        for i in range(n):
+            see = visible(i, size, keep)
+            row = s[i, :i + 1][see]
+            top = max(row.max(), sink[h])
+            e = np.exp(row - top)
+            out[i, h] = (e / (e.sum() + np.exp(sink[h] - top))) @ vh[:i + 1][see]
+    return out
+
+
+def head_normed_attention(h, w, m, eps):
+    """Queries and keys normed per head, interleaved rotation, a window with kept first tokens, a learned sink."""
+    n, H, G, pos = h.shape[0], m["heads"], m["kv_heads"], np.arange(h.shape[0])
+    f, c = rotation(m["rot"], "yarn")
+    q = rotate(rms_norm((h @ w("q").T).reshape(n, H, m["dim"]), w("q.norm"), eps), pos, f, c, True)
+    k = rotate(rms_norm((h @ w("k").T).reshape(n, G, m["dim"]), w("k.norm"), eps), pos, f, c, True)
+    v = (h @ w("v").T).reshape(n, G, m["vdim"])
+    mask = m.get("mask") or {}
+    return sink_attention(q, k, v, m["scale"], w("sink"), mask.get("size"), mask.get("keep_first", 0)).reshape(n, H * m["vdim"]) @ w("o").T
+
+
+def row_normed_attention(h, w, m, eps):
+    """Biased projections, queries and keys normed over all heads at once, halves rotated, a sink of score zero."""
+    n, H, G, pos = h.shape[0], m["heads"], m["kv_heads"], np.arange(h.shape[0])
+    f, c = rotation(m["rot"], "linear")
+    q = rotate(rms_norm(h @ w("q").T + w("q.b"), w("q.norm"), eps).reshape(n, H, m["dim"]), pos, f, c, False)
+    k = rotate(rms_norm(h @ w("k").T + w("k.b"), w("k.norm"), eps).reshape(n, G, m["dim"]), pos, f, c, False)
+    v = (h @ w("v").T + w("v.b")).reshape(n, G, m["vdim"])
+    return sink_attention(q, k, v, m["scale"], np.zeros(H, h.dtype)).reshape(n, H * m["vdim"]) @ w("o").T
+
+
+def linear_attention_states(h, w, m):
+    """What is read, [tokens, heads, dv], and the last states [heads, d, dv]: a key channel decays, a token is written, then read."""
+    n, H, d, dv = h.shape[0], m["heads"], m["dim"], m["vdim"]
+    q, k, v = (h @ w("q").T).reshape(n, H, d) * d ** -0.5, (h @ w("k").T).reshape(n, H, d), (h @ w("v").T).reshape(n, H, dv)
+    z = ((h @ w("a1").T) @ w("a2").T + w("a2.b")).reshape(n, H, d)
+    alpha = sigmoid(z) ** (1.0 / m["tau"])
+    o, last = np.zeros_like(v), []
+    for i in range(H):
+        S = np.zeros((d, dv), h.dtype)
+        for t in range(n):
+            S = alpha[t, i][:, None] * S + np.outer(k[t, i], v[t, i])
+            o[t, i] = S.T @ q[t, i]
+        last.append(S)
+    return o, np.stack(last)
+
+
+def gated_linear_attention(h, w, m, eps):
+    o, _ = linear_attention_states(h, w, m)
+    n, H, dv = o.shape
+    return (rms_norm(o, w("norm"), eps).reshape(n, H * dv) * silu(h @ w("g").T)) @ w("o").T
+
+
+def route(z, top):
+    """z: [tokens, experts] -> chosen experts [tokens, top], largest first, and their softmax weights."""
+    chosen = np.argsort(-z, axis=1, kind="stable")[:, :top]
+    e = np.take_along_axis(z, chosen, 1)
+    e = np.exp(e - e.max(1, keepdims=True))
+    return chosen, e / e.sum(1, keepdims=True)
+
+
+def mixture_ff(h, w, m):
+    chosen, weight = route(h @ w("router").T + w("router.b"), m["router"]["top"])
+    out = np.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, g in zip(chosen[t], weight[t]):
+            out[t] += g * silu_glu_ff(h[t:t + 1], lambda n: w(f"e{e}.{n}"))[0]
+    return out
+
+
+def bigram_rows(tokens, b):
+    """Row of the bigram table for every token; the last row for the first token."""
+    return [b["buckets"] if i == 0 else (int(tokens[i - 1]) * b["mul_prev"] + int(t) * b["mul_cur"]) % b["buckets"] for i, t in enumerate(tokens)]
+
+
 def mixer_of(kind, h, w, m, eps):
     if kind == "latent_attention":
         return latent_attention(h, w, m, eps)
+    if kind in ("attention", "attention_2", "gla"):
+        return {"attention": head_normed_attention, "attention_2": row_normed_attention, "gla": gated_linear_attention}[kind](h, w, m, eps)
     return {"delta": gated_delta, "channel_delta": channel_delta, "parallel": parallel_pair}[kind](h, w, m, eps)
 
 
@@ -257,8 +378,11 @@ class LayerStack:
         self.cfg = config
         self.t = {k: np.asarray(v, dtype) for k, v in tensors.items()}
         self.dtype = dtype
+        self.side_by_side = config["architecture"] == "Mokatar"
 
     def norm(self, x, name):
+        if self.side_by_side:
+            return rms_norm(x, 1.0 + self.t[name], self.cfg["norm"]["eps"])
         return dynamic_tanh(x, self.t[name + ".alpha"], self.t[name], self.t[name + ".b"])
 
     def layer(self, x, i):
@@ -267,6 +391,11 @@ class LayerStack:
         mix, mlp = (lambda n: self.t[p + "mix." + n]), (lambda n: self.t[p + "mlp." + n])
         h = self.norm(x, p + "norm1")
         y = mixer_of(L["type"], h, mix, L["mixer"], self.cfg["norm"]["eps"])
+        if self.side_by_side:
+            if L.get("mlp"):
+                h = self.norm(x, p + "norm2")
+                y = y + (mixture_ff(h, mlp, L["mlp"]) if L["mlp"]["kind"] == "moe" else silu_glu_ff(h, mlp))
+            return x + y
         if self.cfg["architecture"] == "Bolenex":
             if L.get("mlp"):
                 y = y + dense_ff(h, mlp, L["mlp"])
@@ -276,10 +405,15 @@ class LayerStack:
 
     def residuals(self, tokens):
         """The residual stream after every layer run: [runs, tokens, width]."""
-        x0 = x = self.t["embed"][np.asarray(tokens, np.int64)]
+        x = self.t["embed"][np.asarray(tokens, np.int64)]
+        if self.side_by_side:
+            x = x * self.dtype(self.cfg["embedding"]["scale"]) + self.t["bigram"][bigram_rows(tokens, self.cfg["embedding"]["bigram"])]
+        x0 = x
         out = []
         for i, start in layer_runs(self.cfg):
-            if start is not None:
+            if start is not None and self.side_by_side:
+                x = (x + x0 if start else x) + self.t["loop.step"][start]
+            elif start is not None:
                 x = np.concatenate([x, x0], axis=1) @ self.t["loop.in"].T + self.t["loop.step"][start]
             x = self.layer(x, i)
             out.append(x)
@@ -287,7 +421,7 @@ class LayerStack:
 
     def logits(self, tokens):
         """[tokens, vocab]: the logits behind every position."""
-        return self.norm(self.residuals(tokens)[-1], "final.norm") @ self.t["head"].T
+        return self.norm(self.residuals(tokens)[-1], "final.norm") @ self.t["head"].T * self.cfg.get("logit_scale", 1.0)
 
     def generate_greedy(self, prompt, n_new):
         """The next n_new tokens, the last index winning a tie."""
