@@ -3,7 +3,7 @@
 // lazy running maximum, probabilities back into tensor memory as the operand of O += P V, three overlapped stages - with these
 // differences: the query / key width (a part per head plus, optionally, a part whose keys all heads share) and the value width
 // are independent run-time sizes, several query heads may share a key head, the scores may be capped and the keys limited to the
-// query's chunk, several sequences' tiles run in one launch (a table gives each tile's rows, position and context), and the
+// query's chunk or window (with the first tokens kept: their key tiles come first), a sink may stand in the denominator, several sequences' tiles run in one launch (a table gives each tile's rows, position and context), and the
 // epilogue applies an output gate per value or per head.
 // Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = softmax, rescale, store.
 // Tensor memory: S [0, 64), P0 [64, 96), P1 [96, 128), O from 128.
@@ -51,8 +51,11 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = blockIdx.x;
     const PromptTile t = p.a.tiles[blockIdx.y];
-    const int jb = (d.chunk > 0 ? t.pos0 / d.chunk * d.chunk : 0) / BN;   // the first key tile anybody sees
-    const int nblk = (t.pos0 + t.rows - 1) / BN + 1 - jb;
+    auto first_key = [&](int pos) { return d.chunk > 0 ? pos / d.chunk * d.chunk : d.window > 0 && pos >= d.window ? pos - d.window + 1 : 0; };
+    // key tiles: `head` tiles of kept first tokens, then from the first one that anybody's chunk or window reaches
+    const int jb = first_key(t.pos0) / BN, head = d.window > 0 ? min(jb, (d.keep + BN - 1) / BN) : 0;
+    const int nblk = head + (t.pos0 + t.rows - 1) / BN + 1 - jb;
+    auto key_tile = [&](int j) { return j < head ? j : jb + j - head; };
 
     if (tid == 0) {
         mbar_init(&q_full, 1);
@@ -76,7 +79,7 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
             for (int j = 0; j < nblk; ++j) {
                 const int s = j % KVS, use = j / KVS;
                 if (use > 0 && !mbar_wait(&kv_empty[s], (use - 1) & 1, &s_err)) { atomicExch(&s_err, 1); break; }
-                const int row = p.a.pages ? p.a.pages[t.ctx0 / BN + jb + j] * BN : t.ctx0 + (jb + j) * BN, hk = h / d.share;
+                const int row = p.a.pages ? p.a.pages[t.ctx0 / BN + key_tile(j)] * BN : t.ctx0 + key_tile(j) * BN, hk = h / d.share;
                 unsigned char* dst = sKV + size_t(s) * stage_bytes;
                 mbar_expect_tx(&kv_full[s], uint32_t(stage_bytes));
                 for (int c = 0; c < kch; ++c) tma_3d(dst + c * KV_CHUNK, &map_k, c * 64, hk, row, &kv_full[s]);
@@ -121,15 +124,15 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
     } else {
         const int quad = warp & 3;
         const int r = quad * 32 + lane;
-        const int pq = t.pos0 + r, lo = d.chunk > 0 ? pq / d.chunk * d.chunk : 0;
-        const int lo_last = d.chunk > 0 ? (t.pos0 + t.rows - 1) / d.chunk * d.chunk : 0;   // of the tile's last row
+        const int pq = t.pos0 + r, lo = first_key(pq), keep = d.window > 0 ? d.keep : 0;
+        const int lo_last = first_key(t.pos0 + t.rows - 1);   // of the tile's last row
         const float scale2 = d.softcap > 0.f ? d.softcap * 1.4426950408889634f : p.scale2, cap2 = d.softcap > 0.f ? 2.f * p.scale2 / d.softcap : 0.f;
         const uint32_t lane_addr = tmem + (uint32_t(quad * 32) << 16);
         const uint32_t masked = scale2 < 0.f ? 0x7f800000u : 0xff800000u;   // -inf behind the scale
         float m_ref = -INFINITY, l_run = 0.f;
         bool ok = true;
         for (int j = 0; j < nblk; ++j) {
-            const int t0 = (jb + j) * BN;
+            const int t0 = key_tile(j) * BN;
             if (ok && !mbar_wait(&s_full, j & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
             fence_after();
             uint32_t sv[2][32];
@@ -143,10 +146,10 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
 #pragma unroll
                 for (int c = 0; c < 64; ++c) sv[c >> 5][c & 31] = __float_as_uint(1.f - __fdividef(2.f, 1.f + ex2(fminf(__uint_as_float(sv[c >> 5][c & 31]) * cap2, 120.f))));
             }
-            if (t0 + BN - 1 > t.pos0 || t0 < lo_last) {
+            if (t0 + BN - 1 > t.pos0 || (t0 < lo_last && t0 + BN > keep)) {
 #pragma unroll
                 for (int c = 0; c < 64; ++c)
-                    if (t0 + c > pq || t0 + c < lo) sv[c >> 5][c & 31] = masked;
+                    if (t0 + c > pq || (t0 + c < lo && t0 + c >= keep)) sv[c >> 5][c & 31] = masked;
             }
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -189,7 +192,11 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
         if (ok && !mbar_wait(&pv_done[(nblk - 1) & 1], ((nblk - 1) >> 1) & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
         fence_after();
         const bool per_value = p.a.gate != nullptr;
-        const float head_gate = per_value || r >= t.rows ? 1.f : p.a.head_gate[size_t(t.row0 + r) * d.heads + h];
+        if (p.a.sink) {
+            const float own = p.a.sink[h] * 1.4426950408889634f;
+            l_run += m_ref == -INFINITY ? 1.f : ex2(own - m_ref);
+        }
+        const float head_gate = per_value || r >= t.rows || !p.a.head_gate ? 1.f : p.a.head_gate[size_t(t.row0 + r) * d.heads + h];
         const float inv = l_run > 0.f ? head_gate / l_run : 0.f;
         const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(p.a.gate) + size_t(t.row0 + r) * p.a.gate_ld + h * d.vdim;
         __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.a.out) + size_t(t.row0 + r) * p.a.out_ld + h * d.vdim;

@@ -11,18 +11,19 @@ struct PromptDims {
     int dim = 0, rot = 0, vdim = 0;           // query / key part of the head, part whose keys all heads share, values
     int dim_p = 0, rot_p = 0, vdim_p = 0;     // padded to 64
     float scale = 1.f, softcap = 0.f;
-    int chunk = 0;
+    int chunk = 0, window = 0, keep = 0;      // as in AttnDims
     PromptDims() = default;
     explicit PromptDims(const LatentDims& d) : heads(d.heads), dim(d.dim), rot(d.rot), vdim(d.vdim), dim_p(d.dim_p), rot_p(d.rot_p), vdim_p(d.vdim_p), scale(d.scale) {}
     explicit PromptDims(const AttnDims& d)
-        : heads(d.heads), share(d.heads / d.groups), dim(d.dim), vdim(d.vdim), dim_p(d.dim_p), vdim_p(d.vdim_p), scale(d.scale), softcap(d.softcap), chunk(d.chunk) {}
+        : heads(d.heads), share(d.heads / d.groups), dim(d.dim), vdim(d.vdim), dim_p(d.dim_p), vdim_p(d.vdim_p), scale(d.scale), softcap(d.softcap), chunk(d.chunk), window(d.window), keep(d.keep) {}
 };
 struct PromptTile { int32_t row0, rows, pos0, ctx0; };   // query rows of the step, position of the first, first context row of its sequence
 struct PromptAttnArgs {
     // [q_rows][heads][dim_p + rot_p], [ctx][heads / share][dim_p], [ctx][rot_p], [ctx][heads / share][vdim_p]
     const void* q = nullptr; const void* k = nullptr; const void* krot = nullptr; const void* v = nullptr;
     const void* gate = nullptr; int gate_ld = 0;      // out[row][head * vdim + i] = gate * attention: bf16 per value,
-    const float* head_gate = nullptr;                 // or, without gate, f32 per head
+    const float* head_gate = nullptr;                 // or, without gate, f32 per head, or none
+    const float* sink = nullptr;                      // score per head that enters the denominator
     void* out = nullptr; int out_ld = 0;
     int q_rows = 0, ctx_rows = 0;
     const PromptTile* tiles = nullptr; int n_tiles = 0;   // device

@@ -174,18 +174,52 @@ __global__ void embed_rows_kernel(const EmbedArgs a) {
         if (a.hist) a.hist[size_t(*a.step) * gridDim.x + r] = a.tokens[r];
         if (a.place) a.place[r] = int32_t(cache_row(a.rows, r, a.rows.pos[r]));
     }
-    const T* src = static_cast<const T*>(a.table) + size_t(a.tokens[r]) * a.width;
-    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < a.width_p; i += gridDim.y * blockDim.x) {
-        const float v = i < a.width ? to_f(src[i]) : 0.f;
-        if (i < a.width) a.x[size_t(r) * a.width + i] = v;
-        static_cast<T*>(a.after.dst)[size_t(r) * a.after.ld + i] =
-            to_t<T>(i >= a.width ? 0.f : a.after.kind == AFTER_DYT ? dynamic_tanh(v, a.after.alpha, a.after.w[i], a.after.b[i]) : v);
+    const uint32_t tok = a.tokens[r];
+    const T* src = static_cast<const T*>(a.table) + size_t(tok) * a.width;
+    const T* pair = nullptr;
+    if (a.bigram) {
+        uint32_t row = a.buckets;
+        const int pos = a.rows.pos[r];
+        if (pos > 0) {
+            const bool inside = r > 0 && a.rows.seq && a.rows.seq[r - 1] == a.rows.seq[r];   // a sequence's rows of a step are consecutive
+            const uint32_t before = inside ? a.tokens[r - 1] : a.prev[state_slot(a.rows, r)];
+            row = uint32_t((uint64_t(before) * a.mul_prev + uint64_t(tok) * a.mul_cur) % a.buckets);
+        }
+        pair = static_cast<const T*>(a.bigram) + size_t(row) * a.width;
+    }
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < a.width_p; i += gridDim.y * blockDim.x) {   // width_p is a multiple of 64: whole warps
+        const bool ok = i < a.width;
+        float v = ok ? to_f(src[i]) * a.scale : 0.f;
+        if (pair && ok) v += to_f(pair[i]);
+        if (ok && a.x0_f32) a.x0_f32[size_t(r) * a.width + i] = v;
         if (a.x0) static_cast<T*>(a.x0)[size_t(r) * a.x0_ld + i] = to_t<T>(v);
+        if (!ok) {
+            static_cast<T*>(a.after.dst)[size_t(r) * a.after.ld + i] = to_t<T>(0.f);
+            if (a.after.w2) static_cast<T*>(a.after.dst)[size_t(r) * a.after.ld + a.after.col2 + i] = to_t<T>(0.f);
+        }
+        v = leave_value<T>(a.after, v, size_t(r), size_t(a.width), i, ok);
+        if (ok) a.x[size_t(r) * a.width + i] = v;
     }
 }
 
-__global__ void gather_act_kernel(uint4* dst, const uint4* src, const int32_t* idx, int ld16) {
-    for (int i = threadIdx.x; i < ld16; i += blockDim.x) dst[size_t(blockIdx.x) * ld16 + i] = src[size_t(idx[blockIdx.x]) * ld16 + i];
+__global__ void keep_tokens_kernel(uint32_t* prev, const uint32_t* tokens, const StepRows rows) {
+    const int r = blockIdx.x * blockDim.x + threadIdx.x;
+    if (r >= rows.n) return;
+    if (!rows.seq || r + 1 == rows.n || rows.seq[r + 1] != rows.seq[r]) prev[state_slot(rows, r)] = tokens[r];
+}
+
+// a warp per row
+__global__ void row_sums_kernel(float* dst, const float* sums, int rows, int parts) {
+    const int r = blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (r >= rows) return;
+    float s = 0.f;
+    for (int i = threadIdx.x & 31; i < parts; i += 32) s += sums[size_t(r) * parts + i];
+    s = warp_sum(s);
+    if ((threadIdx.x & 31) == 0) dst[r] = s;
+}
+
+__global__ void gather_act_kernel(uint4* dst, const uint4* src, const int32_t* idx, int n16, int ld16) {
+    for (int i = threadIdx.x; i < n16; i += blockDim.x) dst[size_t(blockIdx.x) * n16 + i] = src[size_t(idx[blockIdx.x]) * ld16 + i];
 }
 
 __global__ void kv_append_contig_kernel(__half* kc, __half* vc, const float* k, const float* v, size_t n, size_t off) {
@@ -570,23 +604,33 @@ int32_t embed_rows(const EmbedArgs& a, int dtype, cudaStream_t st) {
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
-int32_t gather_act_rows(void* dst, const void* src, const int32_t* idx, int rows, int ld, int dtype, cudaStream_t st) {
+int32_t gather_act_rows(void* dst, const void* src, int src_ld, const int32_t* idx, int rows, int cols, int dtype, cudaStream_t st) {
     if (rows <= 0) return FORGE_OK;
-    gather_act_kernel<<<rows, 128, 0, st>>>(static_cast<uint4*>(dst), static_cast<const uint4*>(src), idx, int(ld * dense_size(dtype) / 16));
+    gather_act_kernel<<<rows, 128, 0, st>>>(static_cast<uint4*>(dst), static_cast<const uint4*>(src), idx, int(cols * dense_size(dtype) / 16), int(src_ld * dense_size(dtype) / 16));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
-// {cos, sin} of p / base^(2 i / dims), angles formed in double
-int32_t rope_half_table(float* table, int n_pos, int dims, double base) {
-    const int half = dims / 2;
-    for (int i = 0; i < half; ++i) {
-        const double f = std::pow(base, -2.0 * i / dims);
+int32_t keep_tokens(uint32_t* prev, const uint32_t* tokens, const StepRows& rows, cudaStream_t st) {
+    if (rows.n <= 0) return FORGE_OK;
+    keep_tokens_kernel<<<(rows.n + 127) / 128, 128, 0, st>>>(prev, tokens, rows);
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+int32_t row_sums(float* dst, const float* sums, int rows, int parts, cudaStream_t st) {
+    if (rows <= 0) return FORGE_OK;
+    row_sums_kernel<<<(rows + 7) / 8, 256, 0, st>>>(dst, sums, rows, parts);
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+// {cos, sin} * factor of p * freq[i], angles formed in double
+int32_t rope_table(float* table, int n_pos, const std::vector<double>& freq, double factor) {
+    const size_t half = freq.size();
+    for (size_t i = 0; i < half; ++i)
         for (int p = 0; p < n_pos; ++p) {
-            const double a = p * f;
-            table[(size_t(p) * half + i) * 2] = float(std::cos(a));
-            table[(size_t(p) * half + i) * 2 + 1] = float(std::sin(a));
+            const double a = p * freq[i];
+            table[(size_t(p) * half + i) * 2] = float(std::cos(a) * factor);
+            table[(size_t(p) * half + i) * 2 + 1] = float(std::sin(a) * factor);
         }
-    }
     return FORGE_OK;
 }
 

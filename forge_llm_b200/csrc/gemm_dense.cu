@@ -15,6 +15,9 @@
 // Accumulators are double buffered in tensor memory: the epilogue of one tile runs under the products of the next.
 // The weight stages of the ring are requested before the dependency wait of a programmatic launch, the activations after.
 //
+// Products in groups (GROUPED) take their tiles of tokens, each with the matrix it meets, from a table in memory; listed products
+// (LISTED) take a fixed run of K steps and then those of the groups that the table names.  Both read the table behind the dependency wait.
+//
 // float32 (gemm_f32_kernel): a tiled product on the CUDA cores in plain f32 fused multiply-adds.
 #include <algorithm>
 #include <cstring>
@@ -48,8 +51,17 @@ struct RowOut {
     const int32_t* place;
     int after;
     T* next; size_t next_ld;
-    float limit, mul, add, alpha, nw, nb;
-    __device__ __forceinline__ float next_value(float x) const { return after == AFTER_DYT ? dynamic_tanh(x, alpha, nw, nb) : x; }
+    T* next2;                // the second norm's
+    float* sums; size_t parts;
+    float* keep; const float* again;
+    float limit, mul, add, alpha, nw, nb, plus;
+    __device__ __forceinline__ float next_value(float x) const { return after == AFTER_DYT ? dynamic_tanh(x, alpha, nw, nb) : after == AFTER_RMS ? x * nw : x; }
+    // a finished value of the stream (token t): the entry of a pass of a loop
+    __device__ __forceinline__ float enter(float x, size_t t) const {
+        if (keep) keep[t * ld] = x;
+        if (again) x += again[t * ld];
+        return x + plus;
+    }
 };
 template <typename T>
 __device__ __forceinline__ RowOut<T> row_out(const DenseOut& o, int row, int first_row) {
@@ -70,13 +82,20 @@ __device__ __forceinline__ RowOut<T> row_out(const DenseOut& o, int row, int fir
     q.t = static_cast<T*>(g.dst) + col;
     q.place = g.place;
     q.limit = g.limit;
+    if (q.kind == SEG_RESID) {
+        q.after = g.after.kind;   // of the whole warp
+        if (q.after == AFTER_RMS) { q.sums = g.after.sums + (first_row - g.row0) / 32; q.parts = size_t(g.after.parts); }
+    }
     if (q.ok) {
         if (g.mul) q.mul = g.mul[r];
         if (g.add) q.add = g.add[r];
         if (q.kind == SEG_RESID) {
-            q.after = g.after.kind;
             if (q.after == AFTER_DYT) { q.alpha = g.after.alpha; q.nw = g.after.w[r]; q.nb = g.after.b[r]; }
+            if (q.after == AFTER_RMS) { q.nw = g.after.w[r]; if (g.after.w2) { q.nb = g.after.w2[r]; q.next2 = static_cast<T*>(g.after.dst) + g.after.col2 + r; } }
             q.next = static_cast<T*>(g.after.dst) + r; q.next_ld = size_t(g.after.ld);
+            if (g.after.plus) q.plus = g.after.plus[r];
+            if (g.after.again) q.again = g.after.again + r;
+            if (g.after.keep) q.keep = g.after.keep + r;
         }
     }
     return q;
@@ -88,30 +107,38 @@ __device__ __forceinline__ int act_col(const DenseOut& o, int row) {
     return c;
 }
 
-// the epilogue of one value; `up`: the value of the next row, used by the even rows of gated pairs; `old`: what dst holds, if it is known
+// the epilogue of one value v; `up`: the value of the next row, used by the even rows of gated pairs, w: what those are multiplied with; `old`: what dst
+// holds, if it is known; returns the stream's new value
 template <typename T>
-__device__ __forceinline__ void put_one(const RowOut<T>& g, float v, float up, size_t t, float old, bool old_known, bool even_row) {
+__device__ __forceinline__ float put_one(const RowOut<T>& g, float v, float up, float w, size_t t, float old, bool old_known, bool even_row) {
     float* f = g.f32 + t * g.ld;
     T* h = g.t + t * g.ld;
     switch (g.kind) {
-        case SEG_CLAMPED_GLU: if (even_row) *h = to_t<T>(clamped_glu(v, up, g.limit)); break;
-        case SEG_SILU_GLU: if (even_row) *h = to_t<T>(silu(v) * up); break;
+        case SEG_CLAMPED_GLU: if (even_row) *h = to_t<T>(clamped_glu(v, up, g.limit) * w); break;
+        case SEG_SILU_GLU: if (even_row) *h = to_t<T>(silu(v) * up * w); break;
         case SEG_CAST: g.t[(g.place ? size_t(g.place[t]) : t) * g.ld] = to_t<T>(v); break;
         case SEG_SIGMOID: *h = to_t<T>(sigmoid(v)); break;
         case SEG_SILU: *h = to_t<T>(silu(v)); break;
         case SEG_TANH: *h = to_t<T>(tanhf(v)); break;
         case SEG_SIGMOID_F32: *f = sigmoid(v); break;
-        case SEG_DECAY: *f = -g.mul * softplus(v + g.add); break;
-        case SEG_EXP_DECAY: *f = -expf(v + g.add); break;
+        case SEG_DECAY: *f = -g.mul * softplus(v); break;
+        case SEG_EXP_DECAY: *f = -expf(v); break;
         case SEG_RESID: {
-            const float x = (g.fresh ? 0.f : old_known ? old : *f) + v + g.add;
+            const float x = g.enter((g.fresh ? 0.f : old_known ? old : *f) + v, t);
             *f = x;
             if (g.after) g.next[t * g.next_ld] = to_t<T>(g.next_value(x));
-            break;
+            if (g.next2) g.next2[t * g.next_ld] = to_t<T>(x * g.nb);
+            return x;
         }
         default: *f = v;
     }
+    return 0.f;
 }
+
+// the sum of squares behind a token's scale
+__device__ __forceinline__ float row_scale(const RowScale& s, float sum) { return s.mul / sqrtf(sum * s.inv_n + s.eps); }
+
+enum Mode { PLAIN = 0, GROUPED, LISTED };
 
 struct GemmParams {
     DenseOut out;
@@ -124,6 +151,13 @@ struct GemmParams {
     int cluster;             // > 0: CTA i takes part i % cluster of the K steps of tile i / cluster, and nothing is dealt out
     float* part; int* tickets;
     int* err;
+    RowScale scale;
+    int pitch, k_off;        // images per row tile, and in front of the first K step
+    // GROUPED: row tiles per group, images from one group to the next, elements of the output from one group to the next
+    GroupTable groups;
+    int row_tiles; uint32_t group_images; long long group_dst;
+    // LISTED: K steps in front of the groups', and of a group
+    int k_fixed, k_group;
 };
 
 // (32-bit: the host checks that units * sharers fits; 64-bit divisions in front of the first load cost microseconds)
@@ -131,12 +165,23 @@ __device__ __forceinline__ uint32_t share_begin(uint32_t units, uint32_t g, uint
 __device__ __forceinline__ int share_of(uint32_t units, uint32_t u, uint32_t sharers) { return int(((u + 1) * sharers - 1) / units); }
 
 // the pieces of work of one CTA, in order: [k0, k0 + n) K steps of `tile`
-struct Work {
+template <int MODE> struct Work {
     int cta, grid, waves, nk, wave = 0;
     uint32_t u, u1;
     int tile, k0, n;
-    __device__ __forceinline__ Work(const GemmParams& p, uint32_t u_begin, uint32_t u_end)
-        : cta(blockIdx.x), grid(gridDim.x), waves(p.waves), nk(p.nk), u(u_begin), u1(u_end) {}
+    // groups: how many the table names (of a listed product the host's bound, until it is read)
+    __device__ __forceinline__ Work(const GemmParams& p, uint32_t u_begin, uint32_t u_end, int groups)
+        : cta(blockIdx.x), grid(gridDim.x), waves(p.waves), nk(p.nk), u(u_begin), u1(u_end) {
+        if (MODE == GROUPED) {   // whole tiles in turn, or one part of one tile
+            const int tiles = groups * p.row_tiles;
+            if (p.cluster > 0) { if (int(u / uint32_t(nk)) >= tiles) u1 = u; waves = 0; }
+            else waves = tiles > cta ? (tiles - cta + grid - 1) / grid : 0;
+        }
+        if (MODE == LISTED) {
+            const uint32_t end = u / uint32_t(nk) * uint32_t(nk) + uint32_t(p.k_fixed + groups * p.k_group);
+            u1 = min(u1, end);
+        }
+    }
     __device__ __forceinline__ bool next() {
         if (wave < waves) { tile = wave++ * grid + cta; k0 = 0; n = nk; return true; }
         if (u >= u1) return false;
@@ -148,6 +193,21 @@ struct Work {
         return true;
     }
 };
+// where a tile's rows, tokens and weights lie
+struct Tile { int row_tile, tok0, cols, group, w0; };
+template <int NT, int MODE> __device__ __forceinline__ Tile tile_at(const GemmParams& p, int tile, int groups) {
+    if constexpr (MODE == GROUPED) {
+        const GroupTile g = p.groups.tiles[tile % groups];
+        return Tile{tile / groups, g.row0, g.rows, g.group, g.w0};
+    }
+    const int tok0 = (tile % p.tt_count) * NT;
+    return Tile{tile / p.tt_count, tok0, min(NT, p.m - tok0), 0, 0};
+}
+template <int MODE> __device__ __forceinline__ int listed_k(const GemmParams& p, int k) {
+    if (MODE != LISTED || k < p.k_fixed) return k;
+    const int a = (k - p.k_fixed) / p.k_group;
+    return k + (p.groups.tiles[a].group - a) * p.k_group;
+}
 
 template <int NT> struct Ring {
     static constexpr int X_BYTES = NT * 128, STAGE = 16384 + X_BYTES;
@@ -156,7 +216,7 @@ template <int NT> struct Ring {
     static constexpr uint32_t COLS = NT <= 16 ? 32 : 2 * NT;   // two accumulators
 };
 
-template <int NT>
+template <int NT, int MODE>
 __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ GemmParams p) {
     constexpr int STAGE = Ring<NT>::STAGE, STAGES = Ring<NT>::STAGES;
     constexpr uint32_t kCols = Ring<NT>::COLS;
@@ -190,30 +250,44 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
     if (warp == 0) {
         if (lane == 0) {
             // two walks over the same pieces: weight stages run up to a whole ring ahead of the dependency wait
-            Work ww(p, u0, u1), wx = ww;
-            int kw = 0, row_tile = 0;
+            int groups = MODE == LISTED ? p.groups.max_tiles : 0;
+            if constexpr (MODE == GROUPED) { pdl_wait(); groups = *p.groups.n; }
+            Work<MODE> ww(p, u0, u1, groups), wx = ww;
+            int kw = 0;
+            size_t image = 0;
             bool more = ww.next();
-            if (more) row_tile = ww.tile / p.tt_count;
+            auto first_image = [&]() {
+                const Tile t = tile_at<NT, MODE>(p, ww.tile, groups);
+                image = size_t(t.row_tile) * p.pitch + size_t(t.group) * p.group_images + p.k_off;
+            };
+            if (more) first_image();
             const unsigned char* const weights = static_cast<const unsigned char*>(p.w);
             auto weight_stage = [&](int s) {   // one contiguous image of 128 rows x 64 columns, already swizzled
                 mbar_expect_tx(&full[s], uint32_t(STAGE));
-                bulk_load(ring + size_t(s) * STAGE, weights + (size_t(row_tile) * p.nk + ww.k0 + kw) * 16384, 16384, &full[s]);
-                if (++kw == ww.n) { kw = 0; more = ww.next(); if (more) row_tile = ww.tile / p.tt_count; }
+                bulk_load(ring + size_t(s) * STAGE, weights + (image + listed_k<MODE>(p, ww.k0 + kw)) * 16384, 16384, &full[s]);
+                if (++kw == ww.n) { kw = 0; more = ww.next(); if (more) first_image(); }
             };
             int ahead = 0;
-            for (; ahead < STAGES && more; ++ahead) weight_stage(ahead);   // constant: may overlap the kernel in front
-            pdl_wait();
+            const int most = MODE == LISTED ? min(STAGES, p.k_fixed - ww.k0) : STAGES;
+            for (; ahead < most && more; ++ahead) weight_stage(ahead);   // constant: may overlap the kernel in front
+            if constexpr (MODE != GROUPED) pdl_wait();
+            if constexpr (MODE == LISTED) {
+                groups = *p.groups.n;
+                wx = Work<MODE>(p, u0, u1, groups);
+                if (more) { Work<MODE> w = wx; more = w.next() && kw < w.n; ww.n = w.n; }
+            }
             int s = 0, i = 0;
             uint32_t phase = 1;   // parity of the round in front of the current one
             bool ok = true;
             while (ok && wx.next()) {
-                const int tok0 = (wx.tile % p.tt_count) * NT, col0 = act_col(p.out, wx.tile / p.tt_count * 128);
+                const Tile t = tile_at<NT, MODE>(p, wx.tile, groups);
+                const int tok0 = t.tok0, col0 = act_col(p.out, t.row_tile * 128);
                 for (int k = 0; k < wx.n; ++k, ++i) {
                     if (i >= ahead) {
                         if (!mbar_wait(&empty[s], phase, &s_err)) { atomicExch(&s_err, 1); ok = false; break; }
                         weight_stage(s);
                     }
-                    tma_2d(ring + size_t(s) * STAGE + 16384, &map_x, col0 + (wx.k0 + k) * BK, tok0, &full[s]);
+                    tma_2d(ring + size_t(s) * STAGE + 16384, &map_x, col0 + listed_k<MODE>(p, wx.k0 + k) * BK, tok0, &full[s]);
                     if (++s == STAGES) { s = 0; phase ^= 1; }
                 }
             }
@@ -228,8 +302,9 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
             int s = 0;
             uint32_t phase = 0;
             bool ok = true;
-            int seg = 0;
-            for (Work w(p, u0, u1); ok && w.next(); ++seg) {
+            int seg = 0, groups = 0;
+            if constexpr (MODE != PLAIN) { pdl_wait(); groups = *p.groups.n; }
+            for (Work<MODE> w(p, u0, u1, groups); ok && w.next(); ++seg) {
                 const int n = w.n, buf = seg & 1;
                 if (seg >= 2 && !mbar_wait(&acc_empty[buf], ((seg >> 1) - 1) & 1, &s_err)) { ok = false; break; }
                 fence_after();
@@ -259,24 +334,55 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
         const uint32_t lane_addr = tmem + (uint32_t(quad * 32) << 16);
         constexpr int CH = NT < 32 ? NT : 32;   // columns per read
         int seg_i = 0;
-        for (Work w(p, u0, u1); w.next(); ++seg_i) {
+        const int groups = MODE != PLAIN ? *p.groups.n : 0;
+        Work<MODE> w(p, u0, u1, groups);
+        // a CTA of a cluster takes part in finishing its tile even if the list left it no steps
+        bool none = false;
+        auto next = [&]() {
+            if (w.next()) return true;
+            if (MODE != LISTED || p.cluster <= 1 || seg_i > 0) return false;
+            none = true;
+            w.tile = int(u0 / uint32_t(p.nk)); w.n = 0;
+            return true;
+        };
+        for (; next(); ++seg_i) {
             const int tile = w.tile, n = w.n, buf = seg_i & 1;
             const uint32_t t_begin = uint32_t((tile - p.waves * int(gridDim.x)) * p.nk), t_end = t_begin + uint32_t(p.nk);   // among the dealt-out steps
-            const int row0 = (tile / p.tt_count) * 128 + quad * 32, tok0 = (tile % p.tt_count) * NT;
+            const Tile at_tile = tile_at<NT, MODE>(p, tile, groups);
+            const int row0 = at_tile.row_tile * 128 + quad * 32, tok0 = at_tile.tok0, cols = at_tile.cols;
             const int row = row0 + lane;
-            const int cols = min(NT, p.m - tok0);
             // every warp's rows lie in one segment (segments start at multiples of 32 rows)
-            const RowOut<__nv_bfloat16> g = row_out<__nv_bfloat16>(p.out, row, row0);
+            RowOut<__nv_bfloat16> g = row_out<__nv_bfloat16>(p.out, row, row0);
+            if constexpr (MODE == GROUPED) { g.t += at_tile.group * p.group_dst; g.f32 += at_tile.group * p.group_dst; }
+            // scales of the tokens, lane c: of column c (few tokens: all of the tile's)
+            float col_scale = 1.f;
+            auto scale_row = [&](int t) { return size_t(p.scale.row ? p.scale.row[t] : t); };
+            if (NT <= 32 && p.scale.sums)
+                for (int c = 0; c < cols; ++c) {
+                    const float* src = p.scale.sums + scale_row(tok0 + c) * p.scale.parts;
+                    float sum = 0.f;
+                    for (int i = lane; i < p.scale.parts; i += 32) sum += src[i];
+                    sum = row_scale(p.scale, warp_sum(sum));
+                    if (lane == c) col_scale = sum;
+                }
+            const float* pair_w = MODE == GROUPED && p.groups.weight ? p.groups.weight + at_tile.w0 : nullptr;
             float x_old[CH];   // few tokens: the residual is on its way while the product is formed
             if (NT <= 32 && g.kind == SEG_RESID && g.ok && !g.fresh)
 #pragma unroll
                 for (int c = 0; c < CH; ++c) if (c < cols && (p.cluster <= 1 || (c >> 2) % p.cluster == rank)) x_old[c] = g.f32[size_t(tok0 + c) * g.ld];
             // the four warps meet at the barriers of a shared tile: one whose wait gave up must not leave the loop alone
-            if (!mbar_wait(&acc_full[buf], (seg_i >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
+            if (!(MODE == LISTED && none) && !mbar_wait(&acc_full[buf], (seg_i >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
             fence_after();
-            auto finish = [&](int c0, const float (&v)[CH]) {
+            auto finish = [&](int c0, float (&v)[CH]) {
                 const int n_c = cols - c0;
                 const size_t t0 = size_t(tok0 + c0);
+                if (p.scale.sums) {
+                    if (NT > 32) col_scale = lane < n_c ? row_scale(p.scale, p.scale.sums[scale_row(tok0 + c0 + lane)]) : 1.f;
+#pragma unroll
+                    for (int c = 0; c < CH; ++c) v[c] *= __shfl_sync(0xffffffffu, col_scale, c);
+                }
+#pragma unroll
+                for (int c = 0; c < CH; ++c) v[c] += g.add;
                 auto put_t = [&](auto f) {
                     __nv_bfloat16* dst = g.t + t0 * g.ld;
 #pragma unroll
@@ -289,19 +395,66 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                 };
                 if (n_c == 1) {   // one token: little code
                     const float got = __shfl_xor_sync(0xffffffffu, v[0], 1);
-                    if (g.ok) put_one(g, v[0], got, t0, NT <= 32 ? x_old[0] : 0.f, NT <= 32, !(lane & 1));
+                    float x = 0.f;
+                    if (g.ok) x = put_one(g, v[0], got, pair_w ? pair_w[c0] : 1.f, t0, NT <= 32 ? x_old[0] : 0.f, NT <= 32, !(lane & 1));
+                    if (g.sums) {
+                        x = warp_sum(x * x);
+                        if (lane == 0) g.sums[t0 * g.parts] = x;
+                    }
                 } else if (g.kind == SEG_CLAMPED_GLU || g.kind == SEG_SILU_GLU) {
                     // neighbouring lanes hold gate_j and up_j: the even lane takes the first half of the columns
                     const bool even = !(lane & 1), clamped = g.kind == SEG_CLAMPED_GLU;
-                    __nv_bfloat16* dst = g.t + (t0 + (even ? 0 : CH / 2)) * g.ld;
+                    const int mine = even ? 0 : CH / 2;
+                    __nv_bfloat16* dst = g.t + (t0 + mine) * g.ld;
 #pragma unroll
                     for (int c = 0; c < CH / 2; ++c) {
                         const float got = __shfl_xor_sync(0xffffffffu, even ? v[CH / 2 + c] : v[c], 1);
                         const float ga = even ? v[c] : got, up = even ? got : v[CH / 2 + c];
-                        if (g.ok && (even ? c : CH / 2 + c) < n_c) dst[c * g.ld] = __float2bfloat16_rn(clamped ? clamped_glu(ga, up, g.limit) : silu(ga) * up);
+                        if (g.ok && mine + c < n_c) dst[c * g.ld] = __float2bfloat16_rn((clamped ? clamped_glu(ga, up, g.limit) : silu(ga) * up) * (pair_w ? pair_w[c0 + mine + c] : 1.f));
+                    }
+                } else if (g.kind == SEG_RESID) {
+                    float* dst = g.f32 + t0 * g.ld;
+                    float x[CH];
+#pragma unroll
+                    for (int c = 0; c < CH; ++c) x[c] = !g.ok || g.fresh ? 0.f : NT <= 32 ? x_old[c] : c < n_c ? dst[c * g.ld] : 0.f;   // all loads before the first store
+                    if (g.keep || g.again) {
+#pragma unroll
+                        for (int c = 0; c < CH; ++c) { x[c] += v[c]; if (c < n_c) x[c] = g.enter(x[c], t0 + c); }
+                    } else {
+#pragma unroll
+                        for (int c = 0; c < CH; ++c) x[c] += v[c] + g.plus;
+                    }
+                    if (g.ok) {
+#pragma unroll
+                        for (int c = 0; c < CH; ++c) if (c < n_c) dst[c * g.ld] = x[c];
+                        if (g.after) {
+                            __nv_bfloat16* nx = g.next + t0 * g.next_ld;
+#pragma unroll
+                            for (int c = 0; c < CH; ++c) if (c < n_c) nx[c * g.next_ld] = __float2bfloat16_rn(g.next_value(x[c]));
+                        }
+                        if (g.next2) {
+                            __nv_bfloat16* nx = g.next2 + t0 * g.next_ld;
+#pragma unroll
+                            for (int c = 0; c < CH; ++c) if (c < n_c) nx[c * g.next_ld] = __float2bfloat16_rn(x[c] * g.nb);
+                        }
+                    }
+                    if (g.sums) {   // lane c ends with the sum over the warp's rows of column c's squares
+#pragma unroll
+                        for (int c = 0; c < CH; ++c) x[c] = g.ok ? x[c] * x[c] : 0.f;
+                        if constexpr (CH == 16)
+#pragma unroll
+                            for (int c = 0; c < CH; ++c) x[c] += __shfl_xor_sync(0xffffffffu, x[c], 16);
+#pragma unroll
+                        for (int o = CH / 2; o > 0; o >>= 1)
+#pragma unroll
+                            for (int c = 0; c < o; ++c) {
+                                const bool up = lane & o;
+                                const float send = up ? x[c] : x[c + o], mine = up ? x[c + o] : x[c];
+                                x[c] = mine + __shfl_xor_sync(0xffffffffu, send, o);
+                            }
+                        if (lane < CH && lane < n_c) g.sums[(t0 + lane) * g.parts] = x[0];
                     }
                 } else if (g.ok) switch (g.kind) {
-                    case SEG_F32: put_f([](float x) { return x; }); break;
                     case SEG_CAST:
                         if (g.place) {
 #pragma unroll
@@ -312,21 +465,9 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                     case SEG_SILU: put_t([](float x) { return silu(x); }); break;
                     case SEG_TANH: put_t([](float x) { return tanhf(x); }); break;
                     case SEG_SIGMOID_F32: put_f([](float x) { return sigmoid(x); }); break;
-                    case SEG_DECAY: put_f([&](float x) { return -g.mul * softplus(x + g.add); }); break;
-                    case SEG_EXP_DECAY: put_f([&](float x) { return -expf(x + g.add); }); break;
-                    default: {
-                        float* dst = g.f32 + t0 * g.ld;
-                        float x[CH];
-#pragma unroll
-                        for (int c = 0; c < CH; ++c) x[c] = g.fresh ? 0.f : NT <= 32 ? x_old[c] : c < n_c ? dst[c * g.ld] : 0.f;   // all loads before the first store
-#pragma unroll
-                        for (int c = 0; c < CH; ++c) { x[c] += v[c] + g.add; if (c < n_c) dst[c * g.ld] = x[c]; }
-                        if (g.after) {
-                            __nv_bfloat16* nx = g.next + t0 * g.next_ld;
-#pragma unroll
-                            for (int c = 0; c < CH; ++c) if (c < n_c) nx[c * g.next_ld] = __float2bfloat16_rn(g.next_value(x[c]));
-                        }
-                    }
+                    case SEG_DECAY: put_f([&](float x) { return -g.mul * softplus(x); }); break;
+                    case SEG_EXP_DECAY: put_f([&](float x) { return -expf(x); }); break;
+                    default: put_f([](float x) { return x; });
                 }
             };
             auto load = [&](int c0, float (&v)[CH]) {
@@ -337,7 +478,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
 #pragma unroll
                 for (int c = 0; c < CH; ++c) v[c] = __uint_as_float(t[c]);
             };
-            if (n == p.nk) {
+            if (MODE == GROUPED || MODE == LISTED ? p.cluster <= 1 : n == p.nk) {
 #pragma unroll 1
                 for (int c0 = 0; c0 < NT && c0 < cols; c0 += CH) {
                     float v[CH];
@@ -349,7 +490,10 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                 const int at = (quad * 32 + lane) * 4, groups = (cols + 3) / 4, senders = p.cluster - 1;
                 float* box = reinterpret_cast<float*>(ring + size_t(STAGES) * STAGE);
                 float v[CH];
-                load(0, v);
+                if (MODE == LISTED && none) {
+#pragma unroll
+                    for (int c = 0; c < CH; ++c) v[c] = 0.f;
+                } else load(0, v);
                 cluster_wait();
 #pragma unroll
                 for (int c = 0; c < CH / 4; ++c) {
@@ -374,13 +518,21 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                     const int c0 = (rank + k * p.cluster) * 4;
 #pragma unroll 1
                     for (int e = 0; e < min(4, cols - c0); ++e) {
-                        const float got = __shfl_xor_sync(0xffffffffu, t[0], 1);
-                        if (g.ok) put_one(g, t[0], got, size_t(tok0 + c0 + e), old[0], true, !(lane & 1));
+                        float val = t[0];
+                        if (p.scale.sums) val *= __shfl_sync(0xffffffffu, col_scale, c0 + e);
+                        val += g.add;
+                        const float got = __shfl_xor_sync(0xffffffffu, val, 1);
+                        float x = 0.f;
+                        if (g.ok) x = put_one(g, val, got, pair_w ? pair_w[c0 + e] : 1.f, size_t(tok0 + c0 + e), old[0], true, !(lane & 1));
+                        if (g.sums) {
+                            x = warp_sum(x * x);
+                            if (lane == 0) g.sums[size_t(tok0 + c0 + e) * g.parts] = x;
+                        }
                         t[0] = t[1]; t[1] = t[2]; t[2] = t[3];
                         old[0] = old[1]; old[1] = old[2]; old[2] = old[3];
                     }
                 }
-            } else {
+            } else if (MODE == PLAIN) {
                 // a shared tile: this CTA's part goes to its slot (0: the part its share starts with, 1: the other one)
                 float* mine = p.part + (size_t(blockIdx.x) * 2 + (u0 >= t_begin ? 0 : 1)) * (NT * 128);
 #pragma unroll 1
@@ -432,6 +584,11 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
             __syncwarp();
             if (lane == 0) mbar_arrive(&acc_empty[buf]);
         }
+        if (MODE == GROUPED && p.cluster > 1 && seg_i == 0) {   // a tile the table does not name
+            __syncwarp();
+            cluster_wait();
+            cluster_sync();
+        }
         fence_before();
     }
     __syncthreads();
@@ -442,39 +599,55 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
     if (tid == 0 && s_err && p.err) atomicExch(p.err, 1);
 }
 
-template <int NT>
-int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmParams& p, int sms, cudaStream_t st) {
+// most CTAs per tile, clusters of which all run at once (a cluster lies within one group of SMs, so large ones leave SMs idle); 0: too few tiles to fill the SMs
+template <int NT, int MODE>
+int32_t cluster_parts(long long tiles, int nk, size_t smem, int* parts) {
+    static int fits[9] = {0};
+    auto kern = gemm_dense_kernel<NT, MODE>;
+    if (!fits[1])
+        for (int c = 1; c <= 8; ++c) {
+            cudaLaunchConfig_t cfg{};
+            cudaLaunchAttribute at[1];
+            cfg.gridDim = dim3(unsigned(c * 148)); cfg.blockDim = dim3(kThreads); cfg.dynamicSmemBytes = std::max(smem, size_t(120) * 1024);   // one CTA per SM
+            at[0].id = cudaLaunchAttributeClusterDimension;
+            at[0].val.clusterDim.x = unsigned(c); at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
+            cfg.attrs = at; cfg.numAttrs = 1;
+            FORGE_CUDA(cudaOccupancyMaxActiveClusters(&fits[c], kern, &cfg));
+        }
+    *parts = 0;
+    for (int c = 1; c <= 8; ++c)
+        if (tiles <= fits[c] && (c == 1 || (nk >= 2 * c && (c - 1) * ((NT / 4 + c - 1) / c) * 2048 <= Ring<NT>::EXCHANGE))) *parts = c;
+    if (tiles * *parts < 90 && tiles > fits[8] && MODE == PLAIN) *parts = 0;
+    return FORGE_OK;
+}
+
+template <int NT, int MODE>
+int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, int act_rows, GemmParams& p, int sms, cudaStream_t st) {
     CUtensorMap mx;
     int last_col = 0;
     for (int i = 0; i < p.out.nseg; ++i) last_col = std::max(last_col, p.out.seg[i].act_col);
-    FORGE_TRY(make_map_2d(&mx, act, uint64_t(last_col + w.K), uint64_t(p.m), uint64_t(act_ld) * 2, NT));
-    p.tt_count = (p.m + NT - 1) / NT;
-    const long long tiles = (long long)((w.N + 127) / 128) * p.tt_count;
-    auto kern = gemm_dense_kernel<NT>;
+    FORGE_TRY(make_map_2d(&mx, act, uint64_t(last_col + (MODE == LISTED ? w.K : p.nk * BK)), uint64_t(act_rows), uint64_t(act_ld) * 2, NT));
+    p.tt_count = MODE == GROUPED ? 1 : (p.m + NT - 1) / NT;
+    const long long tiles = MODE == GROUPED ? (long long)p.groups.max_tiles * p.row_tiles : (long long)((w.N + 127) / 128) * p.tt_count;   // at most
+    auto kern = gemm_dense_kernel<NT, MODE>;
     const size_t smem = size_t(Ring<NT>::STAGES) * Ring<NT>::STAGE + Ring<NT>::EXCHANGE + 1024;
     FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(std::max(smem, size_t(120) * 1024))));
     if (NT <= 32 && tiles <= sms) {
-        // most parts per tile whose clusters all run at once (a cluster lies within one group of SMs, so large ones leave SMs idle)
-        static int fits[9] = {0};
-        if (!fits[1])
-            for (int c = 1; c <= 8; ++c) {
-                cudaLaunchConfig_t cfg{};
-                cudaLaunchAttribute at[1];
-                cfg.gridDim = dim3(unsigned(c * 148)); cfg.blockDim = dim3(kThreads); cfg.dynamicSmemBytes = std::max(smem, size_t(120) * 1024);   // one CTA per SM
-                at[0].id = cudaLaunchAttributeClusterDimension;
-                at[0].val.clusterDim.x = unsigned(c); at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
-                cfg.attrs = at; cfg.numAttrs = 1;
-                FORGE_CUDA(cudaOccupancyMaxActiveClusters(&fits[c], kern, &cfg));
-            }
         int parts = 0;
-        for (int c = 1; c <= 8; ++c)
-            if (tiles <= fits[c] && (c == 1 || (p.nk >= 2 * c && (c - 1) * ((NT / 4 + c - 1) / c) * 2048 <= Ring<NT>::EXCHANGE))) parts = c;
-        if (tiles * parts >= 90 || tiles <= fits[8]) {
+        FORGE_TRY((cluster_parts<NT, MODE>(tiles, p.nk, smem, &parts)));
+        if (parts > 0) {
             p.cluster = parts;
             FORGE_CUDA(launch_pdl_cluster(kern, dim3(unsigned(tiles * parts)), dim3(kThreads), parts, smem, st, mx, p));
             FORGE_LAUNCH_CHECK();
             return FORGE_OK;
         }
+    }
+    if constexpr (MODE == LISTED) { set_error("listed product: %lld tiles are too many", tiles); return FORGE_ERR_SHAPE; }
+    if constexpr (MODE == GROUPED) {   // sixteen-token tiles: two CTAs fit an SM
+        if (tiles * p.nk > INT32_MAX) { set_error("product in groups: %lld tiles of %d K steps are too many", tiles, p.nk); return FORGE_ERR_SHAPE; }
+        FORGE_CUDA(launch_pdl(kern, dim3(unsigned(std::min((long long)sms * (NT <= 16 ? 2 : 1), tiles))), dim3(kThreads), smem, st, mx, p));
+        FORGE_LAUNCH_CHECK();
+        return FORGE_OK;
     }
     const int grid = int(std::max(1LL, std::min((long long)sms, std::max(NT >= 128 ? tiles : 1, tiles * p.nk / 4))));
     p.waves = NT >= 128 ? int(tiles / grid) : 0;   // a weight stream gains nothing from whole tiles in turn
@@ -491,13 +664,37 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, GemmPara
 }
 
 // ------------------------------------------------------------------------------------------------ float32
-// 64 rows x TM tokens per CTA, K in steps of 16, 256 threads
-template <int TM>
-__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ w, const float* __restrict__ x, int ldx, int K, int m, int N, const DenseOut out) {
+// 64 rows x TM tokens per CTA, K in steps of 16, 256 threads.  Groups: blockIdx.y is a tile of the table, blockIdx.z its part of TM tokens.
+struct F32Groups { GroupTable t; size_t group_w; size_t group_dst; };
+template <int TM, bool GROUPS>
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ w, int ldw, const float* __restrict__ x, int ldx, int K, int m, int N, const DenseOut out, const F32Groups gr) {
     constexpr int TN = 64, KS = 16, PT = TM / 16;   // tokens per thread
-    __shared__ float sw[KS][TN + 4], sx[KS][TM + 4];
+    __shared__ float sw[KS][TN + 4], sx[KS][TM + 4], s_scale[TM];
     const int tid = threadIdx.x, rr = (tid & 15) * 4, tt = (tid >> 4) * PT;
-    const int row0 = blockIdx.x * TN, tok0 = blockIdx.y * TM;
+    const int row0 = blockIdx.x * TN;
+    int tok0 = blockIdx.y * TM;
+    const float* pair_w = nullptr;
+    size_t dst_off = 0;
+    if constexpr (GROUPS) {
+        if (int(blockIdx.y) >= *gr.t.n) return;
+        const GroupTile t = gr.t.tiles[blockIdx.y];
+        if (int(blockIdx.z) * TM >= t.rows) return;
+        tok0 = t.row0 + blockIdx.z * TM;
+        m = t.row0 + t.rows;
+        w += size_t(t.group) * gr.group_w;
+        dst_off = size_t(t.group) * gr.group_dst;
+        if (gr.t.weight) pair_w = gr.t.weight + t.w0 + blockIdx.z * TM;
+    }
+    for (int i = tid; i < TM; i += 256) {
+        float sc = 1.f;
+        if (out.scale.sums && tok0 + i < m) {
+            const float* src = out.scale.sums + size_t(out.scale.row ? out.scale.row[tok0 + i] : tok0 + i) * out.scale.parts;
+            float sum = 0.f;
+            for (int j = 0; j < out.scale.parts; ++j) sum += src[j];
+            sc = row_scale(out.scale, sum);
+        }
+        s_scale[i] = sc;
+    }
     x += act_col(out, row0);
     float acc[4][PT];
 #pragma unroll
@@ -507,7 +704,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
     for (int k0 = 0; k0 < K; k0 += KS) {
         for (int i = tid; i < TN * KS; i += 256) {
             const int r = i / KS, k = i % KS;
-            sw[k][r] = row0 + r < N ? w[size_t(row0 + r) * K + k0 + k] : 0.f;
+            sw[k][r] = row0 + r < N ? w[size_t(row0 + r) * ldw + k0 + k] : 0.f;
         }
         for (int i = tid; i < TM * KS; i += 256) {
             const int t = i / KS, k = i % KS;
@@ -530,17 +727,53 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
     }
     RowOut<float> g[4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) g[i] = row_out<float>(out, row0 + rr + i, row0 + rr);   // four consecutive rows lie in one segment or past its end
+    for (int i = 0; i < 4; ++i) {   // four consecutive rows lie in one segment or past its end
+        g[i] = row_out<float>(out, row0 + rr + i, (row0 + rr) & ~31);
+        g[i].t += dst_off; g[i].f32 += dst_off;
+    }
 #pragma unroll
     for (int j = 0; j < PT; ++j) {
         const size_t t = size_t(tok0 + tt + j);
-        if (int(t) >= m) continue;
+        const bool live = int(t) < m;
+        float v[4], sum = 0.f;
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            if (!g[i].ok) continue;
-            put_one(g[i], acc[i][j], acc[i | 1][j], t, 0.f, false, !(i & 1));
+        for (int i = 0; i < 4; ++i) v[i] = acc[i][j] * s_scale[tt + j] + g[i].add;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            if (live && g[i].ok) {
+                const float xn = put_one(g[i], v[i], v[i | 1], pair_w ? pair_w[tt + j] : 1.f, t, 0.f, false, !(i & 1));
+                sum = fmaf(xn, xn, sum);
+            }
+        if (__any_sync(0xffffffffu, g[0].sums != nullptr)) {   // over the 32 rows of eight neighbouring lanes
+            sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+            sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+            sum += __shfl_xor_sync(0xffffffffu, sum, 4);
+            if (live && g[0].sums && !(tid & 7)) g[0].sums[t * g[0].parts] = sum;
         }
     }
+}
+
+int32_t check_out(const DenseWeight& w, int rows, int act_ld, const DenseOut& out) {
+    for (int i = 0; i < out.nseg; ++i) {
+        const OutSeg& g = out.seg[i];
+        const bool glu = g.kind == SEG_CLAMPED_GLU || g.kind == SEG_SILU_GLU, moved = g.act_col != (i ? out.seg[i - 1].act_col : 0);
+        if (g.row0 % kSegAlign || g.row0 + g.rows > rows || (glu && (g.rows % 2 || g.add)) || (i && g.row0 < out.seg[i - 1].row0 + out.seg[i - 1].rows) ||
+            g.act_col % kDensePad || g.act_col + w.K > act_ld || (i && moved && g.row0 % 128)) {
+            set_error("dense product: bad output segment %d", i);
+            return FORGE_ERR_SHAPE;
+        }
+    }
+    return FORGE_OK;
+}
+int32_t check_weight(const DenseWeight& w, int act_ld) {
+    if (w.K % kDensePad || act_ld < w.K || act_ld % kDensePad || w.pitch() % kDensePad || w.col0 % kDensePad || w.col0 + w.K > w.pitch()) { set_error("dense product: K=%d, activation rows of %d", w.K, act_ld); return FORGE_ERR_SHAPE; }
+    return FORGE_OK;
+}
+int sm_count() {
+    int dev = 0, sms = 148;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    return std::min(sms, 148);
 }
 
 }  // namespace
@@ -561,39 +794,78 @@ void dense_tile_image(void* dst, const void* rows, int N, int K) {
 
 int32_t dense_gemm(const DenseWeight& w, const void* act, int act_ld, int m, const DenseOut& out, const DenseScratch& sc, int* err, cudaStream_t st) {
     if (m <= 0) return FORGE_OK;
-    if (w.K % kDensePad || act_ld < w.K || act_ld % kDensePad) { set_error("dense product: K=%d, activation rows of %d", w.K, act_ld); return FORGE_ERR_SHAPE; }
-    for (int i = 0; i < out.nseg; ++i) {
-        const OutSeg& g = out.seg[i];
-        const bool glu = g.kind == SEG_CLAMPED_GLU || g.kind == SEG_SILU_GLU, moved = g.act_col != (i ? out.seg[i - 1].act_col : 0);
-        if (g.row0 % kSegAlign || g.row0 + g.rows > w.N || (glu && g.rows % 2) || (i && g.row0 < out.seg[i - 1].row0 + out.seg[i - 1].rows) ||
-            g.act_col % kDensePad || g.act_col + w.K > act_ld || (i && moved && g.row0 % 128)) {
-            set_error("dense product: bad output segment %d", i);
-            return FORGE_ERR_SHAPE;
-        }
-    }
+    FORGE_TRY(check_weight(w, act_ld));
+    FORGE_TRY(check_out(w, w.N, act_ld, out));
     if (w.dtype == FORGE_F32) {
-        const float* wf = static_cast<const float*>(w.w);
+        const float* wf = static_cast<const float*>(w.w) + w.col0;
         const float* xf = static_cast<const float*>(act);
-        if (m <= 16) gemm_f32_kernel<16><<<dim3((w.N + 63) / 64, 1), 256, 0, st>>>(wf, xf, act_ld, w.K, m, w.N, out);
-        else gemm_f32_kernel<64><<<dim3((w.N + 63) / 64, (m + 63) / 64), 256, 0, st>>>(wf, xf, act_ld, w.K, m, w.N, out);
+        if (m <= 16) gemm_f32_kernel<16, false><<<dim3((w.N + 63) / 64, 1), 256, 0, st>>>(wf, w.pitch(), xf, act_ld, w.K, m, w.N, out, F32Groups{});
+        else gemm_f32_kernel<64, false><<<dim3((w.N + 63) / 64, (m + 63) / 64), 256, 0, st>>>(wf, w.pitch(), xf, act_ld, w.K, m, w.N, out, F32Groups{});
         FORGE_LAUNCH_CHECK();
         return FORGE_OK;
     }
-    int dev = 0, sms = 148;
-    cudaGetDevice(&dev);
-    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-    sms = std::min(sms, 148);
     GemmParams p{};
-    p.out = out; p.w = w.tiles; p.m = m; p.N = w.N; p.nk = w.K / BK; p.part = sc.part; p.tickets = sc.tickets; p.err = err;
-    const int nt = m <= 16 ? 16 : m <= 32 ? 32 : m <= 64 ? 64 : m <= 128 ? 128 : 256;
+    p.out = out; p.scale = out.scale; p.w = w.tiles; p.m = m; p.N = w.N; p.nk = w.K / BK; p.part = sc.part; p.tickets = sc.tickets; p.err = err;
+    p.pitch = w.pitch() / BK; p.k_off = w.col0 / BK;
+    const int sms = sm_count(), nt = group_tile_rows(m);
+    if (out.scale.sums && out.scale.parts > 1 && nt > kScaleRows) { set_error("dense product: %d tokens with scales in parts", m); return FORGE_ERR_SHAPE; }
     if (size_t((w.N + 127) / 128) * ((m + nt - 1) / nt) > sc.tickets_cap) { set_error("dense product: too many tiles for the ticket array"); return FORGE_ERR_SHAPE; }
     switch (nt) {
-        case 16: return launch_dense<16>(w, act, act_ld, p, sms, st);
-        case 32: return launch_dense<32>(w, act, act_ld, p, sms, st);
-        case 64: return launch_dense<64>(w, act, act_ld, p, sms, st);
-        case 128: return launch_dense<128>(w, act, act_ld, p, sms, st);
+        case 16: return launch_dense<16, PLAIN>(w, act, act_ld, m, p, sms, st);
+        case 32: return launch_dense<32, PLAIN>(w, act, act_ld, m, p, sms, st);
+        case 64: return launch_dense<64, PLAIN>(w, act, act_ld, m, p, sms, st);
+        case 128: return launch_dense<128, PLAIN>(w, act, act_ld, m, p, sms, st);
     }
-    return launch_dense<256>(w, act, act_ld, p, sms, st);
+    return launch_dense<256, PLAIN>(w, act, act_ld, m, p, sms, st);
+}
+
+int32_t dense_gemm_groups(const DenseWeight& w, const GroupShape& s, const GroupTable& t, const void* act, int act_ld, int act_rows, const DenseOut& out, int* err, cudaStream_t st) {
+    if (act_rows <= 0 || t.max_tiles <= 0) return FORGE_OK;
+    FORGE_TRY(check_weight(w, act_ld));
+    FORGE_TRY(check_out(w, s.rows, act_ld, out));
+    if (s.group_rows % 128 || s.group_cols % kDensePad) { set_error("product in groups: matrices %d rows and %d columns apart", s.group_rows, s.group_cols); return FORGE_ERR_SHAPE; }
+    if (w.dtype == FORGE_F32) {
+        const F32Groups g{t, size_t(s.group_rows) * w.pitch() + s.group_cols, s.group_dst};
+        const float* wf = static_cast<const float*>(w.w) + w.col0;
+        const float* xf = static_cast<const float*>(act);
+        if (t.tile_rows <= 16) gemm_f32_kernel<16, true><<<dim3((s.rows + 63) / 64, t.max_tiles, 1), 256, 0, st>>>(wf, w.pitch(), xf, act_ld, w.K, 0, s.rows, out, g);
+        else gemm_f32_kernel<64, true><<<dim3((s.rows + 63) / 64, t.max_tiles, (t.tile_rows + 63) / 64), 256, 0, st>>>(wf, w.pitch(), xf, act_ld, w.K, 0, s.rows, out, g);
+        FORGE_LAUNCH_CHECK();
+        return FORGE_OK;
+    }
+    GemmParams p{};
+    p.out = out; p.scale = out.scale; p.w = w.tiles; p.m = act_rows; p.N = s.rows; p.nk = w.K / BK; p.err = err;
+    p.pitch = w.pitch() / BK; p.k_off = w.col0 / BK;
+    p.groups = t; p.row_tiles = (s.rows + 127) / 128; p.group_dst = (long long)s.group_dst;
+    p.group_images = uint32_t(s.group_rows / 128 * p.pitch + s.group_cols / BK);
+    const int sms = sm_count();
+    if (out.scale.sums && out.scale.parts > 1 && t.tile_rows > kScaleRows) { set_error("product in groups: tiles of %d tokens with scales in parts", t.tile_rows); return FORGE_ERR_SHAPE; }
+    switch (t.tile_rows) {
+        case 16: return launch_dense<16, GROUPED>(w, act, act_ld, act_rows, p, sms, st);
+        case 32: return launch_dense<32, GROUPED>(w, act, act_ld, act_rows, p, sms, st);
+        case 64: return launch_dense<64, GROUPED>(w, act, act_ld, act_rows, p, sms, st);
+        case 128: return launch_dense<128, GROUPED>(w, act, act_ld, act_rows, p, sms, st);
+        case 256: return launch_dense<256, GROUPED>(w, act, act_ld, act_rows, p, sms, st);
+    }
+    set_error("product in groups: tiles of %d rows", t.tile_rows);
+    return FORGE_ERR_SHAPE;
+}
+
+bool dense_listed_supported(const DenseWeight& w, int m) { return w.dtype == FORGE_BF16 && m <= kScaleRows && (w.N + 127) / 128 <= 128; }
+
+int32_t dense_gemm_listed(const DenseWeight& w, int k_fixed, int k_group, const GroupTable& t, const void* act, int act_ld, int m, const DenseOut& out, int* err, cudaStream_t st) {
+    if (m <= 0) return FORGE_OK;
+    FORGE_TRY(check_weight(w, act_ld));
+    FORGE_TRY(check_out(w, w.N, act_ld, out));
+    if (!dense_listed_supported(w, m) || k_fixed % BK || k_group % BK || k_fixed <= 0 || k_group <= 0 || w.ld || k_fixed + t.max_tiles * k_group > w.K) {
+        set_error("listed product: %d rows, %d + %d * %d of %d columns", m, k_fixed, t.max_tiles, k_group, w.K);
+        return FORGE_ERR_SHAPE;
+    }
+    GemmParams p{};
+    p.out = out; p.scale = out.scale; p.w = w.tiles; p.m = m; p.N = w.N; p.err = err;
+    p.pitch = w.K / BK; p.groups = t; p.k_fixed = k_fixed / BK; p.k_group = k_group / BK;
+    p.nk = p.k_fixed + t.max_tiles * p.k_group;
+    return m <= 16 ? launch_dense<16, LISTED>(w, act, act_ld, m, p, sm_count(), st) : launch_dense<32, LISTED>(w, act, act_ld, m, p, sm_count(), st);
 }
 
 }  // namespace forge

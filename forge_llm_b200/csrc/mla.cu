@@ -65,7 +65,7 @@ template <> struct Held<__nv_bfloat16> {
 };
 
 template <typename T, int RB>
-__global__ void __launch_bounds__(kThreads) latent_post_kernel(const LatentDims d, const float* __restrict__ proj, int ldp, int dkv_col, const float* __restrict__ kv_norm,
+__global__ void __launch_bounds__(kThreads) latent_post_kernel(const LatentDims d, const float* proj, int ldp, int dkv_col, const float* __restrict__ kv_norm,
                                                                const float2* __restrict__ rope, const T* __restrict__ uk, int uk_ld, T* __restrict__ qabs, T* __restrict__ cache,
                                                                const StepRows rows) {
     extern __shared__ float sm[];   // queries [RB][dim], then partial sums [8][RB][128]
@@ -178,7 +178,7 @@ __global__ void __launch_bounds__(kThreads) latent_prompt_kernel(const LatentDim
 
 // one (row, head, split) per CTA; four warps take its pages' 32-key halves in turn
 template <typename T>
-__global__ void __launch_bounds__(128) latent_attn_kernel(const LatentDims d, const T* __restrict__ qabs, const T* __restrict__ cache, const StepRows rows, float scale2,
+__global__ void __launch_bounds__(128) latent_attn_kernel(const LatentDims d, const T* qabs, const T* cache, const StepRows rows, float scale2,
                                                           float* __restrict__ part, float2* __restrict__ ml) {
     extern __shared__ float sm[];   // query [row], then per warp the running sums [rank_p]
     __shared__ float sml[4][2];
@@ -245,8 +245,8 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentDims d, co
 constexpr int kValueRows = 32;   // rows of W_uv per CTA
 
 template <typename T, int RB>
-__global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentDims d, const float* __restrict__ part, const float2* __restrict__ ml, int splits,
-                                                                const T* __restrict__ uv, int uv_ld, const T* __restrict__ gate, int gate_ld, T* __restrict__ out, int out_ld, int rows, const int32_t* __restrict__ rows_pos) {
+__global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentDims d, const float* part, const float2* ml, int splits,
+                                                                const T* __restrict__ uv, int uv_ld, const T* gate, int gate_ld, T* __restrict__ out, int out_ld, int rows, const int32_t* __restrict__ rows_pos) {
     extern __shared__ __align__(16) float sm[];   // merged latents [RB][rank_p], split factors [RB][splits]
     const int h = blockIdx.y, v0 = blockIdx.z * kValueRows, r0 = blockIdx.x * RB, nr = min(RB, rows - r0);
     const int nv = min(kValueRows, d.vdim - v0);

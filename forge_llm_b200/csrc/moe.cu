@@ -1,0 +1,207 @@
+// Routing of tokens to experts, in f32.  Everything is dealt out in a fixed order (no atomics): the same step gives the same bits.
+#include <algorithm>
+
+#include "moe.cuh"
+
+namespace forge {
+
+namespace {
+
+constexpr int kPerLane = kMaxExperts / 32;
+
+// The warp chooses the `top` largest of z (lower numbers win ties); expert[k] and weight[k] by lane 0.
+__device__ __forceinline__ void choose(const float* z, int experts, int top, int32_t* expert, float* weight) {
+    const int lane = threadIdx.x & 31;
+    float v[kPerLane];
+    uint32_t taken = 0;
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i) v[i] = lane + 32 * i < experts ? z[lane + 32 * i] : 0.f;
+    float first = 0.f, sum = 0.f;
+    for (int k = 0; k < top; ++k) {
+        float best = 0.f;
+        int at = -1;
+#pragma unroll
+        for (int i = 0; i < kPerLane; ++i)
+            if (lane + 32 * i < experts && !(taken >> i & 1) && (at < 0 || v[i] > best)) { best = v[i]; at = lane + 32 * i; }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float other = __shfl_xor_sync(0xffffffffu, best, o);
+            const int whose = __shfl_xor_sync(0xffffffffu, at, o);
+            if (whose >= 0 && (at < 0 || other > best || (other == best && whose < at))) { best = other; at = whose; }
+        }
+        at = __shfl_sync(0xffffffffu, at, 0);      // (values that are no numbers compare differently in different lanes)
+        best = __shfl_sync(0xffffffffu, best, 0);
+        if (k == 0) first = best;
+        const float e = expf(best - first);
+        sum += e;
+        if ((at & 31) == lane) taken |= 1u << (at >> 5);
+        if (lane == 0) { expert[k] = at; weight[k] = e; }
+    }
+    if (lane == 0) for (int k = 0; k < top; ++k) weight[k] /= sum;
+    __syncwarp();
+}
+
+__global__ void __launch_bounds__(1024) route_few_kernel(const RouterDims d, const float* logits, int rows, const RouteTables t) {
+    extern __shared__ float s_w[];                                  // [experts][kScaleRows]
+    int* used = reinterpret_cast<int*>(s_w + d.experts * kScaleRows);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int i = threadIdx.x; i < d.experts * kScaleRows; i += 1024) s_w[i] = 0.f;
+    for (int i = threadIdx.x; i < d.experts; i += 1024) used[i] = 0;
+    __syncthreads();
+    pdl_trigger();
+    pdl_wait();
+    if (warp < rows) {
+        choose(logits + size_t(warp) * d.experts, d.experts, d.top, t.expert + warp * d.top, t.weight + warp * d.top);
+        if (lane == 0)
+            for (int k = 0; k < d.top; ++k) {
+                const int e = t.expert[warp * d.top + k];
+                s_w[e * kScaleRows + warp] = t.weight[warp * d.top + k];
+                used[e] = 1;
+            }
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < d.experts * kScaleRows; i += 1024) t.row_weight[i] = s_w[i];
+    if (warp == 0) {
+        int n = 0;
+        for (int e0 = 0; e0 < d.experts; e0 += 32) {
+            const int e = e0 + lane;
+            const bool on = e < d.experts && used[e];
+            const uint32_t mask = __ballot_sync(0xffffffffu, on);
+            if (on) t.tiles[n + __popc(mask & ((1u << lane) - 1))] = GroupTile{e, 0, rows, e * kScaleRows};
+            n += __popc(mask);
+        }
+        if (lane == 0) *t.n_tiles = n;
+    }
+}
+
+__global__ void __launch_bounds__(256) choose_kernel(const RouterDims d, const float* __restrict__ logits, int rows, const RouteTables t) {
+    const int r = blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (r < rows) choose(logits + size_t(r) * d.experts, d.experts, d.top, t.expert + size_t(r) * d.top, t.weight + size_t(r) * d.top);
+}
+
+// One CTA.  Every warp owns a run of pairs; a pair's place among its expert's is what earlier warps, earlier pairs of the warp and
+// earlier lanes hold.
+__global__ void __launch_bounds__(1024) slots_kernel(const RouterDims d, int rows, int tile_rows, const RouteTables t) {
+    extern __shared__ int s_cnt[];                                  // [32][experts]
+    __shared__ int total[kMaxExperts], start[kMaxExperts], tile0[kMaxExperts];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, E = d.experts, pairs = rows * d.top;
+    const int per = ((pairs + 31) / 32 + 31) & ~31, p0 = warp * per, p1 = min(pairs, p0 + per);
+    int* cnt = s_cnt + warp * E;
+    for (int i = threadIdx.x; i < 32 * E; i += 1024) s_cnt[i] = 0;
+    __syncthreads();
+    for (int p = p0; p < p1; p += 32) {
+        const int e = p + lane < p1 ? t.expert[p + lane] : -1;
+        const uint32_t same = __match_any_sync(0xffffffffu, e);
+        if (e >= 0 && lane == __ffs(same) - 1) cnt[e] += __popc(same);
+        __syncwarp();
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < E; e += 1024) {
+        int sum = 0;
+        for (int w = 0; w < 32; ++w) { const int c = s_cnt[w * E + e]; s_cnt[w * E + e] = sum; sum += c; }
+        total[e] = sum;
+    }
+    __syncthreads();
+    if (warp == 0) {   // where an expert's slots and tiles begin
+        int slots = 0, tiles = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int e = e0 + lane, c = e < E ? total[e] : 0, n = (c + tile_rows - 1) / tile_rows;
+            int sc = c, sn = n;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int a = __shfl_up_sync(0xffffffffu, sc, o), b = __shfl_up_sync(0xffffffffu, sn, o);
+                if (lane >= o) { sc += a; sn += b; }
+            }
+            if (e < E) { start[e] = slots + sc - c; tile0[e] = tiles + sn - n; }
+            slots += __shfl_sync(0xffffffffu, sc, 31);
+            tiles += __shfl_sync(0xffffffffu, sn, 31);
+        }
+        if (lane == 0) *t.n_tiles = tiles;
+    }
+    __syncthreads();
+    for (int e = warp; e < E; e += 32)
+        for (int i = lane; i * tile_rows < total[e]; i += 32) {
+            const int at = start[e] + i * tile_rows;
+            t.tiles[tile0[e] + i] = GroupTile{e, at, min(tile_rows, total[e] - i * tile_rows), at};
+        }
+    for (int p = p0; p < p1; p += 32) {
+        const int i = p + lane, e = i < p1 ? t.expert[i] : -1;
+        const uint32_t same = __match_any_sync(0xffffffffu, e);
+        if (e >= 0) {
+            const int slot = start[e] + cnt[e] + __popc(same & ((1u << lane) - 1));
+            t.slot[i] = slot;
+            t.row[slot] = i / d.top;
+            t.slot_weight[slot] = t.weight[i];
+        }
+        __syncwarp();
+        if (e >= 0 && lane == __ffs(same) - 1) cnt[e] += __popc(same);
+        __syncwarp();
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) add_experts_kernel(float* __restrict__ x, const float* __restrict__ y, const int32_t* __restrict__ slot, int top, int width, const After after) {
+    const int r = blockIdx.x;
+    for (int c0 = blockIdx.y * 256; c0 < width; c0 += gridDim.y * 256) {
+        const int c = c0 + threadIdx.x;
+        const bool ok = c < width;
+        float v = ok ? x[size_t(r) * width + c] : 0.f;
+        for (int k = 0; k < top; ++k) v += ok ? y[size_t(slot[size_t(r) * top + k]) * width + c] : 0.f;
+        v = leave_value<T>(after, v, size_t(r), size_t(width), c, ok);
+        if (ok) x[size_t(r) * width + c] = v;
+    }
+}
+
+size_t align16(size_t n) { return (n + 15) & ~size_t(15); }
+
+}  // namespace
+
+size_t route_bytes(const RouterDims& d, int rows) {
+    const size_t pairs = size_t(rows) * d.top;
+    return 5 * align16(pairs * 4) + size_t(d.experts) * kScaleRows * 4 + (pairs + d.experts) * sizeof(GroupTile) + 16;
+}
+RouteTables route_tables(void* p, const RouterDims& d, int rows) {
+    const size_t pairs = align16(size_t(rows) * d.top * 4);
+    char* b = static_cast<char*>(p);
+    auto take = [&](size_t n) { char* at = b; b += n; return at; };
+    RouteTables t;
+    t.n_tiles = reinterpret_cast<int32_t*>(take(16));
+    t.tiles = reinterpret_cast<GroupTile*>(take((size_t(rows) * d.top + d.experts) * sizeof(GroupTile)));
+    t.row_weight = reinterpret_cast<float*>(take(size_t(d.experts) * kScaleRows * 4));
+    t.expert = reinterpret_cast<int32_t*>(take(pairs)); t.weight = reinterpret_cast<float*>(take(pairs)); t.slot = reinterpret_cast<int32_t*>(take(pairs));
+    t.row = reinterpret_cast<int32_t*>(take(pairs)); t.slot_weight = reinterpret_cast<float*>(take(pairs));
+    return t;
+}
+
+int32_t route_few(const RouterDims& d, const float* logits, int rows, const RouteTables& t, GroupTable* out, cudaStream_t st) {
+    if (rows > kScaleRows || d.experts > kMaxExperts) { set_error("routing: %d rows, %d experts", rows, d.experts); return FORGE_ERR_SHAPE; }
+    *out = GroupTable{t.tiles, t.n_tiles, int(std::min<long long>(d.experts, (long long)rows * d.top)), rows <= 16 ? 16 : 32, t.row_weight};
+    const size_t smem = size_t(d.experts) * (kScaleRows + 1) * 4;
+    FORGE_CUDA(cudaFuncSetAttribute(route_few_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(size_t(kMaxExperts) * (kScaleRows + 1) * 4)));
+    FORGE_CUDA(launch_pdl(route_few_kernel, dim3(1), dim3(1024), smem, st, d, logits, rows, t));
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+
+int32_t route_slots(const RouterDims& d, const float* logits, int rows, const RouteTables& t, GroupTable* out, cudaStream_t st) {
+    if (d.experts > kMaxExperts || (long long)rows * d.top > (1 << 30)) { set_error("routing: %d rows, %d experts", rows, d.experts); return FORGE_ERR_SHAPE; }
+    const int pairs = rows * d.top, tile_rows = group_tile_rows((pairs + d.experts - 1) / d.experts);
+    *out = GroupTable{t.tiles, t.n_tiles, std::min(pairs, pairs / tile_rows + d.experts), tile_rows, t.slot_weight};
+    choose_kernel<<<(rows + 7) / 8, 256, 0, st>>>(d, logits, rows, t);
+    FORGE_LAUNCH_CHECK();
+    FORGE_CUDA(cudaFuncSetAttribute(slots_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 32 * kMaxExperts * 4));
+    slots_kernel<<<1, 1024, size_t(32) * d.experts * 4, st>>>(d, rows, tile_rows, t);
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+
+int32_t add_experts(float* x, const float* y, const RouterDims& d, const RouteTables& t, int rows, int width, const After& after, int dtype, cudaStream_t st) {
+    if (rows <= 0) return FORGE_OK;
+    const dim3 grid(rows, rows < 64 ? (width + 255) / 256 : 1);
+    if (dtype == FORGE_F32) add_experts_kernel<float><<<grid, 256, 0, st>>>(x, y, t.slot, d.top, width, after);
+    else add_experts_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(x, y, t.slot, d.top, width, after);
+    FORGE_LAUNCH_CHECK();
+    return FORGE_OK;
+}
+
+}  // namespace forge

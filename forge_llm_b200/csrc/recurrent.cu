@@ -73,8 +73,9 @@ template <int N> __device__ __forceinline__ void store_cols(float* p, const floa
     else if constexpr (N == 2) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
     else *p = v[0];
 }
-template <typename T, bool DELTA, bool CHANNEL, int RPT, int CPL>
+template <typename T, Rule RULE, bool CHANNEL, int RPT, int CPL>
 __global__ void __launch_bounds__(256, CPL > 1 ? 2 : 1) recur_decode_kernel(const RecurDims d, const RecurArgs a, const StepRows rows) {
+    constexpr bool DELTA = RULE == Rule::Delta;
     extern __shared__ float sm[];
     float* sq = sm;                 // [dim] queries, keys, decays
     float* sk = sq + d.dim;
@@ -149,7 +150,7 @@ __global__ void __launch_bounds__(256, CPL > 1 ? 2 : 1) recur_decode_kernel(cons
         float s0 = 0.f, s1 = 0.f;
         for (int i = tid; i < d.dim; i += 256) {
             if constexpr (DELTA) { s0 = fmaf(sq[i], sq[i], s0); s1 = fmaf(sk[i], sk[i], s1); }
-            else s0 = fmaf(sq[i] * a.bonus[h * d.dim + i], sk[i], s0);
+            else if constexpr (RULE == Rule::TimeMix) s0 = fmaf(sq[i] * a.bonus[h * d.dim + i], sk[i], s0);
         }
         s0 = warp_sum(s0);
         if constexpr (DELTA) s1 = warp_sum(s1);
@@ -158,7 +159,7 @@ __global__ void __launch_bounds__(256, CPL > 1 ? 2 : 1) recur_decode_kernel(cons
     if (two_step) {
         low_d.run(slow, [&](int i, float z) {
             z += a.decay_add[h * d.dim + i];
-            sg[i] = expf(DELTA ? -a.decay_mul[h * d.dim + i] * softplus(z) : -expf(z));
+            sg[i] = expf(RULE != Rule::TimeMix ? -a.decay_mul[h * d.dim + i] * softplus(z) : -expf(z));
         });
         if (low_gate) low_g.run(slow + a.low_k, [&](int i, float z) { sgate[i] = sigmoid(z); });
     }
@@ -169,7 +170,7 @@ __global__ void __launch_bounds__(256, CPL > 1 ? 2 : 1) recur_decode_kernel(cons
     float t0 = 0.f, t1 = 0.f;
 #pragma unroll
     for (int w = 0; w < 8; ++w) { t0 += wsum[w][0]; t1 += wsum[w][1]; }
-    const float qs = DELTA ? d.q_scale / sqrtf(t0 + 1e-6f) : 1.f, ks = DELTA ? 1.0f / sqrtf(t1 + 1e-6f) : 1.f;
+    const float qs = DELTA ? d.q_scale / sqrtf(t0 + 1e-6f) : d.q_scale, ks = DELTA ? 1.0f / sqrtf(t1 + 1e-6f) : 1.f;
     float o[CPL], sum8[CPL];
     auto all_warps = [&](float (*buf)[NC], const float (&mine)[CPL]) {   // sum over the warps' rows
         store_cols<CPL>(&buf[warp][cl], mine);
@@ -220,9 +221,13 @@ __global__ void __launch_bounds__(256, CPL > 1 ? 2 : 1) recur_decode_kernel(cons
         for (int i = 0; i < RPT; ++i) {
             const int row = warp + 8 * i;
             if (row < d.dim) {
-                const float w = CHANNEL ? sg[row] : g1, k = sk[row], q = sq[row];
+                const float w = CHANNEL ? sg[row] : g1, k = sk[row], q = sq[row] * qs;
 #pragma unroll
-                for (int c = 0; c < CPL; ++c) { o[c] = fmaf(st[i][c], q, o[c]); st[i][c] = fmaf(k, v[c], st[i][c] * w); }
+                for (int c = 0; c < CPL; ++c) {
+                    const float next = fmaf(k, v[c], st[i][c] * w);
+                    o[c] = fmaf(RULE == Rule::Linear ? next : st[i][c], q, o[c]);
+                    st[i][c] = next;
+                }
                 if (own) store_cols<CPL>(S + size_t(row) * d.vdim, st[i]);
             }
         }
@@ -233,7 +238,7 @@ __global__ void __launch_bounds__(256, CPL > 1 ? 2 : 1) recur_decode_kernel(cons
 #pragma unroll
         for (int c = 0; c < CPL; ++c) {
             o[c] = sum8[c];
-            if constexpr (!DELTA) o[c] = fmaf(t0, own ? sv[cl + c] : 0.f, o[c]);
+            if constexpr (RULE == Rule::TimeMix) o[c] = fmaf(t0, own ? sv[cl + c] : 0.f, o[c]);
             if (own) ss = fmaf(o[c], o[c], ss);
         }
         ss = warp_sum(ss);
@@ -368,8 +373,9 @@ bool conv_rows8_supported(const RecurDims& d) {
 }
 
 // Token by token: a warp carries four value columns of one head, its lanes share the rows of the state.
-template <typename T, bool DELTA, bool CHANNEL, int RPL>
+template <typename T, Rule RULE, bool CHANNEL, int RPL>
 __global__ void __launch_bounds__(128) scan_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs) {
+    constexpr bool DELTA = RULE == Rule::Delta;
     const ScanSeg s = segs[blockIdx.z];
     const int lane = threadIdx.x & 31, h = blockIdx.y, c0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * 4;
     if (c0 >= d.vdim) return;
@@ -381,7 +387,7 @@ __global__ void __launch_bounds__(128) scan_kernel(const RecurDims d, const Recu
 #pragma unroll
     for (int i = 0; i < RPL; ++i) {
         const int row = lane + 32 * i;
-        bonus[i] = !DELTA && row < d.dim ? a.bonus[h * d.dim + row] : 0.f;
+        bonus[i] = RULE == Rule::TimeMix && row < d.dim ? a.bonus[h * d.dim + row] : 0.f;
 #pragma unroll
         for (int c = 0; c < 4; ++c) st[i][c] = s.pos0 > 0 && row < d.dim && c < nc ? S[size_t(row) * d.vdim + c] : 0.f;
     }
@@ -432,13 +438,18 @@ __global__ void __launch_bounds__(128) scan_kernel(const RecurDims d, const Recu
             const float g1 = CHANNEL ? 0.f : expf(in.g[0]);
 #pragma unroll
             for (int i = 0; i < RPL; ++i) {
-                const float w = CHANNEL ? expf(in.g[CHANNEL ? i : 0]) : g1, k = to_f(in.k[i]), q = to_f(in.q[i]);
+                const float w = CHANNEL ? expf(in.g[CHANNEL ? i : 0]) : g1, k = to_f(in.k[i]), q = to_f(in.q[i]) * d.q_scale;
                 own = fmaf(q * bonus[i], k, own);
 #pragma unroll
-                for (int c = 0; c < 4; ++c) { o[c] = fmaf(st[i][c], q, o[c]); st[i][c] = fmaf(k, to_f(in.v[c]), st[i][c] * w); }
+                for (int c = 0; c < 4; ++c) {
+                    const float next = fmaf(k, to_f(in.v[c]), st[i][c] * w);
+                    o[c] = fmaf(RULE == Rule::Linear ? next : st[i][c], q, o[c]);
+                    st[i][c] = next;
+                }
             }
+            if constexpr (RULE == Rule::TimeMix)
 #pragma unroll
-            for (int c = 0; c < 4; ++c) o[c] = fmaf(own, to_f(in.v[c]), o[c]);
+                for (int c = 0; c < 4; ++c) o[c] = fmaf(own, to_f(in.v[c]), o[c]);
         }
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
@@ -492,7 +503,7 @@ __global__ void __launch_bounds__(256) head_norm4_kernel(const RecurDims d, cons
 // before a segment is the one that leaves the segment's last row there.
 constexpr int kShiftRows = 16;
 template <typename T>
-__global__ void __launch_bounds__(256) token_shift_kernel(T* __restrict__ dst, int ld, int width, int width_p, int n_mix, const float* __restrict__ mu, T* __restrict__ prev, const StepRows rows,
+__global__ void __launch_bounds__(256) token_shift_kernel(T* dst, int ld, int width, int width_p, int n_mix, const float* __restrict__ mu, T* prev, const StepRows rows,
                                                           const ScanSeg* __restrict__ segs) {
     const int c = blockIdx.y * 256 + threadIdx.x;
     ScanSeg s;
@@ -520,7 +531,7 @@ __global__ void __launch_bounds__(256) token_shift_kernel(T* __restrict__ dst, i
 // ------------------------------------------------------------------------------------------------ sum of two normed rows
 // NV: four-value pieces per thread of rows of up to 1024 NV values (a multiple of four); 0: any width
 template <typename T, int NV>
-__global__ void __launch_bounds__(256) add_normed_pair_kernel(float* __restrict__ x, const float* __restrict__ ab, int width, float eps, const float* __restrict__ wa, const float* __restrict__ wb, const After after) {
+__global__ void __launch_bounds__(256) add_normed_pair_kernel(float* x, const float* ab, int width, float eps, const float* __restrict__ wa, const float* __restrict__ wb, const After after) {
     __shared__ float red[8][2];
     const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const float* a = ab + size_t(r) * 2 * width;
@@ -589,39 +600,39 @@ __global__ void __launch_bounds__(256) add_normed_pair_kernel(float* __restrict_
     }
 }
 
-template <typename T, bool DELTA, bool CHANNEL, int RPT, int CPL>
+template <typename T, Rule RULE, bool CHANNEL, int RPT, int CPL>
 int32_t launch_decode(const RecurDims& d, const RecurArgs& a, const StepRows& rows, cudaStream_t st) {
     const int splits = (d.vdim + 32 * CPL - 1) / (32 * CPL);
     const size_t smem = sizeof(float) * (3 * size_t(d.dim) + 64 * CPL + 4 + 2 * size_t(a.low_k));
-    FORGE_CUDA(launch_pdl_cluster(recur_decode_kernel<T, DELTA, CHANNEL, RPT, CPL>, dim3(splits, d.heads, rows.n), dim3(256), splits, smem, st, d, a, rows));
+    FORGE_CUDA(launch_pdl_cluster(recur_decode_kernel<T, RULE, CHANNEL, RPT, CPL>, dim3(splits, d.heads, rows.n), dim3(256), splits, smem, st, d, a, rows));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
-template <typename T, bool DELTA, bool CHANNEL>
+template <typename T, Rule RULE, bool CHANNEL>
 int32_t decode_t(const RecurDims& d, const RecurArgs& a, const StepRows& rows, cudaStream_t st) {
     // enough rows to fill the SMs: whole heads (what all columns of a head share is formed once)
     const bool whole = (long long)rows.n * d.heads >= 148 && d.vdim > 32;
-    if (whole && d.vdim <= 64 && d.vdim % 2 == 0 && d.dim <= 64) return launch_decode<T, DELTA, CHANNEL, 8, 2>(d, a, rows, st);
-    if (whole && d.vdim % 4 == 0 && d.dim <= 64) return launch_decode<T, DELTA, CHANNEL, 8, 4>(d, a, rows, st);
-    if (whole && d.vdim % 4 == 0 && d.dim <= 128) return launch_decode<T, DELTA, CHANNEL, 16, 4>(d, a, rows, st);
-    if (d.dim <= 64) return launch_decode<T, DELTA, CHANNEL, 8, 1>(d, a, rows, st);
-    if (d.dim <= 128) return launch_decode<T, DELTA, CHANNEL, 16, 1>(d, a, rows, st);
-    return launch_decode<T, DELTA, CHANNEL, 32, 1>(d, a, rows, st);
+    if (whole && d.vdim <= 64 && d.vdim % 2 == 0 && d.dim <= 64) return launch_decode<T, RULE, CHANNEL, 8, 2>(d, a, rows, st);
+    if (whole && d.vdim % 4 == 0 && d.dim <= 64) return launch_decode<T, RULE, CHANNEL, 8, 4>(d, a, rows, st);
+    if (whole && d.vdim % 4 == 0 && d.dim <= 128) return launch_decode<T, RULE, CHANNEL, 16, 4>(d, a, rows, st);
+    if (d.dim <= 64) return launch_decode<T, RULE, CHANNEL, 8, 1>(d, a, rows, st);
+    if (d.dim <= 128) return launch_decode<T, RULE, CHANNEL, 16, 1>(d, a, rows, st);
+    return launch_decode<T, RULE, CHANNEL, 32, 1>(d, a, rows, st);
 }
-template <typename T, bool DELTA, bool CHANNEL>
+template <typename T, Rule RULE, bool CHANNEL>
 int32_t scan_t(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, const ScanSeg* segs, int n_segs, cudaStream_t st) {
     const dim3 grid((d.vdim + 15) / 16, d.heads, n_segs);
-    if (d.dim <= 32) scan_kernel<T, DELTA, CHANNEL, 1><<<grid, 128, 0, st>>>(d, a, sc, segs);
-    else if (d.dim <= 64) scan_kernel<T, DELTA, CHANNEL, 2><<<grid, 128, 0, st>>>(d, a, sc, segs);
-    else if (d.dim <= 128) scan_kernel<T, DELTA, CHANNEL, 4><<<grid, 128, 0, st>>>(d, a, sc, segs);
-    else scan_kernel<T, DELTA, CHANNEL, 8><<<grid, 128, 0, st>>>(d, a, sc, segs);
+    if (d.dim <= 32) scan_kernel<T, RULE, CHANNEL, 1><<<grid, 128, 0, st>>>(d, a, sc, segs);
+    else if (d.dim <= 64) scan_kernel<T, RULE, CHANNEL, 2><<<grid, 128, 0, st>>>(d, a, sc, segs);
+    else if (d.dim <= 128) scan_kernel<T, RULE, CHANNEL, 4><<<grid, 128, 0, st>>>(d, a, sc, segs);
+    else scan_kernel<T, RULE, CHANNEL, 8><<<grid, 128, 0, st>>>(d, a, sc, segs);
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
 template <typename T>
 int32_t segments_t(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, const SegTable& t, cudaStream_t st) {
     constexpr bool half = std::is_same<T, __nv_bfloat16>::value;
-    if (d.delta) {
+    if (d.rule == Rule::Delta) {
         const int tiles = (t.max_n + kConvTile - 1) / kConvTile, units = 2 * d.groups + (d.heads * d.vdim + 127) / 128;
         if (half && conv_rows8_supported(d)) conv_rows8_kernel<<<dim3((t.max_n + kConvRun - 1) / kConvRun, (d.channels() + 1023) / 1024, t.n), 128, 0, st>>>(d, a, sc, t.segs);
         else conv_rows_kernel<T><<<dim3(tiles, (units + 7) / 8, t.n), 256, 0, st>>>(d, a, sc, t.segs);
@@ -629,8 +640,9 @@ int32_t segments_t(const RecurDims& d, const RecurArgs& a, const RecurScratch& s
     }
     const int walked = half && recur_chunked_supported(d) ? t.n_short : t.n;   // token by token
     if (walked > 0) {
-        if (!d.delta) FORGE_TRY((scan_t<T, false, true>(d, a, sc, t.segs, walked, st)));
-        else FORGE_TRY(d.channel ? (scan_t<T, true, true>(d, a, sc, t.segs, walked, st)) : (scan_t<T, true, false>(d, a, sc, t.segs, walked, st)));
+        if (d.rule == Rule::TimeMix) FORGE_TRY((scan_t<T, Rule::TimeMix, true>(d, a, sc, t.segs, walked, st)));
+        else if (d.rule == Rule::Linear) FORGE_TRY((scan_t<T, Rule::Linear, true>(d, a, sc, t.segs, walked, st)));
+        else FORGE_TRY(d.channel ? (scan_t<T, Rule::Delta, true>(d, a, sc, t.segs, walked, st)) : (scan_t<T, Rule::Delta, false>(d, a, sc, t.segs, walked, st)));
     }
     FORGE_TRY(recur_chunked(d, a, sc, t.segs + walked, t.n - walked, t.n_chunks, st));
     const int lanes = d.vdim / 4;
@@ -643,14 +655,15 @@ int32_t segments_t(const RecurDims& d, const RecurArgs& a, const RecurScratch& s
 
 }  // namespace
 
-bool recur_supported(const RecurDims& d) { return d.dim <= 256 && d.vdim <= 256 && d.taps <= kConvTile && (d.delta ? d.taps >= 1 : d.channel && d.taps == 0); }
+bool recur_supported(const RecurDims& d) { return d.dim <= 256 && d.vdim <= 256 && d.taps <= kConvTile && (d.rule == Rule::Delta ? d.taps >= 1 : d.channel && d.taps == 0); }
 
 int32_t recur_decode(const RecurDims& d, int dtype, const RecurArgs& a, const StepRows& rows, cudaStream_t st) {
     if (rows.n <= 0) return FORGE_OK;
     auto go = [&](auto t) -> int32_t {
         using T = decltype(t);
-        if (!d.delta) return decode_t<T, false, true>(d, a, rows, st);
-        return d.channel ? decode_t<T, true, true>(d, a, rows, st) : decode_t<T, true, false>(d, a, rows, st);
+        if (d.rule == Rule::TimeMix) return decode_t<T, Rule::TimeMix, true>(d, a, rows, st);
+        if (d.rule == Rule::Linear) return decode_t<T, Rule::Linear, true>(d, a, rows, st);
+        return d.channel ? decode_t<T, Rule::Delta, true>(d, a, rows, st) : decode_t<T, Rule::Delta, false>(d, a, rows, st);
     };
     return dtype == FORGE_F32 ? go(float{}) : go(__nv_bfloat16{});
 }

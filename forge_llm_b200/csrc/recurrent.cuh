@@ -1,6 +1,7 @@
 // Recurrent mixers: per head a state S [dim][vdim] in f32 that every token decays, extends and reads.
 //   delta rule     S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //   time mixing    o = S^T q + (sum_c q_c bonus_c k_c) v;  S <- diag(g) S + k v^T
+//   linear         S <- diag(g) S + k v^T;  o = S^T q
 // g is one decay per head or one per head and key channel, given by its logarithm.  The delta rule's q, k, v come from a short
 // causal convolution per channel with silu behind it, q and k as unit vectors; its last inputs are kept in a ring of `taps` rows,
 // the input of position p in row p % taps.  A sequence's state counts as zero when its first row of a step is at position 0, so
@@ -11,10 +12,12 @@
 
 namespace forge {
 
+enum class Rule { TimeMix, Delta, Linear };
 struct RecurDims {
     int heads = 0, groups = 0, dim = 0, vdim = 0;   // groups: heads of q and k (head h uses h / (heads / groups))
     int taps = 0;                                   // 0: no convolution
-    bool delta = false, channel = false;            // channel: a decay per key channel
+    Rule rule = Rule::TimeMix;
+    bool channel = false;                           // a decay per key channel
     float eps = 0.f, q_scale = 1.f;
     __host__ __device__ int qk() const { return groups * dim; }
     __host__ __device__ int channels() const { return 2 * groups * dim + heads * vdim; }
@@ -39,7 +42,7 @@ struct RecurArgs {
     float* state = nullptr;                              // [slot][heads][dim][vdim]
     // second step of two-step decays and gates, for single tokens (then decay, and gate if gate_w is set, are not read): T rows of low_k values per
     // key channel and per value over the inner values low[row], the gate's from column gate_col; a decay's logarithm is
-    // -mul softplus(z + add) for the delta rule, -exp(z + add) for time mixing
+    // -mul softplus(z + add), for time mixing -exp(z + add)
     const void* decay_w = nullptr; const void* gate_w = nullptr; const void* low = nullptr;
     int low_ld = 0, low_k = 0, gate_col = 0;
     const float* decay_mul = nullptr; const float* decay_add = nullptr;

@@ -4,7 +4,8 @@
 //   delta rule    (I + L) U = R,  R_t = beta_t (v_t - S^T (e^{G_t} k_t)),  L_ts = beta_t sum_c k_tc k_sc e^{G_tc - G_sc}  (s < t)
 //                 o_t = S^T (e^{G_t} q_t) + sum_{s <= t} P_ts u_s,         P_ts = sum_c q_tc k_sc e^{G_tc - G_sc}
 //                 S <- e^{G_end} S + sum_s (e^{G_end - G_s} k_s) u_s^T
-//   time mixing   U = V, o_t reads with e^{G_(t-1)} instead of e^{G_t}, and P_tt = sum_c q_tc bonus_c k_tc.
+//   time mixing   U = V, o_t reads with e^{G_(t-1)} instead of e^{G_t}, and P_tt = sum_c q_tc bonus_c k_tc;
+//   linear        U = V.
 // chunk_prep_kernel (every chunk and head at once) inverts I + L and leaves P, U0 = (I + L)^-1 diag(beta) V and
 // W = (I + L)^-1 diag(beta) e^G K, so that U = U0 - W S; chunk_scan_kernel walks a sequence's chunks with a block of 32 columns of
 // the state in registers: two dependent products per chunk (U, then S), the read-out beside them.  What the walk reads lies in
@@ -36,7 +37,8 @@ using tc5::mbar_wait;
 constexpr int C = kRecurChunk;          // tokens of a chunk
 constexpr int NB = 32;                  // value columns of a CTA of the walk
 constexpr int LDT = C + 8, LDN = NB + 8, TT = C * LDT, VT = C * LDN;
-enum Mode { HEAD_DELTA = 0, CHANNEL_DELTA = 1, TIME_MIX = 2 };
+enum Mode { HEAD_DELTA = 0, CHANNEL_DELTA = 1, TIME_MIX = 2, LINEAR = 3 };
+__host__ __device__ constexpr bool writes_v(int mode) { return mode == TIME_MIX || mode == LINEAR; }   // U = V
 constexpr float kLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return uint32_t(__cvta_generic_to_shared(p)); }
@@ -50,18 +52,19 @@ __device__ __forceinline__ float ex2(float x) {   // 2^x
 // P hi, lo; v in blocks of 32 columns (time mixing).  f32: U0 in blocks [64][32] (delta rules), scale of q and of k's update per
 // token (decay per head), e^{G_end} per channel.
 template <int DK, int MODE> struct Rec {
+    static constexpr bool PLAIN = writes_v(MODE);
     static constexpr int LDK = DK + 8, KT = C * LDK;
-    static constexpr int nw = MODE == TIME_MIX ? 0 : 2, nx = MODE == HEAD_DELTA ? 1 : 2;
+    static constexpr int nw = PLAIN ? 0 : 2, nx = MODE == HEAD_DELTA ? 1 : 2;
     static constexpr int oq = nw * KT, ok = oq + nx * KT, op = ok + nx * KT, ov = op + 2 * TT;
-    static __host__ __device__ size_t halves(int nb) { return size_t(ov) + (MODE == TIME_MIX ? size_t(nb) * VT : 0); }
-    static __host__ __device__ size_t floats(int nb) { return (MODE == TIME_MIX ? 0 : size_t(nb) * C * NB) + 2 * C + DK; }
+    static __host__ __device__ size_t halves(int nb) { return size_t(ov) + (PLAIN ? size_t(nb) * VT : 0); }
+    static __host__ __device__ size_t floats(int nb) { return (PLAIN ? 0 : size_t(nb) * C * NB) + 2 * C + DK; }
     bf16* h; float* f;
     float *scal, *end;
     __device__ __forceinline__ Rec(const ChunkScratch& s, int chunk, int heads, int head, int nb) {
         const size_t i = size_t(chunk) * heads + head;
         h = s.half + i * halves(nb);
         f = s.f32 + i * floats(nb);
-        scal = f + (MODE == TIME_MIX ? 0 : size_t(nb) * C * NB);
+        scal = f + (PLAIN ? 0 : size_t(nb) * C * NB);
         end = scal + 2 * C;
     }
 };
@@ -130,6 +133,7 @@ template <int DK, int MODE> struct Prep {
 
 template <int DK, int MODE>
 __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs, int n_segs) {
+    constexpr bool PLAIN = writes_v(MODE), TIME = MODE == TIME_MIX;
     using L = Prep<DK, MODE>;
     using R = Rec<DK, MODE>;
     constexpr int NT = L::NT, LDK = L::LDK, NW = NT / 32, KT = R::KT;
@@ -153,8 +157,8 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
     const ScanSeg s = segs[s_seg];
     const int t0 = (chunk - s.chunk0) * C, n = min(C, s.n - t0), row0 = s.row0 + t0;
     const R out(sc.chunk, chunk, d.heads, h, nb);
-    const bf16* x = MODE == TIME_MIX ? static_cast<const bf16*>(a.x) : static_cast<const bf16*>(sc.conv);
-    const size_t ld = MODE == TIME_MIX ? a.x_ld : d.channels();
+    const bf16* x = PLAIN ? static_cast<const bf16*>(a.x) : static_cast<const bf16*>(sc.conv);
+    const size_t ld = PLAIN ? a.x_ld : d.channels();
     // [64] rows of the step, `cols` of its columns from col0 (zeros past `valid`)
     auto fetch = [&](bf16* dst, int l, int col0, int cols, int valid) {
         for (int i = tid; i < C * (cols / 8); i += NT) {
@@ -168,8 +172,9 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
     cp_commit();
     if (tid < C) {
         const bool ok = tid < n;
-        s_ks[tid] = s_qs[tid] = s_beta[tid] = 1.f;
-        if constexpr (MODE != TIME_MIX) {
+        s_ks[tid] = s_beta[tid] = 1.f;
+        s_qs[tid] = d.q_scale;
+        if constexpr (!PLAIN) {
             s_ks[tid] = ok ? sc.unit[size_t(row0 + tid) * 2 * d.groups + d.groups + g] : 0.f;   // |k|^-1
             s_qs[tid] = ok ? sc.unit[size_t(row0 + tid) * 2 * d.groups + g] : 0.f;              // q scale
             s_beta[tid] = ok ? a.beta[size_t(row0 + tid) * d.heads + h] : 0.f;
@@ -250,8 +255,8 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
             out.end[c] = ex2(sum);
         }
         // exponents of a query row inside its block: up to and including its own decay, or for time mixing without it
-        auto sum_q = [&](int t) { return MODE == TIME_MIX ? sg + (t - 1) * DK : sg + t * DK; };
-        auto first = [](int t) { return MODE == TIME_MIX && !(t & 15); };   // then they are zero
+        auto sum_q = [&](int t) { return TIME ? sg + (t - 1) * DK : sg + t * DK; };
+        auto first = [](int t) { return TIME && !(t & 15); };   // then they are zero
         // pairs inside a block: a warp per row, DK / 32 neighbouring channels per lane, sixteen partners at once
         constexpr int PL = DK / 32;
         for (int t = warp; t < C; t += NW) {
@@ -271,8 +276,8 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
 #pragma unroll
                 for (int i = 0; i < PL; ++i) {
                     const float ku = __bfloat162float(sk[u * LDK + c + i]), gu = sg[u * DK + c + i];
-                    if constexpr (MODE == TIME_MIX) part[j] = fmaf(qv[i] * ku, u < t ? ex2(eq[i] - gu) : c + i < d.dim ? a.bonus[h * d.dim + c + i] : 0.f, part[j]);
-                    else { const float e = ex2(eq[i] - gu) * ku; part[j] = fmaf(qv[i], e, part[j]); part[16 + j] = fmaf(kv[i], e, part[16 + j]); }
+                    if constexpr (TIME) part[j] = fmaf(qv[i] * ku, u < t ? ex2(eq[i] - gu) : c + i < d.dim ? a.bonus[h * d.dim + c + i] : 0.f, part[j]);
+                    else { const float e = ex2(eq[i] - gu) * ku; part[j] = fmaf(qv[i], e, part[j]); if (!PLAIN) part[16 + j] = fmaf(kv[i], e, part[16 + j]); }
                 }
             }
             // lane l ends with the sum of part[l]
@@ -287,7 +292,7 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
             const int j = lane & 15, u = (t & ~15) + j;
             if (u <= t) {
                 if (lane < 16) sp[t * LDL + u] = part[0] * s_qs[t] * s_ks[u];
-                else if (MODE != TIME_MIX) sl[t * LDL + u] = part[0] * s_beta[t] * s_ks[t] * s_ks[u];
+                else if (!PLAIN) sl[t * LDL + u] = part[0] * s_beta[t] * s_ks[t] * s_ks[u];
             }
         }
         __syncthreads();
@@ -313,7 +318,7 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
             const SmemMat ah{smem_addr(sa), LDK}, al{smem_addr(sa + 32 * LDK), LDK}, bh{smem_addr(so), LDK}, bl{smem_addr(so + 48 * LDK), LDK};
             for (int w = warp; w < 4 * b; w += NW) {   // (k or q) x 8 earlier keys
                 const int is_q = w & 1, n8 = w >> 1;
-                if (MODE == TIME_MIX && !is_q) continue;
+                if (PLAIN && !is_q) continue;
                 float acc[3][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
                 for (int kt = 0; kt < DK / 16; ++kt) {
@@ -348,13 +353,13 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
             split_bf16x2(k.x * ks * ex2(end.x - f.x - w.x), k.y * ks * ex2(end.y - f.y - w.y), hi, lo);
             dst = reinterpret_cast<uint32_t*>(out.h + R::ok + t * LDK + c);
             dst[0] = hi; dst[KT / 2] = lo;
-            if constexpr (MODE != TIME_MIX) {
+            if constexpr (!PLAIN) {
                 split_bf16x2(k.x * ks * ex2(f.x + w.x), k.y * ks * ex2(f.y + w.y), hi, lo);
                 dst = reinterpret_cast<uint32_t*>(sa + t * LDK + c);
                 dst[0] = hi; dst[KT / 2] = lo;
             }
         }
-        if constexpr (MODE == TIME_MIX) {   // v as the walk's tiles
+        if constexpr (PLAIN) {   // v as the walk's tiles
             for (int i = tid; i < nb * C * (NB / 8); i += NT) {
                 const int blk = i / (C * (NB / 8)), t = i / (NB / 8) % C, c = (i % (NB / 8)) * 8;
                 const bool ok = t < n && blk * NB + c < d.vdim;
@@ -364,7 +369,7 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
         }
     }
     put_lower<NT>(out.h + R::op, sp, nullptr, tid);
-    if constexpr (MODE != TIME_MIX) {
+    if constexpr (!PLAIN) {
         __syncthreads();
         fetch(sq, LDK, 2 * d.qk() + h * d.vdim, DK, d.vdim);   // q gives way to the first columns of v
         cp_commit();
@@ -431,11 +436,12 @@ __global__ void __launch_bounds__(Prep<DK, MODE>::NT) chunk_prep_kernel(const Re
 
 // ------------------------------------------------------------------------------------------------ walk over the chunks
 template <int DK, int MODE> struct Scan {
+    static constexpr bool PLAIN = writes_v(MODE);
     using R = Rec<DK, MODE>;
     static constexpr int SS = DK * LDN;                              // one half of a state buffer
     static constexpr int ST = DK <= 64 ? 2 : 1;                      // buffers of every tile
-    static constexpr int ow = 0, oq = R::nw * R::KT, ok = oq + R::nx * R::KT, op = ok + R::nx * R::KT, ov = op + 2 * TT, stage = ov + (MODE == TIME_MIX ? VT : 0), os = ST * stage,
-                         ou = os + 4 * SS, ox = ou + (MODE == TIME_MIX ? 0 : 2 * VT), total = ox + (MODE == HEAD_DELTA ? 2 * VT : 0);
+    static constexpr int ow = 0, oq = R::nw * R::KT, ok = oq + R::nx * R::KT, op = ok + R::nx * R::KT, ov = op + 2 * TT, stage = ov + (PLAIN ? VT : 0), os = ST * stage,
+                         ou = os + 4 * SS, ox = ou + (PLAIN ? 0 : 2 * VT), total = ox + (MODE == HEAD_DELTA ? 2 * VT : 0);
     static constexpr size_t smem = size_t(total) * 2 + 16;
 };
 
@@ -444,6 +450,7 @@ __device__ __forceinline__ void walk_sync() { asm volatile("bar.sync 1, 256;" ::
 
 template <int DK, int MODE>
 __global__ void __launch_bounds__(kScanThreads, 1) chunk_scan_kernel(const RecurDims d, const RecurArgs a, const RecurScratch sc, const ScanSeg* __restrict__ segs, int* err) {
+    constexpr bool PLAIN = writes_v(MODE);
     using L = Scan<DK, MODE>;
     using R = Rec<DK, MODE>;
     constexpr int LDK = R::LDK, KT = R::KT, ST = L::ST;
@@ -474,8 +481,8 @@ __global__ void __launch_bounds__(kScanThreads, 1) chunk_scan_kernel(const Recur
                     bulk_load(sm + b * L::stage + dst, src, uint32_t(elems) * 2, &full[b][buf]);
                     if (more_elems) bulk_load(sm + b * L::stage + more_dst, more, uint32_t(more_elems) * 2, &full[b][buf]);
                 };
-                if constexpr (MODE != TIME_MIX) load(BW, L::ow, r.h, 2 * KT);
-                load(BK, L::ok, r.h + R::ok, R::nx * KT, r.h + R::ov + size_t(blockIdx.x) * VT, L::ov, MODE == TIME_MIX ? VT : 0);
+                if constexpr (!PLAIN) load(BW, L::ow, r.h, 2 * KT);
+                load(BK, L::ok, r.h + R::ok, R::nx * KT, r.h + R::ov + size_t(blockIdx.x) * VT, L::ov, PLAIN ? VT : 0);
                 load(BQ, L::oq, r.h + R::oq, R::nx * KT);
                 load(BP, L::op, r.h + R::op, 2 * TT);
             }
@@ -530,7 +537,7 @@ __global__ void __launch_bounds__(kScanThreads, 1) chunk_scan_kernel(const Recur
             for (int e = 0; e < 2; ++e) {
                 o.end[e] = r.end[sm0 + lr + 8 * e];
                 if constexpr (MODE == HEAD_DELTA) { o.qd[e] = r.scal[t_lo + 8 * e]; o.ko[e] = r.scal[C + t_lo + 8 * e]; }
-                if constexpr (MODE != TIME_MIX)
+                if constexpr (!PLAIN)
 #pragma unroll
                     for (int j = 0; j < 2; ++j) o.u0[j][e] = *reinterpret_cast<const float2*>(r.f + size_t(blockIdx.x) * C * NB + (t_lo + 8 * e) * NB + n0 + j * 8 + lc);
             }
@@ -540,14 +547,14 @@ __global__ void __launch_bounds__(kScanThreads, 1) chunk_scan_kernel(const Recur
         for (int ch = 0; ch < chunks; ++ch) {
             const Own next = own(ch + 1);
             const int at = ch % ST * L::stage;
-            const SmemMat uh = mat(MODE == TIME_MIX ? at + L::ov : L::ou, LDN), ph = mat(at + L::op, LDT), pl = mat(at + L::op + TT, LDT);
+            const SmemMat uh = mat(PLAIN ? at + L::ov : L::ou, LDN), ph = mat(at + L::op, LDT), pl = mat(at + L::op + TT, LDT);
             const SmemMat wh = mat(at + L::ow, LDK), wl = mat(at + L::ow + KT, LDK), qh = mat(at + L::oq, LDK), ql = mat(at + L::oq + KT, LDK), kh = mat(at + L::ok, LDK), kl = mat(at + L::ok + KT, LDK);
             const SmemMat sh = mat(L::os + (ch & 1) * 2 * L::SS, LDN), slo = mat(L::os + (ch & 1) * 2 * L::SS + L::SS, LDN);
             // the state in front of the chunk as B operands of two products (shared-memory reads bound this kernel)
             uint32_t gh[DK / 16][4], gl[DK / 16][4];
 #pragma unroll
             for (int kt = 0; kt < DK / 16; ++kt) { sh.b_t(gh[kt], kt * 16, n0, lane); slo.b_t(gl[kt], kt * 16, n0, lane); }
-            if constexpr (MODE != TIME_MIX) {   // U = U0 - W S
+            if constexpr (!PLAIN) {   // U = U0 - W S
                 take(BW, ch);
                 float acc[3][2][4];
 #pragma unroll
@@ -592,16 +599,16 @@ __global__ void __launch_bounds__(kScanThreads, 1) chunk_scan_kernel(const Recur
                 for (int i = 0; i < NI; ++i) {
                     uint32_t gh[4], gl[4];
                     (MODE == HEAD_DELTA ? xh : uh).b_t(gh, kt * 16, sn0 + i * 16, lane);
-                    if constexpr (MODE != TIME_MIX) (MODE == HEAD_DELTA ? xl : ul).b_t(gl, kt * 16, sn0 + i * 16, lane);
+                    if constexpr (!PLAIN) (MODE == HEAD_DELTA ? xl : ul).b_t(gl, kt * 16, sn0 + i * 16, lane);
 #pragma unroll
                     for (int j = 0; j < 2; ++j) {
                         if constexpr (MODE != HEAD_DELTA) mma(st[i][j], fl, gh[2 * j], gh[2 * j + 1]);
-                        if constexpr (MODE != TIME_MIX) mma(st[i][j], fh, gl[2 * j], gl[2 * j + 1]);
+                        if constexpr (!PLAIN) mma(st[i][j], fh, gl[2 * j], gl[2 * j + 1]);
                         mma(st[i][j], fh, gh[2 * j], gh[2 * j + 1]);
                     }
                 }
             }
-            if constexpr (MODE != TIME_MIX) give(BK, ch);
+            if constexpr (!PLAIN) give(BK, ch);
             put_state((ch + 1) & 1);
             // the read-out: q against the state in front of the chunk, then P U
             take(BQ, ch);
@@ -636,16 +643,16 @@ __global__ void __launch_bounds__(kScanThreads, 1) chunk_scan_kernel(const Recur
                     uint32_t fh[4], fl[4], gh[4], gl[4];
                     ph.a(fh, mt * 16, kt * 16, lane); pl.a(fl, mt * 16, kt * 16, lane);
                     uh.b_t(gh, kt * 16, n0, lane);
-                    if constexpr (MODE != TIME_MIX) ul.b_t(gl, kt * 16, n0, lane);
+                    if constexpr (!PLAIN) ul.b_t(gl, kt * 16, n0, lane);
 #pragma unroll
                     for (int j = 0; j < 2; ++j) {
                         mma(acc[0][j], fl, gh[2 * j], gh[2 * j + 1]);
-                        if constexpr (MODE != TIME_MIX) mma(acc[1][j], fh, gl[2 * j], gl[2 * j + 1]);
+                        if constexpr (!PLAIN) mma(acc[1][j], fh, gl[2 * j], gl[2 * j + 1]);
                         mma(acc[2][j], fh, gh[2 * j], gh[2 * j + 1]);
                     }
                 }
             give(BP, ch);
-            if constexpr (MODE == TIME_MIX) give(BK, ch);   // v lies with k
+            if constexpr (PLAIN) give(BK, ch);   // v lies with k
             const int rows = s.n - ch * C;
 #pragma unroll
             for (int j = 0; j < 2; ++j)
@@ -688,7 +695,8 @@ int32_t launch(const RecurDims& d, const RecurArgs& a, const RecurScratch& sc, c
 
 template <typename F> auto dispatch(const RecurDims& d, F f) {
     auto mode = [&](auto dk) {
-        if (!d.delta) return f(dk, std::integral_constant<int, TIME_MIX>{});
+        if (d.rule == Rule::TimeMix) return f(dk, std::integral_constant<int, TIME_MIX>{});
+        if (d.rule == Rule::Linear) return f(dk, std::integral_constant<int, LINEAR>{});
         return d.channel ? f(dk, std::integral_constant<int, CHANNEL_DELTA>{}) : f(dk, std::integral_constant<int, HEAD_DELTA>{});
     };
     return d.dim <= 64 ? mode(std::integral_constant<int, 64>{}) : mode(std::integral_constant<int, 128>{});

@@ -1,19 +1,58 @@
 // Registry of architectures and the reader of a layer-list model's configuration and tensor names (host code).
+#include <algorithm>
 #include <cmath>
 #include <cstdio>
 #include <cstring>
+#include <tuple>
 
 #include "stack.cuh"
 
 namespace forge {
 
 static const Architecture kArchitectures[] = {
-    {"Bolenex", Norm::DynamicTanh, Arrangement::Parallel, Mlp::ClampedGlu},
-    {"Robazen", Norm::DynamicTanh, Arrangement::Sequential, Mlp::SiluGlu},
+    {"Bolenex", Norm::DynamicTanh, Arrangement::Parallel, Mlp::ClampedGlu, LoopEntry::Project, false},
+    {"Robazen", Norm::DynamicTanh, Arrangement::Sequential, Mlp::SiluGlu, LoopEntry::Project, false},
+    {"Mokatar", Norm::RmsPlusOne, Arrangement::ParallelTwo, Mlp::SiluGlu, LoopEntry::Add, true},
 };
-static const struct { const char* name; Mixer kind; } kMixers[] = {
-    {"latent_attention", Mixer::Latent}, {"delta", Mixer::Delta}, {"channel_delta", Mixer::ChannelDelta}, {"parallel", Mixer::AttnTimeMix},
+// mixers by architecture and the name a layer's "type" gives them
+struct MixerName { const char* architecture; const char* name; Mixer kind; SoftmaxTraits soft; Rotation::Scaling scaling; };
+static SoftmaxTraits traits(QkPost::Scope norm, bool interleaved, bool bias, bool sink) {
+    SoftmaxTraits t;
+    t.qk.norm = norm; t.qk.interleaved = interleaved; t.bias = bias; t.sink = sink;
+    return t;
+}
+static const MixerName kMixers[] = {
+    {"Bolenex", "latent_attention", Mixer::Latent, {}, Rotation::None},
+    {"Robazen", "latent_attention", Mixer::Latent, {}, Rotation::None},
+    {"Robazen", "delta", Mixer::Delta, {}, Rotation::None},
+    {"Robazen", "channel_delta", Mixer::ChannelDelta, {}, Rotation::None},
+    {"Robazen", "parallel", Mixer::AttnTimeMix, {}, Rotation::None},
+    {"Mokatar", "attention", Mixer::Softmax, traits(QkPost::PER_HEAD, true, false, true), Rotation::Yarn},
+    {"Mokatar", "attention_2", Mixer::Softmax, traits(QkPost::WHOLE, false, true, false), Rotation::Linear},
+    {"Mokatar", "gla", Mixer::GatedLinear, {}, Rotation::None},
 };
+
+bool Rotation::operator<(const Rotation& o) const {
+    return std::tie(scaling, dims, base, factor, original, fast, slow) < std::tie(o.scaling, o.dims, o.base, o.factor, o.original, o.fast, o.slow);
+}
+// Yarn: pairs that turn more than `fast` times over the original length keep their frequency, those below `slow` are divided by the
+// factor, with a ramp over the pairs between.
+std::vector<double> Rotation::frequencies() const {
+    std::vector<double> f;
+    for (int i = 0; i < dims / 2; ++i) f.push_back(std::pow(base, -2.0 * i / dims));
+    if (scaling == Linear) for (double& x : f) x /= factor;
+    if (scaling == Yarn && dims > 0) {
+        const double pi = 3.14159265358979323846;
+        auto pair_of = [&](double turns) { return dims * std::log(original / (2 * pi * turns)) / (2 * std::log(base)); };
+        const double lo = std::max(std::floor(pair_of(fast)), 0.0), hi = std::min(std::ceil(pair_of(slow)), double(dims - 1));
+        for (int i = 0; i < dims / 2; ++i) {
+            const double ramp = std::min(1.0, std::max(0.0, (i - lo) / std::max(hi - lo, 0.001)));
+            f[i] = f[i] / factor * ramp + f[i] * (1 - ramp);
+        }
+    }
+    return f;
+}
+double Rotation::magnitude() const { return scaling == Yarn ? 0.1 * std::log(factor) + 1.0 : 1.0; }
 
 namespace {
 
@@ -48,8 +87,9 @@ int32_t parse_latent(const Json* m, float eps, LayerSpec* L) {
     if (d.rot > 0) {
         const Json* rot = m->get("rot");
         FORGE_TRY(need_int(rot, "dims", &d.rot_dims, 0));
-        FORGE_TRY(need_num(rot, "base", &L->rot_base));
-        if (d.rot_dims > d.rot || d.rot_dims % 2 || !(L->rot_base > 0)) { set_error("config.json: rot.dims %d does not fit rot_dim %d", d.rot_dims, d.rot); return FORGE_ERR_SHAPE; }
+        FORGE_TRY(need_num(rot, "base", &L->rot.base));
+        L->rot.dims = d.rot_dims;
+        if (d.rot_dims > d.rot || d.rot_dims % 2 || !(L->rot.base > 0)) { set_error("config.json: rot.dims %d does not fit rot_dim %d", d.rot_dims, d.rot); return FORGE_ERR_SHAPE; }
     }
     d.scale = float(scale); d.eps = eps;
     d.rank_p = pad_to(d.rank, 64); d.rot_p = pad_to(d.rot, 64); d.dim_p = pad_to(d.dim, 64); d.vdim_p = pad_to(d.vdim, 64);
@@ -75,12 +115,14 @@ int32_t parse_delta(const Json* m, float eps, bool channel, LayerSpec* L) {
     FORGE_TRY(need_int(m, "vdim", &d.vdim));
     FORGE_TRY(need_int(m, "conv", &d.taps));
     FORGE_TRY(heads_fit(d.heads, d.groups));
-    d.delta = true; d.channel = channel; d.eps = eps;
+    d.rule = Rule::Delta; d.channel = channel; d.eps = eps;
     d.q_scale = float(1.0 / std::sqrt(double(d.dim)));
     return check_recur(d);
 }
 
-int32_t parse_attn(const Json* m, AttnDims* d) {
+// mask: "size" is the length of chunks, or of a sliding window beside "keep_first" kept tokens
+enum class MaskKind { Chunks, Window };
+int32_t parse_attn(const Json* m, MaskKind kind, AttnDims* d) {
     double scale, cap = 0;
     FORGE_TRY(need_int(m, "heads", &d->heads));
     FORGE_TRY(need_int(m, "kv_heads", &d->groups));
@@ -93,7 +135,10 @@ int32_t parse_attn(const Json* m, AttnDims* d) {
         if (!(cap > 0)) { set_error("config.json: \"softcap\" must be positive"); return FORGE_ERR_SHAPE; }
     }
     const Json* mask = m->get("mask");
-    if (mask && mask->kind != Json::Null) FORGE_TRY(need_int(mask, "size", &d->chunk));
+    if (mask && mask->kind != Json::Null) {
+        FORGE_TRY(need_int(mask, "size", kind == MaskKind::Chunks ? &d->chunk : &d->window));
+        if (kind == MaskKind::Window) FORGE_TRY(need_int(mask, "keep_first", &d->keep, 0));
+    }
     FORGE_TRY(heads_fit(d->heads, d->groups));
     d->scale = float(scale); d->softcap = float(cap);
     d->dim_p = pad_to(d->dim, 64); d->vdim_p = pad_to(d->vdim, 64);
@@ -105,12 +150,64 @@ int32_t parse_attn(const Json* m, AttnDims* d) {
 int32_t parse_pair(const Json* m, float eps, LayerSpec* L) {
     const Json* left = m ? m->get("left") : nullptr;
     const Json* right = m ? m->get("right") : nullptr;
-    FORGE_TRY(parse_attn(left ? left : m, &L->attn));
+    FORGE_TRY(parse_attn(left ? left : m, MaskKind::Chunks, &L->attn));
     RecurDims& d = L->rec;
     FORGE_TRY(need_int(right, "heads", &d.heads));
     FORGE_TRY(need_int(right, "dim", &d.dim));
     d.groups = d.heads; d.vdim = d.dim; d.channel = true; d.eps = eps;
     return check_recur(d);
+}
+
+int32_t parse_rotation(const Json* r, Rotation::Scaling kind, int dim, Rotation* rot) {
+    FORGE_TRY(need_int(r, "dims", &rot->dims, 0));
+    FORGE_TRY(need_num(r, "base", &rot->base));
+    const Json* s = r->get("scaling");
+    if (s && s->kind != Json::Null && kind != Rotation::None) {
+        rot->scaling = kind;
+        FORGE_TRY(need_num(s, "factor", &rot->factor));
+        if (kind == Rotation::Yarn) {
+            FORGE_TRY(need_num(s, "original", &rot->original));
+            FORGE_TRY(need_num(s, "fast", &rot->fast));
+            FORGE_TRY(need_num(s, "slow", &rot->slow));
+        }
+    }
+    const bool yarn = rot->scaling == Rotation::Yarn;
+    if (rot->dims > dim || rot->dims % 2 || !(rot->base > 0) || !(rot->factor > 0) || (yarn && (!(rot->original > 0) || !(rot->fast > 0) || !(rot->slow > 0) || rot->base == 1.0))) {
+        set_error("config.json: \"rot\" does not fit heads of %d", dim);
+        return FORGE_ERR_SHAPE;
+    }
+    return FORGE_OK;
+}
+
+int32_t parse_softmax(const Json* m, float eps, const MixerName& name, LayerSpec* L) {
+    FORGE_TRY(parse_attn(m, MaskKind::Window, &L->attn));
+    if (L->attn.dim > 512) { set_error("attention: head size %d is not supported", L->attn.dim); return FORGE_ERR_UNSUPPORTED; }
+    FORGE_TRY(parse_rotation(m->get("rot"), name.scaling, L->attn.dim, &L->rot));
+    L->soft = name.soft;
+    L->soft.qk.eps = eps; L->soft.qk.rot_dims = L->rot.dims;
+    return FORGE_OK;
+}
+
+int32_t parse_linear(const Json* m, float eps, LayerSpec* L) {
+    RecurDims& d = L->rec;
+    FORGE_TRY(need_int(m, "heads", &d.heads));
+    FORGE_TRY(need_int(m, "dim", &d.dim));
+    FORGE_TRY(need_int(m, "vdim", &d.vdim));
+    FORGE_TRY(need_num(m, "tau", &L->tau));
+    if (!(L->tau > 0)) { set_error("config.json: \"tau\" must be positive"); return FORGE_ERR_SHAPE; }
+    d.groups = d.heads; d.rule = Rule::Linear; d.channel = true; d.eps = eps;
+    d.q_scale = float(1.0 / std::sqrt(double(d.dim)));
+    return check_recur(d);
+}
+
+int32_t parse_experts(const Json* mlp, int layer, LayerSpec* L) {
+    const Json* router = mlp->get("router");
+    FORGE_TRY(need_int(mlp->get("expert"), "ff", &L->ff));
+    FORGE_TRY(need_int(router, "experts", &L->router.experts));
+    FORGE_TRY(need_int(router, "top", &L->router.top));
+    if (L->router.top > L->router.experts) { set_error("layer %d: top %d of %d experts", layer, L->router.top, L->router.experts); return FORGE_ERR_SHAPE; }
+    if (L->router.experts > kMaxExperts) { set_error("layer %d: %d experts are not supported", layer, L->router.experts); return FORGE_ERR_UNSUPPORTED; }
+    return FORGE_OK;
 }
 
 bool same_sizes(const LayerSpec& A, const LayerSpec& B) {
@@ -130,6 +227,20 @@ int32_t stack_parse(const Json& c, StackSpec* s) {
     double eps;
     FORGE_TRY(need_num(c.get("norm"), "eps", &eps));
     s->eps = float(eps);
+    if (s->arch->scaled) {
+        double scale;
+        const Json* e = c.get("embedding");
+        FORGE_TRY(need_num(e, "scale", &scale));
+        s->embed_scale = float(scale);
+        const Json* b = e->get("bigram");
+        if (b && b->kind != Json::Null) {
+            FORGE_TRY(need_int(b, "buckets", &s->buckets));
+            FORGE_TRY(need_int(b, "mul_prev", &s->mul_prev, 0));
+            FORGE_TRY(need_int(b, "mul_cur", &s->mul_cur, 0));
+        }
+        FORGE_TRY(need_num(&c, "logit_scale", &scale));
+        s->logit_scale = float(scale);
+    }
     const Json* layers = c.get("layers");
     if (!layers || layers->kind != Json::Array || layers->items.empty()) { set_error("config.json: \"layers\" must list at least one layer"); return FORGE_ERR_SHAPE; }
     const int n = int(layers->items.size());
@@ -138,9 +249,9 @@ int32_t stack_parse(const Json& c, StackSpec* s) {
         LayerSpec L;
         std::string type;
         FORGE_TRY(need_string(&e, "type", &type));
-        bool known = false;
-        for (const auto& m : kMixers) if (type == m.name) { L.kind = m.kind; known = true; }
-        if (!known || (s->arch->arrangement == Arrangement::Parallel && L.kind != Mixer::Latent)) { set_error("layer %d: mixer \"%s\" is not supported", i, type.c_str()); return FORGE_ERR_UNSUPPORTED; }
+        const MixerName* known = nullptr;
+        for (const MixerName& m : kMixers) if (type == m.name && !strcmp(s->arch->name, m.architecture)) { L.kind = m.kind; known = &m; }
+        if (!known) { set_error("layer %d: mixer \"%s\" is not supported", i, type.c_str()); return FORGE_ERR_UNSUPPORTED; }
         const Json* mx = e.get("mixer");
         if (!mx || mx->kind != Json::Object) { set_error("layer %d: \"mixer\" must be an object", i); return FORGE_ERR_SHAPE; }
         switch (L.kind) {
@@ -148,13 +259,17 @@ int32_t stack_parse(const Json& c, StackSpec* s) {
             case Mixer::Delta: FORGE_TRY(parse_delta(mx, s->eps, false, &L)); break;
             case Mixer::ChannelDelta: FORGE_TRY(parse_delta(mx, s->eps, true, &L)); break;
             case Mixer::AttnTimeMix: FORGE_TRY(parse_pair(mx, s->eps, &L)); break;
+            case Mixer::Softmax: FORGE_TRY(parse_softmax(mx, s->eps, *known, &L)); break;
+            case Mixer::GatedLinear: FORGE_TRY(parse_linear(mx, s->eps, &L)); break;
         }
         const Json* mlp = e.get("mlp");
         if (mlp && mlp->kind != Json::Null) {
             std::string kind;
             FORGE_TRY(need_string(mlp, "kind", &kind));
-            if (kind != "dense") { set_error("layer %d: feed-forward \"%s\" is not supported", i, kind.c_str()); return FORGE_ERR_UNSUPPORTED; }
-            FORGE_TRY(need_int(mlp, "ff", &L.ff));
+            const bool experts = kind == "moe" && s->arch->arrangement == Arrangement::ParallelTwo;
+            if (kind != "dense" && !experts) { set_error("layer %d: feed-forward \"%s\" is not supported", i, kind.c_str()); return FORGE_ERR_UNSUPPORTED; }
+            if (experts) FORGE_TRY(parse_experts(mlp, i, &L));
+            else FORGE_TRY(need_int(mlp, "ff", &L.ff));
             if (s->arch->dense == Mlp::ClampedGlu) {
                 double limit;
                 FORGE_TRY(need_num(mlp, "limit", &limit));
@@ -205,6 +320,7 @@ int32_t stack_find_tensors(const Checkpoint& ck, StackSpec* s, StackTensors* t) 
     };
     auto norm = [&](const std::string& name) -> int32_t {
         FORGE_TRY(get(name, {W}));
+        if (s->arch->norm != Norm::DynamicTanh) return FORGE_OK;
         FORGE_TRY(get(name + ".b", {W}));
         return get(name + ".alpha", {});
     };
@@ -218,7 +334,9 @@ int32_t stack_find_tensors(const Checkpoint& ck, StackSpec* s, StackTensors* t) 
     FORGE_TRY(get("embed", {V, W}));
     FORGE_TRY(get("head", {V, W}));
     FORGE_TRY(norm("final.norm"));
-    if (s->loop_times) { FORGE_TRY(get("loop.in", {W, 2 * W})); FORGE_TRY(get("loop.step", {s->loop_times, W})); }
+    if (s->buckets) FORGE_TRY(get("bigram", {int64_t(s->buckets) + 1, W}));
+    if (s->loop_times && s->arch->loop == LoopEntry::Project) FORGE_TRY(get("loop.in", {W, 2 * W}));
+    if (s->loop_times) FORGE_TRY(get("loop.step", {s->loop_times, W}));
     for (size_t i = 0; i < s->layers.size(); ++i) {
         t->layers.push_back(TensorSet{});
         LayerSpec& L = s->layers[i];
@@ -278,9 +396,32 @@ int32_t stack_find_tensors(const Checkpoint& ck, StackSpec* s, StackTensors* t) 
                 FORGE_TRY(get("mix.right.out", {W}));
                 break;
             }
+            case Mixer::Softmax: {
+                const AttnDims& a = L.attn;
+                const int64_t q = int64_t(a.heads) * a.dim, k = int64_t(a.groups) * a.dim, v = int64_t(a.groups) * a.vdim;
+                const bool whole = L.soft.qk.norm == QkPost::WHOLE;
+                FORGE_TRY(get("mix.q", {q, W})); FORGE_TRY(get("mix.k", {k, W})); FORGE_TRY(get("mix.v", {v, W}));
+                if (L.soft.bias) { FORGE_TRY(get("mix.q.b", {q})); FORGE_TRY(get("mix.k.b", {k})); FORGE_TRY(get("mix.v.b", {v})); }
+                FORGE_TRY(get("mix.q.norm", {whole ? q : a.dim})); FORGE_TRY(get("mix.k.norm", {whole ? k : a.dim}));
+                if (L.soft.sink) FORGE_TRY(get("mix.sink", {a.heads}));
+                FORGE_TRY(get("mix.o", {W, int64_t(a.heads) * a.vdim}));
+                break;
+            }
+            case Mixer::GatedLinear:
+                FORGE_TRY(get("mix.q", {D, W})); FORGE_TRY(get("mix.k", {D, W})); FORGE_TRY(get("mix.v", {HV, W}));
+                FORGE_TRY(rank_of("mix.a1", &L.decay_rank)); FORGE_TRY(get("mix.a2", {D, L.decay_rank})); FORGE_TRY(get("mix.a2.b", {D}));
+                FORGE_TRY(get("mix.g", {HV, W}));
+                FORGE_TRY(get("mix.norm", {r.vdim}));
+                FORGE_TRY(get("mix.o", {W, HV}));
+                break;
         }
-        if (L.ff) {
-            if (s->arch->arrangement == Arrangement::Sequential) FORGE_TRY(norm("norm2"));
+        if (L.ff && s->arch->arrangement != Arrangement::Parallel) FORGE_TRY(norm("norm2"));
+        for (int e = 0; e < L.router.experts; ++e) {
+            const std::string x = "mlp.e" + std::to_string(e);
+            FORGE_TRY(get(x + ".gate", {L.ff, W})); FORGE_TRY(get(x + ".up", {L.ff, W})); FORGE_TRY(get(x + ".down", {W, L.ff}));
+        }
+        if (L.router.experts) { FORGE_TRY(get("mlp.router", {L.router.experts, W})); FORGE_TRY(get("mlp.router.b", {L.router.experts})); }
+        if (L.ff && !L.router.experts) {
             FORGE_TRY(get("mlp.gate", {L.ff, W}));
             FORGE_TRY(get("mlp.up", {L.ff, W}));
             FORGE_TRY(get("mlp.down", {W, L.ff}));
@@ -300,6 +441,7 @@ void stack_fill_info(const StackSpec& s, ForgeCheckpointInfo* out) {
         out->cache_values_per_token += L.cache_row();
         if (L.has_state()) out->state_values_per_sequence += int64_t(L.rec.state_values() + L.rec.ring_values()) + (L.kind == Mixer::AttnTimeMix ? s.width : 0);
     }
+    if (s.buckets) out->state_values_per_sequence += 1;   // the last token
 }
 
 }  // namespace forge

@@ -2,11 +2,13 @@
 // loop, sampling, mixed steps - take such a model like a quantised decoder.
 //
 // A sublayer is a dense product of its normed input (all projections of a mixer in one), the mechanism, and a dense product
-// whose epilogue adds the residual and leaves what the next reader of the stream takes (After): its Dynamic Tanh norm, or the
-// stream itself where a pass of the loop begins.
+// whose epilogue adds the residual and leaves what the next reader of the stream takes (After): its norm, or the stream itself where a
+// pass of the loop begins with a product.
 //   parallel arrangement   the `in` product also holds the feed-forward's rows, and `out` runs over the concatenated columns
 //                          [o | down] of [gated heads | activation], so both sublayers are summed by the product itself;
 //   delta rules            in [q k v | gate | beta | decay] (a second product for two-step gates and decays), recurrence, out;
+//   two parallel norms     the input's columns are [x (1 + w1) | x (1 + w2)], the RMS of the stream is a factor of the product's epilogue; the mixer's rows
+//                          read the first block, the feed-forward's the second; experts: see experts();
 //   attention | time mix   the input's columns are [h | five shifted mixes] and every row of `in` reads the block it belongs to; keys
 //                          and values go from the epilogue into the cache; one product with both outputs, then the sum of their norms.
 #include <algorithm>
@@ -21,10 +23,10 @@
 // ------------------------------------------------------------------------------------------------ structures
 namespace forge {
 
-struct DytNorm { float* w = nullptr; float* b = nullptr; float alpha = 0.f; };
+struct StreamNorm { float* w = nullptr; float* b = nullptr; float alpha = 0.f; };   // RMS norm: w = one plus the weight
 
 struct LayerWeights {
-    DytNorm norm1, norm2;
+    StreamNorm norm1, norm2;
     DenseWeight in, out;
     DenseWeight ff_in, ff_out;    // sequential arrangement
     // latent attention
@@ -42,25 +44,33 @@ struct LayerWeights {
     int k_row = 0, v_row = 0, hg_row = 0, r_row = 0, rk_row = 0, rv_row = 0;
     int out_r_row = 0;            // first row of the second mixer in `out`; it reads the columns behind the first one's
     float *mu = nullptr, *norm_l = nullptr, *norm_r = nullptr;
+    // attention with normed queries and keys (k_row, v_row as above)
+    float *q_norm = nullptr, *k_norm = nullptr, *sink = nullptr, *q_bias = nullptr, *k_bias = nullptr, *v_bias = nullptr;
+    // experts: their columns of `out` follow the heads', ff_k apart
+    int router_row = 0, ff_k = 0;
+    float* router_bias = nullptr;
+    DenseWeight experts;          // gate and up rows, pairs interleaved, expert by expert expert_rows apart
+    int expert_rows = 0;
 };
 
 struct StackModel {
     StackSpec spec;
     int dtype = FORGE_BF16;
     int width_p = 0;
-    void* embed = nullptr;
+    void *embed = nullptr, *bigram = nullptr;
     std::vector<LayerWeights> w;                       // by layer; empty for a layer with weights_of
-    DytNorm final_norm;
+    StreamNorm final_norm;
     DenseWeight head, loop_in;
     float* loop_step = nullptr;                        // [times][width]
-    std::map<std::pair<double, int>, std::pair<int, float*>> ropes;   // (base, dims) -> positions, table
+    std::map<Rotation, std::pair<int, float*>> ropes;   // -> positions, table
     int rope_positions = 0;
     DenseScratch scratch;
     // step buffers, grown on demand (scratch_gen of the model counts the moves)
     struct Buf { void* p = nullptr; size_t cap = 0; };
-    Buf x, h, cat, proj, gate, mid, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, hgate, decay, beta, low, conv, unit, o, pair, place, c_half, c_f32, sel, logits, meta;
+    Buf x, h, cat, proj, gate, mid, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, hgate, decay, beta, low, conv, unit, o, pair, place, c_half, c_f32, sel, logits, meta, x0, sums, sum1, router, route, e_in, e_act, e_out;
     std::vector<Buf*> all() {
-        return {&x, &h, &cat, &proj, &gate, &mid, &q, &part, &ml, &ctx_c, &ctx_r, &ctx_k, &ctx_v, &hgate, &decay, &beta, &low, &conv, &unit, &o, &pair, &place, &c_half, &c_f32, &sel, &logits, &meta};
+        return {&x, &h, &cat, &proj, &gate, &mid, &q, &part, &ml, &ctx_c, &ctx_r, &ctx_k, &ctx_v, &hgate, &decay, &beta, &low, &conv, &unit, &o, &pair, &place, &c_half, &c_f32, &sel, &logits, &meta,
+                &x0, &sums, &sum1, &router, &route, &e_in, &e_act, &e_out};
     }
     const LayerWeights& weights(int layer) const { return w[spec.layers[layer].weights_of >= 0 ? spec.layers[layer].weights_of : layer]; }
 };
@@ -71,6 +81,7 @@ struct StackCache {
     struct Run { void* pool = nullptr; alignas(64) unsigned char map[128]; float* state = nullptr; void* ring = nullptr; void* prev = nullptr; };
     std::vector<Run> runs;
     int splits = 1;     // of a captured decode step
+    uint32_t* prev_token = nullptr;   // by sequence: its last token (bigram embeddings)
 };
 
 namespace {
@@ -135,7 +146,12 @@ struct Image {
     int32_t load(ForgeModel* m, DenseWeight* w, bool row_reads = false) const { return load_dense(m, w, N, K, dtype, img, row_reads); }
 };
 
-int32_t load_norm(ForgeModel* m, DytNorm* n, const TensorSet& t, const std::string& name) {
+int32_t load_norm(ForgeModel* m, StreamNorm* n, const TensorSet& t, const std::string& name) {
+    if (m->stack->spec.arch->norm == Norm::RmsPlusOne) {
+        std::vector<float> w(size_t(t.at(name)->count()));
+        for (size_t i = 0; i < w.size(); ++i) w[i] = 1.f + t.at(name)->at(i);
+        return upload_values(m, &n->w, w);
+    }
     n->alpha = t.at(name + ".alpha")->at(0);
     FORGE_TRY(upload_f32(m, &n->w, *t.at(name)));
     return upload_f32(m, &n->b, *t.at(name + ".b"));
@@ -250,6 +266,77 @@ int32_t load_pair(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWe
     return upload_f32(m, &w->norm_r, *t.at("mix.right.out"));
 }
 
+// Side by side behind two norms: the feed-forward's rows of `in` (or the router's) behind the mixer's `rows`, and `out` over [heads | feed-forward].
+// fill_in puts the mixer's rows.
+template <typename F>
+int32_t load_two_norms(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w, int rows, int heads_cols, F fill_in) {
+    StackModel& S = *m->stack;
+    const int E = L.router.experts;
+    w->glu_row = w->router_row = pad_to(rows, 128);   // a tile of rows reads one block of the activations
+    Image in(E ? w->router_row + E : L.ff ? w->glu_row + 2 * L.ff : rows, S.width_p, S.dtype);
+    fill_in(in);
+    if (E) in.put(t.at("mlp.router"), w->router_row);
+    else if (L.ff) { in.put(t.at("mlp.gate"), w->glu_row, 2); in.put(t.at("mlp.up"), w->glu_row + 1, 2); }
+    FORGE_TRY(in.load(m, &w->in));
+    w->heads_k = pad_to(heads_cols, kDensePad);
+    w->ff_k = pad_to(L.ff, kDensePad);
+    Image out(S.spec.width, w->heads_k + std::max(1, E) * w->ff_k, S.dtype);
+    out.put(t.at("mix.o"), 0);
+    if (E) {
+        FORGE_TRY(upload_f32(m, &w->router_bias, *t.at("mlp.router.b")));
+        w->expert_rows = pad_to(2 * L.ff, 128);
+        Image ex(E * w->expert_rows, S.width_p, S.dtype);
+        for (int e = 0; e < E; ++e) {
+            const std::string x = "mlp.e" + std::to_string(e);
+            ex.put(t.at(x + ".gate"), e * w->expert_rows, 2);
+            ex.put(t.at(x + ".up"), e * w->expert_rows + 1, 2);
+            out.put(t.at(x + ".down"), 0, 1, w->heads_k + e * w->ff_k);
+        }
+        FORGE_TRY(ex.load(m, &w->experts));
+    } else if (L.ff) out.put(t.at("mlp.down"), 0, 1, w->heads_k);
+    return out.load(m, &w->out);
+}
+
+int32_t load_softmax(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
+    const AttnDims& a = L.attn;
+    w->k_row = pad_to(a.heads * a.dim, kSegAlign);
+    w->v_row = w->k_row + pad_to(a.groups * a.dim, kSegAlign);
+    FORGE_TRY(upload_f32(m, &w->q_norm, *t.at("mix.q.norm")));
+    FORGE_TRY(upload_f32(m, &w->k_norm, *t.at("mix.k.norm")));
+    if (L.soft.sink) FORGE_TRY(upload_f32(m, &w->sink, *t.at("mix.sink")));
+    else FORGE_TRY(upload_values(m, &w->sink, std::vector<float>(size_t(a.heads), 0.f)));
+    if (L.soft.bias) {
+        FORGE_TRY(upload_f32(m, &w->q_bias, *t.at("mix.q.b")));
+        FORGE_TRY(upload_f32(m, &w->k_bias, *t.at("mix.k.b")));
+        FORGE_TRY(upload_f32(m, &w->v_bias, *t.at("mix.v.b")));
+    }
+    return load_two_norms(m, L, t, w, w->v_row + a.groups * a.vdim, a.heads * a.vdim, [&](Image& in) {
+        in.put(t.at("mix.q"), 0); in.put(t.at("mix.k"), w->k_row); in.put(t.at("mix.v"), w->v_row);
+    });
+}
+
+int32_t load_linear(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
+    StackModel& S = *m->stack;
+    const RecurDims& d = L.rec;
+    const int D = d.qk(), HV = d.heads * d.vdim;
+    // the logarithm of a decay, log(sigmoid(z)) / tau, is -softplus(-z) / tau: the second step and its bias are kept negated
+    std::vector<float> bias(size_t(D), 0.f);
+    for (int i = 0; i < D; ++i) bias[i] = -t.at("mix.a2.b")->at(size_t(i));
+    FORGE_TRY(upload_values(m, &w->decay_add, bias));
+    FORGE_TRY(upload_values(m, &w->decay_mul, std::vector<float>(size_t(D), float(1.0 / L.tau))));
+    FORGE_TRY(upload_f32(m, &w->head_norm, *t.at("mix.norm")));
+    Image low(D, pad_to(L.decay_rank, kDensePad), S.dtype);
+    low.put(t.at("mix.a2"), 0);
+    for (size_t i = dense_size(S.dtype) - 1; i < low.img.size(); i += dense_size(S.dtype)) low.img[i] ^= 0x80;   // sign bits
+    FORGE_TRY(low.load(m, &w->low, true));
+    w->gate_row = pad_to(d.channels(), kSegAlign);
+    w->decay_row = w->gate_row + pad_to(HV, kSegAlign);
+    return load_two_norms(m, L, t, w, w->decay_row + L.decay_rank, HV, [&](Image& in) {
+        in.put(t.at("mix.q"), 0); in.put(t.at("mix.k"), D); in.put(t.at("mix.v"), 2 * D);
+        in.put(t.at("mix.g"), w->gate_row); in.put(t.at("mix.a1"), w->decay_row);
+    });
+}
+
 int32_t load_layer(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
     StackModel& S = *m->stack;
     FORGE_TRY(load_norm(m, &w->norm1, t, "norm1"));
@@ -257,7 +344,10 @@ int32_t load_layer(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerW
         case Mixer::Latent: FORGE_TRY(load_latent(m, L, t, w)); break;
         case Mixer::Delta: case Mixer::ChannelDelta: FORGE_TRY(load_delta(m, L, t, w)); break;
         case Mixer::AttnTimeMix: FORGE_TRY(load_pair(m, L, t, w)); break;
+        case Mixer::Softmax: FORGE_TRY(load_softmax(m, L, t, w)); break;
+        case Mixer::GatedLinear: FORGE_TRY(load_linear(m, L, t, w)); break;
     }
+    if (L.ff && S.spec.arch->arrangement == Arrangement::ParallelTwo) FORGE_TRY(load_norm(m, &w->norm2, t, "norm2"));
     if (L.ff && S.spec.arch->arrangement == Arrangement::Sequential) {
         FORGE_TRY(load_norm(m, &w->norm2, t, "norm2"));
         Image in(2 * L.ff, S.width_p, S.dtype), out(S.spec.width, pad_to(L.ff, kDensePad), S.dtype);
@@ -269,18 +359,18 @@ int32_t load_layer(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerW
     return FORGE_OK;
 }
 
-// rotation tables of every (base, dims) for at least n positions
+// rotation tables for at least n positions
 int32_t ensure_rope(ForgeModel* m, int n) {
     StackModel& S = *m->stack;
     if (n <= S.rope_positions) return FORGE_OK;
     n = pad_to(n, 1024);
     FORGE_CUDA(cudaStreamSynchronize(m->stream));
     for (const LayerSpec& L : S.spec.layers) {
-        if (!L.has_latent()) continue;
-        auto& e = S.ropes[{L.rot_base, L.mix.rot_dims}];
+        if (!L.has_rotation()) continue;
+        auto& e = S.ropes[L.rot];
         if (e.first >= n) continue;
-        std::vector<float> tab(std::max<size_t>(1, size_t(n) * L.mix.rot_dims));
-        FORGE_TRY(rope_half_table(tab.data(), n, L.mix.rot_dims, L.rot_base));
+        std::vector<float> tab(std::max<size_t>(1, size_t(n) * L.rot.dims));
+        FORGE_TRY(rope_table(tab.data(), n, L.rot.frequencies(), L.rot.magnitude()));
         float* p = nullptr;
         FORGE_CUDA(cudaMalloc(&p, tab.size() * 4));
         if (e.second) cudaFree(e.second);
@@ -309,6 +399,11 @@ int32_t grow(ForgeModel* m, StackModel::Buf& b, size_t bytes) {
 
 bool tensor_core_rows(const StackModel& S, const LatentDims& d) { return S.dtype == FORGE_BF16 && latent_decode_tc_supported(d); }
 
+// A step of few tokens runs an expert over all of them and takes the experts' columns of `out` from a list; otherwise tokens are dealt to the experts.
+bool few_tokens(const StackModel& S, const LayerWeights& w, int rows) { return dense_listed_supported(w.out, rows); }
+// values of a row in front of `out`
+int mid_columns(const StackModel& S, const LayerSpec& L, const LayerWeights& w, int rows) { return L.router.experts && !few_tokens(S, w, rows) ? w.heads_k : w.out.K; }
+
 // splits of the row attention: at most one CTA per SM over all rows and head groups, no more than there are pages
 int row_splits(const StackModel& S, int rows, int pages) {
     int groups = 1;
@@ -320,7 +415,7 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
     StackModel& S = *m->stack;
     const size_t es = dense_size(S.dtype), r = size_t(rows), W = size_t(S.spec.width), WP = size_t(S.width_p);
     // bytes, rows times the widest layer
-    size_t h = WP * es, proj = 0, gate = 0, mid = 0, q = 0, part = 0, heads = 0, cc = 0, cr = 0, ck = 0, cv = 0, hgate = 0, decay = 0, beta = 0, low = 0, conv = 0, unit = 0, o = 0, pair = 0;
+    size_t h = WP * es, proj = 0, gate = 0, mid = 0, q = 0, part = 0, heads = 0, cc = 0, cr = 0, ck = 0, cv = 0, hgate = 0, decay = 0, beta = 0, low = 0, conv = 0, unit = 0, o = 0, pair = 0, router = 0, route = 0, e_in = 0, e_act = 0, e_out = 0;
     ChunkBytes cb{0, 0};
     auto most = [](size_t& a, size_t b) { a = std::max(a, b); };
     size_t n_max = size_t(S.head.N);
@@ -328,7 +423,20 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
         const LayerSpec& L = S.spec.layers[i];
         const LayerWeights& w = S.weights(int(i));
         for (const DenseWeight* d : {&w.in, &w.out, &w.kv, &w.low, &w.ff_in, &w.ff_out}) most(n_max, size_t(d->N));
-        most(mid, r * std::max(w.out.K, w.ff_out.K) * es);
+        most(mid, r * std::max(mid_columns(S, L, w, rows), w.ff_out.K) * es);
+        if (S.spec.arch->arrangement == Arrangement::ParallelTwo) most(h, 2 * WP * es);
+        if (L.router.experts) {
+            const size_t pairs = r * L.router.top;
+            most(mid, std::min<size_t>(r, kScaleRows) * w.out.K * es);
+            most(router, r * L.router.experts * 4);
+            most(route, route_bytes(L.router, rows));
+            if (!few_tokens(S, w, rows)) { most(e_in, pairs * WP * es); most(e_act, pairs * w.ff_k * es); most(e_out, pairs * W * 4); }
+        }
+        if (L.kind == Mixer::Softmax) {
+            most(proj, r * w.v_row * 4);
+            most(q, r * L.attn.heads * L.attn.dim_p * es);
+            continue;
+        }
         if (L.has_latent()) {
             const LatentDims& d = L.mix;
             most(proj, r * w.g_row * 4);
@@ -352,8 +460,8 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
             const ChunkBytes b = recur_chunk_bytes(d);
             most(cb.half, chunks * b.half); most(cb.f32, chunks * b.f32);
         }
-        if (d.delta && seg_rows) { most(conv, r * d.channels() * es); most(unit, r * 2 * d.groups * 4); }
-        if (L.has_attn()) {
+        if (d.rule == Rule::Delta && seg_rows) { most(conv, r * d.channels() * es); most(unit, r * 2 * d.groups * 4); }
+        if (L.kind == Mixer::AttnTimeMix) {
             most(h, (1 + kMixes) * WP * es);
             most(q, r * L.attn.heads * L.attn.dim_p * es);
             most(hgate, r * L.attn.heads * 4);
@@ -363,10 +471,13 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
     }
     FORGE_TRY(grow(m, S.x, r * W * 4));
     FORGE_TRY(grow(m, S.h, r * h));
-    if (S.spec.loop_times) FORGE_TRY(grow(m, S.cat, r * 2 * WP * es));
+    if (S.loop_in.N) FORGE_TRY(grow(m, S.cat, r * 2 * WP * es));
+    if (S.spec.adds_loop()) FORGE_TRY(grow(m, S.x0, r * W * 4));
+    if (S.spec.arch->norm == Norm::RmsPlusOne) { FORGE_TRY(grow(m, S.sums, r * ((W + 31) / 32) * 4)); FORGE_TRY(grow(m, S.sum1, r * 4)); }
     FORGE_TRY(grow(m, S.place, r * sizeof(int32_t)));
     const std::pair<StackModel::Buf*, size_t> sizes[] = {{&S.proj, proj}, {&S.gate, gate}, {&S.mid, mid}, {&S.q, q}, {&S.part, part}, {&S.ml, heads}, {&S.hgate, hgate}, {&S.decay, decay},
-        {&S.beta, beta}, {&S.low, low}, {&S.conv, conv}, {&S.unit, unit}, {&S.o, o}, {&S.pair, pair}, {&S.c_half, cb.half}, {&S.c_f32, cb.f32}, {&S.ctx_c, cc}, {&S.ctx_r, cr}, {&S.ctx_k, ck}, {&S.ctx_v, cv}};
+        {&S.beta, beta}, {&S.low, low}, {&S.conv, conv}, {&S.unit, unit}, {&S.o, o}, {&S.pair, pair}, {&S.c_half, cb.half}, {&S.c_f32, cb.f32}, {&S.ctx_c, cc}, {&S.ctx_r, cr}, {&S.ctx_k, ck}, {&S.ctx_v, cv},
+        {&S.router, router}, {&S.route, route}, {&S.e_in, e_in}, {&S.e_act, e_act}, {&S.e_out, e_out}};
     for (const auto& e : sizes) FORGE_TRY(grow(m, *e.first, e.second));
     // one ticket per output tile of the largest product (128 rows x at least 16 tokens)
     const size_t tiles = ((n_max + 127) / 128) * std::max<size_t>(1, (size_t(std::max(rows, ctx_rows)) + 127) / 128);
@@ -385,6 +496,7 @@ struct Step {
     int ones = 0;                            // rows [0, ones): one token of its sequence each
     int single = 0, splits = 1;              // rows [0, single): attention row by row; the rest are prompt rows
     int max_keys = 1;                        // most keys a row of [0, single) has
+    int scale_rows = 0;                      // most rows of a product that takes scales
     SegTable segs;                           // the rows [ones, n)
     const PromptTile* tiles = nullptr; int n_tiles = 0;
     const int32_t* ctx_pages = nullptr; int ctx_rows = 0;
@@ -394,6 +506,17 @@ struct Step {
 
 char* at(void* p, size_t elems, int dtype) { return static_cast<char*>(p) + elems * dense_size(dtype); }
 
+// the scales of an RMS norm's tokens
+RowScale stream_scale(const StackModel& S, int rows) {
+    RowScale r;
+    if (S.spec.arch->norm != Norm::RmsPlusOne) return r;
+    const bool summed = rows > kScaleRows;
+    r.sums = static_cast<const float*>(summed ? S.sum1.p : S.sums.p);
+    r.parts = summed ? 1 : (S.spec.width + 31) / 32;
+    r.inv_n = 1.0f / float(S.spec.width); r.eps = S.spec.eps;
+    return r;
+}
+
 // The launch sequence of one step.
 struct Sequence {
     ForgeModel* m;
@@ -402,51 +525,84 @@ struct Sequence {
     StackModel& S;
     cudaStream_t st;
     const int n, W, WP, dt;
-    const bool sequential;
+    const bool sequential, two_norms;
     Sequence(ForgeModel* m_, ForgeKV* kv_, const Step& s_)
-        : m(m_), kv(kv_), s(s_), S(*m_->stack), st(m_->stream), n(s_.rows.n), W(S.spec.width), WP(S.width_p), dt(S.dtype), sequential(S.spec.arch->arrangement == Arrangement::Sequential) {}
+        : m(m_), kv(kv_), s(s_), S(*m_->stack), st(m_->stream), n(s_.rows.n), W(S.spec.width), WP(S.width_p), dt(S.dtype), sequential(S.spec.arch->arrangement == Arrangement::Sequential),
+          two_norms(S.spec.arch->arrangement == Arrangement::ParallelTwo) {}
 
     int32_t gemm(const DenseWeight& w, const void* act, int ld, const DenseOut& o, int rows) { return dense_gemm(w, act, ld, rows, o, S.scratch, m->d_err, st); }
     int32_t gemm(const DenseWeight& w, const void* act, int ld, const DenseOut& o) { return gemm(w, act, ld, o, n); }
 
-    After dyt(const DytNorm& d, int ld) { After a; a.kind = AFTER_DYT; a.alpha = d.alpha; a.w = d.w; a.b = d.b; a.dst = S.h.p; a.ld = ld; return a; }
-    int h_ld(int layer) const { return S.spec.layers[layer].has_attn() ? (1 + kMixes) * WP : WP; }
-    After norm1(int layer) { return dyt(S.weights(layer).norm1, h_ld(layer)); }
+    After norm(const StreamNorm& d, int ld) {
+        After a;
+        a.dst = S.h.p; a.ld = ld; a.w = d.w;
+        if (rms()) { a.kind = AFTER_RMS; a.sums = static_cast<float*>(S.sums.p); a.parts = (W + 31) / 32; }
+        else { a.kind = AFTER_DYT; a.alpha = d.alpha; a.b = d.b; }
+        return a;
+    }
+    bool rms() const { return S.spec.arch->norm == Norm::RmsPlusOne; }
+    int h_ld(int layer) const { return S.spec.layers[layer].kind == Mixer::AttnTimeMix ? (1 + kMixes) * WP : two_norms ? 2 * WP : WP; }
+    After norm1(int layer) {
+        After a = norm(S.weights(layer).norm1, h_ld(layer));
+        if (two_norms && S.spec.layers[layer].ff) { a.w2 = S.weights(layer).norm2.w; a.col2 = WP; }
+        return a;
+    }
     // what the first reader of the stream in front of run i takes
     After into(size_t i) {
-        if (i == S.spec.runs.size()) return dyt(S.final_norm, WP);
-        if (S.spec.runs[i].pass < 0) return norm1(S.spec.runs[i].layer);
+        if (i == S.spec.runs.size()) return norm(S.final_norm, WP);
+        const int pass = S.spec.runs[i].pass;
+        if (pass < 0) return norm1(S.spec.runs[i].layer);
         After a;
+        if (S.spec.adds_loop()) {
+            a = norm1(S.spec.runs[i].layer);
+            a.plus = S.loop_step + size_t(pass) * W;
+            if (pass > 0) a.again = static_cast<float*>(S.x0.p);
+            if (s.trace && i > 0) a.keep = s.trace + (i - 1) * s.trace_stride;
+            return a;
+        }
         a.kind = AFTER_CAST; a.dst = S.cat.p; a.ld = 2 * WP;
         return a;
     }
     static void resid(DenseOut* o, float* x, int W, const After& after) { o->add(SEG_RESID, 0, W, x, W).after = after; }
     float* x() { return static_cast<float*>(S.x.p); }
+    // RMS norms: the tokens' scales from the sums that the stream's last writer left
+    int32_t stats() { return rms() && s.scale_rows > kScaleRows ? row_sums(static_cast<float*>(S.sum1.p), static_cast<float*>(S.sums.p), n, (W + 31) / 32, st) : FORGE_OK; }
+    RowScale scale() const { return stream_scale(S, s.scale_rows); }
 
     int32_t run() {
         EmbedArgs e;
         e.x = x(); e.table = S.embed; e.tokens = s.tokens; e.width = W; e.width_p = WP;
         e.after = into(0);
-        if (S.spec.loop_times) { e.x0 = at(S.cat.p, size_t(WP), dt); e.x0_ld = 2 * WP; }
+        if (S.loop_in.N) { e.x0 = at(S.cat.p, size_t(WP), dt); e.x0_ld = 2 * WP; }
+        if (S.spec.adds_loop()) e.x0_f32 = static_cast<float*>(S.x0.p);
+        e.scale = S.spec.embed_scale;
+        if (S.spec.buckets) {
+            e.bigram = S.bigram; e.buckets = uint32_t(S.spec.buckets); e.mul_prev = uint32_t(S.spec.mul_prev); e.mul_cur = uint32_t(S.spec.mul_cur);
+            e.prev = kv->stack->prev_token;
+        }
         e.place = static_cast<int32_t*>(S.place.p); e.rows = s.rows; e.hist = s.hist; e.step = s.step;
         FORGE_TRY(embed_rows(e, dt, st));
+        if (S.spec.buckets) FORGE_TRY(keep_tokens(kv->stack->prev_token, s.tokens, s.rows, st));
         for (size_t i = 0; i < S.spec.runs.size(); ++i) {
             const LayerRun& r = S.spec.runs[i];
             const LayerSpec& L = S.spec.layers[r.layer];
             const LayerWeights& w = S.weights(r.layer);
             StackCache::Run& run = kv->stack->runs[i];
-            if (r.pass >= 0) {
+            if (r.pass >= 0 && !S.spec.adds_loop()) {
                 DenseOut o;
                 OutSeg& g = o.add(SEG_RESID, 0, W, x(), W);
                 g.fresh = true; g.add = S.loop_step + size_t(r.pass) * W; g.after = norm1(r.layer);
                 FORGE_TRY(gemm(S.loop_in, S.cat.p, 2 * WP, o));
             }
             const bool ff = sequential && L.ff;
-            const After after = ff ? dyt(w.norm2, WP) : into(i + 1);
+            const After after = ff ? norm(w.norm2, WP) : into(i + 1);
+            FORGE_TRY(stats());
             switch (L.kind) {
                 case Mixer::Latent: FORGE_TRY(latent(L, w, run, after)); break;
                 case Mixer::Delta: case Mixer::ChannelDelta: FORGE_TRY(delta(L, w, run, after)); break;
                 case Mixer::AttnTimeMix: FORGE_TRY(pair(L, w, run, after)); break;
+                case Mixer::Softmax: FORGE_TRY(softmax(L, w, run, after)); break;
+                case Mixer::GatedLinear: FORGE_TRY(linear(L, w, run, after)); break;
             }
             if (ff) {
                 DenseOut in, out;
@@ -455,16 +611,16 @@ struct Sequence {
                 resid(&out, x(), W, into(i + 1));
                 FORGE_TRY(gemm(w.ff_out, S.mid.p, w.ff_out.K, out));
             }
-            if (s.trace) FORGE_CUDA(cudaMemcpyAsync(s.trace + i * s.trace_stride, S.x.p, sizeof(float) * n * W, cudaMemcpyDeviceToDevice, st));
+            if (s.trace && !after.keep) FORGE_CUDA(cudaMemcpyAsync(s.trace + i * s.trace_stride, S.x.p, sizeof(float) * n * W, cudaMemcpyDeviceToDevice, st));
         }
-        return FORGE_OK;
+        return stats();
     }
 
     int32_t latent(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
         const LatentDims& d = L.mix;
         const int ldp = w.g_row, gate_ld = d.heads * d.vdim, mid_ld = w.out.K, ff = sequential ? 0 : L.ff;
         float* proj = static_cast<float*>(S.proj.p);
-        const float* rope = S.ropes.at({L.rot_base, d.rot_dims}).second;
+        const float* rope = S.ropes.at(L.rot).second;
         {
             DenseOut o;
             o.add(SEG_F32, 0, w.q_rows, proj, ldp);
@@ -525,6 +681,115 @@ struct Sequence {
         a.norm = w.head_norm;
         a.gate = S.gate.p; a.gate_ld = d.heads * d.vdim;
         return a;
+    }
+
+    // rows of `in` that the feed-forward of a layer with two norms takes, or its router
+    void feed_forward_rows(DenseOut* o, const LayerSpec& L, const LayerWeights& w) {
+        if (L.router.experts) {
+            OutSeg& g = o->add(SEG_F32, w.router_row, L.router.experts, S.router.p, L.router.experts);
+            g.add = w.router_bias; g.act_col = WP;
+        } else if (L.ff) o->add(SEG_SILU_GLU, w.glu_row, 2 * L.ff, at(S.mid.p, w.heads_k, dt), w.out.K).act_col = WP;
+    }
+    // x += W_o (heads in front of `out`) + feed-forward
+    int32_t two_norms_out(const LayerSpec& L, const LayerWeights& w, const After& after) {
+        if (L.router.experts) return experts(L, w, after);
+        DenseOut o;
+        resid(&o, x(), W, after);
+        return gemm(w.out, S.mid.p, w.out.K, o);
+    }
+    // Few tokens: every expert that is used runs over all of them (a token that does not use it gets zeros) into its columns in front of `out`, which
+    // then is one product over the heads' columns and those of the experts that are used.  Otherwise the tokens are gathered expert by expert.
+    int32_t experts(const LayerSpec& L, const LayerWeights& w, const After& after) {
+        const RouteTables t = route_tables(S.route.p, L.router, n);
+        const float* logits = static_cast<const float*>(S.router.p);
+        GroupTable table;
+        GroupShape shape;
+        shape.rows = 2 * L.ff; shape.group_rows = w.expert_rows;
+        DenseOut in;
+        in.scale = scale();
+        if (few_tokens(S, w, n)) {
+            FORGE_TRY(route_few(L.router, logits, n, t, &table, st));
+            shape.group_dst = size_t(w.ff_k);
+            in.add(SEG_SILU_GLU, 0, 2 * L.ff, at(S.mid.p, w.heads_k, dt), w.out.K);
+            FORGE_TRY(dense_gemm_groups(w.experts, shape, table, at(S.h.p, WP, dt), 2 * WP, n, in, m->d_err, st));
+            DenseOut out;
+            resid(&out, x(), W, after);
+            return dense_gemm_listed(w.out, w.heads_k, w.ff_k, table, S.mid.p, w.out.K, n, out, m->d_err, st);
+        }
+        {
+            DenseOut o;
+            resid(&o, x(), W, After{});
+            FORGE_TRY(gemm(w.out.columns(0, w.heads_k), S.mid.p, w.heads_k, o));
+        }
+        FORGE_TRY(route_slots(L.router, logits, n, t, &table, st));
+        const int pairs = n * L.router.top;
+        FORGE_TRY(gather_act_rows(S.e_in.p, at(S.h.p, WP, dt), 2 * WP, t.row, pairs, WP, dt, st));
+        in.scale.row = t.row;
+        in.add(SEG_SILU_GLU, 0, 2 * L.ff, S.e_act.p, w.ff_k);
+        FORGE_TRY(dense_gemm_groups(w.experts, shape, table, S.e_in.p, WP, pairs, in, m->d_err, st));
+        DenseOut down;
+        down.add(SEG_F32, 0, W, S.e_out.p, W);
+        GroupShape cols;
+        cols.rows = W; cols.group_cols = w.ff_k;
+        table.weight = nullptr;
+        FORGE_TRY(dense_gemm_groups(w.out.columns(w.heads_k, w.ff_k), cols, table, S.e_act.p, w.ff_k, pairs, down, m->d_err, st));
+        return add_experts(x(), static_cast<const float*>(S.e_out.p), L.router, t, n, W, after, dt, st);
+    }
+
+    int32_t softmax(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
+        const AttnDims& a = L.attn;
+        const int ldp = w.v_row, mid_ld = mid_columns(S, L, w, n);
+        float* proj = static_cast<float*>(S.proj.p);
+        const int32_t* place = static_cast<const int32_t*>(S.place.p);
+        {
+            DenseOut o;
+            o.scale = scale();
+            o.add(SEG_F32, 0, a.heads * a.dim, proj, ldp).add = w.q_bias;
+            o.add(SEG_F32, w.k_row, a.groups * a.dim, proj + w.k_row, ldp).add = w.k_bias;
+            OutSeg& v = o.add(SEG_CAST, w.v_row, a.groups * a.vdim, at(run.pool, size_t(a.groups) * a.dim_p, dt), a.row());
+            v.group = a.vdim; v.group_ld = a.vdim_p; v.place = place; v.add = w.v_bias;
+            feed_forward_rows(&o, L, w);
+            FORGE_TRY(gemm(w.in, S.h.p, 2 * WP, o));
+        }
+        FORGE_TRY(qk_post(a, L.soft.qk, dt, proj, ldp, w.k_row, w.q_norm, w.k_norm, S.ropes.at(L.rot).second, S.q.p, run.pool, place, s.rows, st));
+        StepRows single = s.rows;
+        single.n = s.single;
+        FORGE_TRY(attn_rows(a, dt, S.q.p, run.pool, nullptr, w.sink, S.mid.p, mid_ld, single, a.most_keys(s.max_keys), st));
+        if (n > s.single) {
+            PromptAttnArgs p;
+            p.q = at(S.q.p, size_t(s.single) * a.heads * a.dim_p, dt); p.k = run.pool; p.v = at(run.pool, size_t(a.groups) * a.dim_p, dt);
+            p.sink = w.sink;
+            p.out = at(S.mid.p, size_t(s.single) * mid_ld, dt); p.out_ld = mid_ld;
+            p.q_rows = n - s.single; p.ctx_rows = kv->num_pages * FORGE_KV_PAGE; p.tiles = s.tiles; p.n_tiles = s.n_tiles;
+            p.pages = s.ctx_pages; p.page_row = a.row(); p.err = m->d_err;
+            FORGE_TRY(attn_prefill_kv(PromptDims(a), p, st));
+        }
+        return two_norms_out(L, w, after);
+    }
+
+    int32_t linear(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
+        const RecurDims& d = L.rec;
+        const int D = d.qk(), HV = d.heads * d.vdim;
+        RecurArgs a = recur_args(d, w, run);
+        {
+            DenseOut o;
+            o.scale = scale();
+            o.add(SEG_CAST, 0, d.channels(), S.proj.p, d.channels());
+            o.add(SEG_SILU, w.gate_row, HV, S.gate.p, HV);
+            o.add(SEG_CAST, w.decay_row, L.decay_rank, S.low.p, w.low.K);
+            feed_forward_rows(&o, L, w);
+            FORGE_TRY(gemm(w.in, S.h.p, 2 * WP, o));
+        }
+        if (all_ones()) two_step(&a, w, w.low.K);
+        else {
+            DenseOut lo;
+            OutSeg& g = lo.add(SEG_DECAY, 0, D, S.decay.p, D);
+            g.mul = w.decay_mul; g.add = w.decay_add;
+            FORGE_TRY(gemm(w.low, S.low.p, w.low.K, lo));
+        }
+        a.out = S.mid.p; a.out_ld = mid_columns(S, L, w, n);
+        FORGE_TRY(recur(d, a));
+        return two_norms_out(L, w, after);
     }
 
     // a step of single tokens forms two-step decays and gates inside the recurrence
@@ -602,7 +867,7 @@ struct Sequence {
         }
         StepRows single = s.rows;
         single.n = s.single;
-        FORGE_TRY(attn_rows(t, dt, S.q.p, run.pool, hgate, S.mid.p, mid_ld, single, t.chunk ? std::min(t.chunk, s.max_keys) : s.max_keys, st));
+        FORGE_TRY(attn_rows(t, dt, S.q.p, run.pool, hgate, nullptr, S.mid.p, mid_ld, single, t.most_keys(s.max_keys), st));
         const int np = n - s.single;
         if (np > 0) {
             PromptAttnArgs p;
@@ -625,9 +890,12 @@ struct Sequence {
     }
 };
 
-int32_t run_head(ForgeModel* m, const void* h, int n, float* logits) {
+// rows: of the stream that h's rows were taken from (null: the first n); step_rows: the step's scale_rows
+int32_t run_head(ForgeModel* m, const void* h, const int32_t* rows, int n, int step_rows, float* logits) {
     StackModel& S = *m->stack;
     DenseOut o;
+    o.scale = stream_scale(S, step_rows);
+    o.scale.row = rows; o.scale.mul = S.spec.logit_scale;
     o.nseg = 1;
     o.seg[0].rows = S.spec.vocab; o.seg[0].dst = logits; o.seg[0].ld = S.spec.vocab;
     return dense_gemm(S.head, h, S.width_p, n, o, S.scratch, m->d_err, m->stream);
@@ -668,6 +936,7 @@ int32_t stack_cache_create(ForgeKV* kv) {
         FORGE_CUDA(cudaMemsetAsync(q, 0, bytes, m->stream));
         return FORGE_OK;
     };
+    if (S.spec.buckets) FORGE_TRY(alloc(&kv->stack->prev_token, slots * sizeof(uint32_t)));
     for (size_t i = 0; i < S.spec.runs.size(); ++i) {
         const LayerSpec& L = S.spec.layers[S.spec.runs[i].layer];
         StackCache::Run& r = kv->stack->runs[i];
@@ -688,11 +957,13 @@ int32_t stack_cache_create(ForgeKV* kv) {
 void stack_cache_destroy(ForgeKV* kv) {
     if (!kv->stack) return;
     for (StackCache::Run& r : kv->stack->runs) for (void* p : {r.pool, static_cast<void*>(r.state), r.ring, r.prev}) if (p) cudaFree(p);
+    if (kv->stack->prev_token) cudaFree(kv->stack->prev_token);
     delete kv->stack;
     kv->stack = nullptr;
 }
 
 bool stack_has_state(const ForgeModel* m) {
+    if (m->stack->spec.buckets) return true;
     for (const LayerSpec& L : m->stack->spec.layers) if (L.has_state()) return true;
     return false;
 }
@@ -753,7 +1024,7 @@ size_t stack_kv_bytes_per_token(const ForgeKV* kv) {
 }
 size_t stack_kv_bytes_per_seq(const ForgeKV* kv) {
     const StackModel& S = *kv->model->stack;
-    size_t n = 0;
+    size_t n = S.spec.buckets ? sizeof(uint32_t) : 0;
     for (const LayerRun& r : S.spec.runs) { const LayerSpec& L = S.spec.layers[r.layer]; n += state_bytes(L) + ring_bytes(S, L) + prev_bytes(S, L); }
     return n;
 }
@@ -779,6 +1050,7 @@ int32_t stack_kv_copy(ForgeKV* kv, int seq, int len, char* host, bool to_host) {
         FORGE_TRY(copy(static_cast<char*>(r.ring) + size_t(seq) * ring_bytes(S, L), ring_bytes(S, L)));
         FORGE_TRY(copy(static_cast<char*>(r.prev) + size_t(seq) * prev_bytes(S, L), prev_bytes(S, L)));
     }
+    if (S.spec.buckets) FORGE_TRY(copy(reinterpret_cast<char*>(kv->stack->prev_token + seq), sizeof(uint32_t)));
     FORGE_CUDA(cudaStreamSynchronize(m->stream));
     return FORGE_OK;
 }
@@ -855,11 +1127,12 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
     s.segs = SegTable{reinterpret_cast<const ScanSeg*>(dm + o_segs), int(segs.size()), n_short, max_seg, chunks, ones, rows - ones};
     s.ctx_pages = dm + o_pages; s.ctx_rows = ctx_rows;
     s.tiles = reinterpret_cast<const PromptTile*>(dm + o_tiles); s.n_tiles = int(tiles.size());
+    s.scale_rows = std::max(rows, wants);
     if (trace_rows) { s.trace = m->trace + size_t(trace_row0) * S.spec.width; s.trace_stride = size_t(trace_rows) * S.spec.width; }
     FORGE_TRY(Sequence(m, kv, s).run());
     if (wants) {
-        FORGE_TRY(gather_act_rows(S.sel.p, S.h.p, dm + 3 * rows, wants, S.width_p, S.dtype, m->stream));
-        FORGE_TRY(run_head(m, S.sel.p, wants, static_cast<float*>(S.logits.p)));
+        FORGE_TRY(gather_act_rows(S.sel.p, S.h.p, S.width_p, dm + 3 * rows, wants, S.width_p, S.dtype, m->stream));
+        FORGE_TRY(run_head(m, S.sel.p, dm + 3 * rows, wants, s.scale_rows, static_cast<float*>(S.logits.p)));
     }
     if (d_logits) *d_logits = static_cast<float*>(S.logits.p);
     FORGE_CUDA(cudaStreamSynchronize(m->stream));   // the host's tables are read by the copy
@@ -892,11 +1165,12 @@ int32_t stack_decode_launches(ForgeModel* m, ForgeKV* kv, int batch, bool greedy
     s.tokens = m->d_tok;
     s.rows = StepRows{batch, kv->d_seq_len, nullptr, kv->d_page_table, kv->pages_per_seq};
     s.rows.slot0 = kv->slot0;
+    s.scale_rows = batch;
     s.ones = s.single = batch; s.splits = kv->stack->splits; s.max_keys = kv->max_seq;
     if (record) { s.hist = m->d_hist; s.step = m->d_step; }
     if (m->trace_on) { s.trace = m->trace; s.trace_stride = size_t(batch) * S.spec.width; }
     FORGE_TRY(Sequence(m, kv, s).run());
-    FORGE_TRY(run_head(m, S.h.p, batch, m->d_logits));
+    FORGE_TRY(run_head(m, S.h.p, nullptr, batch, batch, m->d_logits));
     if (greedy) FORGE_TRY(argmax_slices(m->d_tok, m->d_logits, m->V, batch, m->d_amax_val, m->d_amax_idx, m->d_amax_ticket, m->stream));
     return step_advance(kv->d_seq_len, batch, m->d_step, m->stream);
 }
@@ -949,19 +1223,24 @@ int32_t forge_model_open(const char* dir, int32_t dtype, int32_t device, ForgeMo
             put_rows(img, dtype, spec.width, *t.top.at("embed"), 0);
             FORGE_TRY(upload(m, &S.embed, img));
         }
+        if (spec.buckets) {
+            std::vector<uint8_t> img((size_t(spec.buckets) + 1) * spec.width * es);
+            put_rows(img, dtype, spec.width, *t.top.at("bigram"), 0);
+            FORGE_TRY(upload(m, &S.bigram, img));
+        }
         {
             Image head(spec.vocab, S.width_p, dtype);
             head.put(t.top.at("head"), 0);
             FORGE_TRY(head.load(m, &S.head));
         }
-        if (spec.loop_times) {   // columns [stream | embedding], each padded
+        if (spec.loop_times) FORGE_TRY(upload_f32(m, &S.loop_step, *t.top.at("loop.step")));
+        if (spec.loop_times && !spec.adds_loop()) {   // columns [stream | embedding], each padded
             const TensorView& in = *t.top.at("loop.in");
             Image img(spec.width, 2 * S.width_p, dtype);
             for (int r = 0; r < spec.width; ++r)
                 for (int c = 0; c < 2 * spec.width; ++c)
                     store(img.img.data(), dtype, size_t(r) * img.K + (c < spec.width ? c : S.width_p + c - spec.width), in, size_t(r) * 2 * spec.width + c);
             FORGE_TRY(img.load(m, &S.loop_in));
-            FORGE_TRY(upload_f32(m, &S.loop_step, *t.top.at("loop.step")));
         }
         FORGE_TRY(load_norm(m, &S.final_norm, t.top, "final.norm"));
         S.w.resize(spec.layers.size());
