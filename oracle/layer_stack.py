@@ -593,8 +593,133 @@ def random_robazen(cfg, seed=0, rank=20):
     return t
 
 
+def rotation_of(dims, base=1000.0, **scaling):
+    return {"base": float(base), "dims": dims, "scaling": scaling or None}
+
+
+def head_normed_mixer(heads=6, kv_heads=2, dim=24, vdim=40, window=40, keep=5, rot=None, scale=None):
+    return {"dim": dim, "heads": heads, "kv_heads": kv_heads, "mask": {"keep_first": keep, "size": window}, "rot": rot or rotation_of(16, 3000.0, factor=4.0, fast=8.0, original=64, slow=1.0),
+            "scale": float(scale if scale is not None else dim ** -0.5), "vdim": vdim}
+
+
+def row_normed_mixer(heads=4, kv_heads=4, dim=32, vdim=16, rot=None, scale=None):
+    return {"dim": dim, "heads": heads, "kv_heads": kv_heads, "rot": rot or rotation_of(20, 700.0, factor=3.0), "scale": float(scale if scale is not None else dim ** -0.5), "vdim": vdim}
+
+
+def linear_mixer(heads=3, dim=24, vdim=40, tau=8.0):
+    return {"dim": dim, "heads": heads, "tau": float(tau), "vdim": vdim}
+
+
+def make_mokatar(width=136, vocab=203, layers=(), loop=None, eps=1e-5, scale=3.0, bigram=(61, 5, 3), logit_scale=0.7):
+    """``layers``: (type, mixer, feed-forward) per layer, the feed-forward None, a size, or (experts, top, size); ``loop``: (start, stop, times); ``bigram``:
+    (buckets, factor of the token before, factor of the token)."""
+    def ff(f):
+        if f is None:
+            return None
+        return {"ff": f, "kind": "dense"} if isinstance(f, int) else {"expert": {"ff": f[2]}, "kind": "moe", "router": {"experts": f[0], "top": f[1]}}
+    return {"architecture": "Mokatar", "embedding": {"bigram": dict(zip(("buckets", "mul_prev", "mul_cur"), bigram)), "scale": float(scale)},
+            "layers": [{"mixer": mx, "mlp": ff(f), "type": t} for t, mx, f in layers], "logit_scale": float(logit_scale),
+            "loop": None if loop is None else dict(zip(("start", "stop", "times"), loop)), "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+MARKERS = 4
+
+
+def random_mokatar(cfg, seed=0, rank=12, clear=True):
+    """Seeded weights of a Mokatar model, rounded to bfloat16.  clear: routers read MARKERS columns of the stream alone, in which the embedding
+    holds signs and nobody else writes, so that rounding does not change a choice."""
+    rng = np.random.default_rng(seed)
+    W = cfg["width"]
+    t = {}
+
+    def mat(name, out, inp, gain=1.0):
+        t[name] = bf16_round(rng.standard_normal((out, inp)) * (gain / math.sqrt(inp)))
+
+    def vec(name, n, mean, dev):
+        t[name] = bf16_round(mean + dev * rng.standard_normal(n))
+
+    t["embed"] = bf16_round(rng.standard_normal((cfg["vocab"], W)))
+    t["bigram"] = bf16_round(2.0 * rng.standard_normal((cfg["embedding"]["bigram"]["buckets"] + 1, W)))
+    if cfg.get("loop"):
+        t["loop.step"] = bf16_round(1.5 * rng.standard_normal((cfg["loop"]["times"], W)))
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        x = p + "mix."
+        vec(p + "norm1", W, 0.1, 0.3)
+        H, dv = m["heads"], m["vdim"]
+        if L["type"] == "gla":
+            D = H * m["dim"]
+            mat(x + "q", D, W, 1.5)
+            mat(x + "k", D, W)
+            mat(x + "v", H * dv, W)
+            mat(x + "g", H * dv, W, 1.5)
+            mat(x + "a1", rank, W)
+            mat(x + "a2", D, rank, 2.0)
+            vec(x + "a2.b", D, 0.5, 2.0)
+            vec(x + "norm", dv, 1.0, 0.3)
+        else:
+            q, k, v = H * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * dv
+            mat(x + "q", q, W)
+            mat(x + "k", k, W)
+            mat(x + "v", v, W)
+            if L["type"] == "attention":
+                vec(x + "q.norm", m["dim"], 1.2, 0.4)
+                vec(x + "k.norm", m["dim"], 1.2, 0.4)
+                vec(x + "sink", H, 0.5, 1.5)
+            else:
+                for n, c in (("q", q), ("k", k), ("v", v)):
+                    vec(x + n + ".b", c, 0.0, 0.5)
+                vec(x + "q.norm", q, 1.2, 0.4)
+                vec(x + "k.norm", k, 1.2, 0.4)
+        mat(x + "o", W, H * dv, 2.0)
+        f = L.get("mlp")
+        if f:
+            vec(p + "norm2", W, -0.1, 0.3)
+            if f["kind"] == "dense":
+                mat(p + "mlp.gate", f["ff"], W, 1.5)
+                mat(p + "mlp.up", f["ff"], W, 1.5)
+                mat(p + "mlp.down", W, f["ff"], 1.5)
+            else:
+                E, n = f["router"]["experts"], f["expert"]["ff"]
+                for e in range(E):
+                    mat(p + f"mlp.e{e}.gate", n, W, 1.5)
+                    mat(p + f"mlp.e{e}.up", n, W, 1.5)
+                    mat(p + f"mlp.e{e}.down", W, n, 2.0)
+                mat(p + "mlp.router", E, W, 2.0)
+                vec(p + "mlp.router.b", E, 0.0, 0.5)
+    vec("final.norm", W, 0.0, 0.3)
+    mat("head", cfg["vocab"], W)
+    if clear:
+        signs = np.sign(rng.standard_normal((cfg["vocab"], MARKERS)))
+        t["embed"][:, :MARKERS] = signs
+        t["bigram"][:, :MARKERS] = 0
+        if "loop.step" in t:
+            t["loop.step"][:, :MARKERS] = 0
+        patterns = np.array([[1.0 if i >> c & 1 else -1.0 for c in range(MARKERS)] for i in range(1 << MARKERS)])
+        for name in t:
+            if name.endswith(("mix.o", ".down")):
+                t[name][:MARKERS] = 0
+            if name.endswith((".norm1", ".norm2")):
+                t[name][:MARKERS] = 0.5
+            if name.endswith("mlp.router"):
+                best = None
+                for _ in range(200):     # of some routers the one whose closest call is least close
+                    r = np.zeros_like(t[name])
+                    r[:, :MARKERS] = bf16_round(2.0 * rng.standard_normal((len(r), MARKERS)))
+                    z = np.sort(patterns @ r[:, :MARKERS].T, axis=1)[:, ::-1]
+                    top = cfg["layers"][int(name[1:name.index(".")])]["mlp"]["router"]["top"]
+                    gap = (z[:, top - 1] - z[:, top]).min() if top < len(r) else 1e9
+                    if best is None or gap > best[0]:
+                        best = (gap, r)
+                t[name] = best[1]
+                t[name + ".b"] = bf16_round(0.02 * rng.standard_normal(len(best[1])))
+    return t
+
+
 def random_tensors(cfg, seed=0):
     """Seeded weights, rounded to bfloat16, in which every factor matters (norm weights and biases away from 1 and 0)."""
+    if cfg["architecture"] == "Mokatar":
+        return random_mokatar(cfg, seed)
     if cfg["architecture"] == "Robazen":
         return random_robazen(cfg, seed)
     rng = np.random.default_rng(seed)

@@ -45,9 +45,28 @@ ROBAZEN = {
     # wide heads and values beyond the chunked kernels, many query heads on one key head, a chunk larger than the prompt
     "beyond": LS.make_robazen(96, 110, [("delta", _delta(2, 2, 160, 200, 4), None), ("parallel", _pair(10, 1, 72, 136, 1000, 50.0, None, 1, 136), 40), ("channel_delta", _delta(1, 1, 136, 40, 7), None)]),
 }
+_yarn = LS.rotation_of
+MOKATAR = {
+    # every mixer and feed-forward, the middle layers twice
+    "all": LS.make_mokatar(136, 203, [("gla", LS.linear_mixer(), 72), ("attention", LS.head_normed_mixer(), (5, 2, 24)), ("attention_2", LS.row_normed_mixer(), 56), ("gla", LS.linear_mixer(2, 16, 24, 3.0), None)],
+                           (1, 3, 2), eps=1e-3),
+    # the loop is the whole model, three passes; one head; every expert used; no kept tokens; a rotation without scaling
+    "loop_all": LS.make_mokatar(72, 67, [("attention", LS.head_normed_mixer(1, 1, 16, 8, 9, 0, _yarn(16, 50.0), 0.4), (3, 3, 70)), ("gla", LS.linear_mixer(1, 8, 8, 1.0), (4, 1, 16))], (0, 2, 3), eps=1e-2,
+                                scale=1.0, bigram=(7, 1, 0), logit_scale=1.0),
+    # one pass only, at the end; sizes no multiple of eight; layers without a feed-forward
+    "odd": LS.make_mokatar(70, 91, [("attention_2", LS.row_normed_mixer(3, 1, 9, 13, _yarn(6, 77.0, factor=2.5)), 21), ("attention", LS.head_normed_mixer(6, 3, 13, 11, 33, 3, _yarn(10, 90.0, factor=2.0, fast=2.0, original=40, slow=0.5)), (7, 3, 21)),
+                                    ("gla", LS.linear_mixer(2, 11, 9, 5.0), None), ("attention", LS.head_normed_mixer(2, 1, 10, 7, 64, 1, _yarn(4, 20.0)), None)], (3, 4, 1)),
+    # no loop; a real model's head sizes, many experts, several row tiles per expert
+    "wide": LS.make_mokatar(192, 150, [("attention", LS.head_normed_mixer(8, 2, 128, 128, 80, 4, _yarn(64, 10000.0, factor=8.0, fast=32.0, original=256, slow=1.0)), (40, 4, 100)), ("attention_2", LS.row_normed_mixer(4, 2, 128, 64, _yarn(128, 1e6, factor=4.0)), 64),
+                                       ("gla", LS.linear_mixer(2, 128, 128, 16.0), (70, 6, 40))]),
+    # wide heads and values beyond the tensor-core kernels, many query heads on one key head, a window larger than the prompt, more kept tokens than the window holds
+    "beyond": LS.make_mokatar(96, 110, [("attention", LS.head_normed_mixer(10, 1, 72, 272, 1000, 100), (3, 2, 40)), ("gla", LS.linear_mixer(1, 136, 200, 2.0), None), ("attention_2", LS.row_normed_mixer(2, 2, 300, 136), 40),
+                                        ("attention", LS.head_normed_mixer(3, 3, 24, 24, 20, 70), None)]),
+}
+CONFIGS.update({"mokatar_" + k: v for k, v in MOKATAR.items()})
 CONFIGS.update({"robazen_" + k: v for k, v in ROBAZEN.items()})
 ROBAZEN_NAMES = ["robazen_" + k for k in ROBAZEN]
-BOLENEX_NAMES = [k for k in CONFIGS if k not in ROBAZEN_NAMES]
+BOLENEX_NAMES = [k for k in CONFIGS if not k.startswith(("robazen_", "mokatar_"))]
 
 
 def sharp(tensors, cfg, gain=5.0):
