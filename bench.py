@@ -2,7 +2,7 @@
 """Benchmark of the quantized forward path on B200.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
-    python bench.py --design bolenex|robazen  (another model design, one GPU; the default workload is unchanged)
+    python bench.py --design bolenex|robazen|mokatar  (another model design, one GPU; the default workload is unchanged)
 
 One GPU (the default).  Headline workload: the Llama-3.2-1B-shaped Q4_0 decoder of the benchmark definition - one
 "step" is one request: a 1501-token uniform-random prompt through the batched prefill path, then 128 greedy decode
@@ -455,6 +455,38 @@ def robazen_work(cfg: dict, ctx: int, m: int):
     return w, kv, flops
 
 
+def mokatar_work(cfg: dict, ctx: int, m: int):
+    """The same; the weights of a decode step depend on the batch: of a mixture the experts that some token is expected to use (uniform routing)."""
+    from forge_llm_b200 import synth
+    W, V = cfg["width"], cfg["vocab"]
+    shapes = synth.stack_shapes(cfg)
+    loop = cfg.get("loop") or {"start": 0, "stop": 0, "times": 1}
+    dense, mixtures, kv, flops = 2.0 * V * W, [], 0.0, 2.0 * V * W
+    for i, L in enumerate(cfg["layers"]):
+        n = loop["times"] if loop["start"] <= i < loop["stop"] else 1
+        mats = {k: s[0] * s[1] for k, s in shapes.items() if k.startswith(f"l{i}.") and len(s) == 2}
+        exp = sum(v for k, v in mats.items() if ".mlp.e" in k)
+        lin = sum(mats.values()) - exp
+        x, f = L["mixer"], L["mlp"]
+        dense += n * 2.0 * lin
+        flops += n * 2.0 * m * lin
+        if f["kind"] == "moe":
+            E, top = f["router"]["experts"], f["router"]["top"]
+            mixtures.append((n * 2.0 * exp, E, top))
+            flops += n * 2.0 * m * exp * top / E
+        if L["type"] == "gla":
+            state = x["heads"] * x["dim"] * x["vdim"]
+            kv += n * 8.0 * state
+            flops += n * 4.0 * m * state
+        else:
+            c = (x.get("mask") or {}).get("size", m)
+            seen = min(ctx, c + (x.get("mask") or {}).get("keep_first", 0))
+            kv += n * 2.0 * x["kv_heads"] * (x["dim"] + x["vdim"]) * seen
+            pairs = m * (m + 1) / 2 if m <= c else c * (c + 1) / 2 + (m - c) * c
+            flops += n * 2.0 * x["heads"] * (x["dim"] + x["vdim"]) * pairs
+    return (lambda batch: dense + sum(b * (1 - (1 - top / E) ** batch) for b, E, top in mixtures)), kv, flops
+
+
 def run_design(args, device: int):
     """Prefill and decode rates of a layer-list design and, at equal width, depth, heads and feed-forward, of the framework's closest
     decoder (multi-head, head_dim 128, Q8_0), each against its own roofline."""
@@ -465,7 +497,7 @@ def run_design(args, device: int):
     t0 = time.time()
     out, launches = {}, 0
     design = args.design
-    make_config, work = {"bolenex": (synth.bolenex_config, bolenex_work), "robazen": (synth.robazen_config, robazen_work)}[design]
+    make_config, work = {"bolenex": (synth.bolenex_config, bolenex_work), "robazen": (synth.robazen_config, robazen_work), "mokatar": (synth.mokatar_config, mokatar_work)}[design]
     arm = f"{design} bf16"
 
     def measure(model, batch, n_prompt, n_dec, bytes_w, bytes_kv, flops, vocab):
@@ -495,7 +527,7 @@ def run_design(args, device: int):
                 pre.append(p); dec.append(d); host.append(h1 - h0); nl += l
         kv.close()
         step = statistics.median(dec) / n_dec * 1e-3
-        gbs = (bytes_w + batch * bytes_kv) / step / 1e9
+        gbs = ((bytes_w(batch) if callable(bytes_w) else bytes_w) + batch * bytes_kv) / step / 1e9
         tf = batch * flops / (statistics.median(pre) * 1e-3) / 1e12
         return {"batch": batch, "decode_tok_s": batch / step, "us_per_step": step * 1e6,
                 "decode_roofline": {"bound": "hbm", "achieved": gbs, "peak": peaks["hbm_gbs"], "unit": "GB/s", "frac": gbs / peaks["hbm_gbs"]},
@@ -713,7 +745,7 @@ def main():
     ap.add_argument("--prompt-tokens", type=int, default=None, help="override the headline prompt length (profiling / experiments)")
     ap.add_argument("--decode-steps", type=int, default=None, help="override the headline number of decode steps")
     ap.add_argument("--profile", action="store_true", help="short run for ncu: no side configurations, no CPU baseline; prints a non-benchmark line")
-    ap.add_argument("--design", default="headline", choices=["headline", "bolenex", "robazen"], help="bolenex, robazen: that design beside a Llama-shaped decoder of equal size (one GPU)")
+    ap.add_argument("--design", default="headline", choices=["headline", "bolenex", "robazen", "mokatar"], help="bolenex, robazen, mokatar: that design beside a Llama-shaped decoder of equal size (one GPU)")
     ap.add_argument("--sizes", default="w2048,w4096", help="with --design: which sizes")
     ap.add_argument("--batches", default="1,16", help="with --design: sequences decoded together")
     ap.add_argument("--arms", default="design,llama", help="with --design: which models")

@@ -268,15 +268,73 @@ def robazen_shapes(cfg: dict, layer: int, rank: int = 64) -> dict:
     return s
 
 
-LAYER_SHAPES = {"Bolenex": bolenex_shapes, "Robazen": robazen_shapes}
+def mokatar_config(width: int, layers: int, heads: int, ff: int, vocab: int, dim: int = 128, window: int = 1024, experts: int = 8, top: int = 2, loop: bool = True) -> dict:
+    """config.json of a Mokatar stack of ``layers`` layer runs (a multiple of four): groups of (gated linear attention, windowed attention,
+    attention, windowed attention), the windowed ones with a mixture of experts whose used ones have ``ff`` rows together, the others with
+    a dense feed-forward.  With ``loop`` a quarter of the groups (at least one) runs twice with the same weights."""
+    def rot(**scaling):
+        return {"base": 10000.0, "dims": dim, "scaling": scaling}
+
+    kv = max(1, heads // 4)
+    near = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": float(dim ** -0.5), "mask": {"size": window, "keep_first": 16},
+            "rot": rot(factor=4.0, fast=32.0, original=4096, slow=1.0)}
+    far = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": float(dim ** -0.5), "rot": rot(factor=4.0)}
+    lin = {"heads": heads, "dim": dim, "vdim": dim, "tau": 16.0}
+    dense, moe = {"kind": "dense", "ff": ff}, {"kind": "moe", "expert": {"ff": ff // top}, "router": {"experts": experts, "top": top}}
+    group = [("gla", lin, dense), ("attention", near, moe), ("attention_2", far, dense), ("attention", near, moe)]
+    n = layers // 4
+    twice = max(1, n // 4) if loop and n >= 2 else 0
+    out = [{"type": t, "mixer": dict(m), "mlp": dict(f)} for _ in range(n - twice) for t, m, f in group]
+    cfg = {"architecture": "Mokatar", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "layers": out, "loop": None, "logit_scale": 1.0,
+           "embedding": {"scale": 1.0, "bigram": {"buckets": 4093, "mul_prev": 31, "mul_cur": 7}}}
+    if twice:
+        cfg["loop"] = {"start": len(out) - 4 * twice, "stop": len(out), "times": 2}
+    return cfg
+
+
+def mokatar_shapes(cfg: dict, layer: int, rank: int = 64) -> dict:
+    """Tensor shapes of one layer, without its prefix; ``rank``: inner size of the two-step projections."""
+    W, L = cfg["width"], cfg["layers"][layer]
+    m, f = L["mixer"], L.get("mlp")
+    H, hv = m["heads"], m["heads"] * m["vdim"]
+    s = {"norm1": (W,), "mix.o": (W, hv)}
+    if L["type"] == "gla":
+        D = H * m["dim"]
+        s.update({"mix.q": (D, W), "mix.k": (D, W), "mix.v": (hv, W), "mix.g": (hv, W), "mix.a1": (rank, W), "mix.a2": (D, rank), "mix.a2.b": (D,), "mix.norm": (m["vdim"],)})
+    else:
+        q, k, v = H * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"]
+        s.update({"mix.q": (q, W), "mix.k": (k, W), "mix.v": (v, W)})
+        if L["type"] == "attention":
+            s.update({"mix.q.norm": (m["dim"],), "mix.k.norm": (m["dim"],), "mix.sink": (H,)})
+        else:
+            s.update({"mix.q.b": (q,), "mix.k.b": (k,), "mix.v.b": (v,), "mix.q.norm": (q,), "mix.k.norm": (k,)})
+    if f:
+        s["norm2"] = (W,)
+        if f["kind"] == "dense":
+            s.update({"mlp.gate": (f["ff"], W), "mlp.up": (f["ff"], W), "mlp.down": (W, f["ff"])})
+        else:
+            E, n = f["router"]["experts"], f["expert"]["ff"]
+            for e in range(E):
+                s.update({f"mlp.e{e}.gate": (n, W), f"mlp.e{e}.up": (n, W), f"mlp.e{e}.down": (W, n)})
+            s.update({"mlp.router": (E, W), "mlp.router.b": (E,)})
+    return s
+
+
+LAYER_SHAPES = {"Bolenex": bolenex_shapes, "Robazen": robazen_shapes, "Mokatar": mokatar_shapes}
 
 
 def stack_shapes(cfg: dict) -> dict:
     """Tensor shapes of a layer-list model."""
     W, V = cfg["width"], cfg["vocab"]
-    out = {"embed": (V, W), "head": (V, W), "final.norm": (W,), "final.norm.b": (W,), "final.norm.alpha": ()}
+    out = {"embed": (V, W), "head": (V, W), "final.norm": (W,)}
+    if cfg["architecture"] == "Mokatar":
+        out["bigram"] = (cfg["embedding"]["bigram"]["buckets"] + 1, W)
+    else:
+        out.update({"final.norm.b": (W,), "final.norm.alpha": ()})
+        if cfg.get("loop"):
+            out["loop.in"] = (W, 2 * W)
     if cfg.get("loop"):
-        out.update({"loop.in": (W, 2 * W), "loop.step": (cfg["loop"]["times"], W)})
+        out["loop.step"] = (cfg["loop"]["times"], W)
     for i, L in enumerate(cfg["layers"]):
         if "weights_of" not in L:
             out.update({f"l{i}.{n}": s for n, s in LAYER_SHAPES[cfg["architecture"]](cfg, i).items()})

@@ -223,3 +223,13 @@ def test_tensor_errors(tmp_path):
         with pytest.raises(ForgeError) as e:
             _info(_folder(tmp_path / str(i), tensors=edit))
         assert text in str(e.value), e.value
+
+
+def test_shapes_of_the_synthetic_writer_agree(tmp_path):
+    from forge_llm_b200 import synth
+    cfg = synth.mokatar_config(128, 8, 2, 48, 77, dim=64, window=32)
+    synth.write_stack(str(tmp_path), cfg)
+    i = _info(str(tmp_path))
+    assert i["num_layers"] == 8 and i["num_weight_layers"] == 4
+    t = LS.read_safetensors(str(tmp_path / "model.safetensors"))
+    assert np.array_equal(t["l1.mix.q"], t["l3.mix.q"]) and t["l1.mlp.e7.gate"].std() > 0.05
