@@ -1,13 +1,18 @@
 // Attention of single rows (decode, short portions, float32 prompts) over a paged cache.
 //
-// One CTA = up to eight query heads of one key / value head, one row, one of up to eight ranges of its keys; the CTAs of a row form a
-// cluster and merge their sums through distributed shared memory.  A warp takes 32 keys at a time: eight keys by four lanes for
-// the scores, then a lane per pair of value columns for the sums.  Everything behind the loads is f32.
+// One CTA = some query heads of one key / value head, one row, one of up to eight ranges of its keys; the CTAs of a row form a
+// cluster and merge their sums through distributed shared memory.
+//   float32 (and value heads beyond 256)  up to four heads; a warp takes 32 keys at a time: eight keys by four lanes for the scores, then
+//                                         a lane per pair of value columns for the sums.  Everything behind the loads is f32.
+//   bfloat16                              up to sixteen heads are the rows of a tensor-core tile; a warp takes sixteen keys at a time, whose
+//                                         keys and values it copies into its own two buffers in shared memory.  The tiles of earlier
+//                                         steps' keys are requested before the dependency wait.  Probabilities enter their product as bf16 pairs.
 #include <cooperative_groups.h>
 
 #include <algorithm>
 
 #include "attn_rows.cuh"
+#include "mma.cuh"
 
 namespace forge {
 
@@ -20,6 +25,55 @@ constexpr float kLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ float2 load_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
 __device__ __forceinline__ float2 load_pair(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+
+// The warps' maxima and sums (sml [warp][hs][2]) and unnormalised outputs (so, `stride` values per warp, [head][vdim_p]) of a CTA become one, then those of
+// the cluster's CTAs: nh heads from h0, hs the stride of sml in heads, cml [nh][2].
+template <typename T>
+__device__ __forceinline__ void merge_rows(const AttnDims& d, float* so, int stride, float* sml, float* cml, int hs, int nh, int h0, int r, const float* gate, const float* sink, T* out, int out_ld) {
+    const int split = blockIdx.x, splits = gridDim.x;
+    __syncthreads();
+    if (int(threadIdx.x) < nh) {   // maximum and sum of the CTA
+        const int h = threadIdx.x;
+        float mt = -INFINITY, lt = 0.f;
+        for (int w = 0; w < kWarps; ++w) mt = fmaxf(mt, sml[(w * hs + h) * 2]);
+        for (int w = 0; w < kWarps; ++w) {
+            const float f = mt == -INFINITY ? 0.f : exp2f(sml[(w * hs + h) * 2] - mt);
+            lt += sml[(w * hs + h) * 2 + 1] * f;
+            sml[(w * hs + h) * 2] = f;     // the warp's factor
+        }
+        cml[2 * h] = mt; cml[2 * h + 1] = lt;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < nh * d.vdim_p; i += kThreads) {   // own element of every warp: read, then written over warp 0's
+        const int h = i / d.vdim_p;
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < kWarps; ++w) v += so[w * stride + i] * sml[(w * hs + h) * 2];
+        so[i] = v;
+    }
+    cg::cluster_group cl = cg::this_cluster();
+    if (splits > 1) cl.sync();
+    else __syncthreads();
+    const int items = nh * d.vdim, share = (items + splits - 1) / splits;
+    for (int i = split * share + threadIdx.x; i < min(items, (split + 1) * share); i += kThreads) {
+        const int h = i / d.vdim, c = i % d.vdim;
+        const float own = sink ? sink[h0 + h] * kLog2e : -INFINITY;
+        float mt = own, lt = 0.f, v = 0.f;
+        for (int s = 0; s < splits; ++s) mt = fmaxf(mt, splits > 1 ? cl.map_shared_rank(cml, s)[2 * h] : cml[2 * h]);
+        for (int s = 0; s < splits; ++s) {
+            const float* o = splits > 1 ? cl.map_shared_rank(cml, s) : cml;
+            const float* x = splits > 1 ? cl.map_shared_rank(so, s) : so;
+            const float f = o[2 * h] == -INFINITY ? 0.f : exp2f(o[2 * h] - mt);
+            lt = fmaf(o[2 * h + 1], f, lt);
+            v = fmaf(x[h * d.vdim_p + c], f, v);
+        }
+        if (sink) lt += exp2f(own - mt);
+        v /= lt;
+        if (gate) v *= gate[size_t(r) * d.heads + h0 + h];
+        out[size_t(r) * out_ld + (h0 + h) * d.vdim + c] = to_t<T>(v);
+    }
+    if (splits > 1) cl.sync();   // nobody leaves while its shared memory is read
+}
 
 // (What a kernel in front writes is not __restrict__: loads of it may not be moved above the dependency wait.)
 // GQ: query heads per CTA; VP: pairs of value columns per lane
@@ -131,48 +185,7 @@ __global__ void __launch_bounds__(kThreads) attn_rows_kernel(const AttnDims d, c
         for (int c = 0; c < VP; ++c)
             if (2 * lane + 64 * c < d.vdim_p) *reinterpret_cast<float2*>(so + (warp * GQ + h) * d.vdim_p + 2 * lane + 64 * c) = make_float2(acc[h][2 * c], acc[h][2 * c + 1]);
     }
-    __syncthreads();
-    if (threadIdx.x < GQ) {   // maximum and sum of the CTA
-        const int h = threadIdx.x;
-        float mt = -INFINITY, lt = 0.f;
-        for (int w = 0; w < kWarps; ++w) mt = fmaxf(mt, sml[(w * GQ + h) * 2]);
-        for (int w = 0; w < kWarps; ++w) {
-            const float f = mt == -INFINITY ? 0.f : exp2f(sml[(w * GQ + h) * 2] - mt);
-            lt += sml[(w * GQ + h) * 2 + 1] * f;
-            sml[(w * GQ + h) * 2] = f;     // the warp's factor
-        }
-        cml[2 * h] = mt; cml[2 * h + 1] = lt;
-    }
-    __syncthreads();
-    for (int i = threadIdx.x; i < GQ * d.vdim_p; i += kThreads) {   // own element of every warp: read, then written over warp 0's
-        const int h = i / d.vdim_p;
-        float v = 0.f;
-#pragma unroll
-        for (int w = 0; w < kWarps; ++w) v += so[w * GQ * d.vdim_p + i] * sml[(w * GQ + h) * 2];
-        so[i] = v;
-    }
-    cg::cluster_group cl = cg::this_cluster();
-    if (splits > 1) cl.sync();
-    else __syncthreads();
-    const int items = nh * d.vdim, share = (items + splits - 1) / splits;
-    for (int i = split * share + threadIdx.x; i < min(items, (split + 1) * share); i += kThreads) {
-        const int h = i / d.vdim, c = i % d.vdim;
-        const float own = sink ? sink[h0 + h] * kLog2e : -INFINITY;
-        float mt = own, lt = 0.f, v = 0.f;
-        for (int s = 0; s < splits; ++s) mt = fmaxf(mt, splits > 1 ? cl.map_shared_rank(cml, s)[2 * h] : cml[2 * h]);
-        for (int s = 0; s < splits; ++s) {
-            const float* o = splits > 1 ? cl.map_shared_rank(cml, s) : cml;
-            const float* x = splits > 1 ? cl.map_shared_rank(so, s) : so;
-            const float f = o[2 * h] == -INFINITY ? 0.f : exp2f(o[2 * h] - mt);
-            lt = fmaf(o[2 * h + 1], f, lt);
-            v = fmaf(x[h * d.vdim_p + c], f, v);
-        }
-        if (sink) lt += exp2f(own - mt);
-        v /= lt;
-        if (gate) v *= gate[size_t(r) * d.heads + h0 + h];
-        out[size_t(r) * out_ld + (h0 + h) * d.vdim + c] = to_t<T>(v);
-    }
-    if (splits > 1) cl.sync();   // nobody leaves while its shared memory is read
+    merge_rows(d, so, GQ * d.vdim_p, sml, cml, GQ, nh, h0, r, gate, sink, out, out_ld);
 }
 
 size_t smem_bytes(const AttnDims& d, int gq) { return sizeof(float) * (size_t(gq) * d.dim_p + kWarps * gq * 32 + size_t(kWarps) * gq * d.vdim_p + kWarps * gq * 2 + gq * 2); }
@@ -200,6 +213,173 @@ int32_t run(const AttnDims& d, const void* q, const void* cache, const float* ga
     if (gq == 1) return with_vp(std::integral_constant<int, 1>{});
     if (gq == 2) return with_vp(std::integral_constant<int, 2>{});
     return with_vp(std::integral_constant<int, 4>{});
+}
+
+// ------------------------------------------------------------------------------------------------ bfloat16
+using bf16 = __nv_bfloat16;
+constexpr int kTileKeys = 16, kRowHeads = 16;
+struct TileBytes {   // of shared memory, in elements
+    int ldk, ldv, stage;
+    __host__ __device__ explicit TileBytes(const AttnDims& d) : ldk(d.dim_p + 8), ldv(d.vdim_p + 8), stage(kTileKeys * (d.dim_p + 8 + d.vdim_p + 8)) {}
+};
+size_t mma_smem(const AttnDims& d) { return (size_t(kWarps) * 2 * TileBytes(d).stage + kRowHeads * TileBytes(d).ldk) * 2 + (kWarps * kRowHeads * 2 + kRowHeads * 2) * 4; }
+
+// VC: blocks of 64 value columns
+template <int VC>
+__global__ void __launch_bounds__(kThreads, 1) attn_rows_mma_kernel(const AttnDims d, const bf16* q, const bf16* cache, const float* gate, const float* __restrict__ sink, bf16* out, int out_ld, const StepRows rows) {
+    extern __shared__ __align__(16) unsigned char sm_raw[];
+    const TileBytes L(d);
+    bf16* tiles = reinterpret_cast<bf16*>(sm_raw);              // [warp][2]: keys, values
+    bf16* sq = tiles + size_t(kWarps) * 2 * L.stage;            // [16][ldk]
+    float* sml = reinterpret_cast<float*>(sq + kRowHeads * L.ldk);
+    float* cml = sml + kWarps * kRowHeads * 2;
+    const int gq = d.heads / d.groups, blocks = (gq + kRowHeads - 1) / kRowHeads;
+    const int split = blockIdx.x, splits = gridDim.x, g = blockIdx.y / blocks, h0 = g * gq + (blockIdx.y % blocks) * kRowHeads, nh = min(kRowHeads, (g + 1) * gq - h0), r = blockIdx.z;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lr = lane >> 2, lc = (lane & 3) * 2;
+    pdl_trigger();
+    // positions and page tables are written in front of the step's first kernel, which is launched without overlap
+    const int pos = rows.pos[r], seq = rows.seq ? rows.seq[r] : r;
+    const int lo = d.first_key(pos), kept = d.kept(pos), n = kept + pos - lo + 1;   // the visible keys are numbered: the kept first ones, then those from lo
+    const int per = ((n + splits - 1) / splits + kTileKeys - 1) & ~(kTileKeys - 1);
+    const int k_begin = split * per, k_end = min(n, k_begin + per);
+    const int32_t* pt = rows.page_table + size_t(seq) * rows.pages_per_seq;
+    const size_t W = d.row();
+    const bf16* kbase = cache + size_t(g) * d.dim_p;
+    const bf16* vbase = cache + size_t(d.groups) * d.dim_p + size_t(g) * d.vdim_p;
+    bf16* mine = tiles + size_t(warp) * 2 * L.stage;
+    const int kp = d.dim_p / 8, vp = d.vdim_p / 8;              // 16-byte pieces of a row
+    auto fetch = [&](int i) {   // the warp's i-th tile
+        const int key0 = k_begin + (warp + kWarps * i) * kTileKeys;
+        if (key0 < k_end) {
+            const int idx = key0 + min(lane & (kTileKeys - 1), k_end - key0 - 1), key = idx < kept ? idx : lo + idx - kept;
+            const uint32_t row = uint32_t(pt[key / FORGE_KV_PAGE]) * FORGE_KV_PAGE + key % FORGE_KV_PAGE;
+            const uint32_t sk = uint32_t(__cvta_generic_to_shared(mine + (i & 1) * L.stage)), sv = sk + kTileKeys * L.ldk * 2;
+            for (int p = lane; p < kTileKeys * kp; p += 32) {
+                const int k = p / kp, c = (p % kp) * 8;
+                cp_async16(sk + (k * L.ldk + c) * 2, kbase + __shfl_sync(0xffffffffu, row, k) * W + c, true);
+            }
+            for (int p = lane; p < kTileKeys * vp; p += 32) {
+                const int k = p / vp, c = (p % vp) * 8;
+                cp_async16(sv + (k * L.ldv + c) * 2, vbase + __shfl_sync(0xffffffffu, row, k) * W + c, true);
+            }
+        }
+        cp_commit();
+    };
+    // a tile all of whose keys earlier steps have written
+    auto old = [&](int i) { return min(k_end, k_begin + (warp + kWarps * i + 1) * kTileKeys) <= n - rows.fresh; };
+    int ahead = 0;
+    while (ahead < 2 && old(ahead)) fetch(ahead++);
+    pdl_wait();
+    while (ahead < 2) fetch(ahead++);
+    for (int i = threadIdx.x; i < kRowHeads * kp; i += kThreads) {
+        const int h = i / kp, c = (i % kp) * 8;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (h < nh) v = *reinterpret_cast<const uint4*>(q + (size_t(r) * d.heads + h0 + h) * d.dim_p + c);
+        *reinterpret_cast<uint4*>(sq + h * L.ldk + c) = v;
+    }
+    __syncthreads();
+    const SmemMat mq{uint32_t(__cvta_generic_to_shared(sq)), L.ldk};
+    const int ksteps = (d.dim + 15) / 16, vsteps = (d.vdim + 15) / 16;
+    const float scale2 = d.scale * kLog2e, inv_cap = d.softcap > 0.f ? d.scale / d.softcap : 0.f;
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[VC * 4][2][4];
+#pragma unroll
+    for (int v = 0; v < VC * 4; ++v)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[v][e >> 2][e & 3] = 0.f;
+    for (int i = 0;; ++i) {
+        const int key0 = k_begin + (warp + kWarps * i) * kTileKeys;
+        if (key0 >= k_end) break;
+        cp_wait<1>();
+        __syncwarp();
+        const uint32_t at = uint32_t(__cvta_generic_to_shared(mine + (i & 1) * L.stage));
+        const SmemMat mk{at, L.ldk}, mv{at + uint32_t(kTileKeys * L.ldk) * 2, L.ldv};
+        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll 4
+        for (int k = 0; k < ksteps; ++k) {
+            uint32_t fa[4], fb[4];
+            mq.a(fa, 0, k * 16, lane);
+            mk.b(fb, 0, k * 16, lane);
+            mma(s[0], fa, fb[0], fb[1]);
+            mma(s[1], fa, fb[2], fb[3]);
+        }
+        float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                float v = d.softcap > 0.f ? d.softcap * kLog2e * tanhf(s[j][e] * inv_cap) : s[j][e] * scale2;
+                if (key0 + j * 8 + lc + (e & 1) >= k_end) v = -INFINITY;
+                s[j][e] = v;
+                mx[e >> 1] = fmaxf(mx[e >> 1], v);
+            }
+        float alpha[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
+            mx[e] = fmaxf(fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2)), m[e]);
+            alpha[e] = exp2f(m[e] - mx[e]);
+            m[e] = mx[e];
+            l[e] *= alpha[e];
+        }
+        uint32_t ph[4], pl[4];
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const float p0 = exp2f(s[j][2 * e] - m[e]), p1 = exp2f(s[j][2 * e + 1] - m[e]);
+                l[e] += p0 + p1;
+                split_bf16x2(p0, p1, ph[2 * j + e], pl[2 * j + e]);
+            }
+#pragma unroll
+        for (int v = 0; v < VC * 4; ++v) {
+            if (v >= vsteps) break;
+            uint32_t fb[4];
+            mv.b_t(fb, 0, v * 16, lane);
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) o[v][j][e] *= alpha[e >> 1];
+                mma(o[v][j], pl, fb[2 * j], fb[2 * j + 1]);
+                mma(o[v][j], ph, fb[2 * j], fb[2 * j + 1]);
+            }
+        }
+        __syncwarp();   // the buffer is read
+        fetch(i + 2);
+    }
+    cp_wait<0>();
+    __syncwarp();
+    float* so = reinterpret_cast<float*>(mine);                 // [nh][vdim_p]: fits the warp's buffers
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
+        l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
+        const int h = lr + 8 * e;
+        if (h >= nh) continue;
+        if ((lane & 3) == 0) { sml[(warp * kRowHeads + h) * 2] = m[e]; sml[(warp * kRowHeads + h) * 2 + 1] = l[e]; }
+#pragma unroll
+        for (int v = 0; v < VC * 4; ++v)
+            if (v < vsteps)
+#pragma unroll
+                for (int j = 0; j < 2; ++j) *reinterpret_cast<float2*>(so + h * d.vdim_p + v * 16 + j * 8 + lc) = make_float2(o[v][j][2 * e], o[v][j][2 * e + 1]);
+    }
+    merge_rows(d, reinterpret_cast<float*>(tiles), L.stage, sml, cml, kRowHeads, nh, h0, r, gate, sink, out, out_ld);
+}
+
+bool mma_supported(const AttnDims& d) { return d.vdim_p <= 256 && mma_smem(d) <= 220 * 1024; }
+
+int32_t run_mma(const AttnDims& d, const void* q, const void* cache, const float* gate, const float* sink, void* out, int out_ld, const StepRows& rows, int max_keys, cudaStream_t st) {
+    const int gq = d.heads / d.groups, blocks = (gq + kRowHeads - 1) / kRowHeads;
+    const size_t smem = mma_smem(d);
+    int splits = 1;   // at most one CTA per SM, no split shorter than one round of its warps
+    while (splits < 8 && (long long)rows.n * d.groups * blocks * splits * 2 <= 148 && max_keys > splits * kWarps * kTileKeys) splits *= 2;
+    auto go = [&](auto kern) -> int32_t {
+        FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+        FORGE_CUDA(launch_pdl_cluster(kern, dim3(splits, d.groups * blocks, rows.n), dim3(kThreads), splits, smem, st, d, static_cast<const bf16*>(q), static_cast<const bf16*>(cache), gate, sink,
+                                      static_cast<bf16*>(out), out_ld, rows));
+        FORGE_LAUNCH_CHECK();
+        return FORGE_OK;
+    };
+    return d.vdim_p <= 64 ? go(attn_rows_mma_kernel<1>) : d.vdim_p <= 128 ? go(attn_rows_mma_kernel<2>) : go(attn_rows_mma_kernel<4>);
 }
 
 // ------------------------------------------------------------------------------------------------ queries and keys
@@ -264,6 +444,92 @@ __global__ void __launch_bounds__(256) qk_post_kernel(const AttnDims d, const Qk
     }
 }
 
+// The same for sizes in whole pieces of four values: a lane holds up to four pieces of its head, its rotation partners come through shared
+// memory for halves and lie in the same piece for interleaved pairs.
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+__device__ __forceinline__ float sum4(float4 v) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))); }
+template <typename T, int P>
+__global__ void __launch_bounds__(256) qk_post4_kernel(const AttnDims d, const QkPost p, const float* proj, int ldp, int k_col, const float* __restrict__ q_norm,
+                                                       const float* __restrict__ k_norm, const float2* __restrict__ rope, T* q, T* cache, const int32_t* place, const StepRows rows) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[2][8];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = blockIdx.y, h = blockIdx.x * 8 + warp;
+    const bool on = h < d.heads + d.groups, is_q = h < d.heads;
+    const int g = is_q ? h : h - d.heads, half = p.rot_dims / 2, pieces = d.dim / 4;
+    const float* w = is_q ? q_norm : k_norm;
+    if (p.norm == QkPost::WHOLE) w += size_t(g) * d.dim;
+    pdl_trigger();
+    const float2* turn = rope + size_t(rows.pos[r]) * half;
+    float4 nw[P], v[P], t0[P], t1[P];
+#pragma unroll
+    for (int i = 0; i < P; ++i) {
+        const int c = (lane + 32 * i) * 4;
+        const bool ok = on && c < d.dim;
+        nw[i] = ok ? *reinterpret_cast<const float4*>(w + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        t0[i] = t1[i] = make_float4(1.f, 0.f, 1.f, 0.f);
+        if (ok && c < 2 * half) {   // {cos, sin} of the piece's pairs
+            const int pair = p.interleaved ? c / 2 : c < half ? c : c - half;
+            t0[i] = *reinterpret_cast<const float4*>(turn + pair);
+            if (!p.interleaved) t1[i] = *reinterpret_cast<const float4*>(turn + pair + 2);
+        }
+    }
+    pdl_wait();
+    const float* row = proj + size_t(r) * ldp;
+    const float* src = is_q ? row + size_t(g) * d.dim : row + k_col + size_t(g) * d.dim;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < P; ++i) {
+        v[i] = on && lane + 32 * i < pieces ? reinterpret_cast<const float4*>(src)[lane + 32 * i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss += sum4(v[i]);
+    }
+    float n = float(d.dim);
+    if (p.norm == QkPost::WHOLE) {   // this CTA sums up the rows that its heads belong to
+        const int last = min(d.heads + d.groups, int(blockIdx.x) * 8 + 8) - 1;
+        const int nq = int(blockIdx.x) * 8 < d.heads ? d.heads * pieces : 0, nk = last >= d.heads ? d.groups * pieces : 0;
+        float sq = 0.f, sk = 0.f;
+#pragma unroll 4
+        for (int i = threadIdx.x; i < nq; i += 256) sq += sum4(reinterpret_cast<const float4*>(row)[i]);
+#pragma unroll 2
+        for (int i = threadIdx.x; i < nk; i += 256) sk += sum4(reinterpret_cast<const float4*>(row + k_col)[i]);
+        sq = warp_sum(sq); sk = warp_sum(sk);
+        if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+        __syncthreads();
+        ss = 0.f;
+        for (int i = 0; i < 8; ++i) ss += red[is_q ? 0 : 1][i];
+        n = float(is_q ? d.heads : d.groups) * d.dim;
+    } else ss = warp_sum(ss);
+    const float inv = 1.0f / sqrtf(ss / n + p.eps);
+    float* s = sm + warp * d.dim_p;
+#pragma unroll
+    for (int i = 0; i < P; ++i) {
+        v[i] = make_float4(v[i].x * inv * nw[i].x, v[i].y * inv * nw[i].y, v[i].z * inv * nw[i].z, v[i].w * inv * nw[i].w);
+        if (!p.interleaved && (lane + 32 * i) * 4 < 2 * half) store4(s + (lane + 32 * i) * 4, v[i]);
+    }
+    __syncwarp();
+    if (!on) return;
+    T* dst = is_q ? q + (size_t(r) * d.heads + g) * d.dim_p : cache + size_t(place[r]) * d.row() + size_t(g) * d.dim_p;
+#pragma unroll
+    for (int i = 0; i < P; ++i) {
+        const int c = (lane + 32 * i) * 4;
+        if (c >= d.dim) continue;
+        float4 x = v[i];
+        if (c < 2 * half) {
+            if (p.interleaved) {
+                x = make_float4(fmaf(v[i].x, t0[i].x, -v[i].y * t0[i].y), fmaf(v[i].y, t0[i].x, v[i].x * t0[i].y), fmaf(v[i].z, t0[i].z, -v[i].w * t0[i].w), fmaf(v[i].w, t0[i].z, v[i].z * t0[i].w));
+            } else {
+                const float4 y = *reinterpret_cast<const float4*>(s + (c < half ? c + half : c - half));
+                const float sign = c < half ? -1.f : 1.f;
+                x = make_float4(fmaf(x.x, t0[i].x, sign * y.x * t0[i].y), fmaf(x.y, t0[i].z, sign * y.y * t0[i].w), fmaf(x.z, t1[i].x, sign * y.z * t1[i].y), fmaf(x.w, t1[i].z, sign * y.w * t1[i].w));
+            }
+        }
+        store4(dst + c, x);
+    }
+}
+
 }  // namespace
 
 int32_t qk_post(const AttnDims& d, const QkPost& p, int dtype, const float* proj, int ldp, int k_col, const float* q_norm, const float* k_norm, const float* rope, void* q, void* cache,
@@ -277,7 +543,9 @@ int32_t qk_post(const AttnDims& d, const QkPost& p, int dtype, const float* proj
             StepRows part = rows;
             part.n = std::min(65535, rows.n - r0);
             part.pos += r0;
-            FORGE_CUDA(launch_pdl(qk_post_kernel<T>, dim3((d.heads + d.groups + 7) / 8, part.n), dim3(256), smem, st, d, p, proj + size_t(r0) * ldp, ldp, k_col, q_norm, k_norm,
+            const bool four = d.dim % 4 == 0 && ldp % 4 == 0 && k_col % 4 == 0 && p.rot_dims % (p.interleaved ? 4 : 8) == 0;
+            auto kern = !four ? qk_post_kernel<T> : d.dim <= 128 ? qk_post4_kernel<T, 1> : d.dim <= 256 ? qk_post4_kernel<T, 2> : qk_post4_kernel<T, 4>;
+            FORGE_CUDA(launch_pdl(kern, dim3((d.heads + d.groups + 7) / 8, part.n), dim3(256), smem, st, d, p, proj + size_t(r0) * ldp, ldp, k_col, q_norm, k_norm,
                                   reinterpret_cast<const float2*>(rope), static_cast<T*>(q) + size_t(r0) * d.heads * d.dim_p, static_cast<T*>(cache), place + r0, part));
             FORGE_LAUNCH_CHECK();
         }
@@ -291,6 +559,7 @@ bool attn_rows_supported(const AttnDims& d) { return d.vdim_p <= 512 && smem_byt
 int32_t attn_rows(const AttnDims& d, int dtype, const void* q, const void* cache, const float* gate, const float* sink, void* out, int out_ld, const StepRows& rows, int max_keys, cudaStream_t st) {
     if (rows.n <= 0) return FORGE_OK;
     if (!attn_rows_supported(d)) { set_error("row attention: head sizes %d / %d unsupported", d.dim, d.vdim); return FORGE_ERR_SHAPE; }
+    if (dtype == FORGE_BF16 && mma_supported(d)) return run_mma(d, q, cache, gate, sink, out, out_ld, rows, max_keys, st);
     const int gq = d.heads / d.groups, blocks = (gq + 3) / 4;
     int splits = 1;   // about two CTAs per SM, no split shorter than one round of its warps
     while (splits < 8 && rows.n * d.groups * blocks * splits * 2 <= 296 && max_keys > splits * kThreads) splits *= 2;

@@ -66,6 +66,7 @@ struct RowScale {
     float inv_n = 0.f, eps = 0.f, mul = 1.f;
     const int32_t* row = nullptr;
 };
+inline int scale_parts(int width) { return pad_to((width + 31) / 32, 4); }   // (the padding stays zero)
 constexpr int kScaleRows = 32;   // products of more tokens take one sum per row (row_sums)
 struct OutSeg {
     int kind = SEG_F32, row0 = 0, rows = 0, ld = 0;
@@ -191,6 +192,41 @@ __device__ __forceinline__ float leave_value(const After& a, float x, size_t t, 
     if (a.kind == AFTER_RMS) {
         const float s = warp_sum(ok ? x * x : 0.f);
         if ((threadIdx.x & 31) == 0 && ok) a.sums[t * a.parts + col / 32] = s;
+    }
+    return x;
+}
+// The same with four neighbouring columns from `col` per lane, eight lanes per part; sizes and strides are multiples of four.
+__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put4(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+__device__ __forceinline__ float4 get4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 get4(const __nv_bfloat16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+__device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+template <typename T>
+__device__ __forceinline__ float4 leave_four(const After& a, float4 x, size_t t, size_t stride, int col, bool ok) {
+    if (ok) {
+        if (a.keep) put4(a.keep + t * stride + col, x);
+        if (a.plus) x = add4(x, get4(a.plus + col));
+        if (a.again) x = add4(x, get4(a.again + t * stride + col));
+        T* dst = static_cast<T*>(a.dst) + t * a.ld + col;
+        if (a.kind == AFTER_DYT) {
+            const float4 w = get4(a.w + col), b = get4(a.b + col);
+            put4(dst, make_float4(dynamic_tanh(x.x, a.alpha, w.x, b.x), dynamic_tanh(x.y, a.alpha, w.y, b.y), dynamic_tanh(x.z, a.alpha, w.z, b.z), dynamic_tanh(x.w, a.alpha, w.w, b.w)));
+        } else if (a.kind == AFTER_CAST) put4(dst, x);
+        else if (a.kind == AFTER_RMS) { put4(dst, mul4(x, get4(a.w + col))); if (a.w2) put4(dst + a.col2, mul4(x, get4(a.w2 + col))); }
+    }
+    if (a.kind == AFTER_RMS) {
+        float s = ok ? fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w))) : 0.f;
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        if ((threadIdx.x & 7) == 0 && ok) a.sums[t * a.parts + col / 32] = s;
     }
     return x;
 }

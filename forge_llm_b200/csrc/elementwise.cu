@@ -187,6 +187,26 @@ __global__ void embed_rows_kernel(const EmbedArgs a) {
         }
         pair = static_cast<const T*>(a.bigram) + size_t(row) * a.width;
     }
+    T* const next = static_cast<T*>(a.after.dst) + size_t(r) * a.after.ld;
+    if (a.width % 4 == 0) {   // four columns per thread; whole warps stay in the loop
+        const int n = (a.width_p / 4 + 31) & ~31;
+        for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < n; i += gridDim.y * blockDim.x) {
+            const int c = i * 4;
+            const bool ok = c < a.width;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (ok) {
+                v = get4(src + c);
+                v = make_float4(v.x * a.scale, v.y * a.scale, v.z * a.scale, v.w * a.scale);
+                if (pair) v = add4(v, get4(pair + c));
+                if (a.x0_f32) put4(a.x0_f32 + size_t(r) * a.width + c, v);
+            }
+            if (a.x0 && c < a.width_p) put4(static_cast<T*>(a.x0) + size_t(r) * a.x0_ld + c, v);
+            if (!ok && c < a.width_p) { put4(next + c, v); if (a.after.w2) put4(next + a.after.col2 + c, v); }
+            v = leave_four<T>(a.after, v, size_t(r), size_t(a.width), c, ok);
+            if (ok) put4(a.x + size_t(r) * a.width + c, v);
+        }
+        return;
+    }
     for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < a.width_p; i += gridDim.y * blockDim.x) {   // width_p is a multiple of 64: whole warps
         const bool ok = i < a.width;
         float v = ok ? to_f(src[i]) * a.scale : 0.f;
@@ -194,8 +214,8 @@ __global__ void embed_rows_kernel(const EmbedArgs a) {
         if (ok && a.x0_f32) a.x0_f32[size_t(r) * a.width + i] = v;
         if (a.x0) static_cast<T*>(a.x0)[size_t(r) * a.x0_ld + i] = to_t<T>(v);
         if (!ok) {
-            static_cast<T*>(a.after.dst)[size_t(r) * a.after.ld + i] = to_t<T>(0.f);
-            if (a.after.w2) static_cast<T*>(a.after.dst)[size_t(r) * a.after.ld + a.after.col2 + i] = to_t<T>(0.f);
+            next[i] = to_t<T>(0.f);
+            if (a.after.w2) next[a.after.col2 + i] = to_t<T>(0.f);
         }
         v = leave_value<T>(a.after, v, size_t(r), size_t(a.width), i, ok);
         if (ok) a.x[size_t(r) * a.width + i] = v;

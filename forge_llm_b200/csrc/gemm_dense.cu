@@ -10,7 +10,8 @@
 // arrival.  Nobody waits for another CTA.  Up to 32 tokens with at most one tile per SM, the CTAs of a tile form a cluster instead: each takes
 // an equal part of its K steps and finishes some of its tokens, for which the others store their parts into its shared memory.  The ring of the sixteen-token form leaves room for a second CTA on the SM: the next product's weights are
 // requested while this one ends.
-// Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = epilogue (TMEM lane = weight row).
+// Warp roles: 0 = TMA producer, 1 = TMEM allocation and MMA issue, the rest = epilogue (TMEM lane = weight row): four warps, or for more than 32
+// tokens eight, two per 32 rows, each with half of the columns.
 // The weights lie in memory as the very images the ring holds (dense_tile_image), so a stage is one contiguous 16 KB bulk copy.
 // Accumulators are double buffered in tensor memory: the epilogue of one tile runs under the products of the next.
 // The weight stages of the ring are requested before the dependency wait of a programmatic launch, the activations after.
@@ -32,36 +33,30 @@ namespace {
 using namespace tc5;
 
 constexpr int BK = 64;
-constexpr int kThreads = 192;
+template <int NT> constexpr int kEpilogueWarps = NT <= 32 ? 4 : 8;
+template <int NT> constexpr int kThreads = 64 + 32 * kEpilogueWarps<NT>;
 
-__device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
+// activations: bfloat16 models take the fast exponential and quotient, whose errors are far inside the rounding of what is stored
+template <typename T> __device__ __forceinline__ float act_sigmoid(float x, float v) {   // x * sigmoid(v)
+    if constexpr (sizeof(T) == 2) return __fdividef(x, 1.0f + __expf(-v));
+    else return x / (1.0f + expf(-v));
+}
+template <typename T> __device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
-    return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+    return act_sigmoid<T>(g, 1.702f * g) * (u + 1.0f);
 }
 
 // The fields of a segment this thread's row needs, in registers: a store through a pointer may not make the compiler fetch them
 // again for every value.
 template <typename T>
 struct RowOut {
-    int kind;
+    int kind, seg;
     bool ok;                 // the row belongs to a segment
     bool fresh;
     size_t ld;
     float* f32; T* t;        // the row's place of token 0
     const int32_t* place;
-    int after;
-    T* next; size_t next_ld;
-    T* next2;                // the second norm's
-    float* sums; size_t parts;
-    float* keep; const float* again;
-    float limit, mul, add, alpha, nw, nb, plus;
-    __device__ __forceinline__ float next_value(float x) const { return after == AFTER_DYT ? dynamic_tanh(x, alpha, nw, nb) : after == AFTER_RMS ? x * nw : x; }
-    // a finished value of the stream (token t): the entry of a pass of a loop
-    __device__ __forceinline__ float enter(float x, size_t t) const {
-        if (keep) keep[t * ld] = x;
-        if (again) x += again[t * ld];
-        return x + plus;
-    }
+    float limit, mul, add, nw, nb, plus;
 };
 template <typename T>
 __device__ __forceinline__ RowOut<T> row_out(const DenseOut& o, int row, int first_row) {
@@ -74,6 +69,7 @@ __device__ __forceinline__ RowOut<T> row_out(const DenseOut& o, int row, int fir
     const OutSeg& g = o.seg[s];
     const int r = row - g.row0, group = g.group;
     q.kind = g.kind;
+    q.seg = s;
     q.ok = r < g.rows;
     q.ld = size_t(g.ld);
     q.fresh = g.fresh;
@@ -82,24 +78,44 @@ __device__ __forceinline__ RowOut<T> row_out(const DenseOut& o, int row, int fir
     q.t = static_cast<T*>(g.dst) + col;
     q.place = g.place;
     q.limit = g.limit;
-    if (q.kind == SEG_RESID) {
-        q.after = g.after.kind;   // of the whole warp
-        if (q.after == AFTER_RMS) { q.sums = g.after.sums + (first_row - g.row0) / 32; q.parts = size_t(g.after.parts); }
-    }
     if (q.ok) {
         if (g.mul) q.mul = g.mul[r];
         if (g.add) q.add = g.add[r];
         if (q.kind == SEG_RESID) {
-            if (q.after == AFTER_DYT) { q.alpha = g.after.alpha; q.nw = g.after.w[r]; q.nb = g.after.b[r]; }
-            if (q.after == AFTER_RMS) { q.nw = g.after.w[r]; if (g.after.w2) { q.nb = g.after.w2[r]; q.next2 = static_cast<T*>(g.after.dst) + g.after.col2 + r; } }
-            q.next = static_cast<T*>(g.after.dst) + r; q.next_ld = size_t(g.after.ld);
+            if (g.after.w) q.nw = g.after.w[r];
+            if (g.after.kind == AFTER_DYT) q.nb = g.after.b[r];
+            if (g.after.w2) q.nb = g.after.w2[r];
             if (g.after.plus) q.plus = g.after.plus[r];
-            if (g.after.again) q.again = g.after.again + r;
-            if (g.after.keep) q.keep = g.after.keep + r;
         }
     }
     return q;
 }
+// what a finished row of the stream leaves
+template <typename T>
+struct Leave {
+    int kind;
+    bool two;                // a second norm's input
+    size_t ld, next_ld, parts;
+    T *next, *next2;
+    float alpha, nw, nb, plus;
+    float* sums; float* keep; const float* again;
+    __device__ __forceinline__ Leave(const OutSeg& g, const RowOut<T>& q, int row, int first_row)
+        : kind(g.after.kind), two(g.after.w2 != nullptr), ld(q.ld), next_ld(size_t(g.after.ld)), parts(size_t(g.after.parts)), alpha(g.after.alpha), nw(q.nw), nb(q.nb), plus(q.plus) {
+        const int r = row - g.row0;
+        next = static_cast<T*>(g.after.dst) + r;
+        next2 = next + g.after.col2;
+        sums = kind == AFTER_RMS ? g.after.sums + (first_row - g.row0) / 32 : nullptr;
+        keep = g.after.keep ? g.after.keep + r : nullptr;
+        again = g.after.again ? g.after.again + r : nullptr;
+    }
+    __device__ __forceinline__ float next_value(float x) const { return kind == AFTER_DYT ? dynamic_tanh(x, alpha, nw, nb) : kind == AFTER_RMS ? x * nw : x; }
+    // a finished value of the stream (token t): the entry of a pass of a loop
+    __device__ __forceinline__ float enter(float x, size_t t) const {
+        if (keep) keep[t * ld] = x;
+        if (again) x += again[t * ld];
+        return x + plus;
+    }
+};
 // column of the activations the rows of the tile at `row` are multiplied with
 __device__ __forceinline__ int act_col(const DenseOut& o, int row) {
     int c = 0;
@@ -110,24 +126,24 @@ __device__ __forceinline__ int act_col(const DenseOut& o, int row) {
 // the epilogue of one value v; `up`: the value of the next row, used by the even rows of gated pairs, w: what those are multiplied with; `old`: what dst
 // holds, if it is known; returns the stream's new value
 template <typename T>
-__device__ __forceinline__ float put_one(const RowOut<T>& g, float v, float up, float w, size_t t, float old, bool old_known, bool even_row) {
+__device__ __forceinline__ float put_one(const RowOut<T>& g, const Leave<T>& n, float v, float up, float w, size_t t, float old, bool old_known, bool even_row) {
     float* f = g.f32 + t * g.ld;
     T* h = g.t + t * g.ld;
     switch (g.kind) {
-        case SEG_CLAMPED_GLU: if (even_row) *h = to_t<T>(clamped_glu(v, up, g.limit) * w); break;
-        case SEG_SILU_GLU: if (even_row) *h = to_t<T>(silu(v) * up * w); break;
+        case SEG_CLAMPED_GLU: if (even_row) *h = to_t<T>(clamped_glu<T>(v, up, g.limit) * w); break;
+        case SEG_SILU_GLU: if (even_row) *h = to_t<T>(act_sigmoid<T>(v, v) * up * w); break;
         case SEG_CAST: g.t[(g.place ? size_t(g.place[t]) : t) * g.ld] = to_t<T>(v); break;
-        case SEG_SIGMOID: *h = to_t<T>(sigmoid(v)); break;
-        case SEG_SILU: *h = to_t<T>(silu(v)); break;
+        case SEG_SIGMOID: *h = to_t<T>(act_sigmoid<T>(1.f, v)); break;
+        case SEG_SILU: *h = to_t<T>(act_sigmoid<T>(v, v)); break;
         case SEG_TANH: *h = to_t<T>(tanhf(v)); break;
         case SEG_SIGMOID_F32: *f = sigmoid(v); break;
         case SEG_DECAY: *f = -g.mul * softplus(v); break;
         case SEG_EXP_DECAY: *f = -expf(v); break;
         case SEG_RESID: {
-            const float x = g.enter((g.fresh ? 0.f : old_known ? old : *f) + v, t);
+            const float x = n.enter((g.fresh ? 0.f : old_known ? old : *f) + v, t);
             *f = x;
-            if (g.after) g.next[t * g.next_ld] = to_t<T>(g.next_value(x));
-            if (g.next2) g.next2[t * g.next_ld] = to_t<T>(x * g.nb);
+            if (n.kind) n.next[t * n.next_ld] = to_t<T>(n.next_value(x));
+            if (n.two) n.next2[t * n.next_ld] = to_t<T>(x * n.nb);
             return x;
         }
         default: *f = v;
@@ -137,6 +153,25 @@ __device__ __forceinline__ float put_one(const RowOut<T>& g, float v, float up, 
 
 // the sum of squares behind a token's scale
 __device__ __forceinline__ float row_scale(const RowScale& s, float sum) { return s.mul / sqrtf(sum * s.inv_n + s.eps); }
+
+// of few tokens, lane c: token tok0 + c (parts a multiple of four, or one)
+template <int NT> __device__ __forceinline__ float lane_scale(const RowScale& s, int tok0, int cols, int lane) {
+    constexpr int SHARE = 32 / NT;   // lanes per token
+    const int c = lane % NT, i0 = lane / NT;
+    const bool ok = c < cols;
+    const float* src = s.sums + size_t(ok ? (s.row ? s.row[tok0 + c] : tok0 + c) : 0) * s.parts;
+    float sum = 0.f;
+    if (s.parts == 1) sum = ok ? *src : 0.f;
+    else {
+#pragma unroll 8
+        for (int i = i0; i < s.parts / 4; i += SHARE) {
+            const float4 v = ok ? reinterpret_cast<const float4*>(src)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+            sum += (v.x + v.y) + (v.z + v.w);
+        }
+        if (SHARE == 2) sum += __shfl_xor_sync(0xffffffffu, sum, 16);
+    }
+    return row_scale(s, sum);
+}
 
 enum Mode { PLAIN = 0, GROUPED, LISTED };
 
@@ -203,11 +238,22 @@ template <int NT, int MODE> __device__ __forceinline__ Tile tile_at(const GemmPa
     const int tok0 = (tile % p.tt_count) * NT;
     return Tile{tile / p.tt_count, tok0, min(NT, p.m - tok0), 0, 0};
 }
-template <int MODE> __device__ __forceinline__ int listed_k(const GemmParams& p, int k) {
-    if (MODE != LISTED || k < p.k_fixed) return k;
-    const int a = (k - p.k_fixed) / p.k_group;
-    return k + (p.groups.tiles[a].group - a) * p.k_group;
-}
+// K steps in order -> where they lie
+template <int MODE> struct KMap {
+    int end = 0, shift = 0;
+    __device__ __forceinline__ int at(const GemmParams& p, int k) {
+        if (MODE != LISTED) return k;
+        if (k >= end) {
+            if (k < p.k_fixed) end = p.k_fixed;
+            else {
+                const int a = (k - p.k_fixed) / p.k_group;
+                end = p.k_fixed + (a + 1) * p.k_group;
+                shift = (p.groups.tiles[a].group - a) * p.k_group;
+            }
+        }
+        return k + shift;
+    }
+};
 
 template <int NT> struct Ring {
     static constexpr int X_BYTES = NT * 128, STAGE = 16384 + X_BYTES;
@@ -217,7 +263,7 @@ template <int NT> struct Ring {
 };
 
 template <int NT, int MODE>
-__global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ GemmParams p) {
+__global__ void __launch_bounds__(kThreads<NT>, NT <= 16 ? 2 : 1) gemm_dense_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ GemmParams p) {
     constexpr int STAGE = Ring<NT>::STAGE, STAGES = Ring<NT>::STAGES;
     constexpr uint32_t kCols = Ring<NT>::COLS;
     extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -235,7 +281,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
     } else if (int(blockIdx.x) < p.sharers) { u0 = share_begin(p.units, blockIdx.x, p.sharers); u1 = share_begin(p.units, blockIdx.x + 1, p.sharers); }
     if (tid == 0) {
         for (int s = 0; s < STAGES; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
-        for (int s = 0; s < 2; ++s) { mbar_init(&acc_full[s], 1); mbar_init(&acc_empty[s], 4); }
+        for (int s = 0; s < 2; ++s) { mbar_init(&acc_full[s], 1); mbar_init(&acc_empty[s], kEpilogueWarps<NT>); }
         s_err = 0;
         mbar_fence_init();
     }
@@ -253,6 +299,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
             int groups = MODE == LISTED ? p.groups.max_tiles : 0;
             if constexpr (MODE == GROUPED) { pdl_wait(); groups = *p.groups.n; }
             Work<MODE> ww(p, u0, u1, groups), wx = ww;
+            KMap<MODE> mw, mx;
             int kw = 0;
             size_t image = 0;
             bool more = ww.next();
@@ -264,7 +311,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
             const unsigned char* const weights = static_cast<const unsigned char*>(p.w);
             auto weight_stage = [&](int s) {   // one contiguous image of 128 rows x 64 columns, already swizzled
                 mbar_expect_tx(&full[s], uint32_t(STAGE));
-                bulk_load(ring + size_t(s) * STAGE, weights + (image + listed_k<MODE>(p, ww.k0 + kw)) * 16384, 16384, &full[s]);
+                bulk_load(ring + size_t(s) * STAGE, weights + (image + mw.at(p, ww.k0 + kw)) * 16384, 16384, &full[s]);
                 if (++kw == ww.n) { kw = 0; more = ww.next(); if (more) first_image(); }
             };
             int ahead = 0;
@@ -287,7 +334,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                         if (!mbar_wait(&empty[s], phase, &s_err)) { atomicExch(&s_err, 1); ok = false; break; }
                         weight_stage(s);
                     }
-                    tma_2d(ring + size_t(s) * STAGE + 16384, &map_x, col0 + listed_k<MODE>(p, wx.k0 + k) * BK, tok0, &full[s]);
+                    tma_2d(ring + size_t(s) * STAGE + 16384, &map_x, col0 + mx.at(p, wx.k0 + k) * BK, tok0, &full[s]);
                     if (++s == STAGES) { s = 0; phase ^= 1; }
                 }
             }
@@ -332,8 +379,13 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
         pdl_wait();
         const int quad = warp & 3;
         const uint32_t lane_addr = tmem + (uint32_t(quad * 32) << 16);
-        constexpr int CH = NT < 32 ? NT : 32;   // columns per read
+        constexpr int CH = NT == 32 ? 32 : 16;   // columns per read
+        constexpr int EW = kEpilogueWarps<NT>, MINE = NT / (EW / 4);
+        const int c_begin = (warp - 2) / 4 * MINE, c_end = c_begin + MINE;   // this warp's columns
+        auto epilogue_sync = [&]() { asm volatile("bar.sync 1, %0;" ::"n"(EW * 32) : "memory"); };
         int seg_i = 0;
+        float col_scale = 1.f;   // of the tokens, lane c: of column c (few tokens: all of the tile's)
+        int scaled_tok0 = -1, scaled_cols = 0;
         const int groups = MODE != PLAIN ? *p.groups.n : 0;
         Work<MODE> w(p, u0, u1, groups);
         // a CTA of a cluster takes part in finishing its tile even if the list left it no steps
@@ -354,17 +406,10 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
             // every warp's rows lie in one segment (segments start at multiples of 32 rows)
             RowOut<__nv_bfloat16> g = row_out<__nv_bfloat16>(p.out, row, row0);
             if constexpr (MODE == GROUPED) { g.t += at_tile.group * p.group_dst; g.f32 += at_tile.group * p.group_dst; }
-            // scales of the tokens, lane c: of column c (few tokens: all of the tile's)
-            float col_scale = 1.f;
-            auto scale_row = [&](int t) { return size_t(p.scale.row ? p.scale.row[t] : t); };
-            if (NT <= 32 && p.scale.sums)
-                for (int c = 0; c < cols; ++c) {
-                    const float* src = p.scale.sums + scale_row(tok0 + c) * p.scale.parts;
-                    float sum = 0.f;
-                    for (int i = lane; i < p.scale.parts; i += 32) sum += src[i];
-                    sum = row_scale(p.scale, warp_sum(sum));
-                    if (lane == c) col_scale = sum;
-                }
+            if (NT <= 32 && p.scale.sums && (tok0 != scaled_tok0 || cols != scaled_cols)) {
+                col_scale = lane_scale<NT <= 32 ? NT : 32>(p.scale, tok0, cols, lane);
+                scaled_tok0 = tok0; scaled_cols = cols;
+            }
             const float* pair_w = MODE == GROUPED && p.groups.weight ? p.groups.weight + at_tile.w0 : nullptr;
             float x_old[CH];   // few tokens: the residual is on its way while the product is formed
             if (NT <= 32 && g.kind == SEG_RESID && g.ok && !g.fresh)
@@ -377,7 +422,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                 const int n_c = cols - c0;
                 const size_t t0 = size_t(tok0 + c0);
                 if (p.scale.sums) {
-                    if (NT > 32) col_scale = lane < n_c ? row_scale(p.scale, p.scale.sums[scale_row(tok0 + c0 + lane)]) : 1.f;
+                    if (NT > 32) col_scale = lane < n_c ? row_scale(p.scale, p.scale.sums[p.scale.row ? p.scale.row[t0 + lane] : t0 + lane]) : 1.f;
 #pragma unroll
                     for (int c = 0; c < CH; ++c) v[c] *= __shfl_sync(0xffffffffu, col_scale, c);
                 }
@@ -396,10 +441,11 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                 if (n_c == 1) {   // one token: little code
                     const float got = __shfl_xor_sync(0xffffffffu, v[0], 1);
                     float x = 0.f;
-                    if (g.ok) x = put_one(g, v[0], got, pair_w ? pair_w[c0] : 1.f, t0, NT <= 32 ? x_old[0] : 0.f, NT <= 32, !(lane & 1));
-                    if (g.sums) {
+                    const Leave<__nv_bfloat16> n(p.out.seg[g.seg], g, row, row0);
+                    if (g.ok) x = put_one(g, n, v[0], got, pair_w ? pair_w[c0] : 1.f, t0, NT <= 32 ? x_old[0] : 0.f, NT <= 32, !(lane & 1));
+                    if (g.kind == SEG_RESID && n.sums) {
                         x = warp_sum(x * x);
-                        if (lane == 0) g.sums[t0 * g.parts] = x;
+                        if (lane == 0) n.sums[t0 * n.parts] = x;
                     }
                 } else if (g.kind == SEG_CLAMPED_GLU || g.kind == SEG_SILU_GLU) {
                     // neighbouring lanes hold gate_j and up_j: the even lane takes the first half of the columns
@@ -410,35 +456,36 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                     for (int c = 0; c < CH / 2; ++c) {
                         const float got = __shfl_xor_sync(0xffffffffu, even ? v[CH / 2 + c] : v[c], 1);
                         const float ga = even ? v[c] : got, up = even ? got : v[CH / 2 + c];
-                        if (g.ok && mine + c < n_c) dst[c * g.ld] = __float2bfloat16_rn((clamped ? clamped_glu(ga, up, g.limit) : silu(ga) * up) * (pair_w ? pair_w[c0 + mine + c] : 1.f));
+                        if (g.ok && mine + c < n_c) dst[c * g.ld] = __float2bfloat16_rn((clamped ? clamped_glu<__nv_bfloat16>(ga, up, g.limit) : act_sigmoid<__nv_bfloat16>(ga, ga) * up) * (pair_w ? pair_w[c0 + mine + c] : 1.f));
                     }
                 } else if (g.kind == SEG_RESID) {
+                    const Leave<__nv_bfloat16> n(p.out.seg[g.seg], g, row, row0);
                     float* dst = g.f32 + t0 * g.ld;
                     float x[CH];
 #pragma unroll
                     for (int c = 0; c < CH; ++c) x[c] = !g.ok || g.fresh ? 0.f : NT <= 32 ? x_old[c] : c < n_c ? dst[c * g.ld] : 0.f;   // all loads before the first store
-                    if (g.keep || g.again) {
+                    if (n.keep || n.again) {
 #pragma unroll
-                        for (int c = 0; c < CH; ++c) { x[c] += v[c]; if (c < n_c) x[c] = g.enter(x[c], t0 + c); }
+                        for (int c = 0; c < CH; ++c) { x[c] += v[c]; if (g.ok && c < n_c) x[c] = n.enter(x[c], t0 + c); }
                     } else {
 #pragma unroll
-                        for (int c = 0; c < CH; ++c) x[c] += v[c] + g.plus;
+                        for (int c = 0; c < CH; ++c) x[c] += v[c] + n.plus;
                     }
                     if (g.ok) {
 #pragma unroll
                         for (int c = 0; c < CH; ++c) if (c < n_c) dst[c * g.ld] = x[c];
-                        if (g.after) {
-                            __nv_bfloat16* nx = g.next + t0 * g.next_ld;
+                        if (n.kind) {
+                            __nv_bfloat16* nx = n.next + t0 * n.next_ld;
 #pragma unroll
-                            for (int c = 0; c < CH; ++c) if (c < n_c) nx[c * g.next_ld] = __float2bfloat16_rn(g.next_value(x[c]));
+                            for (int c = 0; c < CH; ++c) if (c < n_c) nx[c * n.next_ld] = __float2bfloat16_rn(n.next_value(x[c]));
                         }
-                        if (g.next2) {
-                            __nv_bfloat16* nx = g.next2 + t0 * g.next_ld;
+                        if (n.two) {
+                            __nv_bfloat16* nx = n.next2 + t0 * n.next_ld;
 #pragma unroll
-                            for (int c = 0; c < CH; ++c) if (c < n_c) nx[c * g.next_ld] = __float2bfloat16_rn(x[c] * g.nb);
+                            for (int c = 0; c < CH; ++c) if (c < n_c) nx[c * n.next_ld] = __float2bfloat16_rn(x[c] * n.nb);
                         }
                     }
-                    if (g.sums) {   // lane c ends with the sum over the warp's rows of column c's squares
+                    if (n.sums) {   // lane c ends with the sum over the warp's rows of column c's squares
 #pragma unroll
                         for (int c = 0; c < CH; ++c) x[c] = g.ok ? x[c] * x[c] : 0.f;
                         if constexpr (CH == 16)
@@ -452,17 +499,20 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                                 const float send = up ? x[c] : x[c + o], mine = up ? x[c + o] : x[c];
                                 x[c] = mine + __shfl_xor_sync(0xffffffffu, send, o);
                             }
-                        if (lane < CH && lane < n_c) g.sums[(t0 + lane) * g.parts] = x[0];
+                        if (lane < CH && lane < n_c) n.sums[(t0 + lane) * n.parts] = x[0];
                     }
                 } else if (g.ok) switch (g.kind) {
                     case SEG_CAST:
                         if (g.place) {
+                            int to[CH];
 #pragma unroll
-                            for (int c = 0; c < CH; ++c) if (c < n_c) g.t[size_t(g.place[t0 + c]) * g.ld] = __float2bfloat16_rn(v[c]);
+                            for (int c = 0; c < CH; ++c) to[c] = c < n_c ? g.place[t0 + c] : 0;
+#pragma unroll
+                            for (int c = 0; c < CH; ++c) if (c < n_c) g.t[size_t(to[c]) * g.ld] = __float2bfloat16_rn(v[c]);
                         } else put_t([](float x) { return x; });
                         break;
-                    case SEG_SIGMOID: put_t([](float x) { return sigmoid(x); }); break;
-                    case SEG_SILU: put_t([](float x) { return silu(x); }); break;
+                    case SEG_SIGMOID: put_t([](float x) { return act_sigmoid<__nv_bfloat16>(1.f, x); }); break;
+                    case SEG_SILU: put_t([](float x) { return act_sigmoid<__nv_bfloat16>(x, x); }); break;
                     case SEG_TANH: put_t([](float x) { return tanhf(x); }); break;
                     case SEG_SIGMOID_F32: put_f([](float x) { return sigmoid(x); }); break;
                     case SEG_DECAY: put_f([&](float x) { return -g.mul * softplus(x); }); break;
@@ -480,13 +530,14 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
             };
             if (MODE == GROUPED || MODE == LISTED ? p.cluster <= 1 : n == p.nk) {
 #pragma unroll 1
-                for (int c0 = 0; c0 < NT && c0 < cols; c0 += CH) {
+                for (int c0 = c_begin; c0 < c_end && c0 < cols; c0 += CH) {
                     float v[CH];
                     load(c0, v);
                     finish(c0, v);
                 }
             } else if (NT <= 32 && p.cluster > 1) {
                 // the tokens 4 c .. 4 c + 3 are finished by CTA c % cluster: box [c / cluster][sender][row][4]
+                const Leave<__nv_bfloat16> nx(p.out.seg[g.seg], g, row, row0);
                 const int at = (quad * 32 + lane) * 4, groups = (cols + 3) / 4, senders = p.cluster - 1;
                 float* box = reinterpret_cast<float*>(ring + size_t(STAGES) * STAGE);
                 float v[CH];
@@ -523,10 +574,10 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                         val += g.add;
                         const float got = __shfl_xor_sync(0xffffffffu, val, 1);
                         float x = 0.f;
-                        if (g.ok) x = put_one(g, val, got, pair_w ? pair_w[c0 + e] : 1.f, size_t(tok0 + c0 + e), old[0], true, !(lane & 1));
-                        if (g.sums) {
+                        if (g.ok) x = put_one(g, nx, val, got, pair_w ? pair_w[c0 + e] : 1.f, size_t(tok0 + c0 + e), old[0], true, !(lane & 1));
+                        if (g.kind == SEG_RESID && nx.sums) {
                             x = warp_sum(x * x);
-                            if (lane == 0) g.sums[size_t(tok0 + c0 + e) * g.parts] = x;
+                            if (lane == 0) nx.sums[size_t(tok0 + c0 + e) * nx.parts] = x;
                         }
                         t[0] = t[1]; t[1] = t[2]; t[2] = t[3];
                         old[0] = old[1]; old[1] = old[2]; old[2] = old[3];
@@ -536,7 +587,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                 // a shared tile: this CTA's part goes to its slot (0: the part its share starts with, 1: the other one)
                 float* mine = p.part + (size_t(blockIdx.x) * 2 + (u0 >= t_begin ? 0 : 1)) * (NT * 128);
 #pragma unroll 1
-                for (int c0 = 0; c0 < NT && c0 < cols; c0 += CH) {
+                for (int c0 = c_begin; c0 < c_end && c0 < cols; c0 += CH) {
                     float v[CH];
                     load(c0, v);
 #pragma unroll
@@ -544,22 +595,22 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                 }
                 const int first = share_of(p.units, t_begin, p.sharers), last = share_of(p.units, t_end - 1, p.sharers);
                 __threadfence();
-                asm volatile("bar.sync 1, 128;" ::: "memory");
+                epilogue_sync();
                 if (tid == 64) {
                     const int old = atomicAdd(p.tickets + tile, 1);
                     s_last = old == last - first;
                     if (s_last) p.tickets[tile] = 0;
                 }
-                asm volatile("bar.sync 1, 128;" ::: "memory");
+                epilogue_sync();
                 if (s_last) {
                     __threadfence();
 #pragma unroll 1
-                    for (int c0 = 0; c0 < NT && c0 < cols; c0 += CH) {
+                    for (int c0 = c_begin; c0 < c_end && c0 < cols; c0 += CH) {
                         float v[CH];
 #pragma unroll
                         for (int c = 0; c < CH; ++c) v[c] = 0.f;
                         // only the first share of the tile may be the second part of its CTA; loads of QB shares in flight together
-                        constexpr int QB = CH == 16 ? 4 : 2;
+                        constexpr int QB = NT <= 16 ? 4 : 2;
                         const int n_c = cols - c0;
                         const int first_slot = share_begin(p.units, first, p.sharers) >= t_begin ? 0 : 1;
                         for (int q = first; q <= last; q += QB) {
@@ -578,7 +629,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 16 ? 2 : 1) gemm_dense_kernel(
                         finish(c0, v);
                     }
                 }
-                asm volatile("bar.sync 1, 128;" ::: "memory");   // s_last is read before it is written again
+                epilogue_sync();   // s_last is read before it is written again
             }
             fence_before();
             __syncwarp();
@@ -608,7 +659,7 @@ int32_t cluster_parts(long long tiles, int nk, size_t smem, int* parts) {
         for (int c = 1; c <= 8; ++c) {
             cudaLaunchConfig_t cfg{};
             cudaLaunchAttribute at[1];
-            cfg.gridDim = dim3(unsigned(c * 148)); cfg.blockDim = dim3(kThreads); cfg.dynamicSmemBytes = std::max(smem, size_t(120) * 1024);   // one CTA per SM
+            cfg.gridDim = dim3(unsigned(c * 148)); cfg.blockDim = dim3(kThreads<NT>); cfg.dynamicSmemBytes = std::max(smem, size_t(120) * 1024);   // one CTA per SM
             at[0].id = cudaLaunchAttributeClusterDimension;
             at[0].val.clusterDim.x = unsigned(c); at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
             cfg.attrs = at; cfg.numAttrs = 1;
@@ -621,6 +672,7 @@ int32_t cluster_parts(long long tiles, int nk, size_t smem, int* parts) {
     return FORGE_OK;
 }
 
+constexpr int kShareSteps = 96;   // what sharing a tile of 256 tokens costs, in K steps (measured)
 template <int NT, int MODE>
 int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, int act_rows, GemmParams& p, int sms, cudaStream_t st) {
     CUtensorMap mx;
@@ -637,7 +689,7 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, int act_
         FORGE_TRY((cluster_parts<NT, MODE>(tiles, p.nk, smem, &parts)));
         if (parts > 0) {
             p.cluster = parts;
-            FORGE_CUDA(launch_pdl_cluster(kern, dim3(unsigned(tiles * parts)), dim3(kThreads), parts, smem, st, mx, p));
+            FORGE_CUDA(launch_pdl_cluster(kern, dim3(unsigned(tiles * parts)), dim3(kThreads<NT>), parts, smem, st, mx, p));
             FORGE_LAUNCH_CHECK();
             return FORGE_OK;
         }
@@ -645,7 +697,7 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, int act_
     if constexpr (MODE == LISTED) { set_error("listed product: %lld tiles are too many", tiles); return FORGE_ERR_SHAPE; }
     if constexpr (MODE == GROUPED) {   // sixteen-token tiles: two CTAs fit an SM
         if (tiles * p.nk > INT32_MAX) { set_error("product in groups: %lld tiles of %d K steps are too many", tiles, p.nk); return FORGE_ERR_SHAPE; }
-        FORGE_CUDA(launch_pdl(kern, dim3(unsigned(std::min((long long)sms * (NT <= 16 ? 2 : 1), tiles))), dim3(kThreads), smem, st, mx, p));
+        FORGE_CUDA(launch_pdl(kern, dim3(unsigned(std::min((long long)sms * (NT <= 16 ? 2 : 1), tiles))), dim3(kThreads<NT>), smem, st, mx, p));
         FORGE_LAUNCH_CHECK();
         return FORGE_OK;
     }
@@ -655,10 +707,10 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, int act_
     if (tiles * p.nk > INT32_MAX || (units + 1) * grid > INT32_MAX) { set_error("dense product: %lld tiles of %d K steps are too many", tiles, p.nk); return FORGE_ERR_SHAPE; }
     p.units = uint32_t(units);
     p.sharers = int(std::min((long long)grid, (units + 1) / 2));
-    // leaving and adding shares costs about NT / 32 K steps: where whole tiles are no dearer, every CTA takes at most one
+    // leaving and adding shares costs about NT * kShareSteps / 256 K steps: where whole tiles are no dearer, every CTA takes at most one
     const long long rest = tiles - (long long)p.waves * grid;
-    if (rest > 0 && rest <= grid && p.nk <= units / grid + NT / 32) p.sharers = int(rest);
-    FORGE_CUDA(launch_pdl(kern, dim3(grid), dim3(kThreads), smem, st, mx, p));
+    if (rest > 0 && rest <= grid && p.nk <= units / grid + NT * kShareSteps / 256) p.sharers = int(rest);
+    FORGE_CUDA(launch_pdl(kern, dim3(grid), dim3(kThreads<NT>), smem, st, mx, p));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
@@ -731,6 +783,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
         g[i] = row_out<float>(out, row0 + rr + i, (row0 + rr) & ~31);
         g[i].t += dst_off; g[i].f32 += dst_off;
     }
+    const bool resid = g[0].kind == SEG_RESID;
 #pragma unroll
     for (int j = 0; j < PT; ++j) {
         const size_t t = size_t(tok0 + tt + j);
@@ -741,14 +794,16 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 #pragma unroll
         for (int i = 0; i < 4; ++i)
             if (live && g[i].ok) {
-                const float xn = put_one(g[i], v[i], v[i | 1], pair_w ? pair_w[tt + j] : 1.f, t, 0.f, false, !(i & 1));
+                const Leave<float> n(out.seg[g[i].seg], g[i], row0 + rr + i, (row0 + rr) & ~31);
+                const float xn = put_one(g[i], n, v[i], v[i | 1], pair_w ? pair_w[tt + j] : 1.f, t, 0.f, false, !(i & 1));
                 sum = fmaf(xn, xn, sum);
             }
-        if (__any_sync(0xffffffffu, g[0].sums != nullptr)) {   // over the 32 rows of eight neighbouring lanes
+        if (__any_sync(0xffffffffu, resid)) {   // over the 32 rows of eight neighbouring lanes
             sum += __shfl_xor_sync(0xffffffffu, sum, 1);
             sum += __shfl_xor_sync(0xffffffffu, sum, 2);
             sum += __shfl_xor_sync(0xffffffffu, sum, 4);
-            if (live && g[0].sums && !(tid & 7)) g[0].sums[t * g[0].parts] = sum;
+            const After& a = out.seg[g[0].seg].after;
+            if (live && resid && a.kind == AFTER_RMS && !(tid & 7)) a.sums[t * a.parts + (((row0 + rr) & ~31) - out.seg[g[0].seg].row0) / 32] = sum;
         }
     }
 }

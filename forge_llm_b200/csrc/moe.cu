@@ -142,6 +142,21 @@ __global__ void __launch_bounds__(1024) slots_kernel(const RouterDims d, int row
 template <typename T>
 __global__ void __launch_bounds__(256) add_experts_kernel(float* __restrict__ x, const float* __restrict__ y, const int32_t* __restrict__ slot, int top, int width, const After after) {
     const int r = blockIdx.x;
+    if (width % 4 == 0) {   // four columns per thread
+        for (int c0 = blockIdx.y * 1024; c0 < width; c0 += gridDim.y * 1024) {
+            const int c = c0 + threadIdx.x * 4;
+            const bool ok = c < width;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (ok) {
+                v = get4(x + size_t(r) * width + c);
+#pragma unroll 2
+                for (int k = 0; k < top; ++k) v = add4(v, get4(y + size_t(slot[size_t(r) * top + k]) * width + c));
+            }
+            v = leave_four<T>(after, v, size_t(r), size_t(width), c, ok);
+            if (ok) put4(x + size_t(r) * width + c, v);
+        }
+        return;
+    }
     for (int c0 = blockIdx.y * 256; c0 < width; c0 += gridDim.y * 256) {
         const int c = c0 + threadIdx.x;
         const bool ok = c < width;

@@ -473,7 +473,7 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
     FORGE_TRY(grow(m, S.h, r * h));
     if (S.loop_in.N) FORGE_TRY(grow(m, S.cat, r * 2 * WP * es));
     if (S.spec.adds_loop()) FORGE_TRY(grow(m, S.x0, r * W * 4));
-    if (S.spec.arch->norm == Norm::RmsPlusOne) { FORGE_TRY(grow(m, S.sums, r * ((W + 31) / 32) * 4)); FORGE_TRY(grow(m, S.sum1, r * 4)); }
+    if (S.spec.arch->norm == Norm::RmsPlusOne) { FORGE_TRY(grow(m, S.sums, r * scale_parts(int(W)) * 4)); FORGE_TRY(grow(m, S.sum1, r * 4)); }
     FORGE_TRY(grow(m, S.place, r * sizeof(int32_t)));
     const std::pair<StackModel::Buf*, size_t> sizes[] = {{&S.proj, proj}, {&S.gate, gate}, {&S.mid, mid}, {&S.q, q}, {&S.part, part}, {&S.ml, heads}, {&S.hgate, hgate}, {&S.decay, decay},
         {&S.beta, beta}, {&S.low, low}, {&S.conv, conv}, {&S.unit, unit}, {&S.o, o}, {&S.pair, pair}, {&S.c_half, cb.half}, {&S.c_f32, cb.f32}, {&S.ctx_c, cc}, {&S.ctx_r, cr}, {&S.ctx_k, ck}, {&S.ctx_v, cv},
@@ -512,7 +512,7 @@ RowScale stream_scale(const StackModel& S, int rows) {
     if (S.spec.arch->norm != Norm::RmsPlusOne) return r;
     const bool summed = rows > kScaleRows;
     r.sums = static_cast<const float*>(summed ? S.sum1.p : S.sums.p);
-    r.parts = summed ? 1 : (S.spec.width + 31) / 32;
+    r.parts = summed ? 1 : scale_parts(S.spec.width);
     r.inv_n = 1.0f / float(S.spec.width); r.eps = S.spec.eps;
     return r;
 }
@@ -536,7 +536,7 @@ struct Sequence {
     After norm(const StreamNorm& d, int ld) {
         After a;
         a.dst = S.h.p; a.ld = ld; a.w = d.w;
-        if (rms()) { a.kind = AFTER_RMS; a.sums = static_cast<float*>(S.sums.p); a.parts = (W + 31) / 32; }
+        if (rms()) { a.kind = AFTER_RMS; a.sums = static_cast<float*>(S.sums.p); a.parts = scale_parts(W); }
         else { a.kind = AFTER_DYT; a.alpha = d.alpha; a.b = d.b; }
         return a;
     }
@@ -566,7 +566,7 @@ struct Sequence {
     static void resid(DenseOut* o, float* x, int W, const After& after) { o->add(SEG_RESID, 0, W, x, W).after = after; }
     float* x() { return static_cast<float*>(S.x.p); }
     // RMS norms: the tokens' scales from the sums that the stream's last writer left
-    int32_t stats() { return rms() && s.scale_rows > kScaleRows ? row_sums(static_cast<float*>(S.sum1.p), static_cast<float*>(S.sums.p), n, (W + 31) / 32, st) : FORGE_OK; }
+    int32_t stats() { return rms() && s.scale_rows > kScaleRows ? row_sums(static_cast<float*>(S.sum1.p), static_cast<float*>(S.sums.p), n, scale_parts(W), st) : FORGE_OK; }
     RowScale scale() const { return stream_scale(S, s.scale_rows); }
 
     int32_t run() {
