@@ -258,7 +258,10 @@ int32_t attn_prefill_kv(const PromptDims& d, const PromptAttnArgs& a, cudaStream
     if (d.rot_p == 0) mr = mk;   // no rotated part: never read
     else FORGE_TRY(make_map_2d(&mr, a.krot, uint64_t(d.rot_p), uint64_t(a.ctx_rows), uint64_t(d.rot_p) * 2, BN));
     FORGE_TRY(make_map_3d(&mv, a.v, uint64_t(d.vdim_p), G, uint64_t(a.ctx_rows), uint64_t(d.vdim_p) * 2, v_row, BN));
-    Params p{d, a, d.scale * 1.4426950408889634f, smem_bytes(d, 3) <= 220 * 1024 ? 3 : 2};
+    // three stages, or two where that lets two CTAs share an SM
+    auto fit = [&](int stages, size_t ctas) { return ctas * (smem_bytes(d, stages) + 1024) <= 226 * 1024; };
+    const int stages = fit(3, 2) ? 3 : fit(2, 2) && d.vdim_p <= 128 ? 2 : fit(3, 1) ? 3 : 2;
+    Params p{d, a, d.scale * 1.4426950408889634f, stages};
     const size_t smem = smem_bytes(d, p.stages);
     auto go = [&](auto kern) -> int32_t {
         FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));

@@ -387,10 +387,18 @@ int32_t run_mma(const AttnDims& d, const void* q, const void* cache, const float
 constexpr int kQkDims = 16;   // values per lane at most
 template <typename T>
 __global__ void __launch_bounds__(256) qk_post_kernel(const AttnDims d, const QkPost p, const float* proj, int ldp, int k_col, const float* __restrict__ q_norm,
-                                                      const float* __restrict__ k_norm, const float2* __restrict__ rope, T* q, T* cache, const int32_t* place, const StepRows rows) {
+                                                      const float* __restrict__ k_norm, const float2* __restrict__ rope, T* q, T* cache, const int32_t* place, const StepRows rows, const RouteBeside route) {
     extern __shared__ float sm[];
     __shared__ float red[2][8];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = blockIdx.y, h = blockIdx.x * 8 + warp;
+    if (route.logits && blockIdx.x == gridDim.x - 1) {
+        if (r > 0) return;
+        pdl_trigger();
+        route_few_clear(route.d, sm);
+        pdl_wait();
+        route_few_rows(route.d, route.logits, rows.n, route.t, sm);
+        return;
+    }
     const bool on = h < d.heads + d.groups, is_q = h < d.heads;
     const int g = is_q ? h : h - d.heads, half = p.rot_dims / 2;
     const float* w = is_q ? q_norm : k_norm;
@@ -454,10 +462,18 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
 __device__ __forceinline__ float sum4(float4 v) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))); }
 template <typename T, int P>
 __global__ void __launch_bounds__(256) qk_post4_kernel(const AttnDims d, const QkPost p, const float* proj, int ldp, int k_col, const float* __restrict__ q_norm,
-                                                       const float* __restrict__ k_norm, const float2* __restrict__ rope, T* q, T* cache, const int32_t* place, const StepRows rows) {
+                                                       const float* __restrict__ k_norm, const float2* __restrict__ rope, T* q, T* cache, const int32_t* place, const StepRows rows, const RouteBeside route) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float red[2][8];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = blockIdx.y, h = blockIdx.x * 8 + warp;
+    if (route.logits && blockIdx.x == gridDim.x - 1) {
+        if (r > 0) return;
+        pdl_trigger();
+        route_few_clear(route.d, sm);
+        pdl_wait();
+        route_few_rows(route.d, route.logits, rows.n, route.t, sm);
+        return;
+    }
     const bool on = h < d.heads + d.groups, is_q = h < d.heads;
     const int g = is_q ? h : h - d.heads, half = p.rot_dims / 2, pieces = d.dim / 4;
     const float* w = is_q ? q_norm : k_norm;
@@ -533,20 +549,23 @@ __global__ void __launch_bounds__(256) qk_post4_kernel(const AttnDims d, const Q
 }  // namespace
 
 int32_t qk_post(const AttnDims& d, const QkPost& p, int dtype, const float* proj, int ldp, int k_col, const float* q_norm, const float* k_norm, const float* rope, void* q, void* cache,
-                const int32_t* place, const StepRows& rows, cudaStream_t st) {
+                const int32_t* place, const StepRows& rows, const RouteBeside* route, cudaStream_t st) {
     if (rows.n <= 0) return FORGE_OK;
+    if (route && (rows.n > kScaleRows || route->d.experts > kMaxExperts)) { set_error("routing: %d rows, %d experts", rows.n, route->d.experts); return FORGE_ERR_SHAPE; }
     if (d.dim > kQkDims * 32 || p.rot_dims > d.dim || p.rot_dims % 2) { set_error("attention: head size %d with %d rotated dimensions", d.dim, p.rot_dims); return FORGE_ERR_SHAPE; }
     auto go = [&](auto t) -> int32_t {
         using T = decltype(t);
-        const size_t smem = size_t(8) * d.dim_p * 4;
+        const RouteBeside beside = route ? *route : RouteBeside{};
+        const size_t smem = std::max(size_t(8) * d.dim_p * 4, route ? route_few_smem(route->d) : 0);
         for (int r0 = 0; r0 < rows.n; r0 += 65535) {
             StepRows part = rows;
             part.n = std::min(65535, rows.n - r0);
             part.pos += r0;
             const bool four = d.dim % 4 == 0 && ldp % 4 == 0 && k_col % 4 == 0 && p.rot_dims % (p.interleaved ? 4 : 8) == 0;
             auto kern = !four ? qk_post_kernel<T> : d.dim <= 128 ? qk_post4_kernel<T, 1> : d.dim <= 256 ? qk_post4_kernel<T, 2> : qk_post4_kernel<T, 4>;
-            FORGE_CUDA(launch_pdl(kern, dim3((d.heads + d.groups + 7) / 8, part.n), dim3(256), smem, st, d, p, proj + size_t(r0) * ldp, ldp, k_col, q_norm, k_norm,
-                                  reinterpret_cast<const float2*>(rope), static_cast<T*>(q) + size_t(r0) * d.heads * d.dim_p, static_cast<T*>(cache), place + r0, part));
+            if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+            FORGE_CUDA(launch_pdl(kern, dim3((d.heads + d.groups + 7) / 8 + (route ? 1 : 0), part.n), dim3(256), smem, st, d, p, proj + size_t(r0) * ldp, ldp, k_col, q_norm, k_norm,
+                                  reinterpret_cast<const float2*>(rope), static_cast<T*>(q) + size_t(r0) * d.heads * d.dim_p, static_cast<T*>(cache), place + r0, part, beside));
             FORGE_LAUNCH_CHECK();
         }
         return FORGE_OK;

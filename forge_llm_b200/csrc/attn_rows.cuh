@@ -4,6 +4,7 @@
 #pragma once
 
 #include "dense.cuh"
+#include "moe.cuh"
 
 namespace forge {
 
@@ -29,8 +30,10 @@ struct QkPost {
     float eps = 0.f;
 };
 // proj: f32 rows [q of all heads | ... | k of all groups from k_col | ...] of ldp floats; rope: {cos, sin} by position and pair; place: cache row of each row
+// route (may be null): a routing of the step's rows (route_few) done by one more CTA of the launch
+struct RouteBeside { RouterDims d; const float* logits = nullptr; RouteTables t; };
 int32_t qk_post(const AttnDims& d, const QkPost& p, int dtype, const float* proj, int ldp, int k_col, const float* q_norm, const float* k_norm, const float* rope, void* q, void* cache,
-                const int32_t* place, const StepRows& rows, cudaStream_t st);
+                const int32_t* place, const StepRows& rows, const RouteBeside* route, cudaStream_t st);
 
 bool attn_rows_supported(const AttnDims& d);
 // q: T rows [heads][dim_p]; out[row][head * vdim + i] = gate[row][head] * attention, T (gate null: ungated).  sink: score per head, or null.

@@ -411,10 +411,15 @@ __global__ void __launch_bounds__(kThreads<NT>, NT <= 16 ? 2 : 1) gemm_dense_ker
                 scaled_tok0 = tok0; scaled_cols = cols;
             }
             const float* pair_w = MODE == GROUPED && p.groups.weight ? p.groups.weight + at_tile.w0 : nullptr;
-            float x_old[CH];   // few tokens: the residual is on its way while the product is formed
-            if (NT <= 32 && g.kind == SEG_RESID && g.ok && !g.fresh)
+            // what dst holds is on its way while the product, or the chunk before, is finished
+            float x_old[CH];
+            const bool adds = g.kind == SEG_RESID && g.ok && !g.fresh;
+            auto fetch_old = [&](int c0) {
 #pragma unroll
-                for (int c = 0; c < CH; ++c) if (c < cols && (p.cluster <= 1 || (c >> 2) % p.cluster == rank)) x_old[c] = g.f32[size_t(tok0 + c) * g.ld];
+                for (int c = 0; c < CH; ++c)
+                    x_old[c] = adds && c < cols - c0 && (p.cluster <= 1 || (c >> 2) % p.cluster == rank) ? g.f32[size_t(tok0 + c0 + c) * g.ld] : 0.f;
+            };
+            if (g.kind == SEG_RESID) fetch_old(c_begin);
             // the four warps meet at the barriers of a shared tile: one whose wait gave up must not leave the loop alone
             if (!(MODE == LISTED && none) && !mbar_wait(&acc_full[buf], (seg_i >> 1) & 1, &s_err)) atomicExch(&s_err, 1);
             fence_after();
@@ -442,7 +447,7 @@ __global__ void __launch_bounds__(kThreads<NT>, NT <= 16 ? 2 : 1) gemm_dense_ker
                     const float got = __shfl_xor_sync(0xffffffffu, v[0], 1);
                     float x = 0.f;
                     const Leave<__nv_bfloat16> n(p.out.seg[g.seg], g, row, row0);
-                    if (g.ok) x = put_one(g, n, v[0], got, pair_w ? pair_w[c0] : 1.f, t0, NT <= 32 ? x_old[0] : 0.f, NT <= 32, !(lane & 1));
+                    if (g.ok) x = put_one(g, n, v[0], got, pair_w ? pair_w[c0] : 1.f, t0, x_old[0], true, !(lane & 1));
                     if (g.kind == SEG_RESID && n.sums) {
                         x = warp_sum(x * x);
                         if (lane == 0) n.sums[t0 * n.parts] = x;
@@ -463,7 +468,8 @@ __global__ void __launch_bounds__(kThreads<NT>, NT <= 16 ? 2 : 1) gemm_dense_ker
                     float* dst = g.f32 + t0 * g.ld;
                     float x[CH];
 #pragma unroll
-                    for (int c = 0; c < CH; ++c) x[c] = !g.ok || g.fresh ? 0.f : NT <= 32 ? x_old[c] : c < n_c ? dst[c * g.ld] : 0.f;   // all loads before the first store
+                    for (int c = 0; c < CH; ++c) x[c] = x_old[c];
+                    if (c0 + CH < c_end) fetch_old(c0 + CH);
                     if (n.keep || n.again) {
 #pragma unroll
                         for (int c = 0; c < CH; ++c) { x[c] += v[c]; if (g.ok && c < n_c) x[c] = n.enter(x[c], t0 + c); }
@@ -604,6 +610,7 @@ __global__ void __launch_bounds__(kThreads<NT>, NT <= 16 ? 2 : 1) gemm_dense_ker
                 epilogue_sync();
                 if (s_last) {
                     __threadfence();
+                    if (g.kind == SEG_RESID) fetch_old(c_begin);
 #pragma unroll 1
                     for (int c0 = c_begin; c0 < c_end && c0 < cols; c0 += CH) {
                         float v[CH];

@@ -7,71 +7,12 @@ namespace forge {
 
 namespace {
 
-constexpr int kPerLane = kMaxExperts / 32;
-
-// The warp chooses the `top` largest of z (lower numbers win ties); expert[k] and weight[k] by lane 0.
-__device__ __forceinline__ void choose(const float* z, int experts, int top, int32_t* expert, float* weight) {
-    const int lane = threadIdx.x & 31;
-    float v[kPerLane];
-    uint32_t taken = 0;
-#pragma unroll
-    for (int i = 0; i < kPerLane; ++i) v[i] = lane + 32 * i < experts ? z[lane + 32 * i] : 0.f;
-    float first = 0.f, sum = 0.f;
-    for (int k = 0; k < top; ++k) {
-        float best = 0.f;
-        int at = -1;
-#pragma unroll
-        for (int i = 0; i < kPerLane; ++i)
-            if (lane + 32 * i < experts && !(taken >> i & 1) && (at < 0 || v[i] > best)) { best = v[i]; at = lane + 32 * i; }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float other = __shfl_xor_sync(0xffffffffu, best, o);
-            const int whose = __shfl_xor_sync(0xffffffffu, at, o);
-            if (whose >= 0 && (at < 0 || other > best || (other == best && whose < at))) { best = other; at = whose; }
-        }
-        at = __shfl_sync(0xffffffffu, at, 0);      // (values that are no numbers compare differently in different lanes)
-        best = __shfl_sync(0xffffffffu, best, 0);
-        if (k == 0) first = best;
-        const float e = expf(best - first);
-        sum += e;
-        if ((at & 31) == lane) taken |= 1u << (at >> 5);
-        if (lane == 0) { expert[k] = at; weight[k] = e; }
-    }
-    if (lane == 0) for (int k = 0; k < top; ++k) weight[k] /= sum;
-    __syncwarp();
-}
-
 __global__ void __launch_bounds__(1024) route_few_kernel(const RouterDims d, const float* logits, int rows, const RouteTables t) {
-    extern __shared__ float s_w[];                                  // [experts][kScaleRows]
-    int* used = reinterpret_cast<int*>(s_w + d.experts * kScaleRows);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int i = threadIdx.x; i < d.experts * kScaleRows; i += 1024) s_w[i] = 0.f;
-    for (int i = threadIdx.x; i < d.experts; i += 1024) used[i] = 0;
-    __syncthreads();
+    extern __shared__ float s_w[];
+    route_few_clear(d, s_w);
     pdl_trigger();
     pdl_wait();
-    if (warp < rows) {
-        choose(logits + size_t(warp) * d.experts, d.experts, d.top, t.expert + warp * d.top, t.weight + warp * d.top);
-        if (lane == 0)
-            for (int k = 0; k < d.top; ++k) {
-                const int e = t.expert[warp * d.top + k];
-                s_w[e * kScaleRows + warp] = t.weight[warp * d.top + k];
-                used[e] = 1;
-            }
-    }
-    __syncthreads();
-    for (int i = threadIdx.x; i < d.experts * kScaleRows; i += 1024) t.row_weight[i] = s_w[i];
-    if (warp == 0) {
-        int n = 0;
-        for (int e0 = 0; e0 < d.experts; e0 += 32) {
-            const int e = e0 + lane;
-            const bool on = e < d.experts && used[e];
-            const uint32_t mask = __ballot_sync(0xffffffffu, on);
-            if (on) t.tiles[n + __popc(mask & ((1u << lane) - 1))] = GroupTile{e, 0, rows, e * kScaleRows};
-            n += __popc(mask);
-        }
-        if (lane == 0) *t.n_tiles = n;
-    }
+    route_few_rows(d, logits, rows, t, s_w);
 }
 
 __global__ void __launch_bounds__(256) choose_kernel(const RouterDims d, const float* __restrict__ logits, int rows, const RouteTables t) {
@@ -175,6 +116,9 @@ size_t route_bytes(const RouterDims& d, int rows) {
     const size_t pairs = size_t(rows) * d.top;
     return 5 * align16(pairs * 4) + size_t(d.experts) * kScaleRows * 4 + (pairs + d.experts) * sizeof(GroupTile) + 16;
 }
+GroupTable few_table(const RouterDims& d, int rows, const RouteTables& t) {
+    return GroupTable{t.tiles, t.n_tiles, int(std::min<long long>(d.experts, (long long)rows * d.top)), rows <= 16 ? 16 : 32, t.row_weight};
+}
 RouteTables route_tables(void* p, const RouterDims& d, int rows) {
     const size_t pairs = align16(size_t(rows) * d.top * 4);
     char* b = static_cast<char*>(p);
@@ -190,9 +134,9 @@ RouteTables route_tables(void* p, const RouterDims& d, int rows) {
 
 int32_t route_few(const RouterDims& d, const float* logits, int rows, const RouteTables& t, GroupTable* out, cudaStream_t st) {
     if (rows > kScaleRows || d.experts > kMaxExperts) { set_error("routing: %d rows, %d experts", rows, d.experts); return FORGE_ERR_SHAPE; }
-    *out = GroupTable{t.tiles, t.n_tiles, int(std::min<long long>(d.experts, (long long)rows * d.top)), rows <= 16 ? 16 : 32, t.row_weight};
-    const size_t smem = size_t(d.experts) * (kScaleRows + 1) * 4;
-    FORGE_CUDA(cudaFuncSetAttribute(route_few_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(size_t(kMaxExperts) * (kScaleRows + 1) * 4)));
+    *out = few_table(d, rows, t);
+    const size_t smem = route_few_smem(d);
+    FORGE_CUDA(cudaFuncSetAttribute(route_few_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(route_few_smem(RouterDims{kMaxExperts, 1}))));
     FORGE_CUDA(launch_pdl(route_few_kernel, dim3(1), dim3(1024), smem, st, d, logits, rows, t));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;

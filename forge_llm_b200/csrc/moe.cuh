@@ -19,6 +19,8 @@ struct RouteTables {
 size_t route_bytes(const RouterDims& d, int rows);
 RouteTables route_tables(void* p, const RouterDims& d, int rows);
 
+GroupTable few_table(const RouterDims& d, int rows, const RouteTables& t);   // of route_few
+inline size_t route_few_smem(const RouterDims& d) { return size_t(d.experts) * (kScaleRows + 1) * 4; }
 // logits: f32 [rows][experts].  The `top` largest of a row, weighted by the softmax over them.
 // Few rows (at most kScaleRows): a tile of all rows per expert that any of them uses.
 int32_t route_few(const RouterDims& d, const float* logits, int rows, const RouteTables& t, GroupTable* out, cudaStream_t st);
@@ -26,5 +28,73 @@ int32_t route_few(const RouterDims& d, const float* logits, int rows, const Rout
 int32_t route_slots(const RouterDims& d, const float* logits, int rows, const RouteTables& t, GroupTable* out, cudaStream_t st);
 // x[r] += sum over k of y[slot(r, k)], f32 rows of `width`, then `after`
 int32_t add_experts(float* x, const float* y, const RouterDims& d, const RouteTables& t, int rows, int width, const After& after, int dtype, cudaStream_t st);
+
+#ifdef __CUDACC__
+constexpr int kPerLane = kMaxExperts / 32;
+
+// The warp chooses the `top` largest of z (lower numbers win ties); expert[k] and weight[k] by lane 0.
+__device__ __forceinline__ void choose(const float* z, int experts, int top, int32_t* expert, float* weight) {
+    const int lane = threadIdx.x & 31;
+    float v[kPerLane];
+    uint32_t taken = 0;
+#pragma unroll
+    for (int i = 0; i < kPerLane; ++i) v[i] = lane + 32 * i < experts ? z[lane + 32 * i] : 0.f;
+    float first = 0.f, sum = 0.f;
+    for (int k = 0; k < top; ++k) {
+        float best = 0.f;
+        int at = -1;
+#pragma unroll
+        for (int i = 0; i < kPerLane; ++i)
+            if (lane + 32 * i < experts && !(taken >> i & 1) && (at < 0 || v[i] > best)) { best = v[i]; at = lane + 32 * i; }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float other = __shfl_xor_sync(0xffffffffu, best, o);
+            const int whose = __shfl_xor_sync(0xffffffffu, at, o);
+            if (whose >= 0 && (at < 0 || other > best || (other == best && whose < at))) { best = other; at = whose; }
+        }
+        at = __shfl_sync(0xffffffffu, at, 0);      // (values that are no numbers compare differently in different lanes)
+        best = __shfl_sync(0xffffffffu, best, 0);
+        if (k == 0) first = best;
+        const float e = expf(best - first);
+        sum += e;
+        if ((at & 31) == lane) taken |= 1u << (at >> 5);
+        if (lane == 0) { expert[k] = at; weight[k] = e; }
+    }
+    if (lane == 0) for (int k = 0; k < top; ++k) weight[k] /= sum;
+    __syncwarp();
+}
+
+// Routing of few rows by one CTA of whole warps; s_w: route_few_smem(d) bytes, cleared before.  (Also run by a kernel that stands beside it in a step.)
+__device__ __forceinline__ void route_few_clear(const RouterDims& d, float* s_w) {
+    for (int i = threadIdx.x; i < d.experts * (kScaleRows + 1); i += blockDim.x) s_w[i] = 0.f;
+    __syncthreads();
+}
+__device__ __forceinline__ void route_few_rows(const RouterDims& d, const float* logits, int rows, const RouteTables& t, float* s_w) {
+    int* used = reinterpret_cast<int*>(s_w + d.experts * kScaleRows);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int r = warp; r < rows; r += blockDim.x / 32) {
+        choose(logits + size_t(r) * d.experts, d.experts, d.top, t.expert + r * d.top, t.weight + r * d.top);
+        if (lane == 0)
+            for (int k = 0; k < d.top; ++k) {
+                const int e = t.expert[r * d.top + k];
+                s_w[e * kScaleRows + r] = t.weight[r * d.top + k];
+                used[e] = 1;
+            }
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < d.experts * kScaleRows; i += blockDim.x) t.row_weight[i] = s_w[i];
+    if (warp == 0) {
+        int n = 0;
+        for (int e0 = 0; e0 < d.experts; e0 += 32) {
+            const int e = e0 + lane;
+            const bool on = e < d.experts && used[e];
+            const uint32_t mask = __ballot_sync(0xffffffffu, on);
+            if (on) t.tiles[n + __popc(mask & ((1u << lane) - 1))] = GroupTile{e, 0, rows, e * kScaleRows};
+            n += __popc(mask);
+        }
+        if (lane == 0) *t.n_tiles = n;
+    }
+}
+#endif
 
 }  // namespace forge

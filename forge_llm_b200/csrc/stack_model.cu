@@ -691,15 +691,16 @@ struct Sequence {
         } else if (L.ff) o->add(SEG_SILU_GLU, w.glu_row, 2 * L.ff, at(S.mid.p, w.heads_k, dt), w.out.K).act_col = WP;
     }
     // x += W_o (heads in front of `out`) + feed-forward
-    int32_t two_norms_out(const LayerSpec& L, const LayerWeights& w, const After& after) {
-        if (L.router.experts) return experts(L, w, after);
+    int32_t two_norms_out(const LayerSpec& L, const LayerWeights& w, const After& after, bool routed = false) {
+        if (L.router.experts) return experts(L, w, after, routed);
         DenseOut o;
         resid(&o, x(), W, after);
         return gemm(w.out, S.mid.p, w.out.K, o);
     }
     // Few tokens: every expert that is used runs over all of them (a token that does not use it gets zeros) into its columns in front of `out`, which
     // then is one product over the heads' columns and those of the experts that are used.  Otherwise the tokens are gathered expert by expert.
-    int32_t experts(const LayerSpec& L, const LayerWeights& w, const After& after) {
+    // routed: a launch of the mixer has routed few tokens already.
+    int32_t experts(const LayerSpec& L, const LayerWeights& w, const After& after, bool routed) {
         const RouteTables t = route_tables(S.route.p, L.router, n);
         const float* logits = static_cast<const float*>(S.router.p);
         GroupTable table;
@@ -708,7 +709,8 @@ struct Sequence {
         DenseOut in;
         in.scale = scale();
         if (few_tokens(S, w, n)) {
-            FORGE_TRY(route_few(L.router, logits, n, t, &table, st));
+            if (routed) table = few_table(L.router, n, t);
+            else FORGE_TRY(route_few(L.router, logits, n, t, &table, st));
             shape.group_dst = size_t(w.ff_k);
             in.add(SEG_SILU_GLU, 0, 2 * L.ff, at(S.mid.p, w.heads_k, dt), w.out.K);
             FORGE_TRY(dense_gemm_groups(w.experts, shape, table, at(S.h.p, WP, dt), 2 * WP, n, in, m->d_err, st));
@@ -751,7 +753,9 @@ struct Sequence {
             feed_forward_rows(&o, L, w);
             FORGE_TRY(gemm(w.in, S.h.p, 2 * WP, o));
         }
-        FORGE_TRY(qk_post(a, L.soft.qk, dt, proj, ldp, w.k_row, w.q_norm, w.k_norm, S.ropes.at(L.rot).second, S.q.p, run.pool, place, s.rows, st));
+        const bool routed = L.router.experts && few_tokens(S, w, n);
+        const RouteBeside route{L.router, static_cast<const float*>(S.router.p), route_tables(S.route.p, L.router, n)};
+        FORGE_TRY(qk_post(a, L.soft.qk, dt, proj, ldp, w.k_row, w.q_norm, w.k_norm, S.ropes.at(L.rot).second, S.q.p, run.pool, place, s.rows, routed ? &route : nullptr, st));
         StepRows single = s.rows;
         single.n = s.single;
         FORGE_TRY(attn_rows(a, dt, S.q.p, run.pool, nullptr, w.sink, S.mid.p, mid_ld, single, a.most_keys(s.max_keys), st));
@@ -764,7 +768,7 @@ struct Sequence {
             p.pages = s.ctx_pages; p.page_row = a.row(); p.err = m->d_err;
             FORGE_TRY(attn_prefill_kv(PromptDims(a), p, st));
         }
-        return two_norms_out(L, w, after);
+        return two_norms_out(L, w, after, routed);
     }
 
     int32_t linear(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
