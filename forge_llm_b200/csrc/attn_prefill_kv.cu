@@ -29,6 +29,10 @@ struct Params {
     int stages;
 };
 
+__host__ __device__ __forceinline__ int first_visible(const PromptDims& d, int pos) { return d.chunk > 0 ? pos / d.chunk * d.chunk : d.window > 0 && pos >= d.window ? pos - d.window + 1 : 0; }
+// key tiles: `head` tiles of kept first tokens, then from jb, the first one that anybody's chunk or window reaches
+__host__ __device__ __forceinline__ int head_tiles(const PromptDims& d, int jb) { const int k = (d.keep + BN - 1) / BN; return d.window > 0 ? (jb < k ? jb : k) : 0; }
+
 __device__ __forceinline__ float ex2(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -51,9 +55,8 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = blockIdx.x;
     const PromptTile t = p.a.tiles[blockIdx.y];
-    auto first_key = [&](int pos) { return d.chunk > 0 ? pos / d.chunk * d.chunk : d.window > 0 && pos >= d.window ? pos - d.window + 1 : 0; };
-    // key tiles: `head` tiles of kept first tokens, then from the first one that anybody's chunk or window reaches
-    const int jb = first_key(t.pos0) / BN, head = d.window > 0 ? min(jb, (d.keep + BN - 1) / BN) : 0;
+    auto first_key = [&](int pos) { return first_visible(d, pos); };
+    const int jb = first_key(t.pos0) / BN, head = head_tiles(d, jb);
     const int nblk = head + (t.pos0 + t.rows - 1) / BN + 1 - jb;
     auto key_tile = [&](int j) { return j < head ? j : jb + j - head; };
 
@@ -258,10 +261,18 @@ int32_t attn_prefill_kv(const PromptDims& d, const PromptAttnArgs& a, cudaStream
     if (d.rot_p == 0) mr = mk;   // no rotated part: never read
     else FORGE_TRY(make_map_2d(&mr, a.krot, uint64_t(d.rot_p), uint64_t(a.ctx_rows), uint64_t(d.rot_p) * 2, BN));
     FORGE_TRY(make_map_3d(&mv, a.v, uint64_t(d.vdim_p), G, uint64_t(a.ctx_rows), uint64_t(d.vdim_p) * 2, v_row, BN));
-    // three stages, or two where that lets two CTAs share an SM
+    // three stages, or two where that lets two CTAs share an SM: if the work of an SM, not the longest tile, decides
     auto fit = [&](int stages, size_t ctas) { return ctas * (smem_bytes(d, stages) + 1024) <= 226 * 1024; };
-    const int stages = fit(3, 2) ? 3 : fit(2, 2) && d.vdim_p <= 128 ? 2 : fit(3, 1) ? 3 : 2;
-    Params p{d, a, d.scale * 1.4426950408889634f, stages};
+    long long total = 0, longest = 0;
+    for (int i = 0; i < a.n_tiles && a.host_tiles; ++i) {
+        const PromptTile& t = a.host_tiles[i];
+        const int jb = first_visible(d, t.pos0) / BN;
+        const long long n = head_tiles(d, jb) + (t.pos0 + t.rows - 1) / BN + 1 - jb;
+        total += n * d.heads;
+        longest = std::max(longest, n);
+    }
+    const bool share = longest * 148 < total && d.vdim_p <= 128;
+    Params p{d, a, d.scale * 1.4426950408889634f, fit(3, share ? 2 : 1) ? 3 : fit(2, share ? 2 : 1) ? 2 : fit(3, 1) ? 3 : 2};
     const size_t smem = smem_bytes(d, p.stages);
     auto go = [&](auto kern) -> int32_t {
         FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));

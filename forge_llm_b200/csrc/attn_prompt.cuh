@@ -27,6 +27,7 @@ struct PromptAttnArgs {
     void* out = nullptr; int out_ld = 0;
     int q_rows = 0, ctx_rows = 0;
     const PromptTile* tiles = nullptr; int n_tiles = 0;   // device
+    const PromptTile* host_tiles = nullptr;               // the same on the host, if they are at hand
     // k and v are the pool of the cache: rows of page_row values, context rows 64 i .. lie in page pages[i] (device)
     const int32_t* pages = nullptr; int page_row = 0;
     int* err = nullptr;

@@ -499,6 +499,7 @@ struct Step {
     int scale_rows = 0;                      // most rows of a product that takes scales
     SegTable segs;                           // the rows [ones, n)
     const PromptTile* tiles = nullptr; int n_tiles = 0;
+    const PromptTile* host_tiles = nullptr;
     const int32_t* ctx_pages = nullptr; int ctx_rows = 0;
     uint32_t* hist = nullptr; const int32_t* step = nullptr;
     float* trace = nullptr; size_t trace_stride = 0;
@@ -655,7 +656,7 @@ struct Sequence {
             a.q = S.q.p; a.k = S.ctx_k.p; a.krot = S.ctx_r.p; a.v = S.ctx_v.p;
             a.gate = at(S.gate.p, size_t(s.single) * gate_ld, dt); a.gate_ld = gate_ld;
             a.out = at(S.mid.p, size_t(s.single) * mid_ld, dt); a.out_ld = mid_ld;
-            a.q_rows = np; a.ctx_rows = s.ctx_rows; a.tiles = s.tiles; a.n_tiles = s.n_tiles; a.err = m->d_err;
+            a.q_rows = np; a.ctx_rows = s.ctx_rows; a.tiles = s.tiles; a.n_tiles = s.n_tiles; a.host_tiles = s.host_tiles; a.err = m->d_err;
             FORGE_TRY(attn_prefill_kv(PromptDims(d), a, st));
         }
         DenseOut o;
@@ -764,7 +765,7 @@ struct Sequence {
             p.q = at(S.q.p, size_t(s.single) * a.heads * a.dim_p, dt); p.k = run.pool; p.v = at(run.pool, size_t(a.groups) * a.dim_p, dt);
             p.sink = w.sink;
             p.out = at(S.mid.p, size_t(s.single) * mid_ld, dt); p.out_ld = mid_ld;
-            p.q_rows = n - s.single; p.ctx_rows = kv->num_pages * FORGE_KV_PAGE; p.tiles = s.tiles; p.n_tiles = s.n_tiles;
+            p.q_rows = n - s.single; p.ctx_rows = kv->num_pages * FORGE_KV_PAGE; p.tiles = s.tiles; p.n_tiles = s.n_tiles; p.host_tiles = s.host_tiles;
             p.pages = s.ctx_pages; p.page_row = a.row(); p.err = m->d_err;
             FORGE_TRY(attn_prefill_kv(PromptDims(a), p, st));
         }
@@ -878,7 +879,7 @@ struct Sequence {
             p.q = at(S.q.p, size_t(s.single) * t.heads * t.dim_p, dt); p.k = run.pool; p.v = at(run.pool, size_t(t.groups) * t.dim_p, dt);
             p.head_gate = hgate + size_t(s.single) * t.heads;
             p.out = at(S.mid.p, size_t(s.single) * mid_ld, dt); p.out_ld = mid_ld;
-            p.q_rows = np; p.ctx_rows = kv->num_pages * FORGE_KV_PAGE; p.tiles = s.tiles; p.n_tiles = s.n_tiles;
+            p.q_rows = np; p.ctx_rows = kv->num_pages * FORGE_KV_PAGE; p.tiles = s.tiles; p.n_tiles = s.n_tiles; p.host_tiles = s.host_tiles;
             p.pages = s.ctx_pages; p.page_row = t.row(); p.err = m->d_err;
             FORGE_TRY(attn_prefill_kv(PromptDims(t), p, st));
         }
@@ -1130,7 +1131,7 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
     s.ones = ones; s.single = single; s.splits = splits; s.max_keys = max_keys;
     s.segs = SegTable{reinterpret_cast<const ScanSeg*>(dm + o_segs), int(segs.size()), n_short, max_seg, chunks, ones, rows - ones};
     s.ctx_pages = dm + o_pages; s.ctx_rows = ctx_rows;
-    s.tiles = reinterpret_cast<const PromptTile*>(dm + o_tiles); s.n_tiles = int(tiles.size());
+    s.tiles = reinterpret_cast<const PromptTile*>(dm + o_tiles); s.n_tiles = int(tiles.size()); s.host_tiles = tiles.data();
     s.scale_rows = std::max(rows, wants);
     if (trace_rows) { s.trace = m->trace + size_t(trace_row0) * S.spec.width; s.trace_stride = size_t(trace_rows) * S.spec.width; }
     FORGE_TRY(Sequence(m, kv, s).run());
