@@ -224,8 +224,8 @@ struct TileBytes {   // of shared memory, in elements
 };
 size_t mma_smem(const AttnDims& d) { return (size_t(kWarps) * 2 * TileBytes(d).stage + kRowHeads * TileBytes(d).ldk) * 2 + (kWarps * kRowHeads * 2 + kRowHeads * 2) * 4; }
 
-// VC: blocks of 64 value columns
-template <int VC>
+// VC: blocks of 64 value columns at most; KP, VP: 16-byte pieces of a row's key and values (0: any number)
+template <int VC, int KP, int VP>
 __global__ void __launch_bounds__(kThreads, 1) attn_rows_mma_kernel(const AttnDims d, const bf16* q, const bf16* cache, const float* gate, const float* __restrict__ sink, bf16* out, int out_ld, const StepRows rows) {
     extern __shared__ __align__(16) unsigned char sm_raw[];
     const TileBytes L(d);
@@ -247,21 +247,22 @@ __global__ void __launch_bounds__(kThreads, 1) attn_rows_mma_kernel(const AttnDi
     const bf16* kbase = cache + size_t(g) * d.dim_p;
     const bf16* vbase = cache + size_t(d.groups) * d.dim_p + size_t(g) * d.vdim_p;
     bf16* mine = tiles + size_t(warp) * 2 * L.stage;
-    const int kp = d.dim_p / 8, vp = d.vdim_p / 8;              // 16-byte pieces of a row
+    const int kp = KP ? KP : d.dim_p / 8, vp = VP ? VP : d.vdim_p / 8;
     auto fetch = [&](int i) {   // the warp's i-th tile
         const int key0 = k_begin + (warp + kWarps * i) * kTileKeys;
         if (key0 < k_end) {
             const int idx = key0 + min(lane & (kTileKeys - 1), k_end - key0 - 1), key = idx < kept ? idx : lo + idx - kept;
             const uint32_t row = uint32_t(pt[key / FORGE_KV_PAGE]) * FORGE_KV_PAGE + key % FORGE_KV_PAGE;
             const uint32_t sk = uint32_t(__cvta_generic_to_shared(mine + (i & 1) * L.stage)), sv = sk + kTileKeys * L.ldk * 2;
-            for (int p = lane; p < kTileKeys * kp; p += 32) {
-                const int k = p / kp, c = (p % kp) * 8;
-                cp_async16(sk + (k * L.ldk + c) * 2, kbase + __shfl_sync(0xffffffffu, row, k) * W + c, true);
-            }
-            for (int p = lane; p < kTileKeys * vp; p += 32) {
-                const int k = p / vp, c = (p % vp) * 8;
-                cp_async16(sv + (k * L.ldv + c) * 2, vbase + __shfl_sync(0xffffffffu, row, k) * W + c, true);
-            }
+            auto copy = [&](uint32_t dst, int ld, const bf16* src, int pieces) {
+#pragma unroll
+                for (int p = lane; p < kTileKeys * pieces; p += 32) {
+                    const int k = p / pieces, c = (p % pieces) * 8;
+                    cp_async16(dst + (k * ld + c) * 2, src + __shfl_sync(0xffffffffu, row, k) * W + c, true);
+                }
+            };
+            copy(sk, L.ldk, kbase, kp);
+            copy(sv, L.ldv, vbase, vp);
         }
         cp_commit();
     };
@@ -370,16 +371,32 @@ bool mma_supported(const AttnDims& d) { return d.vdim_p <= 256 && mma_smem(d) <=
 int32_t run_mma(const AttnDims& d, const void* q, const void* cache, const float* gate, const float* sink, void* out, int out_ld, const StepRows& rows, int max_keys, cudaStream_t st) {
     const int gq = d.heads / d.groups, blocks = (gq + kRowHeads - 1) / kRowHeads;
     const size_t smem = mma_smem(d);
-    int splits = 1;   // at most one CTA per SM, no split shorter than one round of its warps
-    while (splits < 8 && (long long)rows.n * d.groups * blocks * splits * 2 <= 148 && max_keys > splits * kWarps * kTileKeys) splits *= 2;
     auto go = [&](auto kern) -> int32_t {
         FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+        // the most splits whose clusters all run at once, none shorter than one round of its warps
+        static int fits[9] = {0};   // one CTA per SM
+        if (!fits[1])
+            for (int c = 1; c <= 8; ++c) {
+                cudaLaunchConfig_t cfg{};
+                cudaLaunchAttribute at[1];
+                cfg.gridDim = dim3(unsigned(c * 148)); cfg.blockDim = dim3(kThreads); cfg.dynamicSmemBytes = std::max(smem, size_t(120) * 1024);
+                at[0].id = cudaLaunchAttributeClusterDimension;
+                at[0].val.clusterDim.x = unsigned(c); at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
+                cfg.attrs = at; cfg.numAttrs = 1;
+                FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(std::max(smem, size_t(120) * 1024))));
+                FORGE_CUDA(cudaOccupancyMaxActiveClusters(&fits[c], kern, &cfg));
+            }
+        int splits = 1;
+        for (int c = 2; c <= 8; ++c)
+            if ((long long)rows.n * d.groups * blocks <= fits[c] && max_keys > (c - 1) * kWarps * kTileKeys) splits = c;
         FORGE_CUDA(launch_pdl_cluster(kern, dim3(splits, d.groups * blocks, rows.n), dim3(kThreads), splits, smem, st, d, static_cast<const bf16*>(q), static_cast<const bf16*>(cache), gate, sink,
                                       static_cast<bf16*>(out), out_ld, rows));
         FORGE_LAUNCH_CHECK();
         return FORGE_OK;
     };
-    return d.vdim_p <= 64 ? go(attn_rows_mma_kernel<1>) : d.vdim_p <= 128 ? go(attn_rows_mma_kernel<2>) : go(attn_rows_mma_kernel<4>);
+    if (d.dim_p == 64 && d.vdim_p == 64) return go(attn_rows_mma_kernel<1, 8, 8>);
+    if (d.dim_p == 128 && d.vdim_p == 128) return go(attn_rows_mma_kernel<2, 16, 16>);
+    return d.vdim_p <= 64 ? go(attn_rows_mma_kernel<1, 0, 0>) : d.vdim_p <= 128 ? go(attn_rows_mma_kernel<2, 0, 0>) : go(attn_rows_mma_kernel<4, 0, 0>);
 }
 
 // ------------------------------------------------------------------------------------------------ queries and keys
