@@ -477,14 +477,14 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
 }
 __device__ __forceinline__ float sum4(float4 v) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))); }
-template <typename T, int P>
+template <typename T, int P, int R>   // R: rows per CTA, whose loads are in flight together
 __global__ void __launch_bounds__(256) qk_post4_kernel(const AttnDims d, const QkPost p, const float* proj, int ldp, int k_col, const float* __restrict__ q_norm,
                                                        const float* __restrict__ k_norm, const float2* __restrict__ rope, T* q, T* cache, const int32_t* place, const StepRows rows, const RouteBeside route) {
     extern __shared__ __align__(16) float sm[];
-    __shared__ float red[2][8];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = blockIdx.y, h = blockIdx.x * 8 + warp;
+    __shared__ float red[R][2][8];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = blockIdx.y * R, h = blockIdx.x * 8 + warp;
     if (route.logits && blockIdx.x == gridDim.x - 1) {
-        if (r > 0) return;
+        if (r0 > 0) return;
         pdl_trigger();
         route_few_clear(route.d, sm);
         pdl_wait();
@@ -496,70 +496,99 @@ __global__ void __launch_bounds__(256) qk_post4_kernel(const AttnDims d, const Q
     const float* w = is_q ? q_norm : k_norm;
     if (p.norm == QkPost::WHOLE) w += size_t(g) * d.dim;
     pdl_trigger();
-    const float2* turn = rope + size_t(rows.pos[r]) * half;
-    float4 nw[P], v[P], t0[P], t1[P];
+    float4 nw[P], v[R][P], t0[R][P], t1[R][P];
 #pragma unroll
     for (int i = 0; i < P; ++i) {
         const int c = (lane + 32 * i) * 4;
-        const bool ok = on && c < d.dim;
-        nw[i] = ok ? *reinterpret_cast<const float4*>(w + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-        t0[i] = t1[i] = make_float4(1.f, 0.f, 1.f, 0.f);
-        if (ok && c < 2 * half) {   // {cos, sin} of the piece's pairs
-            const int pair = p.interleaved ? c / 2 : c < half ? c : c - half;
-            t0[i] = *reinterpret_cast<const float4*>(turn + pair);
-            if (!p.interleaved) t1[i] = *reinterpret_cast<const float4*>(turn + pair + 2);
+        nw[i] = on && c < d.dim ? *reinterpret_cast<const float4*>(w + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int j = 0; j < R; ++j) {
+        const float2* turn = rope + size_t(rows.pos[min(r0 + j, rows.n - 1)]) * half;
+#pragma unroll
+        for (int i = 0; i < P; ++i) {
+            const int c = (lane + 32 * i) * 4;
+            t0[j][i] = t1[j][i] = make_float4(1.f, 0.f, 1.f, 0.f);
+            if (on && c < d.dim && c < 2 * half) {   // {cos, sin} of the piece's pairs
+                const int pair = p.interleaved ? c / 2 : c < half ? c : c - half;
+                t0[j][i] = *reinterpret_cast<const float4*>(turn + pair);
+                if (!p.interleaved) t1[j][i] = *reinterpret_cast<const float4*>(turn + pair + 2);
+            }
         }
     }
     pdl_wait();
-    const float* row = proj + size_t(r) * ldp;
-    const float* src = is_q ? row + size_t(g) * d.dim : row + k_col + size_t(g) * d.dim;
-    float ss = 0.f;
+    float ss[R];
+    int to[R];
 #pragma unroll
-    for (int i = 0; i < P; ++i) {
-        v[i] = on && lane + 32 * i < pieces ? reinterpret_cast<const float4*>(src)[lane + 32 * i] : make_float4(0.f, 0.f, 0.f, 0.f);
-        ss += sum4(v[i]);
+    for (int j = 0; j < R; ++j) {
+        const int r = min(r0 + j, rows.n - 1);
+        const float* row = proj + size_t(r) * ldp;
+        const float* src = is_q ? row + size_t(g) * d.dim : row + k_col + size_t(g) * d.dim;
+        to[j] = place[r];
+        ss[j] = 0.f;
+#pragma unroll
+        for (int i = 0; i < P; ++i) v[j][i] = on && lane + 32 * i < pieces ? reinterpret_cast<const float4*>(src)[lane + 32 * i] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     float n = float(d.dim);
     if (p.norm == QkPost::WHOLE) {   // this CTA sums up the rows that its heads belong to
         const int last = min(d.heads + d.groups, int(blockIdx.x) * 8 + 8) - 1;
         const int nq = int(blockIdx.x) * 8 < d.heads ? d.heads * pieces : 0, nk = last >= d.heads ? d.groups * pieces : 0;
-        float sq = 0.f, sk = 0.f;
+#pragma unroll
+        for (int j = 0; j < R; ++j) {
+            const float* row = proj + size_t(min(r0 + j, rows.n - 1)) * ldp;
+            float sq = 0.f, sk = 0.f;
 #pragma unroll 4
-        for (int i = threadIdx.x; i < nq; i += 256) sq += sum4(reinterpret_cast<const float4*>(row)[i]);
+            for (int i = threadIdx.x; i < nq; i += 256) sq += sum4(reinterpret_cast<const float4*>(row)[i]);
 #pragma unroll 2
-        for (int i = threadIdx.x; i < nk; i += 256) sk += sum4(reinterpret_cast<const float4*>(row + k_col)[i]);
-        sq = warp_sum(sq); sk = warp_sum(sk);
-        if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+            for (int i = threadIdx.x; i < nk; i += 256) sk += sum4(reinterpret_cast<const float4*>(row + k_col)[i]);
+            sq = warp_sum(sq); sk = warp_sum(sk);
+            if (lane == 0) { red[j][0][warp] = sq; red[j][1][warp] = sk; }
+        }
         __syncthreads();
-        ss = 0.f;
-        for (int i = 0; i < 8; ++i) ss += red[is_q ? 0 : 1][i];
+#pragma unroll
+        for (int j = 0; j < R; ++j)
+            for (int i = 0; i < 8; ++i) ss[j] += red[j][is_q ? 0 : 1][i];
         n = float(is_q ? d.heads : d.groups) * d.dim;
-    } else ss = warp_sum(ss);
-    const float inv = 1.0f / sqrtf(ss / n + p.eps);
+    } else {
+#pragma unroll
+        for (int j = 0; j < R; ++j) {
+#pragma unroll
+            for (int i = 0; i < P; ++i) ss[j] += sum4(v[j][i]);
+            ss[j] = warp_sum(ss[j]);
+        }
+    }
     float* s = sm + warp * d.dim_p;
 #pragma unroll
-    for (int i = 0; i < P; ++i) {
-        v[i] = make_float4(v[i].x * inv * nw[i].x, v[i].y * inv * nw[i].y, v[i].z * inv * nw[i].z, v[i].w * inv * nw[i].w);
-        if (!p.interleaved && (lane + 32 * i) * 4 < 2 * half) store4(s + (lane + 32 * i) * 4, v[i]);
-    }
-    __syncwarp();
-    if (!on) return;
-    T* dst = is_q ? q + (size_t(r) * d.heads + g) * d.dim_p : cache + size_t(place[r]) * d.row() + size_t(g) * d.dim_p;
+    for (int j = 0; j < R; ++j) {
+        const int r = r0 + j;
+        const float inv = 1.0f / sqrtf(ss[j] / n + p.eps);
+        __syncwarp();
 #pragma unroll
-    for (int i = 0; i < P; ++i) {
-        const int c = (lane + 32 * i) * 4;
-        if (c >= d.dim) continue;
-        float4 x = v[i];
-        if (c < 2 * half) {
-            if (p.interleaved) {
-                x = make_float4(fmaf(v[i].x, t0[i].x, -v[i].y * t0[i].y), fmaf(v[i].y, t0[i].x, v[i].x * t0[i].y), fmaf(v[i].z, t0[i].z, -v[i].w * t0[i].w), fmaf(v[i].w, t0[i].z, v[i].z * t0[i].w));
-            } else {
-                const float4 y = *reinterpret_cast<const float4*>(s + (c < half ? c + half : c - half));
-                const float sign = c < half ? -1.f : 1.f;
-                x = make_float4(fmaf(x.x, t0[i].x, sign * y.x * t0[i].y), fmaf(x.y, t0[i].z, sign * y.y * t0[i].w), fmaf(x.z, t1[i].x, sign * y.z * t1[i].y), fmaf(x.w, t1[i].z, sign * y.w * t1[i].w));
-            }
+        for (int i = 0; i < P; ++i) {
+            float4& x = v[j][i];
+            x = make_float4(x.x * inv * nw[i].x, x.y * inv * nw[i].y, x.z * inv * nw[i].z, x.w * inv * nw[i].w);
+            if (!p.interleaved && (lane + 32 * i) * 4 < 2 * half) store4(s + (lane + 32 * i) * 4, x);
         }
-        store4(dst + c, x);
+        __syncwarp();
+        if (!on || r >= rows.n) continue;
+        T* dst = is_q ? q + (size_t(r) * d.heads + g) * d.dim_p : cache + size_t(to[j]) * d.row() + size_t(g) * d.dim_p;
+#pragma unroll
+        for (int i = 0; i < P; ++i) {
+            const int c = (lane + 32 * i) * 4;
+            if (c >= d.dim) continue;
+            float4 x = v[j][i];
+            const float4 a = t0[j][i], b = t1[j][i];
+            if (c < 2 * half) {
+                if (p.interleaved) {
+                    x = make_float4(fmaf(x.x, a.x, -x.y * a.y), fmaf(x.y, a.x, x.x * a.y), fmaf(x.z, a.z, -x.w * a.w), fmaf(x.w, a.z, x.z * a.w));
+                } else {
+                    const float4 y = *reinterpret_cast<const float4*>(s + (c < half ? c + half : c - half));
+                    const float sign = c < half ? -1.f : 1.f;
+                    x = make_float4(fmaf(x.x, a.x, sign * y.x * a.y), fmaf(x.y, a.z, sign * y.y * a.w), fmaf(x.z, b.x, sign * y.z * b.y), fmaf(x.w, b.z, sign * y.w * b.w));
+                }
+            }
+            store4(dst + c, x);
+        }
     }
 }
 
@@ -573,15 +602,16 @@ int32_t qk_post(const AttnDims& d, const QkPost& p, int dtype, const float* proj
     auto go = [&](auto t) -> int32_t {
         using T = decltype(t);
         const RouteBeside beside = route ? *route : RouteBeside{};
-        const size_t smem = std::max(size_t(8) * d.dim_p * 4, route ? route_few_smem(route->d) : 0);
         for (int r0 = 0; r0 < rows.n; r0 += 65535) {
             StepRows part = rows;
             part.n = std::min(65535, rows.n - r0);
             part.pos += r0;
             const bool four = d.dim % 4 == 0 && ldp % 4 == 0 && k_col % 4 == 0 && p.rot_dims % (p.interleaved ? 4 : 8) == 0;
-            auto kern = !four ? qk_post_kernel<T> : d.dim <= 128 ? qk_post4_kernel<T, 1> : d.dim <= 256 ? qk_post4_kernel<T, 2> : qk_post4_kernel<T, 4>;
+            const int per = four && d.dim <= 128 && part.n >= 512 && p.norm == QkPost::PER_HEAD ? 4 : 1;
+            auto kern = !four ? qk_post_kernel<T> : per == 4 ? qk_post4_kernel<T, 1, 4> : d.dim <= 128 ? qk_post4_kernel<T, 1, 1> : d.dim <= 256 ? qk_post4_kernel<T, 2, 1> : qk_post4_kernel<T, 4, 1>;
+            const size_t smem = std::max(size_t(8) * d.dim_p * 4, route ? route_few_smem(route->d) : 0);
             if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
-            FORGE_CUDA(launch_pdl(kern, dim3((d.heads + d.groups + 7) / 8 + (route ? 1 : 0), part.n), dim3(256), smem, st, d, p, proj + size_t(r0) * ldp, ldp, k_col, q_norm, k_norm,
+            FORGE_CUDA(launch_pdl(kern, dim3((d.heads + d.groups + 7) / 8 + (route ? 1 : 0), (part.n + per - 1) / per), dim3(256), smem, st, d, p, proj + size_t(r0) * ldp, ldp, k_col, q_norm, k_norm,
                                   reinterpret_cast<const float2*>(rope), static_cast<T*>(q) + size_t(r0) * d.heads * d.dim_p, static_cast<T*>(cache), place + r0, part, beside));
             FORGE_LAUNCH_CHECK();
         }

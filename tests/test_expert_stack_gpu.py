@@ -112,6 +112,7 @@ ATTENTION = {
     "row": ("attention_2", LS.row_normed_mixer()),
     "row_wide": ("attention_2", LS.row_normed_mixer(6, 2, 128, 160, LS.rotation_of(96, 1e6, factor=5.0))),
     "row_odd": ("attention_2", LS.row_normed_mixer(3, 1, 7, 11, LS.rotation_of(2, 9.0), 0.7)),
+    "row_blocks": ("attention_2", LS.row_normed_mixer(40, 2, 64, 64, LS.rotation_of(64, 200.0, factor=1.5))),     # more heads on a key head than one tile holds
     "row_many": ("attention_2", LS.row_normed_mixer(21, 7, 16, 24, LS.rotation_of(16, 200.0, factor=1.5))),
 }
 
@@ -349,6 +350,17 @@ def test_prompt_decode_and_portions(opened, dtype, name):
         at += n
     assert at == 170 and U.err(got, want) < tol(dtype)
     kv.close()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_a_long_prompt_in_one_step(root, dtype):
+    """More rows than the passes in front of the attention take one by one, an uneven number of them."""
+    cfg = LS.make_mokatar(104, 90, [("attention", LS.head_normed_mixer(), 40), ("attention_2", LS.row_normed_mixer(6, 2, 40, 24, LS.rotation_of(24, 500.0)), (5, 2, 24))])
+    m, orc = open_custom(root, cfg, LS.random_tensors(cfg, 6), dtype, "long")
+    toks = U.tokens(cfg, 1031, 8)
+    kv = m.new_cache(max_seq=1088)
+    assert U.err(all_logits(m, toks, kv), orc.logits(toks)) < tol(dtype)
+    kv.close(); m.close()
 
 
 def test_a_router_that_reads_the_whole_stream(root):
