@@ -7,6 +7,9 @@ decay per head or per key channel) and a pair of chunked attention and time mixi
 Mokatar: mixer and feed-forward side by side, each behind its own RMS norm of the same stream; mixers are softmax attentions with
 normed and rotated queries and keys (a window with kept first tokens and a learned sink per head, or the whole past and a sink of
 score zero) and gated linear attention; feed-forwards may be mixtures of experts; bigram embeddings; some layers run several times.
+Tarulix: norms on the outputs of the sublayers only; mixers are windowed attention with learned distance biases, sinks and values
+blended with an earlier layer's, and a pair of attention over a window and pooled blocks, whose heads' weights are mixed, beside a
+selective scan; feed-forwards are mixtures of experts, some of which pass their input on, beside a shared expert.
 
 TEST INFRASTRUCTURE ONLY, like the rest of this folder; it shares no code with the shipped package.  Everything is computed in
 ``dtype`` (float64 by default).  A sequence is evaluated as a whole: there is no cache, no page and no batch here.
@@ -347,6 +350,156 @@ def mixture_ff(h, w, m):
     return out
 
 
+# ------------------------------------------------------- distance biases, pooled blocks, mixed heads, selective scan, shared experts
+def unit_rms(x, eps):
+    """x divided by its root mean square over the last axis."""
+    return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps)
+
+
+def distance_bucket(n, buckets, longest):
+    """Bucket of the distance n: one each for the first half, then logarithmic ones up to the distance ``longest``."""
+    half = buckets // 2
+    if n < half:
+        return n
+    x = math.log(n / half) / math.log(longest / half) * (buckets - half)
+    if abs(x - round(x)) < 1e-9:       # an edge: exactly there, whatever the logarithms round to
+        x = round(x)
+    return min(buckets - 1, half + math.floor(x))
+
+
+def windowed(i, size=None):
+    """Positions 0 .. i: which of them position i sees."""
+    j = np.arange(i + 1)
+    return np.ones(i + 1, bool) if size is None else i - j < size
+
+
+def blocks_seen(i, size, pool):
+    """How many blocks of ``pool`` positions lie wholly in front of position i's window."""
+    return sum(1 for b in range(i // pool + 1) if b * pool + pool - 1 <= i - size) if size and pool else 0
+
+
+def head_scores(q, k, group):
+    """[heads, queries, keys]: query head h meets key head h / group."""
+    return np.stack([q[:, h] @ k[:, h // group].T for h in range(q.shape[1])])
+
+
+def soft_weights(row, sink=None):
+    """Softmax of a row of scores; a sink is one more score whose weight is left out."""
+    top = row.max() if sink is None else max(row.max(), sink)
+    e = np.exp(row - top)
+    return e / (e.sum() + (0.0 if sink is None else np.exp(sink - top)))
+
+
+def biased_attention(q, k, v, scale, rel, longest, sink, size):
+    """A window, a learned bias per distance bucket and head, a sink per head."""
+    n, H, _ = q.shape
+    group = H // k.shape[1]
+    s = head_scores(q, k, group) * scale
+    bucket = np.array([distance_bucket(d, len(rel), longest) for d in range(n)])
+    out = np.zeros((n, H, v.shape[2]), q.dtype)
+    for h in range(H):
+        for i in range(n):
+            j = np.flatnonzero(windowed(i, size))
+            out[i, h] = soft_weights(s[h, i, j] + rel[bucket[i - j], h], sink[h]) @ v[j, h // group]
+    return out
+
+
+def pooled_attention(q, k, v, scale, softcap, size, pool, talk):
+    """A window of tokens and the blocks in front of it, each as the mean of its keys and values, under one softmax with capped scores; the
+    heads' weights are mixed before they meet the values of each head's own key / value head."""
+    n, H, _ = q.shape
+    group = H // k.shape[1]
+    nb = n // pool if pool else 0
+    mean = lambda x: x[:nb * pool].reshape((nb, pool) + x.shape[1:]).mean(1) if nb else x[:0]
+    kk, vv = np.concatenate([mean(k), k]), np.concatenate([mean(v), v])      # blocks, then tokens
+    s = head_scores(q, kk, group) * scale
+    if softcap:
+        s = softcap * np.tanh(s / softcap)
+    out = np.zeros((n, H, v.shape[2]), q.dtype)
+    for i in range(n):
+        j = np.concatenate([np.arange(blocks_seen(i, size, pool)), nb + np.flatnonzero(windowed(i, size))])
+        w = talk @ np.stack([soft_weights(s[h, i, j]) for h in range(H)])
+        for h in range(H):
+            out[i, h] = w[h] @ vv[j, h // group]
+    return out
+
+
+def biased_qkv(h, w, m):
+    n = h.shape[0]
+    shape = {"q": (n, m["heads"], m["dim"]), "k": (n, m["kv_heads"], m["dim"]), "v": (n, m["kv_heads"], m["vdim"])}
+    return [(h @ w(x).T + w(x + ".b")).reshape(shape[x]) for x in "qkv"]
+
+
+def blended_values(v, first, lam):
+    return (1 - lam) * v + lam * first
+
+
+def distance_attention(h, w, m, eps, first=None):
+    """(output, values in front of blending).  first: an earlier layer's values, blended in."""
+    q, k, own = biased_qkv(h, w, m)
+    q, k = unit_rms(q, eps), unit_rms(k, eps)
+    v = own if first is None else blended_values(own, first, w("vmix"))
+    o = biased_attention(q, k, v, m["scale"], w("rel"), m["bias_max"], w("sink"), (m.get("mask") or {}).get("size"))
+    return o.reshape(len(h), -1) @ w("o").T + w("o.b"), own
+
+
+def talking_attention(h, w, m, eps):
+    q, k, v = biased_qkv(h, w, m)
+    rot = m["rot"]
+    q, k = (unit_rms(rotate_half(x, np.arange(len(h)), rot["base"], rot["dims"]), eps) for x in (q, k))
+    mask = m.get("mask") or {}
+    o = pooled_attention(q, k, v, m["scale"], m.get("softcap"), mask.get("size"), mask.get("pool"), w("talk"))
+    return o.reshape(len(h), -1) @ w("o").T + w("o.b")
+
+
+def selective_inputs(h, w, m):
+    """(x behind the convolution, step sizes, B, C, z)"""
+    n = m["inner"]
+    xz = h @ w("in").T
+    x = silu(short_convolution(xz[:, :n], w("conv")) + w("conv.b"))
+    p = x @ w("x").T
+    r, s = m["dt_rank"], m["state"]
+    return x, softplus(p[:, :r] @ w("dt").T + w("dt.b")), p[:, r:r + s], p[:, r + s:], xz[:, n:]
+
+
+def selective_scan(x, dt, A, B, C, D):
+    """(y [tokens, channels], last state [channels, states])"""
+    S, y = np.zeros(A.shape, x.dtype), np.zeros_like(x)
+    for t in range(len(x)):
+        S = np.exp(dt[t][:, None] * A) * S + (dt[t] * x[t])[:, None] * B[t]
+        y[t] = S @ C[t] + D * x[t]
+    return y, S
+
+
+def selective_mixer(h, w, m):
+    x, dt, B, C, z = selective_inputs(h, w, m)
+    y, _ = selective_scan(x, dt, -np.exp(w("A_log")), B, C, w("D"))
+    return (y * silu(z)) @ w("o").T
+
+
+def attention_beside_scan(h, w, m, eps):
+    return m["left_scale"] * talking_attention(h, lambda n: w("left." + n), m["left"], eps) + m["right_scale"] * selective_mixer(h, lambda n: w("right." + n), m["right"])
+
+
+def route_corrected(z, correction, top):
+    """The ``top`` largest of softmax(z) + correction, and their softmax values as they are."""
+    e = np.exp(z - z.max(1, keepdims=True))
+    s = e / e.sum(1, keepdims=True)
+    chosen = np.argsort(-(s + correction), axis=1, kind="stable")[:, :top]
+    return chosen, np.take_along_axis(s, chosen, 1)
+
+
+def shared_mixture_ff(h, w, m):
+    """Experts, the last ``identity`` choices passing their input on, beside a shared expert."""
+    r = m["router"]
+    chosen, weight = route_corrected(h @ w("router").T, w("correction"), r["top"])
+    out = silu_glu_ff(h, lambda n: w("shared." + n))
+    for t in range(h.shape[0]):
+        for e, g in zip(chosen[t], weight[t]):
+            out[t] += g * (h[t] if e >= r["experts"] else silu_glu_ff(h[t:t + 1], lambda n: w(f"e{e}.{n}"))[0])
+    return out
+
+
 def bigram_rows(tokens, b):
     """Row of the bigram table for every token; the last row for the first token."""
     return [b["buckets"] if i == 0 else (int(tokens[i - 1]) * b["mul_prev"] + int(t) * b["mul_cur"]) % b["buckets"] for i, t in enumerate(tokens)]
@@ -379,8 +532,11 @@ class LayerStack:
         self.t = {k: np.asarray(v, dtype) for k, v in tensors.items()}
         self.dtype = dtype
         self.side_by_side = config["architecture"] == "Mokatar"
+        self.post_norm = config["architecture"] == "Tarulix"
 
     def norm(self, x, name):
+        if self.post_norm:
+            return unit_rms(x, self.cfg["norm"]["eps"]) * self.t[name]
         if self.side_by_side:
             return rms_norm(x, 1.0 + self.t[name], self.cfg["norm"]["eps"])
         return dynamic_tanh(x, self.t[name + ".alpha"], self.t[name], self.t[name + ".b"])
@@ -389,6 +545,16 @@ class LayerStack:
         L = self.cfg["layers"][i]
         p = f"l{L.get('weights_of', i)}."
         mix, mlp = (lambda n: self.t[p + "mix." + n]), (lambda n: self.t[p + "mlp." + n])
+        if self.post_norm:
+            m, eps = L["mixer"], self.cfg["norm"]["eps"]
+            if L["type"] == "parallel":
+                y = attention_beside_scan(x, mix, m, eps)
+            else:
+                y, own = distance_attention(x, mix, m, eps, self.first_values if m.get("v_mix") else None)
+                if m.get("v_mix") and self.first_values is None:
+                    self.first_values = own
+            x = x + self.norm(y, p + "norm1")
+            return x + self.norm(shared_mixture_ff(x, mlp, L["mlp"]), p + "norm2") if L.get("mlp") else x
         h = self.norm(x, p + "norm1")
         y = mixer_of(L["type"], h, mix, L["mixer"], self.cfg["norm"]["eps"])
         if self.side_by_side:
@@ -409,6 +575,7 @@ class LayerStack:
         if self.side_by_side:
             x = x * self.dtype(self.cfg["embedding"]["scale"]) + self.t["bigram"][bigram_rows(tokens, self.cfg["embedding"]["bigram"])]
         x0 = x
+        self.first_values = None
         out = []
         for i, start in layer_runs(self.cfg):
             if start is not None and self.side_by_side:
