@@ -17,7 +17,7 @@ LIB = os.path.join(HERE, "libforge_b200.so")
 STAMP = LIB + ".sha256"
 SOURCES = ["pack.cu", "gemv_tc.cu", "gemv_batch.cu", "elementwise.cu", "attn_decode.cu", "attn_prefill_tc5.cu", "gemm_mma.cu", "gemm_tc5.cu",
            "tp_comm.cu", "gguf_reader.cu", "kquant_host.cu", "sampler.cu", "api_ops.cu", "model.cu",
-           "checkpoint.cu", "gemm_dense.cu", "mla.cu", "mla_decode.cu", "attn_prefill_kv.cu", "attn_rows.cu", "moe.cu", "recurrent.cu", "recurrent_chunk.cu", "stack_config.cu", "stack_model.cu"]
+           "checkpoint.cu", "gemm_dense.cu", "mla.cu", "mla_decode.cu", "attn_prefill_kv.cu", "attn_rows.cu", "moe.cu", "attn_pool.cu", "attn_talk.cu", "selective.cu", "recurrent.cu", "recurrent_chunk.cu", "stack_config.cu", "stack_model.cu"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC,-fopenmp,-O3", "-Xptxas", "-v"]
 

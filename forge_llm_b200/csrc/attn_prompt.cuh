@@ -11,13 +11,15 @@ struct PromptDims {
     int dim = 0, rot = 0, vdim = 0;           // query / key part of the head, part whose keys all heads share, values
     int dim_p = 0, rot_p = 0, vdim_p = 0;     // padded to 64
     float scale = 1.f, softcap = 0.f;
-    int chunk = 0, window = 0, keep = 0;      // as in AttnDims
+    int chunk = 0, window = 0, keep = 0, pool = 0, bias_n = 0;   // as in AttnDims
+    bool joint = false;                       // every head meets the values of all groups: out [row][head][group][vdim_p]
     PromptDims() = default;
     explicit PromptDims(const LatentDims& d) : heads(d.heads), dim(d.dim), rot(d.rot), vdim(d.vdim), dim_p(d.dim_p), rot_p(d.rot_p), vdim_p(d.vdim_p), scale(d.scale) {}
     explicit PromptDims(const AttnDims& d)
-        : heads(d.heads), share(d.heads / d.groups), dim(d.dim), vdim(d.vdim), dim_p(d.dim_p), vdim_p(d.vdim_p), scale(d.scale), softcap(d.softcap), chunk(d.chunk), window(d.window), keep(d.keep) {}
+        : heads(d.heads), share(d.heads / d.groups), dim(d.dim), vdim(d.vdim), dim_p(d.dim_p), vdim_p(d.vdim_p), scale(d.scale), softcap(d.softcap), chunk(d.chunk), window(d.window), keep(d.keep), pool(d.pool), bias_n(d.bias_n) {}
 };
-struct PromptTile { int32_t row0, rows, pos0, ctx0; };   // query rows of the step, position of the first, first context row of its sequence
+// query rows of the step, position of the first, first context row of its sequence, first row of its blocks
+struct PromptTile { int32_t row0, rows, pos0, ctx0, pool0, unused[3]; };
 struct PromptAttnArgs {
     // [q_rows][heads][dim_p + rot_p], [ctx][heads / share][dim_p], [ctx][rot_p], [ctx][heads / share][vdim_p]
     const void* q = nullptr; const void* k = nullptr; const void* krot = nullptr; const void* v = nullptr;
@@ -30,6 +32,8 @@ struct PromptAttnArgs {
     const PromptTile* host_tiles = nullptr;               // the same on the host, if they are at hand
     // k and v are the pool of the cache: rows of page_row values, context rows 64 i .. lie in page pages[i] (device)
     const int32_t* pages = nullptr; int page_row = 0;
+    const float* bias = nullptr;                      // [heads][bias_n]
+    const void* blocks = nullptr; int block_rows = 0; // rows like the cache's
     int* err = nullptr;
 };
 bool attn_prefill_kv_supported(const PromptDims& d);

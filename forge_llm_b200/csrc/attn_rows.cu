@@ -79,7 +79,7 @@ __device__ __forceinline__ void merge_rows(const AttnDims& d, float* so, int str
 // GQ: query heads per CTA; VP: pairs of value columns per lane
 template <typename T, int GQ, int VP>
 __global__ void __launch_bounds__(kThreads) attn_rows_kernel(const AttnDims d, const T* q, const T* cache, const float* gate, const float* __restrict__ sink,
-                                                             T* __restrict__ out, int out_ld, const StepRows rows) {
+                                                             const float* __restrict__ bias, T* __restrict__ out, int out_ld, const StepRows rows) {
     extern __shared__ float sm[];
     const int gq = d.heads / d.groups, blocks = (gq + GQ - 1) / GQ;
     const int split = blockIdx.x, splits = gridDim.x, g = blockIdx.y / blocks, h0 = g * gq + (blockIdx.y % blocks) * GQ, nh = min(GQ, (g + 1) * gq - h0), r = blockIdx.z;
@@ -92,8 +92,7 @@ __global__ void __launch_bounds__(kThreads) attn_rows_kernel(const AttnDims d, c
     pdl_trigger();
     // positions and page tables are written in front of the step's first kernel, which is launched without overlap
     const int pos = rows.pos[r], seq = rows.seq ? rows.seq[r] : r;
-    // the visible keys are numbered: the kept first ones, then those from lo
-    const int lo = d.first_key(pos), kept = d.kept(pos), n = kept + pos - lo + 1;
+    const int lo = d.first_key(pos), front = d.front(pos), n = front + pos - lo + 1;
     const int per = ((n + splits - 1) / splits + 31) & ~31;
     const int k_begin = split * per, k_end = min(n, k_begin + per);
     const int32_t* pt = rows.page_table + size_t(seq) * rows.pages_per_seq;
@@ -114,7 +113,7 @@ __global__ void __launch_bounds__(kThreads) attn_rows_kernel(const AttnDims d, c
     const float inv_cap = d.softcap > 0.f ? 1.0f / d.softcap : 0.f;
     const T* kbase = cache + size_t(g) * d.dim_p;
     const T* vbase = cache + size_t(d.groups) * d.dim_p + size_t(g) * d.vdim_p;
-    auto row_of = [&](int i) { const int key = i < kept ? i : lo + i - kept; return size_t(pt[key / FORGE_KV_PAGE]) * FORGE_KV_PAGE + key % FORGE_KV_PAGE; };
+    auto row_of = [&](int i) { return d.key_row(pt, i, front, lo); };
     for (int key0 = k_begin + warp * 32; key0 < k_end; key0 += kThreads) {
         const int nk = min(32, k_end - key0);
         const size_t my_row = row_of(key0 + min(lane, nk - 1));
@@ -145,6 +144,10 @@ __global__ void __launch_bounds__(kThreads) attn_rows_kernel(const AttnDims d, c
                 s[h] += __shfl_xor_sync(0xffffffffu, s[h], 2);
                 float v = s[h] * d.scale;
                 if (d.softcap > 0.f) v = d.softcap * tanhf(v * inv_cap);
+                if (bias && h < nh) {
+                    const int i = min(key0 + key, n - 1), dist = pos - (i < front ? i : lo + i - front);
+                    v += bias[size_t(h0 + h) * d.bias_n + min(dist, d.bias_n - 1)];
+                }
                 if ((lane & 3) == 0) sp[h * 32 + key] = key < nk ? v * kLog2e : -INFINITY;
             }
         }
@@ -191,24 +194,24 @@ __global__ void __launch_bounds__(kThreads) attn_rows_kernel(const AttnDims d, c
 size_t smem_bytes(const AttnDims& d, int gq) { return sizeof(float) * (size_t(gq) * d.dim_p + kWarps * gq * 32 + size_t(kWarps) * gq * d.vdim_p + kWarps * gq * 2 + gq * 2); }
 
 template <typename T, int GQ, int VP>
-int32_t launch(const AttnDims& d, const void* q, const void* cache, const float* gate, const float* sink, void* out, int out_ld, const StepRows& rows, int splits, cudaStream_t st) {
+int32_t launch(const AttnDims& d, const void* q, const void* cache, const float* gate, const float* sink, const float* bias, void* out, int out_ld, const StepRows& rows, int splits, cudaStream_t st) {
     auto kern = attn_rows_kernel<T, GQ, VP>;
     const size_t smem = smem_bytes(d, GQ);
     if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
     const int gq = d.heads / d.groups, blocks = (gq + GQ - 1) / GQ;
-    FORGE_CUDA(launch_pdl_cluster(kern, dim3(splits, d.groups * blocks, rows.n), dim3(kThreads), splits, smem, st, d, static_cast<const T*>(q), static_cast<const T*>(cache), gate, sink, static_cast<T*>(out), out_ld, rows));
+    FORGE_CUDA(launch_pdl_cluster(kern, dim3(splits, d.groups * blocks, rows.n), dim3(kThreads), splits, smem, st, d, static_cast<const T*>(q), static_cast<const T*>(cache), gate, sink, bias, static_cast<T*>(out), out_ld, rows));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
 
 template <typename T>
-int32_t run(const AttnDims& d, const void* q, const void* cache, const float* gate, const float* sink, void* out, int out_ld, const StepRows& rows, int splits, cudaStream_t st) {
+int32_t run(const AttnDims& d, const void* q, const void* cache, const float* gate, const float* sink, const float* bias, void* out, int out_ld, const StepRows& rows, int splits, cudaStream_t st) {
     const int gq = d.heads / d.groups, vp = d.vdim_p / 64;
     auto with_vp = [&](auto gqc) -> int32_t {
         constexpr int GQ = decltype(gqc)::value;
-        if (vp <= 1) return launch<T, GQ, 1>(d, q, cache, gate, sink, out, out_ld, rows, splits, st);
-        if (vp <= 2) return launch<T, GQ, 2>(d, q, cache, gate, sink, out, out_ld, rows, splits, st);
-        return launch<T, GQ, 8>(d, q, cache, gate, sink, out, out_ld, rows, splits, st);
+        if (vp <= 1) return launch<T, GQ, 1>(d, q, cache, gate, sink, bias, out, out_ld, rows, splits, st);
+        if (vp <= 2) return launch<T, GQ, 2>(d, q, cache, gate, sink, bias, out, out_ld, rows, splits, st);
+        return launch<T, GQ, 8>(d, q, cache, gate, sink, bias, out, out_ld, rows, splits, st);
     };
     if (gq == 1) return with_vp(std::integral_constant<int, 1>{});
     if (gq == 2) return with_vp(std::integral_constant<int, 2>{});
@@ -226,7 +229,8 @@ size_t mma_smem(const AttnDims& d) { return (size_t(kWarps) * 2 * TileBytes(d).s
 
 // VC: blocks of 64 value columns at most; KP, VP: 16-byte pieces of a row's key and values (0: any number)
 template <int VC, int KP, int VP>
-__global__ void __launch_bounds__(kThreads, 1) attn_rows_mma_kernel(const AttnDims d, const bf16* q, const bf16* cache, const float* gate, const float* __restrict__ sink, bf16* out, int out_ld, const StepRows rows) {
+__global__ void __launch_bounds__(kThreads, 1) attn_rows_mma_kernel(const AttnDims d, const bf16* q, const bf16* cache, const float* gate, const float* __restrict__ sink, const float* __restrict__ bias,
+                                                                    bf16* out, int out_ld, const StepRows rows) {
     extern __shared__ __align__(16) unsigned char sm_raw[];
     const TileBytes L(d);
     bf16* tiles = reinterpret_cast<bf16*>(sm_raw);              // [warp][2]: keys, values
@@ -239,7 +243,7 @@ __global__ void __launch_bounds__(kThreads, 1) attn_rows_mma_kernel(const AttnDi
     pdl_trigger();
     // positions and page tables are written in front of the step's first kernel, which is launched without overlap
     const int pos = rows.pos[r], seq = rows.seq ? rows.seq[r] : r;
-    const int lo = d.first_key(pos), kept = d.kept(pos), n = kept + pos - lo + 1;   // the visible keys are numbered: the kept first ones, then those from lo
+    const int lo = d.first_key(pos), front = d.front(pos), n = front + pos - lo + 1;
     const int per = ((n + splits - 1) / splits + kTileKeys - 1) & ~(kTileKeys - 1);
     const int k_begin = split * per, k_end = min(n, k_begin + per);
     const int32_t* pt = rows.page_table + size_t(seq) * rows.pages_per_seq;
@@ -251,8 +255,7 @@ __global__ void __launch_bounds__(kThreads, 1) attn_rows_mma_kernel(const AttnDi
     auto fetch = [&](int i) {   // the warp's i-th tile
         const int key0 = k_begin + (warp + kWarps * i) * kTileKeys;
         if (key0 < k_end) {
-            const int idx = key0 + min(lane & (kTileKeys - 1), k_end - key0 - 1), key = idx < kept ? idx : lo + idx - kept;
-            const uint32_t row = uint32_t(pt[key / FORGE_KV_PAGE]) * FORGE_KV_PAGE + key % FORGE_KV_PAGE;
+            const uint32_t row = uint32_t(d.key_row(pt, key0 + min(lane & (kTileKeys - 1), k_end - key0 - 1), front, lo));
             const uint32_t sk = uint32_t(__cvta_generic_to_shared(mine + (i & 1) * L.stage)), sv = sk + kTileKeys * L.ldk * 2;
             auto copy = [&](uint32_t dst, int ld, const bf16* src, int pieces) {
 #pragma unroll
@@ -266,8 +269,9 @@ __global__ void __launch_bounds__(kThreads, 1) attn_rows_mma_kernel(const AttnDi
         }
         cp_commit();
     };
-    // a tile all of whose keys earlier steps have written
-    auto old = [&](int i) { return min(k_end, k_begin + (warp + kWarps * i + 1) * kTileKeys) <= n - rows.fresh; };
+    // a tile all of whose keys earlier steps have written (a block that this step completes is seen by rows a window behind it)
+    const int written = d.pool > 0 && rows.fresh > d.window ? 0 : n - rows.fresh;
+    auto old = [&](int i) { return min(k_end, k_begin + (warp + kWarps * i + 1) * kTileKeys) <= written; };
     int ahead = 0;
     while (ahead < 2 && old(ahead)) fetch(ahead++);
     pdl_wait();
@@ -290,6 +294,15 @@ __global__ void __launch_bounds__(kThreads, 1) attn_rows_mma_kernel(const AttnDi
     for (int i = 0;; ++i) {
         const int key0 = k_begin + (warp + kWarps * i) * kTileKeys;
         if (key0 >= k_end) break;
+        float far[2][4];   // biases
+        if (bias)
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int idx = min(key0 + j * 8 + lc + (e & 1), k_end - 1), dist = pos - (idx < front ? idx : lo + idx - front);
+                    far[j][e] = bias[size_t(h0 + min(lr + (e >> 1) * 8, nh - 1)) * d.bias_n + min(dist, d.bias_n - 1)];
+                }
         cp_wait<1>();
         __syncwarp();
         const uint32_t at = uint32_t(__cvta_generic_to_shared(mine + (i & 1) * L.stage));
@@ -309,6 +322,7 @@ __global__ void __launch_bounds__(kThreads, 1) attn_rows_mma_kernel(const AttnDi
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 float v = d.softcap > 0.f ? d.softcap * kLog2e * tanhf(s[j][e] * inv_cap) : s[j][e] * scale2;
+                if (bias) v = fmaf(far[j][e], kLog2e, v);
                 if (key0 + j * 8 + lc + (e & 1) >= k_end) v = -INFINITY;
                 s[j][e] = v;
                 mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -368,7 +382,7 @@ __global__ void __launch_bounds__(kThreads, 1) attn_rows_mma_kernel(const AttnDi
 
 bool mma_supported(const AttnDims& d) { return d.vdim_p <= 256 && mma_smem(d) <= 220 * 1024; }
 
-int32_t run_mma(const AttnDims& d, const void* q, const void* cache, const float* gate, const float* sink, void* out, int out_ld, const StepRows& rows, int max_keys, cudaStream_t st) {
+int32_t run_mma(const AttnDims& d, const void* q, const void* cache, const float* gate, const float* sink, const float* bias, void* out, int out_ld, const StepRows& rows, int max_keys, cudaStream_t st) {
     const int gq = d.heads / d.groups, blocks = (gq + kRowHeads - 1) / kRowHeads;
     const size_t smem = mma_smem(d);
     auto go = [&](auto kern) -> int32_t {
@@ -389,7 +403,7 @@ int32_t run_mma(const AttnDims& d, const void* q, const void* cache, const float
         int splits = 1;
         for (int c = 2; c <= 8; ++c)
             if ((long long)rows.n * d.groups * blocks <= fits[c] && max_keys > (c - 1) * kWarps * kTileKeys) splits = c;
-        FORGE_CUDA(launch_pdl_cluster(kern, dim3(splits, d.groups * blocks, rows.n), dim3(kThreads), splits, smem, st, d, static_cast<const bf16*>(q), static_cast<const bf16*>(cache), gate, sink,
+        FORGE_CUDA(launch_pdl_cluster(kern, dim3(splits, d.groups * blocks, rows.n), dim3(kThreads), splits, smem, st, d, static_cast<const bf16*>(q), static_cast<const bf16*>(cache), gate, sink, bias,
                                       static_cast<bf16*>(out), out_ld, rows));
         FORGE_LAUNCH_CHECK();
         return FORGE_OK;
@@ -597,7 +611,7 @@ __global__ void __launch_bounds__(256) qk_post4_kernel(const AttnDims d, const Q
 int32_t qk_post(const AttnDims& d, const QkPost& p, int dtype, const float* proj, int ldp, int k_col, const float* q_norm, const float* k_norm, const float* rope, void* q, void* cache,
                 const int32_t* place, const StepRows& rows, const RouteBeside* route, cudaStream_t st) {
     if (rows.n <= 0) return FORGE_OK;
-    if (route && (rows.n > kScaleRows || route->d.experts > kMaxExperts)) { set_error("routing: %d rows, %d experts", rows.n, route->d.experts); return FORGE_ERR_SHAPE; }
+    if (route && (rows.n > kScaleRows || route->d.choices() > kMaxExperts)) { set_error("routing: %d rows, %d experts", rows.n, route->d.experts); return FORGE_ERR_SHAPE; }
     if (d.dim > kQkDims * 32 || p.rot_dims > d.dim || p.rot_dims % 2) { set_error("attention: head size %d with %d rotated dimensions", d.dim, p.rot_dims); return FORGE_ERR_SHAPE; }
     auto go = [&](auto t) -> int32_t {
         using T = decltype(t);
@@ -622,14 +636,15 @@ int32_t qk_post(const AttnDims& d, const QkPost& p, int dtype, const float* proj
 
 bool attn_rows_supported(const AttnDims& d) { return d.vdim_p <= 512 && smem_bytes(d, 4) <= 200 * 1024; }
 
-int32_t attn_rows(const AttnDims& d, int dtype, const void* q, const void* cache, const float* gate, const float* sink, void* out, int out_ld, const StepRows& rows, int max_keys, cudaStream_t st) {
+int32_t attn_rows(const AttnDims& d, int dtype, const void* q, const void* cache, const float* gate, const float* sink, const float* bias, void* out, int out_ld, const StepRows& rows, int max_keys,
+                  cudaStream_t st) {
     if (rows.n <= 0) return FORGE_OK;
     if (!attn_rows_supported(d)) { set_error("row attention: head sizes %d / %d unsupported", d.dim, d.vdim); return FORGE_ERR_SHAPE; }
-    if (dtype == FORGE_BF16 && mma_supported(d)) return run_mma(d, q, cache, gate, sink, out, out_ld, rows, max_keys, st);
+    if (dtype == FORGE_BF16 && mma_supported(d)) return run_mma(d, q, cache, gate, sink, bias, out, out_ld, rows, max_keys, st);
     const int gq = d.heads / d.groups, blocks = (gq + 3) / 4;
     int splits = 1;   // about two CTAs per SM, no split shorter than one round of its warps
     while (splits < 8 && rows.n * d.groups * blocks * splits * 2 <= 296 && max_keys > splits * kThreads) splits *= 2;
-    return dtype == FORGE_F32 ? run<float>(d, q, cache, gate, sink, out, out_ld, rows, splits, st) : run<__nv_bfloat16>(d, q, cache, gate, sink, out, out_ld, rows, splits, st);
+    return dtype == FORGE_F32 ? run<float>(d, q, cache, gate, sink, bias, out, out_ld, rows, splits, st) : run<__nv_bfloat16>(d, q, cache, gate, sink, bias, out, out_ld, rows, splits, st);
 }
 
 }  // namespace forge

@@ -1,6 +1,7 @@
 // Softmax attention over a paged cache of keys and values, grouped heads, optional cap on the scores, optional chunks (position i
-// sees the keys of its own chunk of positions only) or a sliding window with kept first tokens, optional sinks (a learned score per
-// head that enters the denominator only); and what stands in front of it: norms and rotation of queries and keys.
+// sees the keys of its own chunk of positions only) or a sliding window, in front of which first tokens are kept or blocks of tokens are
+// seen as the mean of their keys and values, optional learned biases by distance, optional sinks (a learned score per head that enters
+// the denominator only), optional mixing of the heads' weights; and what stands in front of it: norms and rotation of queries and keys.
 #pragma once
 
 #include "dense.cuh"
@@ -14,11 +15,29 @@ struct AttnDims {
     float scale = 1.f, softcap = 0.f;               // softcap > 0: score <- softcap * tanh(score / softcap)
     int chunk = 0;                                  // > 0: key j is visible to i only if j / chunk == i / chunk
     int window = 0, keep = 0;                       // window > 0: key j is visible to i only if i - j < window or j < keep
+    // pool > 0 (keep is 0): of the blocks of `pool` tokens those that lie wholly in front of the window are seen, a block as one key and value.  A block's
+    // row belongs to the page of its first token; these rows follow those of the pages, from cache row pool_row0.
+    int pool = 0, pool_row0 = 0;
+    int bias_n = 0;                                 // > 0: scores get bias[head][min(i - j, bias_n - 1)]
     __host__ __device__ int row() const { return groups * (dim_p + vdim_p); }
+    __host__ __device__ int pool_slots() const { return pool > 0 ? (FORGE_KV_PAGE + pool - 1) / pool : 0; }   // block rows of a page
+    __host__ __device__ int blocks(int pos) const { return pool > 0 ? first_key(pos) / pool : 0; }
+    // cache row of block b; pt: the sequence's pages
+    __device__ size_t block_row(const int32_t* pt, int b) const {
+        const int page = b * pool / FORGE_KV_PAGE, first = (page * FORGE_KV_PAGE + pool - 1) / pool;
+        return size_t(pool_row0) + size_t(pt[page]) * pool_slots() + (b - first);
+    }
+    // The keys that a position sees are numbered: `front` blocks or kept tokens, then the tokens from `lo` on.
+    __host__ __device__ int front(int pos) const { return pool > 0 ? blocks(pos) : kept(pos); }
+    __device__ size_t key_row(const int32_t* pt, int i, int front, int lo) const {
+        if (pool > 0 && i < front) return block_row(pt, i);
+        const int key = i < front ? i : lo + i - front;
+        return size_t(pt[key / FORGE_KV_PAGE]) * FORGE_KV_PAGE + key % FORGE_KV_PAGE;
+    }
     // position pos sees the keys first_key(pos) .. pos, and the first kept(pos) in front of them
     __host__ __device__ int first_key(int pos) const { return chunk > 0 ? pos / chunk * chunk : window > 0 && pos >= window ? pos - window + 1 : 0; }
     __host__ __device__ int kept(int pos) const { const int lo = first_key(pos); return window > 0 ? (keep < lo ? keep : lo) : 0; }
-    int most_keys(int n) const { return chunk > 0 ? (n < chunk ? n : chunk) : window > 0 && (long long)window + keep < n ? window + keep : n; }
+    int most_keys(int n) const { return chunk > 0 ? (n < chunk ? n : chunk) : window > 0 && (long long)window + keep + (pool > 0 ? n / pool : 0) < n ? window + keep + (pool > 0 ? n / pool : 0) : n; }
 };
 
 // Queries and keys of a step's rows: rms norm (per head, or over all heads at once), rotary positions on the first rot_dims dimensions,
@@ -37,7 +56,24 @@ int32_t qk_post(const AttnDims& d, const QkPost& p, int dtype, const float* proj
 
 bool attn_rows_supported(const AttnDims& d);
 // q: T rows [heads][dim_p]; out[row][head * vdim + i] = gate[row][head] * attention, T (gate null: ungated).  sink: score per head, or null.
-// max_keys: most keys a row sees.
-int32_t attn_rows(const AttnDims& d, int dtype, const void* q, const void* cache, const float* gate, const float* sink, void* out, int out_ld, const StepRows& rows, int max_keys, cudaStream_t st);
+// bias: f32 [heads][bias_n], or null.  max_keys: most keys a row sees.
+int32_t attn_rows(const AttnDims& d, int dtype, const void* q, const void* cache, const float* gate, const float* sink, const float* bias, void* out, int out_ld, const StepRows& rows, int max_keys,
+                  cudaStream_t st);
+
+// ---- blocks seen as one key (attn_pool.cu)
+// The means of the blocks that the step's rows complete.
+int32_t pool_blocks(const AttnDims& d, int dtype, void* cache, const StepRows& rows, cudaStream_t st);
+// For prompts: block rows of sequences in a row, 64 per table entry.  dst: rows like the cache's.
+struct PoolChunk { int32_t pages0, block0, len, unused; };   // first entry of the sequence in `pages`, first block, positions of the sequence
+int32_t gather_blocks(const AttnDims& d, int dtype, void* dst, const void* cache, const int32_t* pages, const PoolChunk* chunks, int n_chunks, cudaStream_t st);
+
+// ---- mixed heads (attn_talk.cu): the weight of head h becomes the sum over heads g of talk[h][g] times the weight of g
+bool talk_rows_supported(const AttnDims& d);
+size_t talk_rows_bytes(const AttnDims& d, int rows, int max_keys);
+// out[row][head * vdim + i] = factor * attention, T; scratch: talk_rows_bytes of at most max_bytes (more rows go in turn).
+int32_t talk_rows(const AttnDims& d, int dtype, const void* q, const void* cache, const float* talk, float factor, void* scratch, size_t max_bytes, void* out, int out_ld, const StepRows& rows, int max_keys,
+                  cudaStream_t st);
+// out[row][h * vdim + i] = factor * sum over g of talk[h][g] o[row][g][group of h][i]: o bf16 [rows][heads][groups][vdim_p], every head's weights on all groups' values
+int32_t talk_heads(const AttnDims& d, const void* o, const float* talk, float factor, void* out, int out_ld, int rows, cudaStream_t st);
 
 }  // namespace forge

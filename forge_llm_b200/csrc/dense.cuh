@@ -75,6 +75,8 @@ struct OutSeg {
     float limit = 0.f;
     const float* mul = nullptr; const float* add = nullptr;   // per row (add: not with gated pairs)
     const int32_t* place = nullptr;   // SEG_CAST: row of dst that token goes to (null: the token's own number)
+    // SEG_CAST, blending: what is stored is own * v + other * blend[row of dst * blend_ld + column of dst], blend being T rows
+    const void* blend = nullptr; int blend_ld = 0; float own = 1.f, other = 0.f;
     bool fresh = false;               // SEG_RESID: dst is written, not added to
     int act_col = 0;                  // first column of the activations these rows are multiplied with (segments that differ in it start at multiples of 128 rows)
     After after;

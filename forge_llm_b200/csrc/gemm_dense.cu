@@ -56,7 +56,10 @@ struct RowOut {
     size_t ld;
     float* f32; T* t;        // the row's place of token 0
     const int32_t* place;
+    const T* blend; size_t blend_ld; float own, other;   // blend: the row's place of row 0
     float limit, mul, add, nw, nb, plus;
+    // what is stored for v in row `to` of dst
+    __device__ __forceinline__ float blended(float v, size_t to) const { return blend ? fmaf(other, to_f(blend[to * blend_ld]), own * v) : v; }
 };
 template <typename T>
 __device__ __forceinline__ RowOut<T> row_out(const DenseOut& o, int row, int first_row) {
@@ -77,6 +80,7 @@ __device__ __forceinline__ RowOut<T> row_out(const DenseOut& o, int row, int fir
     q.f32 = static_cast<float*>(g.dst) + col;
     q.t = static_cast<T*>(g.dst) + col;
     q.place = g.place;
+    if (q.kind == SEG_CAST && g.blend && q.ok) { q.blend = static_cast<const T*>(g.blend) + col; q.blend_ld = size_t(g.blend_ld); q.own = g.own; q.other = g.other; }
     q.limit = g.limit;
     if (q.ok) {
         if (g.mul) q.mul = g.mul[r];
@@ -132,7 +136,7 @@ __device__ __forceinline__ float put_one(const RowOut<T>& g, const Leave<T>& n, 
     switch (g.kind) {
         case SEG_CLAMPED_GLU: if (even_row) *h = to_t<T>(clamped_glu<T>(v, up, g.limit) * w); break;
         case SEG_SILU_GLU: if (even_row) *h = to_t<T>(act_sigmoid<T>(v, v) * up * w); break;
-        case SEG_CAST: g.t[(g.place ? size_t(g.place[t]) : t) * g.ld] = to_t<T>(v); break;
+        case SEG_CAST: { const size_t to = g.place ? size_t(g.place[t]) : t; g.t[to * g.ld] = to_t<T>(g.blended(v, to)); break; }
         case SEG_SIGMOID: *h = to_t<T>(act_sigmoid<T>(1.f, v)); break;
         case SEG_SILU: *h = to_t<T>(act_sigmoid<T>(v, v)); break;
         case SEG_TANH: *h = to_t<T>(tanhf(v)); break;
@@ -509,10 +513,17 @@ __global__ void __launch_bounds__(kThreads<NT>, NT <= 16 ? 2 : 1) gemm_dense_ker
                     }
                 } else if (g.ok) switch (g.kind) {
                     case SEG_CAST:
-                        if (g.place) {
+                        if (g.place || g.blend) {
                             int to[CH];
 #pragma unroll
-                            for (int c = 0; c < CH; ++c) to[c] = c < n_c ? g.place[t0 + c] : 0;
+                            for (int c = 0; c < CH; ++c) to[c] = c >= n_c ? 0 : g.place ? g.place[t0 + c] : int(t0) + c;
+                            if (g.blend) {
+                                float other[CH];
+#pragma unroll
+                                for (int c = 0; c < CH; ++c) other[c] = c < n_c ? to_f(g.blend[size_t(to[c]) * g.blend_ld]) : 0.f;
+#pragma unroll
+                                for (int c = 0; c < CH; ++c) v[c] = fmaf(g.other, other[c], g.own * v[c]);
+                            }
 #pragma unroll
                             for (int c = 0; c < CH; ++c) if (c < n_c) g.t[size_t(to[c]) * g.ld] = __float2bfloat16_rn(v[c]);
                         } else put_t([](float x) { return x; });

@@ -17,7 +17,13 @@ __global__ void __launch_bounds__(1024) route_few_kernel(const RouterDims d, con
 
 __global__ void __launch_bounds__(256) choose_kernel(const RouterDims d, const float* __restrict__ logits, int rows, const RouteTables t) {
     const int r = blockIdx.x * 8 + (threadIdx.x >> 5);
-    if (r < rows) choose(logits + size_t(r) * d.experts, d.experts, d.top, t.expert + size_t(r) * d.top, t.weight + size_t(r) * d.top);
+    if (r >= rows) return;
+    choose(logits + size_t(r) * d.choices(), d, t.expert + size_t(r) * d.top, t.weight + size_t(r) * d.top);
+    if (d.identity && (threadIdx.x & 31) == 0) {
+        float passed = 0.f;
+        for (int k = 0; k < d.top; ++k) if (t.expert[size_t(r) * d.top + k] >= d.experts) passed += t.weight[size_t(r) * d.top + k];
+        t.passed[r] = passed;
+    }
 }
 
 // One CTA.  Every warp owns a run of pairs; a pair's place among its expert's is what earlier warps, earlier pairs of the warp and
@@ -31,7 +37,8 @@ __global__ void __launch_bounds__(1024) slots_kernel(const RouterDims d, int row
     for (int i = threadIdx.x; i < 32 * E; i += 1024) s_cnt[i] = 0;
     __syncthreads();
     for (int p = p0; p < p1; p += 32) {
-        const int e = p + lane < p1 ? t.expert[p + lane] : -1;
+        int e = p + lane < p1 ? t.expert[p + lane] : -1;
+        if (e >= E) e = -1;     // passed on: no slot
         const uint32_t same = __match_any_sync(0xffffffffu, e);
         if (e >= 0 && lane == __ffs(same) - 1) cnt[e] += __popc(same);
         __syncwarp();
@@ -58,6 +65,7 @@ __global__ void __launch_bounds__(1024) slots_kernel(const RouterDims d, int row
             tiles += __shfl_sync(0xffffffffu, sn, 31);
         }
         if (lane == 0) *t.n_tiles = tiles;
+        for (int i = slots + lane; i < pairs; i += 32) { t.row[i] = 0; t.slot_weight[i] = 0.f; }   // slots that nobody took are gathered, too
     }
     __syncthreads();
     for (int e = warp; e < E; e += 32)
@@ -66,7 +74,9 @@ __global__ void __launch_bounds__(1024) slots_kernel(const RouterDims d, int row
             t.tiles[tile0[e] + i] = GroupTile{e, at, min(tile_rows, total[e] - i * tile_rows), at};
         }
     for (int p = p0; p < p1; p += 32) {
-        const int i = p + lane, e = i < p1 ? t.expert[i] : -1;
+        const int i = p + lane;
+        int e = i < p1 ? t.expert[i] : -1;
+        if (e >= E) { e = -1; t.slot[i] = -1; }
         const uint32_t same = __match_any_sync(0xffffffffu, e);
         if (e >= 0) {
             const int slot = start[e] + cnt[e] + __popc(same & ((1u << lane) - 1));
@@ -108,13 +118,90 @@ __global__ void __launch_bounds__(256) add_experts_kernel(float* __restrict__ x,
     }
 }
 
+// A CTA per row.  NV: pieces of four columns per thread (rows of up to 1024 NV); 0: any width.
+template <typename T, int NV>
+__global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* y, int width, float eps, float gain, const MixtureSum mix, const After after) {
+    __shared__ float red[8];
+    const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    float* xr = x + size_t(r) * width;
+    const float* yr = y + size_t(r) * width;
+    auto factor = [&](float ss) {
+        ss = warp_sum(ss);
+        if (lane == 0) red[warp] = ss;
+        __syncthreads();
+        ss = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) ss += red[w];
+        return gain / sqrtf(ss / float(width) + eps);
+    };
+    pdl_trigger();
+    pdl_wait();
+    const float passed = mix.passed ? mix.passed[r] : 0.f;
+    if constexpr (NV > 0) {
+        float4 vx[NV], vy[NV];
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int c = 4 * (threadIdx.x + 256 * j);
+            const bool ok = c < width;
+            vx[j] = ok ? get4(xr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            vy[j] = ok ? get4(yr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        if (mix.e)
+            for (int k = 0; k < mix.top; ++k) {
+                const int s = mix.slot[size_t(r) * mix.top + k];
+                if (s < 0) continue;
+#pragma unroll
+                for (int j = 0; j < NV; ++j) {
+                    const int c = 4 * (threadIdx.x + 256 * j);
+                    if (c < width) vy[j] = add4(vy[j], get4(mix.e + size_t(s) * width + c));
+                }
+            }
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            float4& v = vy[j];
+            v = make_float4(fmaf(passed, vx[j].x, v.x), fmaf(passed, vx[j].y, v.y), fmaf(passed, vx[j].z, v.z), fmaf(passed, vx[j].w, v.w));
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+        }
+        const float f = factor(ss);
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {   // whole warps stay
+            const int c = 4 * (threadIdx.x + 256 * j);
+            const bool ok = c < width;
+            float4 v = make_float4(fmaf(f, vy[j].x, vx[j].x), fmaf(f, vy[j].y, vx[j].y), fmaf(f, vy[j].z, vx[j].z), fmaf(f, vy[j].w, vx[j].w));
+            v = leave_four<T>(after, v, size_t(r), size_t(width), c, ok);
+            if (ok) put4(xr + c, v);
+        }
+    } else {
+        auto value = [&](int c) {
+            float v = yr[c];
+            if (mix.e)
+                for (int k = 0; k < mix.top; ++k) {
+                    const int s = mix.slot[size_t(r) * mix.top + k];
+                    if (s >= 0) v += mix.e[size_t(s) * width + c];
+                }
+            return fmaf(passed, xr[c], v);
+        };
+        float ss = 0.f;
+        for (int c = threadIdx.x; c < width; c += 256) { const float v = value(c); ss = fmaf(v, v, ss); }
+        const float f = factor(ss);
+        for (int c0 = 0; c0 < width; c0 += 256) {
+            const int c = c0 + threadIdx.x;
+            const bool ok = c < width;
+            float v = ok ? fmaf(f, value(c), xr[c]) : 0.f;
+            v = leave_value<T>(after, v, size_t(r), size_t(width), c, ok);
+            if (ok) xr[c] = v;
+        }
+    }
+}
+
 size_t align16(size_t n) { return (n + 15) & ~size_t(15); }
 
 }  // namespace
 
 size_t route_bytes(const RouterDims& d, int rows) {
     const size_t pairs = size_t(rows) * d.top;
-    return 5 * align16(pairs * 4) + size_t(d.experts) * kScaleRows * 4 + (pairs + d.experts) * sizeof(GroupTile) + 16;
+    return 5 * align16(pairs * 4) + align16(size_t(rows) * 4) + size_t(d.experts) * kScaleRows * 4 + (pairs + d.experts) * sizeof(GroupTile) + 16;
 }
 GroupTable few_table(const RouterDims& d, int rows, const RouteTables& t) {
     return GroupTable{t.tiles, t.n_tiles, int(std::min<long long>(d.experts, (long long)rows * d.top)), rows <= 16 ? 16 : 32, t.row_weight};
@@ -129,11 +216,12 @@ RouteTables route_tables(void* p, const RouterDims& d, int rows) {
     t.row_weight = reinterpret_cast<float*>(take(size_t(d.experts) * kScaleRows * 4));
     t.expert = reinterpret_cast<int32_t*>(take(pairs)); t.weight = reinterpret_cast<float*>(take(pairs)); t.slot = reinterpret_cast<int32_t*>(take(pairs));
     t.row = reinterpret_cast<int32_t*>(take(pairs)); t.slot_weight = reinterpret_cast<float*>(take(pairs));
+    t.passed = reinterpret_cast<float*>(take(align16(size_t(rows) * 4)));
     return t;
 }
 
 int32_t route_few(const RouterDims& d, const float* logits, int rows, const RouteTables& t, GroupTable* out, cudaStream_t st) {
-    if (rows > kScaleRows || d.experts > kMaxExperts) { set_error("routing: %d rows, %d experts", rows, d.experts); return FORGE_ERR_SHAPE; }
+    if (rows > kScaleRows || d.choices() > kMaxExperts) { set_error("routing: %d rows, %d experts", rows, d.experts); return FORGE_ERR_SHAPE; }
     *out = few_table(d, rows, t);
     const size_t smem = route_few_smem(d);
     FORGE_CUDA(cudaFuncSetAttribute(route_few_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(route_few_smem(RouterDims{kMaxExperts, 1}))));
@@ -143,7 +231,7 @@ int32_t route_few(const RouterDims& d, const float* logits, int rows, const Rout
 }
 
 int32_t route_slots(const RouterDims& d, const float* logits, int rows, const RouteTables& t, GroupTable* out, cudaStream_t st) {
-    if (d.experts > kMaxExperts || (long long)rows * d.top > (1 << 30)) { set_error("routing: %d rows, %d experts", rows, d.experts); return FORGE_ERR_SHAPE; }
+    if (d.choices() > kMaxExperts || (long long)rows * d.top > (1 << 30)) { set_error("routing: %d rows, %d experts", rows, d.experts); return FORGE_ERR_SHAPE; }
     const int pairs = rows * d.top, tile_rows = group_tile_rows((pairs + d.experts - 1) / d.experts);
     *out = GroupTable{t.tiles, t.n_tiles, std::min(pairs, pairs / tile_rows + d.experts), tile_rows, t.slot_weight};
     choose_kernel<<<(rows + 7) / 8, 256, 0, st>>>(d, logits, rows, t);
@@ -161,6 +249,19 @@ int32_t add_experts(float* x, const float* y, const RouterDims& d, const RouteTa
     else add_experts_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(x, y, t.slot, d.top, width, after);
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
+}
+
+int32_t add_normed(float* x, const float* y, int rows, int width, float eps, float gain, const MixtureSum& mix, const After& after, int dtype, cudaStream_t st) {
+    if (rows <= 0) return FORGE_OK;
+    auto go = [&](auto type) -> int32_t {
+        using T = decltype(type);
+        const bool four = width % 4 == 0 && after.ld % 4 == 0 && after.col2 % 4 == 0;
+        auto kern = !four || width > 8192 ? add_normed_kernel<T, 0> : width <= 1024 ? add_normed_kernel<T, 1> : width <= 2048 ? add_normed_kernel<T, 2> : width <= 4096 ? add_normed_kernel<T, 4> : add_normed_kernel<T, 8>;
+        FORGE_CUDA(launch_pdl(kern, dim3(rows), dim3(256), 0, st, x, y, width, eps, gain, mix, after));
+        FORGE_LAUNCH_CHECK();
+        return FORGE_OK;
+    };
+    return dtype == FORGE_F32 ? go(float{}) : go(__nv_bfloat16{});
 }
 
 }  // namespace forge

@@ -7,13 +7,20 @@ namespace forge {
 
 constexpr int kMaxExperts = 512;
 
-struct RouterDims { int experts = 0, top = 0; };
+// Choices behind the experts pass a token's input on (identity).  correction (device, null: none): the `top` largest of softmax(logits) +
+// correction are chosen and weighted with their softmax over all choices; without it the largest logits, weighted by the softmax over the chosen.
+struct RouterDims {
+    int experts = 0, top = 0, identity = 0;
+    const float* correction = nullptr;
+    __host__ __device__ int choices() const { return experts + identity; }
+};
 // Device tables of one routing.  A pair is (row, k), k = 0 .. top - 1; pairs are dealt to slots expert by expert, in the order of
 // rows within an expert.
 struct RouteTables {
     int32_t* expert = nullptr; float* weight = nullptr; int32_t* slot = nullptr;   // [rows][top]
     int32_t* row = nullptr; float* slot_weight = nullptr;                          // [rows * top], by slot
     float* row_weight = nullptr;                                                   // few rows: [experts][kScaleRows], zero where the expert is not used
+    float* passed = nullptr;                                                       // [rows]: weight of the choices that pass the input on
     GroupTile* tiles = nullptr; int32_t* n_tiles = nullptr;
 };
 size_t route_bytes(const RouterDims& d, int rows);
@@ -21,25 +28,43 @@ RouteTables route_tables(void* p, const RouterDims& d, int rows);
 
 GroupTable few_table(const RouterDims& d, int rows, const RouteTables& t);   // of route_few
 inline size_t route_few_smem(const RouterDims& d) { return size_t(d.experts) * (kScaleRows + 1) * 4; }
-// logits: f32 [rows][experts].  The `top` largest of a row, weighted by the softmax over them.
+// logits: f32 [rows][choices].
 // Few rows (at most kScaleRows): a tile of all rows per expert that any of them uses.
 int32_t route_few(const RouterDims& d, const float* logits, int rows, const RouteTables& t, GroupTable* out, cudaStream_t st);
 // Any number: tiles of slots.
 int32_t route_slots(const RouterDims& d, const float* logits, int rows, const RouteTables& t, GroupTable* out, cudaStream_t st);
 // x[r] += sum over k of y[slot(r, k)], f32 rows of `width`, then `after`
 int32_t add_experts(float* x, const float* y, const RouterDims& d, const RouteTables& t, int rows, int width, const After& after, int dtype, cudaStream_t st);
+// x += gain * y / rms(y), then `after`.  y: f32 rows; with a mixture first y[r] += passed[r] x[r], and with expert outputs e (f32 rows by slot) += those of the
+// row's slots.
+struct MixtureSum { const float* passed = nullptr; const float* e = nullptr; const int32_t* slot = nullptr; int top = 0; };
+int32_t add_normed(float* x, const float* y, int rows, int width, float eps, float gain, const MixtureSum& mix, const After& after, int dtype, cudaStream_t st);
 
 #ifdef __CUDACC__
 constexpr int kPerLane = kMaxExperts / 32;
 
-// The warp chooses the `top` largest of z (lower numbers win ties); expert[k] and weight[k] by lane 0.
-__device__ __forceinline__ void choose(const float* z, int experts, int top, int32_t* expert, float* weight) {
-    const int lane = threadIdx.x & 31;
+// The warp chooses a row's experts (lower numbers win ties); expert[k] and weight[k] by lane 0.
+__device__ __forceinline__ void choose(const float* z, const RouterDims& d, int32_t* expert, float* weight) {
+    const int lane = threadIdx.x & 31, experts = d.choices(), top = d.top;
     float v[kPerLane];
     uint32_t taken = 0;
 #pragma unroll
     for (int i = 0; i < kPerLane; ++i) v[i] = lane + 32 * i < experts ? z[lane + 32 * i] : 0.f;
     float first = 0.f, sum = 0.f;
+    if (d.correction) {
+        float mx = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < kPerLane; ++i) if (lane + 32 * i < experts) mx = fmaxf(mx, v[i]);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < kPerLane; ++i) if (lane + 32 * i < experts) s += v[i] = expf(v[i] - mx);
+        s = warp_sum(s);
+        first = mx; sum = s;
+#pragma unroll
+        for (int i = 0; i < kPerLane; ++i) if (lane + 32 * i < experts) v[i] = v[i] / s + d.correction[lane + 32 * i];
+    }
     for (int k = 0; k < top; ++k) {
         float best = 0.f;
         int at = -1;
@@ -54,10 +79,11 @@ __device__ __forceinline__ void choose(const float* z, int experts, int top, int
         }
         at = __shfl_sync(0xffffffffu, at, 0);      // (values that are no numbers compare differently in different lanes)
         best = __shfl_sync(0xffffffffu, best, 0);
+        if ((at & 31) == lane) taken |= 1u << (at >> 5);
+        if (d.correction) { if (lane == 0) { expert[k] = at; weight[k] = expf(z[at] - first); } continue; }
         if (k == 0) first = best;
         const float e = expf(best - first);
         sum += e;
-        if ((at & 31) == lane) taken |= 1u << (at >> 5);
         if (lane == 0) { expert[k] = at; weight[k] = e; }
     }
     if (lane == 0) for (int k = 0; k < top; ++k) weight[k] /= sum;
@@ -73,13 +99,18 @@ __device__ __forceinline__ void route_few_rows(const RouterDims& d, const float*
     int* used = reinterpret_cast<int*>(s_w + d.experts * kScaleRows);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int r = warp; r < rows; r += blockDim.x / 32) {
-        choose(logits + size_t(r) * d.experts, d.experts, d.top, t.expert + r * d.top, t.weight + r * d.top);
-        if (lane == 0)
+        choose(logits + size_t(r) * d.choices(), d, t.expert + r * d.top, t.weight + r * d.top);
+        if (lane == 0) {
+            float passed = 0.f;
             for (int k = 0; k < d.top; ++k) {
                 const int e = t.expert[r * d.top + k];
-                s_w[e * kScaleRows + r] = t.weight[r * d.top + k];
+                const float w = t.weight[r * d.top + k];
+                if (e >= d.experts) { passed += w; continue; }
+                s_w[e * kScaleRows + r] = w;
                 used[e] = 1;
             }
+            t.passed[r] = passed;
+        }
     }
     __syncthreads();
     for (int i = threadIdx.x; i < d.experts * kScaleRows; i += blockDim.x) t.row_weight[i] = s_w[i];

@@ -1,0 +1,41 @@
+// Selective scan: per channel c a state S [states] in f32 that every token decays by its own step size and extends,
+//   S <- exp(dt_c A[c]) S + dt_c x_c B;  y_c = S . C + D_c x_c,  out = factor y gate,
+// with x behind a short causal convolution per channel (bias, silu), whose last inputs are kept in a ring of `taps` rows, the input of
+// position p in row p % taps.  A sequence's state counts as zero when its first row of a step is at position 0.
+#pragma once
+
+#include "recurrent.cuh"
+
+namespace forge {
+
+struct SelectiveDims {
+    int inner = 0, state = 0, rank = 0, taps = 0;   // channels, states per channel, inner size of the step sizes' projection
+    size_t state_values() const { return size_t(inner) * state; }
+    __host__ __device__ size_t ring_values() const { return size_t(taps) * inner; }
+};
+
+struct SelectiveArgs {
+    const void* in = nullptr; int in_ld = 0;               // T rows [inner]: in front of the convolution
+    const float* conv = nullptr; const float* conv_add = nullptr; void* ring = nullptr;   // [taps][inner], [inner]; T [slot][taps][inner]
+    void* x = nullptr; int x_ld = 0;                       // T rows [inner] behind it
+    const float* bc = nullptr; int bc_ld = 0;              // f32 rows [B | C]
+    const float* dt = nullptr; int dt_ld = 0;              // f32 rows [inner]: step sizes
+    // or, for single tokens, the projection that forms them: T rows of low_k values per channel over low[row]; a step size is softplus(z + dt_add)
+    const void* dt_w = nullptr; const void* low = nullptr; int low_ld = 0, low_k = 0;
+    const float* dt_add = nullptr;
+    const float* a2 = nullptr;                             // [inner][state]: A in the base of exp2
+    const float* skip = nullptr;                           // D
+    float* state = nullptr;                                // [slot][inner][state]
+    const void* gate = nullptr; int gate_ld = 0;           // T rows [inner]
+    float factor = 1.f;
+    void* out = nullptr; int out_ld = 0;                   // T rows [inner]
+};
+
+bool selective_supported(const SelectiveDims& d);
+// the convolution of single tokens (rows) and of segments
+int32_t selective_conv(const SelectiveDims& d, int dtype, const SelectiveArgs& a, const StepRows& ones, const SegTable& t, cudaStream_t st);
+// the recurrence of single tokens, and of segments of any length (these take step sizes from dt)
+int32_t selective_decode(const SelectiveDims& d, int dtype, const SelectiveArgs& a, const StepRows& ones, cudaStream_t st);
+int32_t selective_segments(const SelectiveDims& d, int dtype, const SelectiveArgs& a, const SegTable& t, cudaStream_t st);
+
+}  // namespace forge

@@ -9,13 +9,14 @@
 #include "checkpoint.cuh"
 #include "moe.cuh"
 #include "recurrent.cuh"
+#include "selective.cuh"
 
 namespace forge {
 
-enum class Norm { DynamicTanh, RmsPlusOne };   // RmsPlusOne: the weight is stored around zero
+enum class Norm { DynamicTanh, RmsPlusOne, RmsScalar };   // RmsPlusOne: the weight is stored around zero; RmsScalar: one weight for all columns
 // Parallel: x += mixer(h) + ff(h) behind one norm.  Sequential: x += mixer(norm1(x)), then x += ff(norm2(x)).
-// ParallelTwo: x += mixer(norm1(x)) + ff(norm2(x)).
-enum class Arrangement { Parallel, Sequential, ParallelTwo };
+// ParallelTwo: x += mixer(norm1(x)) + ff(norm2(x)).  PostNorm: x += norm1(mixer(x)), then x += norm2(ff(x)).
+enum class Arrangement { Parallel, Sequential, ParallelTwo, PostNorm };
 enum class Mlp { ClampedGlu, SiluGlu };
 // What stands in front of a pass of the loop.  Project: a product over [stream | embedding] plus the pass's vector.  Add: the embedding
 // (not in front of the first pass) and the pass's vector are added.
@@ -31,7 +32,8 @@ enum class Mixer {
     ChannelDelta,  // gated delta rule, one decay per head and key channel
     AttnTimeMix,   // gated attention and time mixing side by side, half the sum of their normed outputs
     Softmax,       // attention with normed and rotated queries and keys
-    GatedLinear    // gated linear attention, one decay per head and key channel
+    GatedLinear,   // gated linear attention, one decay per head and key channel
+    AttnSelective  // attention with mixed heads and a selective scan side by side, a weighted sum of their outputs
 };
 // Rotary positions: frequencies base^(-2 i / dims), scaled.
 struct Rotation {
@@ -42,24 +44,41 @@ struct Rotation {
     std::vector<double> frequencies() const;
     double magnitude() const;          // of cos and sin
 };
-struct SoftmaxTraits { QkPost qk; bool bias = false, sink = false; };   // sink: a learned score per head, else one of zero
+// sink: a learned score per head, else one of zero (not with mixed heads).  plain: norms of queries and keys have no weights, the output projection has a bias too, a
+// mask is a plain window or one with blocks in front.  distance: a learned bias by distance.  talk: the heads' weights are mixed.
+struct SoftmaxTraits { QkPost qk; bool bias = false, sink = false, plain = false, distance = false, talk = false; };
+// learned biases by distance n: a bucket each up to half of them, then logarithmic ones up to the distance `longest`
+struct DistanceBuckets {
+    int count = 0, longest = 0;
+    int of(int n) const;
+};
 struct LayerSpec {
     Mixer kind = Mixer::Latent;
     LatentDims mix;                          // Latent
     AttnDims attn;                           // AttnTimeMix, Softmax
     Rotation rot;                            // Latent, Softmax
-    SoftmaxTraits soft;                      // Softmax
+    SoftmaxTraits soft;                      // Softmax, AttnSelective
+    DistanceBuckets distance;
+    int blend_layer = -1;                    // values are blended with those of this earlier layer
+    bool blends = false;                     // takes part in it (the first such layer lends its values)
+    SelectiveDims sel;                       // AttnSelective
+    float left_scale = 1.f, right_scale = 1.f;
     RecurDims rec;                           // Delta, ChannelDelta, AttnTimeMix, GatedLinear
     int decay_rank = 0, gate_rank = 0;       // inner sizes of the two-step projections, from the tensors' shapes
     double tau = 1.0;                        // GatedLinear: a decay is sigmoid(z)^(1 / tau)
     int ff = 0;                              // 0: no feed-forward
     RouterDims router;                       // experts > 0: a mixture of experts of size ff
+    int shared_ff = 0;                       // beside a shared expert
     float limit = 0.f;
     int weights_of = -1;                     // layer whose tensors are used
-    bool has_attn() const { return kind == Mixer::AttnTimeMix || kind == Mixer::Softmax; }
+    bool has_attn() const { return kind == Mixer::AttnTimeMix || kind == Mixer::Softmax || kind == Mixer::AttnSelective; }
     bool has_latent() const { return kind == Mixer::Latent; }
     bool has_state() const { return kind != Mixer::Latent && kind != Mixer::Softmax; }
-    bool has_rotation() const { return kind == Mixer::Latent || kind == Mixer::Softmax; }
+    bool has_rotation() const { return kind == Mixer::Latent || kind == Mixer::Softmax || kind == Mixer::AttnSelective; }
+    // what a sequence keeps besides cache rows: f32 state values and values of the convolution's ring
+    size_t state_values() const { return kind == Mixer::AttnSelective ? sel.state_values() : has_state() ? rec.state_values() : 0; }
+    size_t ring_values() const { return kind == Mixer::AttnSelective ? sel.ring_values() : has_state() ? rec.ring_values() : 0; }
+    int page_rows() const { return FORGE_KV_PAGE + (has_attn() ? attn.pool_slots() : 0); }   // cache rows of a page, those of blocks included
     int cache_row() const { return has_latent() ? mix.row() : has_attn() ? attn.row() : 0; }   // values per position, padding included
 };
 struct LayerRun { int layer, pass; };   // pass >= 0: this pass of the loop starts in front of the layer

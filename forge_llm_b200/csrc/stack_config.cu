@@ -13,12 +13,18 @@ static const Architecture kArchitectures[] = {
     {"Bolenex", Norm::DynamicTanh, Arrangement::Parallel, Mlp::ClampedGlu, LoopEntry::Project, false},
     {"Robazen", Norm::DynamicTanh, Arrangement::Sequential, Mlp::SiluGlu, LoopEntry::Project, false},
     {"Mokatar", Norm::RmsPlusOne, Arrangement::ParallelTwo, Mlp::SiluGlu, LoopEntry::Add, true},
+    {"Tarulix", Norm::RmsScalar, Arrangement::PostNorm, Mlp::SiluGlu, LoopEntry::Project, false},
 };
 // mixers by architecture and the name a layer's "type" gives them
 struct MixerName { const char* architecture; const char* name; Mixer kind; SoftmaxTraits soft; Rotation::Scaling scaling; };
 static SoftmaxTraits traits(QkPost::Scope norm, bool interleaved, bool bias, bool sink) {
     SoftmaxTraits t;
     t.qk.norm = norm; t.qk.interleaved = interleaved; t.bias = bias; t.sink = sink;
+    return t;
+}
+static SoftmaxTraits plain_traits(bool distance, bool sink, bool talk) {
+    SoftmaxTraits t = traits(QkPost::PER_HEAD, false, true, sink);
+    t.plain = true; t.distance = distance; t.talk = talk;
     return t;
 }
 static const MixerName kMixers[] = {
@@ -30,7 +36,19 @@ static const MixerName kMixers[] = {
     {"Mokatar", "attention", Mixer::Softmax, traits(QkPost::PER_HEAD, true, false, true), Rotation::Yarn},
     {"Mokatar", "attention_2", Mixer::Softmax, traits(QkPost::WHOLE, false, true, false), Rotation::Linear},
     {"Mokatar", "gla", Mixer::GatedLinear, {}, Rotation::None},
+    {"Tarulix", "attention", Mixer::Softmax, plain_traits(true, true, false), Rotation::None},
+    {"Tarulix", "parallel", Mixer::AttnSelective, plain_traits(false, false, true), Rotation::None},
 };
+
+int DistanceBuckets::of(int n) const {
+    const int half = count / 2;
+    if (n < half) return n;
+    if (half < 1 || longest <= half) return count - 1;
+    // the quotient of logarithms is an integer where a bucket begins: there rounding must not decide
+    const double x = std::log(double(n) / half) / std::log(double(longest) / half) * (count - half), near = std::round(x);
+    const double b = half + (std::fabs(x - near) < 1e-9 ? near : std::floor(x));
+    return b < count - 1 ? int(b) : count - 1;
+}
 
 bool Rotation::operator<(const Rotation& o) const {
     return std::tie(scaling, dims, base, factor, original, fast, slow) < std::tie(o.scaling, o.dims, o.base, o.factor, o.original, o.fast, o.slow);
@@ -120,8 +138,8 @@ int32_t parse_delta(const Json* m, float eps, bool channel, LayerSpec* L) {
     return check_recur(d);
 }
 
-// mask: "size" is the length of chunks, or of a sliding window beside "keep_first" kept tokens
-enum class MaskKind { Chunks, Window };
+// mask: "size" is the length of chunks, or of a sliding window: beside "keep_first" kept tokens, alone, or behind blocks of "pool" tokens
+enum class MaskKind { Chunks, Kept, Window, Pooled };
 int32_t parse_attn(const Json* m, MaskKind kind, AttnDims* d) {
     double scale, cap = 0;
     FORGE_TRY(need_int(m, "heads", &d->heads));
@@ -137,7 +155,8 @@ int32_t parse_attn(const Json* m, MaskKind kind, AttnDims* d) {
     const Json* mask = m->get("mask");
     if (mask && mask->kind != Json::Null) {
         FORGE_TRY(need_int(mask, "size", kind == MaskKind::Chunks ? &d->chunk : &d->window));
-        if (kind == MaskKind::Window) FORGE_TRY(need_int(mask, "keep_first", &d->keep, 0));
+        if (kind == MaskKind::Kept) FORGE_TRY(need_int(mask, "keep_first", &d->keep, 0));
+        if (kind == MaskKind::Pooled) FORGE_TRY(need_int(mask, "pool", &d->pool));
     }
     FORGE_TRY(heads_fit(d->heads, d->groups));
     d->scale = float(scale); d->softcap = float(cap);
@@ -180,12 +199,38 @@ int32_t parse_rotation(const Json* r, Rotation::Scaling kind, int dim, Rotation*
 }
 
 int32_t parse_softmax(const Json* m, float eps, const MixerName& name, LayerSpec* L) {
-    FORGE_TRY(parse_attn(m, MaskKind::Window, &L->attn));
-    if (L->attn.dim > 512) { set_error("attention: head size %d is not supported", L->attn.dim); return FORGE_ERR_UNSUPPORTED; }
-    FORGE_TRY(parse_rotation(m->get("rot"), name.scaling, L->attn.dim, &L->rot));
-    L->soft = name.soft;
+    const SoftmaxTraits& soft = name.soft;
+    AttnDims& a = L->attn;
+    FORGE_TRY(parse_attn(m, !soft.plain ? MaskKind::Kept : soft.talk ? MaskKind::Pooled : MaskKind::Window, &a));
+    if (a.dim > 512 || (soft.talk && !talk_rows_supported(a))) { set_error("attention: %d heads of %d / %d are not supported", a.heads, a.dim, a.vdim); return FORGE_ERR_UNSUPPORTED; }
+    if (!soft.plain || m->get("rot")) FORGE_TRY(parse_rotation(m->get("rot"), name.scaling, a.dim, &L->rot));
+    if (soft.distance) {
+        FORGE_TRY(need_int(m, "bias_max", &L->distance.longest));
+        const Json* v = m->get("v_mix");
+        L->blends = v && v->kind == Json::Bool && v->flag;
+        a.bias_n = a.window > 0 && a.window <= L->distance.longest ? a.window : L->distance.longest + 1;   // distances further on share the last bucket
+    }
+    L->soft = soft;
     L->soft.qk.eps = eps; L->soft.qk.rot_dims = L->rot.dims;
     return FORGE_OK;
+}
+
+int32_t parse_attn_selective(const Json* m, float eps, const MixerName& name, LayerSpec* L) {
+    const Json *left = m->get("left"), *right = m->get("right");
+    double l, r;
+    if (!left || left->kind != Json::Object) { set_error("config.json: \"left\" must be an object"); return FORGE_ERR_SHAPE; }
+    FORGE_TRY(need_num(m, "left_scale", &l));
+    FORGE_TRY(need_num(m, "right_scale", &r));
+    L->left_scale = float(l); L->right_scale = float(r);
+    FORGE_TRY(parse_softmax(left, eps, name, L));
+    SelectiveDims& d = L->sel;
+    FORGE_TRY(need_int(right, "inner", &d.inner));
+    FORGE_TRY(need_int(right, "state", &d.state));
+    FORGE_TRY(need_int(right, "dt_rank", &d.rank));
+    FORGE_TRY(need_int(right, "conv", &d.taps));
+    if (selective_supported(d)) return FORGE_OK;
+    set_error("selective scan: %d states with %d taps are not supported", d.state, d.taps);
+    return FORGE_ERR_UNSUPPORTED;
 }
 
 int32_t parse_linear(const Json* m, float eps, LayerSpec* L) {
@@ -200,13 +245,17 @@ int32_t parse_linear(const Json* m, float eps, LayerSpec* L) {
     return check_recur(d);
 }
 
-int32_t parse_experts(const Json* mlp, int layer, LayerSpec* L) {
+int32_t parse_experts(const Json* mlp, int layer, bool shared, LayerSpec* L) {
     const Json* router = mlp->get("router");
     FORGE_TRY(need_int(mlp->get("expert"), "ff", &L->ff));
     FORGE_TRY(need_int(router, "experts", &L->router.experts));
     FORGE_TRY(need_int(router, "top", &L->router.top));
-    if (L->router.top > L->router.experts) { set_error("layer %d: top %d of %d experts", layer, L->router.top, L->router.experts); return FORGE_ERR_SHAPE; }
-    if (L->router.experts > kMaxExperts) { set_error("layer %d: %d experts are not supported", layer, L->router.experts); return FORGE_ERR_UNSUPPORTED; }
+    if (shared) {
+        FORGE_TRY(need_int(mlp->get("shared"), "ff", &L->shared_ff));
+        FORGE_TRY(need_int(router, "identity", &L->router.identity, 0));
+    }
+    if (L->router.top > L->router.choices()) { set_error("layer %d: top %d of %d experts", layer, L->router.top, L->router.choices()); return FORGE_ERR_SHAPE; }
+    if (L->router.choices() > kMaxExperts) { set_error("layer %d: %d experts are not supported", layer, L->router.experts); return FORGE_ERR_UNSUPPORTED; }
     return FORGE_OK;
 }
 
@@ -261,14 +310,15 @@ int32_t stack_parse(const Json& c, StackSpec* s) {
             case Mixer::AttnTimeMix: FORGE_TRY(parse_pair(mx, s->eps, &L)); break;
             case Mixer::Softmax: FORGE_TRY(parse_softmax(mx, s->eps, *known, &L)); break;
             case Mixer::GatedLinear: FORGE_TRY(parse_linear(mx, s->eps, &L)); break;
+            case Mixer::AttnSelective: FORGE_TRY(parse_attn_selective(mx, s->eps, *known, &L)); break;
         }
         const Json* mlp = e.get("mlp");
         if (mlp && mlp->kind != Json::Null) {
             std::string kind;
             FORGE_TRY(need_string(mlp, "kind", &kind));
-            const bool experts = kind == "moe" && s->arch->arrangement == Arrangement::ParallelTwo;
-            if (kind != "dense" && !experts) { set_error("layer %d: feed-forward \"%s\" is not supported", i, kind.c_str()); return FORGE_ERR_UNSUPPORTED; }
-            if (experts) FORGE_TRY(parse_experts(mlp, i, &L));
+            const bool post = s->arch->arrangement == Arrangement::PostNorm, experts = kind == "moe" && (post || s->arch->arrangement == Arrangement::ParallelTwo);
+            if ((kind != "dense" || post) && !experts) { set_error("layer %d: feed-forward \"%s\" is not supported", i, kind.c_str()); return FORGE_ERR_UNSUPPORTED; }
+            if (experts) FORGE_TRY(parse_experts(mlp, i, post, &L));
             else FORGE_TRY(need_int(mlp, "ff", &L.ff));
             if (s->arch->dense == Mlp::ClampedGlu) {
                 double limit;
@@ -291,6 +341,15 @@ int32_t stack_parse(const Json& c, StackSpec* s) {
             set_error("layer %d: weights_of %d names a layer of other sizes or without tensors", i, L.weights_of);
             return FORGE_ERR_SHAPE;
         }
+    }
+    int lender = -1;
+    for (int i = 0; i < n; ++i) {
+        LayerSpec& L = s->layers[i];
+        if (!L.blends) continue;
+        if (lender < 0) { lender = i; continue; }
+        const AttnDims &a = L.attn, &b = s->layers[lender].attn;
+        if (a.groups != b.groups || a.vdim != b.vdim) { set_error("layer %d: its values cannot be blended with those of layer %d", i, lender); return FORGE_ERR_SHAPE; }
+        L.blend_layer = lender;
     }
     const Json* loop = c.get("loop");
     if (loop && loop->kind != Json::Null) {
@@ -319,10 +378,29 @@ int32_t stack_find_tensors(const Checkpoint& ck, StackSpec* s, StackTensors* t) 
         return FORGE_OK;
     };
     auto norm = [&](const std::string& name) -> int32_t {
+        if (s->arch->norm == Norm::RmsScalar) return get(name, {});
         FORGE_TRY(get(name, {W}));
         if (s->arch->norm != Norm::DynamicTanh) return FORGE_OK;
         FORGE_TRY(get(name + ".b", {W}));
         return get(name + ".alpha", {});
+    };
+    // queries, keys and values with their biases, the output's, behind `at`
+    auto plain_attention = [&](const std::string& at, LayerSpec& L) -> int32_t {
+        const AttnDims& a = L.attn;
+        const int64_t q = int64_t(a.heads) * a.dim, k = int64_t(a.groups) * a.dim, v = int64_t(a.groups) * a.vdim;
+        FORGE_TRY(get(at + "q", {q, W})); FORGE_TRY(get(at + "k", {k, W})); FORGE_TRY(get(at + "v", {v, W}));
+        FORGE_TRY(get(at + "q.b", {q})); FORGE_TRY(get(at + "k.b", {k})); FORGE_TRY(get(at + "v.b", {v}));
+        if (L.soft.distance) {
+            const TensorView* rel = ck.find(prefix + at + "rel");
+            if (!rel || rel->shape.size() != 2 || rel->shape[0] < 2 || rel->shape[0] > (1 << 20)) { set_error("tensor \"%srel\" is missing or no matrix", (prefix + at).c_str()); return FORGE_ERR_SHAPE; }
+            L.distance.count = int(rel->shape[0]);
+            FORGE_TRY(get(at + "rel", {rel->shape[0], a.heads}));
+        }
+        if (L.soft.sink) FORGE_TRY(get(at + "sink", {a.heads}));
+        if (L.soft.talk) FORGE_TRY(get(at + "talk", {a.heads, a.heads}));
+        if (L.blend_layer >= 0) FORGE_TRY(get(at + "vmix", {}));
+        FORGE_TRY(get(at + "o", {W, int64_t(a.heads) * a.vdim}));
+        return get(at + "o.b", {W});
     };
     // rows of a matrix [rank][cols] whose first size only its shape gives
     auto rank_of = [&](const std::string& name, int* rank) -> int32_t {
@@ -396,7 +474,19 @@ int32_t stack_find_tensors(const Checkpoint& ck, StackSpec* s, StackTensors* t) 
                 FORGE_TRY(get("mix.right.out", {W}));
                 break;
             }
+            case Mixer::AttnSelective: {
+                const SelectiveDims& d = L.sel;
+                FORGE_TRY(plain_attention("mix.left.", L));
+                FORGE_TRY(get("mix.right.in", {2 * int64_t(d.inner), W}));
+                FORGE_TRY(get("mix.right.conv", {d.inner, d.taps})); FORGE_TRY(get("mix.right.conv.b", {d.inner}));
+                FORGE_TRY(get("mix.right.x", {int64_t(d.rank) + 2 * d.state, d.inner}));
+                FORGE_TRY(get("mix.right.dt", {d.inner, d.rank})); FORGE_TRY(get("mix.right.dt.b", {d.inner}));
+                FORGE_TRY(get("mix.right.A_log", {d.inner, d.state})); FORGE_TRY(get("mix.right.D", {d.inner}));
+                FORGE_TRY(get("mix.right.o", {W, d.inner}));
+                break;
+            }
             case Mixer::Softmax: {
+                if (L.soft.plain) { FORGE_TRY(plain_attention("mix.", L)); break; }
                 const AttnDims& a = L.attn;
                 const int64_t q = int64_t(a.heads) * a.dim, k = int64_t(a.groups) * a.dim, v = int64_t(a.groups) * a.vdim;
                 const bool whole = L.soft.qk.norm == QkPost::WHOLE;
@@ -420,7 +510,11 @@ int32_t stack_find_tensors(const Checkpoint& ck, StackSpec* s, StackTensors* t) 
             const std::string x = "mlp.e" + std::to_string(e);
             FORGE_TRY(get(x + ".gate", {L.ff, W})); FORGE_TRY(get(x + ".up", {L.ff, W})); FORGE_TRY(get(x + ".down", {W, L.ff}));
         }
-        if (L.router.experts) { FORGE_TRY(get("mlp.router", {L.router.experts, W})); FORGE_TRY(get("mlp.router.b", {L.router.experts})); }
+        if (L.router.experts) {
+            FORGE_TRY(get("mlp.router", {L.router.choices(), W}));
+            FORGE_TRY(get(L.shared_ff ? "mlp.correction" : "mlp.router.b", {L.router.choices()}));
+        }
+        if (L.shared_ff) { FORGE_TRY(get("mlp.shared.gate", {L.shared_ff, W})); FORGE_TRY(get("mlp.shared.up", {L.shared_ff, W})); FORGE_TRY(get("mlp.shared.down", {W, L.shared_ff})); }
         if (L.ff && !L.router.experts) {
             FORGE_TRY(get("mlp.gate", {L.ff, W}));
             FORGE_TRY(get("mlp.up", {L.ff, W}));
@@ -438,8 +532,8 @@ void stack_fill_info(const StackSpec& s, ForgeCheckpointInfo* out) {
     for (const LayerSpec& L : s.layers) out->num_weight_layers += L.weights_of < 0;
     for (const LayerRun& r : s.runs) {
         const LayerSpec& L = s.layers[r.layer];
-        out->cache_values_per_token += L.cache_row();
-        if (L.has_state()) out->state_values_per_sequence += int64_t(L.rec.state_values() + L.rec.ring_values()) + (L.kind == Mixer::AttnTimeMix ? s.width : 0);
+        out->cache_values_per_token += L.cache_row();   // (rows of blocks: pool_slots() per page more)
+        if (L.has_state()) out->state_values_per_sequence += int64_t(L.state_values() + L.ring_values()) + (L.kind == Mixer::AttnTimeMix ? s.width : 0);
     }
     if (s.buckets) out->state_values_per_sequence += 1;   // the last token
 }

@@ -9,6 +9,10 @@
 //   delta rules            in [q k v | gate | beta | decay] (a second product for two-step gates and decays), recurrence, out;
 //   two parallel norms     the input's columns are [x (1 + w1) | x (1 + w2)], the RMS of the stream is a factor of the product's epilogue; the mixer's rows
 //                          read the first block, the feed-forward's the second; experts: see experts();
+//   norms on outputs       the stream itself, in the model's type, is every product's input; the sublayer's sum is left as f32 rows, and one
+//                          kernel norms it, adds it and leaves the stream's next form; experts beside a shared one: see mixture();
+//   attention | scan       one `in` product for both, the convolution's projections, one `out` product over [heads | channels] whose
+//                          columns carry the two factors already;
 //   attention | time mix   the input's columns are [h | five shifted mixes] and every row of `in` reads the block it belongs to; keys
 //                          and values go from the epilogue into the cache; one product with both outputs, then the sum of their norms.
 #include <algorithm>
@@ -23,12 +27,12 @@
 // ------------------------------------------------------------------------------------------------ structures
 namespace forge {
 
-struct StreamNorm { float* w = nullptr; float* b = nullptr; float alpha = 0.f; };   // RMS norm: w = one plus the weight
+struct StreamNorm { float* w = nullptr; float* b = nullptr; float alpha = 0.f; };   // RMS norm: w = one plus the weight, or alpha (and in w) the one for all columns
 
 struct LayerWeights {
     StreamNorm norm1, norm2;
     DenseWeight in, out;
-    DenseWeight ff_in, ff_out;    // sequential arrangement
+    DenseWeight ff_in, ff_out;    // sequential arrangement; norms on outputs: [shared | router], [shared | expert 0 | expert 1 ...]
     // latent attention
     DenseWeight kv;               // rows [uk | uv] over the latent
     int q_rows = 0, dkv_row = 0, g_row = 0, glu_row = 0, uv_row = 0;   // first rows of the segments of `in` / `kv`
@@ -46,6 +50,11 @@ struct LayerWeights {
     float *mu = nullptr, *norm_l = nullptr, *norm_r = nullptr;
     // attention with normed queries and keys (k_row, v_row as above)
     float *q_norm = nullptr, *k_norm = nullptr, *sink = nullptr, *q_bias = nullptr, *k_bias = nullptr, *v_bias = nullptr;
+    float *bias = nullptr, *talk = nullptr, *out_bias = nullptr, lambda = 0.f;   // biases by distance, mixing of heads, share of the blended values
+    // selective scan (in_row, gate_row: first rows in `in`; conv, low as above): rows [step sizes' inner values | B C] over the channels
+    DenseWeight scan_in;
+    int in_row = 0, bc_row = 0;
+    float *conv_add = nullptr, *scan_a = nullptr, *skip = nullptr, *minus = nullptr;
     // experts: their columns of `out` follow the heads', ff_k apart
     int router_row = 0, ff_k = 0;
     float* router_bias = nullptr;
@@ -67,11 +76,13 @@ struct StackModel {
     DenseScratch scratch;
     // step buffers, grown on demand (scratch_gen of the model counts the moves)
     struct Buf { void* p = nullptr; size_t cap = 0; };
-    Buf x, h, cat, proj, gate, mid, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, hgate, decay, beta, low, conv, unit, o, pair, place, c_half, c_f32, sel, logits, meta, x0, sums, sum1, router, route, e_in, e_act, e_out;
+    Buf x, h, cat, proj, gate, mid, q, part, ml, ctx_c, ctx_r, ctx_k, ctx_v, hgate, decay, beta, low, conv, unit, o, pair, place, c_half, c_f32, sel, logits, meta, x0, sums, sum1, router, route, e_in, e_act, e_out, scores, joint, blocks, scan, bc;
     std::vector<Buf*> all() {
         return {&x, &h, &cat, &proj, &gate, &mid, &q, &part, &ml, &ctx_c, &ctx_r, &ctx_k, &ctx_v, &hgate, &decay, &beta, &low, &conv, &unit, &o, &pair, &place, &c_half, &c_f32, &sel, &logits, &meta,
-                &x0, &sums, &sum1, &router, &route, &e_in, &e_act, &e_out};
+                &x0, &sums, &sum1, &router, &route, &e_in, &e_act, &e_out, &scores, &joint, &blocks, &scan, &bc};
     }
+    bool rms_stream() const { return spec.arch->norm == Norm::RmsPlusOne; }      // every reader of the stream takes an RMS norm of it
+    bool rms_final() const { return spec.arch->norm != Norm::DynamicTanh; }
     const LayerWeights& weights(int layer) const { return w[spec.layers[layer].weights_of >= 0 ? spec.layers[layer].weights_of : layer]; }
 };
 
@@ -92,11 +103,11 @@ void store(void* dst, int dtype, size_t i, const TensorView& t, size_t j) {
     if (t.dtype == "BF16") { memcpy(static_cast<uint16_t*>(dst) + i, t.data + 2 * j, 2); return; }
     static_cast<__nv_bfloat16*>(dst)[i] = __float2bfloat16_rn(t.at(j));
 }
-// rows of `t` [n][k] into the host image of a matrix with rows of `ld`: row r -> row0 + r * step, columns from col0
-void put_rows(std::vector<uint8_t>& img, int dtype, int ld, const TensorView& t, int row0, int step = 1, int col0 = 0) {
-    const int64_t n = t.shape[0], k = t.shape[1];
-    for (int64_t r = 0; r < n; ++r) {
-        const size_t at = size_t(row0 + r * step) * ld + col0;
+// rows [from, from + count) of `t` [n][k] (count < 0: all) into the host image of a matrix with rows of `ld`: row r -> row0 + (r - from) * step, columns from col0
+void put_rows(std::vector<uint8_t>& img, int dtype, int ld, const TensorView& t, int row0, int step = 1, int col0 = 0, int from = 0, int count = -1) {
+    const int64_t n = count < 0 ? t.shape[0] : from + count, k = t.shape[1];
+    for (int64_t r = from; r < n; ++r) {
+        const size_t at = size_t(row0 + (r - from) * step) * ld + col0;
         if (dtype == FORGE_BF16 && t.dtype == "BF16") memcpy(img.data() + at * 2, t.data + size_t(r) * k * 2, size_t(k) * 2);
         else if (dtype == FORGE_F32 && t.dtype == "F32") memcpy(img.data() + at * 4, t.data + size_t(r) * k * 4, size_t(k) * 4);
         else for (int64_t c = 0; c < k; ++c) store(img.data(), dtype, at + c, t, size_t(r * k + c));
@@ -142,7 +153,7 @@ struct Image {
     std::vector<uint8_t> img;
     int N, K, dtype;
     Image(int n, int k, int dt) : img(size_t(n) * k * dense_size(dt), 0), N(n), K(k), dtype(dt) {}
-    void put(const TensorView* t, int row0, int step = 1, int col0 = 0) { put_rows(img, dtype, K, *t, row0, step, col0); }
+    void put(const TensorView* t, int row0, int step = 1, int col0 = 0, int from = 0, int count = -1) { put_rows(img, dtype, K, *t, row0, step, col0, from, count); }
     int32_t load(ForgeModel* m, DenseWeight* w, bool row_reads = false) const { return load_dense(m, w, N, K, dtype, img, row_reads); }
 };
 
@@ -151,6 +162,10 @@ int32_t load_norm(ForgeModel* m, StreamNorm* n, const TensorSet& t, const std::s
         std::vector<float> w(size_t(t.at(name)->count()));
         for (size_t i = 0; i < w.size(); ++i) w[i] = 1.f + t.at(name)->at(i);
         return upload_values(m, &n->w, w);
+    }
+    if (m->stack->spec.arch->norm == Norm::RmsScalar) {
+        n->alpha = t.at(name)->at(0);
+        return upload_values(m, &n->w, std::vector<float>(size_t(m->stack->spec.width), n->alpha));
     }
     n->alpha = t.at(name + ".alpha")->at(0);
     FORGE_TRY(upload_f32(m, &n->w, *t.at(name)));
@@ -315,6 +330,106 @@ int32_t load_softmax(ForgeModel* m, const LayerSpec& L, const TensorSet& t, Laye
     });
 }
 
+// What the mechanisms of an attention behind `at` need besides its matrices; norms of queries and keys without weights.
+int32_t load_plain_attention(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w, const std::string& at, float factor) {
+    const AttnDims& a = L.attn;
+    const std::vector<float> ones(size_t(a.dim), 1.f);
+    FORGE_TRY(upload_values(m, &w->q_norm, ones));
+    w->k_norm = w->q_norm;
+    FORGE_TRY(upload_f32(m, &w->q_bias, *t.at(at + "q.b")));
+    FORGE_TRY(upload_f32(m, &w->k_bias, *t.at(at + "k.b")));
+    FORGE_TRY(upload_f32(m, &w->v_bias, *t.at(at + "v.b")));
+    std::vector<float> ob;
+    for (int64_t i = 0; i < t.at(at + "o.b")->count(); ++i) ob.push_back(factor * t.at(at + "o.b")->at(size_t(i)));
+    FORGE_TRY(upload_values(m, &w->out_bias, ob));
+    if (L.soft.sink) FORGE_TRY(upload_f32(m, &w->sink, *t.at(at + "sink")));
+    if (L.soft.talk) FORGE_TRY(upload_f32(m, &w->talk, *t.at(at + "talk")));
+    if (L.soft.distance) {
+        std::vector<float> by;   // [head][distance]
+        for (int h = 0; h < a.heads; ++h)
+            for (int n = 0; n < a.bias_n; ++n) by.push_back(t.at(at + "rel")->at(size_t(L.distance.of(n)) * a.heads + h));
+        FORGE_TRY(upload_values(m, &w->bias, by));
+    }
+    if (L.blend_layer >= 0) w->lambda = t.at(at + "vmix")->at(0);
+    return FORGE_OK;
+}
+
+int32_t load_post_softmax(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
+    StackModel& S = *m->stack;
+    const AttnDims& a = L.attn;
+    FORGE_TRY(load_plain_attention(m, L, t, w, "mix.", 1.f));
+    w->k_row = pad_to(a.heads * a.dim, kSegAlign);
+    w->v_row = w->k_row + pad_to(a.groups * a.dim, kSegAlign);
+    Image in(w->v_row + a.groups * a.vdim, S.width_p, S.dtype), out(S.spec.width, pad_to(a.heads * a.vdim, kDensePad), S.dtype);
+    in.put(t.at("mix.q"), 0); in.put(t.at("mix.k"), w->k_row); in.put(t.at("mix.v"), w->v_row);
+    out.put(t.at("mix.o"), 0);
+    FORGE_TRY(in.load(m, &w->in));
+    return out.load(m, &w->out);
+}
+
+int32_t load_attn_selective(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
+    StackModel& S = *m->stack;
+    const AttnDims& a = L.attn;
+    const SelectiveDims& d = L.sel;
+    FORGE_TRY(load_plain_attention(m, L, t, w, "mix.left.", L.left_scale));
+    w->k_row = pad_to(a.heads * a.dim, kSegAlign);
+    w->v_row = w->k_row + pad_to(a.groups * a.dim, kSegAlign);
+    w->in_row = w->v_row + pad_to(a.groups * a.vdim, kSegAlign);
+    w->gate_row = w->in_row + pad_to(d.inner, kSegAlign);
+    Image in(w->gate_row + d.inner, S.width_p, S.dtype);
+    in.put(t.at("mix.left.q"), 0); in.put(t.at("mix.left.k"), w->k_row); in.put(t.at("mix.left.v"), w->v_row);
+    in.put(t.at("mix.right.in"), w->in_row, 1, 0, 0, d.inner);
+    in.put(t.at("mix.right.in"), w->gate_row, 1, 0, d.inner, d.inner);
+    FORGE_TRY(in.load(m, &w->in));
+    const int inner_p = pad_to(d.inner, kDensePad);
+    w->bc_row = pad_to(d.rank, kSegAlign);
+    Image x(w->bc_row + 2 * d.state, inner_p, S.dtype);
+    x.put(t.at("mix.right.x"), 0, 1, 0, 0, d.rank);
+    x.put(t.at("mix.right.x"), w->bc_row, 1, 0, d.rank, 2 * d.state);
+    FORGE_TRY(x.load(m, &w->scan_in));
+    Image low(d.inner, pad_to(d.rank, kDensePad), S.dtype);
+    low.put(t.at("mix.right.dt"), 0);
+    FORGE_TRY(low.load(m, &w->low, true));
+    w->heads_k = pad_to(a.heads * a.vdim, kDensePad);
+    Image out(S.spec.width, w->heads_k + inner_p, S.dtype);
+    out.put(t.at("mix.left.o"), 0);
+    out.put(t.at("mix.right.o"), 0, 1, w->heads_k);
+    FORGE_TRY(out.load(m, &w->out));
+    std::vector<float> conv, a2;   // [taps][channels]; decays are exp2(step size * a2)
+    for (int j = 0; j < d.taps; ++j) for (int c = 0; c < d.inner; ++c) conv.push_back(t.at("mix.right.conv")->at(size_t(c) * d.taps + j));
+    for (size_t i = 0; i < d.state_values(); ++i) a2.push_back(float(-std::exp(double(t.at("mix.right.A_log")->at(i))) / std::log(2.0)));
+    FORGE_TRY(upload_values(m, &w->conv, conv));
+    FORGE_TRY(upload_values(m, &w->scan_a, a2));
+    FORGE_TRY(upload_values(m, &w->minus, std::vector<float>(size_t(d.inner), -1.f)));
+    FORGE_TRY(upload_f32(m, &w->conv_add, *t.at("mix.right.conv.b")));
+    FORGE_TRY(upload_f32(m, &w->decay_add, *t.at("mix.right.dt.b")));
+    return upload_f32(m, &w->skip, *t.at("mix.right.D"));
+}
+
+// A mixture beside a shared expert: [shared gate, up | router] and, over [shared | expert 0 | expert 1 ...], the way back.
+int32_t load_mixture(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
+    StackModel& S = *m->stack;
+    const int E = L.router.experts, shared_k = pad_to(L.shared_ff, kDensePad);
+    w->router_row = pad_to(2 * L.shared_ff, kSegAlign);
+    Image in(w->router_row + L.router.choices(), S.width_p, S.dtype);
+    in.put(t.at("mlp.shared.gate"), 0, 2); in.put(t.at("mlp.shared.up"), 1, 2);
+    in.put(t.at("mlp.router"), w->router_row);
+    FORGE_TRY(in.load(m, &w->ff_in));
+    w->ff_k = pad_to(L.ff, kDensePad);
+    w->expert_rows = pad_to(2 * L.ff, 128);
+    Image ex(E * w->expert_rows, S.width_p, S.dtype), out(S.spec.width, shared_k + E * w->ff_k, S.dtype);
+    out.put(t.at("mlp.shared.down"), 0);
+    for (int e = 0; e < E; ++e) {
+        const std::string x = "mlp.e" + std::to_string(e);
+        ex.put(t.at(x + ".gate"), e * w->expert_rows, 2);
+        ex.put(t.at(x + ".up"), e * w->expert_rows + 1, 2);
+        out.put(t.at(x + ".down"), 0, 1, shared_k + e * w->ff_k);
+    }
+    FORGE_TRY(ex.load(m, &w->experts));
+    FORGE_TRY(out.load(m, &w->ff_out));
+    return upload_f32(m, &w->router_bias, *t.at("mlp.correction"));
+}
+
 int32_t load_linear(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
     StackModel& S = *m->stack;
     const RecurDims& d = L.rec;
@@ -339,13 +454,19 @@ int32_t load_linear(ForgeModel* m, const LayerSpec& L, const TensorSet& t, Layer
 
 int32_t load_layer(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
     StackModel& S = *m->stack;
+    const bool post = S.spec.arch->arrangement == Arrangement::PostNorm;
     FORGE_TRY(load_norm(m, &w->norm1, t, "norm1"));
     switch (L.kind) {
         case Mixer::Latent: FORGE_TRY(load_latent(m, L, t, w)); break;
         case Mixer::Delta: case Mixer::ChannelDelta: FORGE_TRY(load_delta(m, L, t, w)); break;
         case Mixer::AttnTimeMix: FORGE_TRY(load_pair(m, L, t, w)); break;
-        case Mixer::Softmax: FORGE_TRY(load_softmax(m, L, t, w)); break;
+        case Mixer::Softmax: FORGE_TRY(post ? load_post_softmax(m, L, t, w) : load_softmax(m, L, t, w)); break;
         case Mixer::GatedLinear: FORGE_TRY(load_linear(m, L, t, w)); break;
+        case Mixer::AttnSelective: FORGE_TRY(load_attn_selective(m, L, t, w)); break;
+    }
+    if (L.ff && post) {
+        FORGE_TRY(load_norm(m, &w->norm2, t, "norm2"));
+        FORGE_TRY(load_mixture(m, L, t, w));
     }
     if (L.ff && S.spec.arch->arrangement == Arrangement::ParallelTwo) FORGE_TRY(load_norm(m, &w->norm2, t, "norm2"));
     if (L.ff && S.spec.arch->arrangement == Arrangement::Sequential) {
@@ -400,9 +521,14 @@ int32_t grow(ForgeModel* m, StackModel::Buf& b, size_t bytes) {
 bool tensor_core_rows(const StackModel& S, const LatentDims& d) { return S.dtype == FORGE_BF16 && latent_decode_tc_supported(d); }
 
 // A step of few tokens runs an expert over all of them and takes the experts' columns of `out` from a list; otherwise tokens are dealt to the experts.
-bool few_tokens(const StackModel& S, const LayerWeights& w, int rows) { return dense_listed_supported(w.out, rows); }
+bool few_tokens(const StackModel& S, const LayerWeights& w, int rows) { return dense_listed_supported(S.spec.arch->arrangement == Arrangement::PostNorm ? w.ff_out : w.out, rows); }
 // values of a row in front of `out`
-int mid_columns(const StackModel& S, const LayerSpec& L, const LayerWeights& w, int rows) { return L.router.experts && !few_tokens(S, w, rows) ? w.heads_k : w.out.K; }
+int mid_columns(const StackModel& S, const LayerSpec& L, const LayerWeights& w, int rows) {
+    return L.router.experts && S.spec.arch->arrangement == Arrangement::ParallelTwo && !few_tokens(S, w, rows) ? w.heads_k : w.out.K;
+}
+// the same in front of a mixture's way back
+int shared_columns(const LayerSpec& L) { return pad_to(L.shared_ff, kDensePad); }
+constexpr size_t kScoreBytes = size_t(256) << 20;   // scores of rows with mixed heads, at most, if rows may go in turn
 
 // splits of the row attention: at most one CTA per SM over all rows and head groups, no more than there are pages
 int row_splits(const StackModel& S, int rows, int pages) {
@@ -411,30 +537,47 @@ int row_splits(const StackModel& S, int rows, int pages) {
     return std::max(1, std::min(pages, 148 / std::max(1, rows * groups)));
 }
 
-int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt, int ctx_rows, int seg_rows, int chunks) {
+// block_rows: rows of gathered blocks; all_at_once: no row waits for its turn
+int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt, int ctx_rows, int seg_rows, int chunks, int max_keys, int block_rows, bool all_at_once) {
     StackModel& S = *m->stack;
     const size_t es = dense_size(S.dtype), r = size_t(rows), W = size_t(S.spec.width), WP = size_t(S.width_p);
     // bytes, rows times the widest layer
-    size_t h = WP * es, proj = 0, gate = 0, mid = 0, q = 0, part = 0, heads = 0, cc = 0, cr = 0, ck = 0, cv = 0, hgate = 0, decay = 0, beta = 0, low = 0, conv = 0, unit = 0, o = 0, pair = 0, router = 0, route = 0, e_in = 0, e_act = 0, e_out = 0;
+    size_t h = WP * es, proj = 0, gate = 0, mid = 0, q = 0, part = 0, heads = 0, cc = 0, cr = 0, ck = 0, cv = 0, hgate = 0, decay = 0, beta = 0, low = 0, conv = 0, unit = 0, o = 0, pair = 0, router = 0, route = 0, e_in = 0, e_act = 0, e_out = 0, scores = 0, joint = 0, blocks = 0, scan = 0, bc = 0;
     ChunkBytes cb{0, 0};
     auto most = [](size_t& a, size_t b) { a = std::max(a, b); };
     size_t n_max = size_t(S.head.N);
     for (size_t i = 0; i < S.spec.layers.size(); ++i) {
         const LayerSpec& L = S.spec.layers[i];
         const LayerWeights& w = S.weights(int(i));
-        for (const DenseWeight* d : {&w.in, &w.out, &w.kv, &w.low, &w.ff_in, &w.ff_out}) most(n_max, size_t(d->N));
-        most(mid, r * std::max(mid_columns(S, L, w, rows), w.ff_out.K) * es);
+        for (const DenseWeight* d : {&w.in, &w.out, &w.kv, &w.low, &w.scan_in, &w.ff_in, &w.ff_out}) most(n_max, size_t(d->N));
+        most(mid, r * std::max(mid_columns(S, L, w, rows), S.spec.arch->arrangement == Arrangement::PostNorm ? shared_columns(L) : w.ff_out.K) * es);
+        if (S.spec.arch->arrangement == Arrangement::PostNorm) most(pair, r * W * 4);
         if (S.spec.arch->arrangement == Arrangement::ParallelTwo) most(h, 2 * WP * es);
         if (L.router.experts) {
             const size_t pairs = r * L.router.top;
-            most(mid, std::min<size_t>(r, kScaleRows) * w.out.K * es);
-            most(router, r * L.router.experts * 4);
+            most(mid, std::min<size_t>(r, kScaleRows) * std::max(w.out.K, w.ff_out.K) * es);
+            most(router, r * L.router.choices() * 4);
             most(route, route_bytes(L.router, rows));
             if (!few_tokens(S, w, rows)) { most(e_in, pairs * WP * es); most(e_act, pairs * w.ff_k * es); most(e_out, pairs * W * 4); }
         }
-        if (L.kind == Mixer::Softmax) {
+        if (L.kind == Mixer::Softmax || L.kind == Mixer::AttnSelective) {
+            const AttnDims& a = L.attn;
             most(proj, r * w.v_row * 4);
-            most(q, r * L.attn.heads * L.attn.dim_p * es);
+            most(q, r * a.heads * a.dim_p * es);
+            if (L.soft.talk && single) {
+                const size_t one = talk_rows_bytes(a, 1, a.most_keys(max_keys));
+                most(scores, all_at_once ? one * single : std::max(one, std::min(one * single, kScoreBytes)));
+            }
+            if (L.soft.talk) most(joint, size_t(prompt) * a.heads * a.groups * a.vdim_p * es);
+            if (a.pool) most(blocks, size_t(block_rows) * a.row() * es);
+            if (L.kind == Mixer::AttnSelective) {
+                const SelectiveDims& d = L.sel;
+                most(scan, r * 2 * w.scan_in.K * es);
+                most(gate, r * d.inner * es);
+                most(bc, r * 2 * d.state * 4);
+                most(low, r * w.low.K * es);
+                most(decay, r * d.inner * 4);
+            }
             continue;
         }
         if (L.has_latent()) {
@@ -473,11 +616,12 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
     FORGE_TRY(grow(m, S.h, r * h));
     if (S.loop_in.N) FORGE_TRY(grow(m, S.cat, r * 2 * WP * es));
     if (S.spec.adds_loop()) FORGE_TRY(grow(m, S.x0, r * W * 4));
-    if (S.spec.arch->norm == Norm::RmsPlusOne) { FORGE_TRY(grow(m, S.sums, r * scale_parts(int(W)) * 4)); FORGE_TRY(grow(m, S.sum1, r * 4)); }
+    if (S.rms_final()) { FORGE_TRY(grow(m, S.sums, r * scale_parts(int(W)) * 4)); FORGE_TRY(grow(m, S.sum1, r * 4)); }
     FORGE_TRY(grow(m, S.place, r * sizeof(int32_t)));
     const std::pair<StackModel::Buf*, size_t> sizes[] = {{&S.proj, proj}, {&S.gate, gate}, {&S.mid, mid}, {&S.q, q}, {&S.part, part}, {&S.ml, heads}, {&S.hgate, hgate}, {&S.decay, decay},
         {&S.beta, beta}, {&S.low, low}, {&S.conv, conv}, {&S.unit, unit}, {&S.o, o}, {&S.pair, pair}, {&S.c_half, cb.half}, {&S.c_f32, cb.f32}, {&S.ctx_c, cc}, {&S.ctx_r, cr}, {&S.ctx_k, ck}, {&S.ctx_v, cv},
-        {&S.router, router}, {&S.route, route}, {&S.e_in, e_in}, {&S.e_act, e_act}, {&S.e_out, e_out}};
+        {&S.router, router}, {&S.route, route}, {&S.e_in, e_in}, {&S.e_act, e_act}, {&S.e_out, e_out},
+        {&S.scores, scores}, {&S.joint, joint}, {&S.blocks, blocks}, {&S.scan, scan}, {&S.bc, bc}};
     for (const auto& e : sizes) FORGE_TRY(grow(m, *e.first, e.second));
     // one ticket per output tile of the largest product (128 rows x at least 16 tokens)
     const size_t tiles = ((n_max + 127) / 128) * std::max<size_t>(1, (size_t(std::max(rows, ctx_rows)) + 127) / 128);
@@ -501,6 +645,7 @@ struct Step {
     const PromptTile* tiles = nullptr; int n_tiles = 0;
     const PromptTile* host_tiles = nullptr;
     const int32_t* ctx_pages = nullptr; int ctx_rows = 0;
+    const PoolChunk* chunks = nullptr; int n_chunks = 0;   // of the prompts' blocks
     uint32_t* hist = nullptr; const int32_t* step = nullptr;
     float* trace = nullptr; size_t trace_stride = 0;
 };
@@ -510,7 +655,7 @@ char* at(void* p, size_t elems, int dtype) { return static_cast<char*>(p) + elem
 // the scales of an RMS norm's tokens
 RowScale stream_scale(const StackModel& S, int rows) {
     RowScale r;
-    if (S.spec.arch->norm != Norm::RmsPlusOne) return r;
+    if (!S.rms_final()) return r;
     const bool summed = rows > kScaleRows;
     r.sums = static_cast<const float*>(summed ? S.sum1.p : S.sums.p);
     r.parts = summed ? 1 : scale_parts(S.spec.width);
@@ -526,10 +671,10 @@ struct Sequence {
     StackModel& S;
     cudaStream_t st;
     const int n, W, WP, dt;
-    const bool sequential, two_norms;
+    const bool sequential, two_norms, post;
     Sequence(ForgeModel* m_, ForgeKV* kv_, const Step& s_)
         : m(m_), kv(kv_), s(s_), S(*m_->stack), st(m_->stream), n(s_.rows.n), W(S.spec.width), WP(S.width_p), dt(S.dtype), sequential(S.spec.arch->arrangement == Arrangement::Sequential),
-          two_norms(S.spec.arch->arrangement == Arrangement::ParallelTwo) {}
+          two_norms(S.spec.arch->arrangement == Arrangement::ParallelTwo), post(S.spec.arch->arrangement == Arrangement::PostNorm) {}
 
     int32_t gemm(const DenseWeight& w, const void* act, int ld, const DenseOut& o, int rows) { return dense_gemm(w, act, ld, rows, o, S.scratch, m->d_err, st); }
     int32_t gemm(const DenseWeight& w, const void* act, int ld, const DenseOut& o) { return gemm(w, act, ld, o, n); }
@@ -537,15 +682,21 @@ struct Sequence {
     After norm(const StreamNorm& d, int ld) {
         After a;
         a.dst = S.h.p; a.ld = ld; a.w = d.w;
-        if (rms()) { a.kind = AFTER_RMS; a.sums = static_cast<float*>(S.sums.p); a.parts = scale_parts(W); }
+        if (S.rms_final()) { a.kind = AFTER_RMS; a.sums = static_cast<float*>(S.sums.p); a.parts = scale_parts(W); }
         else { a.kind = AFTER_DYT; a.alpha = d.alpha; a.b = d.b; }
         return a;
     }
-    bool rms() const { return S.spec.arch->norm == Norm::RmsPlusOne; }
     int h_ld(int layer) const { return S.spec.layers[layer].kind == Mixer::AttnTimeMix ? (1 + kMixes) * WP : two_norms ? 2 * WP : WP; }
     After norm1(int layer) {
+        if (post) return stream();
         After a = norm(S.weights(layer).norm1, h_ld(layer));
         if (two_norms && S.spec.layers[layer].ff) { a.w2 = S.weights(layer).norm2.w; a.col2 = WP; }
+        return a;
+    }
+    // the stream itself
+    After stream() {
+        After a;
+        a.kind = AFTER_CAST; a.dst = S.h.p; a.ld = WP;
         return a;
     }
     // what the first reader of the stream in front of run i takes
@@ -567,8 +718,8 @@ struct Sequence {
     static void resid(DenseOut* o, float* x, int W, const After& after) { o->add(SEG_RESID, 0, W, x, W).after = after; }
     float* x() { return static_cast<float*>(S.x.p); }
     // RMS norms: the tokens' scales from the sums that the stream's last writer left
-    int32_t stats() { return rms() && s.scale_rows > kScaleRows ? row_sums(static_cast<float*>(S.sum1.p), static_cast<float*>(S.sums.p), n, scale_parts(W), st) : FORGE_OK; }
-    RowScale scale() const { return stream_scale(S, s.scale_rows); }
+    int32_t stats(bool last) { return (last ? S.rms_final() : S.rms_stream()) && s.scale_rows > kScaleRows ? row_sums(static_cast<float*>(S.sum1.p), static_cast<float*>(S.sums.p), n, scale_parts(W), st) : FORGE_OK; }
+    RowScale scale() const { return S.rms_stream() ? stream_scale(S, s.scale_rows) : RowScale{}; }
 
     int32_t run() {
         EmbedArgs e;
@@ -596,15 +747,17 @@ struct Sequence {
                 FORGE_TRY(gemm(S.loop_in, S.cat.p, 2 * WP, o));
             }
             const bool ff = sequential && L.ff;
-            const After after = ff ? norm(w.norm2, WP) : into(i + 1);
-            FORGE_TRY(stats());
+            const After after = ff ? norm(w.norm2, WP) : post && L.ff ? stream() : into(i + 1);
+            FORGE_TRY(stats(false));
             switch (L.kind) {
                 case Mixer::Latent: FORGE_TRY(latent(L, w, run, after)); break;
                 case Mixer::Delta: case Mixer::ChannelDelta: FORGE_TRY(delta(L, w, run, after)); break;
                 case Mixer::AttnTimeMix: FORGE_TRY(pair(L, w, run, after)); break;
                 case Mixer::Softmax: FORGE_TRY(softmax(L, w, run, after)); break;
                 case Mixer::GatedLinear: FORGE_TRY(linear(L, w, run, after)); break;
+                case Mixer::AttnSelective: FORGE_TRY(attn_selective(L, w, run, after)); break;
             }
+            if (post && L.ff) FORGE_TRY(mixture(L, w, into(i + 1)));
             if (ff) {
                 DenseOut in, out;
                 in.add(S.spec.arch->dense == Mlp::ClampedGlu ? SEG_CLAMPED_GLU : SEG_SILU_GLU, 0, 2 * L.ff, S.mid.p, w.ff_out.K).limit = L.limit;
@@ -614,7 +767,7 @@ struct Sequence {
             }
             if (s.trace && !after.keep) FORGE_CUDA(cudaMemcpyAsync(s.trace + i * s.trace_stride, S.x.p, sizeof(float) * n * W, cudaMemcpyDeviceToDevice, st));
         }
-        return stats();
+        return stats(true);
     }
 
     int32_t latent(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
@@ -739,37 +892,169 @@ struct Sequence {
         return add_experts(x(), static_cast<const float*>(S.e_out.p), L.router, t, n, W, after, dt, st);
     }
 
-    int32_t softmax(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
+    // rows of `in` of queries, keys and values
+    void qkv_rows(DenseOut* o, const LayerSpec& L, const LayerWeights& w, StackCache::Run& run) {
         const AttnDims& a = L.attn;
-        const int ldp = w.v_row, mid_ld = mid_columns(S, L, w, n);
         float* proj = static_cast<float*>(S.proj.p);
-        const int32_t* place = static_cast<const int32_t*>(S.place.p);
-        {
-            DenseOut o;
-            o.scale = scale();
-            o.add(SEG_F32, 0, a.heads * a.dim, proj, ldp).add = w.q_bias;
-            o.add(SEG_F32, w.k_row, a.groups * a.dim, proj + w.k_row, ldp).add = w.k_bias;
-            OutSeg& v = o.add(SEG_CAST, w.v_row, a.groups * a.vdim, at(run.pool, size_t(a.groups) * a.dim_p, dt), a.row());
-            v.group = a.vdim; v.group_ld = a.vdim_p; v.place = place; v.add = w.v_bias;
-            feed_forward_rows(&o, L, w);
-            FORGE_TRY(gemm(w.in, S.h.p, 2 * WP, o));
+        o->add(SEG_F32, 0, a.heads * a.dim, proj, w.v_row).add = w.q_bias;
+        o->add(SEG_F32, w.k_row, a.groups * a.dim, proj + w.k_row, w.v_row).add = w.k_bias;
+        OutSeg& v = o->add(SEG_CAST, w.v_row, a.groups * a.vdim, at(run.pool, size_t(a.groups) * a.dim_p, dt), a.row());
+        v.group = a.vdim; v.group_ld = a.vdim_p; v.place = static_cast<const int32_t*>(S.place.p); v.add = w.v_bias;
+        if (L.blend_layer >= 0) {   // the lender's values lie in its cache rows
+            const AttnDims& b = S.spec.layers[L.blend_layer].attn;
+            v.blend = at(lender(L.blend_layer).pool, size_t(b.groups) * b.dim_p, dt); v.blend_ld = b.row();
+            v.own = 1.f - w.lambda; v.other = w.lambda;
         }
-        const bool routed = L.router.experts && few_tokens(S, w, n);
-        const RouteBeside route{L.router, static_cast<const float*>(S.router.p), route_tables(S.route.p, L.router, n)};
-        FORGE_TRY(qk_post(a, L.soft.qk, dt, proj, ldp, w.k_row, w.q_norm, w.k_norm, S.ropes.at(L.rot).second, S.q.p, run.pool, place, s.rows, routed ? &route : nullptr, st));
+    }
+    StackCache::Run& lender(int layer) {
+        size_t i = 0;
+        while (S.spec.runs[i].layer != layer) ++i;
+        return kv->stack->runs[i];
+    }
+    // norms, rotation, attention of all rows of the step: factor * heads to the first columns of mid
+    int32_t attend(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, int mid_ld, float factor, const RouteBeside* route) {
+        AttnDims a = L.attn;
+        a.pool_row0 = kv->num_pages * FORGE_KV_PAGE;
+        const int32_t* place = static_cast<const int32_t*>(S.place.p);
+        FORGE_TRY(qk_post(a, L.soft.qk, dt, static_cast<const float*>(S.proj.p), w.v_row, w.k_row, w.q_norm, w.k_norm, S.ropes.at(L.rot).second, S.q.p, run.pool, place, s.rows, route, st));
+        if (a.pool) FORGE_TRY(pool_blocks(a, dt, run.pool, s.rows, st));
         StepRows single = s.rows;
         single.n = s.single;
-        FORGE_TRY(attn_rows(a, dt, S.q.p, run.pool, nullptr, w.sink, S.mid.p, mid_ld, single, a.most_keys(s.max_keys), st));
-        if (n > s.single) {
-            PromptAttnArgs p;
-            p.q = at(S.q.p, size_t(s.single) * a.heads * a.dim_p, dt); p.k = run.pool; p.v = at(run.pool, size_t(a.groups) * a.dim_p, dt);
-            p.sink = w.sink;
-            p.out = at(S.mid.p, size_t(s.single) * mid_ld, dt); p.out_ld = mid_ld;
-            p.q_rows = n - s.single; p.ctx_rows = kv->num_pages * FORGE_KV_PAGE; p.tiles = s.tiles; p.n_tiles = s.n_tiles; p.host_tiles = s.host_tiles;
-            p.pages = s.ctx_pages; p.page_row = a.row(); p.err = m->d_err;
-            FORGE_TRY(attn_prefill_kv(PromptDims(a), p, st));
+        const int max_keys = a.most_keys(s.max_keys), np = n - s.single;
+        if (L.soft.talk) FORGE_TRY(talk_rows(a, dt, S.q.p, run.pool, w.talk, factor, S.scores.p, S.scores.cap, S.mid.p, mid_ld, single, max_keys, st));
+        else FORGE_TRY(attn_rows(a, dt, S.q.p, run.pool, nullptr, w.sink, w.bias, S.mid.p, mid_ld, single, max_keys, st));
+        if (np <= 0) return FORGE_OK;
+        void* out = at(S.mid.p, size_t(s.single) * mid_ld, dt);
+        PromptDims d(a);
+        PromptAttnArgs p;
+        p.q = at(S.q.p, size_t(s.single) * a.heads * a.dim_p, dt); p.k = run.pool; p.v = at(run.pool, size_t(a.groups) * a.dim_p, dt);
+        p.sink = w.sink; p.bias = w.bias;
+        p.out = out; p.out_ld = mid_ld;
+        p.q_rows = np; p.ctx_rows = kv->num_pages * FORGE_KV_PAGE; p.tiles = s.tiles; p.n_tiles = s.n_tiles; p.host_tiles = s.host_tiles;
+        p.pages = s.ctx_pages; p.page_row = a.row(); p.err = m->d_err;
+        if (a.pool) {
+            FORGE_TRY(gather_blocks(a, dt, S.blocks.p, run.pool, s.ctx_pages, s.chunks, s.n_chunks, st));
+            p.blocks = S.blocks.p; p.block_rows = s.n_chunks * FORGE_KV_PAGE;
         }
+        if (!L.soft.talk) return attn_prefill_kv(d, p, st);
+        d.joint = true;
+        p.out = S.joint.p; p.out_ld = a.heads * a.groups * a.vdim_p;
+        FORGE_TRY(attn_prefill_kv(d, p, st));
+        return talk_heads(a, S.joint.p, w.talk, factor, out, mid_ld, np, st);
+    }
+
+    int32_t softmax(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
+        DenseOut o;
+        qkv_rows(&o, L, w, run);
+        if (post) {
+            FORGE_TRY(gemm(w.in, S.h.p, WP, o));
+            FORGE_TRY(attend(L, w, run, w.out.K, 1.f, nullptr));
+            return post_out(w, after);
+        }
+        o.scale = scale();
+        feed_forward_rows(&o, L, w);
+        FORGE_TRY(gemm(w.in, S.h.p, 2 * WP, o));
+        const bool routed = L.router.experts && few_tokens(S, w, n);
+        const RouteBeside route{L.router, static_cast<const float*>(S.router.p), route_tables(S.route.p, L.router, n)};
+        FORGE_TRY(attend(L, w, run, mid_columns(S, L, w, n), 1.f, routed ? &route : nullptr));
         return two_norms_out(L, w, after, routed);
+    }
+
+    // x += norm1(W_o mid)
+    int32_t post_out(const LayerWeights& w, const After& after) {
+        DenseOut o;
+        o.add(SEG_F32, 0, W, S.pair.p, W).add = w.out_bias;
+        FORGE_TRY(gemm(w.out, S.mid.p, w.out.K, o));
+        return add_normed(x(), static_cast<const float*>(S.pair.p), n, W, S.spec.eps, w.norm1.alpha, MixtureSum{}, after, dt, st);
+    }
+
+    int32_t attn_selective(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
+        const SelectiveDims& d = L.sel;
+        const int inner_p = w.scan_in.K;
+        void *in = S.scan.p, *xc = at(S.scan.p, size_t(n) * pad_to(d.inner, kDensePad), dt);   // rows [inner], then padded ones
+        {
+            DenseOut o;
+            qkv_rows(&o, L, w, run);
+            o.add(SEG_CAST, w.in_row, d.inner, in, d.inner);
+            o.add(SEG_SILU, w.gate_row, d.inner, S.gate.p, d.inner);
+            FORGE_TRY(gemm(w.in, S.h.p, WP, o));
+        }
+        SelectiveArgs a;
+        a.in = in; a.in_ld = d.inner; a.conv = w.conv; a.conv_add = w.conv_add; a.ring = run.ring;
+        a.x = xc; a.x_ld = inner_p;
+        a.bc = static_cast<const float*>(S.bc.p); a.bc_ld = 2 * d.state;
+        a.a2 = w.scan_a; a.skip = w.skip; a.state = run.state;
+        a.gate = S.gate.p; a.gate_ld = d.inner; a.factor = L.right_scale;
+        a.out = at(S.mid.p, w.heads_k, dt); a.out_ld = w.out.K;
+        StepRows ones = s.rows;
+        ones.n = s.ones;
+        FORGE_TRY(selective_conv(d, dt, a, ones, s.segs, st));
+        {
+            DenseOut o;
+            o.add(SEG_CAST, 0, d.rank, S.low.p, w.low.K);
+            o.add(SEG_F32, w.bc_row, 2 * d.state, S.bc.p, 2 * d.state);
+            FORGE_TRY(gemm(w.scan_in, xc, inner_p, o));
+        }
+        if (all_ones() && n <= kFewSteps) {
+            a.dt_w = w.low.w; a.low = S.low.p; a.low_ld = a.low_k = w.low.K; a.dt_add = w.decay_add;
+        } else {   // softplus: the epilogue of decays with a factor of minus one
+            DenseOut o;
+            OutSeg& g = o.add(SEG_DECAY, 0, d.inner, S.decay.p, d.inner);
+            g.mul = w.minus; g.add = w.decay_add;
+            FORGE_TRY(gemm(w.low, S.low.p, w.low.K, o));
+            a.dt = static_cast<const float*>(S.decay.p); a.dt_ld = d.inner;
+        }
+        FORGE_TRY(selective_decode(d, dt, a, ones, st));
+        FORGE_TRY(selective_segments(d, dt, a, s.segs, st));
+        FORGE_TRY(attend(L, w, run, w.out.K, L.left_scale, nullptr));
+        return post_out(w, after);
+    }
+    static constexpr int kFewSteps = 4;   // single tokens whose step sizes are formed inside the recurrence
+
+    // x += norm2(shared expert + experts + what is passed on); see experts() for few and many tokens
+    int32_t mixture(const LayerSpec& L, const LayerWeights& w, const After& after) {
+        RouterDims r = L.router;
+        r.correction = w.router_bias;
+        const bool few = few_tokens(S, w, n);
+        const int shared_k = shared_columns(L), mid_ld = few ? w.ff_out.K : shared_k;
+        const RouteTables t = route_tables(S.route.p, r, n);
+        const float* logits = static_cast<const float*>(S.router.p);
+        float* y = static_cast<float*>(S.pair.p);
+        MixtureSum sum;
+        if (r.identity) sum.passed = t.passed;
+        {
+            DenseOut o;
+            o.add(SEG_SILU_GLU, 0, 2 * L.shared_ff, S.mid.p, mid_ld);
+            o.add(SEG_F32, w.router_row, r.choices(), S.router.p, r.choices());
+            FORGE_TRY(gemm(w.ff_in, S.h.p, WP, o));
+        }
+        GroupTable table;
+        GroupShape shape;
+        shape.rows = 2 * L.ff; shape.group_rows = w.expert_rows;
+        DenseOut in, out;
+        out.add(SEG_F32, 0, W, y, W);
+        if (few) {
+            FORGE_TRY(route_few(r, logits, n, t, &table, st));
+            shape.group_dst = size_t(w.ff_k);
+            in.add(SEG_SILU_GLU, 0, 2 * L.ff, at(S.mid.p, shared_k, dt), mid_ld);
+            FORGE_TRY(dense_gemm_groups(w.experts, shape, table, S.h.p, WP, n, in, m->d_err, st));
+            FORGE_TRY(dense_gemm_listed(w.ff_out, shared_k, w.ff_k, table, S.mid.p, mid_ld, n, out, m->d_err, st));
+            return add_normed(x(), y, n, W, S.spec.eps, w.norm2.alpha, sum, after, dt, st);
+        }
+        FORGE_TRY(gemm(w.ff_out.columns(0, shared_k), S.mid.p, mid_ld, out));
+        FORGE_TRY(route_slots(r, logits, n, t, &table, st));
+        const int pairs = n * r.top;
+        FORGE_TRY(gather_act_rows(S.e_in.p, S.h.p, WP, t.row, pairs, WP, dt, st));
+        in.add(SEG_SILU_GLU, 0, 2 * L.ff, S.e_act.p, w.ff_k);
+        FORGE_TRY(dense_gemm_groups(w.experts, shape, table, S.e_in.p, WP, pairs, in, m->d_err, st));
+        DenseOut down;
+        down.add(SEG_F32, 0, W, S.e_out.p, W);
+        GroupShape cols;
+        cols.rows = W; cols.group_cols = w.ff_k;
+        table.weight = nullptr;
+        FORGE_TRY(dense_gemm_groups(w.ff_out.columns(shared_k, w.ff_k), cols, table, S.e_act.p, w.ff_k, pairs, down, m->d_err, st));
+        sum.e = static_cast<const float*>(S.e_out.p); sum.slot = t.slot; sum.top = r.top;
+        return add_normed(x(), y, n, W, S.spec.eps, w.norm2.alpha, sum, after, dt, st);
     }
 
     int32_t linear(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
@@ -872,7 +1157,7 @@ struct Sequence {
         }
         StepRows single = s.rows;
         single.n = s.single;
-        FORGE_TRY(attn_rows(t, dt, S.q.p, run.pool, hgate, nullptr, S.mid.p, mid_ld, single, t.most_keys(s.max_keys), st));
+        FORGE_TRY(attn_rows(t, dt, S.q.p, run.pool, hgate, nullptr, nullptr, S.mid.p, mid_ld, single, t.most_keys(s.max_keys), st));
         const int np = n - s.single;
         if (np > 0) {
             PromptAttnArgs p;
@@ -922,8 +1207,8 @@ void stack_destroy(ForgeModel* m) {
 }
 
 // ------------------------------------------------------------------------------------------------ cache
-static size_t state_bytes(const LayerSpec& L) { return L.has_state() ? L.rec.state_values() * 4 : 0; }
-static size_t ring_bytes(const StackModel& S, const LayerSpec& L) { return L.has_state() ? L.rec.ring_values() * dense_size(S.dtype) : 0; }
+static size_t state_bytes(const LayerSpec& L) { return L.state_values() * 4; }
+static size_t ring_bytes(const StackModel& S, const LayerSpec& L) { return L.ring_values() * dense_size(S.dtype); }
 static size_t prev_bytes(const StackModel& S, const LayerSpec& L) { return L.kind == Mixer::AttnTimeMix ? size_t(S.spec.width) * dense_size(S.dtype) : 0; }
 
 int32_t stack_cache_create(ForgeKV* kv) {
@@ -932,7 +1217,7 @@ int32_t stack_cache_create(ForgeKV* kv) {
     FORGE_TRY(ensure_rope(m, kv->max_seq));
     kv->stack = new StackCache();
     kv->stack->runs.resize(S.spec.runs.size());
-    const size_t rows = size_t(kv->num_pages) * FORGE_KV_PAGE, slots = size_t(kv->batch);
+    const size_t slots = size_t(kv->batch);
     auto alloc = [&](auto** p, size_t bytes) -> int32_t {
         if (!bytes) return FORGE_OK;
         void* q = nullptr;
@@ -946,6 +1231,7 @@ int32_t stack_cache_create(ForgeKV* kv) {
         const LayerSpec& L = S.spec.layers[S.spec.runs[i].layer];
         StackCache::Run& r = kv->stack->runs[i];
         char *pool = nullptr, *ring = nullptr, *prev = nullptr;
+        const size_t rows = size_t(kv->num_pages) * L.page_rows();
         FORGE_TRY(alloc(&pool, rows * L.cache_row() * dense_size(S.dtype)));
         r.pool = pool;
         if (L.has_latent() && tensor_core_rows(S, L.mix)) FORGE_TRY(latent_cache_map(r.map, r.pool, L.mix, rows));
@@ -1024,7 +1310,10 @@ int32_t stack_state_read(ForgeKV* kv, int seq, int run, float* out_host) {
 size_t stack_kv_bytes_per_token(const ForgeKV* kv) {
     const StackModel& S = *kv->model->stack;
     size_t n = 0;
-    for (const LayerRun& r : S.spec.runs) n += S.spec.layers[r.layer].cache_row();
+    for (const LayerRun& r : S.spec.runs) {   // blocks: their rows of a page, rounded up per position
+        const LayerSpec& L = S.spec.layers[r.layer];
+        n += (size_t(L.cache_row()) * L.page_rows() + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE;
+    }
     return n * dense_size(S.dtype);
 }
 size_t stack_kv_bytes_per_seq(const ForgeKV* kv) {
@@ -1050,6 +1339,8 @@ int32_t stack_kv_copy(ForgeKV* kv, int seq, int len, char* host, bool to_host) {
         for (int t0 = 0; row && t0 < len; t0 += FORGE_KV_PAGE) {
             const int pg = kv->h_page_table[size_t(seq) * kv->pages_per_seq + t0 / FORGE_KV_PAGE];
             FORGE_TRY(copy(static_cast<char*>(r.pool) + size_t(pg) * FORGE_KV_PAGE * row, row * std::min(FORGE_KV_PAGE, len - t0)));
+            const size_t blocks = size_t(L.page_rows() - FORGE_KV_PAGE);
+            FORGE_TRY(copy(static_cast<char*>(r.pool) + (size_t(kv->num_pages) * FORGE_KV_PAGE + size_t(pg) * blocks) * row, row * blocks));
         }
         FORGE_TRY(copy(reinterpret_cast<char*>(r.state) + size_t(seq) * state_bytes(L), state_bytes(L)));
         FORGE_TRY(copy(static_cast<char*>(r.ring) + size_t(seq) * ring_bytes(S, L), ring_bytes(S, L)));
@@ -1065,8 +1356,13 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
                    int trace_rows, int trace_row0) {
     StackModel& S = *m->stack;
     bool prompt_ok = S.dtype == FORGE_BF16;
-    for (const LayerSpec& L : S.spec.layers)
-        prompt_ok = prompt_ok && (L.has_latent() ? attn_prefill_kv_supported(PromptDims(L.mix)) : !L.has_attn() || attn_prefill_kv_supported(PromptDims(L.attn)));
+    int least_pool = 0;   // of all layers
+    for (const LayerSpec& L : S.spec.layers) {
+        PromptDims d = L.has_latent() ? PromptDims(L.mix) : PromptDims(L.attn);
+        d.joint = L.soft.talk;
+        prompt_ok = prompt_ok && ((!L.has_latent() && !L.has_attn()) || attn_prefill_kv_supported(d));
+        if (L.has_attn() && L.attn.pool) least_pool = least_pool ? std::min(least_pool, L.attn.pool) : L.attn.pool;
+    }
     // rows: the single tokens first, then the short entries, then the prompt portions
     struct Place { int row, tok, want; };
     std::vector<Place> at_entry(n_entries);
@@ -1088,6 +1384,7 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
     std::vector<int32_t> meta(size_t(3) * rows + wants);
     std::vector<int32_t> pages;
     std::vector<PromptTile> tiles;
+    std::vector<PoolChunk> pools;
     std::vector<ScanSeg> segs;
     int max_seg = 0;
     for (int i = 0; i < n_entries; ++i) {
@@ -1103,7 +1400,9 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
         if (is_prompt(i)) {
             const int ctx0 = int(pages.size()) * FORGE_KV_PAGE, np = (base + e.n_tokens + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE;
             for (int p = 0; p < np; ++p) pages.push_back(kv->h_page_table[size_t(e.seq) * kv->pages_per_seq + p]);
-            for (int t = 0; t < e.n_tokens; t += 128) tiles.push_back({r0 - single + t, std::min(128, e.n_tokens - t), base + t, ctx0});
+            const int len = base + e.n_tokens, pool0 = int(pools.size()) * FORGE_KV_PAGE;
+            for (int b = 0; least_pool && b < len / least_pool; b += FORGE_KV_PAGE) pools.push_back({ctx0 / FORGE_KV_PAGE, b, len, 0});
+            for (int t = 0; t < e.n_tokens; t += 128) tiles.push_back({r0 - single + t, std::min(128, e.n_tokens - t), base + t, ctx0, pool0, {}});
         }
     }
     std::stable_sort(tiles.begin(), tiles.end(), [](const PromptTile& a, const PromptTile& b) { return a.pos0 + a.rows > b.pos0 + b.rows; });   // the longest first
@@ -1111,14 +1410,16 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
     const int n_short = int(first_long - segs.begin());
     int chunks = 0;
     for (auto g = first_long; g != segs.end(); ++g) { g->chunk0 = chunks; chunks += (g->n + kRecurChunk - 1) / kRecurChunk; }
-    static_assert(sizeof(ScanSeg) == 32, "eight words");
-    const size_t o_pages = (meta.size() + 3) & ~size_t(3), o_tiles = (o_pages + pages.size() + 3) & ~size_t(3), o_segs = o_tiles + tiles.size() * 4, total = o_segs + segs.size() * 8;
+    static_assert(sizeof(ScanSeg) == 32 && sizeof(PromptTile) == 32 && sizeof(PoolChunk) == 16, "words");
+    const size_t o_pages = (meta.size() + 3) & ~size_t(3), o_tiles = (o_pages + pages.size() + 3) & ~size_t(3), o_segs = o_tiles + tiles.size() * 8, o_pools = o_segs + segs.size() * 8,
+                 total = o_pools + pools.size() * 4;
     meta.resize(total);
     std::copy(pages.begin(), pages.end(), meta.begin() + o_pages);
     if (!tiles.empty()) memcpy(meta.data() + o_tiles, tiles.data(), tiles.size() * sizeof(PromptTile));
     if (!segs.empty()) memcpy(meta.data() + o_segs, segs.data(), segs.size() * sizeof(ScanSeg));
+    if (!pools.empty()) memcpy(meta.data() + o_pools, pools.data(), pools.size() * sizeof(PoolChunk));
     const int splits = row_splits(S, std::max(1, single), (max_keys + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE), ctx_rows = int(pages.size()) * FORGE_KV_PAGE;
-    FORGE_TRY(ensure_step(m, std::max(rows, wants), single, splits, rows - single, ctx_rows, rows - ones, chunks));
+    FORGE_TRY(ensure_step(m, std::max(rows, wants), single, splits, rows - single, ctx_rows, rows - ones, chunks, max_keys, int(pools.size()) * FORGE_KV_PAGE, false));
     FORGE_TRY(grow(m, S.meta, total * 4));
     FORGE_TRY(grow(m, S.sel, size_t(wants) * S.width_p * dense_size(S.dtype)));
     FORGE_TRY(grow(m, S.logits, size_t(wants) * S.spec.vocab * 4));
@@ -1131,6 +1432,7 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
     s.ones = ones; s.single = single; s.splits = splits; s.max_keys = max_keys;
     s.segs = SegTable{reinterpret_cast<const ScanSeg*>(dm + o_segs), int(segs.size()), n_short, max_seg, chunks, ones, rows - ones};
     s.ctx_pages = dm + o_pages; s.ctx_rows = ctx_rows;
+    s.chunks = reinterpret_cast<const PoolChunk*>(dm + o_pools); s.n_chunks = int(pools.size());
     s.tiles = reinterpret_cast<const PromptTile*>(dm + o_tiles); s.n_tiles = int(tiles.size()); s.host_tiles = tiles.data();
     s.scale_rows = std::max(rows, wants);
     if (trace_rows) { s.trace = m->trace + size_t(trace_row0) * S.spec.width; s.trace_stride = size_t(trace_rows) * S.spec.width; }
@@ -1162,7 +1464,7 @@ int32_t stack_prefill(ForgeModel* m, ForgeKV* kv, int seq, const uint32_t* token
     return rc;
 }
 
-int32_t stack_ensure_decode(ForgeModel* m, ForgeKV* kv, int batch) { return ensure_step(m, batch, batch, kv->stack->splits, 0, 0, 0, 0); }
+int32_t stack_ensure_decode(ForgeModel* m, ForgeKV* kv, int batch) { return ensure_step(m, batch, batch, kv->stack->splits, 0, 0, 0, 0, kv->max_seq, 0, true); }
 
 int32_t stack_decode_launches(ForgeModel* m, ForgeKV* kv, int batch, bool greedy, bool record) {
     StackModel& S = *m->stack;
