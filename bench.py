@@ -2,7 +2,7 @@
 """Benchmark of the quantized forward path on B200.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
-    python bench.py --design bolenex|robazen|mokatar  (another model design, one GPU; the default workload is unchanged)
+    python bench.py --design bolenex|robazen|mokatar|tarulix  (another model design, one GPU; the default workload is unchanged)
 
 One GPU (the default).  Headline workload: the Llama-3.2-1B-shaped Q4_0 decoder of the benchmark definition - one
 "step" is one request: a 1501-token uniform-random prompt through the batched prefill path, then 128 greedy decode
@@ -487,6 +487,35 @@ def mokatar_work(cfg: dict, ctx: int, m: int):
     return (lambda batch: dense + sum(b * (1 - (1 - top / E) ** batch) for b, E, top in mixtures)), kv, flops
 
 
+def tarulix_work(cfg: dict, ctx: int, m: int):
+    """The same.  Attention over a window of tokens and the blocks in front of it; a scan's states are read and written every step; experts are drawn among the
+    choices that pass the input on, too."""
+    from forge_llm_b200 import synth
+    W, V = cfg["width"], cfg["vocab"]
+    shapes = synth.stack_shapes(cfg)
+    dense, mixtures, kv, flops = 2.0 * V * W, [], 0.0, 2.0 * V * W
+    for i, L in enumerate(cfg["layers"]):
+        mats = {k: s[0] * s[1] for k, s in shapes.items() if k.startswith(f"l{i}.") and len(s) == 2 and not k.endswith((".conv", ".A_log", ".rel", ".talk"))}
+        exp = sum(v for k, v in mats.items() if ".mlp.e" in k)
+        lin = sum(mats.values()) - exp
+        x, r = L["mixer"], L["mlp"]["router"]
+        C = r["experts"] + r["identity"]
+        dense += 2.0 * lin
+        mixtures.append((2.0 * exp, C, r["top"]))
+        flops += 2.0 * m * (lin + exp * r["top"] / C)
+        a = x.get("left", x)
+        c, p = a["mask"]["size"], a["mask"].get("pool", 0)
+        keys = lambda i: min(i + 1, c) + (max(0, i - c + 1) // p if p else 0)
+        kv += 2.0 * a["kv_heads"] * (a["dim"] + a["vdim"]) * keys(ctx)
+        flops += 2.0 * a["heads"] * (a["dim"] + a["vdim"]) * sum(keys(i) for i in range(m))
+        if "right" in x:
+            n, s = x["right"]["inner"], x["right"]["state"]
+            kv += 8.0 * n * s
+            dense += 4.0 * n * s
+            flops += 6.0 * m * n * s
+    return (lambda batch: dense + sum(b * (1 - (1 - top / C) ** batch) for b, C, top in mixtures)), kv, flops
+
+
 def run_design(args, device: int):
     """Prefill and decode rates of a layer-list design and, at equal width, depth, heads and feed-forward, of the framework's closest
     decoder (multi-head, head_dim 128, Q8_0), each against its own roofline."""
@@ -497,7 +526,8 @@ def run_design(args, device: int):
     t0 = time.time()
     out, launches = {}, 0
     design = args.design
-    make_config, work = {"bolenex": (synth.bolenex_config, bolenex_work), "robazen": (synth.robazen_config, robazen_work), "mokatar": (synth.mokatar_config, mokatar_work)}[design]
+    make_config, work = {"bolenex": (synth.bolenex_config, bolenex_work), "robazen": (synth.robazen_config, robazen_work), "mokatar": (synth.mokatar_config, mokatar_work),
+                         "tarulix": (synth.tarulix_config, tarulix_work)}[design]
     arm = f"{design} bf16"
 
     def measure(model, batch, n_prompt, n_dec, bytes_w, bytes_kv, flops, vocab):
@@ -745,7 +775,7 @@ def main():
     ap.add_argument("--prompt-tokens", type=int, default=None, help="override the headline prompt length (profiling / experiments)")
     ap.add_argument("--decode-steps", type=int, default=None, help="override the headline number of decode steps")
     ap.add_argument("--profile", action="store_true", help="short run for ncu: no side configurations, no CPU baseline; prints a non-benchmark line")
-    ap.add_argument("--design", default="headline", choices=["headline", "bolenex", "robazen", "mokatar"], help="bolenex, robazen, mokatar: that design beside a Llama-shaped decoder of equal size (one GPU)")
+    ap.add_argument("--design", default="headline", choices=["headline", "bolenex", "robazen", "mokatar", "tarulix"], help="bolenex, robazen, mokatar, tarulix: that design beside a Llama-shaped decoder of equal size (one GPU)")
     ap.add_argument("--sizes", default="w2048,w4096", help="with --design: which sizes")
     ap.add_argument("--batches", default="1,16", help="with --design: sequences decoded together")
     ap.add_argument("--arms", default="design,llama", help="with --design: which models")

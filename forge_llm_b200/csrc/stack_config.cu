@@ -255,7 +255,7 @@ int32_t parse_experts(const Json* mlp, int layer, bool shared, LayerSpec* L) {
         FORGE_TRY(need_int(router, "identity", &L->router.identity, 0));
     }
     if (L->router.top > L->router.choices()) { set_error("layer %d: top %d of %d experts", layer, L->router.top, L->router.choices()); return FORGE_ERR_SHAPE; }
-    if (L->router.choices() > kMaxExperts) { set_error("layer %d: %d experts are not supported", layer, L->router.experts); return FORGE_ERR_UNSUPPORTED; }
+    if (L->router.choices() > kMaxExperts) { set_error("layer %d: %d experts are not supported", layer, L->router.choices()); return FORGE_ERR_UNSUPPORTED; }
     return FORGE_OK;
 }
 

@@ -320,14 +320,53 @@ def mokatar_shapes(cfg: dict, layer: int, rank: int = 64) -> dict:
     return s
 
 
-LAYER_SHAPES = {"Bolenex": bolenex_shapes, "Robazen": robazen_shapes, "Mokatar": mokatar_shapes}
+def tarulix_config(width: int, layers: int, heads: int, ff: int, vocab: int, dim: int = 128, window: int = 1024, pool: int = 16, state: int = 16, experts: int = 8, identity: int = 2, top: int = 2) -> dict:
+    """config.json of a Tarulix stack: attention over a window and blocks beside a selective scan of twice the width, and windowed attention, in turn; a
+    mixture whose used experts and shared expert have ``ff`` rows together."""
+    kv = max(1, heads // 4)
+    left = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": float(dim ** -0.5), "softcap": 30.0, "mask": {"size": window, "pool": pool}, "rot": {"base": 10000.0, "dims": dim}}
+    pair = {"left": left, "left_scale": 0.9, "right": {"inner": 2 * width, "state": state, "dt_rank": max(1, width // 16), "conv": 4}, "right_scale": 1.1}
+    near = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": float(dim ** -0.5), "bias_max": 4 * window, "mask": {"size": window}, "v_mix": True}
+    moe = {"kind": "moe", "expert": {"ff": ff // 2 // top}, "shared": {"ff": ff // 2}, "router": {"experts": experts, "identity": identity, "top": top}}
+    return {"architecture": "Tarulix", "width": width, "vocab": vocab, "norm": {"eps": 1e-5},
+            "layers": [{"type": "attention" if i % 2 else "parallel", "mixer": dict(near if i % 2 else pair), "mlp": dict(moe)} for i in range(layers)]}
+
+
+def tarulix_shapes(cfg: dict, layer: int, buckets: int = 32) -> dict:
+    """Tensor shapes of one layer, without its prefix; ``buckets``: of the biases by distance."""
+    W, L = cfg["width"], cfg["layers"][layer]
+    m, f = L["mixer"], L.get("mlp")
+    a, p = (m["left"], "mix.left.") if L["type"] == "parallel" else (m, "mix.")
+    q, k, v, hv = a["heads"] * a["dim"], a["kv_heads"] * a["dim"], a["kv_heads"] * a["vdim"], a["heads"] * a["vdim"]
+    s = {"norm1": (), p + "q": (q, W), p + "q.b": (q,), p + "k": (k, W), p + "k.b": (k,), p + "v": (v, W), p + "v.b": (v,), p + "o": (W, hv), p + "o.b": (W,)}
+    if L["type"] == "parallel":
+        r = m["right"]
+        n, st, k = r["inner"], r["state"], r["dt_rank"]
+        s[p + "talk"] = (a["heads"], a["heads"])
+        s.update({"mix.right." + x: y for x, y in (("in", (2 * n, W)), ("conv", (n, r["conv"])), ("conv.b", (n,)), ("x", (k + 2 * st, n)), ("dt", (n, k)), ("dt.b", (n,)), ("A_log", (n, st)), ("D", (n,)), ("o", (W, n)))})
+    else:
+        s.update({"mix.rel": (buckets, a["heads"]), "mix.sink": (a["heads"],)})
+        if a.get("v_mix"):
+            s["mix.vmix"] = ()
+    if f:
+        E, n, sh = f["router"]["experts"], f["expert"]["ff"], f["shared"]["ff"]
+        s["norm2"] = ()
+        for e, c in [(f"e{e}", n) for e in range(E)] + [("shared", sh)]:
+            s.update({f"mlp.{e}.gate": (c, W), f"mlp.{e}.up": (c, W), f"mlp.{e}.down": (W, c)})
+        s.update({"mlp.router": (E + f["router"]["identity"], W), "mlp.correction": (E + f["router"]["identity"],)})
+    return s
+
+
+LAYER_SHAPES = {"Bolenex": bolenex_shapes, "Robazen": robazen_shapes, "Mokatar": mokatar_shapes, "Tarulix": tarulix_shapes}
 
 
 def stack_shapes(cfg: dict) -> dict:
     """Tensor shapes of a layer-list model."""
     W, V = cfg["width"], cfg["vocab"]
-    out = {"embed": (V, W), "head": (V, W), "final.norm": (W,)}
-    if cfg["architecture"] == "Mokatar":
+    out = {"embed": (V, W), "head": (V, W), "final.norm": () if cfg["architecture"] == "Tarulix" else (W,)}
+    if cfg["architecture"] == "Tarulix":
+        pass
+    elif cfg["architecture"] == "Mokatar":
         out["bigram"] = (cfg["embedding"]["bigram"]["buckets"] + 1, W)
     else:
         out.update({"final.norm.b": (W,), "final.norm.alpha": ()})

@@ -883,8 +883,113 @@ def random_mokatar(cfg, seed=0, rank=12, clear=True):
     return t
 
 
+def distance_mixer(heads=6, kv_heads=2, dim=24, vdim=40, window=40, bias_max=64, scale=None, v_mix=True):
+    m = {"bias_max": bias_max, "dim": dim, "heads": heads, "kv_heads": kv_heads, "mask": None if window is None else {"size": window}, "scale": float(scale if scale is not None else dim ** -0.5), "vdim": vdim}
+    return {**m, "v_mix": True} if v_mix else m
+
+
+def scan_pair(heads=6, kv_heads=2, dim=24, vdim=40, window=40, pool=8, rot=16, base=3000.0, softcap=20.0, scale=None, inner=72, state=16, rank=12, conv=4, scales=(0.7, 1.2)):
+    left = {"dim": dim, "heads": heads, "kv_heads": kv_heads, "mask": None if window is None else {"pool": pool, "size": window}, "rot": {"base": float(base), "dims": rot},
+            "scale": float(scale if scale is not None else 1.5 * dim ** -0.5), "softcap": float(softcap), "vdim": vdim}
+    return {"left": left, "left_scale": scales[0], "right": {"conv": conv, "dt_rank": rank, "inner": inner, "state": state}, "right_scale": scales[1]}
+
+
+def make_tarulix(width=136, vocab=203, layers=(), eps=1e-5):
+    """``layers``: (type, mixer, feed-forward) per layer, the feed-forward None or (experts, top, size, identity choices, size of the shared expert)."""
+    def ff(f):
+        return f and {"expert": {"ff": f[2]}, "kind": "moe", "router": {"experts": f[0], "identity": f[3], "top": f[1]}, "shared": {"ff": f[4]}}
+    return {"architecture": "Tarulix", "layers": [{"mixer": m, "mlp": ff(f), "type": t} for t, m, f in layers], "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def random_tarulix(cfg, seed=0, clear=True, buckets=16):
+    """Seeded weights of a Tarulix model, rounded to bfloat16.  clear: as for Mokatar; what is passed on scales the marked columns up, so routers are
+    drawn for a range of scales."""
+    rng = np.random.default_rng(seed)
+    W = cfg["width"]
+    t = {}
+
+    def mat(name, out, inp, gain=1.0):
+        t[name] = bf16_round(rng.standard_normal((out, inp)) * (gain / math.sqrt(inp)))
+
+    def vec(name, n, mean, dev):
+        t[name] = bf16_round(mean + dev * rng.standard_normal(n))
+
+    def scalar(name, lo, hi):
+        t[name] = bf16_round(np.asarray(lo + (hi - lo) * rng.random()))
+
+    def attention(x, m):
+        H, q, k, v = m["heads"], m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"]
+        for n, c in (("q", q), ("k", k), ("v", v)):
+            mat(x + n, c, W)
+            vec(x + n + ".b", c, 0.0, 1.0 if n == "k" and x.endswith("left.") else 0.5)     # keys of a block have something in common
+        mat(x + "o", W, H * m["vdim"], 4.0 if x.endswith("left.") else 2.0)
+        vec(x + "o.b", W, 0.0, 0.2)
+        return H
+
+    t["embed"] = bf16_round(rng.standard_normal((cfg["vocab"], W)))
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        x = p + "mix."
+        scalar(p + "norm1", 0.6, 1.4)
+        if L["type"] == "parallel":
+            H = attention(x + "left.", m["left"])
+            t[x + "left.talk"] = bf16_round(np.eye(H) + 0.4 * rng.standard_normal((H, H)))
+            r = m["right"]
+            n, s, k = r["inner"], r["state"], r["dt_rank"]
+            x += "right."
+            mat(x + "in", 2 * n, W, 0.7)
+            t[x + "conv"] = bf16_round(0.6 * rng.standard_normal((n, r["conv"])))
+            vec(x + "conv.b", n, 0.0, 0.3)
+            mat(x + "x", k + 2 * s, n, 0.7)
+            mat(x + "dt", n, k, 1.5)
+            vec(x + "dt.b", n, -2.5, 1.5)
+            t[x + "A_log"] = bf16_round(-1.0 + 1.5 * rng.standard_normal((n, s)))
+            vec(x + "D", n, 0.8, 0.3)
+            mat(x + "o", W, n, 2.0)
+        else:
+            H = attention(x, m)
+            t[x + "rel"] = bf16_round(rng.standard_normal((buckets, H)))
+            vec(x + "sink", H, 1.0, 1.5)
+            if m.get("v_mix"):
+                scalar(x + "vmix", 0.2, 0.8)
+        f = L.get("mlp")
+        if f:
+            scalar(p + "norm2", 0.6, 1.4)
+            E, C, n, sh = f["router"]["experts"], f["router"]["experts"] + f["router"]["identity"], f["expert"]["ff"], f["shared"]["ff"]
+            for e, c in [(f"e{e}", n) for e in range(E)] + [("shared", sh)]:
+                mat(p + f"mlp.{e}.gate", c, W, 1.5)
+                mat(p + f"mlp.{e}.up", c, W, 1.5)
+                mat(p + f"mlp.{e}.down", W, c, 2.0)
+            mat(p + "mlp.router", C, W, 2.0)
+            vec(p + "mlp.correction", C, 0.3, 0.3)
+    scalar("final.norm", 0.6, 1.4)
+    mat("head", cfg["vocab"], W)
+    if clear:
+        t["embed"][:, :MARKERS] = np.sign(rng.standard_normal((cfg["vocab"], MARKERS)))
+        patterns = np.array([[1.0 if i >> c & 1 else -1.0 for c in range(MARKERS)] for i in range(1 << MARKERS)])
+        patterns = np.concatenate([s * patterns for s in np.linspace(1.0, 2.5, 16)])
+        for name in t:
+            if name.endswith((".o", ".down", ".o.b")):
+                t[name][:MARKERS] = 0
+            if name.endswith("mlp.router"):
+                top, best = cfg["layers"][int(name[1:name.index(".")])]["mlp"]["router"]["top"], None
+                for _ in range(300):     # of some routers the one whose closest call is least close
+                    r = np.zeros_like(t[name])
+                    r[:, :MARKERS] = bf16_round(2.0 * rng.standard_normal((len(r), MARKERS)))
+                    corr = bf16_round(0.3 + (0.3 if len(r) < 20 else 0.6) * rng.standard_normal(len(r)))
+                    e = np.exp(patterns @ r[:, :MARKERS].T)
+                    z = np.sort(e / e.sum(1, keepdims=True) + corr, axis=1)[:, ::-1]
+                    gap = (z[:, top - 1] - z[:, top]).min() if top < len(r) else 1e9
+                    if best is None or gap > best[0]:
+                        best = (gap, r, corr)
+                _, t[name], t[name[:-6] + "correction"] = best
+    return t
+
+
 def random_tensors(cfg, seed=0):
     """Seeded weights, rounded to bfloat16, in which every factor matters (norm weights and biases away from 1 and 0)."""
+    if cfg["architecture"] == "Tarulix":
+        return random_tarulix(cfg, seed)
     if cfg["architecture"] == "Mokatar":
         return random_mokatar(cfg, seed)
     if cfg["architecture"] == "Robazen":

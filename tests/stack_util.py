@@ -63,10 +63,30 @@ MOKATAR = {
     "beyond": LS.make_mokatar(96, 110, [("attention", LS.head_normed_mixer(10, 1, 72, 272, 1000, 100), (3, 2, 40)), ("gla", LS.linear_mixer(1, 136, 200, 2.0), None), ("attention_2", LS.row_normed_mixer(2, 2, 300, 136), 40),
                                         ("attention", LS.head_normed_mixer(3, 3, 24, 24, 20, 70), None)]),
 }
+_far, _scan = LS.distance_mixer, LS.scan_pair
+TARULIX = {
+    # every mechanism: windows shorter and longer than the biases reach, blocks that divide a page and blocks that do not, a layer without a feed-forward, values
+    # blended twice (between heads of different sizes) and not at all
+    "all": LS.make_tarulix(136, 203, [("parallel", _scan(), (5, 2, 24, 2, 40)), ("attention", _far(), None), ("parallel", _scan(4, 4, 16, 24, 33, 24, 10, 50.0, 8.0, 0.6, 40, 6, 9, 3, (1.3, 0.6)), (4, 3, 40, 0, 72)),
+                                      ("attention", _far(8, 2, 32, 40, 50, 20), (3, 4, 16, 3, 24)), ("attention", _far(3, 1, 16, 24, 20, 100, None, False), (6, 1, 24, 1, 16)), ("attention", _far(2, 2, 16, 40, 64, 64), None)], eps=1e-3),
+    # one of everything: a window of one token, blocks of one, two and sixty-four, no history in the convolution, every choice taken
+    "ones": LS.make_tarulix(72, 67, [("parallel", _scan(1, 1, 8, 8, 1, 2, 8, 9.0, 5.0, 0.9, 8, 1, 1, 1, (1.0, 1.0)), (1, 2, 16, 1, 8)), ("parallel", _scan(2, 1, 16, 16, 7, 1, 2, 90.0, 50.0, 0.3, 24, 4, 2, 2), None),
+                                     ("parallel", _scan(2, 2, 8, 16, 20, 64, 0, 90.0, 50.0, 0.5, 16, 8, 5, 2, (0.5, 2.0)), (2, 1, 40, 2, 8)), ("attention", _far(1, 1, 8, 8, 1, 2), (1, 1, 8, 0, 40))], eps=1e-2),
+    # sizes no multiple of eight
+    "odd": LS.make_tarulix(70, 91, [("attention", _far(6, 3, 13, 11, 33, 37), (7, 3, 21, 2, 13)), ("parallel", _scan(3, 1, 9, 13, 45, 5, 6, 77.0, 11.0, 0.4, 37, 5, 3, 5, (0.9, -0.8)), (3, 2, 9, 4, 21)), ("attention", _far(9, 3, 7, 11, None, 30), None),
+                                    ("parallel", _scan(4, 2, 10, 7, 70, 48, 4, 20.0, 40.0, 0.5, 50, 20, 33, 2), (4, 2, 30, 1, 9))]),
+    # a real model's head sizes, many experts, several row tiles per expert
+    "wide": LS.make_tarulix(192, 150, [("parallel", _scan(8, 2, 128, 128, 80, 16, 64, 10000.0, 30.0, None, 256, 16, 64, 4), (40, 4, 100, 8, 136)), ("attention", _far(8, 2, 128, 64, 70, 300), (70, 6, 40, 10, 64)),
+                                       ("parallel", _scan(6, 6, 64, 64, 100, 32, 64, 1e6, 30.0, None, 192, 64, 72, 4), None)]),
+    # beyond the tensor-core kernels: wide heads and values, many query heads on a key head, blocks longer than a page, many states and taps, the whole past
+    "beyond": LS.make_tarulix(96, 110, [("parallel", _scan(20, 1, 72, 272, 60, 70, 40, 500.0, 25.0, None, 40, 200, 20, 6), (3, 2, 40, 1, 24)), ("attention", _far(10, 1, 300, 24, 1000, 500), None),
+                                        ("parallel", _scan(34, 2, 24, 24, None, 0, 24, 500.0, 25.0, None, 24, 33, 6, 4), None)]),
+}
+CONFIGS.update({"tarulix_" + k: v for k, v in TARULIX.items()})
 CONFIGS.update({"mokatar_" + k: v for k, v in MOKATAR.items()})
 CONFIGS.update({"robazen_" + k: v for k, v in ROBAZEN.items()})
 ROBAZEN_NAMES = ["robazen_" + k for k in ROBAZEN]
-BOLENEX_NAMES = [k for k in CONFIGS if not k.startswith(("robazen_", "mokatar_"))]
+BOLENEX_NAMES = [k for k in CONFIGS if not k.startswith(("robazen_", "mokatar_", "tarulix_"))]
 
 
 def sharp(tensors, cfg, gain=5.0):
