@@ -291,7 +291,7 @@ int32_t attn_prefill_kv(const PromptDims& d, const PromptAttnArgs& a, cudaStream
     if (d.rot_p == 0) mr = mk;   // no rotated part: never read
     else FORGE_TRY(make_map_2d(&mr, a.krot, uint64_t(d.rot_p), uint64_t(a.ctx_rows), uint64_t(d.rot_p) * 2, BN));
     FORGE_TRY(make_map_3d(&mv, a.v, uint64_t(d.vdim_p), G, uint64_t(a.ctx_rows), uint64_t(d.vdim_p) * 2, v_row, BN));
-    if (d.pool > 0 && a.blocks) {
+    if (d.pool > 0 && a.block_rows > 0) {
         FORGE_TRY(make_map_3d(&bk, a.blocks, uint64_t(d.dim_p), G, uint64_t(a.block_rows), uint64_t(d.dim_p) * 2, k_row, BN));
         FORGE_TRY(make_map_3d(&bv, static_cast<const __nv_bfloat16*>(a.blocks) + G * d.dim_p, uint64_t(d.vdim_p), G, uint64_t(a.block_rows), uint64_t(d.vdim_p) * 2, v_row, BN));
     } else { bk = mk; bv = mv; }

@@ -457,7 +457,7 @@ __global__ void __launch_bounds__(kThreads) talk_values_mma_kernel(const AttnDim
 }
 
 // ------------------------------------------------------------------------------------------------ behind prompt attention
-constexpr int kMixHeads = 8;     // heads of a group that a thread carries
+constexpr int kMixHeads = 4;     // heads of a group that a thread carries
 // A thread = eight columns of one group of one row.
 __global__ void __launch_bounds__(256) talk_heads_kernel(const AttnDims d, const bf16* __restrict__ o, const float* __restrict__ talk, float factor, bf16* __restrict__ out, int out_ld, int rows) {
     extern __shared__ float mix[];      // [heads][heads], transposed: the weights of one source head lie side by side
@@ -476,7 +476,7 @@ __global__ void __launch_bounds__(256) talk_heads_kernel(const AttnDims d, const
 #pragma unroll
             for (int e = 0; e < 8; ++e) acc[h][e] = 0.f;
         const int nh = min(kMixHeads, gq - h0);
-#pragma unroll 4
+#pragma unroll 8
         for (int x = 0; x < d.heads; ++x) {
             float v[8];
             load8(v, src + size_t(x) * W);

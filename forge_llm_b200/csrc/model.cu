@@ -1078,7 +1078,7 @@ int32_t kv_copy_rows(ForgeKV* kv, int seq, int layer, int which, int len, __half
 size_t forge_kv_save_size(const ForgeKV* kv, int32_t seq) {
     if (!kv || !kv->model || seq < 0 || seq >= kv->batch) return 0;
     const ForgeModel* m = kv->model;
-    if (m->stack) return sizeof(KvHeader) + stack_kv_bytes_per_token(kv) * kv->len[seq] + stack_kv_bytes_per_seq(kv);
+    if (m->stack) return sizeof(KvHeader) + stack_kv_bytes(kv, kv->len[seq]);
     return sizeof(KvHeader) + size_t(2) * m->cfg.num_layers * kv->len[seq] * m->kv * sizeof(__half);
 }
 
@@ -1120,7 +1120,7 @@ int32_t forge_kv_load(ForgeKV* kv, int32_t seq, const void* data_host, size_t n)
         if (n < sizeof(h)) { set_error("forge_kv_load: no data"); return FORGE_ERR_INVALID_ARG; }
         memcpy(&h, p, sizeof(h));
         if (memcmp(h.magic, kLatentMagic, 4) || h.layers != uint32_t(L) || h.width != uint32_t(stack_kv_bytes_per_token(kv))) { set_error("forge_kv_load: not a cache file of this model"); return FORGE_ERR_SHAPE; }
-        if (h.len > uint64_t(kv->max_seq) || n != sizeof(h) + size_t(h.width) * h.len + stack_kv_bytes_per_seq(kv)) { set_error("forge_kv_load: bad length"); return FORGE_ERR_SHAPE; }
+        if (h.len > uint64_t(kv->max_seq) || n != sizeof(h) + stack_kv_bytes(kv, int(h.len))) { set_error("forge_kv_load: bad length"); return FORGE_ERR_SHAPE; }
         FORGE_TRY(forge_kv_free_seq(kv, seq));
         FORGE_TRY(ensure_pages(kv, seq, int(h.len)));
         FORGE_TRY(stack_kv_copy(kv, seq, int(h.len), reinterpret_cast<char*>(const_cast<uint8_t*>(p)) + sizeof(h), false));

@@ -145,7 +145,7 @@ int32_t stack_kv_read(ForgeKV* kv, int seq, int run, int which, float* out_host)
 size_t stack_state_values(const ForgeKV* kv, int run);
 int32_t stack_state_read(ForgeKV* kv, int seq, int run, float* out_host);
 size_t stack_kv_bytes_per_token(const ForgeKV* kv);
-size_t stack_kv_bytes_per_seq(const ForgeKV* kv);
+size_t stack_kv_bytes(const ForgeKV* kv, int len);   // of a sequence
 int32_t stack_kv_copy(ForgeKV* kv, int seq, int len, char* host, bool to_host);
 
 }  // namespace forge

@@ -3,8 +3,9 @@
 //
 // A channel's states are dealt to a group of G neighbouring lanes (a power of two), four or eight each; a token's read-out is added over the
 // group.  Over a segment a CTA carries its channels token by token, with the inputs of the next tile of tokens on their way while one is worked off;
-// the read-outs of four tokens are added together, each step of the sum halving how many a lane holds.
+// the read-outs of sixteen tokens are added together, each step of the sum halving how many a lane holds.
 #include <algorithm>
+#include <type_traits>
 
 #include "selective.cuh"
 
@@ -82,6 +83,52 @@ __global__ void __launch_bounds__(128) conv_segments_kernel(const SelectiveDims 
         for (int t = max(0, s.n - d.taps); t < s.n; ++t) ring[size_t((s.pos0 + t) % d.taps) * d.inner] = in[size_t(t) * a.in_ld];
 }
 
+// The same for bfloat16 channels in whole 16-byte pieces and at most four taps: a thread carries eight channels over eight tokens.
+constexpr int kRun8 = 8;
+__global__ void __launch_bounds__(128) conv_segments8_kernel(const SelectiveDims d, const SelectiveArgs a, const ScanSeg* __restrict__ segs) {
+    using bf16 = __nv_bfloat16;
+    const ScanSeg s = segs[blockIdx.z];
+    const int t0 = blockIdx.x * kRun8, c = (blockIdx.y * 128 + threadIdx.x) * 8;
+    if (t0 >= s.n || c >= d.inner) return;
+    const bf16* in = static_cast<const bf16*>(a.in) + size_t(s.row0) * a.in_ld + c;
+    bf16* out = static_cast<bf16*>(a.x) + size_t(s.row0) * a.x_ld + c;
+    bf16* ring = static_cast<bf16*>(a.ring) + size_t(s.slot) * d.ring_values() + c;
+    uint4 now[kRun8];
+#pragma unroll
+    for (int i = 0; i < kRun8; ++i) now[i] = t0 + i < s.n ? *reinterpret_cast<const uint4*>(in + size_t(t0 + i) * a.in_ld) : make_uint4(0, 0, 0, 0);
+    float w[4][8], past[3][8], add[8];   // past[2]: the token before
+    load8(add, a.conv_add + c);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) w[j][e] = 0.f;
+        if (j >= 4 - d.taps) load8(w[j], a.conv + size_t(j - (4 - d.taps)) * d.inner + c);
+    }
+#pragma unroll
+    for (int j = 0; j < 3; ++j) {
+        const int q = t0 - 3 + j, p = s.pos0 + q;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) past[j][e] = 0.f;
+        if (j >= 4 - d.taps && p >= 0) load8(past[j], q >= 0 ? in + size_t(q) * a.in_ld : ring + size_t(p % d.taps) * d.inner);
+    }
+#pragma unroll
+    for (int i = 0; i < kRun8; ++i) {
+        float v[8], y[8];
+        load8(v, reinterpret_cast<const bf16*>(&now[i]));
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            y[e] = conv_act<bf16>(fmaf(w[3][e], v[e], fmaf(w[2][e], past[2][e], fmaf(w[1][e], past[1][e], fmaf(w[0][e], past[0][e], add[e])))));
+            past[0][e] = past[1][e]; past[1][e] = past[2][e]; past[2][e] = v[e];
+        }
+        if (t0 + i < s.n) {
+            put4(out + size_t(t0 + i) * a.x_ld, make_float4(y[0], y[1], y[2], y[3]));
+            put4(out + size_t(t0 + i) * a.x_ld + 4, make_float4(y[4], y[5], y[6], y[7]));
+        }
+    }
+    if (blockIdx.x == 0)
+        for (int t = max(0, s.n - d.taps); t < s.n; ++t) *reinterpret_cast<uint4*>(ring + size_t((s.pos0 + t) % d.taps) * d.inner) = *reinterpret_cast<const uint4*>(in + size_t(t) * a.in_ld);
+}
+
 // ------------------------------------------------------------------------------------------------ recurrence
 template <int SP> struct States {   // states sub * SP .. of a channel
     float v[SP];
@@ -155,12 +202,15 @@ __global__ void __launch_bounds__(kScanThreads) selective_decode_kernel(const Se
     if (sub == 0) static_cast<T*>(a.out)[size_t(r) * a.out_ld + c] = to_t<T>(fmaf(skip, x, y) * gate * a.factor);
 }
 
-constexpr int kTile = 16;     // tokens whose inputs are in shared memory
+constexpr int kTile = 32, kHalf = 16;     // tokens whose inputs are in shared memory, and whose read-outs are in registers
 template <typename T, int G, int SP>
 __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const SelectiveDims d, const SelectiveArgs a, const ScanSeg* __restrict__ segs) {
     constexpr int CB = kScanThreads / G, NP = G * SP, BC = kTile * NP, XC = kTile * CB;   // channels per CTA, padded states
     constexpr int LB = (2 * BC + kScanThreads - 1) / kScanThreads, LX = (XC + kScanThreads - 1) / kScanThreads;
-    __shared__ __align__(16) float s_bc[2][kTile][NP], s_dt[kTile][CB], s_x[kTile][CB], s_g[kTile][CB], s_y[kTile][CB];
+    extern __shared__ __align__(16) float sm[];
+    float* s_bc = sm;                                             // [B | C][kTile][NP]
+    float2* s_dx = reinterpret_cast<float2*>(s_bc + 2 * BC);      // [kTile][CB]: step size, times x
+    float* s_y = reinterpret_cast<float*>(s_dx + XC);             // [kTile][CB]
     const ScanSeg s = segs[blockIdx.y];
     const int tid = threadIdx.x, sub = tid % G, cl = tid / G, c0 = blockIdx.x * CB, c = c0 + cl;
     const bool ok = c < d.inner;
@@ -178,7 +228,8 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Sele
     const float* dt = a.dt + size_t(s.row0) * a.dt_ld + c0;
     const float* bc = a.bc + size_t(s.row0) * a.bc_ld;
     T* out = static_cast<T*>(a.out) + size_t(s.row0) * a.out_ld + c0;
-    float rb[LB], rd[LX], rg[LX], rx[LX];
+    float rb[LB], rd[LX];
+    T rg[LX], rx[LX];
     auto fetch = [&](int t0) {
 #pragma unroll
         for (int j = 0; j < LB; ++j) {
@@ -190,65 +241,70 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Sele
             const int i = tid + kScanThreads * j, t = i / CB, k = i % CB;
             const bool in = i < XC && t0 + t < s.n && c0 + k < d.inner;
             rd[j] = in ? dt[size_t(t0 + t) * a.dt_ld + k] : 0.f;
-            rx[j] = in ? to_f(x[size_t(t0 + t) * a.x_ld + k]) : 0.f;
-            rg[j] = in ? to_f(gate[size_t(t0 + t) * a.gate_ld + k]) * a.factor : 0.f;
+            rx[j] = in ? x[size_t(t0 + t) * a.x_ld + k] : to_t<T>(0.f);
+            rg[j] = in ? gate[size_t(t0 + t) * a.gate_ld + k] : to_t<T>(0.f);
         }
     };
     fetch(0);
-    float skip[LX];
-#pragma unroll
-    for (int j = 0; j < LX; ++j) { const int k = (tid + kScanThreads * j) % CB; skip[j] = c0 + k < d.inner ? a.skip[c0 + k] : 0.f; }
+    const int own = tid % CB;      // the channel of all elements that this thread fetches and finishes (CB divides the threads)
+    const float skip = c0 + own < d.inner ? a.skip[c0 + own] : 0.f;
     for (int t0 = 0; t0 < s.n; t0 += kTile) {
-        __syncthreads();
+        float cx[LX], cg[LX];
 #pragma unroll
-        for (int j = 0; j < LB; ++j) { const int i = tid + kScanThreads * j; if (i < 2 * BC) (&s_bc[0][0][0])[i] = rb[j]; }
+        for (int j = 0; j < LB; ++j) { const int i = tid + kScanThreads * j; if (i < 2 * BC) s_bc[i] = rb[j]; }
 #pragma unroll
         for (int j = 0; j < LX; ++j) {
             const int i = tid + kScanThreads * j;
-            if (i < XC) { (&s_dt[0][0])[i] = rd[j]; (&s_x[0][0])[i] = rx[j]; (&s_g[0][0])[i] = rg[j]; }
+            cx[j] = to_f(rx[j]); cg[j] = to_f(rg[j]) * a.factor;
+            if (i < XC) s_dx[i] = make_float2(rd[j], rd[j] * cx[j]);
         }
         __syncthreads();
         if (t0 + kTile < s.n) fetch(t0 + kTile);
         // tokens behind the segment have a step size of zero: they change nothing
+#pragma unroll 1
+        for (int h = 0; h < kTile && t0 + h < s.n; h += kHalf) {
+            float y[kHalf];
+            const float* b_at = s_bc + h * NP + n0;
+            const float2* d_at = s_dx + h * CB + cl;
 #pragma unroll
-        for (int t = 0; t < kTile; t += 4) {
-            float y[4];
-#pragma unroll
-            for (int q = 0; q < 4; ++q) {
-                const float step = s_dt[t + q][cl], dx = step * s_x[t + q][cl];
+            for (int q = 0; q < kHalf; ++q) {
+                const float2 dx = d_at[q * CB];
                 y[q] = 0.f;
 #pragma unroll
                 for (int i = 0; i < SP; i += 4) {
-                    const float4 b = get4(&s_bc[0][t + q][n0 + i]), cv = get4(&s_bc[1][t + q][n0 + i]);
-                    S.v[i] = fmaf(decay<T>(step * A.v[i]), S.v[i], dx * b.x);
-                    S.v[i + 1] = fmaf(decay<T>(step * A.v[i + 1]), S.v[i + 1], dx * b.y);
-                    S.v[i + 2] = fmaf(decay<T>(step * A.v[i + 2]), S.v[i + 2], dx * b.z);
-                    S.v[i + 3] = fmaf(decay<T>(step * A.v[i + 3]), S.v[i + 3], dx * b.w);
-                    y[q] = fmaf(S.v[i], cv.x, fmaf(S.v[i + 1], cv.y, fmaf(S.v[i + 2], cv.z, fmaf(S.v[i + 3], cv.w, y[q]))));
+                    const float4 b = get4(b_at + q * NP + i), cv = get4(b_at + BC + q * NP + i);
+                    S.v[i] = fmaf(decay<T>(dx.x * A.v[i]), S.v[i], dx.y * b.x);
+                    S.v[i + 1] = fmaf(decay<T>(dx.x * A.v[i + 1]), S.v[i + 1], dx.y * b.y);
+                    S.v[i + 2] = fmaf(decay<T>(dx.x * A.v[i + 2]), S.v[i + 2], dx.y * b.z);
+                    S.v[i + 3] = fmaf(decay<T>(dx.x * A.v[i + 3]), S.v[i + 3], dx.y * b.w);
+                    y[q] += fmaf(S.v[i], cv.x, S.v[i + 1] * cv.y) + fmaf(S.v[i + 2], cv.z, S.v[i + 3] * cv.w);
                 }
             }
-            if constexpr (G >= 2) {   // lanes with bit 0 go on with the tokens 2, 3
-                const bool up = sub & 1;
-                const float o0 = __shfl_xor_sync(0xffffffffu, up ? y[0] : y[2], 1), o1 = __shfl_xor_sync(0xffffffffu, up ? y[1] : y[3], 1);
-                y[0] = (up ? y[2] : y[0]) + o0; y[1] = (up ? y[3] : y[1]) + o1;
+            // sums over the group: with every bit of the lane's number it goes on with half of the tokens, as far as they go
+            int left = kHalf, first = 0;
+#pragma unroll
+            for (int o = 1; o < G; o <<= 1) {
+                if (left > 1) {
+                    left >>= 1;
+                    const bool up = sub & o;
+#pragma unroll
+                    for (int q = 0; q < kHalf / 2; ++q)
+                        if (q < left) {
+                            const float got = __shfl_xor_sync(0xffffffffu, up ? y[q] : y[q + left], o);
+                            y[q] = (up ? y[q + left] : y[q]) + got;
+                        }
+                    if (up) first += left;
+                } else y[0] += __shfl_xor_sync(0xffffffffu, y[0], o);
             }
-            if constexpr (G >= 4) {
-                const bool up = sub & 2;
-                const float o0 = __shfl_xor_sync(0xffffffffu, up ? y[0] : y[1], 2);
-                y[0] = (up ? y[1] : y[0]) + o0;
+            if (G <= kHalf || sub < kHalf)
 #pragma unroll
-                for (int o = 4; o < G; o <<= 1) y[0] += __shfl_xor_sync(0xffffffffu, y[0], o);
-                if (sub < 4) s_y[t + (sub & 1) * 2 + (sub >> 1)][cl] = y[0];
-            } else if constexpr (G == 2) { s_y[t + sub * 2][cl] = y[0]; s_y[t + sub * 2 + 1][cl] = y[1]; }
-            else
-#pragma unroll
-                for (int q = 0; q < 4; ++q) s_y[t + q][cl] = y[q];
+                for (int q = 0; q < kHalf; ++q) if (q < left) s_y[(h + first + q) * CB + cl] = y[q];
         }
         __syncthreads();
 #pragma unroll
         for (int j = 0; j < LX; ++j) {
-            const int i = tid + kScanThreads * j, t = i / CB, k = i % CB;
-            if (i < XC && t0 + t < s.n && c0 + k < d.inner) out[size_t(t0 + t) * a.out_ld + k] = to_t<T>(fmaf(skip[j], s_x[t][k], s_y[t][k]) * s_g[t][k]);
+            const int i = tid + kScanThreads * j, t = i / CB;
+            if (i < XC && t0 + t < s.n && c0 + own < d.inner) out[size_t(t0 + t) * a.out_ld + own] = to_t<T>(fmaf(skip, cx[j], s_y[i]) * cg[j]);
         }
     }
     if (ok) S.store(at, n, whole);
@@ -280,7 +336,9 @@ int32_t selective_conv(const SelectiveDims& d, int dtype, const SelectiveArgs& a
             FORGE_LAUNCH_CHECK();
         }
         if (t.n > 0) {
-            conv_segments_kernel<T><<<dim3((t.max_n + kRun - 1) / kRun, (d.inner + 127) / 128, t.n), 128, 0, st>>>(d, a, t.segs);
+            const bool eight = std::is_same<T, __nv_bfloat16>::value && d.inner % 8 == 0 && a.in_ld % 8 == 0 && a.x_ld % 8 == 0 && d.taps <= 4;
+            if (eight) conv_segments8_kernel<<<dim3((t.max_n + kRun8 - 1) / kRun8, (d.inner + 1023) / 1024, t.n), 128, 0, st>>>(d, a, t.segs);
+            else conv_segments_kernel<T><<<dim3((t.max_n + kRun - 1) / kRun, (d.inner + 127) / 128, t.n), 128, 0, st>>>(d, a, t.segs);
             FORGE_LAUNCH_CHECK();
         }
         return FORGE_OK;
@@ -304,7 +362,9 @@ int32_t selective_segments(const SelectiveDims& d, int dtype, const SelectiveArg
     return with_group(d.state, [&](auto g, auto sp) -> int32_t {
         constexpr int G = decltype(g)::value, SP = decltype(sp)::value, CB = kScanThreads / G;
         auto kern = dtype == FORGE_F32 ? selective_scan_kernel<float, G, SP> : selective_scan_kernel<__nv_bfloat16, G, SP>;
-        kern<<<dim3((d.inner + CB - 1) / CB, t.n), kScanThreads, 0, st>>>(d, a, t.segs);
+        const size_t smem = size_t(kTile) * (2 * G * SP + 3 * CB) * sizeof(float);
+        if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+        kern<<<dim3((d.inner + CB - 1) / CB, t.n), kScanThreads, smem, st>>>(d, a, t.segs);
         FORGE_LAUNCH_CHECK();
         return FORGE_OK;
     });

@@ -624,7 +624,7 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
         {&S.scores, scores}, {&S.joint, joint}, {&S.blocks, blocks}, {&S.scan, scan}, {&S.bc, bc}};
     for (const auto& e : sizes) FORGE_TRY(grow(m, *e.first, e.second));
     // one ticket per output tile of the largest product (128 rows x at least 16 tokens)
-    const size_t tiles = ((n_max + 127) / 128) * std::max<size_t>(1, (size_t(std::max(rows, ctx_rows)) + 127) / 128);
+    const size_t tiles = std::max<size_t>(256, ((n_max + 127) / 128) * std::max<size_t>(1, (size_t(std::max(rows, ctx_rows)) + 127) / 128));
     if (tiles > S.scratch.tickets_cap) {
         FORGE_TRY(dev_alloc(m, &S.scratch.tickets, tiles));
         FORGE_CUDA(cudaMemsetAsync(S.scratch.tickets, 0, tiles * sizeof(int), m->stream));
@@ -1316,10 +1316,14 @@ size_t stack_kv_bytes_per_token(const ForgeKV* kv) {
     }
     return n * dense_size(S.dtype);
 }
-size_t stack_kv_bytes_per_seq(const ForgeKV* kv) {
+size_t stack_kv_bytes(const ForgeKV* kv, int len) {
     const StackModel& S = *kv->model->stack;
     size_t n = S.spec.buckets ? sizeof(uint32_t) : 0;
-    for (const LayerRun& r : S.spec.runs) { const LayerSpec& L = S.spec.layers[r.layer]; n += state_bytes(L) + ring_bytes(S, L) + prev_bytes(S, L); }
+    const size_t pages = size_t(len + FORGE_KV_PAGE - 1) / FORGE_KV_PAGE;
+    for (const LayerRun& r : S.spec.runs) {
+        const LayerSpec& L = S.spec.layers[r.layer];
+        n += (size_t(len) + pages * size_t(L.page_rows() - FORGE_KV_PAGE)) * L.cache_row() * dense_size(S.dtype) + state_bytes(L) + ring_bytes(S, L) + prev_bytes(S, L);
+    }
     return n;
 }
 
