@@ -41,13 +41,6 @@ template <typename T> __device__ __forceinline__ float act_sigmoid(float x, floa
     if constexpr (sizeof(T) == 2) return __fdividef(x, 1.0f + __expf(-v));
     else return x / (1.0f + expf(-v));
 }
-// step sizes and logarithms of decays of bfloat16 models: log(1 + u) with u = exp(-|v|) by its series where u is small (log near one has no relative accuracy)
-template <typename T> __device__ __forceinline__ float act_softplus(float v) {
-    if constexpr (sizeof(T) == 4) return softplus(v);
-    const float u = __expf(-fabsf(v));
-    const float series = u * fmaf(u, fmaf(u, fmaf(u, fmaf(u, fmaf(u, -1.f / 6.f, 0.2f), -0.25f), 1.f / 3.f), -0.5f), 1.f);
-    return fmaxf(v, 0.f) + (u < 0.0625f ? series : __logf(1.f + u));
-}
 template <typename T> __device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
     return act_sigmoid<T>(g, 1.702f * g) * (u + 1.0f);
@@ -148,7 +141,7 @@ __device__ __forceinline__ float put_one(const RowOut<T>& g, const Leave<T>& n, 
         case SEG_SILU: *h = to_t<T>(act_sigmoid<T>(v, v)); break;
         case SEG_TANH: *h = to_t<T>(tanhf(v)); break;
         case SEG_SIGMOID_F32: *f = sigmoid(v); break;
-        case SEG_DECAY: *f = -g.mul * act_softplus<T>(v); break;
+        case SEG_DECAY: *f = -g.mul * softplus(v); break;
         case SEG_EXP_DECAY: *f = -expf(v); break;
         case SEG_RESID: {
             const float x = n.enter((g.fresh ? 0.f : old_known ? old : *f) + v, t);
@@ -539,7 +532,7 @@ __global__ void __launch_bounds__(kThreads<NT>, NT <= 16 ? 2 : 1) gemm_dense_ker
                     case SEG_SILU: put_t([](float x) { return act_sigmoid<__nv_bfloat16>(x, x); }); break;
                     case SEG_TANH: put_t([](float x) { return tanhf(x); }); break;
                     case SEG_SIGMOID_F32: put_f([](float x) { return sigmoid(x); }); break;
-                    case SEG_DECAY: put_f([&](float x) { return -g.mul * act_softplus<__nv_bfloat16>(x); }); break;
+                    case SEG_DECAY: put_f([&](float x) { return -g.mul * softplus(x); }); break;
                     case SEG_EXP_DECAY: put_f([&](float x) { return -expf(x); }); break;
                     default: put_f([](float x) { return x; });
                 }
@@ -889,9 +882,13 @@ int32_t dense_gemm(const DenseWeight& w, const void* act, int act_ld, int m, con
     p.pitch = w.pitch() / BK; p.k_off = w.col0 / BK;
     const int sms = sm_count();
     int nt = group_tile_rows(m);
-    for (; nt > 32; nt /= 2) {   // where few whole tiles would leave SMs idle: narrower ones
-        const long long tiles = (long long)((w.N + 127) / 128) * ((m + nt - 1) / nt);
-        if (tiles * 2 > sms || p.nk > tiles * p.nk / sms + nt * kShareSteps / 256) break;
+    const long long row_tiles = (w.N + 127) / 128;
+    if (nt > 32 && row_tiles * ((m + nt - 1) / nt) * 2 <= sms) {   // wide tiles would leave SMs idle or share most of their steps: the width whose longest CTA moves least
+        auto moved = [&](int n) {
+            const long long tiles = row_tiles * ((m + n - 1) / n), steps = tiles > sms ? (tiles + sms - 1) / sms * p.nk : std::min<long long>(p.nk, tiles * p.nk / sms + n * kShareSteps / 256);
+            return steps * (128 + n);
+        };
+        for (int n = nt / 2; n >= 32; n /= 2) if (moved(n) < moved(nt)) nt = n;
     }
     if (out.scale.sums && out.scale.parts > 1 && nt > kScaleRows) { set_error("dense product: %d tokens with scales in parts", m); return FORGE_ERR_SHAPE; }
     if (size_t((w.N + 127) / 128) * ((m + nt - 1) / nt) > sc.tickets_cap) { set_error("dense product: too many tiles for the ticket array"); return FORGE_ERR_SHAPE; }

@@ -20,7 +20,8 @@ struct SelectiveArgs {
     void* x = nullptr; int x_ld = 0;                       // T rows [inner] behind it
     const float* bc = nullptr; int bc_ld = 0;              // f32 rows [B | C]
     const float* dt = nullptr; int dt_ld = 0;              // f32 rows [inner]: step sizes
-    // or, for single tokens, the projection that forms them: T rows of low_k values per channel over low[row]; a step size is softplus(z + dt_add)
+    // or the projection that forms them (single tokens; segments if selective_steps_inside): T rows of low_k values per channel over low[row]; a step size is
+    // softplus(z + dt_add)
     const void* dt_w = nullptr; const void* low = nullptr; int low_ld = 0, low_k = 0;
     const float* dt_add = nullptr;
     const float* a2 = nullptr;                             // [inner][state]: A in the base of exp2
@@ -34,7 +35,8 @@ struct SelectiveArgs {
 bool selective_supported(const SelectiveDims& d);
 // the convolution of single tokens (rows) and of segments
 int32_t selective_conv(const SelectiveDims& d, int dtype, const SelectiveArgs& a, const StepRows& ones, const SegTable& t, cudaStream_t st);
-// the recurrence of single tokens, and of segments of any length (these take step sizes from dt)
+bool selective_steps_inside(int dtype, int low_k);
+// the recurrence of single tokens, and of segments of any length
 int32_t selective_decode(const SelectiveDims& d, int dtype, const SelectiveArgs& a, const StepRows& ones, cudaStream_t st);
 int32_t selective_segments(const SelectiveDims& d, int dtype, const SelectiveArgs& a, const SegTable& t, cudaStream_t st);
 

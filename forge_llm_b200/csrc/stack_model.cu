@@ -995,7 +995,8 @@ struct Sequence {
             o.add(SEG_F32, w.bc_row, 2 * d.state, S.bc.p, 2 * d.state);
             FORGE_TRY(gemm(w.scan_in, xc, inner_p, o));
         }
-        if (all_ones() && n <= kFewSteps) {
+        // formed inside the recurrence, if every kernel of the step can
+        if (all_ones() || selective_steps_inside(dt, w.low.K)) {
             a.dt_w = w.low.w; a.low = S.low.p; a.low_ld = a.low_k = w.low.K; a.dt_add = w.decay_add;
         } else {   // softplus: the epilogue of decays with a factor of minus one
             DenseOut o;
@@ -1009,7 +1010,6 @@ struct Sequence {
         FORGE_TRY(attend(L, w, run, w.out.K, L.left_scale, nullptr));
         return post_out(w, after);
     }
-    static constexpr int kFewSteps = 4;   // single tokens whose step sizes are formed inside the recurrence
 
     // x += norm2(shared expert + experts + what is passed on); see experts() for few and many tokens
     int32_t mixture(const LayerSpec& L, const LayerWeights& w, const After& after) {

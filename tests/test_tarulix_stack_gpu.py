@@ -145,7 +145,7 @@ def test_pooled_attention_with_mixed_heads_alone(root, dtype, name):
     m.close()
 
 
-SCAN = {"small": (72, 16, 12, 4), "one": (8, 1, 1, 1), "odd": (37, 5, 3, 5), "wide": (320, 64, 96, 4), "beyond": (40, 250, 70, 16), "whole": (64, 32, 64, 2), "lanes": (33, 128, 8, 3), "eight": (48, 8, 20, 4)}
+SCAN = {"small": (72, 16, 12, 4), "one": (8, 1, 1, 1), "odd": (37, 5, 3, 5), "wide": (320, 64, 96, 4), "beyond": (40, 250, 70, 16), "whole": (64, 32, 64, 2), "lanes": (33, 128, 8, 3), "eight": (48, 8, 20, 4), "ranks": (24, 16, 200, 4), "far_ranks": (16, 4, 300, 2)}
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
