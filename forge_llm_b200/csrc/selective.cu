@@ -138,19 +138,9 @@ __global__ void __launch_bounds__(128) conv_segments8_kernel(const SelectiveDims
 }
 
 // ------------------------------------------------------------------------------------------------ recurrence
-// two f32 operations by one instruction
-__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
-    float2 r;
-    asm("{\n.reg .b64 x, y;\nmov.b64 x, {%2, %3};\nmov.b64 y, {%4, %5};\nmul.rn.f32x2 x, x, y;\nmov.b64 {%0, %1}, x;\n}" : "=f"(r.x), "=f"(r.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
-    return r;
-}
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-    float2 r;
-    asm("{\n.reg .b64 x, y, z;\nmov.b64 x, {%2, %3};\nmov.b64 y, {%4, %5};\nmov.b64 z, {%6, %7};\nfma.rn.f32x2 x, x, y, z;\nmov.b64 {%0, %1}, x;\n}"
-        : "=f"(r.x), "=f"(r.y)
-        : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
-    return r;
-}
+// (by one instruction for both they are slower here: its latency counts, with few warps per SM)
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) { return make_float2(a.x * b.x, a.y * b.y); }
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) { return make_float2(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y)); }
 template <int SP> struct States {   // states sub * SP .. of a channel, in pairs
     float2 v[SP / 2];
     __device__ __forceinline__ void load(const float* p, int n) {   // n: how many there are
@@ -175,11 +165,11 @@ template <int SP> struct States {   // states sub * SP .. of a channel, in pairs
     }
 };
 
-constexpr int kScanThreads = 128;
+constexpr int kDecodeThreads = 128;
 
 template <typename T, int G, int SP>
-__global__ void __launch_bounds__(kScanThreads) selective_decode_kernel(const SelectiveDims d, const SelectiveArgs a, const StepRows rows) {
-    constexpr int CB = kScanThreads / G;
+__global__ void __launch_bounds__(kDecodeThreads) selective_decode_kernel(const SelectiveDims d, const SelectiveArgs a, const StepRows rows) {
+    constexpr int CB = kDecodeThreads / G;
     const int r = blockIdx.y, sub = threadIdx.x % G, c = blockIdx.x * CB + threadIdx.x / G;
     const bool ok = c < d.inner;
     const int cc = ok ? c : 0, n0 = sub * SP, n = max(0, d.state - n0);
@@ -233,22 +223,22 @@ __global__ void __launch_bounds__(kScanThreads) selective_decode_kernel(const Se
 }
 
 constexpr int kTile = 32, kHalf = 16, kGroup = 4;     // tokens whose inputs are in shared memory, whose read-outs are in registers, whose factors are formed together
-// What a CTA holds in shared memory: two tiles of B and C, step sizes, x and gates, one of read-outs, and (KS > 0) two of the step sizes' inner values.
-template <typename T, int G, int SP, int KS> struct ScanSmem {
-    static constexpr int CB = kScanThreads / G, NP = G * SP, BC = kTile * NP, XC = kTile * CB, LD = KS * 16 + 8;
-    static constexpr size_t X = (4 * size_t(BC) + 3 * XC) * 4, LOW = X + 4 * size_t(XC) * sizeof(T), BYTES = LOW + (KS ? 2 * size_t(kTile) * LD * 2 : 0);
+// What a CTA holds in shared memory: three tiles of B and C, step sizes, x and gates, and (KS > 0) the step sizes' inner values, one of read-outs.
+template <typename T, int TH, int G, int SP, int KS> struct ScanSmem {
+    static constexpr int CB = TH / G, NP = G * SP, BC = kTile * NP, XC = kTile * CB, LD = KS * 16 + 8;
+    static constexpr size_t X = (6 * size_t(BC) + 4 * XC) * 4, LOW = X + 6 * size_t(XC) * sizeof(T), BYTES = LOW + (KS ? 3 * size_t(kTile) * LD * 2 : 0);
 };
 // KS > 0: step sizes are formed here, from inner values of 16 KS columns, on the tensor cores.  ASYNC: all rows are copied in 16-byte pieces (bfloat16, channels in
 // eights, states in fours).
-template <typename T, int G, int SP, int KS, bool ASYNC>
-__global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const SelectiveDims d, const SelectiveArgs a, const ScanSeg* __restrict__ segs) {
-    using L = ScanSmem<T, G, SP, KS>;
+template <typename T, int TH, int G, int SP, int KS, bool ASYNC>
+__global__ void __launch_bounds__(TH) selective_scan_kernel(const SelectiveDims d, const SelectiveArgs a, const ScanSeg* __restrict__ segs) {
+    using L = ScanSmem<T, TH, G, SP, KS>;
     constexpr int CB = L::CB, NP = L::NP, BC = L::BC, XC = L::XC;   // channels per CTA, padded states
     extern __shared__ __align__(16) unsigned char sm[];
-    float* const s_bc = reinterpret_cast<float*>(sm);     // [2][B | C][kTile][NP]
-    float* const s_dt = s_bc + 4 * BC;                    // [2][kTile][CB]
-    float* const s_y = s_dt + 2 * XC;                     // [kTile][CB]
-    T* const s_x = reinterpret_cast<T*>(sm + L::X);       // [2][x | gate][kTile][CB]
+    float* const s_bc = reinterpret_cast<float*>(sm);     // [3][B | C][kTile][NP]
+    float* const s_dt = s_bc + 6 * BC;                    // [3][kTile][CB]
+    float* const s_y = s_dt + 3 * XC;                     // [kTile][CB]
+    T* const s_x = reinterpret_cast<T*>(sm + L::X);       // [3][x | gate][kTile][CB]
     const uint32_t s_low = uint32_t(__cvta_generic_to_shared(sm + L::LOW));
     const ScanSeg s = segs[blockIdx.y];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, sub = tid % G, cl = tid / G, c0 = blockIdx.x * CB, c = c0 + cl;
@@ -273,37 +263,37 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Sele
         if (ASYNC) {
             const uint32_t x_at = uint32_t(__cvta_generic_to_shared(s_x + buf * 2 * XC)), bc_at = uint32_t(__cvta_generic_to_shared(s_bc + buf * 2 * BC));
             constexpr int XP = CB >= 8 ? CB / 8 : 1, BP = NP / 4;   // pieces per row
-            for (int i = tid; i < 2 * kTile * XP; i += kScanThreads) {
+            for (int i = tid; i < 2 * kTile * XP; i += TH) {
                 const int which = i / (kTile * XP), t = i / XP % kTile, k = i % XP * 8;
                 const bool in = t0 + t < s.n && c0 + k < d.inner;
                 const T* src = which ? gate + size_t(in ? t0 + t : 0) * a.gate_ld : x + size_t(in ? t0 + t : 0) * a.x_ld;
                 cp_async16(x_at + uint32_t(which * XC + t * CB + k) * 2, src + (in ? k : 0), in);
             }
-            for (int i = tid; i < 2 * kTile * BP; i += kScanThreads) {
+            for (int i = tid; i < 2 * kTile * BP; i += TH) {
                 const int which = i / (kTile * BP), t = i / BP % kTile, k = i % BP * 4;
                 const bool in = t0 + t < s.n && k < d.state;
                 cp_async16(bc_at + uint32_t(which * BC + t * NP + k) * 4, bc + size_t(in ? t0 + t : 0) * a.bc_ld + (in ? which * d.state + k : 0), in);
             }
         } else {
-            for (int i = tid; i < XC; i += kScanThreads) {
+            for (int i = tid; i < XC; i += TH) {
                 const int t = i / CB, k = i % CB;
                 const bool in = t0 + t < s.n && c0 + k < d.inner;
                 s_x[buf * 2 * XC + i] = in ? x[size_t(t0 + t) * a.x_ld + k] : to_t<T>(0.f);
                 s_x[buf * 2 * XC + XC + i] = in ? gate[size_t(t0 + t) * a.gate_ld + k] : to_t<T>(0.f);
             }
-            for (int i = tid; i < 2 * BC; i += kScanThreads) {
+            for (int i = tid; i < 2 * BC; i += TH) {
                 const int which = i / BC, t = i % BC / NP, k = i % NP;
                 s_bc[buf * 2 * BC + i] = t0 + t < s.n && k < d.state ? bc[size_t(t0 + t) * a.bc_ld + which * d.state + k] : 0.f;
             }
         }
         if constexpr (KS > 0) {
-            for (int i = tid; i < kTile * KS * 2; i += kScanThreads) {
+            for (int i = tid; i < kTile * KS * 2; i += TH) {
                 const int t = i / (KS * 2), k = i % (KS * 2) * 8;
                 const bool in = t0 + t < s.n;
                 cp_async16(s_low + uint32_t((buf * kTile + t) * L::LD + k) * 2, low + size_t(in ? t0 + t : 0) * a.low_ld + k, in);
             }
         } else {
-            for (int i = tid; i < XC; i += kScanThreads) {
+            for (int i = tid; i < XC; i += TH) {
                 const int t = i / CB, k = i % CB;
                 s_dt[buf * XC + i] = t0 + t < s.n && c0 + k < d.inner ? dt[size_t(t0 + t) * a.dt_ld + k] : 0.f;
             }
@@ -311,28 +301,28 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Sele
         cp_commit();
     };
     // step sizes on the tensor cores: 16 tokens by eight channels per tile; a warp keeps its channels' weights
-    constexpr int NTILES = (CB + 7) / 8, PER = (NTILES + 3) / 4;
+    constexpr int WARPS = TH / 32, NTILES = (CB + 7) / 8, PER = (NTILES + WARPS - 1) / WARPS;
     uint32_t wf[KS ? PER : 1][KS ? KS : 1][2];
     float dt_add[PER][2];
     if constexpr (KS > 0)
 #pragma unroll
         for (int p = 0; p < PER; ++p) {
-            const int ch = (warp + 4 * p) * 8 + (lane >> 2), lc = (lane & 3) * 2;
-            const bool in = warp + 4 * p < NTILES && c0 + ch < d.inner && ch < CB;
+            const int ch = (warp + WARPS * p) * 8 + (lane >> 2), lc = (lane & 3) * 2;
+            const bool in = warp + WARPS * p < NTILES && c0 + ch < d.inner && ch < CB;
             const T* w = static_cast<const T*>(a.dt_w) + size_t(in ? c0 + ch : 0) * a.low_k;
 #pragma unroll
             for (int k = 0; k < KS; ++k)
 #pragma unroll
                 for (int h = 0; h < 2; ++h) wf[p][k][h] = in ? *reinterpret_cast<const uint32_t*>(w + k * 16 + h * 8 + lc) : 0u;
 #pragma unroll
-            for (int e = 0; e < 2; ++e) { const int own = c0 + (warp + 4 * p) * 8 + lc + e; dt_add[p][e] = own < d.inner ? a.dt_add[own] : 0.f; }
+            for (int e = 0; e < 2; ++e) { const int own = c0 + (warp + WARPS * p) * 8 + lc + e; dt_add[p][e] = own < d.inner ? a.dt_add[own] : 0.f; }
         }
     auto step_sizes = [&](int t0, int buf) {
         if constexpr (KS > 0) {
             const SmemMat m{s_low + uint32_t(buf * kTile * L::LD) * 2, L::LD};
 #pragma unroll
             for (int p = 0; p < PER; ++p) {
-                if (warp + 4 * p >= NTILES) continue;
+                if (warp + WARPS * p >= NTILES) continue;
                 float z[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
                 for (int k = 0; k < KS; ++k)
@@ -346,7 +336,7 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Sele
                 for (int h = 0; h < 2; ++h)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
-                        const int t = h * 16 + (lane >> 2) + (e >> 1) * 8, k = (warp + 4 * p) * 8 + (lane & 3) * 2 + (e & 1);
+                        const int t = h * 16 + (lane >> 2) + (e >> 1) * 8, k = (warp + WARPS * p) * 8 + (lane & 3) * 2 + (e & 1);
                         if (k < CB) s_dt[buf * XC + t * CB + k] = t0 + t < s.n ? fast_softplus(z[h][e] + dt_add[p][e & 1]) : 0.f;
                     }
             }
@@ -361,10 +351,11 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Sele
         step_sizes(0, 0);
     }
     if (s.n > kTile) fetch(kTile, 1);
-    for (int t0 = 0, buf = 0; t0 < s.n; t0 += kTile, buf ^= 1) {
-        cp_wait<0>();
+    for (int t0 = 0, buf = 0, next_buf = 1, free_buf = 2; t0 < s.n; t0 += kTile) {
+        cp_wait<0>();      // the tile behind this one, requested a tile ago
         __syncthreads();
-        if (t0 + kTile < s.n) step_sizes(t0 + kTile, buf ^ 1);
+        if (t0 + 2 * kTile < s.n) fetch(t0 + 2 * kTile, free_buf);
+        if (t0 + kTile < s.n) step_sizes(t0 + kTile, next_buf);
         // tokens behind the segment have a step size of zero: they change nothing
 #pragma unroll 1
         for (int h = 0; h < kTile && t0 + h < s.n; h += kHalf) {
@@ -425,15 +416,13 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Sele
         __syncthreads();
         if (c0 + own < d.inner)
 #pragma unroll 4
-            for (int i = tid; i < XC; i += kScanThreads) {
+            for (int i = tid; i < XC; i += TH) {
                 const int t = i / CB;
                 const T *xs = s_x + buf * 2 * XC + i;
                 if (t0 + t < s.n) out[size_t(t0 + t) * a.out_ld + own] = to_t<T>(fmaf(skip, to_f(xs[0]), s_y[i]) * (to_f(xs[XC]) * a.factor));
             }
-        if (t0 + 2 * kTile < s.n) {
-            __syncthreads();    // the buffer is read
-            fetch(t0 + 2 * kTile, buf);
-        }
+        const int done = buf;
+        buf = next_buf; next_buf = free_buf; free_buf = done;
     }
     if (ok) {
         if (whole) S.store_pairs(at);
@@ -456,27 +445,27 @@ int32_t with_group(int states, F go) {
     return go(integral_constant<int, 32>{}, integral_constant<int, 8>{});
 }
 
-template <typename T, int G, int SP, int KS, bool ASYNC>
+template <typename T, int TH, int G, int SP, int KS, bool ASYNC>
 int32_t launch_scan(const SelectiveDims& d, const SelectiveArgs& a, const SegTable& t, cudaStream_t st) {
-    constexpr int CB = kScanThreads / G;
-    constexpr size_t smem = ScanSmem<T, G, SP, KS>::BYTES;
-    auto kern = selective_scan_kernel<T, G, SP, KS, ASYNC>;
+    constexpr int CB = TH / G;
+    constexpr size_t smem = ScanSmem<T, TH, G, SP, KS>::BYTES;
+    auto kern = selective_scan_kernel<T, TH, G, SP, KS, ASYNC>;
     if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
-    kern<<<dim3((d.inner + CB - 1) / CB, t.n), kScanThreads, smem, st>>>(d, a, t.segs);
+    kern<<<dim3((d.inner + CB - 1) / CB, t.n), TH, smem, st>>>(d, a, t.segs);
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }
-template <int G, int SP, int KS>
+template <int TH, int G, int SP, int KS>
 int32_t scan_steps(const SelectiveDims& d, const SelectiveArgs& a, const SegTable& t, cudaStream_t st) {
     using bf16 = __nv_bfloat16;
-    const bool pieces = d.inner % 8 == 0 && kScanThreads / G >= 8 && a.x_ld % 8 == 0 && a.gate_ld % 8 == 0 && d.state % 4 == 0;
-    return pieces ? launch_scan<bf16, G, SP, KS, true>(d, a, t, st) : launch_scan<bf16, G, SP, KS, false>(d, a, t, st);
+    const bool pieces = d.inner % 8 == 0 && TH / G >= 8 && a.x_ld % 8 == 0 && a.gate_ld % 8 == 0 && d.state % 4 == 0;
+    return pieces ? launch_scan<bf16, TH, G, SP, KS, true>(d, a, t, st) : launch_scan<bf16, TH, G, SP, KS, false>(d, a, t, st);
 }
-template <int G, int SP>
+template <int TH, int G, int SP>
 int32_t scan_segments(const SelectiveDims& d, int dtype, const SelectiveArgs& a, const SegTable& t, cudaStream_t st) {
-    if (dtype == FORGE_F32) return launch_scan<float, G, SP, 0, false>(d, a, t, st);
-    if (!a.dt_w) return scan_steps<G, SP, 0>(d, a, t, st);
-    return a.low_k == 64 ? scan_steps<G, SP, 4>(d, a, t, st) : a.low_k == 128 ? scan_steps<G, SP, 8>(d, a, t, st) : scan_steps<G, SP, 16>(d, a, t, st);
+    if (dtype == FORGE_F32) return launch_scan<float, TH, G, SP, 0, false>(d, a, t, st);
+    if (!a.dt_w) return scan_steps<TH, G, SP, 0>(d, a, t, st);
+    return a.low_k == 64 ? scan_steps<TH, G, SP, 4>(d, a, t, st) : a.low_k == 128 ? scan_steps<TH, G, SP, 8>(d, a, t, st) : scan_steps<TH, G, SP, 16>(d, a, t, st);
 }
 
 }  // namespace
@@ -505,9 +494,9 @@ int32_t selective_conv(const SelectiveDims& d, int dtype, const SelectiveArgs& a
 int32_t selective_decode(const SelectiveDims& d, int dtype, const SelectiveArgs& a, const StepRows& ones, cudaStream_t st) {
     if (ones.n <= 0) return FORGE_OK;
     return with_group(d.state, [&](auto g, auto sp) -> int32_t {
-        constexpr int G = decltype(g)::value, SP = decltype(sp)::value, CB = kScanThreads / G;
+        constexpr int G = decltype(g)::value, SP = decltype(sp)::value, CB = kDecodeThreads / G;
         auto kern = dtype == FORGE_F32 ? selective_decode_kernel<float, G, SP> : selective_decode_kernel<__nv_bfloat16, G, SP>;
-        FORGE_CUDA(launch_pdl(kern, dim3((d.inner + CB - 1) / CB, ones.n), dim3(kScanThreads), 0, st, d, a, ones));
+        FORGE_CUDA(launch_pdl(kern, dim3((d.inner + CB - 1) / CB, ones.n), dim3(kDecodeThreads), 0, st, d, a, ones));
         FORGE_LAUNCH_CHECK();
         return FORGE_OK;
     });
@@ -515,7 +504,7 @@ int32_t selective_decode(const SelectiveDims& d, int dtype, const SelectiveArgs&
 
 int32_t selective_segments(const SelectiveDims& d, int dtype, const SelectiveArgs& a, const SegTable& t, cudaStream_t st) {
     if (t.n <= 0) return FORGE_OK;
-    return with_group(d.state, [&](auto g, auto sp) -> int32_t { return scan_segments<decltype(g)::value, decltype(sp)::value>(d, dtype, a, t, st); });
+    return with_group(d.state, [&](auto g, auto sp) -> int32_t { return scan_segments<(decltype(g)::value >= 8 ? 256 : 128), decltype(g)::value, decltype(sp)::value>(d, dtype, a, t, st); });
 }
 
 }  // namespace forge
