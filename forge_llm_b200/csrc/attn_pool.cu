@@ -11,26 +11,8 @@ __global__ void __launch_bounds__(128) pool_blocks_kernel(const AttnDims d, T* c
     const int r = blockIdx.x, pos = rows.pos[r], seq = rows.seq ? rows.seq[r] : r;
     pdl_trigger();
     pdl_wait();
-    if ((pos + 1) % d.pool) return;
-    const int b = pos / d.pool, t0 = b * d.pool;
     const int32_t* pt = rows.page_table + size_t(seq) * rows.pages_per_seq;
-    const size_t W = d.row();
-    T* dst = cache + d.block_row(pt, b) * W;
-    const float inv = 1.0f / float(d.pool);
-    for (int c = threadIdx.x * 8; c < int(W); c += 128 * 8) {
-        float sum[8];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) sum[e] = 0.f;
-#pragma unroll 8
-        for (int t = t0; t < t0 + d.pool; ++t) {
-            float v[8];
-            load8(v, cache + (size_t(pt[t / FORGE_KV_PAGE]) * FORGE_KV_PAGE + t % FORGE_KV_PAGE) * W + c);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) sum[e] += v[e];
-        }
-        put4(dst + c, make_float4(sum[0] * inv, sum[1] * inv, sum[2] * inv, sum[3] * inv));
-        put4(dst + c + 4, make_float4(sum[4] * inv, sum[5] * inv, sum[6] * inv, sum[7] * inv));
-    }
+    for (int c = 0; c < d.row(); c += 128 * 8) pool_columns(d, cache, pt, pos, c, min(128, (d.row() - c) / 8));
 }
 
 // Rows that are no block yet become zeros: their weights are zero, so they must be finite.

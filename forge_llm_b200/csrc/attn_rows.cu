@@ -418,10 +418,14 @@ int32_t run_mma(const AttnDims& d, const void* q, const void* cache, const float
 constexpr int kQkDims = 16;   // values per lane at most
 template <typename T>
 __global__ void __launch_bounds__(256) qk_post_kernel(const AttnDims d, const QkPost p, const float* proj, int ldp, int k_col, const float* __restrict__ q_norm,
-                                                      const float* __restrict__ k_norm, const float2* __restrict__ rope, T* q, T* cache, const int32_t* place, const StepRows rows, const RouteBeside route) {
+                                                      const float* __restrict__ k_norm, const float2* __restrict__ rope, T* q, T* cache, const int32_t* place, const StepRows rows, const RouteBeside route, const ConvBeside conv) {
     extern __shared__ float sm[];
     __shared__ float red[2][8];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = blockIdx.y, h = blockIdx.x * 8 + warp;
+    if (conv.blocks && int(blockIdx.x) >= int(gridDim.x) - conv.blocks) {
+        conv_one<T>(conv.d, conv.a, rows, r, (int(blockIdx.x) - int(gridDim.x) + conv.blocks) * 256 + int(threadIdx.x));
+        return;
+    }
     if (route.logits && blockIdx.x == gridDim.x - 1) {
         if (r > 0) return;
         pdl_trigger();
@@ -493,10 +497,14 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
 __device__ __forceinline__ float sum4(float4 v) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))); }
 template <typename T, int P, int R>   // R: rows per CTA, whose loads are in flight together
 __global__ void __launch_bounds__(256) qk_post4_kernel(const AttnDims d, const QkPost p, const float* proj, int ldp, int k_col, const float* __restrict__ q_norm,
-                                                       const float* __restrict__ k_norm, const float2* __restrict__ rope, T* q, T* cache, const int32_t* place, const StepRows rows, const RouteBeside route) {
+                                                       const float* __restrict__ k_norm, const float2* __restrict__ rope, T* q, T* cache, const int32_t* place, const StepRows rows, const RouteBeside route, const ConvBeside conv) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float red[R][2][8];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = blockIdx.y * R, h = blockIdx.x * 8 + warp;
+    if (conv.blocks && int(blockIdx.x) >= int(gridDim.x) - conv.blocks) {
+        for (int r = r0; r < min(r0 + R, rows.n); ++r) conv_one<T>(conv.d, conv.a, rows, r, (int(blockIdx.x) - int(gridDim.x) + conv.blocks) * 256 + int(threadIdx.x));
+        return;
+    }
     if (route.logits && blockIdx.x == gridDim.x - 1) {
         if (r0 > 0) return;
         pdl_trigger();
@@ -609,13 +617,16 @@ __global__ void __launch_bounds__(256) qk_post4_kernel(const AttnDims d, const Q
 }  // namespace
 
 int32_t qk_post(const AttnDims& d, const QkPost& p, int dtype, const float* proj, int ldp, int k_col, const float* q_norm, const float* k_norm, const float* rope, void* q, void* cache,
-                const int32_t* place, const StepRows& rows, const RouteBeside* route, cudaStream_t st) {
+                const int32_t* place, const StepRows& rows, const RouteBeside* route, const ConvBeside* conv, cudaStream_t st) {
     if (rows.n <= 0) return FORGE_OK;
     if (route && (rows.n > kScaleRows || route->d.choices() > kMaxExperts)) { set_error("routing: %d rows, %d experts", rows.n, route->d.experts); return FORGE_ERR_SHAPE; }
+    if ((route && conv) || (conv && rows.n > 65535)) { set_error("queries and keys: nothing more fits beside them"); return FORGE_ERR_SHAPE; }
     if (d.dim > kQkDims * 32 || p.rot_dims > d.dim || p.rot_dims % 2) { set_error("attention: head size %d with %d rotated dimensions", d.dim, p.rot_dims); return FORGE_ERR_SHAPE; }
     auto go = [&](auto t) -> int32_t {
         using T = decltype(t);
         const RouteBeside beside = route ? *route : RouteBeside{};
+        ConvBeside scan = conv ? *conv : ConvBeside{};
+        if (conv) scan.blocks = (conv->d.inner + 255) / 256;
         for (int r0 = 0; r0 < rows.n; r0 += 65535) {
             StepRows part = rows;
             part.n = std::min(65535, rows.n - r0);
@@ -625,8 +636,8 @@ int32_t qk_post(const AttnDims& d, const QkPost& p, int dtype, const float* proj
             auto kern = !four ? qk_post_kernel<T> : per == 4 ? qk_post4_kernel<T, 1, 4> : d.dim <= 128 ? qk_post4_kernel<T, 1, 1> : d.dim <= 256 ? qk_post4_kernel<T, 2, 1> : qk_post4_kernel<T, 4, 1>;
             const size_t smem = std::max(size_t(8) * d.dim_p * 4, route ? route_few_smem(route->d) : 0);
             if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
-            FORGE_CUDA(launch_pdl(kern, dim3((d.heads + d.groups + 7) / 8 + (route ? 1 : 0), (part.n + per - 1) / per), dim3(256), smem, st, d, p, proj + size_t(r0) * ldp, ldp, k_col, q_norm, k_norm,
-                                  reinterpret_cast<const float2*>(rope), static_cast<T*>(q) + size_t(r0) * d.heads * d.dim_p, static_cast<T*>(cache), place + r0, part, beside));
+            FORGE_CUDA(launch_pdl(kern, dim3((d.heads + d.groups + 7) / 8 + (route ? 1 : 0) + scan.blocks, (part.n + per - 1) / per), dim3(256), smem, st, d, p, proj + size_t(r0) * ldp, ldp, k_col, q_norm, k_norm,
+                                  reinterpret_cast<const float2*>(rope), static_cast<T*>(q) + size_t(r0) * d.heads * d.dim_p, static_cast<T*>(cache), place + r0, part, beside, scan));
             FORGE_LAUNCH_CHECK();
         }
         return FORGE_OK;

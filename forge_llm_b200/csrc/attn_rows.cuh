@@ -6,6 +6,7 @@
 
 #include "dense.cuh"
 #include "moe.cuh"
+#include "selective.cuh"
 
 namespace forge {
 
@@ -50,9 +51,11 @@ struct QkPost {
 };
 // proj: f32 rows [q of all heads | ... | k of all groups from k_col | ...] of ldp floats; rope: {cos, sin} by position and pair; place: cache row of each row
 // route (may be null): a routing of the step's rows (route_few) done by one more CTA of the launch
+// conv (may be null): the convolution of single tokens of a scan beside the attention, by further CTAs
 struct RouteBeside { RouterDims d; const float* logits = nullptr; RouteTables t; };
+struct ConvBeside { SelectiveDims d; SelectiveArgs a; int blocks = 0; };
 int32_t qk_post(const AttnDims& d, const QkPost& p, int dtype, const float* proj, int ldp, int k_col, const float* q_norm, const float* k_norm, const float* rope, void* q, void* cache,
-                const int32_t* place, const StepRows& rows, const RouteBeside* route, cudaStream_t st);
+                const int32_t* place, const StepRows& rows, const RouteBeside* route, const ConvBeside* conv, cudaStream_t st);
 
 bool attn_rows_supported(const AttnDims& d);
 // q: T rows [heads][dim_p]; out[row][head * vdim + i] = gate[row][head] * attention, T (gate null: ungated).  sink: score per head, or null.
@@ -62,6 +65,29 @@ int32_t attn_rows(const AttnDims& d, int dtype, const void* q, const void* cache
 
 // ---- blocks seen as one key (attn_pool.cu)
 // The means of the blocks that the step's rows complete.
+#ifdef __CUDACC__
+// columns of the block that position pos completes, if it does: `pieces` pieces of eight from `col`, piece i by thread i
+template <typename T>
+__device__ __forceinline__ void pool_columns(const AttnDims& d, T* cache, const int32_t* pt, int pos, int col, int pieces) {
+    if ((pos + 1) % d.pool || int(threadIdx.x) >= pieces) return;
+    const int b = pos / d.pool, c = col + int(threadIdx.x) * 8;
+    const size_t W = d.row();
+    float sum[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sum[e] = 0.f;
+#pragma unroll 8
+    for (int t = b * d.pool; t <= pos; ++t) {
+        float v[8];
+        load8(v, cache + (size_t(pt[t / FORGE_KV_PAGE]) * FORGE_KV_PAGE + t % FORGE_KV_PAGE) * W + c);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum[e] += v[e];
+    }
+    const float inv = 1.0f / float(d.pool);
+    T* dst = cache + d.block_row(pt, b) * W + c;
+    put4(dst, make_float4(sum[0] * inv, sum[1] * inv, sum[2] * inv, sum[3] * inv));
+    put4(dst + 4, make_float4(sum[4] * inv, sum[5] * inv, sum[6] * inv, sum[7] * inv));
+}
+#endif
 int32_t pool_blocks(const AttnDims& d, int dtype, void* cache, const StepRows& rows, cudaStream_t st);
 // For prompts: block rows of sequences in a row, 64 per table entry.  dst: rows like the cache's.
 struct PoolChunk { int32_t pages0, block0, len, unused; };   // first entry of the sequence in `pages`, first block, positions of the sequence
@@ -70,8 +96,9 @@ int32_t gather_blocks(const AttnDims& d, int dtype, void* dst, const void* cache
 // ---- mixed heads (attn_talk.cu): the weight of head h becomes the sum over heads g of talk[h][g] times the weight of g
 bool talk_rows_supported(const AttnDims& d);
 size_t talk_rows_bytes(const AttnDims& d, int rows, int max_keys);
-// out[row][head * vdim + i] = factor * attention, T; scratch: talk_rows_bytes of at most max_bytes (more rows go in turn).
-int32_t talk_rows(const AttnDims& d, int dtype, const void* q, const void* cache, const float* talk, float factor, void* scratch, size_t max_bytes, void* out, int out_ld, const StepRows& rows, int max_keys,
+// out[row][head * vdim + i] = factor * attention, T; scratch: talk_rows_bytes of at most max_bytes (more rows go in turn).  pools: the rows' sequences have one row
+// each, and the blocks that they complete (which nobody sees yet) are formed here.
+int32_t talk_rows(const AttnDims& d, int dtype, const void* q, void* cache, bool pools, const float* talk, float factor, void* scratch, size_t max_bytes, void* out, int out_ld, const StepRows& rows, int max_keys,
                   cudaStream_t st);
 // out[row][h * vdim + i] = factor * sum over g of talk[h][g] o[row][g][group of h][i]: o bf16 [rows][heads][groups][vdim_p], every head's weights on all groups' values
 int32_t talk_heads(const AttnDims& d, const void* o, const float* talk, float factor, void* out, int out_ld, int rows, cudaStream_t st);

@@ -40,9 +40,16 @@ struct Range {
     }
 };
 
+// keys and values of one group of the block that a row completes
+template <typename T>
+__device__ __forceinline__ void pool_group(const AttnDims& d, T* cache, const int32_t* pt, int pos, int g) {
+    pool_columns(d, cache, pt, pos, g * d.dim_p, d.dim_p / 8);
+    pool_columns(d, cache, pt, pos, d.groups * d.dim_p + g * d.vdim_p, d.vdim_p / 8);
+}
+
 // ------------------------------------------------------------------------------------------------ float32
 template <typename T>
-__global__ void __launch_bounds__(kThreads) talk_scores_kernel(const AttnDims d, const T* q, const T* cache, float* scratch, const ScoreRow sr, const StepRows rows) {
+__global__ void __launch_bounds__(kThreads) talk_scores_kernel(const AttnDims d, const T* q, T* cache, bool pools, float* scratch, const ScoreRow sr, const StepRows rows) {
     extern __shared__ float sm[];
     const int gq = d.heads / d.groups, blocks = (gq + kHeads - 1) / kHeads;
     const int split = blockIdx.x, splits = gridDim.x, g = blockIdx.y / blocks, h0 = g * gq + (blockIdx.y % blocks) * kHeads, nh = min(kHeads, (g + 1) * gq - h0), r = blockIdx.z;
@@ -65,6 +72,7 @@ __global__ void __launch_bounds__(kThreads) talk_scores_kernel(const AttnDims d,
 #pragma unroll
     for (int h = 0; h < kHeads; ++h) { m[h] = -INFINITY; l[h] = 0.f; }
     const float inv_cap = d.softcap > 0.f ? 1.0f / d.softcap : 0.f;
+    if (pools && split == splits - 1 && blockIdx.y % blocks == 0) pool_group(d, cache, pt, pos, g);
     const T* kbase = cache + size_t(g) * d.dim_p;
     float* out = sr.scores(scratch, r);
     for (int key0 = k.begin + warp * 32; key0 < k.end; key0 += kThreads) {
@@ -259,7 +267,7 @@ struct TileWalk {
     __device__ __forceinline__ bool old(int i) const { return min(k.end, first(i) + kTileKeys) <= written; }
 };
 
-__global__ void __launch_bounds__(kThreads) talk_scores_mma_kernel(const AttnDims d, const bf16* q, const bf16* cache, float* scratch, const ScoreRow sr, const StepRows rows) {
+__global__ void __launch_bounds__(kThreads) talk_scores_mma_kernel(const AttnDims d, const bf16* q, bf16* cache, bool pools, float* scratch, const ScoreRow sr, const StepRows rows) {
     extern __shared__ __align__(16) unsigned char sm_raw[];
     __shared__ float sml[kWarps][kTileHeads][2];
     const Tiles L(d.dim_p);
@@ -282,6 +290,7 @@ __global__ void __launch_bounds__(kThreads) talk_scores_mma_kernel(const AttnDim
         *reinterpret_cast<uint4*>(sq + h * L.ld + c) = h < nh ? *reinterpret_cast<const uint4*>(q + (size_t(r) * d.heads + h0 + h) * d.dim_p + c) : make_uint4(0, 0, 0, 0);
     }
     __syncthreads();
+    if (pools && split == splits - 1 && blockIdx.y % blocks == 0) pool_group(d, cache, walk.pt, pos, g);
     const SmemMat mq{uint32_t(__cvta_generic_to_shared(sq)), L.ld};
     const int ksteps = (d.dim + 15) / 16;
     const float scale2 = d.scale * kLog2e, inv_cap = d.softcap > 0.f ? d.scale / d.softcap : 0.f;
@@ -516,12 +525,12 @@ int32_t allow_smem(K kern, size_t smem) {
 }
 
 template <typename T>
-int32_t run_plain(const AttnDims& d, const void* q, const void* cache, const float* talk, float factor, float* scratch, const ScoreRow& sr, void* out, int out_ld, const StepRows& rows, int max_keys, cudaStream_t st) {
+int32_t run_plain(const AttnDims& d, const void* q, void* cache, bool pools, const float* talk, float factor, float* scratch, const ScoreRow& sr, void* out, int out_ld, const StepRows& rows, int max_keys, cudaStream_t st) {
     const int gq = d.heads / d.groups, y = d.groups * ((gq + kHeads - 1) / kHeads), vp = d.vdim_p / 64;
     int splits = 1;   // about two CTAs per SM, no split shorter than one round of its warps
     while (splits < kMaxSplits && rows.n * y * splits * 2 <= 296 && max_keys > splits * kThreads) splits *= 2;
     FORGE_TRY(allow_smem(talk_scores_kernel<T>, plain_score_smem(d)));
-    FORGE_CUDA(launch_pdl(talk_scores_kernel<T>, dim3(splits, y, rows.n), dim3(kThreads), plain_score_smem(d), st, d, static_cast<const T*>(q), static_cast<const T*>(cache), scratch, sr, rows));
+    FORGE_CUDA(launch_pdl(talk_scores_kernel<T>, dim3(splits, y, rows.n), dim3(kThreads), plain_score_smem(d), st, d, static_cast<const T*>(q), static_cast<T*>(cache), pools, scratch, sr, rows));
     FORGE_LAUNCH_CHECK();
     auto go = [&](auto kern) -> int32_t {
         FORGE_TRY(allow_smem(kern, plain_value_smem(d)));
@@ -532,12 +541,12 @@ int32_t run_plain(const AttnDims& d, const void* q, const void* cache, const flo
     return vp <= 1 ? go(talk_values_kernel<T, 1>) : vp <= 2 ? go(talk_values_kernel<T, 2>) : go(talk_values_kernel<T, 8>);
 }
 
-int32_t run_mma(const AttnDims& d, const void* q, const void* cache, const float* talk, float factor, float* scratch, const ScoreRow& sr, void* out, int out_ld, const StepRows& rows, int max_keys, cudaStream_t st) {
+int32_t run_mma(const AttnDims& d, const void* q, void* cache, bool pools, const float* talk, float factor, float* scratch, const ScoreRow& sr, void* out, int out_ld, const StepRows& rows, int max_keys, cudaStream_t st) {
     const int gq = d.heads / d.groups, y = d.groups * ((gq + kTileHeads - 1) / kTileHeads);
     int splits = 1;
     while (splits < kMaxSplits && (long long)rows.n * y * splits * 2 <= 296 && max_keys > splits * kWarps * kTileKeys) splits *= 2;
     FORGE_TRY(allow_smem(talk_scores_mma_kernel, score_smem(d)));
-    FORGE_CUDA(launch_pdl(talk_scores_mma_kernel, dim3(splits, y, rows.n), dim3(kThreads), score_smem(d), st, d, static_cast<const bf16*>(q), static_cast<const bf16*>(cache), scratch, sr, rows));
+    FORGE_CUDA(launch_pdl(talk_scores_mma_kernel, dim3(splits, y, rows.n), dim3(kThreads), score_smem(d), st, d, static_cast<const bf16*>(q), static_cast<bf16*>(cache), pools, scratch, sr, rows));
     FORGE_LAUNCH_CHECK();
     const size_t smem = value_smem(d, sr);
     auto go = [&](auto kern) -> int32_t {
@@ -554,7 +563,7 @@ int32_t run_mma(const AttnDims& d, const void* q, const void* cache, const float
 bool talk_rows_supported(const AttnDims& d) { return d.heads <= 128 && d.vdim_p <= 512 && d.keep == 0 && d.bias_n == 0 && plain_score_smem(d) <= 200 * 1024 && plain_value_smem(d) <= 200 * 1024; }
 size_t talk_rows_bytes(const AttnDims& d, int rows, int max_keys) { return size_t(rows) * score_row(d, max_keys).floats() * sizeof(float); }
 
-int32_t talk_rows(const AttnDims& d, int dtype, const void* q, const void* cache, const float* talk, float factor, void* scratch, size_t max_bytes, void* out, int out_ld, const StepRows& rows, int max_keys,
+int32_t talk_rows(const AttnDims& d, int dtype, const void* q, void* cache, bool pools, const float* talk, float factor, void* scratch, size_t max_bytes, void* out, int out_ld, const StepRows& rows, int max_keys,
                   cudaStream_t st) {
     if (rows.n <= 0) return FORGE_OK;
     const ScoreRow sr = score_row(d, max_keys);
@@ -569,9 +578,9 @@ int32_t talk_rows(const AttnDims& d, int dtype, const void* q, const void* cache
         const void* pq = static_cast<const char*>(q) + size_t(r0) * d.heads * d.dim_p * es;
         void* po = static_cast<char*>(out) + size_t(r0) * out_ld * es;
         float* sc = static_cast<float*>(scratch);
-        if (dtype == FORGE_BF16 && mma_supported(d)) FORGE_TRY(run_mma(d, pq, cache, talk, factor, sc, sr, po, out_ld, part, max_keys, st));
-        else if (dtype == FORGE_BF16) FORGE_TRY(run_plain<bf16>(d, pq, cache, talk, factor, sc, sr, po, out_ld, part, max_keys, st));
-        else FORGE_TRY(run_plain<float>(d, pq, cache, talk, factor, sc, sr, po, out_ld, part, max_keys, st));
+        if (dtype == FORGE_BF16 && mma_supported(d)) FORGE_TRY(run_mma(d, pq, cache, pools, talk, factor, sc, sr, po, out_ld, part, max_keys, st));
+        else if (dtype == FORGE_BF16) FORGE_TRY(run_plain<bf16>(d, pq, cache, pools, talk, factor, sc, sr, po, out_ld, part, max_keys, st));
+        else FORGE_TRY(run_plain<float>(d, pq, cache, pools, talk, factor, sc, sr, po, out_ld, part, max_keys, st));
     }
     return FORGE_OK;
 }

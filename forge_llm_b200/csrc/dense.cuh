@@ -25,6 +25,14 @@ struct DenseWeight {
     // a view of some columns: K columns from col0 of rows of ld (0: K) columns; col0 and ld are multiples of 64
     int ld = 0, col0 = 0;
     int pitch() const { return ld ? ld : K; }
+    // a view of n rows from row `from` (a multiple of 128)
+    DenseWeight rows(int from, int n) const {
+        DenseWeight v = *this;
+        v.N = n;
+        if (w) v.w = static_cast<char*>(w) + size_t(from) * pitch() * dense_size(dtype);
+        if (tiles) v.tiles = static_cast<char*>(tiles) + size_t(from) * pitch() * 2;
+        return v;
+    }
     DenseWeight columns(int from, int n) const { DenseWeight v = *this; v.ld = pitch(); v.col0 = col0 + from; v.K = n; return v; }
 };
 

@@ -71,7 +71,7 @@ __global__ void __launch_bounds__(1024) slots_kernel(const RouterDims d, int row
     for (int e = warp; e < E; e += 32)
         for (int i = lane; i * tile_rows < total[e]; i += 32) {
             const int at = start[e] + i * tile_rows;
-            t.tiles[tile0[e] + i] = GroupTile{e, at, min(tile_rows, total[e] - i * tile_rows), at};
+            t.tiles[tile0[e] + i] = GroupTile{d.always + e, at, min(tile_rows, total[e] - i * tile_rows), at};
         }
     for (int p = p0; p < p1; p += 32) {
         const int i = p + lane;
@@ -120,8 +120,10 @@ __global__ void __launch_bounds__(256) add_experts_kernel(float* __restrict__ x,
 
 // A CTA per row.  NV: pieces of four columns per thread (rows of up to 1024 NV); 0: any width.
 template <typename T, int NV>
-__global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* y, int width, float eps, float gain, const MixtureSum mix, const After after) {
+__global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* y, int width, float eps, float gain, const MixtureSum mix, const After after, const RouteBehind route) {
+    extern __shared__ __align__(16) float s_row[];     // routing: the row, its logits, then the tables
     __shared__ float red[8];
+    __shared__ int s_last;
     const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     float* xr = x + size_t(r) * width;
     const float* yr = y + size_t(r) * width;
@@ -135,6 +137,14 @@ __global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* 
         return gain / sqrtf(ss / float(width) + eps);
     };
     pdl_trigger();
+    // routing, a warp per choice: the first one's weights are on their way before the wait
+    constexpr int KEEP = NV * 4;     // pieces of eight columns per lane
+    uint4 held[KEEP > 0 ? KEEP : 1];
+    const T* own_w = static_cast<const T*>(route.w) + size_t(warp) * route.ld;
+    if constexpr (NV > 0 && sizeof(T) == 2)
+        if (route.w && warp < route.d.choices())
+#pragma unroll
+            for (int i = 0; i < KEEP; ++i) { const int c = (lane + 32 * i) * 8; held[i] = c < width ? *reinterpret_cast<const uint4*>(own_w + c) : make_uint4(0, 0, 0, 0); }
     pdl_wait();
     const float passed = mix.passed ? mix.passed[r] : 0.f;
     if constexpr (NV > 0) {
@@ -171,6 +181,47 @@ __global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* 
             float4 v = make_float4(fmaf(f, vy[j].x, vx[j].x), fmaf(f, vy[j].y, vx[j].y), fmaf(f, vy[j].z, vx[j].z), fmaf(f, vy[j].w, vx[j].w));
             v = leave_four<T>(after, v, size_t(r), size_t(width), c, ok);
             if (ok) put4(xr + c, v);
+            if (ok && route.w) put4(s_row + c, v);
+        }
+        if constexpr (sizeof(T) == 2) {
+            if (!route.w) return;
+            const int C = route.d.choices(), rows = gridDim.x;
+            float* s_z = s_row + 1024 * NV;
+            for (int i = width + threadIdx.x; i < 1024 * NV; i += 256) s_row[i] = 0.f;
+            __syncthreads();
+            for (int e = warp; e < C; e += 8) {
+                float z = 0.f;
+#pragma unroll
+                for (int i = 0; i < KEEP; ++i) {
+                    const int c = (lane + 32 * i) * 8;
+                    float w[8], v[8];
+                    if (e != warp) held[i] = c < width ? *reinterpret_cast<const uint4*>(own_w + size_t(e - warp) * route.ld + c) : make_uint4(0, 0, 0, 0);
+                    load8(w, reinterpret_cast<const T*>(&held[i]));
+                    load8(v, s_row + c);
+#pragma unroll
+                    for (int k = 0; k < 8; ++k) z = fmaf(w[k], v[k], z);
+                }
+                z = warp_sum(z);
+                if (lane == 0) s_z[e] = z;
+            }
+            float* s_w = s_z + ((C + 3) & ~3);
+            for (int i = threadIdx.x; i < route.d.groups() * (kScaleRows + 1); i += 256) s_w[i] = 0.f;
+            __syncthreads();
+            if (warp == 0) choose(s_z, route.d, route.t.expert + r * route.d.top, route.t.weight + r * route.d.top);
+            if (rows > 1) {     // the last row makes the tables
+                if (threadIdx.x == 0) {
+                    __threadfence();
+                    const int before = atomicAdd(route.ticket, 1);
+                    s_last = before == rows - 1;
+                    if (s_last) { *route.ticket = 0; __threadfence(); }
+                }
+                __syncthreads();
+                if (!s_last) return;
+            } else {
+                __threadfence_block();
+                __syncthreads();
+            }
+            route_few_tables(route.d, rows, route.t, s_w);
         }
     } else {
         auto value = [&](int c) {
@@ -201,10 +252,15 @@ size_t align16(size_t n) { return (n + 15) & ~size_t(15); }
 
 size_t route_bytes(const RouterDims& d, int rows) {
     const size_t pairs = size_t(rows) * d.top;
-    return 5 * align16(pairs * 4) + align16(size_t(rows) * 4) + size_t(d.experts) * kScaleRows * 4 + (pairs + d.experts) * sizeof(GroupTile) + 16;
+    return 5 * align16(pairs * 4) + align16(size_t(rows) * 4) + size_t(d.groups()) * kScaleRows * 4 + (pairs + d.groups() + d.experts) * sizeof(GroupTile) + 16;
 }
 GroupTable few_table(const RouterDims& d, int rows, const RouteTables& t) {
-    return GroupTable{t.tiles, t.n_tiles, int(std::min<long long>(d.experts, (long long)rows * d.top)), rows <= 16 ? 16 : 32, t.row_weight};
+    return GroupTable{t.tiles, t.n_tiles, d.always + int(std::min<long long>(d.experts, (long long)rows * d.top)), rows <= 16 ? 16 : 32, t.row_weight};
+}
+GroupTable listed_table(const RouterDims& d, int rows, const RouteTables& t) {
+    GroupTable l = few_table(d, rows, t);
+    l.tiles = t.listed; l.n = t.n_listed; l.max_tiles -= d.always;
+    return l;
 }
 RouteTables route_tables(void* p, const RouterDims& d, int rows) {
     const size_t pairs = align16(size_t(rows) * d.top * 4);
@@ -212,8 +268,10 @@ RouteTables route_tables(void* p, const RouterDims& d, int rows) {
     auto take = [&](size_t n) { char* at = b; b += n; return at; };
     RouteTables t;
     t.n_tiles = reinterpret_cast<int32_t*>(take(16));
-    t.tiles = reinterpret_cast<GroupTile*>(take((size_t(rows) * d.top + d.experts) * sizeof(GroupTile)));
-    t.row_weight = reinterpret_cast<float*>(take(size_t(d.experts) * kScaleRows * 4));
+    t.n_listed = t.n_tiles + 1;
+    t.tiles = reinterpret_cast<GroupTile*>(take((size_t(rows) * d.top + d.groups()) * sizeof(GroupTile)));
+    t.listed = reinterpret_cast<GroupTile*>(take(size_t(d.experts) * sizeof(GroupTile)));
+    t.row_weight = reinterpret_cast<float*>(take(size_t(d.groups()) * kScaleRows * 4));
     t.expert = reinterpret_cast<int32_t*>(take(pairs)); t.weight = reinterpret_cast<float*>(take(pairs)); t.slot = reinterpret_cast<int32_t*>(take(pairs));
     t.row = reinterpret_cast<int32_t*>(take(pairs)); t.slot_weight = reinterpret_cast<float*>(take(pairs));
     t.passed = reinterpret_cast<float*>(take(align16(size_t(rows) * 4)));
@@ -224,7 +282,7 @@ int32_t route_few(const RouterDims& d, const float* logits, int rows, const Rout
     if (rows > kScaleRows || d.choices() > kMaxExperts) { set_error("routing: %d rows, %d experts", rows, d.experts); return FORGE_ERR_SHAPE; }
     *out = few_table(d, rows, t);
     const size_t smem = route_few_smem(d);
-    FORGE_CUDA(cudaFuncSetAttribute(route_few_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(route_few_smem(RouterDims{kMaxExperts, 1}))));
+    if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(route_few_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
     FORGE_CUDA(launch_pdl(route_few_kernel, dim3(1), dim3(1024), smem, st, d, logits, rows, t));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
@@ -251,13 +309,22 @@ int32_t add_experts(float* x, const float* y, const RouterDims& d, const RouteTa
     return FORGE_OK;
 }
 
-int32_t add_normed(float* x, const float* y, int rows, int width, float eps, float gain, const MixtureSum& mix, const After& after, int dtype, cudaStream_t st) {
+// (a CTA per row reads all of the router; what it holds on to lies in registers)
+static int norm_pieces(int width) { return width <= 1024 ? 1 : width <= 2048 ? 2 : width <= 4096 ? 4 : 8; }
+static size_t route_behind_smem(const RouterDims& d, int width) { return size_t(1024) * norm_pieces(width) * 4 + size_t((d.choices() + 3) & ~3) * 4 + route_few_smem(d); }
+bool route_behind_supported(const RouterDims& d, int width, int rows) { return rows <= kScaleRows && width % 8 == 0 && width <= 4096 && d.choices() <= 64 && route_behind_smem(d, width) <= 200 * 1024; }
+
+int32_t add_normed(float* x, const float* y, int rows, int width, float eps, float gain, const MixtureSum& mix, const After& after, const RouteBehind* route, int dtype, cudaStream_t st) {
     if (rows <= 0) return FORGE_OK;
+    const bool wide = width % 4 != 0 || after.ld % 4 != 0 || after.col2 % 4 != 0 || width > 8192;
+    if (route && (wide || dtype != FORGE_BF16 || route->ld % 8 || !route_behind_supported(route->d, width, rows))) { set_error("routing behind a norm: %d rows of %d", rows, width); return FORGE_ERR_SHAPE; }
     auto go = [&](auto type) -> int32_t {
         using T = decltype(type);
-        const bool four = width % 4 == 0 && after.ld % 4 == 0 && after.col2 % 4 == 0;
-        auto kern = !four || width > 8192 ? add_normed_kernel<T, 0> : width <= 1024 ? add_normed_kernel<T, 1> : width <= 2048 ? add_normed_kernel<T, 2> : width <= 4096 ? add_normed_kernel<T, 4> : add_normed_kernel<T, 8>;
-        FORGE_CUDA(launch_pdl(kern, dim3(rows), dim3(256), 0, st, x, y, width, eps, gain, mix, after));
+        const int nv = norm_pieces(width);
+        auto kern = wide ? add_normed_kernel<T, 0> : nv == 1 ? add_normed_kernel<T, 1> : nv == 2 ? add_normed_kernel<T, 2> : nv == 4 ? add_normed_kernel<T, 4> : add_normed_kernel<T, 8>;
+        const size_t smem = route ? route_behind_smem(route->d, width) : 0;
+        if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+        FORGE_CUDA(launch_pdl(kern, dim3(rows), dim3(256), smem, st, x, y, width, eps, gain, mix, after, route ? *route : RouteBehind{}));
         FORGE_LAUNCH_CHECK();
         return FORGE_OK;
     };

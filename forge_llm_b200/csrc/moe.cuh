@@ -9,25 +9,29 @@ constexpr int kMaxExperts = 512;
 
 // Choices behind the experts pass a token's input on (identity).  correction (device, null: none): the `top` largest of softmax(logits) +
 // correction are chosen and weighted with their softmax over all choices; without it the largest logits, weighted by the softmax over the chosen.
+// always: groups of the products in front of the experts that every token uses with weight one (pieces of a shared expert).
 struct RouterDims {
-    int experts = 0, top = 0, identity = 0;
+    int experts = 0, top = 0, identity = 0, always = 0;
     const float* correction = nullptr;
     __host__ __device__ int choices() const { return experts + identity; }
+    __host__ __device__ int groups() const { return always + experts; }
 };
 // Device tables of one routing.  A pair is (row, k), k = 0 .. top - 1; pairs are dealt to slots expert by expert, in the order of
 // rows within an expert.
 struct RouteTables {
     int32_t* expert = nullptr; float* weight = nullptr; int32_t* slot = nullptr;   // [rows][top]
     int32_t* row = nullptr; float* slot_weight = nullptr;                          // [rows * top], by slot
-    float* row_weight = nullptr;                                                   // few rows: [experts][kScaleRows], zero where the expert is not used
+    float* row_weight = nullptr;                                                   // few rows: [groups][kScaleRows], zero where the group is not used
     float* passed = nullptr;                                                       // [rows]: weight of the choices that pass the input on
     GroupTile* tiles = nullptr; int32_t* n_tiles = nullptr;
+    GroupTile* listed = nullptr; int32_t* n_listed = nullptr;                      // few rows: the experts among them, numbered without the groups in front
 };
 size_t route_bytes(const RouterDims& d, int rows);
 RouteTables route_tables(void* p, const RouterDims& d, int rows);
 
 GroupTable few_table(const RouterDims& d, int rows, const RouteTables& t);   // of route_few
-inline size_t route_few_smem(const RouterDims& d) { return size_t(d.experts) * (kScaleRows + 1) * 4; }
+GroupTable listed_table(const RouterDims& d, int rows, const RouteTables& t);   // the same for a listed product whose fixed columns are those of the groups in front
+inline size_t route_few_smem(const RouterDims& d) { return size_t(d.groups()) * (kScaleRows + 1) * 4; }
 // logits: f32 [rows][choices].
 // Few rows (at most kScaleRows): a tile of all rows per expert that any of them uses.
 int32_t route_few(const RouterDims& d, const float* logits, int rows, const RouteTables& t, GroupTable* out, cudaStream_t st);
@@ -38,7 +42,10 @@ int32_t add_experts(float* x, const float* y, const RouterDims& d, const RouteTa
 // x += gain * y / rms(y), then `after`.  y: f32 rows; with a mixture first y[r] += passed[r] x[r], and with expert outputs e (f32 rows by slot) += those of the
 // row's slots.
 struct MixtureSum { const float* passed = nullptr; const float* e = nullptr; const int32_t* slot = nullptr; int top = 0; };
-int32_t add_normed(float* x, const float* y, int rows, int width, float eps, float gain, const MixtureSum& mix, const After& after, int dtype, cudaStream_t st);
+// Few rows: the finished rows of the stream are routed, too (route_few's tables): w: T rows [choices][ld]; ticket: one self-resetting word.
+struct RouteBehind { RouterDims d; const void* w = nullptr; int ld = 0; RouteTables t; int* ticket = nullptr; };
+bool route_behind_supported(const RouterDims& d, int width, int rows);
+int32_t add_normed(float* x, const float* y, int rows, int width, float eps, float gain, const MixtureSum& mix, const After& after, const RouteBehind* route, int dtype, cudaStream_t st);
 
 #ifdef __CUDACC__
 constexpr int kPerLane = kMaxExperts / 32;
@@ -92,39 +99,50 @@ __device__ __forceinline__ void choose(const float* z, const RouterDims& d, int3
 
 // Routing of few rows by one CTA of whole warps; s_w: route_few_smem(d) bytes, cleared before.  (Also run by a kernel that stands beside it in a step.)
 __device__ __forceinline__ void route_few_clear(const RouterDims& d, float* s_w) {
-    for (int i = threadIdx.x; i < d.experts * (kScaleRows + 1); i += blockDim.x) s_w[i] = 0.f;
+    for (int i = threadIdx.x; i < d.groups() * (kScaleRows + 1); i += blockDim.x) s_w[i] = 0.f;
     __syncthreads();
 }
-__device__ __forceinline__ void route_few_rows(const RouterDims& d, const float* logits, int rows, const RouteTables& t, float* s_w) {
-    int* used = reinterpret_cast<int*>(s_w + d.experts * kScaleRows);
+// the tables of rows whose choices lie in t.expert and t.weight
+__device__ __forceinline__ void route_few_tables(const RouterDims& d, int rows, const RouteTables& t, float* s_w) {
+    const int G = d.groups();
+    int* used = reinterpret_cast<int*>(s_w + G * kScaleRows);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int r = warp; r < rows; r += blockDim.x / 32) {
-        choose(logits + size_t(r) * d.choices(), d, t.expert + r * d.top, t.weight + r * d.top);
-        if (lane == 0) {
-            float passed = 0.f;
-            for (int k = 0; k < d.top; ++k) {
-                const int e = t.expert[r * d.top + k];
-                const float w = t.weight[r * d.top + k];
-                if (e >= d.experts) { passed += w; continue; }
-                s_w[e * kScaleRows + r] = w;
-                used[e] = 1;
-            }
-            t.passed[r] = passed;
+    for (int i = threadIdx.x; i < d.always * kScaleRows; i += blockDim.x) {
+        s_w[i] = 1.f;
+        if (i % kScaleRows == 0) used[i / kScaleRows] = 1;
+    }
+    for (int r = threadIdx.x; r < rows; r += blockDim.x) {
+        float passed = 0.f;
+        for (int k = 0; k < d.top; ++k) {
+            const int e = __ldcg(t.expert + r * d.top + k);
+            const float w = __ldcg(t.weight + r * d.top + k);
+            if (e >= d.experts) { passed += w; continue; }
+            s_w[(d.always + e) * kScaleRows + r] = w;
+            used[d.always + e] = 1;
         }
+        t.passed[r] = passed;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < d.experts * kScaleRows; i += blockDim.x) t.row_weight[i] = s_w[i];
+    for (int i = threadIdx.x; i < G * kScaleRows; i += blockDim.x) t.row_weight[i] = s_w[i];
     if (warp == 0) {
         int n = 0;
-        for (int e0 = 0; e0 < d.experts; e0 += 32) {
-            const int e = e0 + lane;
-            const bool on = e < d.experts && used[e];
+        for (int g0 = 0; g0 < G; g0 += 32) {
+            const int g = g0 + lane;
+            const bool on = g < G && used[g];
             const uint32_t mask = __ballot_sync(0xffffffffu, on);
-            if (on) t.tiles[n + __popc(mask & ((1u << lane) - 1))] = GroupTile{e, 0, rows, e * kScaleRows};
+            const int at = n + __popc(mask & ((1u << lane) - 1));
+            if (on) t.tiles[at] = GroupTile{g, 0, rows, g * kScaleRows};
+            if (on && g >= d.always) t.listed[at - d.always] = GroupTile{g - d.always, 0, rows, g * kScaleRows};
             n += __popc(mask);
         }
-        if (lane == 0) *t.n_tiles = n;
+        if (lane == 0) { *t.n_tiles = n; *t.n_listed = n - d.always; }
     }
+}
+__device__ __forceinline__ void route_few_rows(const RouterDims& d, const float* logits, int rows, const RouteTables& t, float* s_w) {
+    for (int r = threadIdx.x >> 5; r < rows; r += blockDim.x / 32) choose(logits + size_t(r) * d.choices(), d, t.expert + r * d.top, t.weight + r * d.top);
+    __threadfence_block();
+    __syncthreads();
+    route_few_tables(d, rows, t, s_w);
 }
 #endif
 

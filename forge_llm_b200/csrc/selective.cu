@@ -27,32 +27,11 @@ __device__ __forceinline__ float fast_softplus(float v) {
     const float series = u * fmaf(u, fmaf(u, fmaf(u, fmaf(u, fmaf(u, -1.f / 6.f, 0.2f), -0.25f), 1.f / 3.f), -0.5f), 1.f);
     return fmaxf(v, 0.f) + (u < 0.0625f ? series : __logf(1.f + u));
 }
-template <typename T> __device__ __forceinline__ float conv_act(float v) {
-    if constexpr (sizeof(T) == 4) return silu(v);
-    return __fdividef(v, 1.0f + __expf(-v));   // far inside a bfloat16 rounding
-}
 
 // ------------------------------------------------------------------------------------------------ convolution
 template <typename T>
 __global__ void __launch_bounds__(256) conv_one_kernel(const SelectiveDims d, const SelectiveArgs a, const StepRows rows) {
-    const int r = blockIdx.y, c = blockIdx.x * 256 + threadIdx.x;
-    pdl_trigger();
-    const int pos = rows.pos[r], slot = state_slot(rows, r);
-    T* ring = static_cast<T*>(a.ring) + size_t(slot) * d.ring_values() + c;
-    float v = 0.f, w = 0.f;
-    if (c < d.inner) {   // what earlier steps have left
-        v = a.conv_add[c];
-        w = a.conv[size_t(d.taps - 1) * d.inner + c];
-        for (int j = 0; j < d.taps - 1; ++j) {
-            const int p = pos - (d.taps - 1 - j);
-            if (p >= 0) v = fmaf(a.conv[size_t(j) * d.inner + c], to_f(ring[size_t(p % d.taps) * d.inner]), v);
-        }
-    }
-    pdl_wait();
-    if (c >= d.inner) return;
-    const T in = static_cast<const T*>(a.in)[size_t(r) * a.in_ld + c];
-    static_cast<T*>(a.x)[size_t(r) * a.x_ld + c] = to_t<T>(conv_act<T>(fmaf(w, to_f(in), v)));
-    ring[size_t(pos % d.taps) * d.inner] = in;
+    conv_one<T>(d, a, rows, blockIdx.y, blockIdx.x * 256 + threadIdx.x);
 }
 
 // A thread = one channel over a run of tokens; the first run's thread alone reads what the ring keeps of its channel and then leaves there the segment's

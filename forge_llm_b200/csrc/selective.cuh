@@ -32,6 +32,35 @@ struct SelectiveArgs {
     void* out = nullptr; int out_ld = 0;                   // T rows [inner]
 };
 
+#ifdef __CUDACC__
+// convolutions end in silu; bfloat16 models take the fast exponential and quotient (far inside a rounding)
+template <typename T> __device__ __forceinline__ float conv_act(float v) {
+    if constexpr (sizeof(T) == 4) return silu(v);
+    else return __fdividef(v, 1.0f + __expf(-v));
+}
+// The convolution of channel c of row r, a single token.  What earlier steps have left is read in front of the dependency wait (rows of a loop: of the first).
+template <typename T>
+__device__ __forceinline__ void conv_one(const SelectiveDims& d, const SelectiveArgs& a, const StepRows& rows, int r, int c) {
+    pdl_trigger();
+    const int pos = rows.pos[r], slot = state_slot(rows, r);
+    T* ring = static_cast<T*>(a.ring) + size_t(slot) * d.ring_values() + c;
+    float v = 0.f, w = 0.f;
+    if (c < d.inner) {
+        v = a.conv_add[c];
+        w = a.conv[size_t(d.taps - 1) * d.inner + c];
+        for (int j = 0; j < d.taps - 1; ++j) {
+            const int p = pos - (d.taps - 1 - j);
+            if (p >= 0) v = fmaf(a.conv[size_t(j) * d.inner + c], to_f(ring[size_t(p % d.taps) * d.inner]), v);
+        }
+    }
+    pdl_wait();
+    if (c >= d.inner) return;
+    const T in = static_cast<const T*>(a.in)[size_t(r) * a.in_ld + c];
+    static_cast<T*>(a.x)[size_t(r) * a.x_ld + c] = to_t<T>(conv_act<T>(fmaf(w, to_f(in), v)));
+    ring[size_t(pos % d.taps) * d.inner] = in;
+}
+#endif
+
 bool selective_supported(const SelectiveDims& d);
 // the convolution of single tokens (rows) and of segments
 int32_t selective_conv(const SelectiveDims& d, int dtype, const SelectiveArgs& a, const StepRows& ones, const SegTable& t, cudaStream_t st);

@@ -253,8 +253,10 @@ int32_t parse_experts(const Json* mlp, int layer, bool shared, LayerSpec* L) {
     if (shared) {
         FORGE_TRY(need_int(mlp->get("shared"), "ff", &L->shared_ff));
         FORGE_TRY(need_int(router, "identity", &L->router.identity, 0));
+        L->router.always = (L->shared_ff + L->ff - 1) / L->ff;
     }
     if (L->router.top > L->router.choices()) { set_error("layer %d: top %d of %d experts", layer, L->router.top, L->router.choices()); return FORGE_ERR_SHAPE; }
+    if (L->router.always > kMaxExperts) { set_error("layer %d: a shared expert of %d beside experts of %d is not supported", layer, L->shared_ff, L->ff); return FORGE_ERR_UNSUPPORTED; }
     if (L->router.choices() > kMaxExperts) { set_error("layer %d: %d experts are not supported", layer, L->router.choices()); return FORGE_ERR_UNSUPPORTED; }
     return FORGE_OK;
 }

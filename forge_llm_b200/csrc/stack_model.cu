@@ -32,7 +32,7 @@ struct StreamNorm { float* w = nullptr; float* b = nullptr; float alpha = 0.f; }
 struct LayerWeights {
     StreamNorm norm1, norm2;
     DenseWeight in, out;
-    DenseWeight ff_in, ff_out;    // sequential arrangement; norms on outputs: [shared | router], [shared | expert 0 | expert 1 ...]
+    DenseWeight ff_in, ff_out;    // sequential arrangement; norms on outputs: [router | shared], [shared | expert 0 | expert 1 ...]
     // latent attention
     DenseWeight kv;               // rows [uk | uv] over the latent
     int q_rows = 0, dkv_row = 0, g_row = 0, glu_row = 0, uv_row = 0;   // first rows of the segments of `in` / `kv`
@@ -58,7 +58,8 @@ struct LayerWeights {
     // experts: their columns of `out` follow the heads', ff_k apart
     int router_row = 0, ff_k = 0;
     float* router_bias = nullptr;
-    DenseWeight experts;          // gate and up rows, pairs interleaved, expert by expert expert_rows apart
+    DenseWeight experts;          // gate and up rows, pairs interleaved, group by group expert_rows apart (norms on outputs: those of the shared expert's pieces first)
+    void* router = nullptr;       // its rows
     int expert_rows = 0;
 };
 
@@ -154,6 +155,12 @@ struct Image {
     int N, K, dtype;
     Image(int n, int k, int dt) : img(size_t(n) * k * dense_size(dt), 0), N(n), K(k), dtype(dt) {}
     void put(const TensorView* t, int row0, int step = 1, int col0 = 0, int from = 0, int count = -1) { put_rows(img, dtype, K, *t, row0, step, col0, from, count); }
+    // columns [from, from + count) of all rows of `t` to columns from col0
+    void put_columns(const TensorView* t, int from, int count, int col0) {
+        const int64_t k = t->shape[1];
+        for (int64_t r = 0; r < t->shape[0]; ++r)
+            for (int c = 0; c < count; ++c) store(img.data(), dtype, size_t(r) * K + col0 + c, *t, size_t(r * k + from + c));
+    }
     int32_t load(ForgeModel* m, DenseWeight* w, bool row_reads = false) const { return load_dense(m, w, N, K, dtype, img, row_reads); }
 };
 
@@ -406,26 +413,33 @@ int32_t load_attn_selective(ForgeModel* m, const LayerSpec& L, const TensorSet& 
     return upload_f32(m, &w->skip, *t.at("mix.right.D"));
 }
 
-// A mixture beside a shared expert: [shared gate, up | router] and, over [shared | expert 0 | expert 1 ...], the way back.
+// A mixture beside a shared expert: [router | shared gate, up | experts' gate, up] and, over [shared | expert 0 | expert 1 ...], the way back.
 int32_t load_mixture(ForgeModel* m, const LayerSpec& L, const TensorSet& t, LayerWeights* w) {
     StackModel& S = *m->stack;
-    const int E = L.router.experts, shared_k = pad_to(L.shared_ff, kDensePad);
-    w->router_row = pad_to(2 * L.shared_ff, kSegAlign);
-    Image in(w->router_row + L.router.choices(), S.width_p, S.dtype);
-    in.put(t.at("mlp.shared.gate"), 0, 2); in.put(t.at("mlp.shared.up"), 1, 2);
-    in.put(t.at("mlp.router"), w->router_row);
-    FORGE_TRY(in.load(m, &w->ff_in));
+    const int E = L.router.experts, A = L.router.always;
     w->ff_k = pad_to(L.ff, kDensePad);
     w->expert_rows = pad_to(2 * L.ff, 128);
-    Image ex(E * w->expert_rows, S.width_p, S.dtype), out(S.spec.width, shared_k + E * w->ff_k, S.dtype);
-    out.put(t.at("mlp.shared.down"), 0);
+    w->glu_row = pad_to(L.router.choices(), 128);
+    Image in(w->glu_row + (A + E) * w->expert_rows, S.width_p, S.dtype), out(S.spec.width, (A + E) * w->ff_k, S.dtype), router(L.router.choices(), S.width_p, S.dtype);
+    in.put(t.at("mlp.router"), 0);
+    router.put(t.at("mlp.router"), 0);
+    FORGE_TRY(upload(m, &w->router, router.img));
+    for (int a = 0; a < A; ++a) {   // a piece of the shared expert has as many rows as an expert
+        const int from = a * L.ff, n = std::min(L.ff, L.shared_ff - from), row = w->glu_row + a * w->expert_rows;
+        in.put(t.at("mlp.shared.gate"), row, 2, 0, from, n);
+        in.put(t.at("mlp.shared.up"), row + 1, 2, 0, from, n);
+        out.put_columns(t.at("mlp.shared.down"), from, n, a * w->ff_k);
+    }
     for (int e = 0; e < E; ++e) {
         const std::string x = "mlp.e" + std::to_string(e);
-        ex.put(t.at(x + ".gate"), e * w->expert_rows, 2);
-        ex.put(t.at(x + ".up"), e * w->expert_rows + 1, 2);
-        out.put(t.at(x + ".down"), 0, 1, shared_k + e * w->ff_k);
+        const int row = w->glu_row + (A + e) * w->expert_rows;
+        in.put(t.at(x + ".gate"), row, 2);
+        in.put(t.at(x + ".up"), row + 1, 2);
+        out.put(t.at(x + ".down"), 0, 1, (A + e) * w->ff_k);
     }
-    FORGE_TRY(ex.load(m, &w->experts));
+    FORGE_TRY(in.load(m, &w->ff_in));
+    w->experts = w->ff_in.rows(w->glu_row, (A + E) * w->expert_rows);
+    w->ff_in = w->ff_in.rows(0, w->glu_row + A * w->expert_rows);
     FORGE_TRY(out.load(m, &w->ff_out));
     return upload_f32(m, &w->router_bias, *t.at("mlp.correction"));
 }
@@ -527,7 +541,7 @@ int mid_columns(const StackModel& S, const LayerSpec& L, const LayerWeights& w, 
     return L.router.experts && S.spec.arch->arrangement == Arrangement::ParallelTwo && !few_tokens(S, w, rows) ? w.heads_k : w.out.K;
 }
 // the same in front of a mixture's way back
-int shared_columns(const LayerSpec& L) { return pad_to(L.shared_ff, kDensePad); }
+int shared_columns(const LayerSpec& L, const LayerWeights& w) { return L.router.always * w.ff_k; }
 constexpr size_t kScoreBytes = size_t(256) << 20;   // scores of rows with mixed heads, at most, if rows may go in turn
 
 // splits of the row attention: at most one CTA per SM over all rows and head groups, no more than there are pages
@@ -550,7 +564,7 @@ int32_t ensure_step(ForgeModel* m, int rows, int single, int splits, int prompt,
         const LayerSpec& L = S.spec.layers[i];
         const LayerWeights& w = S.weights(int(i));
         for (const DenseWeight* d : {&w.in, &w.out, &w.kv, &w.low, &w.scan_in, &w.ff_in, &w.ff_out}) most(n_max, size_t(d->N));
-        most(mid, r * std::max(mid_columns(S, L, w, rows), S.spec.arch->arrangement == Arrangement::PostNorm ? shared_columns(L) : w.ff_out.K) * es);
+        most(mid, r * std::max(mid_columns(S, L, w, rows), S.spec.arch->arrangement == Arrangement::PostNorm ? shared_columns(L, w) : w.ff_out.K) * es);
         if (S.spec.arch->arrangement == Arrangement::PostNorm) most(pair, r * W * 4);
         if (S.spec.arch->arrangement == Arrangement::ParallelTwo) most(h, 2 * WP * es);
         if (L.router.experts) {
@@ -911,17 +925,20 @@ struct Sequence {
         while (S.spec.runs[i].layer != layer) ++i;
         return kv->stack->runs[i];
     }
-    // norms, rotation, attention of all rows of the step: factor * heads to the first columns of mid
-    int32_t attend(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, int mid_ld, float factor, const RouteBeside* route) {
+    // norms and rotation; then the attention of all rows of the step: factor * heads to the first columns of mid
+    int32_t queries_and_keys(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const RouteBeside* route, const ConvBeside* conv) {
+        return qk_post(L.attn, L.soft.qk, dt, static_cast<const float*>(S.proj.p), w.v_row, w.k_row, w.q_norm, w.k_norm, S.ropes.at(L.rot).second, S.q.p, run.pool, static_cast<const int32_t*>(S.place.p),
+                       s.rows, route, conv, st);
+    }
+    int32_t attend(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, int mid_ld, float factor) {
         AttnDims a = L.attn;
         a.pool_row0 = kv->num_pages * FORGE_KV_PAGE;
-        const int32_t* place = static_cast<const int32_t*>(S.place.p);
-        FORGE_TRY(qk_post(a, L.soft.qk, dt, static_cast<const float*>(S.proj.p), w.v_row, w.k_row, w.q_norm, w.k_norm, S.ropes.at(L.rot).second, S.q.p, run.pool, place, s.rows, route, st));
-        if (a.pool) FORGE_TRY(pool_blocks(a, dt, run.pool, s.rows, st));
+        const bool pools = a.pool && L.soft.talk && all_ones();
+        if (a.pool && !pools) FORGE_TRY(pool_blocks(a, dt, run.pool, s.rows, st));
         StepRows single = s.rows;
         single.n = s.single;
         const int max_keys = a.most_keys(s.max_keys), np = n - s.single;
-        if (L.soft.talk) FORGE_TRY(talk_rows(a, dt, S.q.p, run.pool, w.talk, factor, S.scores.p, S.scores.cap, S.mid.p, mid_ld, single, max_keys, st));
+        if (L.soft.talk) FORGE_TRY(talk_rows(a, dt, S.q.p, run.pool, pools, w.talk, factor, S.scores.p, S.scores.cap, S.mid.p, mid_ld, single, max_keys, st));
         else FORGE_TRY(attn_rows(a, dt, S.q.p, run.pool, nullptr, w.sink, w.bias, S.mid.p, mid_ld, single, max_keys, st));
         if (np <= 0) return FORGE_OK;
         void* out = at(S.mid.p, size_t(s.single) * mid_ld, dt);
@@ -948,24 +965,34 @@ struct Sequence {
         qkv_rows(&o, L, w, run);
         if (post) {
             FORGE_TRY(gemm(w.in, S.h.p, WP, o));
-            FORGE_TRY(attend(L, w, run, w.out.K, 1.f, nullptr));
-            return post_out(w, after);
+            FORGE_TRY(queries_and_keys(L, w, run, nullptr, nullptr));
+            FORGE_TRY(attend(L, w, run, w.out.K, 1.f));
+            return post_out(L, w, after);
         }
         o.scale = scale();
         feed_forward_rows(&o, L, w);
         FORGE_TRY(gemm(w.in, S.h.p, 2 * WP, o));
         const bool routed = L.router.experts && few_tokens(S, w, n);
         const RouteBeside route{L.router, static_cast<const float*>(S.router.p), route_tables(S.route.p, L.router, n)};
-        FORGE_TRY(attend(L, w, run, mid_columns(S, L, w, n), 1.f, routed ? &route : nullptr));
+        FORGE_TRY(queries_and_keys(L, w, run, routed ? &route : nullptr, nullptr));
+        FORGE_TRY(attend(L, w, run, mid_columns(S, L, w, n), 1.f));
         return two_norms_out(L, w, after, routed);
     }
 
-    // x += norm1(W_o mid)
-    int32_t post_out(const LayerWeights& w, const After& after) {
+    // x += norm1(W_o mid); few tokens are routed there, too
+    RouterDims router_dims(const LayerSpec& L, const LayerWeights& w) {
+        RouterDims r = L.router;
+        r.correction = w.router_bias;
+        return r;
+    }
+    bool routed_behind(const LayerSpec& L, const LayerWeights& w) { return L.router.experts && few_tokens(S, w, n) && route_behind_supported(L.router, W, n); }
+    int32_t post_out(const LayerSpec& L, const LayerWeights& w, const After& after) {
         DenseOut o;
         o.add(SEG_F32, 0, W, S.pair.p, W).add = w.out_bias;
         FORGE_TRY(gemm(w.out, S.mid.p, w.out.K, o));
-        return add_normed(x(), static_cast<const float*>(S.pair.p), n, W, S.spec.eps, w.norm1.alpha, MixtureSum{}, after, dt, st);
+        const RouterDims r = router_dims(L, w);
+        const RouteBehind route{r, w.router, WP, route_tables(S.route.p, r, n), S.scratch.tickets};
+        return add_normed(x(), static_cast<const float*>(S.pair.p), n, W, S.spec.eps, w.norm1.alpha, MixtureSum{}, after, routed_behind(L, w) ? &route : nullptr, dt, st);
     }
 
     int32_t attn_selective(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
@@ -988,7 +1015,13 @@ struct Sequence {
         a.out = at(S.mid.p, w.heads_k, dt); a.out_ld = w.out.K;
         StepRows ones = s.rows;
         ones.n = s.ones;
-        FORGE_TRY(selective_conv(d, dt, a, ones, s.segs, st));
+        if (all_ones()) {
+            const ConvBeside conv{d, a};
+            FORGE_TRY(queries_and_keys(L, w, run, nullptr, &conv));
+        } else {
+            FORGE_TRY(selective_conv(d, dt, a, ones, s.segs, st));
+            FORGE_TRY(queries_and_keys(L, w, run, nullptr, nullptr));
+        }
         {
             DenseOut o;
             o.add(SEG_CAST, 0, d.rank, S.low.p, w.low.K);
@@ -1007,26 +1040,29 @@ struct Sequence {
         }
         FORGE_TRY(selective_decode(d, dt, a, ones, st));
         FORGE_TRY(selective_segments(d, dt, a, s.segs, st));
-        FORGE_TRY(attend(L, w, run, w.out.K, L.left_scale, nullptr));
-        return post_out(w, after);
+        FORGE_TRY(attend(L, w, run, w.out.K, L.left_scale));
+        return post_out(L, w, after);
     }
 
     // x += norm2(shared expert + experts + what is passed on); see experts() for few and many tokens
     int32_t mixture(const LayerSpec& L, const LayerWeights& w, const After& after) {
-        RouterDims r = L.router;
-        r.correction = w.router_bias;
-        const bool few = few_tokens(S, w, n);
-        const int shared_k = shared_columns(L), mid_ld = few ? w.ff_out.K : shared_k;
+        const RouterDims r = router_dims(L, w);
+        const bool few = few_tokens(S, w, n), routed = routed_behind(L, w);
+        const int shared_k = shared_columns(L, w), mid_ld = few ? w.ff_out.K : shared_k;
         const RouteTables t = route_tables(S.route.p, r, n);
         const float* logits = static_cast<const float*>(S.router.p);
         float* y = static_cast<float*>(S.pair.p);
         MixtureSum sum;
         if (r.identity) sum.passed = t.passed;
-        {
+        if (!few) {
             DenseOut o;
-            o.add(SEG_SILU_GLU, 0, 2 * L.shared_ff, S.mid.p, mid_ld);
-            o.add(SEG_F32, w.router_row, r.choices(), S.router.p, r.choices());
+            o.add(SEG_F32, 0, r.choices(), S.router.p, r.choices());
+            o.add(SEG_SILU_GLU, w.glu_row, r.always * w.expert_rows, S.mid.p, mid_ld);
             FORGE_TRY(gemm(w.ff_in, S.h.p, WP, o));
+        } else if (!routed) {
+            DenseOut o;
+            o.add(SEG_F32, 0, r.choices(), S.router.p, r.choices());
+            FORGE_TRY(gemm(w.ff_in.rows(0, w.glu_row), S.h.p, WP, o));
         }
         GroupTable table;
         GroupShape shape;
@@ -1034,12 +1070,13 @@ struct Sequence {
         DenseOut in, out;
         out.add(SEG_F32, 0, W, y, W);
         if (few) {
-            FORGE_TRY(route_few(r, logits, n, t, &table, st));
+            if (routed) table = few_table(r, n, t);
+            else FORGE_TRY(route_few(r, logits, n, t, &table, st));
             shape.group_dst = size_t(w.ff_k);
-            in.add(SEG_SILU_GLU, 0, 2 * L.ff, at(S.mid.p, shared_k, dt), mid_ld);
+            in.add(SEG_SILU_GLU, 0, 2 * L.ff, S.mid.p, mid_ld);
             FORGE_TRY(dense_gemm_groups(w.experts, shape, table, S.h.p, WP, n, in, m->d_err, st));
-            FORGE_TRY(dense_gemm_listed(w.ff_out, shared_k, w.ff_k, table, S.mid.p, mid_ld, n, out, m->d_err, st));
-            return add_normed(x(), y, n, W, S.spec.eps, w.norm2.alpha, sum, after, dt, st);
+            FORGE_TRY(dense_gemm_listed(w.ff_out, shared_k, w.ff_k, listed_table(r, n, t), S.mid.p, mid_ld, n, out, m->d_err, st));
+            return add_normed(x(), y, n, W, S.spec.eps, w.norm2.alpha, sum, after, nullptr, dt, st);
         }
         FORGE_TRY(gemm(w.ff_out.columns(0, shared_k), S.mid.p, mid_ld, out));
         FORGE_TRY(route_slots(r, logits, n, t, &table, st));
@@ -1052,9 +1089,9 @@ struct Sequence {
         GroupShape cols;
         cols.rows = W; cols.group_cols = w.ff_k;
         table.weight = nullptr;
-        FORGE_TRY(dense_gemm_groups(w.ff_out.columns(shared_k, w.ff_k), cols, table, S.e_act.p, w.ff_k, pairs, down, m->d_err, st));
+        FORGE_TRY(dense_gemm_groups(w.ff_out.columns(0, w.ff_k), cols, table, S.e_act.p, w.ff_k, pairs, down, m->d_err, st));
         sum.e = static_cast<const float*>(S.e_out.p); sum.slot = t.slot; sum.top = r.top;
-        return add_normed(x(), y, n, W, S.spec.eps, w.norm2.alpha, sum, after, dt, st);
+        return add_normed(x(), y, n, W, S.spec.eps, w.norm2.alpha, sum, after, nullptr, dt, st);
     }
 
     int32_t linear(const LayerSpec& L, const LayerWeights& w, StackCache::Run& run, const After& after) {
