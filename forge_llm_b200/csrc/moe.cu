@@ -119,7 +119,7 @@ __global__ void __launch_bounds__(256) add_experts_kernel(float* __restrict__ x,
 }
 
 // A CTA per row.  NV: pieces of four columns per thread (rows of up to 1024 NV); 0: any width.
-template <typename T, int NV>
+template <typename T, int NV, bool ROUTE>
 __global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* y, int width, float eps, float gain, const MixtureSum mix, const After after, const RouteBehind route) {
     extern __shared__ __align__(16) float s_row[];     // routing: the row, its logits, then the tables
     __shared__ float red[8];
@@ -138,13 +138,14 @@ __global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* 
     };
     pdl_trigger();
     // routing, a warp per choice: the first one's weights are on their way before the wait
-    constexpr int KEEP = NV * 4;     // pieces of eight columns per lane
-    uint4 held[KEEP > 0 ? KEEP : 1];
+    constexpr int KEEP = ROUTE ? NV * 4 : 1;     // pieces of eight columns per lane
+    uint4 held[KEEP];
     const T* own_w = static_cast<const T*>(route.w) + size_t(warp) * route.ld;
-    if constexpr (NV > 0 && sizeof(T) == 2)
-        if (route.w && warp < route.d.choices())
+    if constexpr (ROUTE) {
+        if (warp < route.d.choices())
 #pragma unroll
             for (int i = 0; i < KEEP; ++i) { const int c = (lane + 32 * i) * 8; held[i] = c < width ? *reinterpret_cast<const uint4*>(own_w + c) : make_uint4(0, 0, 0, 0); }
+    }
     pdl_wait();
     const float passed = mix.passed ? mix.passed[r] : 0.f;
     if constexpr (NV > 0) {
@@ -181,10 +182,9 @@ __global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* 
             float4 v = make_float4(fmaf(f, vy[j].x, vx[j].x), fmaf(f, vy[j].y, vx[j].y), fmaf(f, vy[j].z, vx[j].z), fmaf(f, vy[j].w, vx[j].w));
             v = leave_four<T>(after, v, size_t(r), size_t(width), c, ok);
             if (ok) put4(xr + c, v);
-            if (ok && route.w) put4(s_row + c, v);
+            if (ROUTE && ok) put4(s_row + c, v);
         }
-        if constexpr (sizeof(T) == 2) {
-            if (!route.w) return;
+        if constexpr (ROUTE) {
             const int C = route.d.choices(), rows = gridDim.x;
             float* s_z = s_row + 1024 * NV;
             for (int i = width + threadIdx.x; i < 1024 * NV; i += 256) s_row[i] = 0.f;
@@ -205,23 +205,32 @@ __global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* 
                 if (lane == 0) s_z[e] = z;
             }
             float* s_w = s_z + ((C + 3) & ~3);
+            int32_t* s_expert = reinterpret_cast<int32_t*>(s_w + route.d.groups() * (kScaleRows + 1));      // the row's choice, in the end of all rows
+            const int top = route.d.top;
+            float* s_weight = reinterpret_cast<float*>(s_expert + kScaleRows * top);
             for (int i = threadIdx.x; i < route.d.groups() * (kScaleRows + 1); i += 256) s_w[i] = 0.f;
             __syncthreads();
-            if (warp == 0) choose(s_z, route.d, route.t.expert + r * route.d.top, route.t.weight + r * route.d.top);
+            if (warp == 0) {
+                if (C <= 32) choose<1>(s_z, route.d, s_expert, s_weight);
+                else choose<2>(s_z, route.d, s_expert, s_weight);
+            }
             if (rows > 1) {     // the last row makes the tables
-                if (threadIdx.x == 0) {
+                if (warp == 0) {
+                    for (int k = lane; k < top; k += 32) { route.t.expert[r * top + k] = s_expert[k]; route.t.weight[r * top + k] = s_weight[k]; }
                     __threadfence();
-                    const int before = atomicAdd(route.ticket, 1);
-                    s_last = before == rows - 1;
-                    if (s_last) { *route.ticket = 0; __threadfence(); }
+                    __syncwarp();
+                    if (lane == 0) {
+                        s_last = atomicAdd(route.ticket, 1) == rows - 1;
+                        if (s_last) *route.ticket = 0;
+                        __threadfence();
+                    }
                 }
                 __syncthreads();
                 if (!s_last) return;
-            } else {
-                __threadfence_block();
-                __syncthreads();
+                for (int i = threadIdx.x; i < rows * top; i += 256) { s_expert[i] = __ldcg(route.t.expert + i); s_weight[i] = __ldcg(route.t.weight + i); }
             }
-            route_few_tables(route.d, rows, route.t, s_w);
+            __syncthreads();
+            route_few_tables(route.d, rows, route.t, s_expert, s_weight, s_w);
         }
     } else {
         auto value = [&](int c) {
@@ -311,7 +320,7 @@ int32_t add_experts(float* x, const float* y, const RouterDims& d, const RouteTa
 
 // (a CTA per row reads all of the router; what it holds on to lies in registers)
 static int norm_pieces(int width) { return width <= 1024 ? 1 : width <= 2048 ? 2 : width <= 4096 ? 4 : 8; }
-static size_t route_behind_smem(const RouterDims& d, int width) { return size_t(1024) * norm_pieces(width) * 4 + size_t((d.choices() + 3) & ~3) * 4 + route_few_smem(d); }
+static size_t route_behind_smem(const RouterDims& d, int width) { return size_t(1024) * norm_pieces(width) * 4 + size_t((d.choices() + 3) & ~3) * 4 + route_few_smem(d) + size_t(kScaleRows) * d.top * 8; }
 bool route_behind_supported(const RouterDims& d, int width, int rows) { return rows <= kScaleRows && width % 8 == 0 && width <= 4096 && d.choices() <= 64 && route_behind_smem(d, width) <= 200 * 1024; }
 
 int32_t add_normed(float* x, const float* y, int rows, int width, float eps, float gain, const MixtureSum& mix, const After& after, const RouteBehind* route, int dtype, cudaStream_t st) {
@@ -321,7 +330,8 @@ int32_t add_normed(float* x, const float* y, int rows, int width, float eps, flo
     auto go = [&](auto type) -> int32_t {
         using T = decltype(type);
         const int nv = norm_pieces(width);
-        auto kern = wide ? add_normed_kernel<T, 0> : nv == 1 ? add_normed_kernel<T, 1> : nv == 2 ? add_normed_kernel<T, 2> : nv == 4 ? add_normed_kernel<T, 4> : add_normed_kernel<T, 8>;
+        auto kern = wide ? add_normed_kernel<T, 0, false> : nv == 1 ? add_normed_kernel<T, 1, false> : nv == 2 ? add_normed_kernel<T, 2, false> : nv == 4 ? add_normed_kernel<T, 4, false> : add_normed_kernel<T, 8, false>;
+        if (route) kern = nv == 1 ? add_normed_kernel<__nv_bfloat16, 1, true> : nv == 2 ? add_normed_kernel<__nv_bfloat16, 2, true> : add_normed_kernel<__nv_bfloat16, 4, true>;
         const size_t smem = route ? route_behind_smem(route->d, width) : 0;
         if (smem > 48 * 1024) FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
         FORGE_CUDA(launch_pdl(kern, dim3(rows), dim3(256), smem, st, x, y, width, eps, gain, mix, after, route ? *route : RouteBehind{}));

@@ -50,8 +50,10 @@ int32_t add_normed(float* x, const float* y, int rows, int width, float eps, flo
 #ifdef __CUDACC__
 constexpr int kPerLane = kMaxExperts / 32;
 
-// The warp chooses a row's experts (lower numbers win ties); expert[k] and weight[k] by lane 0.
+// The warp chooses a row's experts (lower numbers win ties); expert[k] and weight[k] by lane 0.  PER: choices per lane.
+template <int PER = kPerLane>
 __device__ __forceinline__ void choose(const float* z, const RouterDims& d, int32_t* expert, float* weight) {
+    constexpr int kPerLane = PER;
     const int lane = threadIdx.x & 31, experts = d.choices(), top = d.top;
     float v[kPerLane];
     uint32_t taken = 0;
@@ -87,13 +89,13 @@ __device__ __forceinline__ void choose(const float* z, const RouterDims& d, int3
         at = __shfl_sync(0xffffffffu, at, 0);      // (values that are no numbers compare differently in different lanes)
         best = __shfl_sync(0xffffffffu, best, 0);
         if ((at & 31) == lane) taken |= 1u << (at >> 5);
-        if (d.correction) { if (lane == 0) { expert[k] = at; weight[k] = expf(z[at] - first); } continue; }
+        if (d.correction) { if (lane == 0) { expert[k] = at; weight[k] = expf(z[at] - first) / sum; } continue; }
         if (k == 0) first = best;
         const float e = expf(best - first);
         sum += e;
         if (lane == 0) { expert[k] = at; weight[k] = e; }
     }
-    if (lane == 0) for (int k = 0; k < top; ++k) weight[k] /= sum;
+    if (lane == 0 && !d.correction) for (int k = 0; k < top; ++k) weight[k] /= sum;
     __syncwarp();
 }
 
@@ -102,8 +104,8 @@ __device__ __forceinline__ void route_few_clear(const RouterDims& d, float* s_w)
     for (int i = threadIdx.x; i < d.groups() * (kScaleRows + 1); i += blockDim.x) s_w[i] = 0.f;
     __syncthreads();
 }
-// the tables of rows whose choices lie in t.expert and t.weight
-__device__ __forceinline__ void route_few_tables(const RouterDims& d, int rows, const RouteTables& t, float* s_w) {
+// the tables of rows whose choices lie in expert and weight, [rows][top]
+__device__ __forceinline__ void route_few_tables(const RouterDims& d, int rows, const RouteTables& t, const int32_t* expert, const float* weight, float* s_w) {
     const int G = d.groups();
     int* used = reinterpret_cast<int*>(s_w + G * kScaleRows);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -113,9 +115,10 @@ __device__ __forceinline__ void route_few_tables(const RouterDims& d, int rows, 
     }
     for (int r = threadIdx.x; r < rows; r += blockDim.x) {
         float passed = 0.f;
+#pragma unroll 4
         for (int k = 0; k < d.top; ++k) {
-            const int e = __ldcg(t.expert + r * d.top + k);
-            const float w = __ldcg(t.weight + r * d.top + k);
+            const int e = expert[r * d.top + k];
+            const float w = weight[r * d.top + k];
             if (e >= d.experts) { passed += w; continue; }
             s_w[(d.always + e) * kScaleRows + r] = w;
             used[d.always + e] = 1;
@@ -142,7 +145,7 @@ __device__ __forceinline__ void route_few_rows(const RouterDims& d, const float*
     for (int r = threadIdx.x >> 5; r < rows; r += blockDim.x / 32) choose(logits + size_t(r) * d.choices(), d, t.expert + r * d.top, t.weight + r * d.top);
     __threadfence_block();
     __syncthreads();
-    route_few_tables(d, rows, t, s_w);
+    route_few_tables(d, rows, t, t.expert, t.weight, s_w);
 }
 #endif
 
