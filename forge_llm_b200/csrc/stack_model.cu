@@ -1399,9 +1399,10 @@ int32_t stack_step(ForgeModel* m, ForgeKV* kv, const ForgeStepEntry* entries, in
     bool prompt_ok = S.dtype == FORGE_BF16;
     int least_pool = 0;   // of all layers
     for (const LayerSpec& L : S.spec.layers) {
+        if (!L.has_latent() && !L.has_attn()) continue;
         PromptDims d = L.has_latent() ? PromptDims(L.mix) : PromptDims(L.attn);
         d.joint = L.soft.talk;
-        prompt_ok = prompt_ok && ((!L.has_latent() && !L.has_attn()) || attn_prefill_kv_supported(d));
+        prompt_ok = prompt_ok && attn_prefill_kv_supported(d);
         if (L.has_attn() && L.attn.pool) least_pool = least_pool ? std::min(least_pool, L.attn.pool) : L.attn.pool;
     }
     // rows: the single tokens first, then the short entries, then the prompt portions
