@@ -5,14 +5,24 @@ namespace forge {
 
 namespace {
 
-// A CTA per row of the step; eight columns per thread.
+// A CTA per eight rows of the step; eight columns per thread.
+constexpr int kPoolRows = 8;
 template <typename T>
 __global__ void __launch_bounds__(128) pool_blocks_kernel(const AttnDims d, T* cache, const StepRows rows) {
-    const int r = blockIdx.x, pos = rows.pos[r], seq = rows.seq ? rows.seq[r] : r;
     pdl_trigger();
     pdl_wait();
-    const int32_t* pt = rows.page_table + size_t(seq) * rows.pages_per_seq;
-    for (int c = 0; c < d.row(); c += 128 * 8) pool_columns(d, cache, pt, pos, c, min(128, (d.row() - c) / 8));
+    const int r0 = blockIdx.x * kPoolRows;
+    int at[kPoolRows];
+#pragma unroll
+    for (int i = 0; i < kPoolRows; ++i) at[i] = r0 + i < rows.n ? rows.pos[r0 + i] : 0;
+#pragma unroll
+    for (int i = 0; i < kPoolRows; ++i) {
+        const int r = r0 + i, pos = at[i];
+        if (r >= rows.n || (pos + 1) % d.pool) continue;
+        const int seq = rows.seq ? rows.seq[r] : r;
+        const int32_t* pt = rows.page_table + size_t(seq) * rows.pages_per_seq;
+        for (int c = 0; c < d.row(); c += 128 * 8) pool_columns(d, cache, pt, pos, c, min(128, (d.row() - c) / 8));
+    }
 }
 
 // Rows that are no block yet become zeros: their weights are zero, so they must be finite.
@@ -31,8 +41,8 @@ __global__ void __launch_bounds__(128) gather_blocks_kernel(const AttnDims d, in
 
 int32_t pool_blocks(const AttnDims& d, int dtype, void* cache, const StepRows& rows, cudaStream_t st) {
     if (rows.n <= 0) return FORGE_OK;
-    if (dtype == FORGE_F32) FORGE_CUDA(launch_pdl(pool_blocks_kernel<float>, dim3(rows.n), dim3(128), 0, st, d, static_cast<float*>(cache), rows));
-    else FORGE_CUDA(launch_pdl(pool_blocks_kernel<__nv_bfloat16>, dim3(rows.n), dim3(128), 0, st, d, static_cast<__nv_bfloat16*>(cache), rows));
+    if (dtype == FORGE_F32) FORGE_CUDA(launch_pdl(pool_blocks_kernel<float>, dim3((rows.n + kPoolRows - 1) / kPoolRows), dim3(128), 0, st, d, static_cast<float*>(cache), rows));
+    else FORGE_CUDA(launch_pdl(pool_blocks_kernel<__nv_bfloat16>, dim3((rows.n + kPoolRows - 1) / kPoolRows), dim3(128), 0, st, d, static_cast<__nv_bfloat16*>(cache), rows));
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }

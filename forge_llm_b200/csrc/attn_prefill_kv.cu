@@ -7,7 +7,8 @@
 // those come first, gathered into rows by sequence), scores may have a bias by distance, a sink may stand in the denominator, several sequences'
 // tiles run in one launch (a table gives each tile's rows, position and context), and the epilogue applies an output gate per value or per
 // head.  Joint values: a CTA meets up to four 64-column pieces of all groups' values, so that heads' weights can be mixed behind it.
-// Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = softmax, rescale, store.
+// Warp roles (192 threads): 0 = TMA producer, 1 = TMEM allocation and MMA issue, 2..5 = softmax, rescale, store.  Where a bound of the scores is known
+// (BOUND, 320 threads) it stands in for the maximum: nothing is ever rescaled, and eight warps, two per 32 rows, take half of a tile's columns each.
 // Tensor memory: S [0, 64), P0 [64, 96), P1 [96, 128), O from 128.
 #include <algorithm>
 
@@ -20,9 +21,10 @@ namespace {
 
 using namespace tc5;
 
-constexpr int BM = 128, BN = 64, kThreads = 192;
+constexpr int BM = 128, BN = 64;
 constexpr uint32_t kColS = 0, kColP = 64, kColO = 128;
 constexpr float kLazy = 8.f;
+constexpr float kMostBound = 35.f;   // weights from exp(-2 * 35) on are far from the smallest numbers
 
 struct Params {
     PromptDims d;
@@ -49,10 +51,11 @@ __device__ __forceinline__ float ex2(float x) {
     return y;
 }
 
-template <uint32_t COLS>
-__global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+template <uint32_t COLS, bool BOUND>
+__global__ void __launch_bounds__(BOUND ? 320 : 192, COLS <= 256 ? 2 : 1) attn_prefill_kv_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                                                                    const __grid_constant__ CUtensorMap map_r, const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_bk,
                                                                    const __grid_constant__ CUtensorMap map_bv, const __grid_constant__ Params p) {
+    constexpr int WARPS = BOUND ? 8 : 4, kThreads = 64 + 32 * WARPS, NC = BOUND ? 32 : 64;   // softmax warps; columns of a tile per thread
     constexpr int Q_CHUNK = BM * 128, KV_CHUNK = BN * 128, kMaxStages = 3;
     const PromptDims& d = p.d;
     const int h = int(blockIdx.x) % d.heads, vp0 = int(blockIdx.x) / d.heads * p.pieces;   // first piece of the values
@@ -65,6 +68,7 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
     __shared__ uint64_t q_full, kv_full[kMaxStages], kv_empty[kMaxStages], s_full, s_free, p_full[2], pv_done[2];
     __shared__ uint32_t s_tmem;
     __shared__ int s_err;
+    __shared__ float s_sum[BOUND ? 2 : 1][BM];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const PromptTile t = p.a.tiles[blockIdx.y];
     auto first_key = [&](int pos) { return first_visible(d, pos); };
@@ -76,8 +80,8 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
         mbar_init(&q_full, 1);
         for (int s = 0; s < kMaxStages; ++s) { mbar_init(&kv_full[s], 1); mbar_init(&kv_empty[s], 1); }
         mbar_init(&s_full, 1);
-        mbar_init(&s_free, 4);
-        for (int s = 0; s < 2; ++s) { mbar_init(&p_full[s], 4); mbar_init(&pv_done[s], 1); }
+        mbar_init(&s_free, WARPS);
+        for (int s = 0; s < 2; ++s) { mbar_init(&p_full[s], WARPS); mbar_init(&pv_done[s], 1); }
         s_err = 0;
         mbar_fence_init();
     }
@@ -142,7 +146,7 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
             if (!ok) atomicExch(&s_err, 1);
         }
     } else {
-        const int quad = warp & 3;
+        const int quad = warp & 3, half = BOUND ? (warp - 2) / 4 : 0, col0 = half * NC;   // of the tile
         const int r = quad * 32 + lane;
         const int pq = t.pos0 + r, lo = first_key(pq), keep = d.window > 0 ? d.keep : 0;
         const int lo_last = first_key(t.pos0 + t.rows - 1);   // of the tile's last row
@@ -151,49 +155,51 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
         const float own2 = d.softcap > 0.f ? d.softcap * 1.4426950408889634f : p.scale2, scale2 = bias ? 1.f : own2, cap2 = d.softcap > 0.f ? 2.f * p.scale2 / d.softcap : 0.f;
         const uint32_t lane_addr = tmem + (uint32_t(quad * 32) << 16);
         const uint32_t masked = scale2 < 0.f ? 0x7f800000u : 0xff800000u;   // -inf behind the scale
-        float m_ref = -INFINITY, l_run = 0.f;
+        float m_ref = BOUND ? d.bound * 1.4426950408889634f : -INFINITY, l_run = 0.f;
         bool ok = true;
         for (int j = 0; j < nblk; ++j) {
-            const int t0 = key_tile(j) * BN;
+            const int t0 = key_tile(j) * BN + col0;
             if (ok && !mbar_wait(&s_full, j & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
             fence_after();
-            uint32_t sv[2][32];
-            tmem_ld32(lane_addr + kColS, sv[0]);
-            tmem_ld32(lane_addr + kColS + 32, sv[1]);
+            uint32_t sv[NC / 32][32];
+#pragma unroll
+            for (int c = 0; c < NC / 32; ++c) tmem_ld32(lane_addr + kColS + col0 + 32 * c, sv[c]);
             wait_ld();
             fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(&s_free);
             if (d.softcap > 0.f) {   // tanh(x) = 1 - 2 / (1 + exp(2 x)); own2 then holds the cap
 #pragma unroll
-                for (int c = 0; c < 64; ++c) sv[c >> 5][c & 31] = __float_as_uint(1.f - __fdividef(2.f, 1.f + ex2(fminf(__uint_as_float(sv[c >> 5][c & 31]) * cap2, 120.f))));
+                for (int c = 0; c < NC; ++c) sv[c >> 5][c & 31] = __float_as_uint(1.f - __fdividef(2.f, 1.f + ex2(fminf(__uint_as_float(sv[c >> 5][c & 31]) * cap2, 120.f))));
             }
             if (bias) {   // scores and biases in the logarithm's base: scale2 is one
 #pragma unroll
-                for (int c = 0; c < 64; ++c)
+                for (int c = 0; c < NC; ++c)
                     sv[c >> 5][c & 31] = __float_as_uint(fmaf(__uint_as_float(sv[c >> 5][c & 31]), own2, bias[max(0, min(pq - t0 - c, d.bias_n - 1))] * bias2));
             }
             if (d.pool > 0 && j < head) {
                 const int seen = lo / d.pool;
 #pragma unroll
-                for (int c = 0; c < 64; ++c) if (t0 + c >= seen) sv[c >> 5][c & 31] = masked;
-            } else if (t0 + BN - 1 > t.pos0 || (t0 < lo_last && t0 + BN > keep)) {
+                for (int c = 0; c < NC; ++c) if (t0 + c >= seen) sv[c >> 5][c & 31] = masked;
+            } else if (t0 + NC - 1 > t.pos0 || (t0 < lo_last && t0 + NC > keep)) {
 #pragma unroll
-                for (int c = 0; c < 64; ++c)
+                for (int c = 0; c < NC; ++c)
                     if (t0 + c > pq || (t0 + c < lo && t0 + c >= keep)) sv[c >> 5][c & 31] = masked;
             }
-            float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-#pragma unroll
-            for (int c = 0; c < 64; ++c) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(sv[c >> 5][c & 31]) * scale2);   // the scale may have either sign
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
             float alpha = 1.f;
-            if (m_ref == -INFINITY) m_ref = mx;
-            else if (mx > m_ref + kLazy) { alpha = ex2(m_ref - mx); m_ref = mx; }
+            if constexpr (!BOUND) {
+                float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+                for (int c = 0; c < NC; ++c) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(sv[c >> 5][c & 31]) * scale2);   // the scale may have either sign
+                const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+                if (m_ref == -INFINITY) m_ref = mx;
+                else if (mx > m_ref + kLazy) { alpha = ex2(m_ref - mx); m_ref = mx; }
+            }
             const float m_use = m_ref == -INFINITY ? 0.f : m_ref;
             float sum4[4] = {0.f, 0.f, 0.f, 0.f};
-            uint32_t ph[32];
+            uint32_t ph[NC / 2];
 #pragma unroll
-            for (int c = 0; c < 64; c += 2) {
+            for (int c = 0; c < NC; c += 2) {
                 const float p0 = ex2(fmaf(__uint_as_float(sv[c >> 5][c & 31]), scale2, -m_use));
                 const float p1 = ex2(fmaf(__uint_as_float(sv[c >> 5][(c & 31) + 1]), scale2, -m_use));
                 sum4[(c >> 1) & 3] += p0 + p1;
@@ -201,7 +207,7 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
             }
             l_run = l_run * alpha + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
             if (j >= 2 && ok && !mbar_wait(&pv_done[j & 1], ((j >> 1) - 1) & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
-            if (j > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
+            if (!BOUND && j > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
                 if (ok && !mbar_wait(&pv_done[(j - 1) & 1], ((j - 1) >> 1) & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
                 fence_after();
                 for (int c0 = 0; c0 < vch * 64; c0 += 32) {
@@ -214,7 +220,8 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
                 }
             }
             fence_after();
-            tmem_st32(lane_addr + kColP + uint32_t((j & 1) * 32), ph);
+            if constexpr (BOUND) tmem_st16(lane_addr + kColP + uint32_t((j & 1) * 32 + half * 16), ph);
+            else tmem_st32(lane_addr + kColP + uint32_t((j & 1) * 32), ph);
             wait_st();
             fence_before();
             __syncwarp();
@@ -222,6 +229,11 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
         }
         if (ok && !mbar_wait(&pv_done[(nblk - 1) & 1], ((nblk - 1) >> 1) & 1, &s_err)) { atomicExch(&s_err, 1); ok = false; }
         fence_after();
+        if constexpr (BOUND) {   // both halves of a row
+            s_sum[half][r] = l_run;
+            asm volatile("bar.sync 1, %0;" ::"n"(32 * WARPS) : "memory");
+            l_run += s_sum[half ^ 1][r];
+        }
         const bool per_value = p.a.gate != nullptr;
         if (p.a.sink) {
             const float own = p.a.sink[h] * 1.4426950408889634f;
@@ -233,7 +245,7 @@ __global__ void __launch_bounds__(kThreads) attn_prefill_kv_kernel(const __grid_
         const int width = d.joint ? vch * 64 : d.vdim;
         __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.a.out) + size_t(t.row0 + r) * p.a.out_ld + (d.joint ? h * value_pieces(d) * 64 + vp0 * 64 : h * d.vdim);
         const bool vec = !(width & 7) && !(p.a.gate_ld & 7) && !(p.a.out_ld & 7);   // 16-byte pieces stay aligned
-        for (int c0 = 0; c0 < width; c0 += 32) {
+        for (int c0 = half * 32; c0 < width; c0 += 32 * (WARPS / 4)) {
             uint32_t o[32];
             tmem_ld32(lane_addr + kColO + c0, o);
             wait_ld();
@@ -296,7 +308,7 @@ int32_t attn_prefill_kv(const PromptDims& d, const PromptAttnArgs& a, cudaStream
         FORGE_TRY(make_map_3d(&bv, static_cast<const __nv_bfloat16*>(a.blocks) + G * d.dim_p, uint64_t(d.vdim_p), G, uint64_t(a.block_rows), uint64_t(d.vdim_p) * 2, v_row, BN));
     } else { bk = mk; bv = mv; }
     // three stages, or two where that lets two CTAs share an SM: if the work of an SM, not the longest tile, decides
-    auto fit = [&](int stages, size_t ctas) { return ctas * (smem_bytes(d, stages) + 1024) <= 226 * 1024; };
+    auto fit = [&](int stages, size_t ctas) { return ctas * (smem_bytes(d, stages) + 2048) <= 226 * 1024; };
     long long total = 0, longest = 0;
     for (int i = 0; i < a.n_tiles && a.host_tiles; ++i) {
         const PromptTile& t = a.host_tiles[i];
@@ -309,13 +321,15 @@ int32_t attn_prefill_kv(const PromptDims& d, const PromptAttnArgs& a, cudaStream
     const bool share = longest * 148 < total * parts && pieces <= 2;
     Params p{d, a, d.scale * 1.4426950408889634f, fit(3, share ? 2 : 1) ? 3 : fit(2, share ? 2 : 1) ? 2 : fit(3, 1) ? 3 : 2, pieces};
     const size_t smem = smem_bytes(d, p.stages);
+    const bool bound = d.bound > 0.f && d.bound <= kMostBound;
     auto go = [&](auto kern) -> int32_t {
         FORGE_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
-        kern<<<dim3(d.heads * parts, a.n_tiles), kThreads, smem, st>>>(mq, mk, mr, mv, bk, bv, p);
+        kern<<<dim3(d.heads * parts, a.n_tiles), bound ? 320 : 192, smem, st>>>(mq, mk, mr, mv, bk, bv, p);
         FORGE_LAUNCH_CHECK();
         return FORGE_OK;
     };
-    return pieces <= 2 ? go(attn_prefill_kv_kernel<256>) : go(attn_prefill_kv_kernel<512>);
+    if (bound) return pieces <= 2 ? go(attn_prefill_kv_kernel<256, true>) : go(attn_prefill_kv_kernel<512, true>);
+    return pieces <= 2 ? go(attn_prefill_kv_kernel<256, false>) : go(attn_prefill_kv_kernel<512, false>);
 }
 
 }  // namespace forge

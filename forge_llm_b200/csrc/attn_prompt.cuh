@@ -12,6 +12,7 @@ struct PromptDims {
     int dim_p = 0, rot_p = 0, vdim_p = 0;     // padded to 64
     float scale = 1.f, softcap = 0.f;
     int chunk = 0, window = 0, keep = 0, pool = 0, bias_n = 0;   // as in AttnDims
+    float bound = 0.f;                        // > 0: no score (bias included) is larger or smaller than this
     bool joint = false;                       // every head meets the values of all groups: out [row][head][group][vdim_p]
     PromptDims() = default;
     explicit PromptDims(const LatentDims& d) : heads(d.heads), dim(d.dim), rot(d.rot), vdim(d.vdim), dim_p(d.dim_p), rot_p(d.rot_p), vdim_p(d.vdim_p), scale(d.scale) {}

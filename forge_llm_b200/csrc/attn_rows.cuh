@@ -75,7 +75,7 @@ __device__ __forceinline__ void pool_columns(const AttnDims& d, T* cache, const 
     float sum[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) sum[e] = 0.f;
-#pragma unroll 8
+#pragma unroll 16
     for (int t = b * d.pool; t <= pos; ++t) {
         float v[8];
         load8(v, cache + (size_t(pt[t / FORGE_KV_PAGE]) * FORGE_KV_PAGE + t % FORGE_KV_PAGE) * W + c);

@@ -467,48 +467,64 @@ __global__ void __launch_bounds__(kThreads) talk_values_mma_kernel(const AttnDim
 
 // ------------------------------------------------------------------------------------------------ behind prompt attention
 constexpr int kMixHeads = 4;     // heads of a group that a thread carries
+constexpr int kMixThreads = 128, kAhead = 8;   // sources whose values are requested together
 // A thread = eight columns of one group of one row.
-__global__ void __launch_bounds__(256) talk_heads_kernel(const AttnDims d, const bf16* __restrict__ o, const float* __restrict__ talk, float factor, bf16* __restrict__ out, int out_ld, int rows) {
-    extern __shared__ float mix[];      // [heads][heads], transposed: the weights of one source head lie side by side
-    for (int i = threadIdx.x; i < d.heads * d.heads; i += 256) mix[i] = talk[size_t(i % d.heads) * d.heads + i / d.heads] * factor;
-    __syncthreads();
-    const int pieces = d.vdim_p / 8, per = d.groups * pieces, gq = d.heads / d.groups;
-    const size_t i = size_t(blockIdx.x) * 256 + threadIdx.x;
+__global__ void __launch_bounds__(kMixThreads) talk_heads_kernel(const AttnDims d, const bf16* __restrict__ o, const float* __restrict__ talk, float factor, bf16* __restrict__ out, int out_ld, int rows) {
+    extern __shared__ __align__(16) float mix[];      // [source head][heads, padded]
+    const int pieces = d.vdim_p / 8, per = d.groups * pieces, gq = d.heads / d.groups, gq_p = (gq + kMixHeads - 1) / kMixHeads * kMixHeads, ld = d.groups * gq_p;
+    const size_t i = size_t(blockIdx.x) * kMixThreads + threadIdx.x;
     const int r = int(i / per), g = int(i % per) / pieces, c = int(i % pieces) * 8;
-    if (r >= rows || c >= d.vdim) return;
+    const bool on = r < rows && c < d.vdim;
     const size_t W = size_t(d.groups) * d.vdim_p;
-    const bf16* src = o + size_t(r) * d.heads * W + size_t(g) * d.vdim_p + c;
+    const bf16* src = o + size_t(on ? r : 0) * d.heads * W + size_t(g) * d.vdim_p + c;
+    uint4 held[kAhead];
+    auto fetch = [&](int x0) {
+#pragma unroll
+        for (int j = 0; j < kAhead; ++j) held[j] = on && x0 + j < d.heads ? *reinterpret_cast<const uint4*>(src + size_t(x0 + j) * W) : make_uint4(0, 0, 0, 0);
+    };
+    fetch(0);
+    for (int k = threadIdx.x; k < d.heads * ld; k += kMixThreads) {
+        const int x = k / ld, h = k % ld / gq_p * gq + k % gq_p;
+        mix[k] = k % gq_p < gq ? talk[size_t(h) * d.heads + x] * factor : 0.f;
+    }
+    __syncthreads();
     for (int h0 = 0; h0 < gq; h0 += kMixHeads) {
         float acc[kMixHeads][8];
 #pragma unroll
         for (int h = 0; h < kMixHeads; ++h)
 #pragma unroll
             for (int e = 0; e < 8; ++e) acc[h][e] = 0.f;
-        const int nh = min(kMixHeads, gq - h0);
-#pragma unroll 8
-        for (int x = 0; x < d.heads; ++x) {
-            float v[8];
-            load8(v, src + size_t(x) * W);
-            const float* w = mix + x * d.heads + g * gq + h0;
+        if (h0 > 0) fetch(0);
+        for (int x0 = 0; x0 < d.heads; x0 += kAhead) {
+            uint4 now[kAhead];
 #pragma unroll
-            for (int h = 0; h < kMixHeads; ++h)
-                if (h < nh)
+            for (int j = 0; j < kAhead; ++j) now[j] = held[j];
+            if (x0 + kAhead < d.heads) fetch(x0 + kAhead);
+#pragma unroll
+            for (int j = 0; j < kAhead; ++j) {
+                if (x0 + j >= d.heads) break;
+                float v[8];
+                load8(v, reinterpret_cast<const bf16*>(&now[j]));
+                const float4 w4 = get4(mix + (x0 + j) * ld + g * gq_p + h0);
+                const float w[kMixHeads] = {w4.x, w4.y, w4.z, w4.w};
+#pragma unroll
+                for (int h = 0; h < kMixHeads; ++h)
 #pragma unroll
                     for (int e = 0; e < 8; ++e) acc[h][e] = fmaf(w[h], v[e], acc[h][e]);
+            }
         }
+        if (!on) continue;
 #pragma unroll
         for (int h = 0; h < kMixHeads; ++h)
-            if (h < nh) {
+            if (h0 + h < gq) {
                 bf16* dst = out + size_t(r) * out_ld + size_t(g * gq + h0 + h) * d.vdim + c;
                 if (d.vdim % 8 == 0 && out_ld % 8 == 0) {
-                    uint4 u;
-                    __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&u);
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) p[e] = __floats2bfloat162_rn(acc[h][2 * e], acc[h][2 * e + 1]);
-                    *reinterpret_cast<uint4*>(dst) = u;
-                } else
+                    put4(dst, make_float4(acc[h][0], acc[h][1], acc[h][2], acc[h][3]));
+                    put4(dst + 4, make_float4(acc[h][4], acc[h][5], acc[h][6], acc[h][7]));
+                } else {
 #pragma unroll
                     for (int e = 0; e < 8; ++e) if (c + e < d.vdim) dst[e] = __float2bfloat16_rn(acc[h][e]);
+                }
             }
     }
 }
@@ -560,7 +576,8 @@ int32_t run_mma(const AttnDims& d, const void* q, void* cache, bool pools, const
 
 }  // namespace
 
-bool talk_rows_supported(const AttnDims& d) { return d.heads <= 128 && d.vdim_p <= 512 && d.keep == 0 && d.bias_n == 0 && plain_score_smem(d) <= 200 * 1024 && plain_value_smem(d) <= 200 * 1024; }
+static size_t mix_smem(const AttnDims& d) { return size_t(d.heads) * d.groups * pad_to(d.heads / d.groups, kMixHeads) * 4; }
+bool talk_rows_supported(const AttnDims& d) { return d.heads <= 128 && mix_smem(d) <= 200 * 1024 && d.vdim_p <= 512 && d.keep == 0 && d.bias_n == 0 && plain_score_smem(d) <= 200 * 1024 && plain_value_smem(d) <= 200 * 1024; }
 size_t talk_rows_bytes(const AttnDims& d, int rows, int max_keys) { return size_t(rows) * score_row(d, max_keys).floats() * sizeof(float); }
 
 int32_t talk_rows(const AttnDims& d, int dtype, const void* q, void* cache, bool pools, const float* talk, float factor, void* scratch, size_t max_bytes, void* out, int out_ld, const StepRows& rows, int max_keys,
@@ -587,9 +604,9 @@ int32_t talk_rows(const AttnDims& d, int dtype, const void* q, void* cache, bool
 
 int32_t talk_heads(const AttnDims& d, const void* o, const float* talk, float factor, void* out, int out_ld, int rows, cudaStream_t st) {
     if (rows <= 0) return FORGE_OK;
-    const size_t smem = size_t(d.heads) * d.heads * 4, threads = size_t(rows) * d.groups * (d.vdim_p / 8);
+    const size_t smem = mix_smem(d), threads = size_t(rows) * d.groups * (d.vdim_p / 8);
     FORGE_TRY(allow_smem(talk_heads_kernel, smem));
-    talk_heads_kernel<<<unsigned((threads + 255) / 256), 256, smem, st>>>(d, static_cast<const bf16*>(o), talk, factor, static_cast<bf16*>(out), out_ld, rows);
+    talk_heads_kernel<<<unsigned((threads + kMixThreads - 1) / kMixThreads), kMixThreads, smem, st>>>(d, static_cast<const bf16*>(o), talk, factor, static_cast<bf16*>(out), out_ld, rows);
     FORGE_LAUNCH_CHECK();
     return FORGE_OK;
 }

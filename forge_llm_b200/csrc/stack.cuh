@@ -59,6 +59,7 @@ struct LayerSpec {
     Rotation rot;                            // Latent, Softmax
     SoftmaxTraits soft;                      // Softmax, AttnSelective
     DistanceBuckets distance;
+    float score_bound = 0.f;                 // plain: no score in front of the bias is larger or smaller than this
     int blend_layer = -1;                    // values are blended with those of this earlier layer
     bool blends = false;                     // takes part in it (the first such layer lends its values)
     SelectiveDims sel;                       // AttnSelective

@@ -212,6 +212,10 @@ int32_t parse_softmax(const Json* m, float eps, const MixerName& name, LayerSpec
     }
     L->soft = soft;
     L->soft.qk.eps = eps; L->soft.qk.rot_dims = L->rot.dims;
+    if (soft.plain) {   // queries and keys are no longer than the root of their size (a little for rounding)
+        L->score_bound = 1.01f * std::fabs(a.scale) * float(a.dim);
+        if (a.softcap > 0.f) L->score_bound = std::min(L->score_bound, a.softcap);
+    }
     return FORGE_OK;
 }
 

@@ -50,6 +50,7 @@ struct LayerWeights {
     float *mu = nullptr, *norm_l = nullptr, *norm_r = nullptr;
     // attention with normed queries and keys (k_row, v_row as above)
     float *q_norm = nullptr, *k_norm = nullptr, *sink = nullptr, *q_bias = nullptr, *k_bias = nullptr, *v_bias = nullptr;
+    float bias_bound = 0.f;       // largest bias by distance
     float *bias = nullptr, *talk = nullptr, *out_bias = nullptr, lambda = 0.f;   // biases by distance, mixing of heads, share of the blended values
     // selective scan (in_row, gate_row: first rows in `in`; conv, low as above): rows [step sizes' inner values | B C] over the channels
     DenseWeight scan_in;
@@ -355,6 +356,7 @@ int32_t load_plain_attention(ForgeModel* m, const LayerSpec& L, const TensorSet&
         std::vector<float> by;   // [head][distance]
         for (int h = 0; h < a.heads; ++h)
             for (int n = 0; n < a.bias_n; ++n) by.push_back(t.at(at + "rel")->at(size_t(L.distance.of(n)) * a.heads + h));
+        for (float b : by) w->bias_bound = std::max(w->bias_bound, std::fabs(b));
         FORGE_TRY(upload_values(m, &w->bias, by));
     }
     if (L.blend_layer >= 0) w->lambda = t.at(at + "vmix")->at(0);
@@ -943,6 +945,7 @@ struct Sequence {
         if (np <= 0) return FORGE_OK;
         void* out = at(S.mid.p, size_t(s.single) * mid_ld, dt);
         PromptDims d(a);
+        if (L.score_bound > 0.f) d.bound = L.score_bound + w.bias_bound;
         PromptAttnArgs p;
         p.q = at(S.q.p, size_t(s.single) * a.heads * a.dim_p, dt); p.k = run.pool; p.v = at(run.pool, size_t(a.groups) * a.dim_p, dt);
         p.sink = w.sink; p.bias = w.bias;
