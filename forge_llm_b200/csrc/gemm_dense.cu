@@ -705,6 +705,8 @@ int32_t launch_dense(const DenseWeight& w, const void* act, int act_ld, int act_
     if (NT <= 32 && tiles <= sms) {
         int parts = 0;
         FORGE_TRY((cluster_parts<NT, MODE>(tiles, p.nk, smem, &parts)));
+        // a table stands in front of the first load: two CTAs per SM have twice as much on its way behind it
+        if (MODE == GROUPED && NT <= 16 && parts == 1 && p.nk >= 8) parts = 2;
         if (parts > 0) {
             p.cluster = parts;
             FORGE_CUDA(launch_pdl_cluster(kern, dim3(unsigned(tiles * parts)), dim3(kThreads<NT>), parts, smem, st, mx, p));

@@ -139,12 +139,19 @@ __global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* 
     pdl_trigger();
     // routing, a warp per choice: the first one's weights are on their way before the wait
     constexpr int KEEP = ROUTE ? NV * 4 : 1;     // pieces of eight columns per lane
-    uint4 held[KEEP];
+    uint4 held[KEEP], held2[NV <= 2 ? KEEP : 1];
+    __shared__ float s_corr[ROUTE ? 64 : 1];
     const T* own_w = static_cast<const T*>(route.w) + size_t(warp) * route.ld;
     if constexpr (ROUTE) {
         if (warp < route.d.choices())
 #pragma unroll
             for (int i = 0; i < KEEP; ++i) { const int c = (lane + 32 * i) * 8; held[i] = c < width ? *reinterpret_cast<const uint4*>(own_w + c) : make_uint4(0, 0, 0, 0); }
+        if constexpr (NV <= 2) {
+            if (warp + 8 < route.d.choices())
+#pragma unroll
+                for (int i = 0; i < KEEP; ++i) { const int c = (lane + 32 * i) * 8; held2[i] = c < width ? *reinterpret_cast<const uint4*>(own_w + size_t(8) * route.ld + c) : make_uint4(0, 0, 0, 0); }
+        }
+        if (route.d.correction && int(threadIdx.x) < route.d.choices()) s_corr[threadIdx.x] = route.d.correction[threadIdx.x];
     }
     pdl_wait();
     const float passed = mix.passed ? mix.passed[r] : 0.f;
@@ -195,7 +202,8 @@ __global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* 
                 for (int i = 0; i < KEEP; ++i) {
                     const int c = (lane + 32 * i) * 8;
                     float w[8], v[8];
-                    if (e != warp) held[i] = c < width ? *reinterpret_cast<const uint4*>(own_w + size_t(e - warp) * route.ld + c) : make_uint4(0, 0, 0, 0);
+                    if (NV <= 2 && e == warp + 8) held[i] = held2[NV <= 2 ? i : 0];
+                    else if (e != warp) held[i] = c < width ? *reinterpret_cast<const uint4*>(own_w + size_t(e - warp) * route.ld + c) : make_uint4(0, 0, 0, 0);
                     load8(w, reinterpret_cast<const T*>(&held[i]));
                     load8(v, s_row + c);
 #pragma unroll
@@ -211,8 +219,10 @@ __global__ void __launch_bounds__(256) add_normed_kernel(float* x, const float* 
             for (int i = threadIdx.x; i < route.d.groups() * (kScaleRows + 1); i += 256) s_w[i] = 0.f;
             __syncthreads();
             if (warp == 0) {
-                if (C <= 32) choose<1>(s_z, route.d, s_expert, s_weight);
-                else choose<2>(s_z, route.d, s_expert, s_weight);
+                RouterDims rd = route.d;
+                if (rd.correction) rd.correction = s_corr;
+                if (C <= 32) choose<1>(s_z, rd, s_expert, s_weight);
+                else choose<2>(s_z, rd, s_expert, s_weight);
             }
             if (rows > 1) {     // the last row makes the tables
                 if (warp == 0) {
