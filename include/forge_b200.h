@@ -227,8 +227,10 @@ void* forge_model_stream(ForgeModel* model);
  * there.  Every session call below takes such a model like any other.  (No counterpart in the reference, whose models are
  * GGUF decoders.)  Registered architectures: "Bolenex" (latent attention and a clamped gated feed-forward in parallel behind
  * one Dynamic Tanh norm), "Robazen" (gated delta rules, with one decay per head or per key channel, and pairs of chunked attention
- * and time mixing, a SiLU-gated feed-forward behind its own norm, and a range of layers that may run several times).  An unknown architecture, mixer or feed-forward returns FORGE_ERR_UNSUPPORTED; a missing key, a
- * missing tensor or a wrong shape FORGE_ERR_SHAPE. */
+ * and time mixing, a SiLU-gated feed-forward behind its own norm, and a range of layers that may run several times), "Mokatar" (softmax
+ * attention variants, gated linear attention, mixtures of experts, bigram embeddings) and "Tarulix" (norms on outputs, biases by distance, pooled
+ * blocks, mixed heads, selective scans, shared experts).  An unknown architecture, mixer or feed-forward returns FORGE_ERR_UNSUPPORTED; a missing
+ * key, a missing tensor or a wrong shape FORGE_ERR_SHAPE. */
 typedef struct ForgeCheckpointInfo {
     char architecture[64];
     int32_t hidden_size;
